@@ -93,7 +93,7 @@ def load_weights(cfg: OrchestrationConfig, device):
             shape = shape.with_(nextn_layers=1)
         return synthesize(shape, v.get("synthetic_recipe") or "Q4_K_M", seed=0,
                           device=device if torch.device(device).type == "cuda" else "cpu")
-    return ModelWeights.from_gguf(v["model"], device="cpu")
+    return ModelWeights.from_path(v["model"], device="cpu")
 
 
 def build_engine(cfg: OrchestrationConfig):
@@ -131,6 +131,15 @@ def build_engine(cfg: OrchestrationConfig):
         log.info("model %s (%s): %d layers, d=%d, heads %d/%d, vocab %d", mcfg.name, mcfg.arch, mcfg.n_layers, mcfg.d_model,
                  mcfg.n_heads, mcfg.n_kv_heads, mcfg.vocab_size)
         log.info("placement\n%s", plan.table())
+    fp32 = v.get("activation_precision") == "fp32" and "activation_precision" in cfg.explicitly_set and torch.device(dev).type == "cuda"
+    if fp32 and not mcfg.is_latent:
+        raise ConfigError(["--activation-precision fp32: the CUDA path of this model uses bf16 GEMM operands with an fp32 residual "
+                           "stream (fp32 is available for latent-attention models, and with -d cpu)"])
+    if mcfg.is_latent:
+        refused = [f"{flag} is not available for latent-attention models such as {mcfg.arch}" for flag, on in
+                   (("--kv-cache-precision q8_0", v.get("kv_cache_precision") in ("q8_0", "q8_1")), ("--mtp", v.get("mtp"))) if on]
+        if refused:
+            raise ConfigError(refused)
     if mcfg.is_hybrid:
         # the gated attention blocks append bf16 K/V
         if v.get("kv_cache_precision") in ("q8_0", "q8_1"):
@@ -148,6 +157,8 @@ def build_engine(cfg: OrchestrationConfig):
     eos = tok.eos_id if tok is not None else None
     kw = dict(device=dev, max_batch=v["batch_size"], max_context=v["ctx_size"], prefix_cache=prefix, mtp=mtp, tp=tp,
               eos_token_id=eos)
+    if fp32:
+        kw["dtype"] = torch.float32
     if torch.device(dev).type == "cpu" and "kv_cache_precision" in cfg.explicitly_set:
         kw["kv_dtype"] = {"bf16": torch.bfloat16, "fp16": torch.float16, "fp32": torch.float32}[v["kv_cache_precision"]]
     elif v.get("kv_cache_precision") in ("q8_0", "q8_1"):
@@ -435,10 +446,15 @@ def cmd_plan(cfg: OrchestrationConfig) -> int:
     else:
         from .gguf import GGUFFile
         from .planning import FileRecipe
-        gf = GGUFFile(v["model"])
-        mcfg = ModelConfig.from_gguf(gf)
-        recipe = FileRecipe(gf)                 # budget the formats the file really stores
-        gf.close()
+        if os.path.isdir(v["model"]):
+            from .models.weights import ModelWeights
+            w = ModelWeights.from_directory(v["model"])
+            mcfg, recipe = w.config, FileRecipe.from_weights(w)
+        else:
+            gf = GGUFFile(v["model"])
+            mcfg = ModelConfig.from_gguf(gf)
+            recipe = FileRecipe(gf)             # budget the formats the file really stores
+            gf.close()
     if v.get("suggest_layout"):
         from .planning import suggest_layout
         layout, plan = suggest_layout(mcfg, int(v["suggest_layout"]), recipe, v["ctx_size"], v["batch_size"])

@@ -75,6 +75,8 @@ class ForwardBatch:
     max_q_len: int = 0
     # which hidden rows get logits (None: all rows)
     logit_rows: torch.Tensor | None = None
+    host_cu: list | None = None              # cu_q and ctx_lens on the host, when the caller has them (saves a synchronisation)
+    host_ctx: list | None = None
     embeds: torch.Tensor | None = None       # optional fp32 [T, d] input instead of token embeddings
     state_slots: torch.Tensor | None = None  # [B] hybrid models: the state slot of every sequence (row of block_table)
     defer_state: bool = False                # hybrid models, speculative verification: equal rows per sequence, the recurrent
@@ -275,10 +277,11 @@ def paged_decode_attention_torch(q: torch.Tensor, kv_layer: torch.Tensor, block_
 
 class CudaModel:
     def __init__(self, weights: ModelWeights, device="cuda", max_tokens: int = 4096, tp=None, layer_range=None,
-                 with_head: bool = True, with_embed: bool = True, with_mtp: bool = True):
+                 with_head: bool = True, with_embed: bool = True, with_mtp: bool = True, dtype: torch.dtype = torch.bfloat16):
         self.cfg: ModelConfig = weights.config
         self.device = torch.device(device)
         self.tp = tp
+        self.dtype = dtype                              # of matrices and activations; the residual stream is fp32
         self.max_tokens = max_tokens
         c = self.cfg
         self.scratch = ops.scratch_for(self.device)
@@ -292,6 +295,13 @@ class CudaModel:
         self.q_dim, self.kv_dim = pl.n_heads_local * c.head_dim, pl.n_kv_local * c.head_dim
         self.qkv_dim = self.q_dim + 2 * self.kv_dim
         self.ff_local = pl.ff_stop - pl.ff_start
+        self.stack = None
+        self.kv_row_widths = None
+        if c.is_latent:
+            self._init_latent(weights, max_tokens)
+            return
+        if dtype != torch.bfloat16:
+            raise ValueError("32-bit mode is available for latent-attention models (the other families' kernels are 16-bit)")
 
         if with_embed:
             emb = weights["token_embd.weight"]
@@ -331,6 +341,46 @@ class CudaModel:
             lay.shared_head_norm = _f32(weights[p + "shared_head_norm.weight"], dev)
             self.mtp_layers.append(lay)
         self._alloc_workspace(max_tokens)
+
+    def _init_latent(self, weights: ModelWeights, max_tokens: int) -> None:
+        """Models whose layers attend over a latent cache: dense matrices, one cache layer per layer run (looped layers have
+        one per pass), each with its own row width."""
+        from .latent import DenseLinear, LatentStack
+        c = self.cfg
+        if self.layer_ids != list(range(c.n_layers)):
+            raise ValueError("a latent-attention model cannot be cut into pipeline stages")
+        self.stack = LatentStack(self, weights)
+        self.layers = [self.stack.build_layer(CudaLayer(), weights, i) for i in self.layer_ids]
+        self.out_norm = _f32(weights["output_norm.weight"], self.device)
+        self.head = DenseLinear(self.stack._mat(weights, "output.weight"))
+        self.vocab_local = c.vocab_size
+        self.runs = c.layer_runs()
+        self.kv_row_widths = [c.mixers[i].cache_width for i, _ in self.runs]
+        self.n_kv_layers = self.mtp_kv_base = len(self.runs)
+        self.mtp_layers, self.hybrid_dims, self.graph_safe, self.torch_attention = [], None, True, False
+        self._kv_ids, self._gdn_ids = list(range(len(self.runs))), []
+        self.ws_h = torch.empty(max_tokens, c.d_model, dtype=torch.float32, device=self.device)
+        self.stack.alloc_workspace(max_tokens, self.layers)
+
+    def _run_latent(self, fb: ForwardBatch, kv: PagedKVCache, h: torch.Tensor, debug) -> None:
+        """The layer runs of a latent-attention model on the residual stream ``h``."""
+        st, runs, layers = self.stack, self.runs, self.layers
+        bp = st.plan(fb, h.shape[0], layers)
+        first = layers[runs[0][0]].attn_norm
+        st.embed_tokens(fb.tokens, h, None if runs[0][1] else first)
+        for r, (i, starts_pass) in enumerate(runs):
+            L = layers[i]
+            if starts_pass:
+                st.enter_pass(h, L.attn_norm)
+            nxt, to_pass = None, False
+            if r + 1 < len(runs):
+                to_pass = runs[r + 1][1]
+                nxt = None if to_pass else layers[runs[r + 1][0]].attn_norm
+            st.layer(L, h, fb, bp, kv.layers[r], nxt, to_pass)
+            if debug is not None:
+                debug(r, h)
+            if getattr(self, "taps", None) is not None:
+                self.taps[f"layer{r}"] = h.float().clone()
 
     # ---------------------------------------------------------------------------------------
     def _pack_or_dense(self, t: QTensor):
@@ -444,6 +494,8 @@ class CudaModel:
         return slab
 
     def weight_bytes(self) -> int:
+        if self.stack is not None:
+            return self.stack.nbytes(self.layers) + self.head.nbytes()
         tot = 0
         for L in self.layers + self.mtp_layers:
             tot += L.qkv.nbytes() + L.wo.nbytes()
@@ -710,6 +762,8 @@ class CudaModel:
         rows = h_rows.shape[0]
         if out is None:
             out = torch.empty(rows, self.vocab_local, dtype=torch.float32, device=self.device)
+        if self.stack is not None:
+            return self.stack.final_logits(h_rows, norm_w, self.head, out)
         if rows <= ops.GEMV_MAX_ROWS:
             self.head(h_rows, out, norm_w=norm_w, eps=self.cfg.rms_eps, scratch=self.scratch)
         else:
@@ -726,7 +780,7 @@ class CudaModel:
         of a dense model under fused tensor parallelism: every weight in a packed format, no pipeline input, no debug taps,
         no consumer of the full hidden state (the engine turns ``seq_shard`` off when a NextN head needs all rows)."""
         tp = self.tp
-        if (tp is None or tp.size == 1 or not tp.fused or not getattr(self, "seq_shard", True) or fb.is_decode or fb.embeds is not None
+        if (tp is None or tp.size == 1 or self.stack is not None or not tp.fused or not getattr(self, "seq_shard", True) or fb.is_decode or fb.embeds is not None
                 or self.cfg.is_moe or self.cfg.is_hybrid or getattr(self, "taps", None) is not None or T < self.SEQ_SHARD_MIN_ROWS * tp.size
                 or self.cfg.d_model % 128 or self.cfg.d_model > 8192 or not isinstance(self.embed, PackedWeight)):
             return None
@@ -805,12 +859,14 @@ class CudaModel:
             if errs:
                 raise IndexError("forward batch rejected before launch: " + "; ".join(errs))
         h = self.ws_h[:T]
-        if fb.embeds is not None:
+        if self.stack is not None:
+            self._run_latent(fb, kv, h, debug)
+        elif fb.embeds is not None:
             h.copy_(fb.embeds)
         else:
             self.embed_tokens(fb.tokens, h)
         self._kv = kv
-        for li, L in enumerate(self.layers):
+        for li, L in enumerate(self.layers if self.stack is None else ()):
             self._layer(L, fb, kv.layers[kv_layer_offset + L.kv_index] if L.kv_index is not None else None, T)
             if debug is not None:
                 debug(self.layer_ids[li], h)

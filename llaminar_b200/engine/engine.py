@@ -70,7 +70,10 @@ class LLMEngine:
     def __init__(self, weights: ModelWeights, device: str | torch.device | None = None, max_batch: int = 32,
                  max_context: int = 4096, kv_pages: int | None = None, max_prefill_tokens: int = 8192,
                  use_graphs: bool = True, prefix_cache=None, mtp=None, tp=None, eos_token_id: int | None = None,
-                 model=None, kv_memory_fraction: float = 0.85, kv_dtype: torch.dtype | None = None, agree_group=None):
+                 model=None, kv_memory_fraction: float = 0.85, kv_dtype: torch.dtype | None = None, agree_group=None,
+                 dtype: torch.dtype = torch.bfloat16):
+        """``dtype``: matrices and activations on the GPU (torch.float32: the 32-bit mode of latent-attention models; the CPU
+        back end always computes in 32 bits)."""
         self.cfg: ModelConfig = weights.config if weights is not None else model.cfg
         if device is None:
             device = "cuda" if torch.cuda.is_available() else "cpu"
@@ -85,7 +88,7 @@ class LLMEngine:
             self.model = model
         elif self.is_cuda:
             from .cuda_model import CudaModel
-            self.model = CudaModel(weights, self.device, max_tokens=max(max_prefill_tokens, max_batch * 4), tp=tp)
+            self.model = CudaModel(weights, self.device, max_tokens=max(max_prefill_tokens, max_batch * 4), tp=tp, dtype=dtype)
         else:
             from .torch_model import TorchPagedModel
             self.model = TorchPagedModel(weights, self.device, tp=tp)
@@ -101,12 +104,15 @@ class LLMEngine:
                 raise ValueError("the 8-bit KV cache is not available for hybrid (linear-attention) models: their gated "
                                  "attention blocks append to a bf16 cache")
             hybrid = HybridState(n_slots=max(1, max_batch), device=self.device, **hd)
+        row_widths = getattr(self.model, "kv_row_widths", None)      # latent attention: one shared row per token and layer
+        if row_widths is not None and (kv_dtype == KV_Q8 or mtp is not None):
+            raise ValueError("latent-attention models have no 8-bit KV cache and no multi-token-prediction head")
         n_kv_layers = getattr(self.model, "n_kv_layers", c.n_layers + c.nextn_layers)
         if kv_pages is None:
             need = max_batch * self.max_pages_per_seq + 64
             if self.is_cuda:
                 free, _ = torch.cuda.mem_get_info(self.device)
-                per_page = max(1, PagedKVCache.bytes_per_page(n_kv_layers, self.model.n_kv_local, c.head_dim, 17 / 16 if kv_dtype == KV_Q8 else 2))
+                per_page = max(1, PagedKVCache.bytes_per_page(n_kv_layers, self.model.n_kv_local, c.head_dim, 17 / 16 if kv_dtype == KV_Q8 else dtype.itemsize, row_widths))
                 kv_pages = int(min(need * 2, max(need // 4, int(free * kv_memory_fraction) // per_page)))
             else:
                 kv_pages = need
@@ -116,7 +122,7 @@ class LLMEngine:
         self._agree_group = agree_group if agree_group is not None else (tp.group if tp is not None and tp.size > 1 else None)
         kv_pages = self._agree_kv_pages(kv_pages, self._agree_group)
         self.kv = PagedKVCache(n_kv_layers, self.model.n_kv_local, c.head_dim, kv_pages, self.device,
-                               dtype=(KV_Q8 if kv_dtype == KV_Q8 else torch.bfloat16) if self.is_cuda else (kv_dtype or torch.float32))
+                               dtype=(KV_Q8 if kv_dtype == KV_Q8 else dtype) if self.is_cuda else (kv_dtype or torch.float32), row_widths=row_widths)
         self.kv.hybrid = hybrid
         self.use_graphs = use_graphs and self.is_cuda and not debug_env().no_cuda_graphs and getattr(self.model, "graph_safe", True)
         self.perf = perf_stats()
@@ -170,7 +176,7 @@ class LLMEngine:
     @staticmethod
     def from_gguf(path: str, **kw) -> "LLMEngine":
         dev = kw.get("device") or ("cuda" if torch.cuda.is_available() else "cpu")
-        w = ModelWeights.from_gguf(path, device="cpu")
+        w = ModelWeights.from_path(path, device="cpu")
         eng = LLMEngine(w, **kw)
         eng.metadata = w.metadata
         return eng
@@ -637,6 +643,96 @@ class LLMEngine:
         if hasattr(self.model, "sync_sampled"):
             self.model.token_sync = self.mtp is None and not any(r.params.wants_logprobs for r in reqs)
 
+    def _forward_chunks(self, chunks: list[tuple[Request, int, list[int]]], logit_rows: list[int]):
+        """One forward call over portions of several sequences: (request, first position, tokens), packed in that order.
+        Returns (logits of `logit_rows` or None, hidden rows, the batch)."""
+        dev = self.device
+        toks, pos, sid, cu, ctx = [], [], [], [0], []
+        for b, (r, start, tokens) in enumerate(chunks):
+            n = len(tokens)
+            toks.extend(tokens)
+            pos.extend(range(start, start + n))
+            sid.extend([b] * n)
+            cu.append(cu[-1] + n)
+            ctx.append(start)
+        bt = torch.zeros(len(chunks), max(len(r.kv.pages) for r, _, _ in chunks), dtype=torch.int32)
+        for i, (r, _, _) in enumerate(chunks):
+            bt[i, :len(r.kv.pages)] = torch.tensor(r.kv.pages, dtype=torch.int32)
+        it = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
+        fb = ForwardBatch(tokens=it(toks), positions=it(pos), seq_ids=it(sid), block_table=bt.to(dev), cu_q=it(cu),
+                          ctx_lens=it(ctx), max_q_len=max(cu[i + 1] - cu[i] for i in range(len(ctx))),
+                          max_kv_len=max(ctx[i] + cu[i + 1] - cu[i] for i in range(len(ctx))), host_cu=cu, host_ctx=ctx,
+                          logit_rows=it(logit_rows) if logit_rows else None,
+                          state_slots=it([r.slot for r, _, _ in chunks]) if self.kv.hybrid is not None else None)
+        logits, h = self.model.forward(fb, self.kv, want_logits=bool(logit_rows))
+        return logits, h, fb
+
+    # -- sequences stepped by the caller ------------------------------------------------------------------
+    # The caller names the tokens of every step instead of having them sampled (replaying a recorded run, scoring given
+    # text).  The steps take the paths of generation: portions of prompts and mixed steps one packed forward call, steps of
+    # one token per sequence the (captured) decode step.
+    def open_sequence(self) -> Request:
+        """A sequence that only `feed` advances; it holds pages (and a state slot) until `close_sequence`."""
+        r = Request(next(self._rid), [], SamplingParams(temperature=0.0, max_tokens=1 << 30, ignore_eos=True), state="stepped")
+        if self.kv.hybrid is not None:
+            r.slot = self.kv.hybrid.alloc()
+        self.requests[r.rid] = r
+        return r
+
+    def close_sequence(self, r: Request) -> None:
+        self._finish(r, "abort")
+        self.requests.pop(r.rid, None)
+
+    def feed(self, entries: list[tuple[Request, list[int], list[int]]]) -> torch.Tensor | None:
+        """One step over all entries: (sequence, its next tokens, places among them whose logits are wanted).  Returns the
+        wanted rows [n, vocab] in the order of the entries, or None when nothing is wanted."""
+        V = self._vocab
+        for r, tokens, want in entries:
+            if not tokens or any(not 0 <= t < V for t in tokens) or any(not 0 <= w < len(tokens) for w in want):
+                raise ValueError("an entry needs tokens of the vocabulary, and wanted places among them")
+            if r.kv.length + len(tokens) > self.max_context:
+                raise ValueError(f"sequence of {r.kv.length + len(tokens)} tokens exceeds the context window of {self.max_context}")
+        total = sum(len(t) for _, t, _ in entries)
+        if total > self.max_prefill_tokens:
+            raise ValueError(f"a step of {total} tokens exceeds the engine's {self.max_prefill_tokens}")
+        for r, tokens, _ in entries:
+            self._ensure_pages(r, r.kv.length + len(tokens))
+        single = len(entries) <= self.max_batch and all(len(t) == 1 and r.kv.length > 0 for r, t, _ in entries)
+        if single:
+            for r, tokens, _ in entries:
+                r.output.extend(tokens)
+            logits = self._decode_logits([r for r, _, _ in entries])
+            picked = [i for i, (_, _, want) in enumerate(entries) for _ in want]
+            out = logits[torch.tensor(picked, dtype=torch.long, device=logits.device)] if picked else None
+        else:
+            at, picked = 0, []
+            for r, tokens, want in entries:
+                picked.extend(at + w for w in want)
+                at += len(tokens)
+            out, _, _ = self._forward_chunks([(r, r.kv.length, tokens) for r, tokens, _ in entries], picked)
+            for r, tokens, _ in entries:
+                r.output.extend(tokens)
+        for r, tokens, _ in entries:
+            r.kv.length += len(tokens)
+        self.check_health()
+        return self._gather_vocab(out) if out is not None else None
+
+    def _decode_logits(self, reqs: list[Request]) -> torch.Tensor:
+        """Logits of one decode step (the last token of every request is the step's input), without sampling."""
+        bucket = next((b for b in BUCKETS if b >= len(reqs)), len(reqs))
+        if not self.use_graphs or bucket > self._bmax:
+            return self.model.forward(self._decode_batch_tensors(reqs), self.kv)[0]
+        v = self._dec_views(bucket, 1)
+        self._fill_decode_host(reqs, bucket, v)
+        self._dec_dev[:v["n"]].copy_(self._dec_host[:v["n"]], non_blocking=True)
+        g = self._graphs.get((bucket, "logits"))
+        if g is None:
+            g = self._graphs[(bucket, "logits")] = self._capture_decode(bucket, True, v, sample=False)
+        g.replay()
+        self.stats["graph_replays"] += 1
+        torch.cuda.current_stream(self.device).synchronize()       # the staging buffers are free for the next step
+        return self._logits[:len(reqs)]
+
     def _prefill(self, batch: list[Request]) -> list[StepOutput]:
         t0 = time.perf_counter()
         dev = self.device
@@ -654,9 +750,8 @@ class LLMEngine:
         if self.prefix_cache is not None and self.kv.hybrid is not None:
             snap_at = {r.rid: self.prefix_cache.snapshot_points(len(r.prompt), pending[r.rid]) for r in batch}
         while any(pending[r.rid] < len(r.prompt) for r in batch):
-            toks, pos, sid, cu, ctx, rows_for, chunks = [], [], [], [0], [], [], []
+            chunks, rows_for, T = [], [], 0
             budget = self.max_prefill_tokens
-            btab_rows = []
             for r in batch:
                 done = pending[r.rid]
                 if done >= len(r.prompt) or budget <= 0:
@@ -666,28 +761,12 @@ class LLMEngine:
                 if nxt is not None:                          # a chunk ends where the prefix cache wants the recurrent state
                     n = min(n, nxt - done)
                 budget -= n
-                b = len(ctx)
-                toks.extend(r.prompt[done:done + n])
-                pos.extend(range(done, done + n))
-                sid.extend([b] * n)
-                cu.append(cu[-1] + n)
-                ctx.append(done)
-                btab_rows.append(r.kv.pages)
+                T += n
                 pending[r.rid] = done + n
                 chunks.append((r, done, n))
-                rows_for.append((r, cu[-1] - 1 if done + n == len(r.prompt) else None))
-            P = max(len(p) for p in btab_rows)
-            bt = torch.zeros(len(btab_rows), P, dtype=torch.int32)
-            for i, p in enumerate(btab_rows):
-                bt[i, :len(p)] = torch.tensor(p, dtype=torch.int32)
-            it = lambda x: torch.tensor(x, dtype=torch.int32, device=dev)
-            logit_rows = [row for _, row in rows_for if row is not None]
-            fb = ForwardBatch(tokens=it(toks), positions=it(pos), seq_ids=it(sid), block_table=bt.to(dev), cu_q=it(cu),
-                              ctx_lens=it(ctx), max_q_len=max(cu[i + 1] - cu[i] for i in range(len(ctx))),
-                              max_kv_len=max(ctx[i] + cu[i + 1] - cu[i] for i in range(len(ctx))),
-                              logit_rows=it(logit_rows) if logit_rows else None,
-                              state_slots=it([r.slot for r, _, _ in chunks]) if self.kv.hybrid is not None else None)
-            logits, h = self.model.forward(fb, self.kv, want_logits=bool(logit_rows))
+                rows_for.append((r, T - 1 if done + n == len(r.prompt) else None))
+            logits, h, fb = self._forward_chunks([(r, done, r.prompt[done:done + n]) for r, done, n in chunks],
+                                                 [row for _, row in rows_for if row is not None])
             for r, done, n in chunks:
                 if done + n in snap_at.get(r.rid, ()):
                     self.prefix_cache.store_state(r.prompt[:done + n], self.kv.hybrid.snapshot(r.slot))
@@ -700,7 +779,7 @@ class LLMEngine:
                     final_logits[r.rid] = logits[j]
                     final_hidden[r.rid] = keep[r.rid] if self.mtp is not None else h[row].clone()
                     j += 1
-            self.stats["prefill_tokens"] += len(toks)
+            self.stats["prefill_tokens"] += T
         outs = []
         lg = torch.stack([final_logits[r.rid] for r in batch])
         toks = self._sample_rows(lg, batch)
@@ -931,7 +1010,7 @@ class LLMEngine:
             self._pen_lanes[i] = None
         self._pen_dev.copy_(self._pen_host, non_blocking=True)
 
-    def _decode_body(self, bucket: int, greedy: bool, v: dict, pen: bool = False) -> None:
+    def _decode_body(self, bucket: int, greedy: bool, v: dict, pen: bool = False, sample: bool = True) -> None:
         from .. import ops
         d = self._dec_dev
         P = self.max_pages_per_seq
@@ -940,6 +1019,8 @@ class LLMEngine:
                           n_splits=self._splits_for(bucket),
                           state_slots=d[v["slot"]] if self.kv.hybrid is not None else None)
         logits, _ = self.model.forward(fb, self.kv, logits_out=self._logits[:bucket])
+        if not sample:
+            return
         tok = self._tok_dev[:bucket]
         if pen:
             ops.penalties_dense(logits, self._pen_counts[:bucket], self._pen_dev[:bucket], self._pen_dev[self._bmax:self._bmax + bucket])
@@ -959,7 +1040,7 @@ class LLMEngine:
             v0, V = self._vocab_window()
             ops.count_tokens(self._pen_counts[:bucket], tok, v0, V)
 
-    def _capture_decode(self, bucket: int, greedy: bool, v: dict, pen: bool = False):
+    def _capture_decode(self, bucket: int, greedy: bool, v: dict, pen: bool = False, sample: bool = True):
         torch.cuda.synchronize(self.device)
         if self.kv.hybrid is not None:
             # the warm-up runs are real steps, and a recurrent state (unlike a K/V row) is not the same after being advanced
@@ -969,7 +1050,7 @@ class LLMEngine:
         side.wait_stream(torch.cuda.current_stream(self.device))
         with torch.cuda.stream(side):
             for _ in range(2):                          # warm-up: lazy initialisation must not happen in capture
-                self._decode_body(bucket, greedy, v, pen)
+                self._decode_body(bucket, greedy, v, pen, sample)
             if pen:                                     # the warm-up runs counted tokens: every lane's table is rebuilt below
                 self._pen_lanes = [None] * self._bmax
         torch.cuda.current_stream(self.device).wait_stream(side)
@@ -978,8 +1059,9 @@ class LLMEngine:
         n0 = ops.launch_count()
         g = torch.cuda.CUDAGraph()
         with torch.cuda.graph(g):
-            self._decode_body(bucket, greedy, v, pen)
-        self.launches_per_graph[(bucket, greedy, pen) if pen else (bucket, greedy)] = ops.launch_count() - n0
+            self._decode_body(bucket, greedy, v, pen, sample)
+        key = (bucket, greedy, pen) if pen else (bucket, greedy) if sample else (bucket, "logits")
+        self.launches_per_graph[key] = ops.launch_count() - n0
         if self.kv.hybrid is not None:
             self._dec_dev[:v["n"]].copy_(self._dec_host[:v["n"]], non_blocking=True)
         return g

@@ -114,11 +114,20 @@ Q8 = "q8_0"          # 8-bit cache: int8 values with one fp16 scale per 32 (CUDA
 
 
 class PagedKVCache:
-    def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, n_pages: int, device, dtype=torch.bfloat16):
+    """Pages of 64 tokens per cache layer.  Per-head layout: [2 (K, V), heads, 64, head size].  With ``row_widths`` (one per
+    layer) a layer holds one row of that many values per token instead, shared by all heads (latent attention)."""
+
+    def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, n_pages: int, device, dtype=torch.bfloat16,
+                 row_widths: list[int] | None = None):
         self.n_layers, self.n_kv_heads, self.head_dim, self.n_pages = n_layers, n_kv_heads, head_dim, n_pages
         self.device = torch.device(device)
         self.q8 = dtype == Q8
-        if self.q8:
+        self.row_widths = row_widths
+        if row_widths is not None:
+            if self.q8 or len(row_widths) != n_layers:
+                raise ValueError("a latent cache takes one row width per layer and float rows")
+            self.layers = [torch.zeros(n_pages, PAGE_SIZE, w, dtype=dtype, device=device) for w in row_widths]
+        elif self.q8:
             # a page is [2][n_kv_heads][64][head_dim] int8 followed by [2][n_kv_heads][64][head_dim / 32] fp16 block scales;
             # zero bytes decode to zeros, so untouched positions stay finite
             if head_dim % 32:
@@ -132,8 +141,15 @@ class PagedKVCache:
         self.allocator = PageAllocator(n_pages)
         self.hybrid: HybridState | None = None          # set by the engine for models with linear-attention layers
 
+    @property
+    def page_bytes(self) -> int:
+        """Bytes of one page over all layers."""
+        return sum(l[0].numel() * l.element_size() for l in self.layers)
+
     @staticmethod
-    def bytes_per_page(n_layers: int, n_kv_heads: int, head_dim: int, itemsize: float = 2) -> int:
+    def bytes_per_page(n_layers: int, n_kv_heads: int, head_dim: int, itemsize: float = 2, row_widths: list[int] | None = None) -> int:
+        if row_widths is not None:
+            return int(sum(row_widths) * PAGE_SIZE * itemsize)
         return int(n_layers * 2 * n_kv_heads * PAGE_SIZE * head_dim * itemsize)
 
     def ensure_capacity(self, seq: SequenceKV, n_tokens: int) -> None:
@@ -162,11 +178,19 @@ class PagedKVCache:
         return SequenceKV(list(pages), n_tokens)
 
     # -- page payload movement for the RAM / disk prefix tiers -------------------------------
-    def export_page(self, page: int) -> torch.Tensor:
+    def copy_page(self, page: int) -> torch.Tensor:
+        """One page over all layers, on the device: [layers, ...page], or one flat run where the layers' rows differ."""
         if not self.layers:                      # a pipeline stage of linear-attention blocks only: pages carry no bytes here
             return torch.empty(0)
-        return torch.stack([l[page] for l in self.layers]).to("cpu", non_blocking=False)
+        if self.row_widths is not None:
+            return torch.cat([l[page].reshape(-1) for l in self.layers])
+        return torch.stack([l[page] for l in self.layers])
+
+    def export_page(self, page: int) -> torch.Tensor:
+        return self.copy_page(page).to("cpu", non_blocking=False)
 
     def import_page(self, page: int, payload: torch.Tensor) -> None:
+        if self.row_widths is not None:
+            payload = [x.view(PAGE_SIZE, -1) for x in payload.split([PAGE_SIZE * w for w in self.row_widths])]
         for i, l in enumerate(self.layers):
             l[page].copy_(payload[i].to(self.device, non_blocking=True))

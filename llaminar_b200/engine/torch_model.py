@@ -33,6 +33,7 @@ class TorchPagedModel:
         self.n_heads_local, self.n_kv_local = pl.n_heads_local, pl.n_kv_local
         self.layer_ids = list(range(*layer_range)) if layer_range else list(range(c.n_layers))
         D = c.head_dim
+        self.kv_row_widths = None
         f = lambda name: weights[name].to_float().to(self.device)
         self.embed = f("token_embd.weight") if with_embed else None
         self.head = None
@@ -42,6 +43,9 @@ class TorchPagedModel:
             self.head = head.rows(pl.vocab_start, pl.vocab_stop).to_float().to(self.device)
             self.vocab_local = pl.vocab_stop - pl.vocab_start
 
+        if c.is_latent:
+            self._init_latent(f)
+            return
         kv_ids, gdn_ids = c.kv_layers(self.layer_ids), c.gdn_layers(self.layer_ids)
 
         def ffn(L, p):
@@ -115,6 +119,91 @@ class TorchPagedModel:
 
     def weight_bytes(self) -> int:
         return 0
+
+    # -- latent-attention models ------------------------------------------------------------------------
+    def _init_latent(self, f) -> None:
+        c = self.cfg
+        if self.layer_ids != list(range(c.n_layers)):
+            raise ValueError("a latent-attention model cannot be cut into pipeline stages")
+        self.embed_norm = f("token_embd_norm.weight")
+        self.loop_in = f("loop_in.weight") if c.loop else None
+        names = {"attn_norm": "attn_norm", "post_attn": "post_attention_norm", "qa": "attn_q_a", "qan": "attn_q_a_norm", "qb": "attn_q_b",
+                 "kva": "attn_kv_a", "kvan": "attn_kv_a_norm", "kb": "attn_k_b", "vb": "attn_v_b", "sink": "attn_sinks", "wo": "attn_output"}
+        ffn = {"ffn_norm": "ffn_norm", "post_ffn": "post_ffw_norm", "wg": "ffn_gate", "wu": "ffn_up", "wd": "ffn_down"}
+        self.layers = []
+        for i in self.layer_ids:
+            want = dict(names, **(ffn if c.ff_width(i) else {}))
+            if not c.mixers[i].sinks:
+                want.pop("sink")
+            L = {k: f(f"blk.{i}.{n}.weight") for k, n in want.items()}
+            L["mixer"] = c.mixers[i]
+            L["freqs"] = torch.tensor(c.mixers[i].rotary.frequencies(), dtype=torch.float64, device=self.device)
+            self.layers.append(L)
+        self.runs = c.layer_runs()
+        self.kv_row_widths = [c.mixers[i].cache_width for i, _ in self.runs]
+        self.n_kv_layers = self.mtp_kv_base = len(self.runs)
+        self.mtp_layers, self.hybrid_dims = [], None
+
+    @staticmethod
+    def _turn(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
+        """Rotate the leading 2 x cos.shape[-1] values of the last dimension, pair (i, i + half)."""
+        half = cos.shape[-1]
+        a, b = x[..., :half], x[..., half:2 * half]
+        return torch.cat([a * cos - b * sin, b * cos + a * sin, x[..., 2 * half:]], dim=-1)
+
+    def _latent_attention(self, L, x: torch.Tensor, fb: ForwardBatch, kvl: torch.Tensor) -> torch.Tensor:
+        """Queries in the latent space against the cached latents, sequence by sequence."""
+        c, m = self.cfg, L["mixer"]
+        T, rot_off = x.shape[0], -(-m.kv_rank // 8) * 8
+        pos = fb.positions.long()
+        ang = pos.double()[:, None] * L["freqs"]
+        cos, sin = (ang.cos() * m.rotary.magnitude).float(), (ang.sin() * m.rotary.magnitude).float()
+        q = (rmsnorm(x @ L["qa"].T, L["qan"], c.rms_eps) @ L["qb"].T).view(T, m.heads, m.dim + m.rot_dim)
+        q_rot = self._turn(q[..., m.dim:], cos[:, None], sin[:, None])
+        q_lat = torch.einsum("thd,hdr->thr", q[..., :m.dim], L["kb"].view(m.heads, m.dim, m.kv_rank))
+        down = x @ L["kva"].T
+        sid = fb.seq_ids.long()
+        page, off = fb.block_table.long()[sid, pos // PAGE_SIZE], pos % PAGE_SIZE
+        row = torch.zeros(T, kvl.shape[-1])
+        row[:, :m.kv_rank] = rmsnorm(down[:, :m.kv_rank], L["kvan"], c.rms_eps)
+        row[:, rot_off:rot_off + m.rot_dim] = self._turn(down[:, m.kv_rank:], cos, sin)
+        kvl[page, off] = row.to(kvl.dtype)
+        out = torch.empty(T, m.heads, m.kv_rank)
+        for b in sid.unique().tolist():
+            rows = (sid == b).nonzero(as_tuple=True)[0]
+            p = pos[rows]
+            lo = max(0, int(p.min()) - m.window + 1) if m.window else 0
+            keys = torch.arange(lo, int(p.max()) + 1)
+            kv = kvl[fb.block_table.long()[b, keys // PAGE_SIZE], keys % PAGE_SIZE].float()
+            s = torch.einsum("thr,sr->hts", q_lat[rows], kv[:, :m.kv_rank])
+            s = (s + torch.einsum("the,se->hts", q_rot[rows], kv[:, rot_off:rot_off + m.rot_dim])) * m.scale
+            ahead = keys[None, :] > p[:, None]
+            if m.window:
+                ahead |= keys[None, :] <= p[:, None] - m.window
+            s = s.masked_fill(ahead[None], float("-inf"))
+            if m.sinks:                       # one more column that carries no value
+                s = torch.cat([s, L["sink"][:, None, None].expand(-1, s.shape[1], 1)], dim=-1)
+            w = torch.softmax(s, -1)[..., :len(keys)]
+            out[rows] = torch.einsum("hts,sr->thr", w, kv[:, :m.kv_rank])
+        v = torch.einsum("thr,hvr->thv", out, L["vb"].view(m.heads, m.vdim, m.kv_rank))
+        return v.reshape(T, -1) @ L["wo"].T
+
+    def _run_latent(self, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        eps = self.cfg.rms_eps
+        x0 = rmsnorm(self.embed[fb.tokens.long()].float(), self.embed_norm, eps)
+        h = x0
+        for r, (i, starts_pass) in enumerate(self.runs):
+            L = self.layers[i]
+            if starts_pass:
+                h = torch.cat([h, x0], dim=-1) @ self.loop_in.T
+            h = h + rmsnorm(self._latent_attention(L, rmsnorm(h, L["attn_norm"], eps), fb, kv.layers[r]), L["post_attn"], eps)
+            if "wg" in L:
+                x = rmsnorm(h, L["ffn_norm"], eps)
+                y = (F.gelu(x @ L["wg"].T, approximate="tanh") * (x @ L["wu"].T)) @ L["wd"].T
+                h = h + rmsnorm(y, L["post_ffn"], eps)
+            if getattr(self, "taps", None) is not None:
+                self.taps[f"layer{r}"] = h.clone()
+        return h
 
     # ---------------------------------------------------------------------------------------
     def _sum_ranks(self, x: torch.Tensor) -> torch.Tensor:
@@ -223,8 +312,12 @@ class TorchPagedModel:
 
     @torch.no_grad()
     def forward(self, fb: ForwardBatch, kv: PagedKVCache, logits_out=None, want_logits=True, kv_layer_offset: int = 0):
-        h = fb.embeds.float() if fb.embeds is not None else self.embed[fb.tokens.long()].float()
-        for li, L in enumerate(self.layers):
+        latent = self.cfg.is_latent
+        if latent:
+            h = self._run_latent(fb, kv)
+        else:
+            h = fb.embeds.float() if fb.embeds is not None else self.embed[fb.tokens.long()].float()
+        for li, L in enumerate(() if latent else self.layers):
             kvl = kv.layers[kv_layer_offset + L["kv_index"]] if L.get("kv_index") is not None else None
             h = self._layer(L, h, fb, kvl, kv)
             if getattr(self, "taps", None) is not None:       # per-layer hidden states for the parity report

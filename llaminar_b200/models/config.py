@@ -7,11 +7,77 @@ src/v2/execution/mtp/MTPWeightManifest.cpp:141-156).
 """
 from __future__ import annotations
 
+import json
+import math
 from dataclasses import asdict, dataclass, field, replace
 
 from ..gguf.constants import GGMLType
 
-SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe")
+SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik")
+
+
+@dataclass(frozen=True)
+class RopeScaling:
+    """YaRN: pairs that turn less than `slow` times over the original context are slowed down by `factor`, pairs that turn
+    more than `fast` times keep their frequency, the ones between are blended; sine and cosine grow by a common factor."""
+    factor: float
+    original: float
+    fast: float
+    slow: float
+
+
+@dataclass(frozen=True)
+class Rotary:
+    """Rotation of the first `dims` values of a vector, pair (i, i + dims/2) by position x frequency i."""
+    dims: int
+    base: float
+    scaling: RopeScaling | None = None
+
+    def frequencies(self) -> list[float]:
+        """Angle per position of each of the dims/2 pairs (double precision)."""
+        plain = [self.base ** (-2.0 * i / self.dims) for i in range(self.dims // 2)]
+        s = self.scaling
+        if s is None:
+            return plain
+
+        def pair_with(turns: float) -> float:
+            """The (fractional) pair index that completes `turns` turns over the original context."""
+            return self.dims * math.log(s.original / (turns * 2.0 * math.pi)) / (2.0 * math.log(self.base))
+
+        first = max(math.floor(pair_with(s.fast)), 0)
+        last = min(math.ceil(pair_with(s.slow)), self.dims - 1)
+        out = []
+        for i, f in enumerate(plain):
+            slowed = min(1.0, max(0.0, (i - first) / max(last - first, 0.001)))
+            out.append(f * (1.0 - slowed) + f * slowed / s.factor)
+        return out
+
+    @property
+    def magnitude(self) -> float:
+        return 1.0 if self.scaling is None else 1.0 + 0.1 * math.log(self.scaling.factor)
+
+
+@dataclass(frozen=True)
+class LatentAttention:
+    """Attention over a low-rank latent: the cache holds one normed latent of `kv_rank` values and one rotated key part of
+    `rot_dim` values per token, shared by all heads; per-head keys (`dim` unrotated values) and values (`vdim`) are linear
+    functions of the latent.  Queries pass through a latent of `q_rank` values."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    q_rank: int
+    kv_rank: int
+    scale: float
+    rotary: Rotary
+    window: int = 0                 # keys a query sees, itself included (0: all before it)
+    sinks: bool = True              # one learned logit per head in the softmax denominator
+
+    @property
+    def cache_width(self) -> int:
+        """Values of a token's cache row: the latent and the rotated part, each starting on a 16-byte boundary in 16-bit
+        form, padded to whole 16-value MMA steps."""
+        return (-(-self.kv_rank // 8) * 8 + -(-self.rot_dim // 8) * 8 + 15) // 16 * 16
 
 
 @dataclass
@@ -47,6 +113,14 @@ class ModelConfig:
     ssm_k_heads: int = 0
     ssm_v_heads: int = 0
     rope_dim: int = 0                    # leading dims of each head that are rotated (0: all of head_dim)
+    # layer lists with their own sizes per layer (pozivik): the mixer of every layer, its feed-forward width (0: none), and
+    # the layers [start, stop) that run `times` times in a row, each pass behind a projection of [hidden | embedding]
+    mixers: tuple[LatentAttention, ...] = ()
+    layer_ff: tuple[int, ...] = ()
+    loop: tuple[int, int, int] | None = None
+    embed_norm: bool = False             # RMSNorm on the token embedding
+    post_norms: bool = False             # RMSNorm on the output of a sublayer, before it joins the residual stream
+    ffn_act: str = "silu"                # silu | gelu_tanh: activation of the gated feed-forward
     attn_gate: bool = False              # attn_q holds [q | gate] per head; the attention output is scaled by sigmoid(gate)
     name: str = "tiny-qwen3"
 
@@ -61,6 +135,21 @@ class ModelConfig:
     def is_gdn_layer(self, i: int) -> bool:
         """Trunk layer i is linear attention (NextN layers, i >= n_layers, are always full attention)."""
         return self.is_hybrid and i < self.n_layers and (i + 1) % self.full_attention_interval != 0
+
+    @property
+    def is_latent(self) -> bool:
+        """Latent-attention layers, run by the latent block (their own cache layout, 16- or 32-bit weight matrices)."""
+        return bool(self.mixers)
+
+    def layer_runs(self) -> list[tuple[int, bool]]:
+        """The layers in the order they run: (layer, whether a pass over the looped layers starts before it).  Every run has a
+        cache layer of its own."""
+        start, stop, times = self.loop or (self.n_layers, self.n_layers, 0)
+        body = [(i, i == start) for i in range(start, stop)]
+        return [(i, False) for i in range(start)] + body * times + [(i, False) for i in range(stop, self.n_layers)]
+
+    def ff_width(self, layer: int) -> int:
+        return self.layer_ff[layer] if self.layer_ff else self.d_ff
 
     def kv_layers(self, layer_ids) -> list[int]:
         """Of the given layers, the ones that own a KV-cache layer (all but the linear-attention ones)."""
@@ -111,6 +200,9 @@ class ModelConfig:
         if arch not in SUPPORTED_ARCHS:
             raise ValueError(f"unsupported GGUF architecture '{arch}' (supported: {', '.join(SUPPORTED_ARCHS)}; "
                              "qwen35 / qwen35moe are the hybrid Gated-DeltaNet families)")
+        if arch == "pozivik":
+            from .pozivik import config_from_json
+            return config_from_json(json.loads(gf.get("pozivik.config")))
         a = gf.arch_key
 
         def scalar(v):
@@ -171,6 +263,9 @@ class ModelConfig:
 
     def gguf_metadata(self) -> dict:
         a = self.arch
+        if a == "pozivik":
+            from .pozivik import config_to_json
+            return {"general.architecture": a, "general.name": self.name, "pozivik.config": json.dumps(config_to_json(self))}
         md = {
             "general.architecture": a,
             "general.name": self.name,
@@ -255,6 +350,15 @@ RECIPES = {
     "F32": QuantRecipe(GGMLType.F32, {}, "F32"),
 }
 
+def latent_shape(name: str, n_layers: int, d_model: int, mixer: LatentAttention, ff: int, vocab: int, loop=None, eps: float = 1e-5,
+                 context_length: int = 32768) -> ModelConfig:
+    """A pozivik shape whose layers are all alike."""
+    return ModelConfig(name=name, arch="pozivik", n_layers=n_layers, d_model=d_model, n_heads=mixer.heads, n_kv_heads=1,
+                       head_dim=mixer.cache_width, d_ff=ff, vocab_size=vocab, rope_theta=mixer.rotary.base, rms_eps=eps,
+                       context_length=context_length, qk_norm=False, tie_embeddings=False, mixers=(mixer,) * n_layers,
+                       layer_ff=(ff,) * n_layers, loop=loop, embed_norm=True, post_norms=True, ffn_act="gelu_tanh")
+
+
 # The benchmark shapes (random-init stand-ins for the named public models).
 SHAPES = {
     "tiny-qwen3": ModelConfig(name="tiny-qwen3"),
@@ -283,6 +387,11 @@ SHAPES = {
     "qwen3-30b-a3b": ModelConfig(name="qwen3-30b-a3b", arch="qwen3moe", n_layers=48, d_model=2048, n_heads=32,
                                  n_kv_heads=4, head_dim=128, d_ff=0, vocab_size=151936, tie_embeddings=False,
                                  n_experts=128, n_experts_used=8, expert_ff=768, context_length=40960),
+    "tiny-pozivik": latent_shape("tiny-pozivik", 3, 256, LatentAttention(4, 32, 16, 32, 64, 96, 48 ** -0.5, Rotary(16, 1e4, RopeScaling(4.0, 256, 32.0, 1.0)), 100),
+                                 512, 1024, loop=(1, 3, 2)),
+    # layers the size of qwen3-8b's: the same width, feed-forward, vocabulary and number of heads
+    "pozivik-8b": latent_shape("pozivik-8b", 36, 4096, LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 5e4, RopeScaling(4.0, 8192, 32.0, 1.0)), 1024),
+                               12288, 151936),
     "qwen2.5-7b": ModelConfig(name="qwen2.5-7b", arch="qwen2", n_layers=28, d_model=3584, n_heads=28, n_kv_heads=4,
                               head_dim=128, d_ff=18944, vocab_size=152064, tie_embeddings=False, qk_norm=False,
                               qkv_bias=True, context_length=32768),

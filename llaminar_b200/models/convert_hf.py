@@ -269,6 +269,10 @@ def requantize(w: ModelWeights, recipe: QuantRecipe | str) -> ModelWeights:
 
 def convert_directory(model_dir: str, out_path: str, recipe: str = "Q8_0") -> ModelWeights:
     hf, sd = load_checkpoint(model_dir)
+    if "architecture" in hf:                        # a family with a reader of its own
+        w = requantize(ModelWeights.from_directory(model_dir), recipe)
+        w.save_gguf(out_path)
+        return w
     cfg = config_from_hf(hf)
     w = convert_state_dict(cfg, sd, recipe)
     w.metadata.update(tokenizer_metadata(model_dir))

@@ -6,6 +6,8 @@ or from the synthetic generator, and can be written back to a ``.gguf``.
 """
 from __future__ import annotations
 
+import json
+import os
 from dataclasses import dataclass
 
 import torch
@@ -89,6 +91,26 @@ class ModelWeights:
 
     # -- file I/O ------------------------------------------------------------------------------
     @staticmethod
+    def from_path(path: str, device="cpu") -> "ModelWeights":
+        """A `.gguf` file, or a checkpoint directory of a family that is served without conversion."""
+        return ModelWeights.from_directory(path) if os.path.isdir(path) else ModelWeights.from_gguf(path, device)
+
+    @staticmethod
+    def from_directory(path: str) -> "ModelWeights":
+        """`config.json` + `*.safetensors`; the family's reader is chosen by the configuration's "architecture"."""
+        from .convert_hf import load_checkpoint, tokenizer_metadata
+        with open(os.path.join(path, "config.json")) as f:
+            arch = json.load(f).get("architecture")
+        reader = _directory_readers().get(arch)
+        if reader is None:
+            raise ValueError(f"{path}: no reader for architecture {arch!r} (known: {', '.join(_directory_readers())}; "
+                             "Hugging Face checkpoints are converted to GGUF first: python -m llaminar_b200.models.convert_hf)")
+        w = reader(*load_checkpoint(path))
+        if os.path.exists(os.path.join(path, "tokenizer.json")):
+            w.metadata.update(tokenizer_metadata(path))
+        return w
+
+    @staticmethod
     def from_gguf(path: str, device="cpu") -> "ModelWeights":
         gf = GGUFFile(path)
         cfg = ModelConfig.from_gguf(gf)
@@ -113,6 +135,12 @@ class ModelWeights:
         for name, t in self.tensors.items():
             w.add_raw_tensor(name, t.qtype, t.shape, t.raw)
         w.write(path)
+
+
+def _directory_readers() -> dict:
+    """config.json "architecture" -> function(config dict, {name: tensor}) -> ModelWeights."""
+    from . import pozivik
+    return {pozivik.ARCHITECTURE: pozivik.weights_from_tensors}
 
 
 def qtensor_from_float(x: torch.Tensor, qtype: GGMLType) -> QTensor:

@@ -15,11 +15,15 @@ from pathlib import Path
 NAME = "llaminar_b200_ops"
 CSRC = Path(__file__).resolve().parent / "csrc"
 BUILD_DIR = Path(__file__).resolve().parent / "_build"
-SOURCES = ["binding.cpp", "gemv.cu", "gemv_stream.cu", "gemm_tc.cu", "gemm_tc_small.cu", "attention.cu", "attention_tc.cu", "ops.cu", "gdn.cu", "moe_ep.cu", "no_alloc.cu"]
+LATENT = "llaminar_b200_latent"       # kernels of latent-attention models, built and loaded on their own
+SOURCES = {
+    NAME: ["binding.cpp", "gemv.cu", "gemv_stream.cu", "gemm_tc.cu", "gemm_tc_small.cu", "attention.cu", "attention_tc.cu", "ops.cu", "gdn.cu", "moe_ep.cu", "no_alloc.cu"],
+    LATENT: ["latent_binding.cpp", "latent_attention.cu", "dense_ops.cu"],
+}
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xptxas", "-v"]
 
-_module = None
+_modules: dict = {}
 
 
 def _bounds_check() -> bool:
@@ -36,62 +40,71 @@ def _build_dir() -> Path:
     return BUILD_DIR.with_name("_build_bc") if _bounds_check() else BUILD_DIR
 
 
-def _existing_sources() -> list[Path]:
-    return [CSRC / s for s in SOURCES if (CSRC / s).exists()]
-
-
-def source_hash() -> str:
+def source_hash(name: str = NAME) -> str:
+    """Hash of an extension's own sources, of every header and of the compiler flags."""
     h = hashlib.sha256()
     for p in sorted(CSRC.iterdir()):
-        if p.suffix in (".cu", ".cuh", ".cpp", ".h", ".inc"):
+        if p.name in SOURCES[name] or p.suffix in (".cuh", ".h", ".inc"):
             h.update(p.name.encode())
             h.update(p.read_bytes())
     h.update(" ".join(_flags()).encode())
     return h.hexdigest()
 
 
-def _so_path() -> Path:
-    return _build_dir() / f"{NAME}.so"
+def _so_path(name: str = NAME) -> Path:
+    return _build_dir() / f"{name}.so"
 
 
-def is_built() -> bool:
-    hp = _build_dir() / f"{NAME}.hash"
-    return _so_path().exists() and hp.exists() and hp.read_text().strip() == source_hash()
+def is_built(name: str = NAME) -> bool:
+    hp = _build_dir() / f"{name}.hash"
+    return _so_path(name).exists() and hp.exists() and hp.read_text().strip() == source_hash(name)
 
 
-def _import_so():
+def _import_so(name: str):
     import torch  # noqa: F401  (the extension links against libtorch)
-    spec = importlib.util.spec_from_file_location(NAME, str(_so_path()))
+    spec = importlib.util.spec_from_file_location(name, str(_so_path(name)))
     mod = importlib.util.module_from_spec(spec)
     spec.loader.exec_module(mod)
-    sys.modules[NAME] = mod
+    sys.modules[name] = mod
     return mod
 
 
-def build(verbose: bool = False, force: bool = False):
-    """Compile every source for sm_100a (cross-compiles without a GPU) and return the module."""
-    global _module
-    if not force and is_built():
-        _module = _import_so()
-        return _module
+def build_extension(name: str, verbose: bool = False, force: bool = False):
+    """Compile one extension for sm_100a (cross-compiles without a GPU) unless its binary is current; returns the module."""
+    if not force and is_built(name):
+        _modules[name] = _import_so(name)
+        return _modules[name]
     from torch.utils import cpp_extension
     _build_dir().mkdir(exist_ok=True)
     os.environ.setdefault("TORCH_CUDA_ARCH_LIST", "10.0a")
     os.environ.setdefault("MAX_JOBS", str(max(1, (os.cpu_count() or 2))))
+    # ninja's build file carries one extension: each has its own directory, the finished binary lands beside the others
+    work = _build_dir() if name == NAME else _build_dir() / name
+    work.mkdir(exist_ok=True)
     cpp_extension.load(
-        name=NAME,
-        sources=[str(s) for s in _existing_sources()],
+        name=name,
+        sources=[str(CSRC / s) for s in SOURCES[name]],
         extra_cflags=["-O2", "-std=c++17"] + (["-DLLM_BOUNDS_CHECK"] if _bounds_check() else []),
         extra_cuda_cflags=_flags(),
         extra_include_paths=[str(CSRC)],
-        build_directory=str(_build_dir()),
+        build_directory=str(work),
         with_cuda=True,
         verbose=verbose,
-        is_python_module=True,
+        is_python_module=name == NAME,
+        is_standalone=False,
     )
-    (_build_dir() / f"{NAME}.hash").write_text(source_hash())
-    _module = sys.modules.get(NAME) or _import_so()
-    return _module
+    if work != _build_dir():
+        os.replace(work / f"{name}.so", _so_path(name))
+    (_build_dir() / f"{name}.hash").write_text(source_hash(name))
+    _modules[name] = sys.modules.get(name) or _import_so(name)
+    return _modules[name]
+
+
+def build(verbose: bool = False, force: bool = False):
+    """Compile every extension; returns the main module."""
+    for name in SOURCES:
+        build_extension(name, verbose, force)
+    return _modules[NAME]
 
 
 def build_bounds_check_variant() -> None:
@@ -103,16 +116,15 @@ def build_bounds_check_variant() -> None:
     subprocess.run([sys.executable, "-c", code], check=True, env=env, cwd=str(Path(__file__).resolve().parents[2]))
 
 
-def load():
-    """The extension module; built on first use if the in-tree binary is missing or stale."""
-    global _module
-    if _module is None:
-        _module = build()
-    return _module
+def load(name: str = NAME):
+    """An extension module; built on first use if the in-tree binary is missing or stale."""
+    if name not in _modules:
+        build_extension(name)
+    return _modules[name]
 
 
-def so_path() -> str:
-    return str(_so_path())
+def so_path(name: str = NAME) -> str:
+    return str(_so_path(name))
 
 
 if __name__ == "__main__":

@@ -1,0 +1,105 @@
+// Launchers of the kernels around latent attention (low-rank key/value cache shared by all heads), of the fused norms and of
+// the small-batch matrix product on 16-bit weights.  `f32` selects the 32-bit build of a kernel (activations, weights and cache
+// as float) instead of the bf16 one; residual stream, norms, angles, scores and softmax are 32-bit in both.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stddef.h>
+
+namespace llm {
+
+// h[t] = (add ? h[t] : 0) + RMSNorm(y[row(t)]) * w_post ; xn[t] = RMSNorm(h[t]) * w_next ; copies of h[t] in the activation type
+struct ResidNormParams {
+    const void* y;                 // activation type; nullptr: h is only read
+    size_t y_stride;
+    const int* y_rows;             // optional gather (embedding lookup): row(t) = y_rows[t]
+    int n_y_rows;                  // rows of y (bounds-check build)
+    const float* w_post;           // [d]
+    float* h;                      // [T, d]
+    int add;
+    const float* w_next;           // optional [d]
+    void* xn;                      // [T, d]
+    void *copy0, *copy1;           // optional
+    size_t copy_stride;
+    int d;
+    float eps;
+};
+cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cudaStream_t st);
+
+// act[t, j] = gelu_tanh(gu[t, j]) * gu[t, ff + j]
+cudaError_t launch_gelu_mul(const void* gu, void* act, int rows, int ff, bool f32, cudaStream_t st);
+
+// out[t, i] = magnitude * (cos, sin)(positions[t] * freqs[i])
+cudaError_t launch_rope_angles(const int* positions, const double* freqs, double magnitude, float2* out, int rows, int half, cudaStream_t st);
+
+// Down projection row [q latent | kv latent | rotated key] -> normed query latent, and the token's cache row
+// [normed kv latent, padded to rot_off | rotated key part, padded to width].
+struct LatentPrepParams {
+    const void* down; size_t down_stride;
+    const float *q_norm, *kv_norm;
+    const float2* angles; int half;            // [T, half]
+    const int *positions, *seq_ids, *block_table;
+    int max_pages, n_seqs, n_pages;
+    void* cq; size_t cq_stride;                // [T, cq_stride], columns behind q_rank are zeroed
+    void* kv;                                  // [n_pages, 64, width]
+    int q_rank, kv_rank, rot_dim, rot_off, width;
+    float eps;
+};
+cudaError_t launch_latent_prep(const LatentPrepParams& p, int rows, bool f32, cudaStream_t st);
+
+// Attention of single rows, each with its own sequence and position, over the latent cache: queries are already multiplied
+// into the latent space, the result is the weighted sum of latents per head.
+struct LatentRowsParams {
+    const void* q_lat; size_t ql_row, ql_head; // [row z][head][kv_rank padded to rot_off]
+    const void* q; size_t q_row, q_head;       // [token][head] up-projected query; its rotated part starts at q_rot_off
+    int q_rot_off;
+    const float2* angles; int half;
+    const int* rows;                           // token of row z (nullptr: z)
+    const int *positions, *seq_ids, *block_table;
+    int max_pages, n_seqs, n_pages;
+    const void* kv;                            // [n_pages, 64, width]
+    int width, rot_off, rot_dim;
+    int n_heads, window;
+    float scale;
+    const float* sink;                         // optional [n_heads]
+    void* out; size_t out_row, out_head;       // [row z][head][rot_off]
+    float *part_o, *part_ml;                   // [rows * head groups * splits][16][rot_off], [...][16][2]
+};
+cudaError_t launch_latent_rows(const LatentRowsParams& p, int rows, int n_splits, bool f32, cudaStream_t st);
+// whether the tensor-core kernel takes these sizes (otherwise launch_latent_rows runs the plain kernel)
+bool latent_rows_has_kernel(int width, int rot_off);
+
+// Cache rows of the sequences' visible keys -> contiguous rows: buffer row k_off[s] + i holds position k_pos0[s] + i.
+struct LatentSeq { int seq, q_start, q_len, q_pos0, k_off, k_pos0, k_len, pad; };
+cudaError_t launch_latent_gather(const void* kv, const LatentSeq* seqs, int n, int max_k_len, const int* block_table, int max_pages,
+                                 int n_pages, int width, void* out, bool f32, cudaStream_t st);
+
+// Attention of prompt chunks with keys and values written out per head.
+struct LatentChunkParams {
+    const __nv_bfloat16* q; size_t q_row, q_head;      // [token][head][dim | rot]
+    const float2* angles; int half;
+    const __nv_bfloat16* kvx; size_t kvx_row, kvx_head; // [key][head][dim | vdim]
+    const __nv_bfloat16* lat; size_t lat_row; int rot_off;
+    const LatentSeq* seqs;
+    __nv_bfloat16* out; size_t out_row;                // [token][head * vdim]
+    int dim, rot, vdim, n_heads, window;               // padded to multiples of 8
+    float scale;
+    const float* sink;
+};
+cudaError_t launch_latent_chunk(const LatentChunkParams& p, int n_seqs, int max_q_len, cudaStream_t st);
+bool latent_chunk_has_kernel(int dk, int dv);
+
+// out[z][m, :] = x[z][m, :] W[z]^T for up to 4 rows, bf16 weights.  gelu: W holds 2n rows and out = gelu_tanh(first n) * second n.
+struct GemvDenseParams {
+    const __nv_bfloat16* w; size_t w_z; int ldw;
+    const __nv_bfloat16* x; size_t x_row, x_z;
+    void* out; size_t o_row, o_z;
+    int n, k, m, z;
+    bool out_f32, gelu;
+};
+cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st);
+
+int bounds_status_latent(bool reset);
+int bounds_status_dense(bool reset);
+
+}  // namespace llm

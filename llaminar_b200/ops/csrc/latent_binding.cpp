@@ -1,0 +1,230 @@
+// Python bindings of the kernels of latent-attention models: an extension of its own, so that a process that serves only such
+// a model compiles and loads nothing else.  Every tensor is checked on the host before a launch.
+#include <ATen/cuda/CUDAContext.h>
+#include <torch/extension.h>
+
+#include "latent.h"
+#include "launch.h"
+
+namespace {
+
+using torch::Tensor;
+using OptTensor = c10::optional<Tensor>;
+
+cudaStream_t stream() { return at::cuda::getCurrentCUDAStream().stream(); }
+
+void check(cudaError_t e, const char* what) { TORCH_CHECK(e == cudaSuccess, what, ": ", cudaGetErrorString(e)); }
+
+bool is_f32(const Tensor& t, const char* name) {
+    TORCH_CHECK(t.is_cuda(), name, " must be on the GPU");
+    TORCH_CHECK(t.scalar_type() == torch::kFloat32 || t.scalar_type() == torch::kBFloat16, name, " must be float32 or bfloat16");
+    return t.scalar_type() == torch::kFloat32;
+}
+void want(const Tensor& t, torch::ScalarType st, const char* name) {
+    TORCH_CHECK(t.is_cuda() && t.scalar_type() == st && t.is_contiguous(), name, " must be a contiguous ", st, " CUDA tensor");
+}
+void want_like(const Tensor& t, bool f32, const char* name) {
+    TORCH_CHECK(is_f32(t, name) == f32, name, " has the wrong element type");
+}
+const int* ints(const Tensor& t, const char* name) {
+    want(t, torch::kInt32, name);
+    return t.data_ptr<int>();
+}
+const float* floats(const Tensor& t, int64_t n, const char* name) {
+    want(t, torch::kFloat32, name);
+    TORCH_CHECK(t.numel() == n, name, " must hold ", n, " values");
+    return t.data_ptr<float>();
+}
+const float2* angle_ptr(const Tensor& t, int64_t rows) {
+    want(t, torch::kFloat32, "angles");
+    TORCH_CHECK(t.dim() == 3 && t.size(0) >= rows && t.size(2) == 2, "angles must be [rows, dims/2, 2]");
+    return reinterpret_cast<const float2*>(t.data_ptr<float>());
+}
+
+void resid_norm(const OptTensor& y, const OptTensor& y_rows, const OptTensor& w_post, const Tensor& h, bool add, const OptTensor& w_next,
+                const OptTensor& xn, const OptTensor& copy0, const OptTensor& copy1, double eps) {
+    llm::ResidNormParams p = {};
+    want(h, torch::kFloat32, "h");
+    const int64_t T = h.size(0), d = h.size(1);
+    if (T == 0) return;
+    bool f32 = false, typed = false;
+    auto elem = [&](const Tensor& t, const char* name) {
+        const bool f = is_f32(t, name);
+        TORCH_CHECK(!typed || f == f32, name, " has another element type than the other activations");
+        f32 = f; typed = true;
+        TORCH_CHECK(t.dim() == 2 && t.size(1) == d && t.stride(1) == 1, name, " must be rows of ", d, " values");
+    };
+    if (y) {
+        elem(*y, "y");
+        p.y = y->data_ptr(); p.y_stride = y->stride(0);
+        p.w_post = floats(w_post.value(), d, "w_post");
+        p.n_y_rows = y->size(0);
+        if (y_rows) {
+            p.y_rows = ints(*y_rows, "y_rows");
+            TORCH_CHECK(y_rows->numel() == T, "y_rows must name one row per token");
+        } else {
+            TORCH_CHECK(y->size(0) == T, "y must have as many rows as h");
+        }
+    }
+    p.h = h.data_ptr<float>(); p.add = add;
+    if (w_next) {
+        elem(xn.value(), "xn");
+        TORCH_CHECK(xn->is_contiguous() && xn->size(0) == T, "xn must be contiguous");
+        p.w_next = floats(*w_next, d, "w_next"); p.xn = xn->data_ptr();
+    }
+    if (copy0) { elem(*copy0, "copy0"); TORCH_CHECK(copy0->size(0) == T, "copy0 rows"); p.copy0 = copy0->data_ptr(); p.copy_stride = copy0->stride(0); }
+    if (copy1) {
+        elem(*copy1, "copy1");
+        TORCH_CHECK(copy1->size(0) == T && (!copy0 || copy1->stride(0) == copy0->stride(0)), "copy1 must have copy0's strides");
+        p.copy1 = copy1->data_ptr(); p.copy_stride = copy1->stride(0);
+    }
+    p.d = d; p.eps = eps;
+    check(llm::launch_resid_norm(p, T, f32, stream()), "resid_norm");
+}
+
+void gelu_mul(const Tensor& gu, const Tensor& act) {
+    const bool f32 = is_f32(gu, "gu");
+    want_like(act, f32, "act");
+    TORCH_CHECK(gu.is_contiguous() && act.is_contiguous() && gu.size(0) == act.size(0) && gu.size(1) == 2 * act.size(1), "gu must be [rows, 2 ff]");
+    if (gu.size(0) == 0) return;
+    check(llm::launch_gelu_mul(gu.data_ptr(), act.data_ptr(), gu.size(0), act.size(1), f32, stream()), "gelu_mul");
+}
+
+void rope_angles(const Tensor& positions, const Tensor& freqs, double magnitude, const Tensor& out) {
+    want(freqs, torch::kFloat64, "freqs");
+    const int rows = positions.numel(), half = freqs.numel();
+    angle_ptr(out, rows);
+    TORCH_CHECK(out.size(1) == half, "angles must have one column per frequency");
+    check(llm::launch_rope_angles(ints(positions, "positions"), freqs.data_ptr<double>(), magnitude, reinterpret_cast<float2*>(out.data_ptr<float>()),
+                                  rows, half, stream()), "rope_angles");
+}
+
+void latent_prep(const Tensor& down, const Tensor& q_norm, const Tensor& kv_norm, const Tensor& angles, const Tensor& positions, const Tensor& seq_ids,
+                 const Tensor& block_table, const Tensor& cq, const Tensor& kv, int64_t rot_dim, int64_t rot_off, double eps) {
+    const bool f32 = is_f32(down, "down");
+    want_like(cq, f32, "cq"); want_like(kv, f32, "kv");
+    const int64_t T = down.size(0), q_rank = q_norm.numel(), kv_rank = kv_norm.numel();
+    if (T == 0) return;
+    TORCH_CHECK(down.stride(1) == 1 && down.size(1) >= q_rank + kv_rank + rot_dim, "down: too few columns");
+    TORCH_CHECK(cq.is_contiguous() && cq.size(0) == T && cq.size(1) >= q_rank, "cq shape");
+    TORCH_CHECK(kv.is_contiguous() && kv.dim() == 3 && kv.size(1) == 64, "kv must be [pages, 64, width]");
+    TORCH_CHECK(rot_off >= kv_rank && rot_off + rot_dim <= kv.size(2), "cache row too narrow");
+    TORCH_CHECK(positions.numel() == T && seq_ids.numel() == T, "positions / seq_ids");
+    llm::LatentPrepParams p = {};
+    p.down = down.data_ptr(); p.down_stride = down.stride(0);
+    p.q_norm = floats(q_norm, q_rank, "q_norm"); p.kv_norm = floats(kv_norm, kv_rank, "kv_norm");
+    p.angles = angle_ptr(angles, T); p.half = angles.size(1);
+    TORCH_CHECK(2 * p.half <= rot_dim, "more angles than the rotated part has pairs");
+    p.positions = ints(positions, "positions"); p.seq_ids = ints(seq_ids, "seq_ids"); p.block_table = ints(block_table, "block_table");
+    p.n_seqs = block_table.size(0); p.max_pages = block_table.size(1); p.n_pages = kv.size(0);
+    p.cq = cq.data_ptr(); p.cq_stride = cq.size(1); p.kv = kv.data_ptr();
+    p.q_rank = q_rank; p.kv_rank = kv_rank; p.rot_dim = rot_dim; p.rot_off = rot_off; p.width = kv.size(2); p.eps = eps;
+    check(llm::launch_latent_prep(p, T, f32, stream()), "latent_prep");
+}
+
+// q_lat [heads, rows, rot_off]; q [tokens, heads, head size] (contiguous); out [heads, rows, rot_off]
+void latent_rows(const Tensor& q_lat, const Tensor& q, int64_t q_rot_off, const Tensor& angles, const OptTensor& rows, const Tensor& positions,
+                 const Tensor& seq_ids, const Tensor& block_table, const Tensor& kv, int64_t rot_dim, int64_t window, double scale,
+                 const OptTensor& sink, const Tensor& out, const OptTensor& part_o, const OptTensor& part_ml, int64_t n_splits) {
+    const bool f32 = is_f32(kv, "kv");
+    want_like(q_lat, f32, "q_lat"); want_like(q, f32, "q"); want_like(out, f32, "out");
+    const int64_t H = q_lat.size(0), n = q_lat.size(1), R = q_lat.size(2);
+    if (n == 0) return;
+    TORCH_CHECK(q_lat.stride(2) == 1 && out.stride(2) == 1 && out.sizes() == q_lat.sizes(), "q_lat / out must be [heads, rows, latent]");
+    TORCH_CHECK(q.is_contiguous() && q.dim() == 3 && q.size(1) == H && q.size(2) >= q_rot_off + rot_dim, "q must be [tokens, heads, size]");
+    TORCH_CHECK(kv.is_contiguous() && kv.dim() == 3 && kv.size(1) == 64 && R + rot_dim <= kv.size(2), "kv must be [pages, 64, width]");
+    const int64_t T = q.size(0);
+    TORCH_CHECK(positions.numel() == T && seq_ids.numel() == T && (rows ? rows->numel() == n : T == n), "row description");
+    llm::LatentRowsParams p = {};
+    p.q_lat = q_lat.data_ptr(); p.ql_row = q_lat.stride(1); p.ql_head = q_lat.stride(0);
+    p.q = q.data_ptr(); p.q_row = q.stride(0); p.q_head = q.stride(1); p.q_rot_off = q_rot_off;
+    p.angles = angle_ptr(angles, T); p.half = angles.size(1);
+    TORCH_CHECK(2 * p.half <= rot_dim, "more angles than the rotated part has pairs");
+    p.rows = rows ? ints(*rows, "rows") : nullptr;
+    p.positions = ints(positions, "positions"); p.seq_ids = ints(seq_ids, "seq_ids"); p.block_table = ints(block_table, "block_table");
+    p.n_seqs = block_table.size(0); p.max_pages = block_table.size(1); p.n_pages = kv.size(0);
+    p.kv = kv.data_ptr(); p.width = kv.size(2); p.rot_off = R; p.rot_dim = rot_dim;
+    p.n_heads = H; p.window = window; p.scale = scale;
+    p.sink = sink ? floats(*sink, H, "sink") : nullptr;
+    p.out = out.data_ptr(); p.out_row = out.stride(1); p.out_head = out.stride(0);
+    if (!f32 && llm::latent_rows_has_kernel(p.width, p.rot_off)) {
+        TORCH_CHECK(p.out_row % 4 == 0 && p.out_head % 4 == 0, "out strides must be multiples of 4");
+        TORCH_CHECK(n_splits >= 1 && n_splits <= 65535, "n_splits");
+        if (n_splits > 1) {
+            const int64_t parts = n * ((H + 15) / 16) * n_splits * 16;
+            want(part_o.value(), torch::kFloat32, "part_o"); want(part_ml.value(), torch::kFloat32, "part_ml");
+            TORCH_CHECK(part_o->numel() >= parts * R && part_ml->numel() >= parts * 2, "split scratch too small");
+            p.part_o = part_o->data_ptr<float>(); p.part_ml = part_ml->data_ptr<float>();
+        }
+    }
+    check(llm::launch_latent_rows(p, n, n_splits, f32, stream()), "latent_rows");
+}
+
+// seqs: int32 [n, 8], see LatentSeq; the limits are the host's view of the same numbers
+void latent_gather(const Tensor& kv, const Tensor& seqs, int64_t max_k_len, const Tensor& block_table, const Tensor& out) {
+    const bool f32 = is_f32(kv, "kv");
+    want_like(out, f32, "out");
+    TORCH_CHECK(kv.is_contiguous() && out.is_contiguous() && kv.dim() == 3 && out.size(1) == kv.size(2), "gather shapes");
+    TORCH_CHECK((kv.size(2) * kv.element_size()) % 16 == 0, "cache rows must be whole 16-byte units");
+    TORCH_CHECK(seqs.dim() == 2 && seqs.size(1) == 8, "seqs must be [n, 8]");
+    if (seqs.size(0) == 0 || max_k_len == 0) return;
+    check(llm::launch_latent_gather(kv.data_ptr(), reinterpret_cast<const llm::LatentSeq*>(ints(seqs, "seqs")), seqs.size(0), max_k_len,
+                                    ints(block_table, "block_table"), block_table.size(1), kv.size(0), kv.size(2), out.data_ptr(), f32, stream()),
+          "latent_gather");
+}
+
+void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& kvx, const Tensor& lat, int64_t rot_off, const Tensor& seqs, int64_t max_q_len,
+                  const Tensor& out, int64_t dim, int64_t rot, int64_t vdim, int64_t window, double scale, const OptTensor& sink) {
+    for (auto& t : {q, kvx, lat, out}) want(t, torch::kBFloat16, "latent_chunk operand");
+    const int64_t T = q.size(0), H = q.size(1);
+    TORCH_CHECK(q.dim() == 3 && q.size(2) == dim + rot, "q must be [tokens, heads, dim + rot]");
+    TORCH_CHECK(kvx.size(1) == H * (dim + vdim) && kvx.size(0) <= lat.size(0) && rot_off + rot <= lat.size(1), "key buffers");
+    TORCH_CHECK(out.size(0) == T && out.size(1) == H * vdim, "out must be [tokens, heads * vdim]");
+    TORCH_CHECK(seqs.dim() == 2 && seqs.size(1) == 8, "seqs must be [n, 8]");
+    TORCH_CHECK(dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && rot_off % 8 == 0 && lat.size(1) % 8 == 0, "sizes must be multiples of 8");
+    if (seqs.size(0) == 0) return;
+    llm::LatentChunkParams p = {};
+    auto b = [](const Tensor& t) { return reinterpret_cast<const __nv_bfloat16*>(t.data_ptr()); };
+    p.q = b(q); p.q_row = q.stride(0); p.q_head = q.stride(1);
+    p.angles = angle_ptr(angles, T); p.half = angles.size(1);
+    TORCH_CHECK(2 * p.half <= rot, "more angles than the rotated part has pairs");
+    p.kvx = b(kvx); p.kvx_row = kvx.size(1); p.kvx_head = dim + vdim;
+    p.lat = b(lat); p.lat_row = lat.size(1); p.rot_off = rot_off;
+    p.seqs = reinterpret_cast<const llm::LatentSeq*>(ints(seqs, "seqs"));
+    p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr()); p.out_row = out.size(1);
+    p.dim = dim; p.rot = rot; p.vdim = vdim; p.n_heads = H; p.window = window; p.scale = scale;
+    p.sink = sink ? floats(*sink, H, "sink") : nullptr;
+    check(llm::launch_latent_chunk(p, seqs.size(0), max_q_len, stream()), "latent_chunk");
+}
+
+// w [z, n, k] (gelu: [z, 2n, k]), x [z, m, k], out [z, m, n]; the last dimension of each is dense
+void gemv_dense(const Tensor& w, const Tensor& x, const Tensor& out, bool gelu) {
+    TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && x.scalar_type() == torch::kBFloat16, "gemv_dense takes bf16 operands");
+    TORCH_CHECK(w.dim() == 3 && x.dim() == 3 && out.dim() == 3 && w.stride(2) == 1 && x.stride(2) == 1 && out.stride(2) == 1, "gemv_dense layouts");
+    llm::GemvDenseParams p = {};
+    p.z = w.size(0); p.n = gelu ? w.size(1) / 2 : w.size(1); p.k = w.size(2); p.m = x.size(1);
+    TORCH_CHECK(x.size(0) == p.z && out.size(0) == p.z && x.size(2) == p.k && out.size(1) == p.m && out.size(2) == p.n, "gemv_dense shapes");
+    p.out_f32 = is_f32(out, "out"); p.gelu = gelu;
+    p.w = reinterpret_cast<const __nv_bfloat16*>(w.data_ptr()); p.w_z = w.stride(0); p.ldw = w.stride(1);
+    p.x = reinterpret_cast<const __nv_bfloat16*>(x.data_ptr()); p.x_row = x.stride(1); p.x_z = x.stride(0);
+    p.out = out.data_ptr(); p.o_row = out.stride(1); p.o_z = out.stride(0);
+    TORCH_CHECK(reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "gemv_dense operands must be 16-byte aligned");
+    check(llm::launch_gemv_dense(p, stream()), "gemv_dense");
+}
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+    m.def("resid_norm", &resid_norm);
+    m.def("gelu_mul", &gelu_mul);
+    m.def("rope_angles", &rope_angles);
+    m.def("latent_prep", &latent_prep);
+    m.def("latent_rows", &latent_rows);
+    m.def("latent_rows_has_kernel", &llm::latent_rows_has_kernel);
+    m.def("latent_gather", &latent_gather);
+    m.def("latent_chunk", &latent_chunk);
+    m.def("latent_chunk_has_kernel", &llm::latent_chunk_has_kernel);
+    m.def("gemv_dense", &gemv_dense);
+    m.def("set_pdl", [](bool on) { llm::pdl_enabled() = on; });
+    m.def("bounds_status", [](bool reset) { return llm::bounds_status_latent(reset) | llm::bounds_status_dense(reset); });
+}

@@ -1,0 +1,105 @@
+"""Python surface of the latent-attention extension (csrc/latent_attention.cu, csrc/dense_ops.cu).
+
+As in :mod:`llaminar_b200.ops`, every call launches hand-written CUDA on the current stream; there is no fallback.  The
+extension is separate from the quantised-weight kernels, so a process that serves a latent model loads only this one.
+"""
+from __future__ import annotations
+
+import torch
+
+from . import _count
+from . import build as _build
+
+ROWS_PER_GROUP = 16            # heads that share the M dimension of the row kernel's MMA
+KEYS_PER_TILE = 32
+GEMV_MAX_ROWS = 4
+_GEMV_SMEM = 200 * 1024
+_ready = False
+
+
+def ext():
+    global _ready
+    mod = _build.load(_build.LATENT)
+    if not _ready:
+        from ..utils.env import debug_env
+        mod.set_pdl(bool(debug_env().pdl))
+        _ready = True
+    return mod
+
+
+def resid_norm(h, y=None, w_post=None, *, add=True, y_rows=None, w_next=None, xn=None, copy0=None, copy1=None, eps: float) -> None:
+    """h = (h if add) + RMSNorm(y) * w_post (``y`` None: h is only read; ``y_rows`` gathers rows of y), then
+    xn = RMSNorm(h) * w_next and copies of h in the activation type.  One launch."""
+    ext().resid_norm(y, y_rows, w_post, h, add, w_next, xn, copy0, copy1, eps)
+    _count()
+
+
+def gelu_mul(gu: torch.Tensor, act: torch.Tensor) -> None:
+    """act = gelu_tanh(gu[:, :ff]) * gu[:, ff:]"""
+    ext().gelu_mul(gu, act)
+    _count()
+
+
+def rope_angles(positions: torch.Tensor, freqs: torch.Tensor, magnitude: float, out: torch.Tensor) -> None:
+    """out[t, i] = magnitude * (cos, sin)(positions[t] * freqs[i]); freqs in double precision."""
+    ext().rope_angles(positions, freqs, magnitude, out)
+    _count()
+
+
+def latent_prep(down, q_norm, kv_norm, angles, positions, seq_ids, block_table, cq, kv, rot_dim: int, rot_off: int, eps: float) -> None:
+    """Rows [q latent | kv latent | rotated key part] of the down projection -> normed query latents ``cq`` and the tokens' rows
+    of the latent cache ``kv`` (both norms, the rotation and the append in one launch)."""
+    ext().latent_prep(down, q_norm, kv_norm, angles, positions, seq_ids, block_table, cq, kv, rot_dim, rot_off, eps)
+    _count()
+
+
+def rows_splits(n_rows: int, n_heads: int, max_keys: int, latent: int, capacity: int) -> int:
+    """Key splits of the row kernel: enough CTAs for two per SM, at least two key tiles per split, partial sums within
+    ``capacity`` floats."""
+    groups = -(-n_heads // ROWS_PER_GROUP)
+    tiles = -(-max_keys // KEYS_PER_TILE) + 1
+    want = max(1, min(296 // max(1, n_rows * groups), tiles // 2, 64))
+    return max(1, min(want, capacity // max(1, n_rows * groups * ROWS_PER_GROUP * latent)))
+
+
+def latent_rows(q_lat, q, q_rot_off: int, angles, rows, positions, seq_ids, block_table, kv, rot_dim: int, window: int, scale: float,
+                sink, out, part_o, part_ml, n_splits: int) -> None:
+    """Attention of single rows over the latent cache, queries and results in the latent space ([heads, rows, latent])."""
+    e = ext()
+    e.latent_rows(q_lat, q, q_rot_off, angles, rows, positions, seq_ids, block_table, kv, rot_dim, window, scale, sink, out,
+                  part_o, part_ml, n_splits)
+    _count(2 if n_splits > 1 and kv.dtype == torch.bfloat16 and e.latent_rows_has_kernel(kv.shape[2], q_lat.shape[2]) else 1)
+
+
+def latent_gather(kv, seqs, max_k_len: int, block_table, out) -> None:
+    """The cache rows of the keys that the sequences of ``seqs`` see, one after the other."""
+    ext().latent_gather(kv, seqs, max_k_len, block_table, out)
+    _count()
+
+
+def latent_chunk(q, angles, kvx, lat, rot_off: int, seqs, max_q_len: int, out, dim: int, rot: int, vdim: int, window: int,
+                 scale: float, sink) -> None:
+    """Attention of prompt chunks on keys and values written out per head (``kvx``) and the shared rotated parts in ``lat``."""
+    ext().latent_chunk(q, angles, kvx, lat, rot_off, seqs, max_q_len, out, dim, rot, vdim, window, scale, sink)
+    _count()
+
+
+def chunk_has_kernel(dk: int, dv: int) -> bool:
+    return bool(ext().latent_chunk_has_kernel(dk, dv))
+
+
+def gemv_fits(w: torch.Tensor, x: torch.Tensor) -> bool:
+    """Whether `gemv_dense` takes this product: few bf16 rows, 16-byte rows."""
+    k = w.shape[-1]
+    return (w.dtype == torch.bfloat16 and x.shape[-2] <= GEMV_MAX_ROWS and k % 8 == 0 and x.stride(-2) % 8 == 0 and w.stride(-2) % 8 == 0
+            and x.shape[-2] * k * 2 <= _GEMV_SMEM and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+
+
+def gemv_dense(w, x, out, gelu: bool = False) -> None:
+    """out[z] = x[z] @ w[z]^T for at most four bf16 rows; ``gelu``: w stacks gate and up, out = gelu_tanh(gate) * up."""
+    ext().gemv_dense(w, x, out, gelu)
+    _count()
+
+
+def bounds_status(reset: bool = True) -> int:
+    return int(ext().bounds_status(bool(reset)))

@@ -57,6 +57,9 @@ class TPPlan:
         if tp < 1:
             errs.append("tensor-parallel degree must be >= 1")
             return errs
+        if getattr(cfg, "is_latent", False):
+            # the latent cache is shared by all heads and the matrices are not stored in shardable blocks
+            return errs if tp == 1 else [f"{cfg.arch} models run on one GPU (tp={tp} was asked for)"]
         if cfg.n_heads % tp:
             errs.append(f"n_heads={cfg.n_heads} is not divisible by tp={tp}")
         if cfg.n_kv_heads >= tp:

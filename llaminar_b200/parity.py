@@ -46,6 +46,8 @@ def compare(weights, device: str, prompt_tokens: int = 96, decode_steps: int = 4
     from .models.reference import ReferenceModel
     dev = torch.device(device)
     cfg = weights.config
+    if cfg.is_latent:
+        raise ValueError(f"the layer report has no reference for {cfg.arch} models")
     if dev.type == "cuda":
         from .engine.cuda_model import CudaModel
         model = CudaModel(weights, dev, max_tokens=max(prompt_tokens, 64))

@@ -99,6 +99,11 @@ class ExecutionPlan:
 
 def layer_weight_bytes(cfg: ModelConfig, recipe: QuantRecipe, layer: int, tp: TPPlan) -> float:
     d, D = cfg.d_model, cfg.head_dim
+    if cfg.is_latent:                           # stored as 16-bit matrices whatever the file's format
+        m, ff = cfg.mixers[layer], cfg.ff_width(layer)
+        n = d * (m.q_rank + m.kv_rank + m.rot_dim) + m.heads * (m.dim + m.rot_dim) * m.q_rank
+        n += m.heads * (2 * m.dim + m.vdim) * m.kv_rank + d * m.heads * m.vdim + 3 * d * ff        # the key matrices are held twice
+        return 2.0 * n
     t = lambda name: recipe.for_tensor(f"blk.{layer}.{name}.weight", layer, cfg.n_layers)
     if cfg.is_gdn_layer(layer):
         # linear-attention block: q | k of every key head, this rank's value heads of v and z, alpha / b, output projection
@@ -133,6 +138,9 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
         return plan
     stages = layout["stages"]
     n_stages = len(stages)
+    if cfg.is_latent and n_stages > 1:
+        plan.errors.append(f"{cfg.arch} models run on one GPU ({n_stages} pipeline stages were asked for)")
+        return plan
     rank = 0
     for si, (dom, devices, first, last) in enumerate(stages):
         if last < 0:
@@ -154,6 +162,9 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
             pages = batch_size * ((ctx_size + 63) // 64 + 1) + 64
             stage_layers = range(first, last + 1)
             rp.kv_bytes = int(pages * len(cfg.kv_layers(stage_layers)) * 2 * tp.n_kv_local * 64 * cfg.head_dim * 2)
+            if cfg.is_latent:                   # one cache layer per layer run; input matrix of the looped layers
+                rp.kv_bytes = int(pages * sum(cfg.mixers[i].cache_width for i, _ in cfg.layer_runs()) * 64 * 2)
+                rp.weight_bytes += 4 * cfg.d_model * cfg.d_model if cfg.loop else 0
             if cfg.is_hybrid:
                 # one fp32 state slot per batch lane (+1 scratch) for every linear-attention layer of the stage
                 from .engine.kv_cache import HybridState
@@ -164,6 +175,10 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
             ff = (tp.ff_stop - tp.ff_start) if not cfg.is_moe else cfg.expert_ff
             rp.activation_bytes = int(T * (cfg.d_model * (4 + 2) + (tp.n_heads_local + 2 * tp.n_kv_local) * cfg.head_dim * 2
                                            + 2 * tp.n_heads_local * cfg.head_dim * 2 + ff * 2))
+            if cfg.is_latent:
+                m = max(cfg.mixers, key=lambda m: m.heads * (2 * m.dim + m.rot_dim + 2 * m.vdim))
+                rp.activation_bytes = int(T * (cfg.d_model * (4 + 8) + 2 * (m.heads * (2 * m.dim + m.rot_dim + 2 * m.vdim) + 2 * m.q_rank
+                                                                            + 2 * m.cache_width + 3 * ff)))
             rp.workspace_bytes = int(256 * 65536 * 4 + (1 << 22) * 4 + batch_size * 4 * (tp.vocab_stop - tp.vocab_start) * 4)
             if rp.total_bytes > hbm_bytes * 0.95:
                 plan.errors.append(f"rank {rank} ({dev}): needs {rp.total_bytes / 1e9:.1f} GB, device has {hbm_bytes / 1e9:.0f} GB")
