@@ -45,6 +45,7 @@ def parse_args():
     ap.add_argument("--layers", type=int, default=0, help="debug only: truncate the model (result is not a valid bench)")
     ap.add_argument("--skip-extras", action="store_true", help="only the headline region (no bs1 / prefill / TTFT)")
     ap.add_argument("--no-graphs", action="store_true", help="profiling aid: launch decode kernels one by one instead of replaying a graph")
+    ap.add_argument("--latent", action="store_true", help="instead of the headline: kernels and models with latent attention beside the like parts of a grouped-query model")
     return ap.parse_args()
 
 
@@ -284,7 +285,7 @@ def log(msg: str) -> None:
 
 T_START = time.time()
 MODEL_DEFAULTS = {"qwen3-8b": ("Q4_K_M", 2048), "qwen3-32b": ("Q4_K_S", 1024),
-                  "qwen3.5-27b": ("Q4_K_M", 512), "qwen3.5-35b-a3b": ("Q4_K_M", 512)}      # the hybrid shapes (--model ...)
+                  "pozivik-8b": ("BF16", 2048), "qwen3.5-27b": ("Q4_K_M", 512), "qwen3.5-35b-a3b": ("Q4_K_M", 512)}      # the hybrid shapes (--model ...)
 
 
 def measure(model_name: str, recipe: str, S: int, args, tp, dev, world: int, rank: int, local: int, extras_on: bool) -> dict:
@@ -298,7 +299,8 @@ def measure(model_name: str, recipe: str, S: int, args, tp, dev, world: int, ran
     from llaminar_b200.models.synth import synthesize
     cfg = SHAPES[model_name]
     if args.layers:
-        cfg = cfg.with_(n_layers=args.layers)
+        from llaminar_b200.bench_latent import cut
+        cfg = cut(cfg, args.layers)
     B, K, W = args.batch, args.steps, max(args.warmup, 3)
     t0 = time.time()
     log(f"synthesising {model_name} ({recipe}), {cfg.n_layers} layers")
@@ -430,6 +432,14 @@ def main():
     _keep_stdout_for_the_result()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.latent:
+        from llaminar_b200.bench_latent import run
+        sampler = ClockSampler(0)
+        sampler.start()
+        res = run(args.layers or 8, log)
+        print(json.dumps({"bench": "latent", **res, "clocks": sampler.stop()}))
+        sys.stdout.flush()
+        return 0
     import datetime
     import faulthandler
     import torch

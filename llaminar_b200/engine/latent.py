@@ -102,6 +102,7 @@ class LatentStack:
         c = self.cfg = model.cfg
         self.device, self.dtype = model.device, model.dtype
         self.f32 = self.dtype == torch.float32
+        self.rows_tc = self.chunk_tc = True             # tcgen05 forms of the attention kernels where the sizes fit
         # sums stay in 32 bits: no TF32 operands in 32-bit mode, no 16-bit reduction of split products otherwise
         if self.f32:
             torch.backends.cuda.matmul.allow_tf32 = False
@@ -110,6 +111,8 @@ class LatentStack:
         self.embed = self._mat(weights, "token_embd.weight")
         self.embed_norm = self._vec(weights, "token_embd_norm.weight")
         self.loop_in = DenseLinear(self._mat(weights, "loop_in.weight")) if c.loop else None
+        from .. import ops
+        self.status = ops.scratch_for(self.device).status               # word that a kernel sets when a bounded wait runs out
         self.rotaries: list = []
         self.freqs: list[torch.Tensor] = []
 
@@ -121,6 +124,7 @@ class LatentStack:
 
     # -- weights ---------------------------------------------------------------------------------------------
     def build_layer(self, L, w, i: int):
+        from ..ops import latent as ops
         c, m, p = self.cfg, self.cfg.mixers[i], f"blk.{i}."
         s = PaddedSizes.of(m)
         L.index, L.mixer, L.sizes = i, m, s
@@ -133,15 +137,14 @@ class LatentStack:
         L.q_b = DenseLinear(q.reshape(-1, s.q_rank))
         k = pad_to(self._mat(w, p + "attn_k_b.weight").view(m.heads, m.dim, m.kv_rank), s.heads, s.dim, s.latent)
         v = pad_to(self._mat(w, p + "attn_v_b.weight").view(m.heads, m.vdim, m.kv_rank), s.heads, s.vdim, s.latent)
-        kv = torch.cat([k, v], dim=1).contiguous()                      # [heads, dim | vdim, latent]
-        L.kv_b = DenseLinear(kv.view(-1, s.latent))
-        L.k_b, L.v_b = kv[:, :s.dim], kv[:, s.dim:]
+        L.k_b, L.v_b = k, v                                             # [heads, dim, latent], [heads, vdim, latent]
         L.k_bt = k.transpose(1, 2).contiguous()                         # [heads, latent, dim]: rows of the small-batch product
         o = self._mat(w, p + "attn_output.weight").view(-1, m.heads, m.vdim)
         L.wo = DenseLinear(pad_to(o, o.shape[0], s.heads, s.vdim).view(o.shape[0], -1))
         if m.rotary not in self.rotaries:
             self.rotaries.append(m.rotary)
             self.freqs.append(torch.tensor(m.rotary.frequencies(), dtype=torch.float64, device=self.device))
+        L.chunk_tc = not self.f32 and ops.chunk_tc_fits(s.dim, s.rot, s.vdim)
         L.rot_index = self.rotaries.index(m.rotary)
         L.ff = c.ff_width(i)
         if L.ff:
@@ -151,9 +154,10 @@ class LatentStack:
         return L
 
     def nbytes(self, layers) -> int:
-        n = self.embed.numel() * self.embed.element_size() + (self.loop_in.nbytes() if self.loop_in else 0)
+        n = (self.loop_in.nbytes() if self.loop_in else 0)
         for L in layers:
-            n += sum(x.nbytes() for x in (L.down_a, L.q_b, L.kv_b, L.wo)) + L.k_bt.numel() * L.k_bt.element_size()
+            n += sum(x.nbytes() for x in (L.down_a, L.q_b, L.wo))
+            n += (2 * L.k_b.numel() + L.v_b.numel()) * L.k_b.element_size()
             if L.ff:
                 n += L.gate_up.nbytes() + L.down.nbytes()
         return n
@@ -278,9 +282,10 @@ class LatentStack:
         else:
             torch.bmm(q_nope, L.k_b, out=q_lat)
         max_keys = min(bp.max_keys, m.window) if m.window else bp.max_keys
-        splits = 1 if self.f32 else ops.rows_splits(n, s.heads, max_keys, s.latent, self.part_o.numel())
+        group = ops.rows_group(kv_layer, s.latent, m.rot_dim, s.heads, self.rows_tc)
+        splits = ops.rows_splits(n, s.heads, group, self.rows_tc, max_keys, s.latent, self.part_o.numel())
         ops.latent_rows(q_lat, q, s.dim, bp.angles[L.rot_index], rows, fb.positions, fb.seq_ids, fb.block_table, kv_layer, m.rot_dim, m.window,
-                        m.scale, L.sink, o_lat, self.part_o, self.part_ml, splits)
+                        m.scale, L.sink, o_lat, self.part_o, self.part_ml, splits, group, self.status)
         out = dst.transpose(0, 1) if dst is not None else e(s.vdim)
         if ops.gemv_fits(L.v_b, o_lat):
             ops.gemv_dense(L.v_b, o_lat, out)
@@ -297,18 +302,23 @@ class LatentStack:
                 k0 = max(0, ctx - window + 1) if window else 0
                 kn = ctx + n - k0
                 table.append((b, q0, n, ctx, off, k0, kn, 0))
-                off, longest, max_q = off + kn, max(longest, kn), max(max_q, n)
+                off, longest, max_q = off + pad8(kn), max(longest, kn), max(max_q, n)
             got = bp.keys[window] = (torch.tensor(table, dtype=torch.int32, device=self.device), off, longest, max_q)
         return got
 
     def _attend_chunks(self, L, q: torch.Tensor, o: torch.Tensor, fb, bp: BatchPlan, kv_layer: torch.Tensor) -> None:
         from ..ops import latent as ops
         m, s = L.mixer, L.sizes
-        seqs, n_keys, longest, max_q = self._chunk_keys(bp, m.window)
+        seqs, n_keys, longest, max_q = self._chunk_keys(bp, m.window)      # n_keys: with the rows up to the next multiple of 8
         lat = torch.empty(n_keys, s.width, dtype=self.dtype, device=self.device)
-        ops.latent_gather(kv_layer, seqs, longest, fb.block_table, lat)
-        kvx = torch.mm(lat[:, :s.latent], L.kv_b.w.t())
-        ops.latent_chunk(q, bp.angles[L.rot_index], kvx, lat, s.latent, seqs, max_q, o, s.dim, s.rot, s.vdim, m.window, m.scale, L.sink)
+        ops.latent_gather(kv_layer, seqs, pad8(longest), fb.block_table, lat)
+        c = lat[:, :s.latent]
+        k = torch.mm(c, L.k_b.view(-1, s.latent).t())
+        v_b = L.v_b.view(-1, s.latent)
+        tc = L.chunk_tc and self.chunk_tc
+        v = torch.mm(v_b, c.t()) if tc else torch.mm(c, v_b.t())
+        ops.latent_chunk(q, bp.angles[L.rot_index], k, v, lat, s.latent, seqs, max_q, o, s.dim, s.rot, s.vdim, m.window, m.scale, L.sink,
+                         self.status if tc else None)
 
     def final_logits(self, rows: torch.Tensor, norm: torch.Tensor, head: DenseLinear, out: torch.Tensor) -> torch.Tensor:
         from ..ops import latent as ops

@@ -18,7 +18,7 @@ BUILD_DIR = Path(__file__).resolve().parent / "_build"
 LATENT = "llaminar_b200_latent"       # kernels of latent-attention models, built and loaded on their own
 SOURCES = {
     NAME: ["binding.cpp", "gemv.cu", "gemv_stream.cu", "gemm_tc.cu", "gemm_tc_small.cu", "attention.cu", "attention_tc.cu", "ops.cu", "gdn.cu", "moe_ep.cu", "no_alloc.cu"],
-    LATENT: ["latent_binding.cpp", "latent_attention.cu", "dense_ops.cu"],
+    LATENT: ["latent_binding.cpp", "latent_attention.cu", "latent_tc.cu", "dense_ops.cu"],
 }
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xptxas", "-v"]

@@ -63,11 +63,16 @@ struct LatentRowsParams {
     float scale;
     const float* sink;                         // optional [n_heads]
     void* out; size_t out_row, out_head;       // [row z][head][rot_off]
-    float *part_o, *part_ml;                   // [rows * head groups * splits][16][rot_off], [...][16][2]
+    float *part_o, *part_ml;                   // [rows * head groups * splits][group][rot_off], [...][group][2]
 };
-cudaError_t launch_latent_rows(const LatentRowsParams& p, int rows, int n_splits, bool f32, cudaStream_t st);
-// whether the tensor-core kernel takes these sizes (otherwise launch_latent_rows runs the plain kernel)
+cudaError_t launch_latent_rows(const LatentRowsParams& p, int rows, int n_splits, bool f32, bool plain, cudaStream_t st);
+// whether the mma.sync kernel takes these sizes (otherwise, or with `plain`, launch_latent_rows runs the plain kernel)
 bool latent_rows_has_kernel(int width, int rot_off);
+// tcgen05 form: heads per CTA (the group of the split scratch), 0 where the sizes do not fit
+int latent_rows_tc_heads(int width, int rot_off, int rot_dim, int n_heads);
+cudaError_t launch_latent_rows_tc(const LatentRowsParams& p, int rows, int n_splits, int* status, cudaStream_t st);
+// merges the splits of either form
+cudaError_t launch_latent_merge(const LatentRowsParams& p, int rows, int n_splits, int group, cudaStream_t st);
 
 // Cache rows of the sequences' visible keys -> contiguous rows: buffer row k_off[s] + i holds position k_pos0[s] + i.
 struct LatentSeq { int seq, q_start, q_len, q_pos0, k_off, k_pos0, k_len, pad; };
@@ -78,7 +83,8 @@ cudaError_t launch_latent_gather(const void* kv, const LatentSeq* seqs, int n, i
 struct LatentChunkParams {
     const __nv_bfloat16* q; size_t q_row, q_head;      // [token][head][dim | rot]
     const float2* angles; int half;
-    const __nv_bfloat16* kvx; size_t kvx_row, kvx_head; // [key][head][dim | vdim]
+    const __nv_bfloat16* k;                            // [key][head][dim]
+    const __nv_bfloat16* v;                            // [key][head][vdim]; tcgen05 form: [head][vdim][key]
     const __nv_bfloat16* lat; size_t lat_row; int rot_off;
     const LatentSeq* seqs;
     __nv_bfloat16* out; size_t out_row;                // [token][head * vdim]
@@ -88,6 +94,9 @@ struct LatentChunkParams {
 };
 cudaError_t launch_latent_chunk(const LatentChunkParams& p, int n_seqs, int max_q_len, cudaStream_t st);
 bool latent_chunk_has_kernel(int dk, int dv);
+// tcgen05 form; n_keys (a multiple of 8, as every k_off) rows of k and lat, columns of v.  `status` receives STATUS_TIMEOUT if a wait gave up.
+cudaError_t launch_latent_chunk_tc(const LatentChunkParams& p, int n_keys, int n_seqs, int max_q_len, int* status, cudaStream_t st);
+bool latent_chunk_tc_fits(int dim, int rot, int vdim);
 
 // out[z][m, :] = x[z][m, :] W[z]^T for up to 4 rows, bf16 weights.  gelu: W holds 2n rows and out = gelu_tanh(first n) * second n.
 struct GemvDenseParams {
@@ -100,6 +109,7 @@ struct GemvDenseParams {
 cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st);
 
 int bounds_status_latent(bool reset);
+int bounds_status_latent_tc(bool reset);
 int bounds_status_dense(bool reset);
 
 }  // namespace llm

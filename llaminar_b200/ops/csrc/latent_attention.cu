@@ -64,6 +64,14 @@ template <class T> LLM_DEVICE float rotated(const T* x, int i, const float2* ang
     return to_f(x[i]);
 }
 
+// values i0 .. i0 + 7 of it, zero from `n` on
+LLM_DEVICE uint4 rotated8(const __nv_bfloat16* x, int i0, int n, const float2* ang, int half) {
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = i0 + j < n ? rotated(x, i0 + j, ang, half) : 0.f;
+    return make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+}
+
 LLM_DEVICE int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
 
 // ---- cache rows --------------------------------------------------------------------------------------------------------
@@ -96,13 +104,71 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
     }
 }
 
+// The bf16 form for sizes that are multiples of 8: a thread keeps up to PREP_UNITS 16-byte units of the row in registers.
+constexpr int PREP_UNITS = 4, PREP_THREADS = 256;
+__global__ void __launch_bounds__(PREP_THREADS) latent_prep_vec_kernel(const LatentPrepParams p) {
+    __shared__ float red[2][PREP_THREADS / 32];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x, tid = threadIdx.x;
+    const __nv_bfloat16* d = static_cast<const __nv_bfloat16*>(p.down) + (size_t)t * p.down_stride;
+    const int nq = p.q_rank / 8, n = nq + p.kv_rank / 8;
+    uint4 w[PREP_UNITS];
+    float sq = 0.f, sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < PREP_UNITS; ++i) {
+        const int u = tid + i * PREP_THREADS;
+        w[i] = u < n ? *reinterpret_cast<const uint4*>(d + u * 8) : make_uint4(0, 0, 0, 0);
+    }
+    const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
+    const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
+    __nv_bfloat16* row = static_cast<__nv_bfloat16*>(p.kv) + ((size_t)page * PAGE + pos % PAGE) * p.width;
+    // rotated part and padding by the last threads, while the sums are on their way
+    const int ur = (p.width - p.rot_off) / 8, r = PREP_THREADS - 1 - tid;
+    for (int u = r; u < ur; u += PREP_THREADS)
+        *reinterpret_cast<uint4*>(row + p.rot_off + u * 8) = rotated8(d + p.q_rank + p.kv_rank, u * 8, p.rot_dim, p.angles + (size_t)t * p.half, p.half);
+#pragma unroll
+    for (int i = 0; i < PREP_UNITS; ++i) {
+        const uint32_t x[4] = {w[i].x, w[i].y, w[i].z, w[i].w};
+        float ss = 0.f;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { const float a = bf16_lo(x[j]), b = bf16_hi(x[j]); ss += a * a + b * b; }
+        if (tid + i * PREP_THREADS < nq) sq += ss; else sk += ss;
+    }
+    sq = warp_sum(sq); sk = warp_sum(sk);
+    if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int i = 0; i < PREP_THREADS / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
+    const float iq = 1.f / sqrtf(sq / (float)p.q_rank + p.eps), ik = 1.f / sqrtf(sk / (float)p.kv_rank + p.eps);
+#pragma unroll
+    for (int i = 0; i < PREP_UNITS; ++i) {
+        const int u = tid + i * PREP_THREADS;
+        if (u >= n) break;
+        const bool q = u < nq;
+        const float* g = q ? p.q_norm + u * 8 : p.kv_norm + (u - nq) * 8;
+        const float inv = q ? iq : ik;
+        const float4 g0 = *reinterpret_cast<const float4*>(g), g1 = *reinterpret_cast<const float4*>(g + 4);
+        const uint4 o = make_uint4(pack_bf16(bf16_lo(w[i].x) * inv * g0.x, bf16_hi(w[i].x) * inv * g0.y), pack_bf16(bf16_lo(w[i].y) * inv * g0.z, bf16_hi(w[i].y) * inv * g0.w),
+                                   pack_bf16(bf16_lo(w[i].z) * inv * g1.x, bf16_hi(w[i].z) * inv * g1.y), pack_bf16(bf16_lo(w[i].w) * inv * g1.z, bf16_hi(w[i].w) * inv * g1.w));
+        __nv_bfloat16* dst = q ? static_cast<__nv_bfloat16*>(p.cq) + (size_t)t * p.cq_stride + u * 8 : row + (u - nq) * 8;
+        *reinterpret_cast<uint4*>(dst) = o;
+    }
+}
+
 // one warp per key row
 template <class T>
 __global__ void __launch_bounds__(256) latent_gather_kernel(const T* kv, const LatentSeq* seqs, const int* block_table, int max_pages, int n_pages,
                                                             int width, T* out) {
     const LatentSeq s = seqs[blockIdx.y];
     const int i = blockIdx.x * 8 + (threadIdx.x >> 5);
-    if (i >= s.k_len) return;
+    if (i >= (s.k_len + 7) / 8 * 8) return;
+    if (i >= s.k_len) {                     // the next sequence's rows start at a multiple of 8: zeros in between
+        uint4* dst = reinterpret_cast<uint4*>(out + (size_t)(s.k_off + i) * width);
+        for (int u = threadIdx.x & 31; u < width * (int)sizeof(T) / 16; u += 32) dst[u] = make_uint4(0, 0, 0, 0);
+        return;
+    }
     const int pos = s.k_pos0 + i;
     const int page = LLM_CHECK_INDEX(block_table[(size_t)s.seq * max_pages + pos / PAGE], n_pages);
     const uint4* src = reinterpret_cast<const uint4*>(kv + ((size_t)page * PAGE + pos % PAGE) * width);
@@ -215,18 +281,15 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const LatentRowsParams
     for (int s = 0; s < STAGES - 1; ++s) issue(kt0 + s, s);
 
     // queries of the 16 heads: latent part, rotated part, zero padding (and zero rows past the last head)
-    for (int i = warp; i < 16; i += 4) {
-        const int h = hg * 16 + i;
-        const __nv_bfloat16* ql = static_cast<const __nv_bfloat16*>(p.q_lat) + (size_t)z * p.ql_row + (size_t)h * p.ql_head;
-        const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off;
-        for (int c = lane; c < LD; c += 32) {
-            __nv_bfloat16 v = __float2bfloat16(0.f);
-            if (h < p.n_heads) {
-                if (c < R) v = ql[c];
-                else if (c < R + p.rot_dim) v = __float2bfloat16(rotated(qr, c - R, p.angles + (size_t)t * p.half, p.half));
-            }
-            sq[i * LD + c] = v;
+    for (int i = threadIdx.x; i < 16 * (LD / 8); i += 128) {
+        const int r = i / (LD / 8), u = i % (LD / 8), h = hg * 16 + r;
+        uint4 v = make_uint4(0, 0, 0, 0);
+        if (h < p.n_heads) {
+            if (u * 8 < R) v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q_lat) + (size_t)z * p.ql_row + (size_t)h * p.ql_head + u * 8);
+            else v = rotated8(static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off, u * 8 - R, p.rot_dim,
+                              p.angles + (size_t)t * p.half, p.half);
         }
+        *reinterpret_cast<uint4*>(sq + r * LD + u * 8) = v;
     }
 
     float o[NT][4];
@@ -346,25 +409,36 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const LatentRowsParams
     }
 }
 
-__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentRowsParams p, int n_splits, int groups) {
+constexpr int MAX_SPLITS = 64;
+__global__ void __launch_bounds__(128) latent_merge_kernel(const LatentRowsParams p, int n_splits, int groups, int group) {
+    __shared__ float s_w[MAX_SPLITS];
     pdl_trigger();
     pdl_wait();
-    const int h = blockIdx.x, z = blockIdx.y, R = p.rot_off;
-    const size_t part = ((size_t)z * groups + h / 16) * n_splits * 16 + h % 16;
-    float m = p.sink ? p.sink[h] * LOG2E : -INFINITY;
-    for (int s = 0; s < n_splits; ++s) m = fmaxf(m, p.part_ml[(part + s * 16) * 2]);
-    float l = p.sink ? exp2f(p.sink[h] * LOG2E - m) : 0.f;
-    for (int s = 0; s < n_splits; ++s) l += exp2f(p.part_ml[(part + s * 16) * 2] - m) * p.part_ml[(part + s * 16) * 2 + 1];
-    const float inv = 1.f / l;
+    const int h = blockIdx.x, z = blockIdx.y, R = p.rot_off, lane = threadIdx.x & 31;
+    const size_t part = ((size_t)z * groups + h / group) * n_splits * group + h % group;
+    if (threadIdx.x < 32) {
+        const float2 none = make_float2(-INFINITY, 0.f);
+        const float2 a = lane < n_splits ? *reinterpret_cast<const float2*>(p.part_ml + (part + (size_t)lane * group) * 2) : none;
+        const float2 b = lane + 32 < n_splits ? *reinterpret_cast<const float2*>(p.part_ml + (part + (size_t)(lane + 32) * group) * 2) : none;
+        const float sink = p.sink ? p.sink[h] * LOG2E : -INFINITY;
+        const float m = fmaxf(warp_max(fmaxf(a.x, b.x)), sink);
+        const float wa = exp2f(a.x - m), wb = exp2f(b.x - m);               // 0 for a split without keys
+        const float inv = 1.f / (warp_sum(wa * a.y + wb * b.y) + exp2f(sink - m));
+        s_w[lane] = wa * inv;
+        s_w[lane + 32] = wb * inv;
+    }
+    __syncthreads();
     for (int c = threadIdx.x * 4; c < R; c += 512) {
         float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
         for (int s = 0; s < n_splits; ++s) {
-            const float w = exp2f(p.part_ml[(part + s * 16) * 2] - m);           // 0 for a split without keys
-            const float4 v = *reinterpret_cast<const float4*>(p.part_o + (part + s * 16) * R + c);
+            const float w = s_w[s];
+            if (w == 0.f) continue;                                         // a split without keys wrote no sums
+            const float4 v = *reinterpret_cast<const float4*>(p.part_o + (part + (size_t)s * group) * R + c);
             a.x = fmaf(w, v.x, a.x); a.y = fmaf(w, v.y, a.y); a.z = fmaf(w, v.z, a.z); a.w = fmaf(w, v.w, a.w);
         }
         *reinterpret_cast<uint2*>(static_cast<__nv_bfloat16*>(p.out) + (size_t)z * p.out_row + (size_t)h * p.out_head + c) =
-            make_uint2(pack_bf16(a.x * inv, a.y * inv), pack_bf16(a.z * inv, a.w * inv));
+            make_uint2(pack_bf16(a.x, a.y), pack_bf16(a.z, a.w));
     }
 }
 
@@ -403,10 +477,10 @@ __global__ void __launch_bounds__(256) latent_chunk_kernel(const LatentChunkPara
             // a quarter of a warp per key row: 8 lanes copy 128 contiguous bytes at a time
             for (int r = threadIdx.x >> 3; r < BK; r += 32) {
                 const size_t row = (size_t)(sq.k_off + min(tile * BK + r, sq.k_len - 1));
-                const __nv_bfloat16* src = p.kvx + row * p.kvx_row + (size_t)head * p.kvx_head;
-                for (int u = threadIdx.x & 7; u < uk; u += 8) cp_async16(kd + (r * LK + u * 8) * 2, src + u * 8);
+                const __nv_bfloat16 *ks = p.k + (row * p.n_heads + head) * p.dim, *vs = p.v + (row * p.n_heads + head) * p.vdim;
+                for (int u = threadIdx.x & 7; u < uk; u += 8) cp_async16(kd + (r * LK + u * 8) * 2, ks + u * 8);
                 for (int u = threadIdx.x & 7; u < ur; u += 8) cp_async16(kd + (r * LK + p.dim + u * 8) * 2, p.lat + row * p.lat_row + p.rot_off + u * 8);
-                for (int u = threadIdx.x & 7; u < uv; u += 8) cp_async16(vd + (r * LV + u * 8) * 2, src + p.dim + u * 8);
+                for (int u = threadIdx.x & 7; u < uv; u += 8) cp_async16(vd + (r * LV + u * 8) * 2, vs + u * 8);
             }
         }
         cp_async_commit();
@@ -419,8 +493,8 @@ __global__ void __launch_bounds__(256) latent_chunk_kernel(const LatentChunkPara
             const __nv_bfloat16* src = p.q + t * p.q_row + (size_t)head * p.q_head;
             for (int u = lane; u < uk; u += 32)
                 *reinterpret_cast<uint4*>(s_q + r * LQ + u * 8) = live ? *reinterpret_cast<const uint4*>(src + u * 8) : make_uint4(0, 0, 0, 0);
-            for (int c = p.dim + lane; c < LQ; c += 32)
-                s_q[r * LQ + c] = __float2bfloat16(live && c < p.dim + p.rot ? rotated(src + p.dim, c - p.dim, p.angles + t * p.half, p.half) : 0.f);
+            for (int u = lane; u < LQ / 8 - uk; u += 32)
+                *reinterpret_cast<uint4*>(s_q + r * LQ + p.dim + u * 8) = live ? rotated8(src + p.dim, u * 8, p.rot, p.angles + t * p.half, p.half) : make_uint4(0, 0, 0, 0);
         }
     }
     float o[DV / 8][4];
@@ -531,6 +605,10 @@ template <class K> cudaError_t raise_smem(K kernel, size_t bytes) {
 
 cudaError_t launch_latent_prep(const LatentPrepParams& p, int rows, bool f32, cudaStream_t st) {
     if (f32) return launch_pdl(latent_prep_kernel<float>, dim3(rows), dim3(128), 0, st, p);
+    const bool vec = p.q_rank % 8 == 0 && p.kv_rank % 8 == 0 && p.rot_dim % 8 == 0 && p.down_stride % 8 == 0 && (int)p.cq_stride == p.q_rank &&
+                     p.rot_off == p.kv_rank && (p.q_rank + p.kv_rank) / 8 <= PREP_UNITS * PREP_THREADS &&
+                     !((reinterpret_cast<uintptr_t>(p.down) | reinterpret_cast<uintptr_t>(p.q_norm) | reinterpret_cast<uintptr_t>(p.kv_norm)) & 15);
+    if (vec) return launch_pdl(latent_prep_vec_kernel, dim3(rows), dim3(PREP_THREADS), 0, st, p);
     return launch_pdl(latent_prep_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, st, p);
 }
 
@@ -549,10 +627,10 @@ bool latent_rows_has_kernel(int width, int rot_off) {
     return width % 16 == 0 && width <= 1024 && rot_off % 8 == 0 && rot_off <= 512 && rows_smem(width, 2) <= 220 * 1024;
 }
 
-cudaError_t launch_latent_rows(const LatentRowsParams& p, int rows, int n_splits, bool f32, cudaStream_t st) {
+cudaError_t launch_latent_rows(const LatentRowsParams& p, int rows, int n_splits, bool f32, bool plain, cudaStream_t st) {
     if (rows == 0) return cudaSuccess;
     if (rows > 65535) return cudaErrorInvalidValue;
-    if (f32 || !latent_rows_has_kernel(p.width, p.rot_off)) {
+    if (f32 || plain || !latent_rows_has_kernel(p.width, p.rot_off)) {
         const size_t smem = (size_t)(p.width + p.rot_off) * 4;
         if (smem > 220 * 1024) return cudaErrorInvalidValue;
         auto go = [&](auto kernel) {
@@ -573,8 +651,12 @@ cudaError_t launch_latent_rows(const LatentRowsParams& p, int rows, int n_splits
     else if (p.rot_off <= 128) e = go(latent_rows_kernel<4, 3>, 3);
     else if (p.rot_off <= 256) e = go(latent_rows_kernel<8, 3>, 3);
     else e = go(latent_rows_kernel<16, 2>, 2);
-    if (e != cudaSuccess || n_splits == 1) return e;
-    return launch_pdl(latent_merge_kernel, dim3(p.n_heads, rows), dim3(128), 0, st, p, n_splits, groups);
+    return e != cudaSuccess || n_splits == 1 ? e : launch_latent_merge(p, rows, n_splits, 16, st);
+}
+
+cudaError_t launch_latent_merge(const LatentRowsParams& p, int rows, int n_splits, int group, cudaStream_t st) {
+    if (n_splits > MAX_SPLITS || rows > 65535) return cudaErrorInvalidValue;
+    return launch_pdl(latent_merge_kernel, dim3(p.n_heads, rows), dim3(128), 0, st, p, n_splits, (p.n_heads + group - 1) / group, group);
 }
 
 bool latent_chunk_has_kernel(int dk, int dv) { return dk % 8 == 0 && dv % 8 == 0 && dk <= 256 && dv <= 256; }

@@ -125,7 +125,8 @@ void latent_prep(const Tensor& down, const Tensor& q_norm, const Tensor& kv_norm
 // q_lat [heads, rows, rot_off]; q [tokens, heads, head size] (contiguous); out [heads, rows, rot_off]
 void latent_rows(const Tensor& q_lat, const Tensor& q, int64_t q_rot_off, const Tensor& angles, const OptTensor& rows, const Tensor& positions,
                  const Tensor& seq_ids, const Tensor& block_table, const Tensor& kv, int64_t rot_dim, int64_t window, double scale,
-                 const OptTensor& sink, const Tensor& out, const OptTensor& part_o, const OptTensor& part_ml, int64_t n_splits) {
+                 const OptTensor& sink, const Tensor& out, const OptTensor& part_o, const OptTensor& part_ml, int64_t n_splits, int64_t group,
+                 const OptTensor& status) {
     const bool f32 = is_f32(kv, "kv");
     want_like(q_lat, f32, "q_lat"); want_like(q, f32, "q"); want_like(out, f32, "out");
     const int64_t H = q_lat.size(0), n = q_lat.size(1), R = q_lat.size(2);
@@ -147,17 +148,26 @@ void latent_rows(const Tensor& q_lat, const Tensor& q, int64_t q_rot_off, const 
     p.n_heads = H; p.window = window; p.scale = scale;
     p.sink = sink ? floats(*sink, H, "sink") : nullptr;
     p.out = out.data_ptr(); p.out_row = out.stride(1); p.out_head = out.stride(0);
-    if (!f32 && llm::latent_rows_has_kernel(p.width, p.rot_off)) {
-        TORCH_CHECK(p.out_row % 4 == 0 && p.out_head % 4 == 0, "out strides must be multiples of 4");
-        TORCH_CHECK(n_splits >= 1 && n_splits <= 65535, "n_splits");
+    // group: heads per CTA of the tcgen05 form, 16 of the mma.sync form, 0 the plain kernel
+    const bool tc = group == llm::latent_rows_tc_heads(p.width, p.rot_off, p.rot_dim, H) && group > 0 && status;
+    TORCH_CHECK(group == 0 || (!f32 && (tc || (group == 16 && llm::latent_rows_has_kernel(p.width, p.rot_off)))), "no kernel for this group of heads");
+    if (group) {
+        TORCH_CHECK(p.out_row % 4 == 0 && p.out_head % 4 == 0 && p.ql_row % 8 == 0 && p.ql_head % 8 == 0, "latent strides");
+        TORCH_CHECK(n_splits >= 1 && n_splits <= 64, "n_splits");
         if (n_splits > 1) {
-            const int64_t parts = n * ((H + 15) / 16) * n_splits * 16;
+            const int64_t parts = n * ((H + group - 1) / group) * n_splits * group;
             want(part_o.value(), torch::kFloat32, "part_o"); want(part_ml.value(), torch::kFloat32, "part_ml");
             TORCH_CHECK(part_o->numel() >= parts * R && part_ml->numel() >= parts * 2, "split scratch too small");
             p.part_o = part_o->data_ptr<float>(); p.part_ml = part_ml->data_ptr<float>();
         }
     }
-    check(llm::launch_latent_rows(p, n, n_splits, f32, stream()), "latent_rows");
+    if (tc) {
+        want(*status, torch::kInt32, "status");
+        check(llm::launch_latent_rows_tc(p, n, n_splits, status->data_ptr<int>(), stream()), "latent_rows_tc");
+        if (n_splits > 1) check(llm::launch_latent_merge(p, n, n_splits, group, stream()), "latent_merge");
+        return;
+    }
+    check(llm::launch_latent_rows(p, n, group ? n_splits : 1, f32, group == 0, stream()), "latent_rows");
 }
 
 // seqs: int32 [n, 8], see LatentSeq; the limits are the host's view of the same numbers
@@ -173,12 +183,15 @@ void latent_gather(const Tensor& kv, const Tensor& seqs, int64_t max_k_len, cons
           "latent_gather");
 }
 
-void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& kvx, const Tensor& lat, int64_t rot_off, const Tensor& seqs, int64_t max_q_len,
-                  const Tensor& out, int64_t dim, int64_t rot, int64_t vdim, int64_t window, double scale, const OptTensor& sink) {
-    for (auto& t : {q, kvx, lat, out}) want(t, torch::kBFloat16, "latent_chunk operand");
-    const int64_t T = q.size(0), H = q.size(1);
+// k [keys, heads * dim]; v [keys, heads * vdim], or with status (the tcgen05 form) [heads * vdim, keys]
+void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& k, const Tensor& v, const Tensor& lat, int64_t rot_off, const Tensor& seqs,
+                  int64_t max_q_len, const Tensor& out, int64_t dim, int64_t rot, int64_t vdim, int64_t window, double scale, const OptTensor& sink,
+                  const OptTensor& status) {
+    for (auto& t : {q, k, v, lat, out}) want(t, torch::kBFloat16, "latent_chunk operand");
+    const int64_t T = q.size(0), H = q.size(1), n = lat.size(0);
     TORCH_CHECK(q.dim() == 3 && q.size(2) == dim + rot, "q must be [tokens, heads, dim + rot]");
-    TORCH_CHECK(kvx.size(1) == H * (dim + vdim) && kvx.size(0) <= lat.size(0) && rot_off + rot <= lat.size(1), "key buffers");
+    TORCH_CHECK(k.size(0) == n && k.size(1) == H * dim && rot_off + rot <= lat.size(1), "key buffers");
+    TORCH_CHECK(status ? v.size(0) == H * vdim && v.size(1) == n : v.size(0) == n && v.size(1) == H * vdim, "value buffer");
     TORCH_CHECK(out.size(0) == T && out.size(1) == H * vdim, "out must be [tokens, heads * vdim]");
     TORCH_CHECK(seqs.dim() == 2 && seqs.size(1) == 8, "seqs must be [n, 8]");
     TORCH_CHECK(dim % 8 == 0 && rot % 8 == 0 && vdim % 8 == 0 && rot_off % 8 == 0 && lat.size(1) % 8 == 0, "sizes must be multiples of 8");
@@ -188,13 +201,18 @@ void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& kvx, cons
     p.q = b(q); p.q_row = q.stride(0); p.q_head = q.stride(1);
     p.angles = angle_ptr(angles, T); p.half = angles.size(1);
     TORCH_CHECK(2 * p.half <= rot, "more angles than the rotated part has pairs");
-    p.kvx = b(kvx); p.kvx_row = kvx.size(1); p.kvx_head = dim + vdim;
+    p.k = b(k); p.v = b(v);
     p.lat = b(lat); p.lat_row = lat.size(1); p.rot_off = rot_off;
     p.seqs = reinterpret_cast<const llm::LatentSeq*>(ints(seqs, "seqs"));
     p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr()); p.out_row = out.size(1);
     p.dim = dim; p.rot = rot; p.vdim = vdim; p.n_heads = H; p.window = window; p.scale = scale;
     p.sink = sink ? floats(*sink, H, "sink") : nullptr;
-    check(llm::launch_latent_chunk(p, seqs.size(0), max_q_len, stream()), "latent_chunk");
+    if (status) {
+        want(*status, torch::kInt32, "status");
+        check(llm::launch_latent_chunk_tc(p, n, seqs.size(0), max_q_len, status->data_ptr<int>(), stream()), "latent_chunk_tc");
+    } else {
+        check(llm::launch_latent_chunk(p, seqs.size(0), max_q_len, stream()), "latent_chunk");
+    }
 }
 
 // w [z, n, k] (gelu: [z, 2n, k]), x [z, m, k], out [z, m, n]; the last dimension of each is dense
@@ -221,10 +239,12 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("latent_prep", &latent_prep);
     m.def("latent_rows", &latent_rows);
     m.def("latent_rows_has_kernel", &llm::latent_rows_has_kernel);
+    m.def("latent_rows_tc_heads", &llm::latent_rows_tc_heads);
+    m.def("latent_chunk_tc_fits", &llm::latent_chunk_tc_fits);
     m.def("latent_gather", &latent_gather);
     m.def("latent_chunk", &latent_chunk);
     m.def("latent_chunk_has_kernel", &llm::latent_chunk_has_kernel);
     m.def("gemv_dense", &gemv_dense);
     m.def("set_pdl", [](bool on) { llm::pdl_enabled() = on; });
-    m.def("bounds_status", [](bool reset) { return llm::bounds_status_latent(reset) | llm::bounds_status_dense(reset); });
+    m.def("bounds_status", [](bool reset) { return llm::bounds_status_latent(reset) | llm::bounds_status_latent_tc(reset) | llm::bounds_status_dense(reset); });
 }

@@ -1,0 +1,709 @@
+// Latent attention on the 5th-generation tensor cores: prompt chunks (latent_chunk_tc_kernel) and single rows
+// (latent_rows_tc_kernel).  All operand tiles arrive by TMA in the 128-byte-swizzled form that the MMA reads.
+// Every mbarrier wait is bounded; on a timeout the kernel raises the status word and tears down.
+#include "latent.h"
+#include "launch.h"
+#include "tc_common.cuh"
+
+namespace llm {
+namespace ltc {
+using namespace tc5;
+
+constexpr float LOG2E = 1.4426950408889634f;
+constexpr int ATOM = 128 * 128;                    // 128 rows x 64 bf16
+
+LLM_DEVICE float ex2(float x) {                    // 2^x, approximate; -inf -> 0
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+LLM_DEVICE int first_key(int pos, int window) { return window > 0 ? max(0, pos - window + 1) : 0; }
+// 16-byte unit `unit` (0..7) of row `row` inside one operand atom
+LLM_DEVICE uint32_t atom_addr(uint32_t base, int row, int unit) { return base + row * 128 + (((unit ^ row) & 7) << 4); }
+LLM_DEVICE void st_shared_v4(uint32_t dst, const uint4& v) {
+    asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};" ::"r"(dst), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
+}
+LLM_DEVICE void tmem_st32(uint32_t taddr, const uint32_t (&r)[32]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,"
+                 "%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
+                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+                   "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]),
+                   "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]), "r"(r[21]), "r"(r[22]), "r"(r[23]),
+                   "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31]) : "memory");
+}
+LLM_DEVICE void tmem_wait_st() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
+
+// value i of a rotated part: pairs (i, i + half) turn, the rest passes
+LLM_DEVICE float rotated(const __nv_bfloat16* x, int i, const float2* ang, int half) {
+    const float v = __bfloat162float(x[i]);
+    if (i < half) return v * ang[i].x - __bfloat162float(x[i + half]) * ang[i].y;
+    if (i < 2 * half) return v * ang[i - half].x + __bfloat162float(x[i - half]) * ang[i - half].y;
+    return v;
+}
+LLM_DEVICE uint4 rotated8(const __nv_bfloat16* x, int i0, const float2* ang, int half) {
+    float v[8];
+#pragma unroll
+    for (int j = 0; j < 8; ++j) v[j] = rotated(x, i0 + j, ang, half);
+    return make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+}
+
+LLM_DEVICE void teardown(volatile int* abort_flag, int tid, int* status) {
+    if (abort_flag[0]) {
+        if (tid == 0 && status) atomicExch(status, (int)STATUS_TIMEOUT);
+        for (int i = 0; i < 2000; ++i) __nanosleep(100);      // let copies still in flight land before the memory is reused
+        __syncthreads();
+    }
+}
+
+// ------------------------------------------------------------------------------------------------------------------------
+// prompt chunks: 128 query rows of one head per CTA, keys in tiles of 128
+//   S = Q K^T         M = 128 query rows, N = 128 keys, K = dim + rot; two accumulators
+//   softmax           two threads per query row (= TMEM lane), 64 columns each; P goes back to TMEM as the A operand
+//   O_tile = P V      M = 128, N = vdim, K = 128 keys; B is V^T (vdim rows of keys), which the value product writes directly
+// The softmax threads keep the output row in registers and fold every O_tile in, scaled by the running-max correction.
+// Warps 0-7 softmax, 8 TMA, 9 TMEM allocation and MMA issue.
+// ------------------------------------------------------------------------------------------------------------------------
+constexpr int BQ = 128, BK = 128, CHUNK_THREADS = 320;
+enum Bar { K_FULL = 0, K_EMPTY = 2, V_FULL = 4, V_EMPTY = 6, S_FULL = 8, S_EMPTY = 10, P_FULL = 12, O_FULL = 13, O_EMPTY = 14, Q_FULL = 15, PAIR = 16, N_BARS = 20 };
+constexpr int T_O = 256, T_P = 384;                // TMEM columns: S 0..255, O 256..383, P 384..447
+
+template <int VD>
+__global__ void __launch_bounds__(CHUNK_THREADS, 1) latent_chunk_tc_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_l,
+                                                                           const __grid_constant__ CUtensorMap map_v, const LatentChunkParams p, int* status) {
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t s_bars[N_BARS];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_abort[2];
+    // row maxima (and, at the end, sums) of a thread pair; an entry is overwritten only after the O_FULL wait of the tile, which
+    // needs the partner's P_FULL arrival, which follows the partner's read
+    __shared__ float s_xchg[2][BQ];
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int head = blockIdx.y;
+    const LatentSeq sq = p.seqs[blockIdx.z];
+    const int q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * BQ;      // the last query tiles see the most keys: they go first
+    if (q0 >= sq.q_len) return;                                      // uniform for the CTA, before any barrier or allocation
+    if (sq.k_off % 8) {                                              // a TMA copy of the transposed values would start off a 16-byte boundary
+        if (tid == 0 && status) atomicExch(status, (int)STATUS_BAD_ARG);
+        return;
+    }
+    const int rows = min(BQ, sq.q_len - q0), pos0 = sq.q_pos0 + q0, pos_last = pos0 + rows - 1;
+    const int tile0 = (max(first_key(pos0, p.window), sq.k_pos0) - sq.k_pos0) / BK;
+    const int nt = (pos_last - sq.k_pos0) / BK + 1 - tile0;
+    const int na = (p.dim + 63) / 64, nr = (p.rot + 63) / 64, nk = na + nr;       // operand atoms of a query or key row
+    const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+    const uint32_t sQ = base, sK = sQ + nk * ATOM, sV = sK + 2 * nk * ATOM;       // sV: [2 buffers][2 key halves]
+    const uint32_t bars = smem_u32(s_bars);
+    auto bar = [&](int i) { return bars + i * 8; };
+
+    if (tid == 0) {
+        s_abort[0] = 0; s_abort[1] = 0;
+        const int counts[N_BARS] = {1, 1, 1, 1, 1, 1, 1, 1, 1, 1, 8, 8, 8, 1, 8, 8, 2, 2, 2, 2};
+        for (int i = 0; i < N_BARS; ++i) mbar_init(bar(i), counts[i]);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        fence_proxy_async();
+    }
+    if (warp == 9) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(512) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s_tmem;
+    volatile int* abort_flag = s_abort;
+
+    if (warp < 8) {
+        // queries: unrotated part copied, rotated part turned on the way
+        const int un = p.dim / 8, ur = p.rot / 8;
+        for (int i = tid; i < BQ * un; i += 256) {
+            const int r = i / un, u = i % un;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (r < rows) v = *reinterpret_cast<const uint4*>(p.q + (size_t)(sq.q_start + q0 + r) * p.q_row + (size_t)head * p.q_head + u * 8);
+            st_shared_v4(atom_addr(sQ + (u >> 3) * ATOM, r, u & 7), v);
+        }
+        for (int i = tid; i < BQ * ur; i += 256) {
+            const int r = i / ur, u = i % ur;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (r < rows) {
+                const size_t t = (size_t)sq.q_start + q0 + r;
+                v = rotated8(p.q + t * p.q_row + (size_t)head * p.q_head + p.dim, u * 8, p.angles + t * p.half, p.half);
+            }
+            st_shared_v4(atom_addr(sQ + (na + (u >> 3)) * ATOM, r, u & 7), v);
+        }
+        fence_proxy_async();
+        __syncwarp();
+        mbar_arrive_if(bar(Q_FULL), lane == 0);
+
+        const int row = tid & 127, half = tid >> 7, q4 = warp & 3;
+        const bool valid = row < rows;
+        const int pos = pos0 + min(row, rows - 1);
+        const int lim = pos + 1, low = first_key(pos, p.window);           // this row sees low <= key < lim
+        const uint32_t t_lane = tmem + ((uint32_t)(q4 * 32) << 16);
+        const float sl2 = p.scale * LOG2E;
+        constexpr int HD = VD / 2;
+        float o[HD];
+#pragma unroll
+        for (int i = 0; i < HD; ++i) o[i] = 0.f;
+        float m = -INFINITY, l = 0.f, m_new = -INFINITY, mb = 0.f, alpha = 0.f, alpha_prev = 0.f;
+        bool ok = true;
+        int n_pair = 0;
+        auto pair_meet = [&]() {                   // bounded rendezvous of the two warps that share these 32 rows
+            __syncwarp();
+            mbar_arrive_if(bar(PAIR + q4), lane == 0);
+            const bool r = mbar_wait_warp(bar(PAIR + q4), n_pair & 1, abort_flag);
+            ++n_pair;
+            return r;
+        };
+        uint32_t ra[32], rb[32];
+        // first pass over tile j: row maximum over this thread's 64 columns, exchanged with the partner thread
+        auto pass1 = [&](int j) {
+            if (!mbar_wait_warp(bar(S_FULL + (j & 1)), (j >> 1) & 1, abort_flag)) return false;
+            tc_fence_after();
+            const int key0 = sq.k_pos0 + (tile0 + j) * BK + half * 64;
+            const uint32_t t_s = t_lane + (j & 1) * 128 + half * 64;
+            tmem_ld32_issue(t_s, ra);
+            tmem_ld32_issue(t_s + 32, rb);
+            tmem_wait_ld(ra);
+            tmem_wait_ld(rb);
+            float mx = -INFINITY;
+            if (key0 + 64 > lim || key0 < low) {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) {
+                    const int k0 = key0 + i, k1 = key0 + 32 + i;
+                    mx = fmaxf(mx, k0 >= lim || k0 < low ? -INFINITY : __uint_as_float(ra[i]));
+                    mx = fmaxf(mx, k1 >= lim || k1 < low ? -INFINITY : __uint_as_float(rb[i]));
+                }
+            } else {
+#pragma unroll
+                for (int i = 0; i < 32; ++i) mx = fmaxf(mx, fmaxf(__uint_as_float(ra[i]), __uint_as_float(rb[i])));
+            }
+            s_xchg[half][row] = mx;
+            if (!pair_meet()) return false;
+            mx = fmaxf(mx, s_xchg[half ^ 1][row]);
+            m_new = fmaxf(m, mx * sl2);
+            mb = m_new == -INFINITY ? 0.f : m_new;
+            alpha = ex2(m - mb);
+            return true;
+        };
+        // the tile's P V product is complete: fold it into the register copy of the output row
+        auto fold = [&](int j) {
+            if (!mbar_wait_warp(bar(O_FULL), j & 1, abort_flag)) return false;
+            tc_fence_after();
+            const uint32_t t_o = t_lane + T_O + half * HD;
+            tmem_ld32_issue(t_o, ra);
+            if constexpr (HD == 64) tmem_ld32_issue(t_o + 32, rb);
+            tmem_wait_ld(ra);
+            if constexpr (HD == 64) tmem_wait_ld(rb);
+#pragma unroll
+            for (int i = 0; i < 32; ++i) {
+                o[i] = o[i] * alpha_prev + __uint_as_float(ra[i]);
+                if constexpr (HD == 64) o[32 + i] = o[32 + i] * alpha_prev + __uint_as_float(rb[i]);
+            }
+            tc_fence_before();
+            __syncwarp();
+            mbar_arrive_if(bar(O_EMPTY), lane == 0);
+            return true;
+        };
+        for (int j = 0; j <= nt && ok; ++j) {
+            if (j < nt) ok = pass1(j);
+            if (ok && j > 0) ok = fold(j - 1);               // also frees P
+            if (!ok || j == nt) break;
+            const int key0 = sq.k_pos0 + (tile0 + j) * BK + half * 64;
+            const bool need_mask = key0 + 64 > lim || key0 < low;
+            const uint32_t t_s = t_lane + (j & 1) * 128 + half * 64;
+            tmem_ld32_issue(t_s, ra);
+            tmem_ld32_issue(t_s + 32, rb);
+            tmem_wait_ld(ra);
+            tmem_wait_ld(rb);
+            float sum = 0.f;
+            uint32_t w[32];
+            auto probs_of = [&](int c, const uint32_t (&r)[32]) {
+                if (need_mask) {
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2) {
+                        const int key = key0 + c * 32 + i;
+                        const float p0 = key >= lim || key < low ? 0.f : ex2(__uint_as_float(r[i]) * sl2 - mb);
+                        const float p1 = key + 1 >= lim || key + 1 < low ? 0.f : ex2(__uint_as_float(r[i + 1]) * sl2 - mb);
+                        sum += p0 + p1;
+                        w[c * 16 + (i >> 1)] = pack_bf16(p0, p1);
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; i += 2) {
+                        const float p0 = ex2(__uint_as_float(r[i]) * sl2 - mb), p1 = ex2(__uint_as_float(r[i + 1]) * sl2 - mb);
+                        sum += p0 + p1;
+                        w[c * 16 + (i >> 1)] = pack_bf16(p0, p1);
+                    }
+                }
+            };
+            probs_of(0, ra);
+            probs_of(1, rb);
+            tmem_st32(t_lane + T_P + half * 32, w);
+            tmem_wait_st();
+            tc_fence_before();
+            __syncwarp();
+            mbar_arrive_if(bar(S_EMPTY + (j & 1)), lane == 0); mbar_arrive_if(bar(P_FULL), lane == 0);
+            l = l * alpha + sum;
+            m = m_new;
+            alpha_prev = alpha;
+        }
+        if (ok) {                                  // the row's normaliser: both column halves, and the sink
+            s_xchg[half][row] = l;
+            ok = pair_meet();
+        }
+        if (ok && valid) {
+            float lt = l + s_xchg[half ^ 1][row];
+            if (p.sink) lt += exp2f(p.sink[head] * LOG2E - m);
+            const float inv = 1.f / lt;
+            __nv_bfloat16* dst = p.out + (size_t)(sq.q_start + q0 + row) * p.out_row + (size_t)head * p.vdim + half * HD;
+#pragma unroll
+            for (int u = 0; u < HD / 8; ++u) {
+                if (half * HD + u * 8 >= p.vdim) break;
+                *reinterpret_cast<uint4*>(dst + 8 * u) = make_uint4(pack_bf16(o[8 * u] * inv, o[8 * u + 1] * inv), pack_bf16(o[8 * u + 2] * inv, o[8 * u + 3] * inv),
+                                                                    pack_bf16(o[8 * u + 4] * inv, o[8 * u + 5] * inv), pack_bf16(o[8 * u + 6] * inv, o[8 * u + 7] * inv));
+            }
+        }
+    } else if (warp == 8) {
+        if (elect_one()) {
+            bool ok = true;
+            for (int j = 0; j < nt && ok; ++j) {
+                const int b = j & 1, key = sq.k_off + (tile0 + j) * BK;             // row of the key buffer
+                ok = mbar_wait(bar(K_EMPTY + b), ((j >> 1) & 1) ^ 1, abort_flag);
+                if (!ok) break;
+                mbar_arrive_expect_tx(bar(K_FULL + b), nk * ATOM);
+                for (int a = 0; a < na; ++a) tma_load_2d(sK + (b * nk + a) * ATOM, &map_k, head * p.dim + a * 64, key, bar(K_FULL + b));
+                for (int a = 0; a < nr; ++a) tma_load_2d(sK + (b * nk + na + a) * ATOM, &map_l, p.rot_off + a * 64, key, bar(K_FULL + b));
+                ok = mbar_wait(bar(V_EMPTY + b), ((j >> 1) & 1) ^ 1, abort_flag);
+                if (!ok) break;
+                mbar_arrive_expect_tx(bar(V_FULL + b), 2 * p.vdim * 128);
+                for (int a = 0; a < 2; ++a) tma_load_2d(sV + (b * 2 + a) * ATOM, &map_v, key + a * 64, head * p.vdim, bar(V_FULL + b));
+            }
+        }
+    } else if (elect_one()) {
+        const uint32_t idesc_s = instr_desc(BK), idesc_o = instr_desc(p.vdim);
+        bool ok = mbar_wait(bar(Q_FULL), 0, abort_flag);
+        auto issue_s = [&](int j) {
+            const int b = j & 1;
+            ok = ok && mbar_wait(bar(K_FULL + b), (j >> 1) & 1, abort_flag) && mbar_wait(bar(S_EMPTY + b), ((j >> 1) & 1) ^ 1, abort_flag);
+            if (!ok) return;
+            tc_fence_after();
+            uint32_t acc = 0;
+            for (int a = 0; a < nk; ++a) {
+                const int steps = (a < na ? min(64, p.dim - a * 64) : min(64, p.rot - (a - na) * 64)) / 16;
+                const uint64_t qd = smem_desc_sw128(sQ + a * ATOM), kd = smem_desc_sw128(sK + (b * nk + a) * ATOM);
+                for (int k = 0; k < steps; ++k) {
+                    mma_f16(tmem + b * 128, qd + 2 * k, kd + 2 * k, idesc_s, acc);
+                    acc = 1;
+                }
+            }
+            mma_commit(bar(S_FULL + b));
+            mma_commit(bar(K_EMPTY + b));
+        };
+        issue_s(0);
+        for (int j = 0; j < nt && ok; ++j) {
+            const int b = j & 1;
+            if (j + 1 < nt) issue_s(j + 1);
+            if (!ok) break;
+            ok = mbar_wait(bar(P_FULL), j & 1, abort_flag) && mbar_wait(bar(V_FULL + b), (j >> 1) & 1, abort_flag) &&
+                 mbar_wait(bar(O_EMPTY), (j & 1) ^ 1, abort_flag);
+            if (!ok) break;
+            tc_fence_after();
+#pragma unroll
+            for (int ks = 0; ks < 8; ++ks)          // 16 keys: 8 TMEM columns of P, 32 bytes of a V^T row
+                mma_f16_ts(tmem + T_O, tmem + T_P + ks * 8, smem_desc_sw128(sV + (b * 2 + (ks >> 2)) * ATOM) + 2 * (ks & 3), idesc_o, ks > 0 ? 1u : 0u);
+            mma_commit(bar(O_FULL));
+            mma_commit(bar(V_EMPTY + b));
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    teardown(abort_flag, tid, status);
+    if (warp == 9) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(512) : "memory");
+}
+
+// ------------------------------------------------------------------------------------------------------------------------
+// single rows: N heads of one row per CTA, keys in tiles of 128 (two pages)
+//   S^T = C Q^T       M = 128 keys, N heads, K = latent + rotated part: the cache rows are the A operand as they lie
+//   softmax           one thread per key (= TMEM lane), N columns; the maxima over keys are reduced across lanes
+//   O^T += C^T P^T    M = 128 latent values, N heads, K = 128 keys: the same rows again, read as an MN-major A operand
+// One copy of the cache rows therefore serves both products, and both fill the M dimension whatever the number of heads.
+// The accumulator stays in TMEM and is rescaled only when a running maximum rises by more than 2^RESCALE_STEP.
+// Warps 0-3 softmax, 4 TMA, 5 TMEM allocation and MMA issue.
+// ------------------------------------------------------------------------------------------------------------------------
+constexpr int ROWS_THREADS = 192, PAGE = 64, MAX_SLOTS = 8;
+constexpr float RESCALE_STEP = 8.f;
+enum RBar { R_FULL = 0, R_EMPTY = R_FULL + MAX_SLOTS, ROT_FULL = R_EMPTY + MAX_SLOTS, ROT_EMPTY, RS_FULL, RP_FULL, RO_DONE, RQ_FULL, R_MEET, R_BARS };
+
+struct RowsSmem { int n_blocks, n_slots; size_t bytes; };
+static __host__ __device__ inline RowsSmem rows_layout(int n, int latent) {
+    RowsSmem r;
+    r.n_blocks = latent / 128;
+    const size_t fixed = (size_t)(2 * r.n_blocks + 1 + 2) * n * 128 + ATOM + 1024;
+    r.n_slots = (int)((226 * 1024 + 512 - fixed) / (2 * ATOM));
+    const int want = 2 * r.n_blocks;
+    if (r.n_slots > want) r.n_slots = want;
+    if (r.n_slots > MAX_SLOTS) r.n_slots = MAX_SLOTS;
+    r.bytes = fixed + (size_t)r.n_slots * 2 * ATOM;
+    return r;
+}
+
+// v[c] over the 32 lanes of a warp -> lane c (and c + 16 for N = 16) holds the reduction of v[c]
+template <int N, bool SUM>
+LLM_DEVICE float reduce_columns(float (&v)[N], int lane) {
+    auto op = [](float a, float b) { return SUM ? a + b : fmaxf(a, b); };
+#pragma unroll
+    for (int w = N / 2; w > 0; w >>= 1) {
+        const bool hi = lane & w;
+#pragma unroll
+        for (int i = 0; i < w; ++i) {
+            const float keep = hi ? v[i + w] : v[i], send = hi ? v[i] : v[i + w];
+            v[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, w));
+        }
+    }
+    if (N == 16) v[0] = op(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
+    return v[0];
+}
+
+template <int N> LLM_DEVICE void tmem_ld_n(uint32_t taddr, uint32_t (&r)[N]);
+template <> LLM_DEVICE void tmem_ld_n<32>(uint32_t taddr, uint32_t (&r)[32]) { tmem_ld32_issue(taddr, r); tmem_wait_ld(r); }
+template <> LLM_DEVICE void tmem_ld_n<16>(uint32_t taddr, uint32_t (&r)[16]) {
+    asm volatile("tcgen05.ld.sync.aligned.32x32b.x16.b32 {%0,%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15}, [%16];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
+                   "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]) : "r"(taddr));
+    asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+#pragma unroll
+    for (int i = 0; i < 16; ++i) asm volatile("" : "+r"(r[i]));
+}
+template <int N> LLM_DEVICE void tmem_st_n(uint32_t taddr, const uint32_t (&r)[N]);
+template <> LLM_DEVICE void tmem_st_n<32>(uint32_t taddr, const uint32_t (&r)[32]) { tmem_st32(taddr, r); }
+template <> LLM_DEVICE void tmem_st_n<16>(uint32_t taddr, const uint32_t (&r)[16]) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x16.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16};"
+                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]),
+                   "r"(r[8]), "r"(r[9]), "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]) : "memory");
+}
+// MN-major, 128-byte swizzle: rows of 64 values along M, one row per k; 8-row groups 1024 bytes apart, 64-value groups `lead` apart
+LLM_DEVICE uint64_t smem_desc_mn_sw128(uint32_t addr, uint32_t lead) {
+    return (smem_desc_sw128(addr) & ~((uint64_t)0x3fff << 16)) | ((uint64_t)((lead >> 4) & 0x3fff) << 16);
+}
+
+template <int N>
+__global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const LatentRowsParams p, int* status) {
+    extern __shared__ uint8_t smem_raw[];
+    __shared__ __align__(8) uint64_t s_bars[R_BARS];
+    __shared__ uint32_t s_tmem;
+    __shared__ int s_abort[2];
+    __shared__ float s_red[4][32];                 // per warp: column maxima (and sums at the end)
+    __shared__ __align__(16) float s_head[4][32];  // per warp: running maximum (or factor) of every head, for broadcast reads
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const RowsSmem lay = rows_layout(N, p.rot_off);
+    const int NB = lay.n_blocks, NS = lay.n_slots, NA = 2 * NB + 1;
+    const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
+    const uint32_t sQ = base, sP = sQ + NA * N * 128, sR = sP + 2 * N * 128, sC = sR + ATOM;
+    const uint32_t bars = smem_u32(s_bars);
+    auto bar = [&](int i) { return bars + i * 8; };
+    pdl_trigger();
+    if (tid == 0) {
+        s_abort[0] = 0; s_abort[1] = 0;
+        for (int i = 0; i < R_BARS; ++i) mbar_init(bar(i), i == RP_FULL || i == RQ_FULL || i == R_MEET ? 4 : 1);
+        asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+        fence_proxy_async();
+    }
+    if (warp == 5) {
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(256) : "memory");
+        asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
+    }
+    tc_fence_before();
+    __syncthreads();
+    tc_fence_after();
+    const uint32_t tmem = s_tmem, t_o = tmem + 32;             // S^T in columns [0, N), O^T blocks behind
+    volatile int* abort_flag = s_abort;
+    pdl_wait();
+
+    const int hg = blockIdx.x, split = blockIdx.y, z = blockIdx.z;
+    const int t = p.rows ? p.rows[z] : z;
+    const int pos = p.positions[t], lo = first_key(pos, p.window);
+    const int* btab = p.block_table + (size_t)LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs) * p.max_pages;
+    const int page0 = lo / PAGE, page_last = pos / PAGE;
+    const int n_tiles = (page_last - page0) / 2 + 1, per = (n_tiles + gridDim.y - 1) / gridDim.y;
+    const int j0 = split * per, nt = max(0, min(n_tiles, j0 + per) - j0);
+    const size_t part = (((size_t)z * gridDim.x + hg) * gridDim.y + split) * N;
+
+    if (nt == 0) {
+        if (tid < N) *reinterpret_cast<float2*>(p.part_ml + (part + tid) * 2) = make_float2(-INFINITY, 0.f);
+    } else if (warp < 4) {
+        // query operand: N rows (heads) of [latent | rotated part, zero padded to one atom]
+        const int ul = p.rot_off / 8, ua = NA * 8;
+        for (int i = tid; i < N * ua; i += 128) {
+            const int r = i / ua, u = i % ua, h = hg * N + r;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (h < p.n_heads) {
+                if (u < ul) {
+                    v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q_lat) + (size_t)z * p.ql_row + (size_t)h * p.ql_head + u * 8);
+                } else if ((u - ul) * 8 < p.rot_dim) {
+                    const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off;
+                    const float2* ang = p.angles + (size_t)t * p.half;
+                    float x[8];
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) { const int c = (u - ul) * 8 + j; x[j] = c < p.rot_dim ? rotated(qr, c, ang, p.half) : 0.f; }
+                    v = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
+                }
+            }
+            st_shared_v4(atom_addr(sQ + (u >> 3) * N * 128, r, u & 7), v);
+        }
+        fence_proxy_async();
+        __syncwarp();
+        mbar_arrive_if(bar(RQ_FULL), lane == 0);
+
+        const uint32_t t_lane = (uint32_t)(warp * 32) << 16;
+        const float sl2 = p.scale * LOG2E;
+        float l[N], m = -INFINITY;                  // l: this key lane's share of every head's sum; m: lane c holds head c's maximum
+#pragma unroll
+        for (int c = 0; c < N; ++c) l[c] = 0.f;
+        bool ok = true;
+        int n_meet = 0;
+        auto meet = [&]() {                         // bounded rendezvous of the four softmax warps
+            __syncwarp();
+            mbar_arrive_if(bar(R_MEET), lane == 0);
+            const bool r = mbar_wait_warp(bar(R_MEET), n_meet & 1, abort_flag);
+            ++n_meet;
+            return r;
+        };
+        auto broadcast = [&](float mine, float (&out)[N]) {      // lane c's value -> out[c] in every lane
+            __syncwarp();
+            s_head[warp][lane] = mine;
+            __syncwarp();
+#pragma unroll
+            for (int c = 0; c < N; c += 4) {
+                const float4 f = *reinterpret_cast<const float4*>(&s_head[warp][c]);
+                out[c] = f.x; out[c + 1] = f.y; out[c + 2] = f.z; out[c + 3] = f.w;
+            }
+        };
+        for (int j = 0; j < nt && ok; ++j) {
+            ok = mbar_wait_warp(bar(RS_FULL), j & 1, abort_flag);
+            if (!ok) break;
+            tc_fence_after();
+            uint32_t raw[N];
+            tmem_ld_n<N>(tmem + t_lane, raw);
+            const int key = (page0 + 2 * (j0 + j)) * PAGE + tid;
+            const bool seen = key >= lo && key <= pos;
+            float s[N], red[N];
+#pragma unroll
+            for (int c = 0; c < N; ++c) { s[c] = seen ? __uint_as_float(raw[c]) * sl2 : -INFINITY; red[c] = s[c]; }
+            // (the previous tile's reads of s_red precede its P_FULL arrivals, without which this tile's S cannot be complete)
+            s_red[warp][lane] = reduce_columns<N, false>(red, lane);
+            ok = meet();
+            if (!ok) break;
+            const float mt = fmaxf(fmaxf(s_red[0][lane], s_red[1][lane]), fmaxf(s_red[2][lane], s_red[3][lane]));
+            const bool raise = mt > m + RESCALE_STEP;           // also the first tile, where m is -inf
+            const float m_old = m;
+            if (raise) m = mt;
+            if (j > 0) {                                        // P and the accumulator are free
+                ok = mbar_wait_warp(bar(RO_DONE), (j - 1) & 1, abort_flag);
+                if (!ok) break;
+                tc_fence_after();
+            }
+            if (__any_sync(0xffffffffu, raise) && j > 0) {      // the same in all four warps
+                float f[N];
+                broadcast(raise ? ex2(m_old - m) : 1.f, f);
+#pragma unroll
+                for (int c = 0; c < N; ++c) l[c] *= f[c];
+                for (int b = 0; b < NB; ++b) {
+                    tmem_ld_n<N>(t_o + b * N + t_lane, raw);
+#pragma unroll
+                    for (int c = 0; c < N; ++c) raw[c] = __float_as_uint(__uint_as_float(raw[c]) * f[c]);
+                    tmem_st_n<N>(t_o + b * N + t_lane, raw);
+                }
+                tmem_wait_st();
+            }
+            float mh[N];
+            broadcast(m, mh);
+            const uint32_t dst = sP + (tid >> 6) * N * 128 + (tid & 7) * 2;
+            const int unit = (tid & 63) >> 3;
+#pragma unroll
+            for (int c = 0; c < N; ++c) {
+                const float pr = ex2(s[c] - mh[c]);
+                l[c] += pr;
+                asm volatile("st.shared.b16 [%0], %1;" ::"r"(dst + c * 128 + (((unit ^ c) & 7) << 4)), "h"(__bfloat16_as_ushort(__float2bfloat16(pr))) : "memory");
+            }
+            tc_fence_before();
+            fence_proxy_async();
+            __syncwarp();
+            mbar_arrive_if(bar(RP_FULL), lane == 0);
+        }
+        // the last products are complete, so every warp has arrived with its P and is done with the maxima in s_red
+        ok = ok && mbar_wait_warp(bar(RO_DONE), (nt - 1) & 1, abort_flag);
+        if (ok) {
+            s_red[warp][lane] = reduce_columns<N, true>(l, lane);
+            ok = meet();
+        }
+        if (ok) {
+            tc_fence_after();
+            float lt = s_red[0][lane] + s_red[1][lane] + s_red[2][lane] + s_red[3][lane];       // lane c: head c
+            uint32_t raw[N];
+            if (gridDim.y == 1) {
+                const int h0 = hg * N;
+                if (p.sink && h0 + (lane & (N - 1)) < p.n_heads) lt += exp2f(p.sink[h0 + (lane & (N - 1))] * LOG2E - m);
+                float inv[N];
+                broadcast(1.f / lt, inv);
+                for (int b = 0; b < NB; ++b) {
+                    tmem_ld_n<N>(t_o + b * N + t_lane, raw);
+                    __nv_bfloat16* out = static_cast<__nv_bfloat16*>(p.out) + (size_t)z * p.out_row + b * 128 + tid;
+#pragma unroll
+                    for (int c = 0; c < N; ++c)
+                        if (h0 + c < p.n_heads) out[(size_t)(h0 + c) * p.out_head] = __float2bfloat16(__uint_as_float(raw[c]) * inv[c]);
+                }
+            } else {
+                for (int b = 0; b < NB; ++b) {
+                    tmem_ld_n<N>(t_o + b * N + t_lane, raw);
+                    float* out = p.part_o + part * p.rot_off + b * 128 + tid;
+#pragma unroll
+                    for (int c = 0; c < N; ++c) out[(size_t)c * p.rot_off] = __uint_as_float(raw[c]);
+                }
+                if (tid < N) *reinterpret_cast<float2*>(p.part_ml + (part + tid) * 2) = make_float2(m, lt);
+            }
+        }
+    } else if (warp == 4) {
+        if (elect_one()) {
+            bool ok = true;
+            int it = 0;
+            for (int j = 0; j < nt && ok; ++j) {
+                const int pg = page0 + 2 * (j0 + j);
+                // a page past the end repeats the last one (its keys are masked)
+                const int r0 = LLM_CHECK_INDEX(btab[pg], p.n_pages) * PAGE, r1 = LLM_CHECK_INDEX(btab[min(pg + 1, page_last)], p.n_pages) * PAGE;
+                auto load = [&](uint32_t dst, int col, uint32_t full) {
+                    tma_load_2d(dst, &map_kv, col, r0, full);
+                    tma_load_2d(dst + ATOM / 2, &map_kv, col, r1, full);
+                };
+                ok = mbar_wait(bar(ROT_EMPTY), (j & 1) ^ 1, abort_flag);
+                if (!ok) break;
+                mbar_arrive_expect_tx(bar(ROT_FULL), ATOM);
+                load(sR, p.rot_off, bar(ROT_FULL));
+                for (int b = 0; b < NB; ++b, ++it) {
+                    const int slot = it % NS;
+                    ok = mbar_wait(bar(R_EMPTY + slot), ((it / NS) & 1) ^ 1, abort_flag);
+                    if (!ok) break;
+                    mbar_arrive_expect_tx(bar(R_FULL + slot), 2 * ATOM);
+                    load(sC + slot * 2 * ATOM, b * 128, bar(R_FULL + slot));
+                    load(sC + slot * 2 * ATOM + ATOM, b * 128 + 64, bar(R_FULL + slot));
+                }
+            }
+        }
+    } else if (elect_one()) {
+        const uint32_t idesc_s = instr_desc(N), idesc_o = instr_desc(N) | (1u << 15);       // bit 15: A is MN-major
+        const int rot_steps = (p.width - p.rot_off) / 16;
+        bool ok = mbar_wait(bar(RQ_FULL), 0, abort_flag);
+        for (int j = 0; j < nt && ok; ++j) {
+            for (int b = 0; b < NB && ok; ++b) {
+                const int it = j * NB + b, slot = it % NS;
+                ok = mbar_wait(bar(R_FULL + slot), (it / NS) & 1, abort_flag);
+                if (!ok) break;
+                tc_fence_after();
+#pragma unroll
+                for (int ks = 0; ks < 8; ++ks)
+                    mma_f16(tmem, smem_desc_sw128(sC + slot * 2 * ATOM + (ks >> 2) * ATOM) + 2 * (ks & 3),
+                            smem_desc_sw128(sQ + (2 * b + (ks >> 2)) * N * 128) + 2 * (ks & 3), idesc_s, b > 0 || ks > 0 ? 1u : 0u);
+            }
+            ok = ok && mbar_wait(bar(ROT_FULL), j & 1, abort_flag);
+            if (!ok) break;
+            tc_fence_after();
+            for (int ks = 0; ks < rot_steps; ++ks)
+                mma_f16(tmem, smem_desc_sw128(sR) + 2 * ks, smem_desc_sw128(sQ + 2 * NB * N * 128) + 2 * ks, idesc_s, 1u);
+            mma_commit(bar(RS_FULL));
+            mma_commit(bar(ROT_EMPTY));
+            ok = mbar_wait(bar(RP_FULL), j & 1, abort_flag);
+            if (!ok) break;
+            tc_fence_after();
+            for (int b = 0; b < NB; ++b) {
+                const int slot = (j * NB + b) % NS;
+#pragma unroll
+                for (int ks = 0; ks < 8; ++ks)              // 16 keys: two groups of eight rows
+                    mma_f16(t_o + b * N, smem_desc_mn_sw128(sC + slot * 2 * ATOM + ks * 2048, ATOM), smem_desc_sw128(sP + (ks >> 2) * N * 128) + 2 * (ks & 3),
+                            idesc_o, j > 0 || ks > 0 ? 1u : 0u);
+                mma_commit(bar(R_EMPTY + slot));
+            }
+            mma_commit(bar(RO_DONE));
+        }
+    }
+    tc_fence_before();
+    __syncthreads();
+    teardown(abort_flag, tid, status);
+    if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(256) : "memory");
+}
+
+// ---- host side ---------------------------------------------------------------------------------------------------------
+typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
+                                  const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+static EncodeTiledFn encode_fn() {
+    static EncodeTiledFn fn = nullptr;
+    if (!fn) {
+        void* ptr = nullptr;
+        cudaDriverEntryPointQueryResult qres;
+        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &ptr, cudaEnableDefault, &qres) == cudaSuccess && qres == cudaDriverEntryPointSuccess)
+            fn = reinterpret_cast<EncodeTiledFn>(ptr);
+    }
+    return fn;
+}
+// bf16 matrix [rows, cols] with the given row stride (elements); boxes of 64 columns x box_rows rows, 128-byte swizzle
+static bool make_map(CUtensorMap* m, const void* ptr, uint64_t cols, uint64_t rows, uint64_t stride, uint32_t box_rows) {
+    EncodeTiledFn enc = encode_fn();
+    if (!enc || (reinterpret_cast<uintptr_t>(ptr) & 15) || stride % 8) return false;
+    const cuuint64_t dims[2] = {cols, rows}, strides[1] = {stride * 2};
+    const cuuint32_t box[2] = {64, box_rows}, estr[2] = {1, 1};
+    return enc(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(ptr), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+template <class K> static cudaError_t raise_smem(K kernel, size_t bytes) {
+    return cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes);
+}
+
+}  // namespace ltc
+
+bool latent_chunk_tc_fits(int dim, int rot, int vdim) {
+    const int nk = (dim + 63) / 64 + (rot + 63) / 64;
+    return dim % 16 == 0 && rot % 16 == 0 && vdim % 16 == 0 && dim > 0 && rot > 0 && vdim >= 16 && vdim <= 128 && nk <= 3;
+}
+
+cudaError_t launch_latent_chunk_tc(const LatentChunkParams& p, int n_keys, int n_seqs, int max_q_len, int* status, cudaStream_t st) {
+    using namespace ltc;
+    if (!latent_chunk_tc_fits(p.dim, p.rot, p.vdim) || p.n_heads > 65535 || n_seqs > 65535 || n_keys % 8) return cudaErrorInvalidValue;
+    CUtensorMap mk, ml, mv;
+    if (!make_map(&mk, p.k, (uint64_t)p.n_heads * p.dim, n_keys, (uint64_t)p.n_heads * p.dim, 128) || !make_map(&ml, p.lat, p.lat_row, n_keys, p.lat_row, 128) ||
+        !make_map(&mv, p.v, n_keys, (uint64_t)p.n_heads * p.vdim, n_keys, p.vdim))
+        return cudaErrorInvalidValue;
+    const int nk = (p.dim + 63) / 64 + (p.rot + 63) / 64;
+    const size_t smem = (size_t)(3 * nk + 4) * ATOM + 1024;
+    const dim3 grid((max_q_len + BQ - 1) / BQ, p.n_heads, n_seqs);
+    auto go = [&](auto kernel) {
+        cudaError_t e = raise_smem(kernel, smem);
+        if (e != cudaSuccess) return e;
+        kernel<<<grid, CHUNK_THREADS, smem, st>>>(mk, ml, mv, p, status);
+        return cudaGetLastError();
+    };
+    return p.vdim <= 64 ? go(latent_chunk_tc_kernel<64>) : go(latent_chunk_tc_kernel<128>);
+}
+
+int latent_rows_tc_heads(int width, int rot_off, int rot_dim, int n_heads) {
+    if (rot_off % 128 || rot_off < 128 || rot_off > 512 || width % 16 || width - rot_off > 64 || width <= rot_off || rot_dim <= 0) return 0;
+    const int n = n_heads <= 16 ? 16 : 32;
+    return ltc::rows_layout(n, rot_off).n_slots >= rot_off / 128 ? n : 0;
+}
+
+cudaError_t launch_latent_rows_tc(const LatentRowsParams& p, int rows, int n_splits, int* status, cudaStream_t st) {
+    using namespace ltc;
+    const int n = latent_rows_tc_heads(p.width, p.rot_off, p.rot_dim, p.n_heads);
+    if (!n || rows > 65535 || p.ql_row % 8 || p.ql_head % 8) return cudaErrorInvalidValue;
+    CUtensorMap m;
+    if (!make_map(&m, p.kv, p.width, (uint64_t)p.n_pages * PAGE, p.width, PAGE)) return cudaErrorInvalidValue;
+    const size_t smem = rows_layout(n, p.rot_off).bytes;
+    const dim3 grid((p.n_heads + n - 1) / n, n_splits, rows);
+    auto go = [&](auto kernel) {
+        cudaError_t e = raise_smem(kernel, smem);
+        return e != cudaSuccess ? e : launch_pdl(kernel, grid, dim3(ROWS_THREADS), smem, st, m, p, status);
+    };
+    return n == 16 ? go(latent_rows_tc_kernel<16>) : go(latent_rows_tc_kernel<32>);
+}
+
+int bounds_status_latent_tc(bool reset);
+LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_latent_tc)
+
+}  // namespace llm

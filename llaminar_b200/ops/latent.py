@@ -10,9 +10,8 @@ import torch
 from . import _count
 from . import build as _build
 
-ROWS_PER_GROUP = 16            # heads that share the M dimension of the row kernel's MMA
-KEYS_PER_TILE = 32
-GEMV_MAX_ROWS = 4
+GEMV_MAX_ROWS = 4              # rows the kernel takes
+GEMV_ROWS = 2                  # rows up to which it is preferred to cuBLAS
 _GEMV_SMEM = 200 * 1024
 _ready = False
 
@@ -53,22 +52,36 @@ def latent_prep(down, q_norm, kv_norm, angles, positions, seq_ids, block_table, 
     _count()
 
 
-def rows_splits(n_rows: int, n_heads: int, max_keys: int, latent: int, capacity: int) -> int:
-    """Key splits of the row kernel: enough CTAs for two per SM, at least two key tiles per split, partial sums within
-    ``capacity`` floats."""
-    groups = -(-n_heads // ROWS_PER_GROUP)
-    tiles = -(-max_keys // KEYS_PER_TILE) + 1
-    want = max(1, min(296 // max(1, n_rows * groups), tiles // 2, 64))
-    return max(1, min(want, capacity // max(1, n_rows * groups * ROWS_PER_GROUP * latent)))
+def rows_group(kv: torch.Tensor, latent: int, rot_dim: int, n_heads: int, tensor_core: bool = True) -> int:
+    """Heads that share a CTA of the row kernel for these sizes: the tcgen05 form where it fits, 16 for the mma.sync form,
+    0 for the plain kernel (32-bit cache, unusual sizes)."""
+    if kv.dtype != torch.bfloat16:
+        return 0
+    e, width = ext(), kv.shape[2]
+    tc = e.latent_rows_tc_heads(width, latent, rot_dim, n_heads) if tensor_core else 0
+    return tc or (16 if e.latent_rows_has_kernel(width, latent) else 0)
+
+
+def rows_splits(n_rows: int, n_heads: int, group: int, tensor_core: bool, max_keys: int, latent: int, capacity: int) -> int:
+    """Key splits of the row kernel: about one CTA per SM (tcgen05) or two (mma.sync), whole key tiles per split, evenly
+    shared, partial sums within ``capacity`` floats."""
+    if group == 0:
+        return 1
+    groups = -(-n_heads // group)
+    tiles = max_keys // (128 if tensor_core else 32) + 1            # a window that starts inside a tile touches one more
+    want = max(1, min(tiles, (148 if tensor_core else 296) // max(1, n_rows * groups), 64))
+    want = max(1, min(want, capacity // max(1, n_rows * groups * group * latent)))
+    per = -(-tiles // want)
+    return -(-tiles // per)
 
 
 def latent_rows(q_lat, q, q_rot_off: int, angles, rows, positions, seq_ids, block_table, kv, rot_dim: int, window: int, scale: float,
-                sink, out, part_o, part_ml, n_splits: int) -> None:
-    """Attention of single rows over the latent cache, queries and results in the latent space ([heads, rows, latent])."""
-    e = ext()
-    e.latent_rows(q_lat, q, q_rot_off, angles, rows, positions, seq_ids, block_table, kv, rot_dim, window, scale, sink, out,
-                  part_o, part_ml, n_splits)
-    _count(2 if n_splits > 1 and kv.dtype == torch.bfloat16 and e.latent_rows_has_kernel(kv.shape[2], q_lat.shape[2]) else 1)
+                sink, out, part_o, part_ml, n_splits: int, group: int, status) -> None:
+    """Attention of single rows over the latent cache, queries and results in the latent space ([heads, rows, latent]).
+    ``group``: see `rows_group`; ``status``: device word of the tcgen05 form."""
+    ext().latent_rows(q_lat, q, q_rot_off, angles, rows, positions, seq_ids, block_table, kv, rot_dim, window, scale, sink, out,
+                      part_o, part_ml, n_splits, group, status)
+    _count(2 if n_splits > 1 and group else 1)
 
 
 def latent_gather(kv, seqs, max_k_len: int, block_table, out) -> None:
@@ -77,10 +90,11 @@ def latent_gather(kv, seqs, max_k_len: int, block_table, out) -> None:
     _count()
 
 
-def latent_chunk(q, angles, kvx, lat, rot_off: int, seqs, max_q_len: int, out, dim: int, rot: int, vdim: int, window: int,
-                 scale: float, sink) -> None:
-    """Attention of prompt chunks on keys and values written out per head (``kvx``) and the shared rotated parts in ``lat``."""
-    ext().latent_chunk(q, angles, kvx, lat, rot_off, seqs, max_q_len, out, dim, rot, vdim, window, scale, sink)
+def latent_chunk(q, angles, k, v, lat, rot_off: int, seqs, max_q_len: int, out, dim: int, rot: int, vdim: int, window: int,
+                 scale: float, sink, status=None) -> None:
+    """Attention of prompt chunks on keys and values written out per head and the shared rotated parts in ``lat``.  With
+    ``status`` the tcgen05 form runs, which takes the values transposed ([heads * vdim, keys])."""
+    ext().latent_chunk(q, angles, k, v, lat, rot_off, seqs, max_q_len, out, dim, rot, vdim, window, scale, sink, status)
     _count()
 
 
@@ -88,10 +102,14 @@ def chunk_has_kernel(dk: int, dv: int) -> bool:
     return bool(ext().latent_chunk_has_kernel(dk, dv))
 
 
+def chunk_tc_fits(dim: int, rot: int, vdim: int) -> bool:
+    return bool(ext().latent_chunk_tc_fits(dim, rot, vdim))
+
+
 def gemv_fits(w: torch.Tensor, x: torch.Tensor) -> bool:
     """Whether `gemv_dense` takes this product: few bf16 rows, 16-byte rows."""
     k = w.shape[-1]
-    return (w.dtype == torch.bfloat16 and x.shape[-2] <= GEMV_MAX_ROWS and k % 8 == 0 and x.stride(-2) % 8 == 0 and w.stride(-2) % 8 == 0
+    return (w.dtype == torch.bfloat16 and x.shape[-2] <= GEMV_ROWS and k % 8 == 0 and x.stride(-2) % 8 == 0 and w.stride(-2) % 8 == 0
             and x.shape[-2] * k * 2 <= _GEMV_SMEM and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
