@@ -194,7 +194,7 @@ def norms(cfg: ModelConfig, n: int) -> list[dict]:
     return rows
 
 
-def products(cfg: ModelConfig, rows_list=(1, 2, 4, 32)) -> list[dict]:
+def products(cfg: ModelConfig, rows_list=(1, 4, 8, 32)) -> list[dict]:
     """Matrix products of a decode step: bf16 weights here, 8-bit blocks on the quantised kernels for comparison."""
     from . import ops as base
     from .engine.latent import DenseLinear, PaddedSizes
@@ -210,7 +210,7 @@ def products(cfg: ModelConfig, rows_list=(1, 2, 4, 32)) -> list[dict]:
             c = copies_for(n * k * 2)
             lins = [DenseLinear(torch.randn(n, k, **bf)) for _ in range(c)]
             x, y = torch.randn(rows, k, **bf), torch.empty(rows, n, **bf)
-            kind = "gemv_dense" if rows <= ops.GEMV_ROWS else "cuBLAS"
+            kind = "gemv_dense" if rows <= ops.GEMV_MAX_ROWS else "cuBLAS"
             out.append(_row(f"{name} [{n}, {k}] x {rows} rows ({kind})", time_us([lambda l=l: l(x, y) for l in lins]), n * k * 2, 2.0 * n * k * rows))
             del lins
         c = copies_for(ff * d * 4)

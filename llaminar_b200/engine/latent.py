@@ -8,10 +8,10 @@ Per layer (the residual stream h is fp32, everything else bf16, or float in 32-b
     attention                                                   latent_rows (queries moved into the latent space: decode steps and
                                                                 short portions) or latent_chunk (keys and values written out)
     y = Wo o ; h += norm(y) ; xn = norm(h)                      resid_norm
-    act = gelu(Wg xn) * (Wu xn) ; y = Wd act                    fused into the product up to four rows
+    act = gelu(Wg xn) * (Wu xn) ; y = Wd act                    fused into the product up to eight rows
     h += norm(y) ; xn = norm(h) of the next layer               resid_norm
 
-Matrix products run on `gemv_dense` up to four rows and on cuBLAS above.  Head sizes and the latent are zero-padded to
+Matrix products run on `gemv_dense` up to eight rows and on cuBLAS above.  Head sizes and the latent are zero-padded to
 multiples of 8 values when the weights are loaded, so that every row the kernels copy starts on a 16-byte boundary.
 """
 from __future__ import annotations

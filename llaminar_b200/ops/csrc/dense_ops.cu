@@ -156,72 +156,75 @@ __global__ void rope_angles_kernel(const int* positions, const double* freqs, do
     out[i] = make_float2((float)magnitude * c, (float)magnitude * s);
 }
 
-// A group of LPR lanes computes one output column for all M rows; x is staged in shared memory once per CTA, which walks
-// over the columns with stride gridDim.x.  GELU: two weight rows (gate and up) per output column.
-template <int M, int LPR, bool GELU, class TO>
-__global__ void __launch_bounds__(256) gemv_dense_kernel(const GemvDenseParams p) {
-    extern __shared__ __align__(16) uint8_t smem_x[];
+// Up to eight rows of x against 16 weight rows per warp on the tensor cores (the weights are the M operand).  Thread (g, t) of
+// a warp loads 8 consecutive k of weight rows g and g + 8 and of x row g in one 16-byte access each; since both operands use
+// the same assignment of k to MMA slots, its order does not matter and no operand passes through shared memory.  `wk` warps
+// share the K range of a row block and add up in shared memory.  GELU: a second set of weight rows (n further down) per block.
+constexpr int SKINNY_WARPS = 8;
+LLM_DEVICE void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+template <bool GELU, class TO>
+__global__ void __launch_bounds__(32 * SKINNY_WARPS) gemv_dense_kernel(const GemvDenseParams p, int wk) {
+    __shared__ float s_acc[SKINNY_WARPS][GELU ? 2 : 1][16][9];
     pdl_trigger();
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    constexpr int RPW = 32 / LPR;                               // columns per warp
-    const int sub = lane / LPR, l = lane % LPR;
-    const __nv_bfloat16* W = p.w + (size_t)blockIdx.y * p.w_z;
-    const int units = p.k / 8;
-    pdl_wait();
-    uint4* sx = reinterpret_cast<uint4*>(smem_x);               // [M][units]
-    for (int i = threadIdx.x; i < M * units; i += 256)
-        sx[i] = *reinterpret_cast<const uint4*>(p.x + (size_t)blockIdx.y * p.x_z + (i / units) * p.x_row + (size_t)(i % units) * 8);
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
+    const int part = warp % wk, n0 = (blockIdx.x * (SKINNY_WARPS / wk) + warp / wk) * 16;
+    const int blocks = (p.k + 31) / 32, per = (blocks + wk - 1) / wk, kb0 = part * per, kb1 = min(blocks, kb0 + per);
+    constexpr int UN = GELU ? 4 : 8, NW = GELU ? 4 : 2;
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    float acc[GELU ? 2 : 1][4] = {};
+    // rows past the end repeat the last one (never stored)
+    const __nv_bfloat16* w[NW];
+#pragma unroll
+    for (int i = 0; i < NW; ++i) w[i] = p.w + (size_t)blockIdx.y * p.w_z + (size_t)(min(n0 + g + (i & 1) * 8, p.n - 1) + (i >> 1) * p.n) * p.ldw + t * 8;
+    const __nv_bfloat16* x = p.x + (size_t)blockIdx.y * p.x_z + (size_t)min(g, p.m - 1) * p.x_row + t * 8;
+    const bool live = n0 < p.n;
+    bool waited = false;
+    for (int kb = kb0; kb < kb1 && live; kb += UN) {
+        uint4 wv[UN][NW], xv[UN];
+#pragma unroll
+        for (int u = 0; u < UN; ++u) {
+            const bool in = kb + u < kb1 && (kb + u) * 32 + t * 8 < p.k;
+#pragma unroll
+            for (int i = 0; i < NW; ++i) wv[u][i] = in ? ldg_nc_v4(w[i] + (size_t)(kb + u) * 32) : zero;
+        }
+        if (!waited) { pdl_wait(); waited = true; }             // the first weights are on their way before x is complete
+#pragma unroll
+        for (int u = 0; u < UN; ++u) {
+            const bool in = kb + u < kb1 && (kb + u) * 32 + t * 8 < p.k && g < p.m;
+            xv[u] = in ? *reinterpret_cast<const uint4*>(x + (size_t)(kb + u) * 32) : zero;
+        }
+#pragma unroll
+        for (int u = 0; u < UN; ++u) {
+#pragma unroll
+            for (int i = 0; i < NW / 2; ++i) {
+                mma_bf16(acc[i], wv[u][2 * i].x, wv[u][2 * i + 1].x, wv[u][2 * i].y, wv[u][2 * i + 1].y, xv[u].x, xv[u].y);
+                mma_bf16(acc[i], wv[u][2 * i].z, wv[u][2 * i + 1].z, wv[u][2 * i].w, wv[u][2 * i + 1].w, xv[u].z, xv[u].w);
+            }
+        }
+    }
+    if (!waited) pdl_wait();
+#pragma unroll
+    for (int i = 0; i < NW / 2; ++i) {
+        s_acc[warp][i][g][2 * t] = acc[i][0]; s_acc[warp][i][g][2 * t + 1] = acc[i][1];
+        s_acc[warp][i][g + 8][2 * t] = acc[i][2]; s_acc[warp][i][g + 8][2 * t + 1] = acc[i][3];
+    }
     __syncthreads();
-    constexpr int UN = 4;
-    for (int n0 = (blockIdx.x * 8 + warp) * RPW; n0 < p.n; n0 += gridDim.x * 8 * RPW) {
-        const int n = n0 + sub;
-        const bool live = n < p.n;
-        const __nv_bfloat16* wr = W + (size_t)(live ? n : p.n - 1) * p.ldw;
-        const __nv_bfloat16* wr2 = GELU ? wr + (size_t)p.n * p.ldw : wr;
-        float acc[M] = {}, acc2[M] = {};
-        auto fma8 = [&](const uint4& w, int u, float (&a)[M]) {
-            const uint32_t ws[4] = {w.x, w.y, w.z, w.w};
-#pragma unroll
-            for (int m = 0; m < M; ++m) {
-                const uint4 xv = sx[m * units + u];
-                const uint32_t xs[4] = {xv.x, xv.y, xv.z, xv.w};
-#pragma unroll
-                for (int j = 0; j < 4; ++j) {
-                    a[m] = fmaf(bf16_lo(ws[j]), bf16_lo(xs[j]), a[m]);
-                    a[m] = fmaf(bf16_hi(ws[j]), bf16_hi(xs[j]), a[m]);
-                }
-            }
-        };
-        int u = l;
-        for (; u + (UN - 1) * LPR < units; u += UN * LPR) {
-            uint4 w[UN], w2[GELU ? UN : 1];
-#pragma unroll
-            for (int i = 0; i < UN; ++i) {
-                w[i] = ldg_nc_v4(wr + (size_t)(u + i * LPR) * 8);
-                if constexpr (GELU) w2[i] = ldg_nc_v4(wr2 + (size_t)(u + i * LPR) * 8);
-            }
-#pragma unroll
-            for (int i = 0; i < UN; ++i) {
-                fma8(w[i], u + i * LPR, acc);
-                if constexpr (GELU) fma8(w2[i], u + i * LPR, acc2);
-            }
+    // 16 columns x m rows per row block of the CTA
+    const int rb = SKINNY_WARPS / wk;
+    for (int i = threadIdx.x; i < rb * 16 * p.m; i += 32 * SKINNY_WARPS) {
+        const int c = i % (rb * 16), m = i / (rb * 16), n = blockIdx.x * rb * 16 + c;
+        if (n >= p.n) continue;
+        float v = 0.f, v2 = 0.f;
+        for (int q = 0; q < wk; ++q) {
+            v += s_acc[(c / 16) * wk + q][0][c % 16][m];
+            if constexpr (GELU) v2 += s_acc[(c / 16) * wk + q][1][c % 16][m];
         }
-        for (; u < units; u += LPR) {
-            fma8(ldg_nc_v4(wr + (size_t)u * 8), u, acc);
-            if constexpr (GELU) fma8(ldg_nc_v4(wr2 + (size_t)u * 8), u, acc2);
-        }
-#pragma unroll
-        for (int m = 0; m < M; ++m) {
-#pragma unroll
-            for (int o = LPR / 2; o > 0; o >>= 1) {
-                acc[m] += __shfl_xor_sync(0xffffffffu, acc[m], o);
-                if constexpr (GELU) acc2[m] += __shfl_xor_sync(0xffffffffu, acc2[m], o);
-            }
-            float v = acc[m];
-            // the two halves are rounded like the stored projection of the unfused form
-            if constexpr (GELU) v = gelu_tanh(__bfloat162float(__float2bfloat16(v))) * __bfloat162float(__float2bfloat16(acc2[m]));
-            if (live && l == 0) static_cast<TO*>(p.out)[(size_t)blockIdx.y * p.o_z + m * p.o_row + n] = from_f<TO>(v);
-        }
+        // the two halves are rounded like the stored projection of the unfused form
+        if constexpr (GELU) v = gelu_tanh(__bfloat162float(__float2bfloat16(v))) * __bfloat162float(__float2bfloat16(v2));
+        static_cast<TO*>(p.out)[(size_t)blockIdx.y * p.o_z + m * p.o_row + n] = from_f<TO>(v);
     }
 }
 
@@ -244,28 +247,6 @@ cudaError_t resid_norm_any(const ResidNormParams& p, int rows, cudaStream_t st) 
     return go(resid_norm_kernel<T, 1, 256>, 256);
 }
 
-template <int M, class TO>
-cudaError_t gemv_m(const GemvDenseParams& p, cudaStream_t st) {
-    const int units = p.k / 8;
-    const size_t smem = (size_t)M * p.k * 2;
-    auto go = [&](auto kernel, int lpr) {
-        cudaError_t e = raise_smem(kernel, smem);
-        if (e != cudaSuccess) return e;
-        const int cols = 8 * (32 / lpr);
-        int gx = (p.n + cols - 1) / cols;
-        const int cap = 148 * 8;
-        if (gx > cap) gx = cap;
-        return launch_pdl(kernel, dim3(gx, p.z), dim3(256), smem, st, p);
-    };
-    if (p.gelu) {
-        if constexpr (sizeof(TO) == 2) return go(gemv_dense_kernel<M, 32, true, TO>, 32);
-        return cudaErrorInvalidValue;
-    }
-    if (units <= 8) return go(gemv_dense_kernel<M, 8, false, TO>, 8);
-    if (units <= 24) return go(gemv_dense_kernel<M, 16, false, TO>, 16);
-    return go(gemv_dense_kernel<M, 32, false, TO>, 32);
-}
-
 }  // namespace
 
 cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cudaStream_t st) {
@@ -286,18 +267,16 @@ cudaError_t launch_rope_angles(const int* positions, const double* freqs, double
 }
 
 cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st) {
-    if (p.m < 1 || p.m > 4 || p.k % 8 || p.ldw % 8 || p.w_z % 8 || p.x_row % 8 || p.x_z % 8 || (size_t)p.m * p.k * 2 > 200 * 1024)
-        return cudaErrorInvalidValue;
-    auto by_m = [&](auto tag) {
-        using TO = decltype(tag);
-        switch (p.m) {
-            case 1: return gemv_m<1, TO>(p, st);
-            case 2: return gemv_m<2, TO>(p, st);
-            case 3: return gemv_m<3, TO>(p, st);
-            default: return gemv_m<4, TO>(p, st);
-        }
-    };
-    return p.out_f32 ? by_m(float()) : by_m(__nv_bfloat16());
+    if (p.m < 1 || p.m > 8 || p.n < 1 || p.k % 8 || p.ldw % 8 || p.w_z % 8 || p.x_row % 8 || p.x_z % 8 || (p.gelu && p.out_f32)) return cudaErrorInvalidValue;
+    // split K until every warp has about eight blocks of 32 and the grid fills the machine
+    const int blocks = (p.k + 31) / 32, tiles = (p.n + 15) / 16 * p.z;
+    int wk = 1;
+    while (wk < SKINNY_WARPS && blocks >= 16 * wk && (blocks > 64 * wk || tiles * wk < 148 * 32)) wk *= 2;
+    const int cols = SKINNY_WARPS / wk * 16;
+    const dim3 grid((p.n + cols - 1) / cols, p.z);
+    auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(32 * SKINNY_WARPS), 0, st, p, wk); };
+    if (p.gelu) return go(gemv_dense_kernel<true, __nv_bfloat16>);
+    return p.out_f32 ? go(gemv_dense_kernel<false, float>) : go(gemv_dense_kernel<false, __nv_bfloat16>);
 }
 
 LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_dense)

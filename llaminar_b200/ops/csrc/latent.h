@@ -98,7 +98,7 @@ bool latent_chunk_has_kernel(int dk, int dv);
 cudaError_t launch_latent_chunk_tc(const LatentChunkParams& p, int n_keys, int n_seqs, int max_q_len, int* status, cudaStream_t st);
 bool latent_chunk_tc_fits(int dim, int rot, int vdim);
 
-// out[z][m, :] = x[z][m, :] W[z]^T for up to 4 rows, bf16 weights.  gelu: W holds 2n rows and out = gelu_tanh(first n) * second n.
+// out[z][m, :] = x[z][m, :] W[z]^T for up to 8 rows, bf16 weights.  gelu: W holds 2n rows and out = gelu_tanh(first n) * second n.
 struct GemvDenseParams {
     const __nv_bfloat16* w; size_t w_z; int ldw;
     const __nv_bfloat16* x; size_t x_row, x_z;

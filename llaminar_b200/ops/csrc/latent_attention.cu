@@ -64,7 +64,7 @@ template <class T> LLM_DEVICE float rotated(const T* x, int i, const float2* ang
     return to_f(x[i]);
 }
 
-// values i0 .. i0 + 7 of it, zero from `n` on
+// values i0 .. i0 + 7 of it, zero from `n` on (reads no value past n)
 LLM_DEVICE uint4 rotated8(const __nv_bfloat16* x, int i0, int n, const float2* ang, int half) {
     float v[8];
 #pragma unroll
@@ -104,56 +104,58 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(const LatentPrepParams
     }
 }
 
-// The bf16 form for sizes that are multiples of 8: a thread keeps up to PREP_UNITS 16-byte units of the row in registers.
-constexpr int PREP_UNITS = 4, PREP_THREADS = 256;
-__global__ void __launch_bounds__(PREP_THREADS) latent_prep_vec_kernel(const LatentPrepParams p) {
-    __shared__ float red[2][PREP_THREADS / 32];
+// The bf16 form for sizes that are multiples of 8: a warp per token, which keeps the row in registers as 16-byte units.
+constexpr int PREP_UNITS = 12, PREP_WARPS = 4;
+template <int UNITS>
+__global__ void __launch_bounds__(32 * PREP_WARPS) latent_prep_vec_kernel(const LatentPrepParams p, int rows) {
     pdl_trigger();
     pdl_wait();
-    const int t = blockIdx.x, tid = threadIdx.x;
+    const int lane = threadIdx.x & 31, t = blockIdx.x * PREP_WARPS + (threadIdx.x >> 5);
+    if (t >= rows) return;
     const __nv_bfloat16* d = static_cast<const __nv_bfloat16*>(p.down) + (size_t)t * p.down_stride;
     const int nq = p.q_rank / 8, n = nq + p.kv_rank / 8;
-    uint4 w[PREP_UNITS];
-    float sq = 0.f, sk = 0.f;
+    uint4 w[UNITS];
 #pragma unroll
-    for (int i = 0; i < PREP_UNITS; ++i) {
-        const int u = tid + i * PREP_THREADS;
+    for (int i = 0; i < UNITS; ++i) {
+        const int u = lane + i * 32;
         w[i] = u < n ? *reinterpret_cast<const uint4*>(d + u * 8) : make_uint4(0, 0, 0, 0);
     }
     const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
     const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
     __nv_bfloat16* row = static_cast<__nv_bfloat16*>(p.kv) + ((size_t)page * PAGE + pos % PAGE) * p.width;
-    // rotated part and padding by the last threads, while the sums are on their way
-    const int ur = (p.width - p.rot_off) / 8, r = PREP_THREADS - 1 - tid;
-    for (int u = r; u < ur; u += PREP_THREADS)
+    for (int u = lane; u < (p.width - p.rot_off) / 8; u += 32)           // rotated part and padding
         *reinterpret_cast<uint4*>(row + p.rot_off + u * 8) = rotated8(d + p.q_rank + p.kv_rank, u * 8, p.rot_dim, p.angles + (size_t)t * p.half, p.half);
+    float sq = 0.f, sk = 0.f;
 #pragma unroll
-    for (int i = 0; i < PREP_UNITS; ++i) {
+    for (int i = 0; i < UNITS; ++i) {
         const uint32_t x[4] = {w[i].x, w[i].y, w[i].z, w[i].w};
         float ss = 0.f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) { const float a = bf16_lo(x[j]), b = bf16_hi(x[j]); ss += a * a + b * b; }
-        if (tid + i * PREP_THREADS < nq) sq += ss; else sk += ss;
+        if (lane + i * 32 < nq) sq += ss; else sk += ss;
     }
     sq = warp_sum(sq); sk = warp_sum(sk);
-    if ((tid & 31) == 0) { red[0][tid >> 5] = sq; red[1][tid >> 5] = sk; }
-    __syncthreads();
-    sq = sk = 0.f;
-#pragma unroll
-    for (int i = 0; i < PREP_THREADS / 32; ++i) { sq += red[0][i]; sk += red[1][i]; }
     const float iq = 1.f / sqrtf(sq / (float)p.q_rank + p.eps), ik = 1.f / sqrtf(sk / (float)p.kv_rank + p.eps);
 #pragma unroll
-    for (int i = 0; i < PREP_UNITS; ++i) {
-        const int u = tid + i * PREP_THREADS;
-        if (u >= n) break;
-        const bool q = u < nq;
-        const float* g = q ? p.q_norm + u * 8 : p.kv_norm + (u - nq) * 8;
-        const float inv = q ? iq : ik;
-        const float4 g0 = *reinterpret_cast<const float4*>(g), g1 = *reinterpret_cast<const float4*>(g + 4);
-        const uint4 o = make_uint4(pack_bf16(bf16_lo(w[i].x) * inv * g0.x, bf16_hi(w[i].x) * inv * g0.y), pack_bf16(bf16_lo(w[i].y) * inv * g0.z, bf16_hi(w[i].y) * inv * g0.w),
-                                   pack_bf16(bf16_lo(w[i].z) * inv * g1.x, bf16_hi(w[i].z) * inv * g1.y), pack_bf16(bf16_lo(w[i].w) * inv * g1.z, bf16_hi(w[i].w) * inv * g1.w));
-        __nv_bfloat16* dst = q ? static_cast<__nv_bfloat16*>(p.cq) + (size_t)t * p.cq_stride + u * 8 : row + (u - nq) * 8;
-        *reinterpret_cast<uint4*>(dst) = o;
+    for (int i0 = 0; i0 < UNITS; i0 += 4) {                 // gains of four units in flight at a time
+        float4 g[4][2];
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int u = min(lane + (i0 + i) * 32, n - 1);
+            const float4* gp = reinterpret_cast<const float4*>(u < nq ? p.q_norm + u * 8 : p.kv_norm + (u - nq) * 8);
+            g[i][0] = gp[0];
+            g[i][1] = gp[1];
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+            const int u = lane + (i0 + i) * 32;
+            const uint4 x = w[i0 + i];
+            const float inv = u < nq ? iq : ik;
+            const float4 g0 = g[i][0], g1 = g[i][1];
+            const uint4 o = make_uint4(pack_bf16(bf16_lo(x.x) * inv * g0.x, bf16_hi(x.x) * inv * g0.y), pack_bf16(bf16_lo(x.y) * inv * g0.z, bf16_hi(x.y) * inv * g0.w),
+                                       pack_bf16(bf16_lo(x.z) * inv * g1.x, bf16_hi(x.z) * inv * g1.y), pack_bf16(bf16_lo(x.w) * inv * g1.z, bf16_hi(x.w) * inv * g1.w));
+            if (u < n) *reinterpret_cast<uint4*>(u < nq ? static_cast<__nv_bfloat16*>(p.cq) + (size_t)t * p.cq_stride + u * 8 : row + (u - nq) * 8) = o;
+        }
     }
 }
 
@@ -606,9 +608,15 @@ template <class K> cudaError_t raise_smem(K kernel, size_t bytes) {
 cudaError_t launch_latent_prep(const LatentPrepParams& p, int rows, bool f32, cudaStream_t st) {
     if (f32) return launch_pdl(latent_prep_kernel<float>, dim3(rows), dim3(128), 0, st, p);
     const bool vec = p.q_rank % 8 == 0 && p.kv_rank % 8 == 0 && p.rot_dim % 8 == 0 && p.down_stride % 8 == 0 && (int)p.cq_stride == p.q_rank &&
-                     p.rot_off == p.kv_rank && (p.q_rank + p.kv_rank) / 8 <= PREP_UNITS * PREP_THREADS &&
+                     p.rot_off == p.kv_rank && (p.q_rank + p.kv_rank) / 8 <= PREP_UNITS * 32 &&
                      !((reinterpret_cast<uintptr_t>(p.down) | reinterpret_cast<uintptr_t>(p.q_norm) | reinterpret_cast<uintptr_t>(p.kv_norm)) & 15);
-    if (vec) return launch_pdl(latent_prep_vec_kernel, dim3(rows), dim3(PREP_THREADS), 0, st, p);
+    if (vec) {
+        const dim3 grid((rows + PREP_WARPS - 1) / PREP_WARPS), block(32 * PREP_WARPS);
+        const int units = (p.q_rank + p.kv_rank) / 8;
+        if (units <= 4 * 32) return launch_pdl(latent_prep_vec_kernel<4>, grid, block, 0, st, p, rows);
+        if (units <= 8 * 32) return launch_pdl(latent_prep_vec_kernel<8>, grid, block, 0, st, p, rows);
+        return launch_pdl(latent_prep_vec_kernel<PREP_UNITS>, grid, block, 0, st, p, rows);
+    }
     return launch_pdl(latent_prep_kernel<__nv_bfloat16>, dim3(rows), dim3(128), 0, st, p);
 }
 

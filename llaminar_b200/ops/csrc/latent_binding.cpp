@@ -162,6 +162,7 @@ void latent_rows(const Tensor& q_lat, const Tensor& q, int64_t q_rot_off, const 
         }
     }
     if (tc) {
+        TORCH_CHECK(q_rot_off % 8 == 0 && q.size(2) % 8 == 0, "the rotated query part must start on a 16-byte boundary");
         want(*status, torch::kInt32, "status");
         check(llm::launch_latent_rows_tc(p, n, n_splits, status->data_ptr<int>(), stream()), "latent_rows_tc");
         if (n_splits > 1) check(llm::launch_latent_merge(p, n, n_splits, group, stream()), "latent_merge");

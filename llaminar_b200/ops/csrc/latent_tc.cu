@@ -40,10 +40,25 @@ LLM_DEVICE float rotated(const __nv_bfloat16* x, int i, const float2* ang, int h
     if (i < 2 * half) return v * ang[i - half].x + __bfloat162float(x[i - half]) * ang[i - half].y;
     return v;
 }
-LLM_DEVICE uint4 rotated8(const __nv_bfloat16* x, int i0, const float2* ang, int half) {
+// values i0 .. i0 + 7 of it, zero from `n` on
+LLM_DEVICE uint4 rotated8(const __nv_bfloat16* x, int i0, int n, const float2* ang, int half) {
     float v[8];
+    if (half % 8 == 0 && i0 + 8 <= 2 * half) {                 // eight whole pairs: vector loads
+        const bool first = i0 < half;
+        const int a0 = first ? i0 : i0 - half;
+        const uint4 own = *reinterpret_cast<const uint4*>(x + i0), other = *reinterpret_cast<const uint4*>(x + (first ? i0 + half : i0 - half));
+        const uint32_t a[4] = {own.x, own.y, own.z, own.w}, b[4] = {other.x, other.y, other.z, other.w};
 #pragma unroll
-    for (int j = 0; j < 8; ++j) v[j] = rotated(x, i0 + j, ang, half);
+        for (int j = 0; j < 4; ++j) {
+            const float4 cs = *reinterpret_cast<const float4*>(ang + a0 + 2 * j);       // cos, sin of two pairs
+            const float s0 = first ? -cs.y : cs.y, s1 = first ? -cs.w : cs.w;
+            v[2 * j] = bf16_lo(a[j]) * cs.x + bf16_lo(b[j]) * s0;
+            v[2 * j + 1] = bf16_hi(a[j]) * cs.z + bf16_hi(b[j]) * s1;
+        }
+    } else {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) v[j] = i0 + j < n ? rotated(x, i0 + j, ang, half) : 0.f;
+    }
     return make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
 }
 
@@ -126,7 +141,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS, 1) latent_chunk_tc_kernel(const
             uint4 v = make_uint4(0, 0, 0, 0);
             if (r < rows) {
                 const size_t t = (size_t)sq.q_start + q0 + r;
-                v = rotated8(p.q + t * p.q_row + (size_t)head * p.q_head + p.dim, u * 8, p.angles + t * p.half, p.half);
+                v = rotated8(p.q + t * p.q_row + (size_t)head * p.q_head + p.dim, u * 8, p.rot, p.angles + t * p.half, p.half);
             }
             st_shared_v4(atom_addr(sQ + (na + (u >> 3)) * ATOM, r, u & 7), v);
         }
@@ -332,7 +347,7 @@ __global__ void __launch_bounds__(CHUNK_THREADS, 1) latent_chunk_tc_kernel(const
 // ------------------------------------------------------------------------------------------------------------------------
 constexpr int ROWS_THREADS = 192, PAGE = 64, MAX_SLOTS = 8;
 constexpr float RESCALE_STEP = 8.f;
-enum RBar { R_FULL = 0, R_EMPTY = R_FULL + MAX_SLOTS, ROT_FULL = R_EMPTY + MAX_SLOTS, ROT_EMPTY, RS_FULL, RP_FULL, RO_DONE, RQ_FULL, R_MEET, R_BARS };
+enum RBar { R_FULL = 0, R_EMPTY = R_FULL + MAX_SLOTS, ROT_FULL = R_EMPTY + MAX_SLOTS, ROT_EMPTY, RS_FULL, RP_FULL, RO_DONE, RQ_FULL, RQ_LAT, R_MEET, R_BARS };
 
 struct RowsSmem { int n_blocks, n_slots; size_t bytes; };
 static __host__ __device__ inline RowsSmem rows_layout(int n, int latent) {
@@ -387,7 +402,8 @@ LLM_DEVICE uint64_t smem_desc_mn_sw128(uint32_t addr, uint32_t lead) {
 }
 
 template <int N>
-__global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const LatentRowsParams p, int* status) {
+__global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_q,
+                                                                        const LatentRowsParams p, int* status) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t s_bars[R_BARS];
     __shared__ uint32_t s_tmem;
@@ -431,24 +447,14 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     if (nt == 0) {
         if (tid < N) *reinterpret_cast<float2*>(p.part_ml + (part + tid) * 2) = make_float2(-INFINITY, 0.f);
     } else if (warp < 4) {
-        // query operand: N rows (heads) of [latent | rotated part, zero padded to one atom]
-        const int ul = p.rot_off / 8, ua = NA * 8;
-        for (int i = tid; i < N * ua; i += 128) {
-            const int r = i / ua, u = i % ua, h = hg * N + r;
+        // query operand, N rows (heads): the latent part comes by TMA, the rotated part (one atom, zero padded) is turned here
+        for (int i = tid; i < N * 8; i += 128) {
+            const int r = i >> 3, u = i & 7, h = hg * N + r;
             uint4 v = make_uint4(0, 0, 0, 0);
-            if (h < p.n_heads) {
-                if (u < ul) {
-                    v = *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.q_lat) + (size_t)z * p.ql_row + (size_t)h * p.ql_head + u * 8);
-                } else if ((u - ul) * 8 < p.rot_dim) {
-                    const __nv_bfloat16* qr = static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off;
-                    const float2* ang = p.angles + (size_t)t * p.half;
-                    float x[8];
-#pragma unroll
-                    for (int j = 0; j < 8; ++j) { const int c = (u - ul) * 8 + j; x[j] = c < p.rot_dim ? rotated(qr, c, ang, p.half) : 0.f; }
-                    v = make_uint4(pack_bf16(x[0], x[1]), pack_bf16(x[2], x[3]), pack_bf16(x[4], x[5]), pack_bf16(x[6], x[7]));
-                }
-            }
-            st_shared_v4(atom_addr(sQ + (u >> 3) * N * 128, r, u & 7), v);
+            if (h < p.n_heads && u * 8 < p.rot_dim)
+                v = rotated8(static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off, u * 8, p.rot_dim,
+                             p.angles + (size_t)t * p.half, p.half);
+            st_shared_v4(atom_addr(sQ + 2 * NB * N * 128, r, u), v);
         }
         fence_proxy_async();
         __syncwarp();
@@ -566,6 +572,8 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
         if (elect_one()) {
             bool ok = true;
             int it = 0;
+            mbar_arrive_expect_tx(bar(RQ_LAT), 2 * NB * N * 128);
+            for (int a = 0; a < 2 * NB; ++a) tma_load_3d(sQ + a * N * 128, &map_q, a * 64, z, hg * N, bar(RQ_LAT));      // heads past the last: zeros
             for (int j = 0; j < nt && ok; ++j) {
                 const int pg = page0 + 2 * (j0 + j);
                 // a page past the end repeats the last one (its keys are masked)
@@ -591,7 +599,7 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     } else if (elect_one()) {
         const uint32_t idesc_s = instr_desc(N), idesc_o = instr_desc(N) | (1u << 15);       // bit 15: A is MN-major
         const int rot_steps = (p.width - p.rot_off) / 16;
-        bool ok = mbar_wait(bar(RQ_FULL), 0, abort_flag);
+        bool ok = mbar_wait(bar(RQ_LAT), 0, abort_flag) && mbar_wait(bar(RQ_FULL), 0, abort_flag);
         for (int j = 0; j < nt && ok; ++j) {
             for (int b = 0; b < NB && ok; ++b) {
                 const int it = j * NB + b, slot = it % NS;
@@ -694,11 +702,20 @@ cudaError_t launch_latent_rows_tc(const LatentRowsParams& p, int rows, int n_spl
     if (!n || rows > 65535 || p.ql_row % 8 || p.ql_head % 8) return cudaErrorInvalidValue;
     CUtensorMap m;
     if (!make_map(&m, p.kv, p.width, (uint64_t)p.n_pages * PAGE, p.width, PAGE)) return cudaErrorInvalidValue;
+    CUtensorMap mq;                                          // [head][row][latent], boxes of 64 values x 1 row x n heads
+    {
+        const cuuint64_t dims[3] = {(cuuint64_t)p.rot_off, (cuuint64_t)rows, (cuuint64_t)p.n_heads}, strides[2] = {p.ql_row * 2, p.ql_head * 2};
+        const cuuint32_t box[3] = {64, 1, (cuuint32_t)n}, estr[3] = {1, 1, 1};
+        if (!encode_fn() || (reinterpret_cast<uintptr_t>(p.q_lat) & 15) ||
+            encode_fn()(&mq, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(p.q_lat), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
+                        CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
+            return cudaErrorInvalidValue;
+    }
     const size_t smem = rows_layout(n, p.rot_off).bytes;
     const dim3 grid((p.n_heads + n - 1) / n, n_splits, rows);
     auto go = [&](auto kernel) {
         cudaError_t e = raise_smem(kernel, smem);
-        return e != cudaSuccess ? e : launch_pdl(kernel, grid, dim3(ROWS_THREADS), smem, st, m, p, status);
+        return e != cudaSuccess ? e : launch_pdl(kernel, grid, dim3(ROWS_THREADS), smem, st, m, mq, p, status);
     };
     return n == 16 ? go(latent_rows_tc_kernel<16>) : go(latent_rows_tc_kernel<32>);
 }

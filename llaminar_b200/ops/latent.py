@@ -10,9 +10,7 @@ import torch
 from . import _count
 from . import build as _build
 
-GEMV_MAX_ROWS = 4              # rows the kernel takes
-GEMV_ROWS = 2                  # rows up to which it is preferred to cuBLAS
-_GEMV_SMEM = 200 * 1024
+GEMV_MAX_ROWS = 8
 _ready = False
 
 
@@ -109,12 +107,12 @@ def chunk_tc_fits(dim: int, rot: int, vdim: int) -> bool:
 def gemv_fits(w: torch.Tensor, x: torch.Tensor) -> bool:
     """Whether `gemv_dense` takes this product: few bf16 rows, 16-byte rows."""
     k = w.shape[-1]
-    return (w.dtype == torch.bfloat16 and x.shape[-2] <= GEMV_ROWS and k % 8 == 0 and x.stride(-2) % 8 == 0 and w.stride(-2) % 8 == 0
-            and x.shape[-2] * k * 2 <= _GEMV_SMEM and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
+    return (w.dtype == torch.bfloat16 and x.shape[-2] <= GEMV_MAX_ROWS and k % 8 == 0 and x.stride(-2) % 8 == 0 and w.stride(-2) % 8 == 0
+            and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
 
 
 def gemv_dense(w, x, out, gelu: bool = False) -> None:
-    """out[z] = x[z] @ w[z]^T for at most four bf16 rows; ``gelu``: w stacks gate and up, out = gelu_tanh(gate) * up."""
+    """out[z] = x[z] @ w[z]^T for at most eight bf16 rows; ``gelu``: w stacks gate and up, out = gelu_tanh(gate) * up."""
     ext().gemv_dense(w, x, out, gelu)
     _count()
 
