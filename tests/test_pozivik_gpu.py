@@ -1,0 +1,111 @@
+"""Pozivik on the GPU against the plain oracle, in bf16 and in 32-bit mode, with and without the tcgen05 attention kernels."""
+import pytest
+import torch
+
+from llaminar_b200 import ops
+from llaminar_b200.engine.sampling import SamplingParams
+
+from . import pozivik_cases as cases
+from . import pozivik_oracle as oracle
+
+pytestmark = pytest.mark.gpu
+BF, F32 = torch.bfloat16, torch.float32
+both = pytest.mark.parametrize("dtype", [BF, F32])
+
+
+@both
+@pytest.mark.parametrize("name", [*cases.MODELS, "wide"])
+def test_whole_prompt(name, dtype):
+    cases.whole_prompt(name, "cuda", dtype)
+
+
+@both
+@pytest.mark.parametrize("name", ["mixed", "loop_middle", "wide"])
+def test_portions_and_decoding(name, dtype):
+    cases.portions_and_decoding(name, "cuda", dtype)
+
+
+@both
+@pytest.mark.parametrize("name", ["loop_once", "wide"])
+def test_token_by_token(name, dtype):
+    cases.token_by_token(name, "cuda", dtype)
+
+
+@both
+@pytest.mark.parametrize("name", ["mixed", "loop_end", "wide"])
+def test_mixed_batches(name, dtype):
+    cases.mixed_batches(name, "cuda", dtype)
+
+
+@both
+@pytest.mark.parametrize("check", ["far_keys_and_window_edges", "sinks_matter", "long_decoding", "greedy_generation", "prefix_cache_reuse", "preemption"])
+def test_engine(check, dtype):
+    getattr(cases, check)("cuda", dtype)
+
+
+@pytest.mark.parametrize("rows_tc,chunk_tc", [(True, False), (False, True), (False, False)])
+def test_attention_forms_agree(rows_tc, chunk_tc):
+    m = cases.model("wide", seed=5)
+    t = cases.tokens(330, 6)
+    want = oracle.forward(t, m)
+    eng = cases.engine(m, "cuda", BF)
+    eng.model.stack.rows_tc, eng.model.stack.chunk_tc = rows_tc, chunk_tc
+    cases.assert_close(cases.feed_all(eng, t, [200, 3, 90, 1]), want, BF)
+    eng.check_health()
+
+
+def test_long_context_many_tiles():
+    """Windows of several key tiles and none at all, over a few thousand tokens; the decode step splits the keys."""
+    E = oracle.layer_entry
+    layers = [E(heads=18, dim=64, rot_dim=32, vdim=64, kv_rank=128, q_rank=64, window=1500, ff=None), E(heads=4, window=700, ff=None),
+              E(heads=16, dim=32, rot_dim=16, vdim=32, kv_rank=256, q_rank=40, window=5000, ff=None)]
+    m = oracle.random_model(3, layers=layers, width=64)
+    t = cases.tokens(2100, 7)
+    want = oracle.forward(t, m, dt=torch.float32)
+    eng = cases.engine(m, "cuda", BF, max_context=2176, kv_pages=40, max_prefill_tokens=2176)
+    for cuts in ([2085, 1], [1000, 7, 1000, 78, 1]):
+        cases.assert_close(cases.feed_all(eng, t, cuts), want, BF, cuts)
+
+
+def test_no_window():
+    E = oracle.layer_entry
+    m = oracle.random_model(4, layers=[E(heads=3, window=None), E(heads=17, dim=64, rot_dim=16, vdim=64, kv_rank=128, window=None)], width=48)
+    t = cases.tokens(400, 8)
+    want = oracle.forward(t, m)
+    for dtype in (BF, F32):
+        eng = cases.engine(m, "cuda", dtype)
+        cases.assert_close(cases.feed_all(eng, t, [129, 250, 1]), want, dtype)
+
+
+def test_captured_and_eager_decode_agree_and_launch_own_kernels():
+    m = cases.model("wide", seed=2, gain=1.3)
+    prompts = [cases.tokens(n, n) for n in (5, 100, 64)]
+    sp = SamplingParams(temperature=0.0, max_tokens=20, ignore_eos=True)
+    a, b = cases.engine(m, "cuda", BF), cases.engine(m, "cuda", BF, use_graphs=False)
+    n0 = ops.launch_count()
+    assert a.generate(prompts, sp) == b.generate(prompts, sp)
+    assert a.stats["graph_replays"] > 0 and ops.launch_count() > n0
+    sampled = SamplingParams(temperature=0.9, top_k=30, top_p=0.95, seed=5, max_tokens=12, ignore_eos=True)
+    assert a.generate(prompts, sampled) == b.generate(prompts, sampled)
+
+
+def test_logits_do_not_depend_on_the_batch():
+    """Steps of one to four sequences of different lengths: a sequence's logits stay within rounding of its own alone."""
+    m = cases.model("loop_middle", seed=3)
+    eng = cases.engine(m, "cuda", BF)
+    t = [cases.tokens(n, n) for n in (30, 150, 64, 129)]
+    alone = [cases.feed_all(eng, x, [len(x) - 4, 1]) for x in t]
+    seqs = [eng.open_sequence() for _ in t]
+    eng.feed([(s, x[:-4], []) for s, x in zip(seqs, t)])
+    for k in range(-4, 0):
+        got = eng.feed([(s, [x[k]], [0]) for s, x in zip(seqs, t)])
+        cases.assert_close(got, torch.stack([a[k] for a in alone]).cpu(), BF)
+
+
+def test_synthetic_shape_through_the_engine():
+    from llaminar_b200.engine.engine import LLMEngine
+    from llaminar_b200.models.config import SHAPES
+    from llaminar_b200.models.synth import synthesize
+    eng = LLMEngine(synthesize(SHAPES["tiny-pozivik"], "BF16", seed=0), device="cuda", max_batch=8, max_context=512)
+    outs = eng.generate([cases.tokens(n, n, 1024) for n in (300, 7, 64, 65, 128, 20, 33, 90)], SamplingParams(temperature=0.0, max_tokens=16, ignore_eos=True))
+    assert all(len(o) == 16 for o in outs)
