@@ -337,28 +337,29 @@ __global__ void __launch_bounds__(CHUNK_THREADS, 1) latent_chunk_tc_kernel(const
 }
 
 // ------------------------------------------------------------------------------------------------------------------------
-// single rows: N heads of one row per CTA, keys in tiles of 128 (two pages)
-//   S^T = C Q^T       M = 128 keys, N heads, K = latent + rotated part: the cache rows are the A operand as they lie
-//   softmax           one thread per key (= TMEM lane), N columns; the maxima over keys are reduced across lanes
-//   O^T += C^T P^T    M = 128 latent values, N heads, K = 128 keys: the same rows again, read as an MN-major A operand
+// single rows: N heads of one row per CTA, keys in tiles of 64 (one page)
+//   S^T = C Q^T       M = 64 keys, N heads, K = latent + rotated part: the cache rows are the A operand as they lie; two accumulators
+//   softmax           one thread per key (M = 64 fills TMEM lanes 0-15 of each warp's quarter), N columns; the maxima over keys
+//                     are reduced across lanes
+//   O^T += C^T P^T    M = 128 latent values, N heads, K = 64 keys: the same rows again, read as an MN-major A operand
 // One copy of the cache rows therefore serves both products, and both fill the M dimension whatever the number of heads.
 // The accumulator stays in TMEM and is rescaled only when a running maximum rises by more than 2^RESCALE_STEP.
 // Warps 0-3 softmax, 4 TMA, 5 TMEM allocation and MMA issue.
 // ------------------------------------------------------------------------------------------------------------------------
-constexpr int ROWS_THREADS = 192, PAGE = 64, MAX_SLOTS = 8;
+constexpr int ROWS_THREADS = 192, PAGE = 64, MAX_SLOTS = 12, HALF = 64 * 128;      // HALF: 64 rows x 64 bf16
 constexpr float RESCALE_STEP = 8.f;
-enum RBar { R_FULL = 0, R_EMPTY = R_FULL + MAX_SLOTS, ROT_FULL = R_EMPTY + MAX_SLOTS, ROT_EMPTY, RS_FULL, RP_FULL, RO_DONE, RQ_FULL, RQ_LAT, R_MEET, R_BARS };
+enum RBar { R_FULL = 0, R_EMPTY = R_FULL + MAX_SLOTS, ROT_FULL = R_EMPTY + MAX_SLOTS, ROT_EMPTY = ROT_FULL + 2, RS_FULL = ROT_EMPTY + 2, RP_FULL = RS_FULL + 2, RO_DONE, RQ_FULL, RQ_LAT, R_MEET, R_BARS };
 
 struct RowsSmem { int n_blocks, n_slots; size_t bytes; };
 static __host__ __device__ inline RowsSmem rows_layout(int n, int latent) {
     RowsSmem r;
     r.n_blocks = latent / 128;
-    const size_t fixed = (size_t)(2 * r.n_blocks + 1 + 2) * n * 128 + ATOM + 1024;
-    r.n_slots = (int)((226 * 1024 + 512 - fixed) / (2 * ATOM));
-    const int want = 2 * r.n_blocks;
+    const size_t fixed = (size_t)(2 * r.n_blocks + 1 + 1) * n * 128 + 2 * HALF + 1024;        // queries, P, rotated parts
+    r.n_slots = (int)((226 * 1024 + 512 - fixed) / (2 * HALF));
+    const int want = 3 * r.n_blocks;
     if (r.n_slots > want) r.n_slots = want;
     if (r.n_slots > MAX_SLOTS) r.n_slots = MAX_SLOTS;
-    r.bytes = fixed + (size_t)r.n_slots * 2 * ATOM;
+    r.bytes = fixed + (size_t)r.n_slots * 2 * HALF;
     return r;
 }
 
@@ -408,13 +409,13 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     __shared__ __align__(8) uint64_t s_bars[R_BARS];
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort[2];
-    __shared__ float s_red[4][32];                 // per warp: column maxima (and sums at the end)
+    __shared__ float s_red[2][4][32];              // [tile parity] per warp: column maxima (and sums at the end)
     __shared__ __align__(16) float s_head[4][32];  // per warp: running maximum (or factor) of every head, for broadcast reads
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const RowsSmem lay = rows_layout(N, p.rot_off);
     const int NB = lay.n_blocks, NS = lay.n_slots, NA = 2 * NB + 1;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-    const uint32_t sQ = base, sP = sQ + NA * N * 128, sR = sP + 2 * N * 128, sC = sR + ATOM;
+    const uint32_t sQ = base, sP = sQ + NA * N * 128, sR = sP + N * 128, sC = sR + 2 * HALF;
     const uint32_t bars = smem_u32(s_bars);
     auto bar = [&](int i) { return bars + i * 8; };
     pdl_trigger();
@@ -431,7 +432,7 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t tmem = s_tmem, t_o = tmem + 32;             // S^T in columns [0, N), O^T blocks behind
+    const uint32_t tmem = s_tmem, t_o = tmem + 64;             // S^T in columns [0, N) and [32, 32 + N), O^T blocks behind
     volatile int* abort_flag = s_abort;
     pdl_wait();
 
@@ -440,7 +441,7 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     const int pos = p.positions[t], lo = first_key(pos, p.window);
     const int* btab = p.block_table + (size_t)LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs) * p.max_pages;
     const int page0 = lo / PAGE, page_last = pos / PAGE;
-    const int n_tiles = (page_last - page0) / 2 + 1, per = (n_tiles + gridDim.y - 1) / gridDim.y;
+    const int n_tiles = page_last - page0 + 1, per = (n_tiles + gridDim.y - 1) / gridDim.y;
     const int j0 = split * per, nt = max(0, min(n_tiles, j0 + per) - j0);
     const size_t part = (((size_t)z * gridDim.x + hg) * gridDim.y + split) * N;
 
@@ -461,6 +462,7 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
         mbar_arrive_if(bar(RQ_FULL), lane == 0);
 
         const uint32_t t_lane = (uint32_t)(warp * 32) << 16;
+        const int row = warp * 16 + lane;           // key row of the tile (lanes 0-15)
         const float sl2 = p.scale * LOG2E;
         float l[N], m = -INFINITY;                  // l: this key lane's share of every head's sum; m: lane c holds head c's maximum
 #pragma unroll
@@ -485,21 +487,22 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             }
         };
         for (int j = 0; j < nt && ok; ++j) {
-            ok = mbar_wait_warp(bar(RS_FULL), j & 1, abort_flag);
+            ok = mbar_wait_warp(bar(RS_FULL + (j & 1)), (j >> 1) & 1, abort_flag);
             if (!ok) break;
             tc_fence_after();
             uint32_t raw[N];
-            tmem_ld_n<N>(tmem + t_lane, raw);
-            const int key = (page0 + 2 * (j0 + j)) * PAGE + tid;
-            const bool seen = key >= lo && key <= pos;
+            tmem_ld_n<N>(tmem + (j & 1) * 32 + t_lane, raw);
+            const int key = (page0 + j0 + j) * PAGE + row;
+            const bool seen = lane < 16 && key >= lo && key <= pos;
             float s[N], red[N];
 #pragma unroll
             for (int c = 0; c < N; ++c) { s[c] = seen ? __uint_as_float(raw[c]) * sl2 : -INFINITY; red[c] = s[c]; }
-            // (the previous tile's reads of s_red precede its P_FULL arrivals, without which this tile's S cannot be complete)
-            s_red[warp][lane] = reduce_columns<N, false>(red, lane);
+            // (the reads of s_red two tiles ago precede that tile's P_FULL arrivals, without which this tile's S is not issued)
+            float (&red4)[4][32] = s_red[j & 1];
+            red4[warp][lane] = reduce_columns<N, false>(red, lane);
             ok = meet();
             if (!ok) break;
-            const float mt = fmaxf(fmaxf(s_red[0][lane], s_red[1][lane]), fmaxf(s_red[2][lane], s_red[3][lane]));
+            const float mt = fmaxf(fmaxf(red4[0][lane], red4[1][lane]), fmaxf(red4[2][lane], red4[3][lane]));
             const bool raise = mt > m + RESCALE_STEP;           // also the first tile, where m is -inf
             const float m_old = m;
             if (raise) m = mt;
@@ -523,13 +526,13 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             }
             float mh[N];
             broadcast(m, mh);
-            const uint32_t dst = sP + (tid >> 6) * N * 128 + (tid & 7) * 2;
-            const int unit = (tid & 63) >> 3;
+            const uint32_t dst = sP + (row & 7) * 2;
+            const int unit = (row & 63) >> 3;
 #pragma unroll
             for (int c = 0; c < N; ++c) {
-                const float pr = ex2(s[c] - mh[c]);
+                const float pr = ex2(s[c] - mh[c]);         // 0 on the idle lanes
                 l[c] += pr;
-                asm volatile("st.shared.b16 [%0], %1;" ::"r"(dst + c * 128 + (((unit ^ c) & 7) << 4)), "h"(__bfloat16_as_ushort(__float2bfloat16(pr))) : "memory");
+                if (lane < 16) asm volatile("st.shared.b16 [%0], %1;" ::"r"(dst + c * 128 + (((unit ^ c) & 7) << 4)), "h"(__bfloat16_as_ushort(__float2bfloat16(pr))) : "memory");
             }
             tc_fence_before();
             fence_proxy_async();
@@ -539,12 +542,12 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
         // the last products are complete, so every warp has arrived with its P and is done with the maxima in s_red
         ok = ok && mbar_wait_warp(bar(RO_DONE), (nt - 1) & 1, abort_flag);
         if (ok) {
-            s_red[warp][lane] = reduce_columns<N, true>(l, lane);
+            s_red[0][warp][lane] = reduce_columns<N, true>(l, lane);
             ok = meet();
         }
         if (ok) {
             tc_fence_after();
-            float lt = s_red[0][lane] + s_red[1][lane] + s_red[2][lane] + s_red[3][lane];       // lane c: head c
+            float lt = s_red[0][0][lane] + s_red[0][1][lane] + s_red[0][2][lane] + s_red[0][3][lane];       // lane c: head c
             uint32_t raw[N];
             if (gridDim.y == 1) {
                 const int h0 = hg * N;
@@ -575,61 +578,81 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             mbar_arrive_expect_tx(bar(RQ_LAT), 2 * NB * N * 128);
             for (int a = 0; a < 2 * NB; ++a) tma_load_3d(sQ + a * N * 128, &map_q, a * 64, z, hg * N, bar(RQ_LAT));      // heads past the last: zeros
             for (int j = 0; j < nt && ok; ++j) {
-                const int pg = page0 + 2 * (j0 + j);
-                // a page past the end repeats the last one (its keys are masked)
-                const int r0 = LLM_CHECK_INDEX(btab[pg], p.n_pages) * PAGE, r1 = LLM_CHECK_INDEX(btab[min(pg + 1, page_last)], p.n_pages) * PAGE;
-                auto load = [&](uint32_t dst, int col, uint32_t full) {
-                    tma_load_2d(dst, &map_kv, col, r0, full);
-                    tma_load_2d(dst + ATOM / 2, &map_kv, col, r1, full);
-                };
-                ok = mbar_wait(bar(ROT_EMPTY), (j & 1) ^ 1, abort_flag);
+                const int r0 = LLM_CHECK_INDEX(btab[page0 + j0 + j], p.n_pages) * PAGE, b2 = j & 1;
+                ok = mbar_wait(bar(ROT_EMPTY + b2), ((j >> 1) & 1) ^ 1, abort_flag);
                 if (!ok) break;
-                mbar_arrive_expect_tx(bar(ROT_FULL), ATOM);
-                load(sR, p.rot_off, bar(ROT_FULL));
+                mbar_arrive_expect_tx(bar(ROT_FULL + b2), HALF);
+                tma_load_2d(sR + b2 * HALF, &map_kv, p.rot_off, r0, bar(ROT_FULL + b2));
                 for (int b = 0; b < NB; ++b, ++it) {
                     const int slot = it % NS;
                     ok = mbar_wait(bar(R_EMPTY + slot), ((it / NS) & 1) ^ 1, abort_flag);
                     if (!ok) break;
-                    mbar_arrive_expect_tx(bar(R_FULL + slot), 2 * ATOM);
-                    load(sC + slot * 2 * ATOM, b * 128, bar(R_FULL + slot));
-                    load(sC + slot * 2 * ATOM + ATOM, b * 128 + 64, bar(R_FULL + slot));
+                    mbar_arrive_expect_tx(bar(R_FULL + slot), 2 * HALF);
+                    tma_load_2d(sC + slot * 2 * HALF, &map_kv, b * 128, r0, bar(R_FULL + slot));
+                    tma_load_2d(sC + slot * 2 * HALF + HALF, &map_kv, b * 128 + 64, r0, bar(R_FULL + slot));
                 }
             }
         }
-    } else if (elect_one()) {
-        const uint32_t idesc_s = instr_desc(N), idesc_o = instr_desc(N) | (1u << 15);       // bit 15: A is MN-major
-        const int rot_steps = (p.width - p.rot_off) / 16;
-        bool ok = mbar_wait(bar(RQ_LAT), 0, abort_flag) && mbar_wait(bar(RQ_FULL), 0, abort_flag);
-        for (int j = 0; j < nt && ok; ++j) {
-            for (int b = 0; b < NB && ok; ++b) {
-                const int it = j * NB + b, slot = it % NS;
-                ok = mbar_wait(bar(R_FULL + slot), (it / NS) & 1, abort_flag);
-                if (!ok) break;
-                tc_fence_after();
-#pragma unroll
-                for (int ks = 0; ks < 8; ++ks)
-                    mma_f16(tmem, smem_desc_sw128(sC + slot * 2 * ATOM + (ks >> 2) * ATOM) + 2 * (ks & 3),
-                            smem_desc_sw128(sQ + (2 * b + (ks >> 2)) * N * 128) + 2 * (ks & 3), idesc_s, b > 0 || ks > 0 ? 1u : 0u);
-            }
-            ok = ok && mbar_wait(bar(ROT_FULL), j & 1, abort_flag);
-            if (!ok) break;
-            tc_fence_after();
-            for (int ks = 0; ks < rot_steps; ++ks)
-                mma_f16(tmem, smem_desc_sw128(sR) + 2 * ks, smem_desc_sw128(sQ + 2 * NB * N * 128) + 2 * ks, idesc_s, 1u);
-            mma_commit(bar(RS_FULL));
-            mma_commit(bar(ROT_EMPTY));
-            ok = mbar_wait(bar(RP_FULL), j & 1, abort_flag);
-            if (!ok) break;
-            tc_fence_after();
+    } else {
+        // The whole warp walks the pipeline and elects a lane only around each batch of MMAs: loop counters, slots and
+        // descriptors then stay warp-uniform, which the issue rate depends on.
+        constexpr uint32_t M_MASK = 31u << 24;
+        constexpr uint32_t idesc_s = (instr_desc(N) & ~M_MASK) | (64u >> 4 << 24), idesc_o = instr_desc(N) | (1u << 15);   // bit 15: A is MN-major
+        const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
+        const int n = __shfl_sync(0xffffffffu, nt, 0), rot_steps = (p.width - p.rot_off) / 16;
+        const uint64_t c_desc = smem_desc_sw128(sC), cm_desc = smem_desc_mn_sw128(sC, HALF), q_desc = smem_desc_sw128(sQ), p_desc = smem_desc_sw128(sP),
+                       r_desc = smem_desc_sw128(sR);
+        bool ok = mbar_wait_warp(bar(RQ_LAT), 0, abort_flag) && mbar_wait_warp(bar(RQ_FULL), 0, abort_flag);
+        int s_slot = 0, s_phase = 0, o_slot = 0;
+        // (the softmax has read this accumulator: P of two tiles ago has been waited for)
+        auto issue_s = [&](int j) {
+            const int b2 = j & 1;
+            const uint32_t d = tm + b2 * 32;
             for (int b = 0; b < NB; ++b) {
-                const int slot = (j * NB + b) % NS;
+                ok = mbar_wait_warp(bar(R_FULL + s_slot), s_phase, abort_flag);
+                if (!ok) return;
+                tc_fence_after();
+                const uint64_t a = c_desc + (uint32_t)(s_slot * (2 * HALF / 16)), q = q_desc + (uint32_t)(b * (2 * N * 128 / 16));
+                const uint32_t first = b > 0 ? 1u : 0u;
+                if (elect_one()) {
 #pragma unroll
-                for (int ks = 0; ks < 8; ++ks)              // 16 keys: two groups of eight rows
-                    mma_f16(t_o + b * N, smem_desc_mn_sw128(sC + slot * 2 * ATOM + ks * 2048, ATOM), smem_desc_sw128(sP + (ks >> 2) * N * 128) + 2 * (ks & 3),
-                            idesc_o, j > 0 || ks > 0 ? 1u : 0u);
-                mma_commit(bar(R_EMPTY + slot));
+                    for (int ks = 0; ks < 8; ++ks)
+                        mma_f16(d, a + (ks >> 2) * (HALF / 16) + 2 * (ks & 3), q + (ks >> 2) * (N * 128 / 16) + 2 * (ks & 3), idesc_s, ks > 0 ? 1u : first);
+                }
+                __syncwarp();
+                if (++s_slot == NS) { s_slot = 0; s_phase ^= 1; }
             }
-            mma_commit(bar(RO_DONE));
+            ok = mbar_wait_warp(bar(ROT_FULL + b2), (j >> 1) & 1, abort_flag);
+            if (!ok) return;
+            tc_fence_after();
+            const uint64_t a = r_desc + (uint32_t)(b2 * (HALF / 16)), q = q_desc + (uint32_t)(2 * NB * (N * 128 / 16));
+            if (elect_one()) {
+                for (int ks = 0; ks < rot_steps; ++ks) mma_f16(d, a + 2 * ks, q + 2 * ks, idesc_s, 1u);
+                mma_commit(bar(RS_FULL + b2));
+                mma_commit(bar(ROT_EMPTY + b2));
+            }
+            __syncwarp();
+        };
+        if (ok) issue_s(0);
+        for (int j = 0; j < n && ok; ++j) {
+            if (j + 1 < n) issue_s(j + 1);
+            ok = ok && mbar_wait_warp(bar(RP_FULL), j & 1, abort_flag);
+            if (!ok) break;
+            tc_fence_after();
+            const uint32_t more = j > 0 ? 1u : 0u;
+            for (int b = 0; b < NB; ++b) {
+                const uint64_t a = cm_desc + (uint32_t)(o_slot * (2 * HALF / 16));
+                const uint32_t d = tm + 64 + b * N;
+                if (elect_one()) {
+#pragma unroll
+                    for (int ks = 0; ks < 4; ++ks)              // 16 keys: two groups of eight rows
+                        mma_f16(d, a + ks * (2048 / 16), p_desc + 2 * ks, idesc_o, ks > 0 ? 1u : more);
+                    mma_commit(bar(R_EMPTY + o_slot));
+                    if (b == NB - 1) mma_commit(bar(RO_DONE));
+                }
+                __syncwarp();
+                if (++o_slot == NS) o_slot = 0;
+            }
         }
     }
     tc_fence_before();
@@ -693,7 +716,7 @@ cudaError_t launch_latent_chunk_tc(const LatentChunkParams& p, int n_keys, int n
 int latent_rows_tc_heads(int width, int rot_off, int rot_dim, int n_heads) {
     if (rot_off % 128 || rot_off < 128 || rot_off > 512 || width % 16 || width - rot_off > 64 || width <= rot_off || rot_dim <= 0) return 0;
     const int n = n_heads <= 16 ? 16 : 32;
-    return ltc::rows_layout(n, rot_off).n_slots >= rot_off / 128 ? n : 0;
+    return ltc::rows_layout(n, rot_off).n_slots >= 2 * (rot_off / 128) ? n : 0;        // two tiles are in use at a time
 }
 
 cudaError_t launch_latent_rows_tc(const LatentRowsParams& p, int rows, int n_splits, int* status, cudaStream_t st) {

@@ -66,7 +66,7 @@ def rows_splits(n_rows: int, n_heads: int, group: int, tensor_core: bool, max_ke
     if group == 0:
         return 1
     groups = -(-n_heads // group)
-    tiles = max_keys // (128 if tensor_core else 32) + 1            # a window that starts inside a tile touches one more
+    tiles = max_keys // (64 if tensor_core else 32) + 1             # a window that starts inside a tile touches one more
     want = max(1, min(tiles, (148 if tensor_core else 296) // max(1, n_rows * groups), 64))
     want = max(1, min(want, capacity // max(1, n_rows * groups * group * latent)))
     per = -(-tiles // want)
