@@ -338,47 +338,24 @@ __global__ void __launch_bounds__(CHUNK_THREADS, 1) latent_chunk_tc_kernel(const
 
 // ------------------------------------------------------------------------------------------------------------------------
 // single rows: N heads of one row per CTA, keys in tiles of 64 (one page)
-//   S^T = C Q^T       M = 64 keys, N heads, K = latent + rotated part: the cache rows are the A operand as they lie; two accumulators
-//   softmax           one thread per key (M = 64 fills TMEM lanes 0-15 of each warp's quarter), N columns; the maxima over keys
-//                     are reduced across lanes
+//   S = Q C^T         M = 128, N = 64 keys, K = latent + rotated part.  Q is the A operand in TMEM, its N rows (heads) repeated in
+//                     every warp's lanes: each softmax warp finds all heads in its own lanes and takes 16 of the keys.  The cache
+//                     rows are the B operand as they lie.
+//   softmax           one thread per head and 16 keys: maxima and sums need no shuffles, only an exchange between the four warps
 //   O^T += C^T P^T    M = 128 latent values, N heads, K = 64 keys: the same rows again, read as an MN-major A operand
-// One copy of the cache rows therefore serves both products, and both fill the M dimension whatever the number of heads.
-// The accumulator stays in TMEM and is rescaled only when a running maximum rises by more than 2^RESCALE_STEP.
+// One copy of the cache rows serves both products.  The accumulator O^T stays in TMEM and is rescaled only when a running
+// maximum rises by more than 2^RESCALE_STEP.
 // Warps 0-3 softmax, 4 TMA, 5 TMEM allocation and MMA issue.
 // ------------------------------------------------------------------------------------------------------------------------
-constexpr int ROWS_THREADS = 192, PAGE = 64, MAX_SLOTS = 12, HALF = 64 * 128;      // HALF: 64 rows x 64 bf16
+constexpr int ROWS_THREADS = 192, PAGE = 64, SLOTS = 3, HALF = 64 * 128;      // HALF: an atom of 64 rows x 64 bf16
 constexpr float RESCALE_STEP = 8.f;
-enum RBar { R_FULL = 0, R_EMPTY = R_FULL + MAX_SLOTS, ROT_FULL = R_EMPTY + MAX_SLOTS, ROT_EMPTY = ROT_FULL + 2, RS_FULL = ROT_EMPTY + 2, RP_FULL = RS_FULL + 2, RO_DONE, RQ_FULL, RQ_LAT, R_MEET, R_BARS };
+enum RBar { R_FULL = 0, R_EMPTY = R_FULL + SLOTS, RS_FULL = R_EMPTY + SLOTS, RS_EMPTY, RP_FULL, RO_DONE, RQ_FULL, RQ_LAT, R_MEET, R_BARS };
 
-struct RowsSmem { int n_blocks, n_slots; size_t bytes; };
-static __host__ __device__ inline RowsSmem rows_layout(int n, int latent) {
-    RowsSmem r;
-    r.n_blocks = latent / 128;
-    const size_t fixed = (size_t)(2 * r.n_blocks + 1 + 1) * n * 128 + 2 * HALF + 1024;        // queries, P, rotated parts
-    r.n_slots = (int)((226 * 1024 + 512 - fixed) / (2 * HALF));
-    const int want = 3 * r.n_blocks;
-    if (r.n_slots > want) r.n_slots = want;
-    if (r.n_slots > MAX_SLOTS) r.n_slots = MAX_SLOTS;
-    r.bytes = fixed + (size_t)r.n_slots * 2 * HALF;
-    return r;
-}
-
-// v[c] over the 32 lanes of a warp -> lane c (and c + 16 for N = 16) holds the reduction of v[c]
-template <int N, bool SUM>
-LLM_DEVICE float reduce_columns(float (&v)[N], int lane) {
-    auto op = [](float a, float b) { return SUM ? a + b : fmaxf(a, b); };
-#pragma unroll
-    for (int w = N / 2; w > 0; w >>= 1) {
-        const bool hi = lane & w;
-#pragma unroll
-        for (int i = 0; i < w; ++i) {
-            const float keep = hi ? v[i + w] : v[i], send = hi ? v[i] : v[i + w];
-            v[i] = op(keep, __shfl_xor_sync(0xffffffffu, send, w));
-        }
-    }
-    if (N == 16) v[0] = op(v[0], __shfl_xor_sync(0xffffffffu, v[0], 16));
-    return v[0];
-}
+// Shared memory: a ring of three key tiles (2 atoms per 128 latent values and one for the rotated part), then P.  The queries
+// pass through the third tile's place on their way to TMEM.
+static __host__ __device__ inline int tile_atoms(int latent) { return latent / 64 + 1; }
+static __host__ __device__ inline size_t rows_smem(int n, int latent) { return (size_t)SLOTS * tile_atoms(latent) * HALF + n * 128 + 1024; }
+static __host__ __device__ inline uint32_t pow2_cols(uint32_t n) { uint32_t c = 32; while (c < n) c *= 2; return c; }
 
 template <int N> LLM_DEVICE void tmem_ld_n(uint32_t taddr, uint32_t (&r)[N]);
 template <> LLM_DEVICE void tmem_ld_n<32>(uint32_t taddr, uint32_t (&r)[32]) { tmem_ld32_issue(taddr, r); tmem_wait_ld(r); }
@@ -409,30 +386,32 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     __shared__ __align__(8) uint64_t s_bars[R_BARS];
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort[2];
-    __shared__ float s_red[2][4][32];              // [tile parity] per warp: column maxima (and sums at the end)
+    __shared__ float s_red[2][4][32];              // [tile parity] per warp: maxima (and sums at the end) of its lanes' heads
     __shared__ __align__(16) float s_head[4][32];  // per warp: running maximum (or factor) of every head, for broadcast reads
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const RowsSmem lay = rows_layout(N, p.rot_off);
-    const int NB = lay.n_blocks, NS = lay.n_slots, NA = 2 * NB + 1;
+    const int NB = p.rot_off / 128;
+    const uint32_t tile_bytes = tile_atoms(p.rot_off) * HALF;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-    const uint32_t sQ = base, sP = sQ + NA * N * 128, sR = sP + N * 128, sC = sR + 2 * HALF;
+    const uint32_t sC = base, sQ = sC + 2 * tile_bytes, sP = sC + SLOTS * tile_bytes;
+    // TMEM: S 64 columns, O^T N columns per block, Q one column per two values
+    const uint32_t c_o = 64, c_q = c_o + NB * N, tmem_cols = pow2_cols(c_q + NB * 64 + 32);
     const uint32_t bars = smem_u32(s_bars);
     auto bar = [&](int i) { return bars + i * 8; };
     pdl_trigger();
     if (tid == 0) {
         s_abort[0] = 0; s_abort[1] = 0;
-        for (int i = 0; i < R_BARS; ++i) mbar_init(bar(i), i == RP_FULL || i == RQ_FULL || i == R_MEET ? 4 : 1);
+        for (int i = 0; i < R_BARS; ++i) mbar_init(bar(i), i == RP_FULL || i == RQ_FULL || i == RS_EMPTY || i == R_MEET ? 4 : 1);
         asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
         fence_proxy_async();
     }
     if (warp == 5) {
-        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(256) : "memory");
+        asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(&s_tmem)), "r"(tmem_cols) : "memory");
         asm volatile("tcgen05.relinquish_alloc_permit.cta_group::1.sync.aligned;" ::: "memory");
     }
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
-    const uint32_t tmem = s_tmem, t_o = tmem + 64;             // S^T in columns [0, N) and [32, 32 + N), O^T blocks behind
+    const uint32_t tmem = s_tmem, t_o = tmem + c_o;
     volatile int* abort_flag = s_abort;
     pdl_wait();
 
@@ -448,25 +427,9 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     if (nt == 0) {
         if (tid < N) *reinterpret_cast<float2*>(p.part_ml + (part + tid) * 2) = make_float2(-INFINITY, 0.f);
     } else if (warp < 4) {
-        // query operand, N rows (heads): the latent part comes by TMA, the rotated part (one atom, zero padded) is turned here
-        for (int i = tid; i < N * 8; i += 128) {
-            const int r = i >> 3, u = i & 7, h = hg * N + r;
-            uint4 v = make_uint4(0, 0, 0, 0);
-            if (h < p.n_heads && u * 8 < p.rot_dim)
-                v = rotated8(static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off, u * 8, p.rot_dim,
-                             p.angles + (size_t)t * p.half, p.half);
-            st_shared_v4(atom_addr(sQ + 2 * NB * N * 128, r, u), v);
-        }
-        fence_proxy_async();
-        __syncwarp();
-        mbar_arrive_if(bar(RQ_FULL), lane == 0);
-
+        // query operand: the latent part arrives in shared memory by TMA and moves on to TMEM, the rotated part is turned here
+        const int hl = lane & (N - 1), head = hg * N + hl;      // the head of this lane (its warps hold copies of the same heads)
         const uint32_t t_lane = (uint32_t)(warp * 32) << 16;
-        const int row = warp * 16 + lane;           // key row of the tile (lanes 0-15)
-        const float sl2 = p.scale * LOG2E;
-        float l[N], m = -INFINITY;                  // l: this key lane's share of every head's sum; m: lane c holds head c's maximum
-#pragma unroll
-        for (int c = 0; c < N; ++c) l[c] = 0.f;
         bool ok = true;
         int n_meet = 0;
         auto meet = [&]() {                         // bounded rendezvous of the four softmax warps
@@ -476,6 +439,32 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             ++n_meet;
             return r;
         };
+#pragma unroll
+        for (int k = 0; k < N * 8 / 128; ++k) {
+            const int r = (tid + k * 128) >> 3, u = tid & 7, h = hg * N + r;
+            uint4 v = make_uint4(0, 0, 0, 0);
+            if (h < p.n_heads && u * 8 < p.rot_dim)
+                v = rotated8(static_cast<const __nv_bfloat16*>(p.q) + (size_t)t * p.q_row + (size_t)h * p.q_head + p.q_rot_off, u * 8, p.rot_dim,
+                             p.angles + (size_t)t * p.half, p.half);
+            st_shared_v4(atom_addr(sQ + 2 * NB * N * 128, r, u), v);
+        }
+        ok = meet() && mbar_wait_warp(bar(RQ_LAT), 0, abort_flag);
+        for (int a = 0; a <= 2 * NB && ok; ++a) {
+            uint32_t w[32];
+#pragma unroll
+            for (int u = 0; u < 8; ++u)
+                asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(w[4 * u]), "=r"(w[4 * u + 1]), "=r"(w[4 * u + 2]), "=r"(w[4 * u + 3])
+                             : "r"(atom_addr(sQ + a * N * 128, hl, u)));
+            tmem_st32(tmem + c_q + a * 32 + t_lane, w);
+        }
+        tmem_wait_st();
+        tc_fence_before();
+        fence_proxy_async();                        // the third tile may overwrite the staged queries
+        __syncwarp();
+        mbar_arrive_if(bar(RQ_FULL), lane == 0);
+
+        const float sl2 = p.scale * LOG2E;
+        float l = 0.f, m = -INFINITY;               // l: this warp's keys' share of the head's sum
         auto broadcast = [&](float mine, float (&out)[N]) {      // lane c's value -> out[c] in every lane
             __syncwarp();
             s_head[warp][lane] = mine;
@@ -487,25 +476,41 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             }
         };
         for (int j = 0; j < nt && ok; ++j) {
-            ok = mbar_wait_warp(bar(RS_FULL + (j & 1)), (j >> 1) & 1, abort_flag);
+            ok = mbar_wait_warp(bar(RS_FULL), j & 1, abort_flag);
             if (!ok) break;
             tc_fence_after();
-            uint32_t raw[N];
-            tmem_ld_n<N>(tmem + (j & 1) * 32 + t_lane, raw);
-            const int key = (page0 + j0 + j) * PAGE + row;
-            const bool seen = lane < 16 && key >= lo && key <= pos;
-            float s[N], red[N];
+            float s[16];
+            {
+                uint32_t raw[16];
+                tmem_ld_n<16>(tmem + warp * 16 + t_lane, raw);
+                tc_fence_before();
+                __syncwarp();
+                mbar_arrive_if(bar(RS_EMPTY), lane == 0);       // the next tile's scores may be issued
+                const int key0 = (page0 + j0 + j) * PAGE + warp * 16;
 #pragma unroll
-            for (int c = 0; c < N; ++c) { s[c] = seen ? __uint_as_float(raw[c]) * sl2 : -INFINITY; red[c] = s[c]; }
-            // (the reads of s_red two tiles ago precede that tile's P_FULL arrivals, without which this tile's S is not issued)
+                for (int i = 0; i < 16; ++i) s[i] = key0 + i >= lo && key0 + i <= pos ? __uint_as_float(raw[i]) * sl2 : -INFINITY;
+            }
+            float mx = s[0];
+#pragma unroll
+            for (int i = 1; i < 16; ++i) mx = fmaxf(mx, s[i]);
+            // (the reads of s_red two tiles ago precede the last tile's RS_EMPTY arrivals, without which this tile's S is not issued)
             float (&red4)[4][32] = s_red[j & 1];
-            red4[warp][lane] = reduce_columns<N, false>(red, lane);
+            red4[warp][lane] = mx;
             ok = meet();
             if (!ok) break;
             const float mt = fmaxf(fmaxf(red4[0][lane], red4[1][lane]), fmaxf(red4[2][lane], red4[3][lane]));
             const bool raise = mt > m + RESCALE_STEP;           // also the first tile, where m is -inf
-            const float m_old = m;
+            const float factor = raise ? ex2(m - mt) : 1.f;
             if (raise) m = mt;
+            float sum = 0.f;
+            uint32_t w[8];
+#pragma unroll
+            for (int i = 0; i < 16; i += 2) {
+                const float p0 = ex2(s[i] - m), p1 = ex2(s[i + 1] - m);
+                sum += p0 + p1;
+                w[i >> 1] = pack_bf16(p0, p1);
+            }
+            l = l * factor + sum;
             if (j > 0) {                                        // P and the accumulator are free
                 ok = mbar_wait_warp(bar(RO_DONE), (j - 1) & 1, abort_flag);
                 if (!ok) break;
@@ -513,9 +518,8 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             }
             if (__any_sync(0xffffffffu, raise) && j > 0) {      // the same in all four warps
                 float f[N];
-                broadcast(raise ? ex2(m_old - m) : 1.f, f);
-#pragma unroll
-                for (int c = 0; c < N; ++c) l[c] *= f[c];
+                uint32_t raw[N];
+                broadcast(factor, f);
                 for (int b = 0; b < NB; ++b) {
                     tmem_ld_n<N>(t_o + b * N + t_lane, raw);
 #pragma unroll
@@ -524,15 +528,9 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
                 }
                 tmem_wait_st();
             }
-            float mh[N];
-            broadcast(m, mh);
-            const uint32_t dst = sP + (row & 7) * 2;
-            const int unit = (row & 63) >> 3;
-#pragma unroll
-            for (int c = 0; c < N; ++c) {
-                const float pr = ex2(s[c] - mh[c]);         // 0 on the idle lanes
-                l[c] += pr;
-                if (lane < 16) asm volatile("st.shared.b16 [%0], %1;" ::"r"(dst + c * 128 + (((unit ^ c) & 7) << 4)), "h"(__bfloat16_as_ushort(__float2bfloat16(pr))) : "memory");
+            if (lane < N) {
+                st_shared_v4(atom_addr(sP, lane, 2 * warp), make_uint4(w[0], w[1], w[2], w[3]));
+                st_shared_v4(atom_addr(sP, lane, 2 * warp + 1), make_uint4(w[4], w[5], w[6], w[7]));
             }
             tc_fence_before();
             fence_proxy_async();
@@ -542,7 +540,7 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
         // the last products are complete, so every warp has arrived with its P and is done with the maxima in s_red
         ok = ok && mbar_wait_warp(bar(RO_DONE), (nt - 1) & 1, abort_flag);
         if (ok) {
-            s_red[0][warp][lane] = reduce_columns<N, true>(l, lane);
+            s_red[0][warp][lane] = l;
             ok = meet();
         }
         if (ok) {
@@ -551,7 +549,7 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             uint32_t raw[N];
             if (gridDim.y == 1) {
                 const int h0 = hg * N;
-                if (p.sink && h0 + (lane & (N - 1)) < p.n_heads) lt += exp2f(p.sink[h0 + (lane & (N - 1))] * LOG2E - m);
+                if (p.sink && head < p.n_heads) lt += exp2f(p.sink[head] * LOG2E - m);
                 float inv[N];
                 broadcast(1.f / lt, inv);
                 for (int b = 0; b < NB; ++b) {
@@ -574,64 +572,47 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     } else if (warp == 4) {
         if (elect_one()) {
             bool ok = true;
-            int it = 0;
             mbar_arrive_expect_tx(bar(RQ_LAT), 2 * NB * N * 128);
             for (int a = 0; a < 2 * NB; ++a) tma_load_3d(sQ + a * N * 128, &map_q, a * 64, z, hg * N, bar(RQ_LAT));      // heads past the last: zeros
-            for (int j = 0; j < nt && ok; ++j) {
-                const int r0 = LLM_CHECK_INDEX(btab[page0 + j0 + j], p.n_pages) * PAGE, b2 = j & 1;
-                ok = mbar_wait(bar(ROT_EMPTY + b2), ((j >> 1) & 1) ^ 1, abort_flag);
+            for (int j = 0; j < nt; ++j) {
+                const int r0 = LLM_CHECK_INDEX(btab[page0 + j0 + j], p.n_pages) * PAGE, slot = j % SLOTS;
+                ok = mbar_wait(bar(R_EMPTY + slot), ((j / SLOTS) & 1) ^ 1, abort_flag) && (j != 2 || mbar_wait(bar(RQ_FULL), 0, abort_flag));
                 if (!ok) break;
-                mbar_arrive_expect_tx(bar(ROT_FULL + b2), HALF);
-                tma_load_2d(sR + b2 * HALF, &map_kv, p.rot_off, r0, bar(ROT_FULL + b2));
-                for (int b = 0; b < NB; ++b, ++it) {
-                    const int slot = it % NS;
-                    ok = mbar_wait(bar(R_EMPTY + slot), ((it / NS) & 1) ^ 1, abort_flag);
-                    if (!ok) break;
-                    mbar_arrive_expect_tx(bar(R_FULL + slot), 2 * HALF);
-                    tma_load_2d(sC + slot * 2 * HALF, &map_kv, b * 128, r0, bar(R_FULL + slot));
-                    tma_load_2d(sC + slot * 2 * HALF + HALF, &map_kv, b * 128 + 64, r0, bar(R_FULL + slot));
-                }
+                mbar_arrive_expect_tx(bar(R_FULL + slot), tile_bytes);
+                for (int a = 0; a <= 2 * NB; ++a) tma_load_2d(sC + slot * tile_bytes + a * HALF, &map_kv, a * 64, r0, bar(R_FULL + slot));
             }
         }
     } else {
         // The whole warp walks the pipeline and elects a lane only around each batch of MMAs: loop counters, slots and
         // descriptors then stay warp-uniform, which the issue rate depends on.
-        constexpr uint32_t M_MASK = 31u << 24;
-        constexpr uint32_t idesc_s = (instr_desc(N) & ~M_MASK) | (64u >> 4 << 24), idesc_o = instr_desc(N) | (1u << 15);   // bit 15: A is MN-major
+        constexpr uint32_t idesc_s = instr_desc(PAGE), idesc_o = instr_desc(N) | (1u << 15);         // bit 15: A is MN-major
         const uint32_t tm = __shfl_sync(0xffffffffu, tmem, 0);
         const int n = __shfl_sync(0xffffffffu, nt, 0), rot_steps = (p.width - p.rot_off) / 16;
-        const uint64_t c_desc = smem_desc_sw128(sC), cm_desc = smem_desc_mn_sw128(sC, HALF), q_desc = smem_desc_sw128(sQ), p_desc = smem_desc_sw128(sP),
-                       r_desc = smem_desc_sw128(sR);
-        bool ok = mbar_wait_warp(bar(RQ_LAT), 0, abort_flag) && mbar_wait_warp(bar(RQ_FULL), 0, abort_flag);
+        const uint64_t c_desc = smem_desc_sw128(sC), cm_desc = smem_desc_mn_sw128(sC, HALF), p_desc = smem_desc_sw128(sP);
+        bool ok = mbar_wait_warp(bar(RQ_FULL), 0, abort_flag);
         int s_slot = 0, s_phase = 0, o_slot = 0;
-        // (the softmax has read this accumulator: P of two tiles ago has been waited for)
         auto issue_s = [&](int j) {
-            const int b2 = j & 1;
-            const uint32_t d = tm + b2 * 32;
-            for (int b = 0; b < NB; ++b) {
-                ok = mbar_wait_warp(bar(R_FULL + s_slot), s_phase, abort_flag);
-                if (!ok) return;
-                tc_fence_after();
-                const uint64_t a = c_desc + (uint32_t)(s_slot * (2 * HALF / 16)), q = q_desc + (uint32_t)(b * (2 * N * 128 / 16));
-                const uint32_t first = b > 0 ? 1u : 0u;
-                if (elect_one()) {
-#pragma unroll
-                    for (int ks = 0; ks < 8; ++ks)
-                        mma_f16(d, a + (ks >> 2) * (HALF / 16) + 2 * (ks & 3), q + (ks >> 2) * (N * 128 / 16) + 2 * (ks & 3), idesc_s, ks > 0 ? 1u : first);
-                }
-                __syncwarp();
-                if (++s_slot == NS) { s_slot = 0; s_phase ^= 1; }
-            }
-            ok = mbar_wait_warp(bar(ROT_FULL + b2), (j >> 1) & 1, abort_flag);
+            ok = mbar_wait_warp(bar(R_FULL + s_slot), s_phase, abort_flag) && (j == 0 || mbar_wait_warp(bar(RS_EMPTY), (j - 1) & 1, abort_flag));
             if (!ok) return;
             tc_fence_after();
-            const uint64_t a = r_desc + (uint32_t)(b2 * (HALF / 16)), q = q_desc + (uint32_t)(2 * NB * (N * 128 / 16));
+            uint64_t c = c_desc + (uint32_t)(s_slot * (tile_bytes / 16));
+            uint32_t q = tm + c_q;
             if (elect_one()) {
-                for (int ks = 0; ks < rot_steps; ++ks) mma_f16(d, a + 2 * ks, q + 2 * ks, idesc_s, 1u);
-                mma_commit(bar(RS_FULL + b2));
-                mma_commit(bar(ROT_EMPTY + b2));
+                uint32_t acc = 0;
+                for (int b = 0; b < NB; ++b) {
+#pragma unroll
+                    for (int ks = 0; ks < 8; ++ks) {
+                        mma_f16_ts(tm, q + ks * 8, c + (ks >> 2) * (HALF / 16) + 2 * (ks & 3), idesc_s, acc);
+                        acc = 1;
+                    }
+                    q += 64;
+                    c += 2 * (HALF / 16);
+                }
+                for (int ks = 0; ks < rot_steps; ++ks) mma_f16_ts(tm, q + ks * 8, c + 2 * ks, idesc_s, 1u);
+                mma_commit(bar(RS_FULL));
             }
             __syncwarp();
+            if (++s_slot == SLOTS) { s_slot = 0; s_phase ^= 1; }
         };
         if (ok) issue_s(0);
         for (int j = 0; j < n && ok; ++j) {
@@ -639,26 +620,26 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
             ok = ok && mbar_wait_warp(bar(RP_FULL), j & 1, abort_flag);
             if (!ok) break;
             tc_fence_after();
-            const uint32_t more = j > 0 ? 1u : 0u;
-            for (int b = 0; b < NB; ++b) {
-                const uint64_t a = cm_desc + (uint32_t)(o_slot * (2 * HALF / 16));
-                const uint32_t d = tm + 64 + b * N;
-                if (elect_one()) {
+            if (elect_one()) {
+                uint64_t a = cm_desc + (uint32_t)(o_slot * (tile_bytes / 16));
+                const uint32_t more = j > 0 ? 1u : 0u;
+                for (int b = 0; b < NB; ++b) {
 #pragma unroll
                     for (int ks = 0; ks < 4; ++ks)              // 16 keys: two groups of eight rows
-                        mma_f16(d, a + ks * (2048 / 16), p_desc + 2 * ks, idesc_o, ks > 0 ? 1u : more);
-                    mma_commit(bar(R_EMPTY + o_slot));
-                    if (b == NB - 1) mma_commit(bar(RO_DONE));
+                        mma_f16(tm + c_o + b * N, a + ks * (2048 / 16), p_desc + 2 * ks, idesc_o, ks > 0 ? 1u : more);
+                    a += 2 * (HALF / 16);
                 }
-                __syncwarp();
-                if (++o_slot == NS) o_slot = 0;
+                mma_commit(bar(RO_DONE));
+                mma_commit(bar(R_EMPTY + o_slot));
             }
+            __syncwarp();
+            if (++o_slot == SLOTS) o_slot = 0;
         }
     }
     tc_fence_before();
     __syncthreads();
     teardown(abort_flag, tid, status);
-    if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(256) : "memory");
+    if (warp == 5) asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(tmem), "r"(tmem_cols) : "memory");
 }
 
 // ---- host side ---------------------------------------------------------------------------------------------------------
@@ -715,8 +696,7 @@ cudaError_t launch_latent_chunk_tc(const LatentChunkParams& p, int n_keys, int n
 
 int latent_rows_tc_heads(int width, int rot_off, int rot_dim, int n_heads) {
     if (rot_off % 128 || rot_off < 128 || rot_off > 512 || width % 16 || width - rot_off > 64 || width <= rot_off || rot_dim <= 0) return 0;
-    const int n = n_heads <= 16 ? 16 : 32;
-    return ltc::rows_layout(n, rot_off).n_slots >= 2 * (rot_off / 128) ? n : 0;        // two tiles are in use at a time
+    return n_heads <= 16 ? 16 : 32;
 }
 
 cudaError_t launch_latent_rows_tc(const LatentRowsParams& p, int rows, int n_splits, int* status, cudaStream_t st) {
@@ -734,7 +714,7 @@ cudaError_t launch_latent_rows_tc(const LatentRowsParams& p, int rows, int n_spl
                         CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) != CUDA_SUCCESS)
             return cudaErrorInvalidValue;
     }
-    const size_t smem = rows_layout(n, p.rot_off).bytes;
+    const size_t smem = rows_smem(n, p.rot_off);
     const dim3 grid((p.n_heads + n - 1) / n, n_splits, rows);
     auto go = [&](auto kernel) {
         cudaError_t e = raise_smem(kernel, smem);
