@@ -397,7 +397,8 @@ __global__ void __launch_bounds__(ROWS_THREADS, 1) latent_rows_tc_kernel(const _
     const uint32_t c_o = 64, c_q = c_o + NB * N, tmem_cols = pow2_cols(c_q + NB * 64 + 32);
     const uint32_t bars = smem_u32(s_bars);
     auto bar = [&](int i) { return bars + i * 8; };
-    pdl_trigger();
+    // no early trigger: while this kernel fills the shared memory of its SMs, the CTAs of the kernels behind it would gather on
+    // the few others and stay there
     if (tid == 0) {
         s_abort[0] = 0; s_abort[1] = 0;
         for (int i = 0; i < R_BARS; ++i) mbar_init(bar(i), i == RP_FULL || i == RQ_FULL || i == RS_EMPTY || i == R_MEET ? 4 : 1);

@@ -67,6 +67,28 @@ def test_long_context_many_tiles():
         cases.assert_close(cases.feed_all(eng, t, cuts), want, BF, cuts)
 
 
+@both
+@pytest.mark.parametrize("width", [50, 33, 72])
+def test_widths_off_the_vector_sizes(width, dtype):
+    m = cases.model("loop_middle", seed=11, width=width, vocab=101)
+    t = cases.tokens(150, 12)
+    want = oracle.forward(t, m)
+    eng = cases.engine(m, "cuda", dtype)
+    for cuts in ([150], [120, 7, 1]):
+        cases.assert_close(cases.feed_all(eng, t, cuts), want, dtype, cuts)
+
+
+def test_sizes_without_a_tensor_core_kernel():
+    """A latent beyond the row kernels and heads beyond the chunk kernels run on the plain kernel."""
+    E = oracle.layer_entry
+    m = oracle.random_model(5, layers=[E(heads=2, kv_rank=600, q_rank=40, window=70), E(heads=2, dim=260, rot_dim=24, vdim=264, window=90)], width=48)
+    t = cases.tokens(170, 13)
+    want = oracle.forward(t, m)
+    eng = cases.engine(m, "cuda", BF)
+    for cuts in ([170], [100, 30, 1]):
+        cases.assert_close(cases.feed_all(eng, t, cuts), want, BF, cuts)
+
+
 def test_no_window():
     E = oracle.layer_entry
     m = oracle.random_model(4, layers=[E(heads=3, window=None), E(heads=17, dim=64, rot_dim=16, vdim=64, kv_rank=128, window=None)], width=48)
