@@ -387,10 +387,10 @@ SHAPES = {
     "qwen3-30b-a3b": ModelConfig(name="qwen3-30b-a3b", arch="qwen3moe", n_layers=48, d_model=2048, n_heads=32,
                                  n_kv_heads=4, head_dim=128, d_ff=0, vocab_size=151936, tie_embeddings=False,
                                  n_experts=128, n_experts_used=8, expert_ff=768, context_length=40960),
-    "tiny-pozivik": latent_shape("tiny-pozivik", 3, 256, LatentAttention(4, 32, 16, 32, 64, 96, 48 ** -0.5, Rotary(16, 1e4, RopeScaling(4.0, 256, 32.0, 1.0)), 100),
+    "tiny-pozivik": latent_shape("tiny-pozivik", 3, 256, LatentAttention(4, 32, 16, 32, 64, 120, 48 ** -0.5, Rotary(16, 1e4, RopeScaling(4.0, 256, 32.0, 1.0)), 100),
                                  512, 1024, loop=(1, 3, 2)),
     # layers the size of qwen3-8b's: the same width, feed-forward, vocabulary and number of heads
-    "pozivik-8b": latent_shape("pozivik-8b", 36, 4096, LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 5e4, RopeScaling(4.0, 8192, 32.0, 1.0)), 1024),
+    "pozivik-8b": latent_shape("pozivik-8b", 36, 4096, LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 1e5, RopeScaling(8.0, 4096, 32.0, 1.0)), 1024),
                                12288, 151936),
     "qwen2.5-7b": ModelConfig(name="qwen2.5-7b", arch="qwen2", n_layers=28, d_model=3584, n_heads=28, n_kv_heads=4,
                               head_dim=128, d_ff=18944, vocab_size=152064, tie_embeddings=False, qk_norm=False,

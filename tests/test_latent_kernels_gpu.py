@@ -89,7 +89,7 @@ def test_latent_rows(heads, latent, rot, half, form, window, sinks, splits):
 
 
 @pytest.mark.parametrize("tensor_core", [False, True])
-@pytest.mark.parametrize("heads,dim,rot,vdim,half", [(3, 24, 8, 16, 4), (2, 64, 64, 64, 32), (4, 128, 64, 128, 32), (3, 64, 16, 64, 8), (2, 96, 32, 112, 16), (2, 160, 48, 136, 8)])
+@pytest.mark.parametrize("heads,dim,rot,vdim,half", [(3, 24, 8, 16, 4), (2, 64, 64, 64, 32), (4, 128, 64, 128, 32), (3, 48, 16, 80, 8), (2, 96, 32, 112, 16), (2, 160, 48, 136, 8)])
 @pytest.mark.parametrize("window,sinks", [(0, True), (50, True), (128, False), (300, True), (1, True)])
 def test_latent_chunk(tensor_core, heads, dim, rot, vdim, half, window, sinks):
     from llaminar_b200.ops import latent as ops
@@ -129,7 +129,7 @@ def test_latent_chunk(tensor_core, heads, dim, rot, vdim, half, window, sinks):
 
 
 @pytest.mark.parametrize("dtype", [BF, torch.float32])
-@pytest.mark.parametrize("q_rank,kv_rank,rot,half", [(80, 96, 16, 8), (33, 50, 12, 4), (1536, 512, 64, 32), (24, 40, 8, 2)])
+@pytest.mark.parametrize("q_rank,kv_rank,rot,half", [(72, 104, 24, 8), (33, 50, 12, 4), (1536, 512, 64, 32), (24, 40, 8, 2)])
 def test_latent_prep_and_gather(dtype, q_rank, kv_rank, rot, half):
     from llaminar_b200.ops import latent as ops
     T, off = 150, -(-kv_rank // 8) * 8
