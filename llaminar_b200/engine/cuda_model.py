@@ -297,11 +297,11 @@ class CudaModel:
         self.ff_local = pl.ff_stop - pl.ff_start
         self.stack = None
         self.kv_row_widths = None
-        if c.is_latent:
-            self._init_latent(weights, max_tokens)
+        if c.has_mixers:
+            self._init_stack(weights, max_tokens)
             return
         if dtype != torch.bfloat16:
-            raise ValueError("32-bit mode is available for latent-attention models (the other families' kernels are 16-bit)")
+            raise ValueError("32-bit mode is available for models with per-layer mixers (the other families' kernels are 16-bit)")
 
         if with_embed:
             emb = weights["token_embd.weight"]
@@ -342,45 +342,34 @@ class CudaModel:
             self.mtp_layers.append(lay)
         self._alloc_workspace(max_tokens)
 
-    def _init_latent(self, weights: ModelWeights, max_tokens: int) -> None:
-        """Models whose layers attend over a latent cache: dense matrices, one cache layer per layer run (looped layers have
-        one per pass), each with its own row width."""
-        from .latent import DenseLinear, LatentStack
+    def _init_stack(self, weights: ModelWeights, max_tokens: int) -> None:
+        """Models whose layers have mixers and sizes of their own: unquantised matrices, cache and state layouts per layer."""
+        from .dense import DenseLinear
+        from .latent import LatentStack
+        from .mixers import MixerStack
         c = self.cfg
         if self.layer_ids != list(range(c.n_layers)):
-            raise ValueError("a latent-attention model cannot be cut into pipeline stages")
-        self.stack = LatentStack(self, weights)
-        self.layers = [self.stack.build_layer(CudaLayer(), weights, i) for i in self.layer_ids]
+            raise ValueError(f"a {c.arch} model cannot be cut into pipeline stages")
+        st = self.stack = (LatentStack if c.is_latent else MixerStack)(self, weights)
+        self.layers = [st.build_layer(CudaLayer(), weights, i) for i in self.layer_ids]
         self.out_norm = _f32(weights["output_norm.weight"], self.device)
-        self.head = DenseLinear(self.stack._mat(weights, "output.weight"))
+        self.head = DenseLinear(st._mat(weights, "output.weight"))
         self.vocab_local = c.vocab_size
-        self.runs = c.layer_runs()
-        self.kv_row_widths = [c.mixers[i].cache_width for i, _ in self.runs]
-        self.n_kv_layers = self.mtp_kv_base = len(self.runs)
+        self.kv_row_widths, self.kv_head_shapes, self.state_shapes = st.kv_row_widths, st.kv_head_shapes, st.state_shapes
+        self.n_kv_layers = self.mtp_kv_base = st.n_kv_layers
         self.mtp_layers, self.hybrid_dims, self.graph_safe, self.torch_attention = [], None, True, False
-        self._kv_ids, self._gdn_ids = list(range(len(self.runs))), []
+        self._kv_ids, self._gdn_ids = list(range(self.n_kv_layers)), []
         self.ws_h = torch.empty(max_tokens, c.d_model, dtype=torch.float32, device=self.device)
-        self.stack.alloc_workspace(max_tokens, self.layers)
+        st.alloc_workspace(max_tokens, self.layers)
 
-    def _run_latent(self, fb: ForwardBatch, kv: PagedKVCache, h: torch.Tensor, debug) -> None:
-        """The layer runs of a latent-attention model on the residual stream ``h``."""
-        st, runs, layers = self.stack, self.runs, self.layers
-        bp = st.plan(fb, h.shape[0], layers)
-        first = layers[runs[0][0]].attn_norm
-        st.embed_tokens(fb.tokens, h, None if runs[0][1] else first)
-        for r, (i, starts_pass) in enumerate(runs):
-            L = layers[i]
-            if starts_pass:
-                st.enter_pass(h, L.attn_norm)
-            nxt, to_pass = None, False
-            if r + 1 < len(runs):
-                to_pass = runs[r + 1][1]
-                nxt = None if to_pass else layers[runs[r + 1][0]].attn_norm
-            st.layer(L, h, fb, bp, kv.layers[r], nxt, to_pass)
+    def _run_stack(self, fb: ForwardBatch, kv: PagedKVCache, h: torch.Tensor, debug) -> None:
+        def after_layer(r: int, h: torch.Tensor) -> None:
             if debug is not None:
                 debug(r, h)
             if getattr(self, "taps", None) is not None:
                 self.taps[f"layer{r}"] = h.float().clone()
+
+        self.stack.run(fb, kv, h, self.layers, after_layer)
 
     # ---------------------------------------------------------------------------------------
     def _pack_or_dense(self, t: QTensor):
@@ -860,7 +849,7 @@ class CudaModel:
                 raise IndexError("forward batch rejected before launch: " + "; ".join(errs))
         h = self.ws_h[:T]
         if self.stack is not None:
-            self._run_latent(fb, kv, h, debug)
+            self._run_stack(fb, kv, h, debug)
         elif fb.embeds is not None:
             h.copy_(fb.embeds)
         else:

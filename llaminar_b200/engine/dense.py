@@ -1,0 +1,50 @@
+"""Linear layers with unquantised matrices, shared by the models with per-layer mixers (engine/latent.py, engine/mixers.py)."""
+from __future__ import annotations
+
+import torch
+
+
+def pad8(n: int) -> int:
+    return -(-n // 8) * 8
+
+
+def pad_to(x: torch.Tensor, *shape: int) -> torch.Tensor:
+    out = torch.zeros(*shape, dtype=x.dtype, device=x.device)
+    out[tuple(slice(0, n) for n in x.shape)] = x
+    return out
+
+
+class DenseLinear:
+    """y = x W^T with W as it is stored (bf16, or float in 32-bit mode)."""
+
+    def __init__(self, weight: torch.Tensor, gelu_pair: bool = False):
+        self.w = weight.contiguous()
+        self.n_out, self.k, self.gelu_pair = weight.shape[0], weight.shape[1], gelu_pair
+
+    def nbytes(self) -> int:
+        return self.w.numel() * self.w.element_size()
+
+    def __call__(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+        """``out``: the activation type, or float32 rows (kept at accumulator precision)."""
+        from ..ops import dense as ops
+        if ops.gemv_fits(self.w, x):
+            ops.gemv_dense(self.w.unsqueeze(0), x.unsqueeze(0), out.unsqueeze(0))
+        elif out.dtype != x.dtype:
+            out.copy_(torch.mm(x, self.w.t(), out_dtype=out.dtype))
+        else:
+            torch.mm(x, self.w.t(), out=out)
+        return out
+
+    def activated(self, x: torch.Tensor, act: torch.Tensor, raw: torch.Tensor, kind: int, side=None) -> torch.Tensor:
+        """The product with an activation behind it (`ops.dense.activate`); ``raw`` is workspace for the unfused form."""
+        from ..ops import dense as ops
+        if ops.gemv_fits(self.w, x):
+            ops.gemv_dense(self.w.unsqueeze(0), x.unsqueeze(0), act.unsqueeze(0), act=kind, side=side)
+        else:
+            ops.activate(self(x, raw), act, kind, side)
+        return act
+
+    def gelu(self, x: torch.Tensor, act: torch.Tensor, gu: torch.Tensor) -> torch.Tensor:
+        """act = gelu_tanh(first half) * second half of the product."""
+        from ..ops import dense as ops
+        return self.activated(x, act, gu, ops.ACT_GELU_MUL)

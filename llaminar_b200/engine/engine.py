@@ -18,7 +18,7 @@ import torch
 from ..models.config import ModelConfig
 from ..models.weights import ModelWeights
 from .cuda_model import ForwardBatch
-from .kv_cache import HybridState, PAGE_SIZE, OutOfPages, PagedKVCache, SequenceKV
+from .kv_cache import HybridState, LayerStates, PAGE_SIZE, OutOfPages, PagedKVCache, SequenceKV
 from .kv_cache import Q8 as KV_Q8
 from .sampling import SamplingParams, apply_penalties, sample_row
 from ..utils.env import debug_env
@@ -72,8 +72,8 @@ class LLMEngine:
                  use_graphs: bool = True, prefix_cache=None, mtp=None, tp=None, eos_token_id: int | None = None,
                  model=None, kv_memory_fraction: float = 0.85, kv_dtype: torch.dtype | None = None, agree_group=None,
                  dtype: torch.dtype = torch.bfloat16):
-        """``dtype``: matrices and activations on the GPU (torch.float32: the 32-bit mode of latent-attention models; the CPU
-        back end always computes in 32 bits)."""
+        """``dtype``: matrices and activations on the GPU (torch.float32: the 32-bit mode of models with per-layer mixers; the
+        CPU back end always computes in 32 bits)."""
         self.cfg: ModelConfig = weights.config if weights is not None else model.cfg
         if device is None:
             device = "cuda" if torch.cuda.is_available() else "cpu"
@@ -105,14 +105,18 @@ class LLMEngine:
                                  "attention blocks append to a bf16 cache")
             hybrid = HybridState(n_slots=max(1, max_batch), device=self.device, **hd)
         row_widths = getattr(self.model, "kv_row_widths", None)      # latent attention: one shared row per token and layer
-        if row_widths is not None and (kv_dtype == KV_Q8 or mtp is not None):
-            raise ValueError("latent-attention models have no 8-bit KV cache and no multi-token-prediction head")
+        head_shapes = getattr(self.model, "kv_head_shapes", None)    # layers with keys and values of their own sizes
+        if c.has_mixers and (kv_dtype == KV_Q8 or mtp is not None):
+            raise ValueError(f"{c.arch} models have no 8-bit KV cache and no multi-token-prediction head")
+        state_shapes = getattr(self.model, "state_shapes", None)
+        if state_shapes:
+            hybrid = LayerStates(state_shapes, max(1, max_batch), self.device)
         n_kv_layers = getattr(self.model, "n_kv_layers", c.n_layers + c.nextn_layers)
         if kv_pages is None:
             need = max_batch * self.max_pages_per_seq + 64
             if self.is_cuda:
                 free, _ = torch.cuda.mem_get_info(self.device)
-                per_page = max(1, PagedKVCache.bytes_per_page(n_kv_layers, self.model.n_kv_local, c.head_dim, 17 / 16 if kv_dtype == KV_Q8 else dtype.itemsize, row_widths))
+                per_page = max(1, PagedKVCache.bytes_per_page(n_kv_layers, self.model.n_kv_local, c.head_dim, 17 / 16 if kv_dtype == KV_Q8 else dtype.itemsize, row_widths, head_shapes))
                 kv_pages = int(min(need * 2, max(need // 4, int(free * kv_memory_fraction) // per_page)))
             else:
                 kv_pages = need
@@ -122,7 +126,8 @@ class LLMEngine:
         self._agree_group = agree_group if agree_group is not None else (tp.group if tp is not None and tp.size > 1 else None)
         kv_pages = self._agree_kv_pages(kv_pages, self._agree_group)
         self.kv = PagedKVCache(n_kv_layers, self.model.n_kv_local, c.head_dim, kv_pages, self.device,
-                               dtype=(KV_Q8 if kv_dtype == KV_Q8 else dtype) if self.is_cuda else (kv_dtype or torch.float32), row_widths=row_widths)
+                               dtype=(KV_Q8 if kv_dtype == KV_Q8 else dtype) if self.is_cuda else (kv_dtype or torch.float32), row_widths=row_widths,
+                               head_shapes=head_shapes)
         self.kv.hybrid = hybrid
         self.use_graphs = use_graphs and self.is_cuda and not debug_env().no_cuda_graphs and getattr(self.model, "graph_safe", True)
         self.perf = perf_stats()
@@ -417,7 +422,7 @@ class LLMEngine:
             if self._available_pages() < need:
                 raise OutOfPages("waiting for pages after a preemption")
         hit_pages, hit_tokens = [], 0
-        hybrid = self.cfg.is_hybrid                          # a model property: every rank takes the same branches below
+        hybrid = self.cfg.has_state                          # a model property: every rank takes the same branches below
         if self.prefix_cache is not None:
             term = None if hybrid else self.prefix_cache.lookup_terminal(r.prompt)
             if not self._agree_min(1 if term is not None else 0):
@@ -790,7 +795,7 @@ class LLMEngine:
             self.running.append(r)
             if self.prefix_cache is not None:
                 self.prefix_cache.insert(self, r)
-                if r.terminal is None and not self.cfg.is_hybrid:
+                if r.terminal is None and not self.cfg.has_state:
                     self.prefix_cache.store_terminal(self, r, final_logits[r.rid], final_hidden[r.rid])
             if self.mtp is not None:
                 self.mtp.on_prefill_done(self, r, t, final_hidden[r.rid])

@@ -7,6 +7,7 @@ appends the cached page ids to the new sequence's table and bumps their referenc
 """
 from __future__ import annotations
 
+import math
 from dataclasses import dataclass, field
 
 import torch
@@ -60,17 +61,57 @@ class SequenceKV:
         return len(self.pages) * PAGE_SIZE
 
 
-class HybridState:
+class StateSlots:
+    """Slots of per-sequence recurrent state.  A running sequence owns one slot from admission to its end; slot ``n_slots`` is
+    scratch for the padded lanes of a captured decode step."""
+
+    def __init__(self, n_slots: int):
+        self.n_slots, self.scratch_slot = n_slots, n_slots
+        self.free = list(range(n_slots - 1, -1, -1))
+
+    def alloc(self) -> int:
+        if not self.free:
+            raise OutOfPages("no free state slot")
+        return self.free.pop()
+
+    def release(self, slot: int) -> None:
+        assert 0 <= slot < self.n_slots and slot not in self.free
+        self.free.append(slot)
+
+
+class LayerStates(StateSlots):
+    """State of layers that differ in kind and size: for each layer with a state, one fp32 tensor [slots, ...] per entry of its
+    shape list."""
+
+    def __init__(self, shapes: list[tuple[tuple[int, ...], ...]], n_slots: int, device):
+        super().__init__(n_slots)
+        self.layers = [tuple(torch.zeros(n_slots + 1, *s, dtype=torch.float32, device=device) for s in layer) for layer in shapes]
+
+    def snapshot(self, slot: int) -> tuple[torch.Tensor, ...]:
+        return tuple(t[slot].clone() for layer in self.layers for t in layer)
+
+    def restore(self, slot: int, snap: tuple[torch.Tensor, ...]) -> None:
+        for t, x in zip((t for layer in self.layers for t in layer), snap):
+            t[slot].copy_(x)
+
+    @property
+    def slot_bytes(self) -> int:
+        return 4 * sum(t[0].numel() for layer in self.layers for t in layer)
+
+    @staticmethod
+    def bytes_per_slot(shapes) -> int:
+        return 4 * sum(math.prod(s) for layer in shapes for s in layer)
+
+
+class HybridState(StateSlots):
     """Per-sequence state of the linear-attention layers of a hybrid model: for every such layer and every state slot the
-    last K-1 inputs of the short convolution and one d x d matrix per value head (fp32).  A running sequence owns one slot
-    from admission to its end; slot ``n_slots`` is scratch for the padded lanes of a captured decode step.  (The
-    reference keeps these beside its ring KV cache: src/v2/kernels/cuda/kvcache/CUDAHybridRingKVCache.h.)"""
+    last K-1 inputs of the short convolution and one d x d matrix per value head (fp32).  (The reference keeps these beside
+    its ring KV cache: src/v2/kernels/cuda/kvcache/CUDAHybridRingKVCache.h.)"""
 
     def __init__(self, n_layers: int, n_slots: int, conv_dim: int, conv_kernel: int, n_v_heads: int, d: int, device):
-        self.n_slots, self.scratch_slot = n_slots, n_slots
+        super().__init__(n_slots)
         self.conv = torch.zeros(n_layers, n_slots + 1, conv_dim, conv_kernel - 1, dtype=torch.float32, device=device)
         self.rec = torch.zeros(n_layers, n_slots + 1, n_v_heads, d, d, dtype=torch.float32, device=device)
-        self.free = list(range(n_slots - 1, -1, -1))
         self.stash: dict = {}                  # layer -> what a deferred (speculative) pass left for `commit`
         self.stash_slots = None
 
@@ -83,15 +124,6 @@ class HybridState:
             commit_rows(st, self.conv[layer], self.rec[layer], self.stash_slots, n)
         self.stash.clear()
         self.stash_slots = None
-
-    def alloc(self) -> int:
-        if not self.free:
-            raise OutOfPages("no free state slot")
-        return self.free.pop()
-
-    def release(self, slot: int) -> None:
-        assert 0 <= slot < self.n_slots and slot not in self.free
-        self.free.append(slot)
 
     def snapshot(self, slot: int) -> tuple[torch.Tensor, torch.Tensor]:
         """Copy of one slot's state over all layers (kept by the prefix cache at a block boundary of a prompt)."""
@@ -114,16 +146,21 @@ Q8 = "q8_0"          # 8-bit cache: int8 values with one fp16 scale per 32 (CUDA
 
 
 class PagedKVCache:
-    """Pages of 64 tokens per cache layer.  Per-head layout: [2 (K, V), heads, 64, head size].  With ``row_widths`` (one per
-    layer) a layer holds one row of that many values per token instead, shared by all heads (latent attention)."""
+    """Pages of 64 tokens per cache layer.  Per-head layout: [2 (K, V), heads, 64, head size], with ``head_shapes`` the heads and
+    head size of every layer.  With ``row_widths`` (one per layer) a layer holds one row of that many values per token instead,
+    shared by all heads (latent attention)."""
 
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, n_pages: int, device, dtype=torch.bfloat16,
-                 row_widths: list[int] | None = None):
+                 row_widths: list[int] | None = None, head_shapes: list[tuple[int, int]] | None = None):
         self.n_layers, self.n_kv_heads, self.head_dim, self.n_pages = n_layers, n_kv_heads, head_dim, n_pages
         self.device = torch.device(device)
         self.q8 = dtype == Q8
-        self.row_widths = row_widths
-        if row_widths is not None:
+        self.row_widths, self.head_shapes = row_widths, head_shapes
+        if head_shapes is not None:
+            if self.q8 or len(head_shapes) != n_layers:
+                raise ValueError("a cache of unequal layers takes one (heads, head size) per layer and float values")
+            self.layers = [torch.zeros(n_pages, 2, h, PAGE_SIZE, d, dtype=dtype, device=device) for h, d in head_shapes]
+        elif row_widths is not None:
             if self.q8 or len(row_widths) != n_layers:
                 raise ValueError("a latent cache takes one row width per layer and float rows")
             self.layers = [torch.zeros(n_pages, PAGE_SIZE, w, dtype=dtype, device=device) for w in row_widths]
@@ -139,7 +176,7 @@ class PagedKVCache:
             self.layers = [torch.zeros(n_pages, 2, n_kv_heads, PAGE_SIZE, head_dim, dtype=dtype, device=device)
                            for _ in range(n_layers)]
         self.allocator = PageAllocator(n_pages)
-        self.hybrid: HybridState | None = None          # set by the engine for models with linear-attention layers
+        self.hybrid: HybridState | LayerStates | None = None          # set by the engine for models with recurrent layers
 
     @property
     def page_bytes(self) -> int:
@@ -147,7 +184,10 @@ class PagedKVCache:
         return sum(l[0].numel() * l.element_size() for l in self.layers)
 
     @staticmethod
-    def bytes_per_page(n_layers: int, n_kv_heads: int, head_dim: int, itemsize: float = 2, row_widths: list[int] | None = None) -> int:
+    def bytes_per_page(n_layers: int, n_kv_heads: int, head_dim: int, itemsize: float = 2, row_widths: list[int] | None = None,
+                       head_shapes: list[tuple[int, int]] | None = None) -> int:
+        if head_shapes is not None:
+            return int(sum(2 * h * d for h, d in head_shapes) * PAGE_SIZE * itemsize)
         if row_widths is not None:
             return int(sum(row_widths) * PAGE_SIZE * itemsize)
         return int(n_layers * 2 * n_kv_heads * PAGE_SIZE * head_dim * itemsize)
@@ -182,7 +222,7 @@ class PagedKVCache:
         """One page over all layers, on the device: [layers, ...page], or one flat run where the layers' rows differ."""
         if not self.layers:                      # a pipeline stage of linear-attention blocks only: pages carry no bytes here
             return torch.empty(0)
-        if self.row_widths is not None:
+        if self.row_widths is not None or self.head_shapes is not None:
             return torch.cat([l[page].reshape(-1) for l in self.layers])
         return torch.stack([l[page] for l in self.layers])
 
@@ -190,7 +230,7 @@ class PagedKVCache:
         return self.copy_page(page).to("cpu", non_blocking=False)
 
     def import_page(self, page: int, payload: torch.Tensor) -> None:
-        if self.row_widths is not None:
-            payload = [x.view(PAGE_SIZE, -1) for x in payload.split([PAGE_SIZE * w for w in self.row_widths])]
+        if self.row_widths is not None or self.head_shapes is not None:
+            payload = [x.view(l[page].shape) for x, l in zip(payload.split([l[page].numel() for l in self.layers]), self.layers)]
         for i, l in enumerate(self.layers):
             l[page].copy_(payload[i].to(self.device, non_blocking=True))

@@ -21,45 +21,11 @@ from dataclasses import dataclass, field
 import torch
 
 from ..models.config import LatentAttention
+from .dense import DenseLinear, pad8, pad_to
 
 SHORT_ROWS = 8                 # portions of up to this many tokens attend row by row in the latent space
 PART_FLOATS = 1 << 23          # scratch of the split row kernel
 PLAIN_ROWS = 1024              # rows per launch where the row kernel serves whole prompts (32-bit mode, unusual sizes)
-
-
-def pad8(n: int) -> int:
-    return -(-n // 8) * 8
-
-
-class DenseLinear:
-    """y = x W^T with W as it is stored (bf16, or float in 32-bit mode)."""
-
-    def __init__(self, weight: torch.Tensor, gelu_pair: bool = False):
-        self.w = weight.contiguous()
-        self.n_out, self.k, self.gelu_pair = weight.shape[0], weight.shape[1], gelu_pair
-
-    def nbytes(self) -> int:
-        return self.w.numel() * self.w.element_size()
-
-    def __call__(self, x: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-        """``out``: the activation type, or float32 rows (kept at accumulator precision)."""
-        from ..ops import latent as ops
-        if ops.gemv_fits(self.w, x):
-            ops.gemv_dense(self.w.unsqueeze(0), x.unsqueeze(0), out.unsqueeze(0))
-        elif out.dtype != x.dtype:
-            out.copy_(torch.mm(x, self.w.t(), out_dtype=out.dtype))
-        else:
-            torch.mm(x, self.w.t(), out=out)
-        return out
-
-    def gelu(self, x: torch.Tensor, act: torch.Tensor, gu: torch.Tensor) -> torch.Tensor:
-        """act = gelu_tanh(first half) * second half of the product; ``gu`` is workspace for the unfused form."""
-        from ..ops import latent as ops
-        if ops.gemv_fits(self.w, x):
-            ops.gemv_dense(self.w.unsqueeze(0), x.unsqueeze(0), act.unsqueeze(0), gelu=True)
-        else:
-            ops.gelu_mul(self(x, gu), act)
-        return act
 
 
 @dataclass(frozen=True)
@@ -76,12 +42,6 @@ class PaddedSizes:
     @staticmethod
     def of(m: LatentAttention) -> "PaddedSizes":
         return PaddedSizes(m.heads, pad8(m.dim), pad8(m.rot_dim), pad8(m.vdim), pad8(m.q_rank), pad8(m.kv_rank), m.cache_width)
-
-
-def pad_to(x: torch.Tensor, *shape: int) -> torch.Tensor:
-    out = torch.zeros(*shape, dtype=x.dtype, device=x.device)
-    out[tuple(slice(0, n) for n in x.shape)] = x
-    return out
 
 
 @dataclass
@@ -113,6 +73,10 @@ class LatentStack:
         self.loop_in = DenseLinear(self._mat(weights, "loop_in.weight")) if c.loop else None
         from .. import ops
         self.status = ops.scratch_for(self.device).status               # word that a kernel sets when a bounded wait runs out
+        self.runs = c.layer_runs()                       # looped layers have a cache layer per pass, each with its own row width
+        self.kv_row_widths = [c.mixers[i].cache_width for i, _ in self.runs]
+        self.kv_head_shapes = self.state_shapes = None
+        self.n_kv_layers = len(self.runs)
         self.rotaries: list = []
         self.freqs: list[torch.Tensor] = []
 
@@ -177,6 +141,22 @@ class LatentStack:
         return self._ws[name][:T * cols].view(T, cols)
 
     # -- one forward call ------------------------------------------------------------------------------------
+    def run(self, fb, kv, h: torch.Tensor, layers, after_layer) -> None:
+        """The layer runs on the residual stream ``h``."""
+        bp = self.plan(fb, h.shape[0], layers)
+        first = layers[self.runs[0][0]].attn_norm
+        self.embed_tokens(fb.tokens, h, None if self.runs[0][1] else first)
+        for r, (i, starts_pass) in enumerate(self.runs):
+            L = layers[i]
+            if starts_pass:
+                self.enter_pass(h, L.attn_norm)
+            nxt, to_pass = None, False
+            if r + 1 < len(self.runs):
+                to_pass = self.runs[r + 1][1]
+                nxt = None if to_pass else layers[self.runs[r + 1][0]].attn_norm
+            self.layer(L, h, fb, bp, kv.layers[r], nxt, to_pass)
+            after_layer(r, h)
+
     def plan(self, fb, T: int, layers) -> BatchPlan:
         from ..ops import latent as ops
         angles = []

@@ -12,8 +12,8 @@ import math
 import torch
 import torch.nn.functional as F
 
-from ..models import gdn
-from ..models.config import ModelConfig
+from ..models import gdn, mixers
+from ..models.config import MatrixLSTM, ModelConfig
 from ..models.reference import moe_route, rmsnorm, rope_split_half
 from ..models.weights import ModelWeights
 from ..parallel.tp_plan import TPPlan
@@ -43,8 +43,10 @@ class TorchPagedModel:
             self.head = head.rows(pl.vocab_start, pl.vocab_stop).to_float().to(self.device)
             self.vocab_local = pl.vocab_stop - pl.vocab_start
 
-        if c.is_latent:
-            self._init_latent(f)
+        if c.has_mixers:
+            if self.layer_ids != list(range(c.n_layers)):
+                raise ValueError(f"a {c.arch} model cannot be cut into pipeline stages")
+            self._init_latent(f) if c.is_latent else self._init_mixers(f)
             return
         kv_ids, gdn_ids = c.kv_layers(self.layer_ids), c.gdn_layers(self.layer_ids)
 
@@ -123,8 +125,6 @@ class TorchPagedModel:
     # -- latent-attention models ------------------------------------------------------------------------
     def _init_latent(self, f) -> None:
         c = self.cfg
-        if self.layer_ids != list(range(c.n_layers)):
-            raise ValueError("a latent-attention model cannot be cut into pipeline stages")
         self.embed_norm = f("token_embd_norm.weight")
         self.loop_in = f("loop_in.weight") if c.loop else None
         names = {"attn_norm": "attn_norm", "post_attn": "post_attention_norm", "qa": "attn_q_a", "qan": "attn_q_a_norm", "qb": "attn_q_b",
@@ -203,6 +203,111 @@ class TorchPagedModel:
                 h = h + rmsnorm(y, L["post_ffn"], eps)
             if getattr(self, "taps", None) is not None:
                 self.taps[f"layer{r}"] = h.clone()
+        return h
+
+    # -- layers of windowed attention, retention and matrix LSTMs --------------------------------------------
+    def _init_mixers(self, f) -> None:
+        c = self.cfg
+        self.side_embed = f("side_embd.weight") if c.side_dim else None
+        self.layers, kv_i, st_i = [], 0, 0
+        for i in self.layer_ids:
+            p, m = f"blk.{i}.", c.mixers[i]
+            L = {"mixer": m, "state": st_i, "kv": kv_i, "post_mix": f(p + "post_attention_norm.weight") * f(p + "post_attention_scale.weight")}
+            names = ["lstm_q", "lstm_k", "lstm_v", "lstm_g", "lstm_i", "lstm_f", "lstm_output", "lstm_norm"] if isinstance(m, MatrixLSTM) else \
+                ["attn_q", "attn_k", "attn_gate", "attn_q_norm", "attn_k_norm", "attn_sinks", "attn_output", "attn_out_norm",
+                 "ret_q", "ret_k", "ret_v", "ret_g", "ret_output", "ret_out_norm"]
+            L.update({n: f(f"{p}{n}.weight") for n in names})
+            if isinstance(m, MatrixLSTM):
+                L["bi"], L["bf"] = f(p + "lstm_i.bias"), f(p + "lstm_f.bias")
+            else:
+                L["freqs"] = torch.tensor(m.right.rotary.frequencies(), dtype=torch.float64, device=self.device)
+                kv_i += 1
+            st_i += 1
+            if c.ff_width(i):
+                L["post_ffn"] = f(p + "post_ffw_norm.weight") * f(p + "post_ffw_scale.weight")
+                L["wu"], L["wd"] = f(p + "ffn_up.weight"), f(p + "ffn_down.weight")
+            if c.side_dim:
+                L.update({n: f(f"{p}{n}.weight") for n in ("side_gate", "side_proj", "side_norm")})
+            self.layers.append(L)
+        self.kv_head_shapes = mixers.mixer_kv_shapes(c)
+        self.state_shapes = mixers.mixer_state_shapes(c)
+        self.n_kv_layers = self.mtp_kv_base = len(self.kv_head_shapes)
+        self.mtp_layers, self.hybrid_dims = [], None
+
+    def _recurrent(self, L, m, q, k, v, fb: ForwardBatch, kv: PagedKVCache, rows_fn) -> torch.Tensor:
+        """Runs `rows_fn(q, k, v, first row, end row, *state)` per sequence on its slot's state; returns the heads' outputs, each
+        divided by its root mean square."""
+        state, out = kv.hybrid.layers[L["state"]], torch.empty_like(v)
+        for r0, r1, slot, fresh in gdn.batch_sequences(fb.seq_ids, fb.positions, fb.state_slots):
+            if fresh:
+                for t in state:
+                    t[slot].zero_()
+            out[r0:r1] = rows_fn(q[r0:r1], k[r0:r1], v[r0:r1], r0, r1, *(t[slot] for t in state))
+        return (out * torch.rsqrt(out.pow(2).mean(-1, keepdim=True) + self.cfg.rms_eps)).reshape(q.shape[0], -1)
+
+    def _mlstm(self, L, x: torch.Tensor, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        m, T = L["mixer"], x.shape[0]
+        q, k, v = ((x @ L[f"lstm_{n}"].T).view(T, m.heads, -1) for n in "qkv")
+        i, f = mixers.mlstm_gates(x @ L["lstm_i"].T + L["bi"], x @ L["lstm_f"].T + L["bf"], m.gate_cap)
+        o = self._recurrent(L, m, q * m.dim ** -0.5, k, v, fb, kv, lambda q, k, v, r0, r1, *st: mixers.mlstm_rows(q, k, v, i[r0:r1], f[r0:r1], *st))
+        return (o * L["lstm_norm"] * torch.sigmoid(x @ L["lstm_g"].T)) @ L["lstm_output"].T
+
+    def _retention(self, L, x: torch.Tensor, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        m, T = L["mixer"].right, x.shape[0]
+        q, k, v = ((x @ L[f"ret_{n}"].T).view(T, m.heads, -1) for n in "qkv")
+        ang = fb.positions.double()[:, None] * L["freqs"]
+        cos, sin = ang.cos().float()[:, None], ang.sin().float()[:, None]
+        q, k = self._turn(q, cos, sin), self._turn(k, cos, sin) * m.dim ** -0.5
+        decay = torch.tensor(m.decay)
+        o = self._recurrent(L, m, q, k, v, fb, kv, lambda q, k, v, r0, r1, S: mixers.retention_rows(q, k, v, decay, S))
+        return (o * F.silu(x @ L["ret_g"].T)) @ L["ret_output"].T
+
+    def _window_attention(self, L, x: torch.Tensor, fb: ForwardBatch, kvl: torch.Tensor) -> torch.Tensor:
+        c, m, T = self.cfg, L["mixer"].left, x.shape[0]
+        k = x @ L["attn_k"].T
+        v = k.view(T, m.kv_heads, m.dim)
+        q = rmsnorm(x @ L["attn_q"].T, L["attn_q_norm"], c.rms_eps).view(T, m.kv_heads, -1, m.dim)
+        k = rmsnorm(k, L["attn_k_norm"], c.rms_eps).view(T, m.kv_heads, m.dim)
+        pos, sid = fb.positions.long(), fb.seq_ids.long()
+        page, off = fb.block_table.long()[sid, pos // PAGE_SIZE], pos % PAGE_SIZE
+        kvl[page, 0, :, off], kvl[page, 1, :, off] = k.to(kvl.dtype), v.to(kvl.dtype)
+        out = torch.empty(T, m.heads * m.dim)
+        for b in sid.unique().tolist():
+            rows = (sid == b).nonzero(as_tuple=True)[0]
+            p = pos[rows]
+            keys = torch.arange(max(0, int(p.min()) - m.window + 1) if m.window else 0, int(p.max()) + 1)
+            pages, off = fb.block_table.long()[b, keys // PAGE_SIZE], keys % PAGE_SIZE
+            K, V = kvl[pages, 0, :, off].float(), kvl[pages, 1, :, off].float()                # [keys, kv heads, dim]
+            s = torch.einsum("tghd,sgd->ghts", q[rows], K) * m.scale
+            hidden = keys[None, :] > p[:, None]
+            if m.window:
+                hidden |= keys[None, :] <= p[:, None] - m.window
+            s = s.masked_fill(hidden, float("-inf"))
+            sink = L["attn_sinks"].view(m.kv_heads, -1, 1, 1).expand(*s.shape[:3], 1)          # one more column that carries no value
+            w = torch.softmax(torch.cat([s, sink], dim=-1), -1)[..., :-1]
+            out[rows] = torch.einsum("ghts,sgd->tghd", w, V).reshape(len(rows), -1)
+        return (out * torch.sigmoid(x @ L["attn_gate"].T)) @ L["attn_output"].T
+
+    def _run_mixers(self, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        c, eps = self.cfg, self.cfg.rms_eps
+        tok = fb.tokens.long()
+        h = self.embed[tok].float() * c.embed_scale
+        norm = lambda x, w: F.layer_norm(x, x.shape[-1:], w, None, eps)
+        for i, L in enumerate(self.layers):
+            if isinstance(L["mixer"], MatrixLSTM):
+                y = self._mlstm(L, h, fb, kv)
+            else:
+                y = 0.5 * (rmsnorm(self._window_attention(L, h, fb, kv.layers[L["kv"]]), L["attn_out_norm"], eps)
+                           + rmsnorm(self._retention(L, h, fb, kv), L["ret_out_norm"], eps))
+            h = h + c.residual_mult * norm(y, L["post_mix"])
+            if "wu" in L:
+                h = h + c.residual_mult * norm(F.relu(h @ L["wu"].T).square() @ L["wd"].T, L["post_ffn"])
+            if c.side_dim:
+                e = self.side_embed[tok, i * c.side_dim:(i + 1) * c.side_dim]
+                y = (F.gelu(h @ L["side_gate"].T, approximate="tanh") * e) @ L["side_proj"].T
+                h = h + c.residual_mult * rmsnorm(y, L["side_norm"], eps)
+            if getattr(self, "taps", None) is not None:
+                self.taps[f"layer{i}"] = h.clone()
         return h
 
     # ---------------------------------------------------------------------------------------
@@ -304,7 +409,8 @@ class TorchPagedModel:
         return h + y
 
     def _logits(self, h_rows, norm_w, out):
-        lg = rmsnorm(h_rows, norm_w, self.cfg.rms_eps) @ self.head.T
+        x = F.layer_norm(h_rows, h_rows.shape[-1:], norm_w, None, self.cfg.rms_eps) if self.cfg.norm_kind == "layer" else rmsnorm(h_rows, norm_w, self.cfg.rms_eps)
+        lg = x @ self.head.T
         if out is not None:
             out[:lg.shape[0]].copy_(lg)
             return out[:lg.shape[0]]
@@ -312,12 +418,12 @@ class TorchPagedModel:
 
     @torch.no_grad()
     def forward(self, fb: ForwardBatch, kv: PagedKVCache, logits_out=None, want_logits=True, kv_layer_offset: int = 0):
-        latent = self.cfg.is_latent
-        if latent:
-            h = self._run_latent(fb, kv)
+        own = self.cfg.has_mixers
+        if own:
+            h = self._run_latent(fb, kv) if self.cfg.is_latent else self._run_mixers(fb, kv)
         else:
             h = fb.embeds.float() if fb.embeds is not None else self.embed[fb.tokens.long()].float()
-        for li, L in enumerate(() if latent else self.layers):
+        for li, L in enumerate(() if own else self.layers):
             kvl = kv.layers[kv_layer_offset + L["kv_index"]] if L.get("kv_index") is not None else None
             h = self._layer(L, h, fb, kvl, kv)
             if getattr(self, "taps", None) is not None:       # per-layer hidden states for the parity report

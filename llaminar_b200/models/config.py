@@ -13,7 +13,7 @@ from dataclasses import asdict, dataclass, field, replace
 
 from ..gguf.constants import GGMLType
 
-SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik")
+SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik", "zogepel")
 
 
 @dataclass(frozen=True)
@@ -80,6 +80,54 @@ class LatentAttention:
         return (-(-self.kv_rank // 8) * 8 + -(-self.rot_dim // 8) * 8 + 15) // 16 * 16
 
 
+@dataclass(frozen=True)
+class WindowAttention:
+    """Grouped-query softmax attention with per-head keys and values in the paged cache, no rotation.  Queries and keys are
+    RMS-normed over the whole projection (all heads together, one gain per value)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    scale: float
+    window: int = 0                 # keys a query sees, itself included (0: all before it)
+    sinks: bool = True              # one learned logit per head in the softmax denominator
+    tied_values: bool = True        # the values are the projected keys before their norm
+    gated: bool = True              # heads times sigmoid of a projection of the input, before the output projection
+
+
+@dataclass(frozen=True)
+class Retention:
+    """Linear attention S_t = decay_h S_(t-1) + k_t v_t^T with rotated queries and keys, no denominator; the output of a head is
+    divided by its root mean square and gated by silu."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple[float, ...]        # per head
+    rotary: Rotary
+
+
+@dataclass(frozen=True)
+class MatrixLSTM:
+    """Linear attention with exponential input gate and logistic forget gate per head and token (mLSTM): state S [dim, vdim], the
+    normaliser n [dim] and the running maximum of the log gates.  Both gates are soft-capped; the output of a head is divided by
+    its root mean square, scaled by a gain per value and gated by a sigmoid."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+@dataclass(frozen=True)
+class ParallelMixers:
+    """Two mixers on the same input; half the sum of their outputs, each RMS-normed over the model width."""
+    left: WindowAttention
+    right: Retention
+
+
+def mixer_parts(m) -> tuple:
+    """The elementary mixers of a layer."""
+    return (m.left, m.right) if isinstance(m, ParallelMixers) else (m,)
+
+
 @dataclass
 class ModelConfig:
     arch: str = "qwen3"
@@ -113,14 +161,20 @@ class ModelConfig:
     ssm_k_heads: int = 0
     ssm_v_heads: int = 0
     rope_dim: int = 0                    # leading dims of each head that are rotated (0: all of head_dim)
-    # layer lists with their own sizes per layer (pozivik): the mixer of every layer, its feed-forward width (0: none), and
-    # the layers [start, stop) that run `times` times in a row, each pass behind a projection of [hidden | embedding]
-    mixers: tuple[LatentAttention, ...] = ()
+    # layer lists with their own sizes per layer (pozivik, zogepel): the mixer of every layer, its feed-forward width (0: none),
+    # and the layers [start, stop) that run `times` times in a row, each pass behind a projection of [hidden | embedding]
+    mixers: tuple[LatentAttention | MatrixLSTM | ParallelMixers, ...] = ()
     layer_ff: tuple[int, ...] = ()
     loop: tuple[int, int, int] | None = None
     embed_norm: bool = False             # RMSNorm on the token embedding
-    post_norms: bool = False             # RMSNorm on the output of a sublayer, before it joins the residual stream
-    ffn_act: str = "silu"                # silu | gelu_tanh: activation of the gated feed-forward
+    embed_scale: float = 1.0             # factor on the token embedding
+    pre_norms: bool = True               # norm on the input of a sublayer
+    post_norms: bool = False             # norm on the output of a sublayer, before it joins the residual stream
+    norm_kind: str = "rms"               # rms | layer (mean taken off, no bias): the norms of the residual stream
+    layer_scale: bool = False            # a gain per value on every sublayer's (normed) output
+    residual_mult: float = 1.0           # factor on what joins the residual stream
+    side_dim: int = 0                    # width of the per-layer token input behind the feed-forward (0: none)
+    ffn_act: str = "silu"                # silu | gelu_tanh: activation of the gated feed-forward; relu2: ungated, squared relu
     attn_gate: bool = False              # attn_q holds [q | gate] per head; the attention output is scaled by sigmoid(gate)
     name: str = "tiny-qwen3"
 
@@ -138,8 +192,18 @@ class ModelConfig:
 
     @property
     def is_latent(self) -> bool:
-        """Latent-attention layers, run by the latent block (their own cache layout, 16- or 32-bit weight matrices)."""
+        """Latent-attention layers, run by the latent block (their own cache layout)."""
+        return self.has_mixers and isinstance(self.mixers[0], LatentAttention)
+
+    @property
+    def has_mixers(self) -> bool:
+        """Layers with a mixer and sizes of their own: 16- or 32-bit weight matrices, one GPU."""
         return bool(self.mixers)
+
+    @property
+    def has_state(self) -> bool:
+        """Some layer carries a recurrent state from token to token, in a slot per sequence."""
+        return self.is_hybrid or any(isinstance(p, (Retention, MatrixLSTM)) for m in self.mixers for p in mixer_parts(m))
 
     def layer_runs(self) -> list[tuple[int, bool]]:
         """The layers in the order they run: (layer, whether a pass over the looped layers starts before it).  Every run has a
@@ -200,9 +264,8 @@ class ModelConfig:
         if arch not in SUPPORTED_ARCHS:
             raise ValueError(f"unsupported GGUF architecture '{arch}' (supported: {', '.join(SUPPORTED_ARCHS)}; "
                              "qwen35 / qwen35moe are the hybrid Gated-DeltaNet families)")
-        if arch == "pozivik":
-            from .pozivik import config_from_json
-            return config_from_json(json.loads(gf.get("pozivik.config")))
+        if arch in ("pozivik", "zogepel"):
+            return family_of(arch).config_from_json(json.loads(gf.get(f"{arch}.config")))
         a = gf.arch_key
 
         def scalar(v):
@@ -263,9 +326,8 @@ class ModelConfig:
 
     def gguf_metadata(self) -> dict:
         a = self.arch
-        if a == "pozivik":
-            from .pozivik import config_to_json
-            return {"general.architecture": a, "general.name": self.name, "pozivik.config": json.dumps(config_to_json(self))}
+        if self.has_mixers:
+            return {"general.architecture": a, "general.name": self.name, f"{a}.config": json.dumps(family_of(a).config_to_json(self))}
         md = {
             "general.architecture": a,
             "general.name": self.name,
@@ -298,6 +360,12 @@ class ModelConfig:
             if self.rope_dim:
                 md[f"{a}.rope.dimension_count"] = self.rope_dim
         return md
+
+
+def family_of(arch: str):
+    """The module that reads and writes the checkpoints of a family with per-layer mixers."""
+    import importlib
+    return importlib.import_module(f"{__package__}.{arch}")
 
 
 @dataclass
@@ -359,6 +427,17 @@ def latent_shape(name: str, n_layers: int, d_model: int, mixer: LatentAttention,
                        layer_ff=(ff,) * n_layers, loop=loop, embed_norm=True, post_norms=True, ffn_act="gelu_tanh")
 
 
+def mixed_shape(name: str, d_model: int, mixers: tuple, ff: int, vocab: int, side_dim: int, eps: float = 1e-5, context_length: int = 32768) -> ModelConfig:
+    """A zogepel shape with one feed-forward width."""
+    return ModelConfig(name=name, arch="zogepel", n_layers=len(mixers), d_model=d_model, d_ff=ff, vocab_size=vocab, rms_eps=eps,
+                       context_length=context_length, mixers=mixers, layer_ff=(ff,) * len(mixers), embed_scale=d_model ** 0.5,
+                       residual_mult=0.25, side_dim=side_dim, **ZOGEPEL)
+
+
+# what every zogepel model has in common
+ZOGEPEL = dict(qk_norm=False, tie_embeddings=False, pre_norms=False, post_norms=True, norm_kind="layer", layer_scale=True, ffn_act="relu2")
+
+
 # The benchmark shapes (random-init stand-ins for the named public models).
 SHAPES = {
     "tiny-qwen3": ModelConfig(name="tiny-qwen3"),
@@ -392,6 +471,11 @@ SHAPES = {
     # layers the size of qwen3-8b's: the same width, feed-forward, vocabulary and number of heads
     "pozivik-8b": latent_shape("pozivik-8b", 36, 4096, LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 1e5, RopeScaling(8.0, 4096, 32.0, 1.0)), 1024),
                                12288, 151936),
+    "tiny-zogepel": mixed_shape("tiny-zogepel", 256, (MatrixLSTM(4, 32, 64, 12.0), ParallelMixers(WindowAttention(4, 2, 64, 0.125, 96), Retention(
+                                4, 32, 48, (0.9, 0.97, 0.99, 0.998), Rotary(24, 1e4)))) * 2, 512, 1024, 32),
+    # layers of qwen3-8b's width, feed-forward width and vocabulary, alternating
+    "zogepel-8b": mixed_shape("zogepel-8b", 4096, (MatrixLSTM(16, 128, 256, 15.0), ParallelMixers(WindowAttention(32, 8, 128, 128 ** -0.5, 1024), Retention(
+                              16, 128, 256, tuple(1.0 - 2.0 ** (-5.0 - i / 2) for i in range(16)), Rotary(128, 1e4)))) * 18, 12288, 151936, 256),
     "qwen2.5-7b": ModelConfig(name="qwen2.5-7b", arch="qwen2", n_layers=28, d_model=3584, n_heads=28, n_kv_heads=4,
                               head_dim=128, d_ff=18944, vocab_size=152064, tie_embeddings=False, qk_norm=False,
                               qkv_bias=True, context_length=32768),

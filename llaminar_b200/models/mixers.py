@@ -1,0 +1,84 @@
+"""Mixers with sizes of their own per layer: what they keep in the cache and in the state slots, and their recurrences in plain
+PyTorch (the CPU back end).
+
+Per head, with log input gate i, log forget gate f and running maximum m (which starts at 0):
+
+    mLSTM       m' = max(f + m, i);  S' = e^(f+m-m') S + e^(i-m') v k^T;  n' = e^(f+m-m') n + e^(i-m') k
+                o = S' q / (max(|n'.q|, e^-m') + NORM_FLOOR)
+    retention   S' = decay S + v k^T;  o = S' q
+
+The state matrix is held as [vdim, dim]: a row per value, so that reading it out is a product with q along contiguous memory.
+"""
+from __future__ import annotations
+
+import torch
+import torch.nn.functional as F
+
+from .config import MatrixLSTM, ModelConfig, ParallelMixers, Retention, WindowAttention, mixer_parts
+
+NORM_FLOOR = 1e-6
+
+
+def pad_to_multiple(n: int, of: int) -> int:
+    return -(-n // of) * of
+
+
+def mixer_kv_shapes(cfg: ModelConfig, head_pad=lambda dim: dim) -> list[tuple[int, int]]:
+    """(heads, head size) of every cache layer."""
+    return [(p.kv_heads, head_pad(p.dim)) for m in cfg.mixers for p in mixer_parts(m) if isinstance(p, WindowAttention)]
+
+
+def state_shapes_of(m, pad: int = 1) -> tuple[tuple[int, ...], ...]:
+    d, v = pad_to_multiple(m.dim, pad), pad_to_multiple(m.vdim, pad)
+    if isinstance(m, MatrixLSTM):
+        return (m.heads, v, d), (m.heads, d), (m.heads,)
+    return ((m.heads, v, d),)
+
+
+def mixer_state_shapes(cfg: ModelConfig, pad: int = 1) -> list[tuple[tuple[int, ...], ...]]:
+    """Shapes of the state tensors of every recurrent mixer, in layer order; sizes rounded up to a multiple of ``pad``."""
+    return [state_shapes_of(p, pad) for m in cfg.mixers for p in mixer_parts(m) if isinstance(p, (MatrixLSTM, Retention))]
+
+
+def mixer_columns(m) -> int:
+    """Values per token between a mixer's input and output products (for the memory estimate)."""
+    if isinstance(m, ParallelMixers):
+        return sum(mixer_columns(p) for p in mixer_parts(m))
+    if isinstance(m, WindowAttention):
+        return (4 * m.heads + m.kv_heads) * m.dim
+    if isinstance(m, (MatrixLSTM, Retention)):
+        return m.heads * (2 * m.dim + 4 * m.vdim)
+    return 0
+
+
+def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(x / cap)
+
+
+def mlstm_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float) -> tuple[torch.Tensor, torch.Tensor]:
+    """Log input gate and log forget gate of the gate projections (biases added)."""
+    return soft_cap(zi, cap), F.logsigmoid(soft_cap(zf, cap))
+
+
+def mlstm_rows(q, k, v, i, f, S, n, m):
+    """New tokens of one sequence, one after the other.  q (scaled), k [T, H, d], v [T, H, e], i, f [T, H]; the state S [H, e, d],
+    n [H, d], m [H] is updated in place.  Returns o [T, H, e]."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        top = torch.maximum(f[t] + m, i[t])
+        keep, add = torch.exp(f[t] + m - top), torch.exp(i[t] - top)
+        S.mul_(keep[:, None, None]).add_((add[:, None] * v[t])[:, :, None] * k[t][:, None, :])
+        n.mul_(keep[:, None]).add_(add[:, None] * k[t])
+        m.copy_(top)
+        size = torch.maximum((n * q[t]).sum(-1).abs(), torch.exp(-m)) + NORM_FLOOR
+        out[t] = (S @ q[t][:, :, None])[..., 0] / size[:, None]
+    return out
+
+
+def retention_rows(q, k, v, decay, S):
+    """As `mlstm_rows` for retention: q, k rotated, k scaled, decay [H]."""
+    out = torch.empty_like(v)
+    for t in range(q.shape[0]):
+        S.mul_(decay[:, None, None]).add_(v[t][:, :, None] * k[t][:, None, :])
+        out[t] = (S @ q[t][:, :, None])[..., 0]
+    return out

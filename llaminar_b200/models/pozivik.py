@@ -11,9 +11,8 @@ from typing import Mapping
 
 import torch
 
-from ..gguf import GGMLType
 from .config import LatentAttention, ModelConfig, Rotary, RopeScaling
-from .weights import ModelWeights, QTensor, qtensor_from_float
+from .weights import ModelWeights, named_weights
 
 ARCHITECTURE = "Pozivik"
 CONTEXT_LENGTH = 1 << 20            # a checkpoint states no limit on positions
@@ -102,15 +101,4 @@ def tensor_names(c: ModelConfig) -> list[tuple[str, str, str, tuple[int, ...]]]:
 
 def weights_from_tensors(j: dict, tensors: Mapping[str, torch.Tensor]) -> ModelWeights:
     cfg = config_from_json(j)
-    out: dict[str, QTensor] = {}
-    for src, dst, kind, shape in tensor_names(cfg):
-        if src not in tensors:
-            raise KeyError(f"tensor '{src}' is missing from the checkpoint")
-        x = tensors[src]
-        if tuple(x.shape) != shape:
-            raise ValueError(f"tensor '{src}' has shape {tuple(x.shape)}, the configuration says {shape}")
-        if kind == "mat":
-            out[dst] = qtensor_from_float(x.float().contiguous(), GGMLType.F32 if x.dtype == torch.float32 else GGMLType.BF16)
-        else:
-            out[dst] = qtensor_from_float((1.0 + x.float() if kind == "gain" else x.float()).contiguous(), GGMLType.F32)
-    return ModelWeights(cfg, out, {})
+    return named_weights(cfg, tensor_names(cfg), tensors)

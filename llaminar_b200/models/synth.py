@@ -57,13 +57,13 @@ def synthesize(cfg: ModelConfig, recipe: QuantRecipe | str = "Q8_0", seed: int =
             x = torch.full((n,), value, device=dev, dtype=torch.float32)
         tensors[name] = qtensor_from_float(x, GGMLType.F32)
 
-    if cfg.is_latent:
-        from .pozivik import tensor_names
-        for _, name, kind, shape in tensor_names(cfg):
+    if cfg.has_mixers:
+        from .config import family_of
+        for _, name, kind, shape in family_of(cfg.arch).tensor_names(cfg):
             if kind == "mat":
                 mat(name, *shape, layer=int(name.split(".")[1]) if name.startswith("blk.") else None)
-            else:
-                vec(name, shape[0], None if "sinks" in name else 1.0)
+            else:                                            # norm gains and layer scales 1, sinks near 0, forget gates open
+                vec(name, shape[0], None if "sinks" in name else 4.0 if name.endswith("lstm_f.bias") else 1.0)
         return ModelWeights(cfg, tensors, byte_tokenizer_metadata(cfg.vocab_size) if with_tokenizer else {})
     d, qd, kvd = cfg.d_model, cfg.q_dim, cfg.kv_dim
     mat("token_embd.weight", cfg.vocab_size, d)

@@ -9,6 +9,7 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass
+from typing import Mapping
 
 import torch
 
@@ -139,9 +140,26 @@ class ModelWeights:
 
 def _directory_readers() -> dict:
     """config.json "architecture" -> function(config dict, {name: tensor}) -> ModelWeights."""
-    from . import pozivik
-    return {pozivik.ARCHITECTURE: pozivik.weights_from_tensors}
+    from . import pozivik, zogepel
+    return {m.ARCHITECTURE: m.weights_from_tensors for m in (pozivik, zogepel)}
 
 
 def qtensor_from_float(x: torch.Tensor, qtype: GGMLType) -> QTensor:
     return QTensor(GGMLType(qtype), tuple(x.shape), quantize(x, qtype))
+
+
+def named_weights(cfg: ModelConfig, names: list[tuple[str, str, str, tuple[int, ...]]], tensors: Mapping[str, torch.Tensor]) -> ModelWeights:
+    """A checkpoint's tensors under the package's names.  ``names``: (checkpoint name, package name, kind, shape), kind "mat" a
+    matrix, "vec" a vector kept as it is, "gain" a zero-centred norm gain (stored as 1 + w)."""
+    out: dict[str, QTensor] = {}
+    for src, dst, kind, shape in names:
+        if src not in tensors:
+            raise KeyError(f"tensor '{src}' is missing from the checkpoint")
+        x = tensors[src]
+        if tuple(x.shape) != shape:
+            raise ValueError(f"tensor '{src}' has shape {tuple(x.shape)}, the configuration says {shape}")
+        if kind == "mat":
+            out[dst] = qtensor_from_float(x.float().contiguous(), GGMLType.F32 if x.dtype == torch.float32 else GGMLType.BF16)
+        else:
+            out[dst] = qtensor_from_float((1.0 + x.float() if kind == "gain" else x.float()).contiguous(), GGMLType.F32)
+    return ModelWeights(cfg, out, {})

@@ -15,10 +15,14 @@ from pathlib import Path
 NAME = "llaminar_b200_ops"
 CSRC = Path(__file__).resolve().parent / "csrc"
 BUILD_DIR = Path(__file__).resolve().parent / "_build"
-LATENT = "llaminar_b200_latent"       # kernels of latent-attention models, built and loaded on their own
+# kernels of models with unquantised matrices, built and loaded on their own: shared ones, latent attention, and the mixers with
+# grouped-query attention and recurrent state
+DENSE, LATENT, MIXERS = "llaminar_b200_dense", "llaminar_b200_latent", "llaminar_b200_mixers"
 SOURCES = {
     NAME: ["binding.cpp", "gemv.cu", "gemv_stream.cu", "gemm_tc.cu", "gemm_tc_small.cu", "attention.cu", "attention_tc.cu", "ops.cu", "gdn.cu", "moe_ep.cu", "no_alloc.cu"],
-    LATENT: ["latent_binding.cpp", "latent_attention.cu", "latent_tc.cu", "dense_ops.cu"],
+    DENSE: ["dense_binding.cpp", "dense_ops.cu"],
+    LATENT: ["latent_binding.cpp", "latent_attention.cu", "latent_tc.cu"],
+    MIXERS: ["mixers_binding.cpp", "mixers.cu", "attention.cu", "attention_tc.cu"],
 }
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xptxas", "-v"]

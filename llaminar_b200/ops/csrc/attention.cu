@@ -137,8 +137,9 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
     const int G = p.n_heads / p.n_kv_heads, R = p.rows_per_seq;
     const int seq_len = p.seq_lens[seq];
     const int n_pages = (seq_len + PAGE - 1) / PAGE;
-    const int per = (n_pages + gridDim.y - 1) / gridDim.y;
-    const int pg0 = split * per, pg1 = min(n_pages, pg0 + per);
+    const int first_page = p.window > 0 ? max(0, seq_len - (R - 1) - p.window) / PAGE : 0;      // of the first key that any row sees
+    const int per = (n_pages - first_page + gridDim.y - 1) / gridDim.y;
+    const int pg0 = first_page + split * per, pg1 = min(n_pages, pg0 + per);
     const int* btab = p.block_table + (size_t)seq * p.max_pages;
     using SM = DecodeSmem<D, Q8>;
     const uint32_t wbase = smem_u32(smem) + warp * SM::PER_WARP;
@@ -171,6 +172,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
     // causal limit per MMA row: verify row r sees keys < seq_len - (R - 1 - r)
     const int lim0 = (i0 < G * R) ? seq_len - (R - 1 - i0 / G) : 0;
     const int lim1 = (i1 < G * R) ? seq_len - (R - 1 - i1 / G) : 0;
+    const int low0 = p.window > 0 ? lim0 - p.window : 0, low1 = p.window > 0 ? lim1 - p.window : 0;     // ... and >= low
 
     float o[D / 8][4];
 #pragma unroll
@@ -269,8 +271,8 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = key0 + nb * 8 + e;
-                s[nb][e] = key < lim0 ? s[nb][e] * sl2 : -INFINITY;
-                s[nb][2 + e] = key < lim1 ? s[nb][2 + e] * sl2 : -INFINITY;
+                s[nb][e] = key < lim0 && key >= low0 ? s[nb][e] * sl2 : -INFINITY;
+                s[nb][2 + e] = key < lim1 && key >= low1 ? s[nb][2 + e] * sl2 : -INFINITY;
                 mx0 = fmaxf(mx0, s[nb][e]);
                 mx1 = fmaxf(mx1, s[nb][2 + e]);
             }
@@ -326,6 +328,15 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
     const int rows = G * R;
     // thread t handles column t % D of rows t / D, t / D + 128 / D, ...
     const int col = threadIdx.x % D;
+    // quotient of one output value: the sink's share of the denominator, the output gate
+    auto store = [&](int i, float m, float l, float acc) {
+        const int r = i / G, head = kvh * G + i % G;
+        const size_t row = (size_t)seq * R + r;
+        if (p.sink) l += exp2f(p.sink[head] * 1.4426950408889634f - m);
+        float v = l > 0.f ? acc / l : 0.f;
+        if (p.gate) v *= 1.f / (1.f + __expf(-p.gate[row * p.gate_row + (size_t)head * D + col]));
+        p.out[(row * p.n_heads + head) * D + col] = __float2bfloat16(v);
+    };
     const size_t part_base = (((size_t)seq * p.n_kv_heads + kvh) * gridDim.y + split) * 16;
     for (int i = threadIdx.x / D; i < rows; i += 128 / D) {
         float m = -INFINITY;
@@ -340,8 +351,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
             acc += c * s_o[(w * 16 + i) * D + col];
         }
         if (gridDim.y == 1) {
-            const int r = i / G, g = i % G;
-            p.out[((size_t)(seq * R + r) * p.n_heads + kvh * G + g) * D + col] = __float2bfloat16(l > 0.f ? acc / l : 0.f);
+            store(i, m, l, acc);
         } else {
             p.part_o[(part_base + i) * D + col] = acc;
             if (col == 0) { p.part_ml[(part_base + i) * 2] = m; p.part_ml[(part_base + i) * 2 + 1] = l; }
@@ -372,8 +382,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
             l += c * __ldcg(&p.part_ml[(pb + s * 16 + i) * 2 + 1]);
             acc += c * __ldcg(&p.part_o[(pb + s * 16 + i) * D + col]);
         }
-        const int r = i / G, g = i % G;
-        p.out[((size_t)(seq * R + r) * p.n_heads + kvh * G + g) * D + col] = __float2bfloat16(l > 0.f ? acc / l : 0.f);
+        store(i, m, l, acc);
     }
 }
 
@@ -446,7 +455,10 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
             qa[ks][3] = q1 ? *reinterpret_cast<const uint32_t*>(q1 + d0 + 8) : 0u;
         }
     }
-    const int lim0 = ctx + r0 + 1, lim1 = ctx + r1 + 1;           // row sees keys < lim
+    const int lim0 = ctx + r0 + 1, lim1 = ctx + r1 + 1;           // row sees keys < lim, and >= low
+    const int low0 = p.window > 0 ? lim0 - p.window : 0, low1 = p.window > 0 ? lim1 - p.window : 0;
+    const int first_page = p.window > 0 ? max(0, ctx + qt0 + 1 - p.window) / PAGE : 0;
+    const int w_low = p.window > 0 ? ctx + qt0 + warp * 16 + 1 - p.window : 0;       // keys before it: none for this warp
     const int kv_end = min(ctx + q_len, ctx + qt0 + 64);          // keys needed by this q tile
     const int n_pages = (kv_end + PAGE - 1) / PAGE;
 
@@ -474,18 +486,20 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
         }
         cp_async_commit();
     };
-    issue(0, 0);
-    for (int pg = 0; pg < n_pages; ++pg) {
+    issue(first_page, first_page & 1);
+    for (int pg = first_page; pg < n_pages; ++pg) {
         const int stage = pg & 1;
         issue(pg + 1, stage ^ 1);
         cp_async_wait<1>();
         __syncthreads();
         const uint32_t kb = sbase + stage * 2 * TILE, vb = kb + TILE;
-        const bool need_mask = (pg + 1) * PAGE > ctx + qt0 + warp * 16 + 1;   // page reaches past this warp's first row
+        // page reaches past this warp's first row, or starts before its last row's window
+        const bool need_mask = (pg + 1) * PAGE > ctx + qt0 + warp * 16 + 1 || pg * PAGE < w_low + 15;
 #pragma unroll
         for (int sub = 0; sub < PAGE / 16; ++sub) {
             const int key_base = pg * PAGE + sub * 16;
             if (key_base >= ctx + qt0 + warp * 16 + 16) break;                 // fully masked for every row of this warp
+            if (key_base + 16 <= w_low) continue;
             float s[2][4];
             qk_16keys<D>(qa, kb + sub * 16 * D * 2, lane, s);
             const int key0 = key_base + (lane & 3) * 2;
@@ -495,8 +509,8 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = key0 + nb * 8 + e;
-                    s[nb][e] = (!need_mask || key < lim0) ? s[nb][e] * sl2 : -INFINITY;
-                    s[nb][2 + e] = (!need_mask || key < lim1) ? s[nb][2 + e] * sl2 : -INFINITY;
+                    s[nb][e] = (!need_mask || (key < lim0 && key >= low0)) ? s[nb][e] * sl2 : -INFINITY;
+                    s[nb][2 + e] = (!need_mask || (key < lim1 && key >= low1)) ? s[nb][2 + e] * sl2 : -INFINITY;
                     mx0 = fmaxf(mx0, s[nb][e]);
                     mx1 = fmaxf(mx1, s[nb][2 + e]);
                 }
@@ -529,14 +543,26 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
     cp_async_wait<0>();
     l0 += __shfl_xor_sync(0xffffffffu, l0, 1); l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
     l1 += __shfl_xor_sync(0xffffffffu, l1, 1); l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+    if (p.sink) {
+        const float sk = p.sink[head] * 1.4426950408889634f;
+        l0 += exp2f(sk - m0);
+        l1 += exp2f(sk - m1);
+    }
     const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
+    auto store = [&](int r, int col, float a, float b) {
+        if (r >= q_len) return;
+        if (p.gate) {
+            const uint32_t g = *reinterpret_cast<const uint32_t*>(p.gate + (size_t)(q_start + r) * p.gate_row + head * D + col);
+            a *= 1.f / (1.f + __expf(-bf16_lo(g)));
+            b *= 1.f / (1.f + __expf(-bf16_hi(g)));
+        }
+        *reinterpret_cast<uint32_t*>(p.out + ((size_t)(q_start + r) * p.n_heads + head) * D + col) = pack_bf16(a, b);
+    };
 #pragma unroll
     for (int n = 0; n < D / 8; ++n) {
         const int col = n * 8 + (lane & 3) * 2;
-        if (r0 < q_len)
-            *reinterpret_cast<uint32_t*>(p.out + ((size_t)(q_start + r0) * p.n_heads + head) * D + col) = pack_bf16(o[n][0] * inv0, o[n][1] * inv0);
-        if (r1 < q_len)
-            *reinterpret_cast<uint32_t*>(p.out + ((size_t)(q_start + r1) * p.n_heads + head) * D + col) = pack_bf16(o[n][2] * inv1, o[n][3] * inv1);
+        store(r0, col, o[n][0] * inv0, o[n][1] * inv0);
+        store(r1, col, o[n][2] * inv1, o[n][3] * inv1);
     }
 }
 

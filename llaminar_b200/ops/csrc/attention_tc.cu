@@ -81,7 +81,8 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
     const int ctx = p.ctx_lens[seq];                       // tokens already in the cache before this chunk
     const int rows = min(BQ, q_len - q0);
     const int kv_end = ctx + q0 + rows;                    // keys this query tile can see
-    const int nt = (kv_end + BK - 1) / BK, n_pages = (kv_end + PAGE - 1) / PAGE;
+    const int tile0 = p.window > 0 ? max(0, ctx + q0 + 1 - p.window) / BK : 0;          // tile of the first key that the first row sees
+    const int nt = (kv_end + BK - 1) / BK - tile0, n_pages = (kv_end + PAGE - 1) / PAGE;
     const int* btab = p.block_table + (size_t)seq * p.max_pages;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t sQ = base + OFF_Q, sK = base + OFF_K, sVT = base + OFF_VT, sP = base + OFF_P, sVS = base + OFF_VS;
@@ -111,7 +112,8 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
         // scheduler and halves the work of each)
         const int row = tid & 127, half = tid >> 7, q4 = warp & 3;
         const bool valid = row < rows;
-        const int lim = ctx + min(q0 + row, q_len - 1) + 1;           // this row sees keys < lim
+        const int lim = ctx + min(q0 + row, q_len - 1) + 1;           // this row sees keys < lim, and >= low
+        const int low = p.window > 0 ? lim - p.window : 0;
         const uint32_t t_lane = tmem + ((uint32_t)(q4 * 32) << 16) + half * 64;
         const float sl2 = p.scale * 1.4426950408889634f;
         constexpr int HD = D / 2;
@@ -135,18 +137,19 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             const int b = j & 1;
             if (!mbar_wait_warp(bar(S_FULL + b), (j >> 1) & 1, abort_flag)) return false;
             tc_fence_after();
-            const int key0 = j * BK + half * 64;
+            const int key0 = (tile0 + j) * BK + half * 64;
             const uint32_t t_s = t_lane + b * 128;
             tmem_ld32_issue(t_s, ra);
             tmem_ld32_issue(t_s + 32, rb);
             tmem_wait_ld(ra);
             tmem_wait_ld(rb);
             float mx = -INFINITY;
-            if (key0 + 64 > lim) {
+            if (key0 + 64 > lim || key0 < low) {
 #pragma unroll
                 for (int i = 0; i < 32; ++i) {
-                    const float s0 = key0 + i >= lim ? -INFINITY : __uint_as_float(ra[i]);
-                    const float s1 = key0 + 32 + i >= lim ? -INFINITY : __uint_as_float(rb[i]);
+                    const int k0 = key0 + i, k1 = key0 + 32 + i;
+                    const float s0 = k0 >= lim || k0 < low ? -INFINITY : __uint_as_float(ra[i]);
+                    const float s1 = k1 >= lim || k1 < low ? -INFINITY : __uint_as_float(rb[i]);
                     mx = fmaxf(mx, fmaxf(s0, s1));
                 }
             } else {
@@ -188,8 +191,8 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             if (j < nt) ok = pass1(j);
             if (ok && j > 0) ok = fold(j - 1);
             if (!ok || j == nt) break;
-            const int key0 = j * BK + half * 64;
-            const bool need_mask = key0 + 64 > lim;
+            const int key0 = (tile0 + j) * BK + half * 64;
+            const bool need_mask = key0 + 64 > lim || key0 < low;
             const uint32_t t_s = t_lane + b * 128;
             tmem_ld32_issue(t_s, ra);
             tmem_ld32_issue(t_s + 32, rb);
@@ -202,8 +205,8 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
                         const int key = key0 + c * 32 + i;
-                        const float p0 = key >= lim ? 0.f : ex2(__uint_as_float(r[i]) * sl2 - mb);
-                        const float p1 = key + 1 >= lim ? 0.f : ex2(__uint_as_float(r[i + 1]) * sl2 - mb);
+                        const float p0 = key >= lim || key < low ? 0.f : ex2(__uint_as_float(r[i]) * sl2 - mb);
+                        const float p1 = key + 1 >= lim || key + 1 < low ? 0.f : ex2(__uint_as_float(r[i + 1]) * sl2 - mb);
                         sum += p0 + p1;
                         w[i >> 1] = pack_bf16(p0, p1);
                     }
@@ -237,12 +240,22 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             ok = pair_meet();
         }
         if (ok && valid) {
-            const float lt = l + s_xchg[half ^ 1][row];
+            float lt = l + s_xchg[half ^ 1][row];
+            if (p.sink) lt += exp2f(p.sink[head] * 1.4426950408889634f - m);
             const float inv = lt > 0.f ? 1.f / lt : 0.f;
             __nv_bfloat16* dst = p.out + ((size_t)(q_start + q0 + row) * p.n_heads + head) * D + half * HD;
 #pragma unroll
             for (int u = 0; u < HD / 8; ++u) {
                 uint4 v;
+                if (p.gate) {
+                    const uint4 g = *reinterpret_cast<const uint4*>(p.gate + (size_t)(q_start + q0 + row) * p.gate_row + head * D + half * HD + 8 * u);
+                    const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        o[8 * u + 2 * i] *= __fdividef(1.f, 1.f + __expf(-bf16_lo(gw[i])));
+                        o[8 * u + 2 * i + 1] *= __fdividef(1.f, 1.f + __expf(-bf16_hi(gw[i])));
+                    }
+                }
                 v.x = pack_bf16(o[8 * u] * inv, o[8 * u + 1] * inv); v.y = pack_bf16(o[8 * u + 2] * inv, o[8 * u + 3] * inv);
                 v.z = pack_bf16(o[8 * u + 4] * inv, o[8 * u + 5] * inv); v.w = pack_bf16(o[8 * u + 6] * inv, o[8 * u + 7] * inv);
                 *reinterpret_cast<uint4*>(dst + 8 * u) = v;
@@ -272,7 +285,7 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             if (j < nt) {
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
-                    const __nv_bfloat16* kp = p.kv + ((page_of(2 * j + half) * 2 + 0) * p.n_kv_heads + kvh) * (size_t)(PAGE * D);
+                    const __nv_bfloat16* kp = p.kv + ((page_of(2 * (tile0 + j) + half) * 2 + 0) * p.n_kv_heads + kvh) * (size_t)(PAGE * D);
                     for (int idx = lt; idx < PAGE * 16; idx += N_LOADERS) {
                         const int r = idx >> 4, u = idx & 15;
                         cp_async16(atom_addr(sK + ((j & 1) * 2 + (u >> 3)) * ATOM, half * PAGE + r, u & 7), kp + r * D + u * 8);
@@ -285,7 +298,7 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             if (j < nt) {
 #pragma unroll
                 for (int half = 0; half < 2; ++half) {
-                    const __nv_bfloat16* vp = p.kv + ((page_of(2 * j + half) * 2 + 1) * p.n_kv_heads + kvh) * (size_t)(PAGE * D);
+                    const __nv_bfloat16* vp = p.kv + ((page_of(2 * (tile0 + j) + half) * 2 + 1) * p.n_kv_heads + kvh) * (size_t)(PAGE * D);
                     for (int idx = lt; idx < PAGE * 16; idx += N_LOADERS) {
                         const int r = idx >> 4, u = idx & 15;
                         cp_async16(stage_addr(sVS, half * PAGE + r, u), vp + r * D + u * 8);

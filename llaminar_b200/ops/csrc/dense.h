@@ -1,0 +1,59 @@
+// Launchers of what models with unquantised matrices share: fused norms of the residual stream, activations, rotary angles and
+// the small-batch matrix product.  `f32` selects the 32-bit build of a kernel (activations as float) instead of the bf16 one;
+// residual stream, norms and angles are 32-bit in both.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stddef.h>
+
+namespace llm {
+
+// v = y[row(t)], or half the sum of RMSNorm(y[t]) * w_y and RMSNorm(y2[t]) * w_y2
+// h[t] = (add ? h[t] : 0) + (norm of v) * w_post, or v * factor ; xn[t] = (norm of h[t]) * w_next ; copies of h[t] in the activation type
+struct ResidNormParams {
+    const void* y;                 // activation type; nullptr: h is only read
+    size_t y_stride;
+    const int* y_rows;             // optional gather (embedding lookup): row(t) = y_rows[t]
+    int n_y_rows;                  // rows of y (bounds-check build)
+    const void* y2;                // optional second sublayer output [T, d]
+    size_t y2_stride;
+    const float *w_y, *w_y2;       // [d], with y2
+    const float* w_post;           // [d]; nullptr: no norm, v * factor
+    float factor;
+    int center_post, center_next;  // the norm takes the mean off first
+    float* h;                      // [T, d]
+    int add;
+    const float* w_next;           // optional [d]
+    void* xn;                      // [T, d]
+    void *copy0, *copy1;           // optional
+    size_t copy_stride;
+    int d;
+    float eps;
+};
+cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cudaStream_t st);
+
+// Activations behind a product.  GELU_MUL: gelu_tanh(first half of the columns) * second half; RELU2: squared relu;
+// GELU_SIDE: gelu_tanh times the token's row of a table (columns [0, side_cols), zero behind).
+enum Activation : int { ACT_NONE = 0, ACT_GELU_MUL = 1, ACT_RELU2 = 2, ACT_GELU_SIDE = 3 };
+struct SideTable { const void* table; size_t row; int cols, n_rows; const int* tokens; };
+// act[t, 0..n) from x[t, 0..n) (GELU_MUL: 2n columns)
+cudaError_t launch_activate(const void* x, void* act, int rows, int n, int kind, const SideTable& side, bool f32, cudaStream_t st);
+
+// out[t, i] = magnitude * (cos, sin)(positions[t] * freqs[i])
+cudaError_t launch_rope_angles(const int* positions, const double* freqs, double magnitude, float2* out, int rows, int half, cudaStream_t st);
+
+// out[z][m, :] = act(x[z][m, :] W[z]^T) for up to 8 rows, bf16 weights.  GELU_MUL: W holds 2n rows.
+struct GemvDenseParams {
+    const __nv_bfloat16* w; size_t w_z; int ldw;
+    const __nv_bfloat16* x; size_t x_row, x_z;
+    void* out; size_t o_row, o_z;
+    int n, k, m, z;
+    bool out_f32;
+    int act;                       // with one: out is bf16
+    SideTable side;
+};
+cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st);
+
+int bounds_status_dense(bool reset);
+
+}  // namespace llm

@@ -1,0 +1,115 @@
+// Python bindings of what models with unquantised matrices share (dense_ops.cu): an extension of its own, so that a process that
+// serves only such a model compiles and loads nothing else.
+#include "binding_util.h"
+#include "dense.h"
+#include "launch.h"
+
+namespace {
+using namespace llm_binding;
+
+void resid_norm(const OptTensor& y, const OptTensor& y_rows, const OptTensor& w_post, const Tensor& h, bool add, const OptTensor& w_next,
+                const OptTensor& xn, const OptTensor& copy0, const OptTensor& copy1, double eps, const OptTensor& y2, const OptTensor& w_y,
+                const OptTensor& w_y2, double factor, bool center_post, bool center_next) {
+    llm::ResidNormParams p = {};
+    want(h, torch::kFloat32, "h");
+    const int64_t T = h.size(0), d = h.size(1);
+    if (T == 0) return;
+    bool f32 = false, typed = false;
+    auto elem = [&](const Tensor& t, const char* name) {
+        const bool f = is_f32(t, name);
+        TORCH_CHECK(!typed || f == f32, name, " has another element type than the other activations");
+        f32 = f; typed = true;
+        TORCH_CHECK(t.dim() == 2 && t.size(1) == d && t.stride(1) == 1, name, " must be rows of ", d, " values");
+    };
+    if (y) {
+        elem(*y, "y");
+        p.y = y->data_ptr(); p.y_stride = y->stride(0);
+        if (w_post) p.w_post = floats(*w_post, d, "w_post");
+        p.n_y_rows = y->size(0);
+        if (y_rows) {
+            p.y_rows = ints(*y_rows, "y_rows");
+            TORCH_CHECK(y_rows->numel() == T, "y_rows must name one row per token");
+        } else {
+            TORCH_CHECK(y->size(0) == T, "y must have as many rows as h");
+        }
+        if (y2) {
+            elem(*y2, "y2");
+            TORCH_CHECK(!y_rows && y2->size(0) == T, "y2 must have as many rows as h");
+            p.y2 = y2->data_ptr(); p.y2_stride = y2->stride(0);
+            p.w_y = floats(w_y.value(), d, "w_y"); p.w_y2 = floats(w_y2.value(), d, "w_y2");
+        }
+    }
+    p.h = h.data_ptr<float>(); p.add = add;
+    if (w_next) {
+        elem(xn.value(), "xn");
+        TORCH_CHECK(xn->is_contiguous() && xn->size(0) == T, "xn must be contiguous");
+        p.w_next = floats(*w_next, d, "w_next"); p.xn = xn->data_ptr();
+    }
+    if (copy0) { elem(*copy0, "copy0"); TORCH_CHECK(copy0->size(0) == T, "copy0 rows"); p.copy0 = copy0->data_ptr(); p.copy_stride = copy0->stride(0); }
+    if (copy1) {
+        elem(*copy1, "copy1");
+        TORCH_CHECK(copy1->size(0) == T && (!copy0 || copy1->stride(0) == copy0->stride(0)), "copy1 must have copy0's strides");
+        p.copy1 = copy1->data_ptr(); p.copy_stride = copy1->stride(0);
+    }
+    p.d = d; p.eps = eps; p.factor = factor; p.center_post = center_post; p.center_next = center_next;
+    check(llm::launch_resid_norm(p, T, f32, stream()), "resid_norm");
+}
+
+// table [vocabulary, columns]: columns [first, first + cols) belong to this layer
+llm::SideTable side_table(const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens, int64_t rows, bool f32) {
+    llm::SideTable s = {};
+    if (!table) return s;
+    want_like(*table, f32, "side table");
+    TORCH_CHECK(table->dim() == 2 && table->stride(1) == 1 && first >= 0 && first + cols <= table->size(1), "side table columns");
+    TORCH_CHECK(tokens && tokens->numel() == rows, "one token per row");
+    s.table = static_cast<const char*>(table->data_ptr()) + first * table->element_size();
+    s.row = table->stride(0); s.cols = cols; s.n_rows = table->size(0); s.tokens = ints(*tokens, "tokens");
+    return s;
+}
+
+void activate(const Tensor& x, const Tensor& act, int64_t kind, const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens) {
+    const bool f32 = is_f32(x, "x");
+    want_like(act, f32, "act");
+    TORCH_CHECK(x.is_contiguous() && act.is_contiguous() && x.size(0) == act.size(0), "activation rows");
+    TORCH_CHECK(x.size(1) == act.size(1) * (kind == llm::ACT_GELU_MUL ? 2 : 1), "activation columns");
+    TORCH_CHECK((kind == llm::ACT_GELU_SIDE) == table.has_value(), "a side table goes with the side activation");
+    if (x.size(0) == 0) return;
+    check(llm::launch_activate(x.data_ptr(), act.data_ptr(), x.size(0), act.size(1), kind, side_table(table, first, cols, tokens, x.size(0), f32), f32, stream()), "activate");
+}
+
+void rope_angles(const Tensor& positions, const Tensor& freqs, double magnitude, const Tensor& out) {
+    want(freqs, torch::kFloat64, "freqs");
+    const int rows = positions.numel(), half = freqs.numel();
+    angle_ptr(out, rows);
+    TORCH_CHECK(out.size(1) == half, "angles must have one column per frequency");
+    check(llm::launch_rope_angles(ints(positions, "positions"), freqs.data_ptr<double>(), magnitude, reinterpret_cast<float2*>(out.data_ptr<float>()),
+                                  rows, half, stream()), "rope_angles");
+}
+
+// w [z, n, k] (GELU_MUL: [z, 2n, k]), x [z, m, k], out [z, m, n]; the last dimension of each is dense
+void gemv_dense(const Tensor& w, const Tensor& x, const Tensor& out, int64_t act, const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens) {
+    TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && x.scalar_type() == torch::kBFloat16, "gemv_dense takes bf16 operands");
+    TORCH_CHECK(w.dim() == 3 && x.dim() == 3 && out.dim() == 3 && w.stride(2) == 1 && x.stride(2) == 1 && out.stride(2) == 1, "gemv_dense layouts");
+    llm::GemvDenseParams p = {};
+    p.z = w.size(0); p.n = act == llm::ACT_GELU_MUL ? w.size(1) / 2 : w.size(1); p.k = w.size(2); p.m = x.size(1);
+    TORCH_CHECK(x.size(0) == p.z && out.size(0) == p.z && x.size(2) == p.k && out.size(1) == p.m && out.size(2) == p.n, "gemv_dense shapes");
+    p.out_f32 = is_f32(out, "out"); p.act = act;
+    p.w = reinterpret_cast<const __nv_bfloat16*>(w.data_ptr()); p.w_z = w.stride(0); p.ldw = w.stride(1);
+    p.x = reinterpret_cast<const __nv_bfloat16*>(x.data_ptr()); p.x_row = x.stride(1); p.x_z = x.stride(0);
+    p.out = out.data_ptr(); p.o_row = out.stride(1); p.o_z = out.stride(0);
+    TORCH_CHECK(reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "gemv_dense operands must be 16-byte aligned");
+    TORCH_CHECK((act == llm::ACT_GELU_SIDE) == table.has_value(), "a side table goes with the side activation");
+    p.side = side_table(table, first, cols, tokens, p.m, false);
+    check(llm::launch_gemv_dense(p, stream()), "gemv_dense");
+}
+
+}  // namespace
+
+PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
+    m.def("resid_norm", &resid_norm);
+    m.def("activate", &activate);
+    m.def("rope_angles", &rope_angles);
+    m.def("gemv_dense", &gemv_dense);
+    m.def("set_pdl", [](bool on) { llm::pdl_enabled() = on; });
+    m.def("bounds_status", [](bool reset) { return llm::bounds_status_dense(reset); });
+}

@@ -1,7 +1,7 @@
-// Fused norms of the residual stream, the gated activation, rotary angles and the small-batch matrix product of models whose
-// matrices are stored as bf16 (or float, 32-bit mode).
+// Fused norms of the residual stream, activations, rotary angles and the small-batch matrix product of models whose matrices are
+// stored as bf16 (or float, 32-bit mode).
 #include "common.cuh"
-#include "latent.h"
+#include "dense.h"
 #include "launch.h"
 
 namespace llm {
@@ -51,7 +51,7 @@ template <> struct Vec4<__nv_bfloat16> {
 // VEC 4 needs d and every row stride to be multiples of 4 elements; VEC 1 takes any size.
 template <class T, int VEC, int THREADS>
 __global__ void __launch_bounds__(THREADS) resid_norm_kernel(const ResidNormParams p) {
-    extern __shared__ __align__(16) float row[];              // [d]
+    extern __shared__ __align__(16) float row[];              // [d], with y2 [2][d]
     __shared__ float red[THREADS / 32];
     pdl_trigger();
     pdl_wait();
@@ -69,31 +69,65 @@ __global__ void __launch_bounds__(THREADS) resid_norm_kernel(const ResidNormPara
     auto store_f = [](float* s, const float (&v)[VEC]) {
         if constexpr (VEC == 4) Vec4<float>::store(s, v); else *s = v[0];
     };
-    float inv_y = 0.f;
+    // 1 / root mean square of the row, after its mean (returned in `mean`, 0 unless `center`) is taken off
+    auto norm_of = [&](const float* r, float sum, float ss, bool center, float& mean) {
+        mean = 0.f;
+        if (center) {
+            mean = block_sum<THREADS>(sum, red) / (float)p.d;
+            ss = 0.f;
+            for (int i = threadIdx.x * VEC; i < p.d; i += THREADS * VEC) {
+                float v[VEC];
+                load_f(r + i, v);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) ss += (v[j] - mean) * (v[j] - mean);
+            }
+        }
+        return 1.f / sqrtf(block_sum<THREADS>(ss, red) / (float)p.d + p.eps);
+    };
+    float inv_y = 0.f, mean_y = 0.f;
     const T* y = nullptr;
     if (p.y) {
         const size_t r = p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[t], p.n_y_rows) : t;
         y = static_cast<const T*>(p.y) + r * p.y_stride;
-        float ss = 0.f;
+        const T* y2 = p.y2 ? static_cast<const T*>(p.y2) + t * p.y2_stride : nullptr;
+        float ss = 0.f, ss2 = 0.f, sum = 0.f;
         for (int i = threadIdx.x * VEC; i < p.d; i += THREADS * VEC) {
             float v[VEC];
             load_t(y + i, v);
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
+            for (int j = 0; j < VEC; ++j) { ss += v[j] * v[j]; sum += v[j]; }
             store_f(row + i, v);
+            if (y2) {
+                load_t(y2 + i, v);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) ss2 += v[j] * v[j];
+                store_f(row + p.d + i, v);
+            }
         }
-        ss = block_sum<THREADS>(ss, red);
-        inv_y = 1.f / sqrtf(ss / (float)p.d + p.eps);
+        if (y2) {
+            const float a = 0.5f / sqrtf(block_sum<THREADS>(ss, red) / (float)p.d + p.eps), b = 0.5f / sqrtf(block_sum<THREADS>(ss2, red) / (float)p.d + p.eps);
+            ss = sum = 0.f;
+            for (int i = threadIdx.x * VEC; i < p.d; i += THREADS * VEC) {      // every thread reads back what it wrote
+                float v[VEC], u[VEC], w[VEC], x[VEC];
+                load_f(row + i, v); load_f(row + p.d + i, u); load_f(p.w_y + i, w); load_f(p.w_y2 + i, x);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) { v[j] = v[j] * a * w[j] + u[j] * b * x[j]; ss += v[j] * v[j]; sum += v[j]; }
+                store_f(row + i, v);
+            }
+        }
+        inv_y = p.w_post ? norm_of(row, sum, ss, p.center_post, mean_y) : p.factor;
     }
-    float ss = 0.f;
+    float ss = 0.f, sum = 0.f;
     for (int i = threadIdx.x * VEC; i < p.d; i += THREADS * VEC) {
         float v[VEC];
         if (y) {
             float w[VEC];
             load_f(row + i, v);
-            load_f(p.w_post + i, w);
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) v[j] = v[j] * inv_y * w[j];
+            for (int j = 0; j < VEC; ++j) w[j] = 1.f;
+            if (p.w_post) load_f(p.w_post + i, w);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[j] = (v[j] - mean_y) * inv_y * w[j];
             if (p.add) {
                 float a[VEC];
                 load_f(h + i, a);
@@ -108,40 +142,49 @@ __global__ void __launch_bounds__(THREADS) resid_norm_kernel(const ResidNormPara
         if (p.copy1) store_t(static_cast<T*>(p.copy1) + t * p.copy_stride + i, v);
         store_f(row + i, v);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
+        for (int j = 0; j < VEC; ++j) { ss += v[j] * v[j]; sum += v[j]; }
     }
     if (!p.w_next) return;
-    ss = block_sum<THREADS>(ss, red);
-    const float inv = 1.f / sqrtf(ss / (float)p.d + p.eps);
+    float mean;
+    const float inv = norm_of(row, sum, ss, p.center_next, mean);
     T* xn = static_cast<T*>(p.xn) + t * p.d;
     for (int i = threadIdx.x * VEC; i < p.d; i += THREADS * VEC) {
         float v[VEC], w[VEC];
         load_f(row + i, v);
         load_f(p.w_next + i, w);
 #pragma unroll
-        for (int j = 0; j < VEC; ++j) v[j] = v[j] * inv * w[j];
+        for (int j = 0; j < VEC; ++j) v[j] = (v[j] - mean) * inv * w[j];
         store_t(xn + i, v);
     }
 }
 
-template <class T>
-__global__ void __launch_bounds__(256) gelu_mul_kernel(const T* gu, T* act, int ff) {
+// value `i` of row `t` of the activation of `x`; `u`: the second half's value (GELU_MUL)
+template <int ACT, class T>
+LLM_DEVICE float activated(float x, float u, const SideTable& s, int t, int i) {
+    if (ACT == ACT_GELU_MUL) return gelu_tanh(x) * u;
+    if (ACT == ACT_RELU2) { x = fmaxf(x, 0.f); return x * x; }
+    if (ACT == ACT_GELU_SIDE) return i < s.cols ? gelu_tanh(x) * to_f(static_cast<const T*>(s.table)[(size_t)LLM_CHECK_INDEX(s.tokens[t], s.n_rows) * s.row + i]) : 0.f;
+    return x;
+}
+
+template <class T, int ACT>
+__global__ void __launch_bounds__(256) activate_kernel(const T* x, T* act, int n, const SideTable s) {
     pdl_trigger();
     pdl_wait();
-    const T* g = gu + (size_t)blockIdx.y * 2 * ff;
-    T* a = act + (size_t)blockIdx.y * ff;
-    if (ff % 4 == 0) {
-        const int i = (blockIdx.x * 256 + threadIdx.x) * 4;
-        if (i >= ff) return;
-        float x[4], u[4];
-        Vec4<T>::load(g + i, x);
-        Vec4<T>::load(g + ff + i, u);
+    const T* g = x + (size_t)blockIdx.y * n * (ACT == ACT_GELU_MUL ? 2 : 1);
+    T* a = act + (size_t)blockIdx.y * n;
+    const int i0 = (blockIdx.x * 256 + threadIdx.x) * 4;
+    if (n % 4 == 0) {
+        if (i0 >= n) return;
+        float v[4], u[4] = {};
+        Vec4<T>::load(g + i0, v);
+        if (ACT == ACT_GELU_MUL) Vec4<T>::load(g + n + i0, u);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) x[j] = gelu_tanh(x[j]) * u[j];
-        Vec4<T>::store(a + i, x);
+        for (int j = 0; j < 4; ++j) v[j] = activated<ACT, T>(v[j], u[j], s, blockIdx.y, i0 + j);
+        Vec4<T>::store(a + i0, v);
     } else {
-        for (int i = (blockIdx.x * 256 + threadIdx.x) * 4; i < min(ff, (int)(blockIdx.x * 256 + threadIdx.x + 1) * 4); ++i)
-            a[i] = from_f<T>(gelu_tanh(to_f(g[i])) * to_f(g[ff + i]));
+        for (int i = i0; i < min(n, i0 + 4); ++i)
+            a[i] = from_f<T>(activated<ACT, T>(to_f(g[i]), ACT == ACT_GELU_MUL ? to_f(g[n + i]) : 0.f, s, blockIdx.y, i));
     }
 }
 
@@ -159,14 +202,15 @@ __global__ void rope_angles_kernel(const int* positions, const double* freqs, do
 // Up to eight rows of x against 16 weight rows per warp on the tensor cores (the weights are the M operand).  Thread (g, t) of
 // a warp loads 8 consecutive k of weight rows g and g + 8 and of x row g in one 16-byte access each; since both operands use
 // the same assignment of k to MMA slots, its order does not matter and no operand passes through shared memory.  `wk` warps
-// share the K range of a row block and add up in shared memory.  GELU: a second set of weight rows (n further down) per block.
+// share the K range of a row block and add up in shared memory.  GELU_MUL: a second set of weight rows (n further down) per block.
 constexpr int SKINNY_WARPS = 8;
 LLM_DEVICE void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
-template <bool GELU, class TO>
+template <int ACT, class TO>
 __global__ void __launch_bounds__(32 * SKINNY_WARPS) gemv_dense_kernel(const GemvDenseParams p, int wk) {
+    constexpr bool GELU = ACT == ACT_GELU_MUL;
     __shared__ float s_acc[SKINNY_WARPS][GELU ? 2 : 1][16][9];
     pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
@@ -222,8 +266,9 @@ __global__ void __launch_bounds__(32 * SKINNY_WARPS) gemv_dense_kernel(const Gem
             v += s_acc[(c / 16) * wk + q][0][c % 16][m];
             if constexpr (GELU) v2 += s_acc[(c / 16) * wk + q][1][c % 16][m];
         }
-        // the two halves are rounded like the stored projection of the unfused form
-        if constexpr (GELU) v = gelu_tanh(__bfloat162float(__float2bfloat16(v))) * __bfloat162float(__float2bfloat16(v2));
+        // rounded like the stored projection of the unfused form
+        if constexpr (ACT != ACT_NONE)
+            v = activated<ACT, __nv_bfloat16>(__bfloat162float(__float2bfloat16(v)), __bfloat162float(__float2bfloat16(v2)), p.side, m, n);
         static_cast<TO*>(p.out)[(size_t)blockIdx.y * p.o_z + m * p.o_row + n] = from_f<TO>(v);
     }
 }
@@ -235,9 +280,9 @@ template <class K> cudaError_t raise_smem(K kernel, size_t bytes) {
 
 template <class T>
 cudaError_t resid_norm_any(const ResidNormParams& p, int rows, cudaStream_t st) {
-    const size_t smem = (size_t)p.d * 4;
+    const size_t smem = (size_t)p.d * (p.y2 ? 8 : 4);
     if (smem > 220 * 1024) return cudaErrorInvalidValue;
-    const bool vec = p.d % 4 == 0 && p.y_stride % 4 == 0 && p.copy_stride % 4 == 0;
+    const bool vec = p.d % 4 == 0 && p.y_stride % 4 == 0 && p.y2_stride % 4 == 0 && p.copy_stride % 4 == 0;
     auto go = [&](auto kernel, int threads) {
         cudaError_t e = raise_smem(kernel, smem);
         return e != cudaSuccess ? e : launch_pdl(kernel, dim3(rows), dim3(threads), smem, st, p);
@@ -253,11 +298,17 @@ cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cuda
     return f32 ? resid_norm_any<float>(p, rows, st) : resid_norm_any<__nv_bfloat16>(p, rows, st);
 }
 
-cudaError_t launch_gelu_mul(const void* gu, void* act, int rows, int ff, bool f32, cudaStream_t st) {
-    const dim3 grid((ff + 1023) / 1024, rows);
+cudaError_t launch_activate(const void* x, void* act, int rows, int n, int kind, const SideTable& side, bool f32, cudaStream_t st) {
+    const dim3 grid((n + 1023) / 1024, rows);
     if (rows > 65535) return cudaErrorInvalidValue;
-    if (f32) return launch_pdl(gelu_mul_kernel<float>, grid, dim3(256), 0, st, static_cast<const float*>(gu), static_cast<float*>(act), ff);
-    return launch_pdl(gelu_mul_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(gu), static_cast<__nv_bfloat16*>(act), ff);
+    auto go = [&](auto k32, auto k16) {
+        if (f32) return launch_pdl(k32, grid, dim3(256), 0, st, static_cast<const float*>(x), static_cast<float*>(act), n, side);
+        return launch_pdl(k16, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(act), n, side);
+    };
+    if (kind == ACT_GELU_MUL) return go(activate_kernel<float, ACT_GELU_MUL>, activate_kernel<__nv_bfloat16, ACT_GELU_MUL>);
+    if (kind == ACT_RELU2) return go(activate_kernel<float, ACT_RELU2>, activate_kernel<__nv_bfloat16, ACT_RELU2>);
+    if (kind == ACT_GELU_SIDE) return go(activate_kernel<float, ACT_GELU_SIDE>, activate_kernel<__nv_bfloat16, ACT_GELU_SIDE>);
+    return cudaErrorInvalidValue;
 }
 
 cudaError_t launch_rope_angles(const int* positions, const double* freqs, double magnitude, float2* out, int rows, int half, cudaStream_t st) {
@@ -267,7 +318,7 @@ cudaError_t launch_rope_angles(const int* positions, const double* freqs, double
 }
 
 cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st) {
-    if (p.m < 1 || p.m > 8 || p.n < 1 || p.k % 8 || p.ldw % 8 || p.w_z % 8 || p.x_row % 8 || p.x_z % 8 || (p.gelu && p.out_f32)) return cudaErrorInvalidValue;
+    if (p.m < 1 || p.m > 8 || p.n < 1 || p.k % 8 || p.ldw % 8 || p.w_z % 8 || p.x_row % 8 || p.x_z % 8 || (p.act != ACT_NONE && p.out_f32)) return cudaErrorInvalidValue;
     // split K until every warp has about eight blocks of 32 and the grid fills the machine
     const int blocks = (p.k + 31) / 32, tiles = (p.n + 15) / 16 * p.z;
     int wk = 1;
@@ -275,8 +326,10 @@ cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st) {
     const int cols = SKINNY_WARPS / wk * 16;
     const dim3 grid((p.n + cols - 1) / cols, p.z);
     auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(32 * SKINNY_WARPS), 0, st, p, wk); };
-    if (p.gelu) return go(gemv_dense_kernel<true, __nv_bfloat16>);
-    return p.out_f32 ? go(gemv_dense_kernel<false, float>) : go(gemv_dense_kernel<false, __nv_bfloat16>);
+    if (p.act == ACT_GELU_MUL) return go(gemv_dense_kernel<ACT_GELU_MUL, __nv_bfloat16>);
+    if (p.act == ACT_RELU2) return go(gemv_dense_kernel<ACT_RELU2, __nv_bfloat16>);
+    if (p.act == ACT_GELU_SIDE) return go(gemv_dense_kernel<ACT_GELU_SIDE, __nv_bfloat16>);
+    return p.out_f32 ? go(gemv_dense_kernel<ACT_NONE, float>) : go(gemv_dense_kernel<ACT_NONE, __nv_bfloat16>);
 }
 
 LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_dense)

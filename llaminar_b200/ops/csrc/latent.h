@@ -1,36 +1,11 @@
-// Launchers of the kernels around latent attention (low-rank key/value cache shared by all heads), of the fused norms and of
-// the small-batch matrix product on 16-bit weights.  `f32` selects the 32-bit build of a kernel (activations, weights and cache
-// as float) instead of the bf16 one; residual stream, norms, angles, scores and softmax are 32-bit in both.
+// Launchers of the kernels around latent attention (low-rank key/value cache shared by all heads).  `f32` selects the 32-bit
+// build of a kernel (activations and cache as float) instead of the bf16 one; angles, norms, scores and softmax are 32-bit in both.
 #pragma once
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
 #include <stddef.h>
 
 namespace llm {
-
-// h[t] = (add ? h[t] : 0) + RMSNorm(y[row(t)]) * w_post ; xn[t] = RMSNorm(h[t]) * w_next ; copies of h[t] in the activation type
-struct ResidNormParams {
-    const void* y;                 // activation type; nullptr: h is only read
-    size_t y_stride;
-    const int* y_rows;             // optional gather (embedding lookup): row(t) = y_rows[t]
-    int n_y_rows;                  // rows of y (bounds-check build)
-    const float* w_post;           // [d]
-    float* h;                      // [T, d]
-    int add;
-    const float* w_next;           // optional [d]
-    void* xn;                      // [T, d]
-    void *copy0, *copy1;           // optional
-    size_t copy_stride;
-    int d;
-    float eps;
-};
-cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cudaStream_t st);
-
-// act[t, j] = gelu_tanh(gu[t, j]) * gu[t, ff + j]
-cudaError_t launch_gelu_mul(const void* gu, void* act, int rows, int ff, bool f32, cudaStream_t st);
-
-// out[t, i] = magnitude * (cos, sin)(positions[t] * freqs[i])
-cudaError_t launch_rope_angles(const int* positions, const double* freqs, double magnitude, float2* out, int rows, int half, cudaStream_t st);
 
 // Down projection row [q latent | kv latent | rotated key] -> normed query latent, and the token's cache row
 // [normed kv latent, padded to rot_off | rotated key part, padded to width].
@@ -98,18 +73,7 @@ bool latent_chunk_has_kernel(int dk, int dv);
 cudaError_t launch_latent_chunk_tc(const LatentChunkParams& p, int n_keys, int n_seqs, int max_q_len, int* status, cudaStream_t st);
 bool latent_chunk_tc_fits(int dim, int rot, int vdim);
 
-// out[z][m, :] = x[z][m, :] W[z]^T for up to 8 rows, bf16 weights.  gelu: W holds 2n rows and out = gelu_tanh(first n) * second n.
-struct GemvDenseParams {
-    const __nv_bfloat16* w; size_t w_z; int ldw;
-    const __nv_bfloat16* x; size_t x_row, x_z;
-    void* out; size_t o_row, o_z;
-    int n, k, m, z;
-    bool out_f32, gelu;
-};
-cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st);
-
 int bounds_status_latent(bool reset);
 int bounds_status_latent_tc(bool reset);
-int bounds_status_dense(bool reset);
 
 }  // namespace llm

@@ -1,103 +1,11 @@
 // Python bindings of the kernels of latent-attention models: an extension of its own, so that a process that serves only such
-// a model compiles and loads nothing else.  Every tensor is checked on the host before a launch.
-#include <ATen/cuda/CUDAContext.h>
-#include <torch/extension.h>
-
+// a model compiles and loads nothing else.
+#include "binding_util.h"
 #include "latent.h"
 #include "launch.h"
 
 namespace {
-
-using torch::Tensor;
-using OptTensor = c10::optional<Tensor>;
-
-cudaStream_t stream() { return at::cuda::getCurrentCUDAStream().stream(); }
-
-void check(cudaError_t e, const char* what) { TORCH_CHECK(e == cudaSuccess, what, ": ", cudaGetErrorString(e)); }
-
-bool is_f32(const Tensor& t, const char* name) {
-    TORCH_CHECK(t.is_cuda(), name, " must be on the GPU");
-    TORCH_CHECK(t.scalar_type() == torch::kFloat32 || t.scalar_type() == torch::kBFloat16, name, " must be float32 or bfloat16");
-    return t.scalar_type() == torch::kFloat32;
-}
-void want(const Tensor& t, torch::ScalarType st, const char* name) {
-    TORCH_CHECK(t.is_cuda() && t.scalar_type() == st && t.is_contiguous(), name, " must be a contiguous ", st, " CUDA tensor");
-}
-void want_like(const Tensor& t, bool f32, const char* name) {
-    TORCH_CHECK(is_f32(t, name) == f32, name, " has the wrong element type");
-}
-const int* ints(const Tensor& t, const char* name) {
-    want(t, torch::kInt32, name);
-    return t.data_ptr<int>();
-}
-const float* floats(const Tensor& t, int64_t n, const char* name) {
-    want(t, torch::kFloat32, name);
-    TORCH_CHECK(t.numel() == n, name, " must hold ", n, " values");
-    return t.data_ptr<float>();
-}
-const float2* angle_ptr(const Tensor& t, int64_t rows) {
-    want(t, torch::kFloat32, "angles");
-    TORCH_CHECK(t.dim() == 3 && t.size(0) >= rows && t.size(2) == 2, "angles must be [rows, dims/2, 2]");
-    return reinterpret_cast<const float2*>(t.data_ptr<float>());
-}
-
-void resid_norm(const OptTensor& y, const OptTensor& y_rows, const OptTensor& w_post, const Tensor& h, bool add, const OptTensor& w_next,
-                const OptTensor& xn, const OptTensor& copy0, const OptTensor& copy1, double eps) {
-    llm::ResidNormParams p = {};
-    want(h, torch::kFloat32, "h");
-    const int64_t T = h.size(0), d = h.size(1);
-    if (T == 0) return;
-    bool f32 = false, typed = false;
-    auto elem = [&](const Tensor& t, const char* name) {
-        const bool f = is_f32(t, name);
-        TORCH_CHECK(!typed || f == f32, name, " has another element type than the other activations");
-        f32 = f; typed = true;
-        TORCH_CHECK(t.dim() == 2 && t.size(1) == d && t.stride(1) == 1, name, " must be rows of ", d, " values");
-    };
-    if (y) {
-        elem(*y, "y");
-        p.y = y->data_ptr(); p.y_stride = y->stride(0);
-        p.w_post = floats(w_post.value(), d, "w_post");
-        p.n_y_rows = y->size(0);
-        if (y_rows) {
-            p.y_rows = ints(*y_rows, "y_rows");
-            TORCH_CHECK(y_rows->numel() == T, "y_rows must name one row per token");
-        } else {
-            TORCH_CHECK(y->size(0) == T, "y must have as many rows as h");
-        }
-    }
-    p.h = h.data_ptr<float>(); p.add = add;
-    if (w_next) {
-        elem(xn.value(), "xn");
-        TORCH_CHECK(xn->is_contiguous() && xn->size(0) == T, "xn must be contiguous");
-        p.w_next = floats(*w_next, d, "w_next"); p.xn = xn->data_ptr();
-    }
-    if (copy0) { elem(*copy0, "copy0"); TORCH_CHECK(copy0->size(0) == T, "copy0 rows"); p.copy0 = copy0->data_ptr(); p.copy_stride = copy0->stride(0); }
-    if (copy1) {
-        elem(*copy1, "copy1");
-        TORCH_CHECK(copy1->size(0) == T && (!copy0 || copy1->stride(0) == copy0->stride(0)), "copy1 must have copy0's strides");
-        p.copy1 = copy1->data_ptr(); p.copy_stride = copy1->stride(0);
-    }
-    p.d = d; p.eps = eps;
-    check(llm::launch_resid_norm(p, T, f32, stream()), "resid_norm");
-}
-
-void gelu_mul(const Tensor& gu, const Tensor& act) {
-    const bool f32 = is_f32(gu, "gu");
-    want_like(act, f32, "act");
-    TORCH_CHECK(gu.is_contiguous() && act.is_contiguous() && gu.size(0) == act.size(0) && gu.size(1) == 2 * act.size(1), "gu must be [rows, 2 ff]");
-    if (gu.size(0) == 0) return;
-    check(llm::launch_gelu_mul(gu.data_ptr(), act.data_ptr(), gu.size(0), act.size(1), f32, stream()), "gelu_mul");
-}
-
-void rope_angles(const Tensor& positions, const Tensor& freqs, double magnitude, const Tensor& out) {
-    want(freqs, torch::kFloat64, "freqs");
-    const int rows = positions.numel(), half = freqs.numel();
-    angle_ptr(out, rows);
-    TORCH_CHECK(out.size(1) == half, "angles must have one column per frequency");
-    check(llm::launch_rope_angles(ints(positions, "positions"), freqs.data_ptr<double>(), magnitude, reinterpret_cast<float2*>(out.data_ptr<float>()),
-                                  rows, half, stream()), "rope_angles");
-}
+using namespace llm_binding;
 
 void latent_prep(const Tensor& down, const Tensor& q_norm, const Tensor& kv_norm, const Tensor& angles, const Tensor& positions, const Tensor& seq_ids,
                  const Tensor& block_table, const Tensor& cq, const Tensor& kv, int64_t rot_dim, int64_t rot_off, double eps) {
@@ -216,27 +124,9 @@ void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& k, const 
     }
 }
 
-// w [z, n, k] (gelu: [z, 2n, k]), x [z, m, k], out [z, m, n]; the last dimension of each is dense
-void gemv_dense(const Tensor& w, const Tensor& x, const Tensor& out, bool gelu) {
-    TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && x.scalar_type() == torch::kBFloat16, "gemv_dense takes bf16 operands");
-    TORCH_CHECK(w.dim() == 3 && x.dim() == 3 && out.dim() == 3 && w.stride(2) == 1 && x.stride(2) == 1 && out.stride(2) == 1, "gemv_dense layouts");
-    llm::GemvDenseParams p = {};
-    p.z = w.size(0); p.n = gelu ? w.size(1) / 2 : w.size(1); p.k = w.size(2); p.m = x.size(1);
-    TORCH_CHECK(x.size(0) == p.z && out.size(0) == p.z && x.size(2) == p.k && out.size(1) == p.m && out.size(2) == p.n, "gemv_dense shapes");
-    p.out_f32 = is_f32(out, "out"); p.gelu = gelu;
-    p.w = reinterpret_cast<const __nv_bfloat16*>(w.data_ptr()); p.w_z = w.stride(0); p.ldw = w.stride(1);
-    p.x = reinterpret_cast<const __nv_bfloat16*>(x.data_ptr()); p.x_row = x.stride(1); p.x_z = x.stride(0);
-    p.out = out.data_ptr(); p.o_row = out.stride(1); p.o_z = out.stride(0);
-    TORCH_CHECK(reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "gemv_dense operands must be 16-byte aligned");
-    check(llm::launch_gemv_dense(p, stream()), "gemv_dense");
-}
-
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
-    m.def("resid_norm", &resid_norm);
-    m.def("gelu_mul", &gelu_mul);
-    m.def("rope_angles", &rope_angles);
     m.def("latent_prep", &latent_prep);
     m.def("latent_rows", &latent_rows);
     m.def("latent_rows_has_kernel", &llm::latent_rows_has_kernel);
@@ -245,7 +135,6 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("latent_gather", &latent_gather);
     m.def("latent_chunk", &latent_chunk);
     m.def("latent_chunk_has_kernel", &llm::latent_chunk_has_kernel);
-    m.def("gemv_dense", &gemv_dense);
     m.def("set_pdl", [](bool on) { llm::pdl_enabled() = on; });
-    m.def("bounds_status", [](bool reset) { return llm::bounds_status_latent(reset) | llm::bounds_status_latent_tc(reset) | llm::bounds_status_dense(reset); });
+    m.def("bounds_status", [](bool reset) { return llm::bounds_status_latent(reset) | llm::bounds_status_latent_tc(reset); });
 }

@@ -1,0 +1,379 @@
+// Mixers with grouped-query attention or a recurrent state: the row-wise kernels.
+//
+//   attn_prep      norms of the queries and keys over all heads together, append to the paged cache
+//   window_plain   one row and head per CTA in float arithmetic
+//   linear_rows    mLSTM and retention, row after row.  The state matrix S [vdim, dim] of a head is spread over a cluster of CTAs,
+//                  which take slices of its rows: a warp reads whole rows of S, scales them, adds v k^T and multiplies by q while
+//                  they pass through its registers, so the state is read and written once per token (what bounds a decode step).
+//                  The CTAs of a cluster exchange the sums of squares of their slices through distributed shared memory for the
+//                  norm of the head's output.
+//   head_gate      norm and gate of the heads' outputs behind the chunk kernels (linear_tc.cu)
+#include <cooperative_groups.h>
+
+#include "common.cuh"
+#include "launch.h"
+#include "mixers.h"
+
+namespace llm {
+
+namespace {
+
+namespace cg = cooperative_groups;
+constexpr int PAGE = 64;
+constexpr float NORM_FLOOR = 1e-6f;            // of the mLSTM normaliser
+
+LLM_DEVICE float to_f(float v) { return v; }
+LLM_DEVICE float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <class T> LLM_DEVICE T from_f(float v);
+template <> LLM_DEVICE float from_f<float>(float v) { return v; }
+template <> LLM_DEVICE __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+LLM_DEVICE void load4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+LLM_DEVICE void load4(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    v[0] = bf16_lo(a.x); v[1] = bf16_hi(a.x); v[2] = bf16_lo(a.y); v[3] = bf16_hi(a.y);
+}
+LLM_DEVICE void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+LLM_DEVICE void store4(__nv_bfloat16* p, const float (&v)[4]) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3])); }
+
+LLM_DEVICE float sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
+
+template <int THREADS>
+LLM_DEVICE float block_sum(float v, float* red) {
+    v = warp_sum(v);
+    __syncthreads();                               // red may still be read from the sum before
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) s += red[i];
+    return s;
+}
+
+// ---- attention -----------------------------------------------------------------------------------------------------------
+template <class TI, class T>
+__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrepParams p) {
+    __shared__ float red[8];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const TI* row = static_cast<const TI*>(p.in) + (size_t)t * p.in_row;
+    const TI *q = row + p.q_off, *k = row + p.k_off, *v = row + p.v_off;
+    const int nq = p.n_heads * p.dim, nk = p.n_kv_heads * p.dim;
+    const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
+    const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
+    float sq = 0.f, sk = 0.f, x[4], w[4];
+    for (int i = threadIdx.x * 4; i < nq; i += 1024) {
+        load4(q + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sq += x[j] * x[j];
+    }
+    for (int i = threadIdx.x * 4; i < nk; i += 1024) {
+        load4(k + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sk += x[j] * x[j];
+    }
+    const float iq = 1.f / sqrtf(block_sum<256>(sq, red) / (float)(p.n_heads * p.true_dim) + p.eps);
+    const float ik = 1.f / sqrtf(block_sum<256>(sk, red) / (float)(p.n_kv_heads * p.true_dim) + p.eps);
+    T* qo = static_cast<T*>(p.q_out) + (size_t)t * nq;
+    for (int i = threadIdx.x * 4; i < nq; i += 1024) {
+        load4(q + i, x); load4(p.q_norm + i, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] *= iq * w[j];
+        store4(qo + i, x);
+    }
+    for (int i = threadIdx.x * 4; i < nk; i += 1024) {
+        const int g = i / p.dim, c = i - g * p.dim;
+        T* dst = static_cast<T*>(p.kv) + (((size_t)page * 2 * p.n_kv_heads + g) * PAGE + pos % PAGE) * p.dim + c;
+        load4(k + i, x); load4(p.k_norm + i, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] *= ik * w[j];
+        store4(dst, x);
+        load4(v + i, x);
+        store4(dst + (size_t)p.n_kv_heads * PAGE * p.dim, x);
+    }
+}
+
+template <class TG, class T>
+__global__ void __launch_bounds__(128) window_plain_kernel(const WindowPlainParams p) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float s_score[64];
+    pdl_trigger();
+    pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y, D = p.dim, g = h / (p.n_heads / p.n_kv_heads);
+    float *sq = sm, *so = sm + D;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int pos = p.positions[t];
+    const int* btab = p.block_table + (size_t)LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs) * p.max_pages;
+    const T* q = static_cast<const T*>(p.q) + ((size_t)t * p.n_heads + h) * D;
+    for (int i = threadIdx.x; i < D; i += 128) { sq[i] = to_f(q[i]); so[i] = 0.f; }
+    __syncthreads();
+    auto key_row = [&](int key, int which) {
+        const int page = LLM_CHECK_INDEX(btab[key / PAGE], p.n_pages);
+        return static_cast<const T*>(p.kv) + ((((size_t)page * 2 + which) * p.n_kv_heads + g) * PAGE + key % PAGE) * D;
+    };
+    float m = p.sink ? p.sink[h] : -INFINITY, l = p.sink ? 1.f : 0.f;
+    for (int k0 = p.window > 0 ? max(0, pos - p.window + 1) : 0; k0 <= pos; k0 += 64) {
+        const int n = min(64, pos + 1 - k0);
+        for (int j = warp; j < n; j += 4) {
+            const T* row = key_row(k0 + j, 0);
+            float s = 0.f;
+            for (int i = lane; i < D; i += 32) s = fmaf(sq[i], to_f(row[i]), s);
+            s = warp_sum(s);
+            if (lane == 0) s_score[j] = s * p.scale;
+        }
+        __syncthreads();
+        float nm = m;
+        for (int j = 0; j < n; ++j) nm = fmaxf(nm, s_score[j]);
+        const float c = expf(m - nm);
+        __syncthreads();
+        if ((int)threadIdx.x < n) s_score[threadIdx.x] = expf(s_score[threadIdx.x] - nm);
+        __syncthreads();
+        float ps = 0.f;
+        for (int j = 0; j < n; ++j) ps += s_score[j];
+        l = l * c + ps;
+        m = nm;
+        for (int i = threadIdx.x; i < D; i += 128) {
+            float a = so[i] * c;
+            for (int j = 0; j < n; ++j) a = fmaf(s_score[j], to_f(key_row(k0 + j, 1)[i]), a);
+            so[i] = a;
+        }
+        __syncthreads();
+    }
+    T* o = static_cast<T*>(p.out) + ((size_t)t * p.n_heads + h) * D;
+    for (int i = threadIdx.x; i < D; i += 128) {
+        float v = so[i] / l;
+        if (p.gate) v *= 1.f / (1.f + expf(-to_f(static_cast<const TG*>(p.gate)[(size_t)t * p.gate_row + (size_t)h * D + i])));
+        o[i] = from_f<T>(v);
+    }
+}
+
+// ---- linear attention ------------------------------------------------------------------------------------------------------
+constexpr int LIN_THREADS = 256, LIN_ROWS = 4;         // state rows in flight per warp
+
+// value i of a head's q or k: pairs (i, i + half) turn, the rest passes
+template <class TI> LLM_DEVICE float rotated(const TI* x, int i, const float2* ang, int half) {
+    if (i < half) return to_f(x[i]) * ang[i].x - to_f(x[i + half]) * ang[i].y;
+    if (i < 2 * half) return to_f(x[i]) * ang[i - half].x + to_f(x[i - half]) * ang[i - half].y;
+    return to_f(x[i]);
+}
+
+// Soft-capped log gates of one token and head: log input gate, log of the logistic forget gate
+LLM_DEVICE void lstm_gates(float zi, float zf, float cap, float& i, float& f) {
+    i = cap * tanhf(zi / cap);
+    const float z = cap * tanhf(zf / cap);
+    f = z >= 0.f ? -log1pf(expf(-z)) : z - log1pf(expf(z));
+}
+
+template <class TI, class TO>
+__global__ void __launch_bounds__(LIN_THREADS) linear_rows_kernel(const LinearParams p, int slice) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float red[LIN_THREADS / 32];
+    __shared__ float s_sum[2];                         // this CTA's sum of squares, by token parity
+    pdl_trigger();
+    pdl_wait();
+    cg::cluster_group cluster = cg::this_cluster();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = p.dim;
+    const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * slice, nv = min(slice, p.vdim - v0);
+    float *s_q = sm, *s_k = s_q + D, *s_n = s_k + D, *s_v = s_n + D, *s_o = s_v + slice;
+    const int r0 = p.cu ? p.cu[b] : b, r1 = p.cu ? p.cu[b + 1] : b + 1;
+    const int slot = LLM_CHECK_INDEX(p.slots[b], p.n_slots);
+    const bool lstm = p.gates != nullptr;
+    bool fresh = r0 < r1 && p.positions[r0] == 0;      // a sequence starts from zeros, whatever its slot holds
+    float* S = p.S + (((size_t)slot * p.heads + h) * p.vdim + v0) * D;
+    float* n_pool = lstm ? p.n + ((size_t)slot * p.heads + h) * D : nullptr;
+    float* m_pool = lstm ? p.m + (size_t)slot * p.heads + h : nullptr;
+    float m = lstm && !fresh ? *m_pool : 0.f;
+    if (lstm) for (int i = threadIdx.x; i < D; i += LIN_THREADS) s_n[i] = fresh ? 0.f : n_pool[i];
+    const TI* in = static_cast<const TI*>(p.in);
+    TO* out = static_cast<TO*>(p.out);
+    for (int t = r0; t < r1; ++t) {
+        const TI* row = in + (size_t)t * p.in_row;
+        const TI *q = row + p.q_off + h * D, *k = row + p.k_off + h * D, *v = row + p.v_off + h * p.vdim + v0;
+        const float2* ang = p.half ? p.angles + (size_t)t * p.half : nullptr;
+        float keep, add = 1.f, den = 1.f;
+        if (lstm) {
+            float gi, gf;
+            const float* z = p.gates + (size_t)t * p.gate_row;
+            lstm_gates(z[h] + p.bias_i[h], z[p.heads + h] + p.bias_f[h], p.cap, gi, gf);
+            const float top = fmaxf(gf + m, gi);
+            keep = expf(gf + m - top);
+            add = expf(gi - top);
+            m = top;
+        } else {
+            keep = p.decay[h];
+        }
+        float nq = 0.f;
+        for (int i = threadIdx.x; i < D; i += LIN_THREADS) {
+            const float a = rotated(q, i, ang, p.half) * p.q_scale, c = rotated(k, i, ang, p.half) * p.k_scale;
+            s_q[i] = a;
+            s_k[i] = c;
+            if (lstm) {
+                const float x = keep * s_n[i] + add * c;
+                s_n[i] = x;
+                nq += x * a;
+            }
+        }
+        for (int i = threadIdx.x; i < nv; i += LIN_THREADS) s_v[i] = to_f(v[i]);
+        if (lstm) den = 1.f / (fmaxf(fabsf(block_sum<LIN_THREADS>(nq, red)), expf(-m)) + NORM_FLOOR);
+        else __syncthreads();
+        for (int r = warp * LIN_ROWS; r < nv; r += LIN_THREADS / 32 * LIN_ROWS) {
+            float acc[LIN_ROWS] = {};
+            for (int c = lane * 4; c < D; c += 128) {
+                float s[LIN_ROWS][4], kk[4], qq[4];
+#pragma unroll
+                for (int j = 0; j < LIN_ROWS; ++j) {
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+                    if (!fresh && r + j < nv) load4(S + (size_t)(r + j) * D + c, s[j]);
+                }
+                load4(s_k + c, kk); load4(s_q + c, qq);
+#pragma unroll
+                for (int j = 0; j < LIN_ROWS; ++j) {
+                    if (r + j >= nv) continue;
+                    const float w = add * s_v[r + j];
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) {
+                        s[j][e] = keep * s[j][e] + w * kk[e];
+                        acc[j] += s[j][e] * qq[e];
+                    }
+                    store4(S + (size_t)(r + j) * D + c, s[j]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < LIN_ROWS; ++j) {
+                const float a = warp_sum(acc[j]);
+                if (lane == 0 && r + j < nv) s_o[r + j] = a;
+            }
+        }
+        __syncthreads();
+        float ss = 0.f;
+        for (int i = threadIdx.x; i < nv; i += LIN_THREADS) { const float o = s_o[i] * den; ss += o * o; }
+        ss = block_sum<LIN_THREADS>(ss, red);
+        if (gridDim.x > 1) {                           // the head's rows are spread over the cluster
+            const int par = (t - r0) & 1;
+            if (threadIdx.x == 0) s_sum[par] = ss;
+            cluster.sync();
+            ss = 0.f;
+            for (int c = 0; c < (int)gridDim.x; ++c) ss += *cluster.map_shared_rank(&s_sum[par], c);
+        }
+        const float inv = den / sqrtf(ss / (float)p.true_vdim + p.eps);
+        for (int i = threadIdx.x; i < nv; i += LIN_THREADS) {
+            const int col = h * p.vdim + v0 + i;
+            const float z = to_f(row[p.g_off + col]);
+            float o = s_o[i] * inv * (p.silu ? z : 1.f) / (1.f + expf(-z));
+            if (p.norm_w) o *= p.norm_w[col];
+            out[(size_t)t * p.out_row + col] = from_f<TO>(o);
+        }
+        fresh = false;
+        __syncthreads();                               // shared arrays are filled anew for the next token
+    }
+    if (gridDim.x > 1) cluster.sync();                 // every CTA has read n and m, and the others' sums
+    if (lstm && blockIdx.x == 0 && r0 < r1) {
+        for (int i = threadIdx.x; i < D; i += LIN_THREADS) n_pool[i] = s_n[i];
+        if (threadIdx.x == 0) *m_pool = m;
+    }
+}
+
+// a warp per token and head
+__global__ void __launch_bounds__(256) head_gate_kernel(const LinearParams p, const __nv_bfloat16* o, int rows) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31, unit = blockIdx.x * 8 + (threadIdx.x >> 5);
+    const int t = unit / p.heads, h = unit - t * p.heads, col0 = h * p.vdim;
+    if (t >= rows) return;
+    const __nv_bfloat16* src = o + (size_t)t * p.heads * p.vdim + col0;
+    const __nv_bfloat16* g = static_cast<const __nv_bfloat16*>(p.in) + (size_t)t * p.in_row + p.g_off + col0;
+    __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.out) + (size_t)t * p.out_row + col0;
+    constexpr int UN = 2;                              // units of eight values a lane keeps; wider heads are read again
+    uint4 keep[UN];
+    float ss = 0.f;
+    for (int i = 0; i * 256 < p.vdim; ++i) {
+        const int c = i * 256 + lane * 8;
+        const uint4 w = c < p.vdim ? *reinterpret_cast<const uint4*>(src + c) : make_uint4(0, 0, 0, 0);
+        const uint32_t x[4] = {w.x, w.y, w.z, w.w};
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { const float a = bf16_lo(x[j]), b = bf16_hi(x[j]); ss += a * a + b * b; }
+#pragma unroll
+        for (int u = 0; u < UN; ++u) if (u == i) keep[u] = w;
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.true_vdim + p.eps);
+    for (int i = 0; i * 256 < p.vdim; ++i) {
+        const int c = i * 256 + lane * 8;
+        if (c >= p.vdim) break;
+        uint4 w = keep[0];
+        if (i == 1) w = keep[1];
+        if (i >= UN) w = *reinterpret_cast<const uint4*>(src + c);
+        const uint4 z = *reinterpret_cast<const uint4*>(g + c);
+        const uint32_t x[4] = {w.x, w.y, w.z, w.w}, y[4] = {z.x, z.y, z.z, z.w};
+        uint32_t r[4];
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float za = bf16_lo(y[j]), zb = bf16_hi(y[j]);
+            float a = bf16_lo(x[j]) * inv * (p.silu ? za : 1.f) * sigmoid(za), b = bf16_hi(x[j]) * inv * (p.silu ? zb : 1.f) * sigmoid(zb);
+            if (p.norm_w) { a *= p.norm_w[col0 + c + 2 * j]; b *= p.norm_w[col0 + c + 2 * j + 1]; }
+            r[j] = pack_bf16(a, b);
+        }
+        *reinterpret_cast<uint4*>(dst + c) = make_uint4(r[0], r[1], r[2], r[3]);
+    }
+}
+
+}  // namespace
+
+cudaError_t launch_attn_prep(const AttnPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    if (p.dim % 8 || p.in_row % 4 || p.q_off % 4 || p.k_off % 4 || p.v_off % 4 || (f32 && !in_f32)) return cudaErrorInvalidValue;
+    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(256), 0, st, p); };
+    if (f32) return go(attn_prep_kernel<float, float>);
+    return in_f32 ? go(attn_prep_kernel<float, __nv_bfloat16>) : go(attn_prep_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
+
+cudaError_t launch_window_plain(const WindowPlainParams& p, int rows, bool gate_f32, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    const size_t smem = (size_t)p.dim * 8;
+    if (rows > 65535 || smem > 48 * 1024 || p.n_heads % p.n_kv_heads) return cudaErrorInvalidValue;
+    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(p.n_heads, rows), dim3(128), smem, st, p); };
+    if (f32) return gate_f32 ? go(window_plain_kernel<float, float>) : go(window_plain_kernel<__nv_bfloat16, float>);
+    return gate_f32 ? go(window_plain_kernel<float, __nv_bfloat16>) : go(window_plain_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
+
+cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, bool f32, cudaStream_t st) {
+    if (n_seqs == 0) return cudaSuccess;
+    if (p.dim % 8 || p.vdim % 8 || p.heads > 65535 || n_seqs > 65535 || (f32 && !in_f32) || (!p.gates == !p.decay)) return cudaErrorInvalidValue;
+    // slices of at least 32 state rows: enough CTAs to fill the machine, clusters of at most eight
+    int slices = 1;
+    while (slices < 8 && p.vdim > 32 * slices && p.heads * n_seqs * slices < 4 * 148) slices *= 2;
+    while ((p.vdim + slices - 1) / slices > 1024 && slices < 8) slices *= 2;
+    const int slice = ((p.vdim + slices - 1) / slices + 7) / 8 * 8;
+    slices = (p.vdim + slice - 1) / slice;
+    const size_t smem = (size_t)(3 * p.dim + 2 * slice) * 4;
+    if (smem > 48 * 1024) return cudaErrorInvalidValue;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(slices, p.heads, n_seqs);
+    cfg.blockDim = dim3(LIN_THREADS);
+    cfg.dynamicSmemBytes = smem;
+    cfg.stream = st;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = slices; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+    attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[1].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = pdl_enabled() ? 2 : 1;
+    if (f32) return cudaLaunchKernelEx(&cfg, linear_rows_kernel<float, float>, p, slice);
+    return in_f32 ? cudaLaunchKernelEx(&cfg, linear_rows_kernel<float, __nv_bfloat16>, p, slice)
+                  : cudaLaunchKernelEx(&cfg, linear_rows_kernel<__nv_bfloat16, __nv_bfloat16>, p, slice);
+}
+
+cudaError_t launch_head_gate(const LinearParams& p, const __nv_bfloat16* o, int rows, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    if (p.vdim % 8 || p.in_row % 8 || p.g_off % 8 || p.out_row % 8) return cudaErrorInvalidValue;
+    return launch_pdl(head_gate_kernel, dim3(((size_t)rows * p.heads + 7) / 8), dim3(256), 0, st, p, o, rows);
+}
+
+LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_mixers)
+
+}  // namespace llm

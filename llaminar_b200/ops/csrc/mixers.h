@@ -1,0 +1,63 @@
+// Launchers of the mixers with grouped-query attention or a recurrent state.  `f32` selects the 32-bit build (activations and
+// cache as float) instead of the bf16 one; norms, scores, softmax, gates and state are 32-bit in both.  The projected rows may be
+// float in the bf16 build as well (`in_f32`): decode steps keep their projections at accumulator precision.
+#pragma once
+#include <cuda_bf16.h>
+#include <cuda_runtime.h>
+#include <stddef.h>
+
+namespace llm {
+
+// Projected rows [q | k | ...] -> queries RMS-normed over all heads, and the token's entry of the paged cache [pages, 2, kv heads, 64,
+// dim]: keys RMS-normed over all heads, values as projected (tied: the keys before their norm).
+struct AttnPrepParams {
+    const void* in; size_t in_row; int q_off, k_off, v_off;      // v_off = k_off: tied values
+    const float *q_norm, *k_norm;                                // [n_heads * dim], [n_kv_heads * dim]
+    const int *positions, *seq_ids, *block_table;
+    int max_pages, n_seqs, n_pages;
+    void* q_out;                                                 // [T, n_heads, dim]
+    void* kv;
+    int n_heads, n_kv_heads, dim, true_dim;                      // padded head size, and the one that the means are taken over
+    float eps;
+};
+cudaError_t launch_attn_prep(const AttnPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st);
+
+// Attention of every row over the paged cache in float arithmetic, any size: the 32-bit mode, and shapes without a tensor-core kernel.
+struct WindowPlainParams {
+    const void* q; const void* kv; void* out;                    // [T, n_heads, dim], cache, [T, n_heads, dim]
+    const int *positions, *seq_ids, *block_table;
+    int max_pages, n_seqs, n_pages;
+    int n_heads, n_kv_heads, dim, window;
+    float scale;
+    const float* sink;                                           // optional [n_heads]
+    const void* gate; size_t gate_row;                           // optional, sigmoid; float if gate_f32
+};
+cudaError_t launch_window_plain(const WindowPlainParams& p, int rows, bool gate_f32, bool f32, cudaStream_t st);
+
+// Linear attention with a recurrent state per head: mLSTM (with `gates`) or retention (with `decay`).
+struct LinearParams {
+    const void* in; size_t in_row;                               // projected rows; head h of q starts at q_off + h * dim
+    int q_off, k_off, v_off, g_off;
+    const float* gates; size_t gate_row;                         // [T][log input gates, then log forget gates, of all heads] before bias and cap
+    const float *bias_i, *bias_f;                                // [heads]
+    float cap;
+    const float* decay;                                          // [heads]
+    const float2* angles; int half;                              // rotation of q and k (half = 0: none)
+    float q_scale, k_scale;
+    const int* cu;                                               // [n_seqs + 1] rows of the sequences (nullptr: one row each)
+    const int *positions, *slots;                                // [T], [n_seqs]
+    float *S, *n, *m;                                            // [slots, heads, vdim, dim], [slots, heads, dim], [slots, heads]
+    int n_slots, heads, dim, vdim, true_vdim;                    // padded to multiples of 8
+    const float* norm_w;                                         // optional [heads * vdim]
+    int silu;                                                    // output gate: silu or sigmoid
+    void* out; size_t out_row;                                   // [T, heads * vdim]
+    float eps;
+};
+// row after row: decode steps, the 32-bit mode, sizes without a chunk kernel
+cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, bool f32, cudaStream_t st);
+// out[t, h] = o[t, h] / rms(o[t, h]) * norm_w * gate(in[t, g_off + ...]), bf16
+cudaError_t launch_head_gate(const LinearParams& p, const __nv_bfloat16* o, int rows, cudaStream_t st);
+
+int bounds_status_mixers(bool reset);
+
+}  // namespace llm

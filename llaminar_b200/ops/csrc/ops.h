@@ -22,6 +22,10 @@ struct AttnDecodeParams {
     // [2][n_kv_heads][64][head_dim / 32] fp16 block scales (value = scale * int8)
     int kv_q8;
     size_t page_bytes, scale_off;
+    int window;                    // keys a row sees, itself included (0: all before it)
+    const float* sink;             // optional [n_heads]: one more logit in the softmax denominator, without a value
+    const float* gate;             // optional [rows, gate_row]: head h of a row is multiplied by sigmoid(gate[h * head_dim ...])
+    size_t gate_row;
 };
 
 struct AttnPrefillParams {
@@ -34,6 +38,10 @@ struct AttnPrefillParams {
     int n_heads, n_kv_heads, head_dim, max_pages;
     float scale;
     int n_pages;                   // pages of the cache (bounds-check build)
+    int window;                    // as in AttnDecodeParams
+    const float* sink;
+    const __nv_bfloat16* gate;
+    size_t gate_row;               // even
 };
 
 int attn_decode_pick_splits(int batch, int n_kv_heads, int max_pages_in_use);

@@ -1,4 +1,4 @@
-"""Python surface of the latent-attention extension (csrc/latent_attention.cu, csrc/dense_ops.cu).
+"""Python surface of the latent-attention extension (csrc/latent_attention.cu, csrc/latent_tc.cu) and of the dense one it builds on.
 
 As in :mod:`llaminar_b200.ops`, every call launches hand-written CUDA on the current stream; there is no fallback.  The
 extension is separate from the quantised-weight kernels, so a process that serves a latent model loads only this one.
@@ -9,8 +9,9 @@ import torch
 
 from . import _count
 from . import build as _build
+from .dense import GEMV_MAX_ROWS, gelu_mul, gemv_dense, gemv_fits, resid_norm, rope_angles  # noqa: F401
+from .dense import bounds_status as _dense_bounds_status
 
-GEMV_MAX_ROWS = 8
 _ready = False
 
 
@@ -22,25 +23,6 @@ def ext():
         mod.set_pdl(bool(debug_env().pdl))
         _ready = True
     return mod
-
-
-def resid_norm(h, y=None, w_post=None, *, add=True, y_rows=None, w_next=None, xn=None, copy0=None, copy1=None, eps: float) -> None:
-    """h = (h if add) + RMSNorm(y) * w_post (``y`` None: h is only read; ``y_rows`` gathers rows of y), then
-    xn = RMSNorm(h) * w_next and copies of h in the activation type.  One launch."""
-    ext().resid_norm(y, y_rows, w_post, h, add, w_next, xn, copy0, copy1, eps)
-    _count()
-
-
-def gelu_mul(gu: torch.Tensor, act: torch.Tensor) -> None:
-    """act = gelu_tanh(gu[:, :ff]) * gu[:, ff:]"""
-    ext().gelu_mul(gu, act)
-    _count()
-
-
-def rope_angles(positions: torch.Tensor, freqs: torch.Tensor, magnitude: float, out: torch.Tensor) -> None:
-    """out[t, i] = magnitude * (cos, sin)(positions[t] * freqs[i]); freqs in double precision."""
-    ext().rope_angles(positions, freqs, magnitude, out)
-    _count()
 
 
 def latent_prep(down, q_norm, kv_norm, angles, positions, seq_ids, block_table, cq, kv, rot_dim: int, rot_off: int, eps: float) -> None:
@@ -104,18 +86,5 @@ def chunk_tc_fits(dim: int, rot: int, vdim: int) -> bool:
     return bool(ext().latent_chunk_tc_fits(dim, rot, vdim))
 
 
-def gemv_fits(w: torch.Tensor, x: torch.Tensor) -> bool:
-    """Whether `gemv_dense` takes this product: few bf16 rows, 16-byte rows."""
-    k = w.shape[-1]
-    return (w.dtype == torch.bfloat16 and x.shape[-2] <= GEMV_MAX_ROWS and k % 8 == 0 and x.stride(-2) % 8 == 0 and w.stride(-2) % 8 == 0
-            and x.data_ptr() % 16 == 0 and w.data_ptr() % 16 == 0)
-
-
-def gemv_dense(w, x, out, gelu: bool = False) -> None:
-    """out[z] = x[z] @ w[z]^T for at most eight bf16 rows; ``gelu``: w stacks gate and up, out = gelu_tanh(gate) * up."""
-    ext().gemv_dense(w, x, out, gelu)
-    _count()
-
-
 def bounds_status(reset: bool = True) -> int:
-    return int(ext().bounds_status(bool(reset)))
+    return int(ext().bounds_status(bool(reset))) | _dense_bounds_status(reset)

@@ -57,8 +57,8 @@ class TPPlan:
         if tp < 1:
             errs.append("tensor-parallel degree must be >= 1")
             return errs
-        if getattr(cfg, "is_latent", False):
-            # the latent cache is shared by all heads and the matrices are not stored in shardable blocks
+        if getattr(cfg, "has_mixers", False):
+            # per-layer sizes, matrices that are not stored in shardable blocks, a latent cache shared by all heads
             return errs if tp == 1 else [f"{cfg.arch} models run on one GPU (tp={tp} was asked for)"]
         if cfg.n_heads % tp:
             errs.append(f"n_heads={cfg.n_heads} is not divisible by tp={tp}")

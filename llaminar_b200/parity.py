@@ -46,7 +46,7 @@ def compare(weights, device: str, prompt_tokens: int = 96, decode_steps: int = 4
     from .models.reference import ReferenceModel
     dev = torch.device(device)
     cfg = weights.config
-    if cfg.is_latent:
+    if cfg.has_mixers:
         raise ValueError(f"the layer report has no reference for {cfg.arch} models")
     if dev.type == "cuda":
         from .engine.cuda_model import CudaModel

@@ -6,10 +6,12 @@ need no devices (reference: src/v2/execution/mpi_orchestration/ExecutionPlanBuil
 """
 from __future__ import annotations
 
+import math
 from dataclasses import asdict, dataclass, field
 
 from .gguf.constants import BLOCK_GEOMETRY, GGMLType
 from .models.config import RECIPES, ModelConfig, QuantRecipe
+from .models.mixers import mixer_columns, mixer_kv_shapes, mixer_state_shapes
 from .parallel.tp_plan import TPPlan
 
 B200_HBM_BYTES = 180 * 10 ** 9
@@ -104,6 +106,10 @@ def layer_weight_bytes(cfg: ModelConfig, recipe: QuantRecipe, layer: int, tp: TP
         n = d * (m.q_rank + m.kv_rank + m.rot_dim) + m.heads * (m.dim + m.rot_dim) * m.q_rank
         n += m.heads * (2 * m.dim + m.vdim) * m.kv_rank + d * m.heads * m.vdim + 3 * d * ff        # the key matrices are held twice
         return 2.0 * n
+    if cfg.has_mixers:
+        from .models.config import family_of
+        return sum((2.0 if kind == "mat" else 4.0) * math.prod(shape) for _, name, kind, shape in family_of(cfg.arch).tensor_names(cfg)
+                   if name.startswith(f"blk.{layer}."))
     t = lambda name: recipe.for_tensor(f"blk.{layer}.{name}.weight", layer, cfg.n_layers)
     if cfg.is_gdn_layer(layer):
         # linear-attention block: q | k of every key head, this rank's value heads of v and z, alpha / b, output projection
@@ -138,7 +144,7 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
         return plan
     stages = layout["stages"]
     n_stages = len(stages)
-    if cfg.is_latent and n_stages > 1:
+    if cfg.has_mixers and n_stages > 1:
         plan.errors.append(f"{cfg.arch} models run on one GPU ({n_stages} pipeline stages were asked for)")
         return plan
     rank = 0
@@ -165,6 +171,11 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
             if cfg.is_latent:                   # one cache layer per layer run; input matrix of the looped layers
                 rp.kv_bytes = int(pages * sum(cfg.mixers[i].cache_width for i, _ in cfg.layer_runs()) * 64 * 2)
                 rp.weight_bytes += 4 * cfg.d_model * cfg.d_model if cfg.loop else 0
+            elif cfg.has_mixers:
+                rp.weight_bytes += 2 * cfg.vocab_size * cfg.side_dim * cfg.n_layers
+                from .engine.kv_cache import LayerStates
+                shapes = mixer_kv_shapes(cfg)
+                rp.kv_bytes = pages * sum(2 * h * d for h, d in shapes) * 64 * 2 + (batch_size + 1) * LayerStates.bytes_per_slot(mixer_state_shapes(cfg))
             if cfg.is_hybrid:
                 # one fp32 state slot per batch lane (+1 scratch) for every linear-attention layer of the stage
                 from .engine.kv_cache import HybridState
@@ -179,6 +190,8 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
                 m = max(cfg.mixers, key=lambda m: m.heads * (2 * m.dim + m.rot_dim + 2 * m.vdim))
                 rp.activation_bytes = int(T * (cfg.d_model * (4 + 8) + 2 * (m.heads * (2 * m.dim + m.rot_dim + 2 * m.vdim) + 2 * m.q_rank
                                                                             + 2 * m.cache_width + 3 * ff)))
+            elif cfg.has_mixers:
+                rp.activation_bytes = int(T * (cfg.d_model * (4 + 6) + 2 * (max(mixer_columns(m) for m in cfg.mixers) + 2 * max(cfg.layer_ff))))
             rp.workspace_bytes = int(256 * 65536 * 4 + (1 << 22) * 4 + batch_size * 4 * (tp.vocab_stop - tp.vocab_start) * 4)
             if rp.total_bytes > hbm_bytes * 0.95:
                 plan.errors.append(f"rank {rank} ({dev}): needs {rp.total_bytes / 1e9:.1f} GB, device has {hbm_bytes / 1e9:.0f} GB")

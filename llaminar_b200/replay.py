@@ -24,7 +24,7 @@ def build_engine(model: str, dtype: torch.dtype, max_tokens: int, device: str):
     from .engine.engine import LLMEngine
     from .models.weights import ModelWeights
     weights = ModelWeights.from_path(model, device="cpu")
-    if dtype == torch.float32 and device != "cpu" and not weights.config.is_latent:
+    if dtype == torch.float32 and device != "cpu" and not weights.config.has_mixers:
         return None
     pages = -(-max_tokens // PAGE)
     return LLMEngine(weights, device=device, max_batch=LIVE_REQUESTS, max_context=pages * PAGE, kv_pages=pages + 1,      # + the scratch page
