@@ -216,7 +216,7 @@ def mlstm_layer(heads=3, dim=24, vdim=16, cap=10.0, ff=56):
 
 
 def parallel_layer(heads=4, kv_heads=2, dim=24, window=20, scale=None, r_heads=3, r_dim=20, r_vdim=28, r_rot=12, base=1000.0, decay=None, ff=56):
-    decay = decay or [1 - 2.0 ** (-3 - i) for i in range(r_heads)]
+    decay = decay or [1 - 2.0 ** (-5 - i) for i in range(r_heads)]
     return {"type": "parallel",
             "mixer": {"left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "mask": {"size": window}, "scale": scale if scale is not None else dim ** -0.5},
                       "right": {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "decay": decay, "rot": {"base": base, "dims": r_rot}}},
