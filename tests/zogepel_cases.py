@@ -14,7 +14,7 @@ M, P = oracle.mlstm_layer, oracle.parallel_layer
 # heads as query heads, rotation of all, some and two values of a head, decays near 0 and 1, windows of one page, of one token and
 # wider than any prompt
 MODELS = {
-    "both": [M(), P(), M(heads=2, dim=16, vdim=40, cap=4.0), P(heads=6, kv_heads=3, dim=16, window=77, r_heads=2, r_dim=32, r_vdim=16, r_rot=32)],
+    "both": [M(), P(), M(heads=2, dim=16, vdim=40, cap=4.0), P(heads=6, kv_heads=3, dim=16, window=77, r_heads=2, r_dim=32, r_vdim=16, r_rot=32, decay=[0.997, 0.98])],
     "lstm": [M(heads=1, dim=30, vdim=22, ff=None), M(heads=5, dim=8, vdim=8, cap=30.0, ff=40)],
     "parallel": [P(heads=2, kv_heads=2, dim=33, window=64, r_heads=1, r_dim=9, r_vdim=13, r_rot=2, decay=[0.5], ff=None), P(heads=5, kv_heads=1, window=1, scale=0.5),
                  P(window=1000, r_heads=4, r_dim=16, r_vdim=64, r_rot=16, decay=[0.999, 0.9, 1.0, 0.05])],
