@@ -24,6 +24,9 @@ from ..models.mixers import mixer_kv_shapes, mixer_state_shapes, pad_to_multiple
 from .dense import DenseLinear, pad8, pad_to
 
 
+SHORT_ROWS = 4              # batches of portions up to this long advance the recurrences row by row
+
+
 def _pad_heads(w: torch.Tensor, heads: int, size: int) -> torch.Tensor:
     """Rows of a projection [heads * n, k] -> [heads * size, k]."""
     k = w.shape[1]
@@ -43,6 +46,7 @@ class MixerPlan:
     """What the layers of one forward call share."""
     angles: list[torch.Tensor]          # per distinct rotation: [T, dims/2, 2]
     rows: torch.dtype                   # type of the projected rows in front of the mixers
+    chunks: tuple | None = None         # how the chunk kernels cut the batch (None: row after row)
 
 
 class MixerStack:
@@ -181,7 +185,7 @@ class MixerStack:
         attn = [L.left.m.heads * L.left.dim for L in layers if L.left is not None]
         lin = [L.right.m.heads * L.right.vdim for L in layers]
         self._ws = {"q": e(max(attn, default=0)), "oa": e(max(attn, default=0)), "ol": e(max(lin)),
-                    "act": e(max(max(L.ff for L in layers), pad8(c.side_dim))), "raw": e(max(max(L.ff for L in layers), pad8(c.side_dim)))}
+                    "act": e(max(max(L.ff for L in layers), pad8(c.side_dim))), "raw": e(max(max(L.ff for L in layers), pad8(c.side_dim), max(lin)))}
         # projected rows: float in a decode step (few rows) and in 32-bit mode, the activation type in prompts; one buffer for both
         self._rows = torch.empty(T * max(L.proj.n_out for L in layers) * (4 if self.f32 else 2), dtype=torch.uint8, device=self.device)
         self._gates = torch.empty(T * 2 * max((L.mixer.heads for L in layers if isinstance(L.mixer, MatrixLSTM)), default=1), dtype=torch.float32, device=self.device)
@@ -203,12 +207,16 @@ class MixerStack:
 
     def plan(self, fb, T: int) -> MixerPlan:
         from ..ops import dense as ops
+        from ..ops import mixers as mixer_ops
         angles = []
         for rot, f in zip(self.rotaries, self.freqs):
             a = torch.empty(T, f.numel(), 2, dtype=torch.float32, device=self.device)
             ops.rope_angles(fb.positions, f, rot.magnitude, a)
             angles.append(a)
-        return MixerPlan(angles, torch.float32 if self.f32 or fb.is_decode else self.dtype)
+        plan = MixerPlan(angles, torch.float32 if self.f32 or fb.is_decode else self.dtype)
+        if not self.f32 and not fb.is_decode and self.linear_tc and fb.max_q_len > SHORT_ROWS:
+            plan.chunks = mixer_ops.chunk_tables(fb.host_cu if fb.host_cu is not None else fb.cu_q.tolist(), self.device)
+        return plan
 
     def layer(self, L, h: torch.Tensor, fb, plan: MixerPlan, kv) -> None:
         """x holds the layer's input in the activation type, and its output's at the end."""
@@ -260,7 +268,11 @@ class MixerStack:
         o = self.ws("ol", T, m.heads * P.vdim)
         state = kv.hybrid.layers[P.state]
         args = (rows, P.offs, (gates, *P.gates) if gates is not None else None, P.decay, plan.angles[P.rot] if P.rot is not None else None, P.q_scale, P.k_scale)
-        ops.linear_rows(*args, None if fb.is_decode else fb.cu_q, fb.positions, fb.state_slots, state, m.vdim, P.norm, gates is None, o, self.cfg.rms_eps)
+        args += (None if fb.is_decode else fb.cu_q, fb.positions, fb.state_slots, state, m.vdim, P.norm, gates is None, o, self.cfg.rms_eps)
+        if plan.chunks is not None and ops.linear_chunk_fits(P.dim, P.vdim):
+            ops.linear_chunk(*args, plan.chunks, self.ws("raw", T, m.heads * P.vdim), self.status)
+        else:
+            ops.linear_rows(*args)
         return o
 
     def final_logits(self, rows: torch.Tensor, norm: torch.Tensor, head: DenseLinear, out: torch.Tensor) -> torch.Tensor:

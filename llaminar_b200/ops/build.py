@@ -22,7 +22,7 @@ SOURCES = {
     NAME: ["binding.cpp", "gemv.cu", "gemv_stream.cu", "gemm_tc.cu", "gemm_tc_small.cu", "attention.cu", "attention_tc.cu", "ops.cu", "gdn.cu", "moe_ep.cu", "no_alloc.cu"],
     DENSE: ["dense_binding.cpp", "dense_ops.cu"],
     LATENT: ["latent_binding.cpp", "latent_attention.cu", "latent_tc.cu"],
-    MIXERS: ["mixers_binding.cpp", "mixers.cu", "attention.cu", "attention_tc.cu"],
+    MIXERS: ["mixers_binding.cpp", "mixers.cu", "linear_tc.cu", "attention.cu", "attention_tc.cu"],
 }
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xptxas", "-v"]

@@ -55,9 +55,24 @@ struct LinearParams {
 };
 // row after row: decode steps, the 32-bit mode, sizes without a chunk kernel
 cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, bool f32, cudaStream_t st);
+// Chunk-parallel form for prompts: bf16 rows, heads of at most 128 key values (linear_tc.cu).  Sequences are cut into chunks of
+// LINEAR_CHUNK rows; `chunks` holds (first row, rows, sequence, 0) of each, `seqs` (first chunk, chunks, 0, 0).  Scratch: state
+// [chunks][heads][vdim][dim] float, vec [chunks][heads][dim] float, scal [chunks][heads][4] float.  o [T, heads * vdim] bf16 receives
+// the heads' outputs before norm and gate.
+constexpr int LINEAR_CHUNK = 128;
+struct LinearChunks {
+    const int4 *chunks, *seqs;
+    int n_chunks, n_seqs, rows;
+    float *state, *vec, *scal;
+    __nv_bfloat16* o;
+    int* status;                                                 // receives STATUS_TIMEOUT if a wait gave up
+};
+bool linear_chunk_fits(int dim, int vdim);
+cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cudaStream_t st);
 // out[t, h] = o[t, h] / rms(o[t, h]) * norm_w * gate(in[t, g_off + ...]), bf16
 cudaError_t launch_head_gate(const LinearParams& p, const __nv_bfloat16* o, int rows, cudaStream_t st);
 
 int bounds_status_mixers(bool reset);
+int bounds_status_linear_tc(bool reset);
 
 }  // namespace llm

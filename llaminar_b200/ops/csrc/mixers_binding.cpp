@@ -166,6 +166,37 @@ void linear_rows(const Tensor& in, const std::vector<int64_t>& offs, const OptTe
     check(llm::launch_linear_rows(p, slots.numel(), is_f32(in, "in"), is_f32(out, "out"), stream()), "linear_rows");
 }
 
+// chunks, seqs: int32 [n, 4], see LinearChunks.  cu is the host's view of the sequences and stays unused on the device.
+void linear_chunk(const Tensor& in, const std::vector<int64_t>& offs, const OptTensor& gates, const OptTensor& bias_i, const OptTensor& bias_f, double cap,
+                  const OptTensor& decay, const OptTensor& angles, double q_scale, double k_scale, const Tensor& cu, const Tensor& positions,
+                  const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps,
+                  const Tensor& chunks, const Tensor& seqs, const Tensor& scratch, const Tensor& vec, const Tensor& scal, const Tensor& o, const Tensor& status) {
+    const llm::LinearParams p = linear_params(in, offs, gates, bias_i, bias_f, cap, decay, angles, q_scale, k_scale, cu, positions, slots, state, true_vdim, norm_w, silu, out, eps);
+    bf16(in, "in"); bf16(out, "out");
+    llm::LinearChunks c = {};
+    auto table = [](const Tensor& t, const char* name) {
+        TORCH_CHECK(t.dim() == 2 && t.size(1) == 4, name, " must be [n, 4]");
+        return reinterpret_cast<const int4*>(ints(t, name));
+    };
+    c.chunks = table(chunks, "chunks"); c.seqs = table(seqs, "seqs");
+    c.n_chunks = chunks.size(0); c.n_seqs = seqs.size(0); c.rows = in.size(0);
+    TORCH_CHECK(slots.numel() == c.n_seqs, "one slot per sequence");
+    const int64_t units = (int64_t)c.n_chunks * p.heads;
+    auto scratch_ptr = [&](const Tensor& t, int64_t n, const char* name) {
+        want(t, torch::kFloat32, name);
+        TORCH_CHECK(t.numel() >= n, name, " too small");
+        want_aligned(t, name);
+        return t.data_ptr<float>();
+    };
+    c.state = scratch_ptr(scratch, units * p.vdim * p.dim, "scratch"); c.vec = scratch_ptr(vec, units * p.dim, "vec"); c.scal = scratch_ptr(scal, units * 4, "scal");
+    TORCH_CHECK(o.is_contiguous() && o.numel() >= (int64_t)c.rows * p.heads * p.vdim, "o too small");
+    c.o = const_cast<__nv_bfloat16*>(bf16(o, "o"));
+    want(status, torch::kInt32, "status");
+    c.status = status.data_ptr<int>();
+    check(llm::launch_linear_chunk(p, c, stream()), "linear_chunk");
+    check(llm::launch_head_gate(p, c.o, c.rows, stream()), "head_gate");
+}
+
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
@@ -174,6 +205,9 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("attn_decode", &attn_decode);
     m.def("attn_prefill", &attn_prefill);
     m.def("linear_rows", &linear_rows);
+    m.def("linear_chunk", &linear_chunk);
+    m.def("linear_chunk_fits", &llm::linear_chunk_fits);
+    m.attr("LINEAR_CHUNK") = llm::LINEAR_CHUNK;
     m.def("set_pdl", [](bool on) { llm::pdl_enabled() = on; });
-    m.def("bounds_status", [](bool reset) { return llm::bounds_status_mixers(reset); });
+    m.def("bounds_status", [](bool reset) { return llm::bounds_status_mixers(reset) | llm::bounds_status_linear_tc(reset); });
 }

@@ -109,6 +109,11 @@ LLM_DEVICE void tma_load_3d(uint32_t dst, const CUtensorMap* tmap, int x, int y,
                  ::"r"(dst), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(x), "r"(y), "r"(z), "r"(bar) : "memory");
 }
 
+LLM_DEVICE void tma_load_4d(uint32_t dst, const CUtensorMap* tmap, int x, int y, int z, int w, uint32_t bar) {
+    asm volatile("cp.async.bulk.tensor.4d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4, %5}], [%6];"
+                 ::"r"(dst), "l"(reinterpret_cast<uint64_t>(tmap)), "r"(x), "r"(y), "r"(z), "r"(w), "r"(bar) : "memory");
+}
+
 // K-major, 128-byte swizzled operand tile: rows of 128 bytes, 8-row groups 1024 bytes apart.
 LLM_DEVICE uint64_t smem_desc_sw128(uint32_t addr) {
     uint64_t d = 0;

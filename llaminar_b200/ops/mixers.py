@@ -71,5 +71,38 @@ def linear_rows(rows, offs, gates, decay, angles, q_scale: float, k_scale: float
     _count()
 
 
+def chunk_tables(cu: list[int], device) -> tuple[torch.Tensor, torch.Tensor]:
+    """How the chunk kernels cut a packed batch whose sequence b has rows cu[b] .. cu[b + 1]: (first row, rows, sequence, last of it)
+    per chunk and (first chunk, chunks, 0, 0) per sequence."""
+    size = ext().LINEAR_CHUNK
+    chunks, seqs = [], []
+    for b in range(len(cu) - 1):
+        first = len(chunks)
+        for r in range(cu[b], cu[b + 1], size):
+            n = min(size, cu[b + 1] - r)
+            chunks.append((r, n, b, int(r + n == cu[b + 1])))
+        seqs.append((first, len(chunks) - first, 0, 0))
+    it = lambda x: torch.tensor(x, dtype=torch.int32, device=device)
+    return it(chunks), it(seqs)
+
+
+def linear_chunk_fits(dim: int, vdim: int) -> bool:
+    return bool(ext().linear_chunk_fits(dim, vdim))
+
+
+def linear_chunk(rows, offs, gates, decay, angles, q_scale: float, k_scale: float, cu, positions, slots, state, true_vdim: int, norm_w,
+                 silu: bool, out, eps: float, tables, raw, status) -> None:
+    """As `linear_rows` for prompts in bf16, chunk-parallel on the tensor cores.  ``tables``: see `chunk_tables`; ``raw``: workspace
+    like ``out``."""
+    g = gates or (None, None, None, 1.0)
+    chunks, seqs = tables
+    _, h, v, d = state[0].shape
+    n = chunks.shape[0]
+    f = lambda *s: torch.empty(*s, dtype=torch.float32, device=rows.device)
+    ext().linear_chunk(rows, list(offs), *g, decay, angles, q_scale, k_scale, cu, positions, slots, list(state), true_vdim, norm_w, silu, out, eps,
+                       chunks, seqs, f(n, h, v, d), f(n, h, d), f(n, h, 4), raw, status)
+    _count(4)
+
+
 def bounds_status(reset: bool = True) -> int:
     return int(ext().bounds_status(bool(reset)))
