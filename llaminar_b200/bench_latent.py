@@ -1,81 +1,17 @@
 """Throughput and kernel times of latent-attention models beside the like parts of a grouped-query model of equal size.
 
 Used by `bench.py --latent`.  Two parts: whole models (prefill and decode tokens per second through the engine, random
-weights, a few layers of full size) and single kernels with their fraction of the memory or tensor roofline.  Kernels are timed
-with CUDA events around a captured graph of many launches that walk over buffers larger than L2 together.
+weights, a few layers of full size) and single kernels with their fraction of the memory or tensor roofline.
 """
 from __future__ import annotations
 
 import json
-import os
-import statistics
 from dataclasses import replace
 
 import torch
 
+from .bench_util import copies_for, cut, measured_peaks, page_tables, row, time_us, visible_pairs, whole_model
 from .models.config import SHAPES, ModelConfig
-
-L2_BYTES = 126 << 20
-
-
-def measured_peaks() -> tuple[float, float, str]:
-    """(memory bandwidth in bytes/s, bf16 FLOP/s, where they come from)"""
-    path = os.path.join(os.path.dirname(os.path.dirname(os.path.abspath(__file__))), "MEASURED_PEAKS.json")
-    if os.path.exists(path):
-        p = json.load(open(path))
-        return p["hbm_gbs"] * 1e9, p["bf16_tflops"] * 1e12, "measured"
-    return 6.65e12, 1.59e15, "fallback"
-
-
-def copies_for(nbytes: int) -> int:
-    """How many copies of a kernel's data make its working set larger than L2."""
-    return max(2, min(256, -(-2 * L2_BYTES // max(nbytes, 1))))
-
-
-def time_us(calls: list, reps: int = 5) -> float:
-    """Device time of one call: `calls` (closures over different buffers) captured back to back in a graph, median of replays."""
-    s = torch.cuda.Stream()
-    s.wait_stream(torch.cuda.current_stream())
-    with torch.cuda.stream(s):
-        for c in calls[:3]:
-            c()
-    torch.cuda.current_stream().wait_stream(s)
-    torch.cuda.synchronize()
-    g = torch.cuda.CUDAGraph()
-    with torch.cuda.graph(g):
-        for c in calls:
-            c()
-    for _ in range(3):
-        g.replay()
-    out = []
-    for _ in range(reps):
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        torch.cuda.synchronize()
-        a.record()
-        g.replay()
-        b.record()
-        torch.cuda.synchronize()
-        out.append(a.elapsed_time(b) * 1e3 / len(calls))
-    return statistics.median(out)
-
-
-def _row(name: str, us: float, nbytes: float, flops: float) -> dict:
-    bw, tf, _ = measured_peaks()
-    roof = max(nbytes / bw, flops / tf) * 1e6
-    return {"kernel": name, "us": round(us, 2), "roofline_us": round(roof, 2), "fraction": round(roof / us, 3),
-            "bound": "memory" if nbytes / bw >= flops / tf else "tensor"}
-
-
-def visible_pairs(n: int, window: int) -> int:
-    """Query-key pairs of a causal prompt of n tokens."""
-    return sum(min(i + 1, window) if window else i + 1 for i in range(n))
-
-
-def _tables(batch: int, ctx: int, dev):
-    P = -(-ctx // 64)
-    bt = (torch.randperm(batch * P, device=dev).to(torch.int32) + 1).view(batch, P).contiguous()
-    return bt, P, batch * P + 1
-
 
 def latent_decode(cfg: ModelConfig, batch: int, ctx: int, tensor_core: bool = True) -> dict:
     """One layer's attention of a decode step: query rotation, split attention and merge."""
@@ -83,7 +19,7 @@ def latent_decode(cfg: ModelConfig, batch: int, ctx: int, tensor_core: bool = Tr
     from .engine.latent import PART_FLOATS, PaddedSizes
     m, dev = cfg.mixers[0], "cuda"
     s = PaddedSizes.of(m)
-    bt, P, pages = _tables(batch, ctx, dev)
+    bt, P, pages = page_tables(batch, ctx, dev)
     keys = min(ctx, m.window) if m.window else ctx
     nbytes = batch * keys * s.width * 2
     bf = dict(dtype=torch.bfloat16, device=dev)
@@ -102,13 +38,13 @@ def latent_decode(cfg: ModelConfig, batch: int, ctx: int, tensor_core: bool = Tr
     us = time_us(calls)
     assert int(status[0]) == 0
     flops = 2.0 * batch * s.heads * keys * (s.width + s.latent)
-    return _row(f"latent_rows ({'tcgen05' if tensor_core else 'mma.sync'}) batch {batch} keys {keys} heads {s.heads} splits {sp}", us, nbytes + 4 * ql.numel(), flops)
+    return row(f"latent_rows ({'tcgen05' if tensor_core else 'mma.sync'}) batch {batch} keys {keys} heads {s.heads} splits {sp}", us, nbytes + 4 * ql.numel(), flops)
 
 
 def gqa_decode(cfg: ModelConfig, batch: int, ctx: int) -> dict:
     from . import ops
     dev, H, Hk, D = "cuda", cfg.n_heads, cfg.n_kv_heads, cfg.head_dim
-    bt, P, pages = _tables(batch, ctx, dev)
+    bt, P, pages = page_tables(batch, ctx, dev)
     nbytes = batch * ctx * 2 * Hk * D * 2
     bf = dict(dtype=torch.bfloat16, device=dev)
     kvs = [torch.randn(pages, 2, Hk, 64, D, **bf) for _ in range(copies_for(nbytes))]
@@ -117,7 +53,7 @@ def gqa_decode(cfg: ModelConfig, batch: int, ctx: int) -> dict:
     sp = max(1, min(16, 296 // max(1, batch * Hk), P // 2))
     sc = ops.scratch_for(torch.device("cuda", torch.cuda.current_device()))
     us = time_us([lambda kv=kv: ops.attn_decode(q, kv, out, bt, lens, H, Hk, D, 1, D ** -0.5, sp, sc) for kv in kvs])
-    return _row(f"attn_decode batch {batch} keys {ctx} heads {H}/{Hk}", us, nbytes + 4 * q.numel(), 4.0 * batch * H * ctx * D)
+    return row(f"attn_decode batch {batch} keys {ctx} heads {H}/{Hk}", us, nbytes + 4 * q.numel(), 4.0 * batch * H * ctx * D)
 
 
 def latent_prefill(cfg: ModelConfig, n: int, window: int) -> list[dict]:
@@ -126,7 +62,7 @@ def latent_prefill(cfg: ModelConfig, n: int, window: int) -> list[dict]:
     from .engine.latent import PaddedSizes
     m, dev = replace(cfg.mixers[0], window=window), "cuda"
     s = PaddedSizes.of(m)
-    bt, P, pages = _tables(1, n, dev)
+    bt, P, pages = page_tables(1, n, dev)
     bf = dict(dtype=torch.bfloat16, device=dev)
     copies = 3
     q = [torch.randn(n, s.heads, s.dim + s.rot, **bf) for _ in range(copies)]
@@ -141,22 +77,22 @@ def latent_prefill(cfg: ModelConfig, n: int, window: int) -> list[dict]:
     pairs, rows = visible_pairs(n, window), []
     for name, v, st in (("tcgen05", vts, status), ("mma.sync", vs, None)):
         us = time_us([lambda i=i: ops.latent_chunk(q[i], ang, ks[i], v[i], lat, s.latent, seqs, n, out, s.dim, s.rot, s.vdim, window, m.scale, sink, st) for i in range(copies)] * 3)
-        rows.append(_row(f"latent_chunk ({name}) rows {n} window {window or 'none'} heads {s.heads}", us, 2 * (q[0].numel() + 3 * ks[0].numel()),
+        rows.append(row(f"latent_chunk ({name}) rows {n} window {window or 'none'} heads {s.heads}", us, 2 * (q[0].numel() + 3 * ks[0].numel()),
                          2.0 * pairs * s.heads * (m.dim + m.rot_dim + m.vdim)))
     assert int(status[0]) == 0
     c = lat[:, :s.latent]
     us = time_us([lambda i=i: (torch.mm(c, wk.t(), out=ks[i]), torch.mm(wv, c.t(), out=vts[i])) for i in range(copies)] * 3)
-    rows.append(_row(f"keys and values from latents (two cuBLAS products) rows {n}", us, 2 * (2 * ks[0].numel() + lat.numel()), 2.0 * n * (wk.numel() + wv.numel())))
+    rows.append(row(f"keys and values from latents (two cuBLAS products) rows {n}", us, 2 * (2 * ks[0].numel() + lat.numel()), 2.0 * n * (wk.numel() + wv.numel())))
     lats = [torch.empty_like(lat) for _ in range(copies_for(4 * lat.numel()))]
     us = time_us([lambda l=l: ops.latent_gather(kv, seqs, n, bt, l) for l in lats])
-    rows.append(_row(f"latent_gather rows {n}", us, 4 * lat.numel(), 0))
+    rows.append(row(f"latent_gather rows {n}", us, 4 * lat.numel(), 0))
     return rows
 
 
 def gqa_prefill(cfg: ModelConfig, n: int) -> dict:
     from . import ops
     dev, H, Hk, D = "cuda", cfg.n_heads, cfg.n_kv_heads, cfg.head_dim
-    bt, P, pages = _tables(1, n, dev)
+    bt, P, pages = page_tables(1, n, dev)
     bf = dict(dtype=torch.bfloat16, device=dev)
     qs = [torch.randn(n, H, D, **bf) for _ in range(3)]
     kvs = [torch.randn(pages, 2, Hk, 64, D, **bf) for _ in range(3)]
@@ -164,7 +100,7 @@ def gqa_prefill(cfg: ModelConfig, n: int) -> dict:
     cu, ctx = torch.tensor([0, n], dtype=torch.int32, device=dev), torch.zeros(1, dtype=torch.int32, device=dev)
     sc = ops.scratch_for(torch.device("cuda", torch.cuda.current_device()))
     us = time_us([lambda q=q, kv=kv: ops.attn_prefill(q, kv, out, bt, cu, ctx, H, Hk, D, D ** -0.5, n, scratch=sc) for q, kv in zip(qs, kvs)] * 3)
-    return _row(f"attn_prefill rows {n} heads {H}/{Hk}", us, 4 * out.numel(), 4.0 * visible_pairs(n, 0) * H * D)
+    return row(f"attn_prefill rows {n} heads {H}/{Hk}", us, 4 * out.numel(), 4.0 * visible_pairs(n, 0) * H * D)
 
 
 def norms(cfg: ModelConfig, n: int) -> list[dict]:
@@ -178,19 +114,19 @@ def norms(cfg: ModelConfig, n: int) -> list[dict]:
     w = torch.ones(d, device=dev)
     k = min(copies_for(n * d * 12), 64)
     hs, ys, xs = [torch.randn(n, d, device=dev) for _ in range(k)], [torch.randn(n, d, **bf) for _ in range(k)], [torch.empty(n, d, **bf) for _ in range(k)]
-    rows = [_row(f"resid_norm rows {n} (two norms, residual update)", time_us([lambda h=h, y=y, x=x: ops.resid_norm(h, y, w, w_next=w, xn=x, eps=1e-6) for h, y, x in zip(hs, ys, xs)]), n * d * 12, 0),
-            _row(f"rmsnorm rows {n} (other families)", time_us([lambda h=h, x=x: base.rmsnorm(h, w, x, 1e-6) for h, x in zip(hs, xs)]), n * d * 6, 0)]
+    rows = [row(f"resid_norm rows {n} (two norms, residual update)", time_us([lambda h=h, y=y, x=x: ops.resid_norm(h, y, w, w_next=w, xn=x, eps=1e-6) for h, y, x in zip(hs, ys, xs)]), n * d * 12, 0),
+            row(f"rmsnorm rows {n} (other families)", time_us([lambda h=h, x=x: base.rmsnorm(h, w, x, 1e-6) for h, x in zip(hs, xs)]), n * d * 6, 0)]
     k = min(copies_for(n * ff * 6), 64)
     gus, act = [torch.randn(n, 2 * ff, **bf) for _ in range(k)], torch.empty(n, ff, **bf)
-    rows.append(_row(f"gelu_mul rows {n}", time_us([lambda g=g: ops.gelu_mul(g, act) for g in gus]), n * ff * 6, 0))
+    rows.append(row(f"gelu_mul rows {n}", time_us([lambda g=g: ops.gelu_mul(g, act) for g in gus]), n * ff * 6, 0))
     cols = m.q_rank + m.kv_rank + m.rot_dim
-    bt, P, pages = _tables(1, n, dev)
+    bt, P, pages = page_tables(1, n, dev)
     k = min(copies_for(n * cols * 4), 64)
     downs, kv = [torch.randn(n, cols, **bf) for _ in range(k)], torch.zeros(pages, 64, s.width, **bf)
     cqs = [torch.empty(n, s.q_rank, **bf) for _ in range(k)]
     pos, sid = torch.arange(n, dtype=torch.int32, device=dev), torch.zeros(n, dtype=torch.int32, device=dev)
     ang, qn, kn = torch.rand(n, m.rotary.dims // 2, 2, device=dev), torch.ones(m.q_rank, device=dev), torch.ones(m.kv_rank, device=dev)
-    rows.append(_row(f"latent_prep rows {n}", time_us([lambda a=a, c=c: ops.latent_prep(a, qn, kn, ang, pos, sid, bt, c, kv, m.rot_dim, s.latent, 1e-6) for a, c in zip(downs, cqs)]), n * cols * 4, 0))
+    rows.append(row(f"latent_prep rows {n}", time_us([lambda a=a, c=c: ops.latent_prep(a, qn, kn, ang, pos, sid, bt, c, kv, m.rot_dim, s.latent, 1e-6) for a, c in zip(downs, cqs)]), n * cols * 4, 0))
     return rows
 
 
@@ -211,20 +147,20 @@ def products(cfg: ModelConfig, rows_list=(1, 4, 8, 32)) -> list[dict]:
             lins = [DenseLinear(torch.randn(n, k, **bf)) for _ in range(c)]
             x, y = torch.randn(rows, k, **bf), torch.empty(rows, n, **bf)
             kind = "gemv_dense" if rows <= ops.GEMV_MAX_ROWS else "cuBLAS"
-            out.append(_row(f"{name} [{n}, {k}] x {rows} rows ({kind})", time_us([lambda l=l: l(x, y) for l in lins]), n * k * 2, 2.0 * n * k * rows))
+            out.append(row(f"{name} [{n}, {k}] x {rows} rows ({kind})", time_us([lambda l=l: l(x, y) for l in lins]), n * k * 2, 2.0 * n * k * rows))
             del lins
         c = copies_for(ff * d * 4)
         lins = [DenseLinear(torch.randn(2 * ff, d, **bf)) for _ in range(c)]
         x, act, gu = torch.randn(rows, d, **bf), torch.empty(rows, ff, **bf), torch.empty(rows, 2 * ff, **bf)
-        out.append(_row(f"gate|up + gelu [{2 * ff}, {d}] x {rows} rows", time_us([lambda l=l: l.gelu(x, act, gu) for l in lins]), ff * d * 4, 4.0 * ff * d * rows))
+        out.append(row(f"gate|up + gelu [{2 * ff}, {d}] x {rows} rows", time_us([lambda l=l: l.gelu(x, act, gu) for l in lins]), ff * d * 4, 4.0 * ff * d * rows))
         del lins
         if rows <= ops.GEMV_MAX_ROWS:
             c = copies_for(s.heads * s.dim * s.latent * 2)
             ws = [torch.randn(s.heads, s.latent, s.dim, **bf) for _ in range(c)]
             vs = [torch.randn(s.heads, s.vdim, s.latent, **bf) for _ in range(c)]
             q, ql, o = torch.randn(s.heads, rows, s.dim, **bf), torch.empty(s.heads, rows, s.latent, **bf), torch.empty(s.heads, rows, s.vdim, **bf)
-            out.append(_row(f"query into latent space x {rows} rows", time_us([lambda w=w: ops.gemv_dense(w, q, ql) for w in ws]), ws[0].numel() * 2, 0))
-            out.append(_row(f"values from latent space x {rows} rows", time_us([lambda w=w: ops.gemv_dense(w, ql, o) for w in vs]), vs[0].numel() * 2, 0))
+            out.append(row(f"query into latent space x {rows} rows", time_us([lambda w=w: ops.gemv_dense(w, q, ql) for w in ws]), ws[0].numel() * 2, 0))
+            out.append(row(f"values from latent space x {rows} rows", time_us([lambda w=w: ops.gemv_dense(w, ql, o) for w in vs]), vs[0].numel() * 2, 0))
         sc = base.scratch_for(torch.device("cuda", torch.cuda.current_device()))
         n, k = d, ff
         packs = [base.pack_matrix(quantize(torch.randn(n, k, device=dev) * 0.05, GGMLType.Q8_0), GGMLType.Q8_0, n, k)]
@@ -232,62 +168,8 @@ def products(cfg: ModelConfig, rows_list=(1, 4, 8, 32)) -> list[dict]:
             packs.append(replace(packs[0], data=packs[0].data.clone()))
         x, y = torch.randn(rows, k, **bf), torch.empty(rows, n, **bf)
         fn = (lambda w: base.gemv(w, x, y, scratch=sc)) if rows <= base.GEMV_MAX_ROWS else (lambda w: base.gemm(w, x, y, scratch=sc))
-        out.append(_row(f"down [{n}, {k}] x {rows} rows (other families: Q8_0 kernel)", time_us([lambda w=w: fn(w) for w in packs]), packs[0].data.numel(), 2.0 * n * k * rows))
+        out.append(row(f"down [{n}, {k}] x {rows} rows (other families: Q8_0 kernel)", time_us([lambda w=w: fn(w) for w in packs]), packs[0].data.numel(), 2.0 * n * k * rows))
     return out
-
-
-def whole_model(cfg: ModelConfig, recipe: str, prompt: int, batch: int, steps: int = 32) -> dict:
-    """Prefill and decode tokens per second through the engine, device-timed."""
-    from .engine.engine import LLMEngine
-    from .engine.sampling import SamplingParams
-    from .models.synth import synthesize
-    w = synthesize(cfg, recipe, seed=0, device="cuda", with_tokenizer=False)
-    eng = LLMEngine(w, device="cuda", max_batch=batch, max_context=prompt + 2 * steps + 80, max_prefill_tokens=8192)
-    del w
-    g = torch.Generator().manual_seed(1)
-    sp = SamplingParams(temperature=0.0, max_tokens=10 ** 6, ignore_eos=True)
-    make = lambda: [torch.randint(0, cfg.vocab_size, (prompt,), generator=g).tolist() for _ in range(batch)]
-    for warm in (True, False):
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        reqs = [eng.add_request(p, sp) for p in make()]
-        torch.cuda.synchronize()
-        a.record()
-        while eng.waiting:
-            eng.step()
-        b.record()
-        torch.cuda.synchronize()
-        pre = batch * prompt / (a.elapsed_time(b) / 1e3)
-        if warm:
-            for r in reqs:
-                eng.abort(r.rid)
-    for _ in range(4):
-        eng.step()
-    evs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(steps)]
-    eng.step_events = list(evs)
-    for _ in range(steps):
-        eng.step()
-    torch.cuda.synchronize()
-    ms = sum(x.elapsed_time(y) for x, y in evs) / steps
-    eng.step_events = None
-    eng.check_health()
-    res = {"model": cfg.name, "recipe": recipe, "layers": cfg.n_layers, "batch": batch, "prompt": prompt, "prefill_tok_s": round(pre),
-           "decode_ms_per_step": round(ms, 4), "decode_tok_s": round(batch / (ms / 1e3)),
-           "weight_gb": round(eng.model.weight_bytes() / 1e9, 2)}
-    for r in reqs:
-        eng.abort(r.rid)
-    del eng
-    import gc
-    gc.collect()
-    torch.cuda.empty_cache()
-    return res
-
-
-def cut(cfg: ModelConfig, n_layers: int) -> ModelConfig:
-    """The first layers of a shape, unlooped."""
-    kw = dict(n_layers=n_layers)
-    if cfg.is_latent:
-        kw.update(mixers=cfg.mixers[:n_layers], layer_ff=cfg.layer_ff[:n_layers], loop=None)
-    return cfg.with_(**kw)
 
 
 def run(layers: int = 8, log=print) -> dict:

@@ -92,16 +92,20 @@ def test_sizes_without_a_tensor_core_kernel():
 
 
 def test_captured_and_eager_decode_agree_and_launch_own_kernels():
+    """In 32-bit mode both give the same tokens; in bf16 (the key splits depend on the table's width) logits within rounding."""
     m = cases.model("wide", seed=2, gain=1.3)
     prompts = [cases.tokens(n, n) for n in (5, 100, 64)]
-    sp = SamplingParams(temperature=0.0, max_tokens=20, ignore_eos=True)
-    a, b = cases.engine(m, "cuda", BF), cases.engine(m, "cuda", BF, use_graphs=False)
-    n0 = ops.launch_count()
-    assert a.generate(prompts, sp) == b.generate(prompts, sp)
-    assert a.stats["graph_replays"] > 0 and ops.launch_count() > n0
+    greedy = SamplingParams(temperature=0.0, max_tokens=20, ignore_eos=True)
     sampled = SamplingParams(temperature=0.9, top_k=30, top_p=0.95, seed=5, max_tokens=12, ignore_eos=True)
     a, b = cases.engine(m, "cuda", F32), cases.engine(m, "cuda", F32, use_graphs=False)
-    assert a.generate(prompts, sampled) == b.generate(prompts, sampled)
+    n0 = ops.launch_count()
+    for sp in (greedy, sampled):
+        assert a.generate(prompts, sp) == b.generate(prompts, sp)
+    assert a.stats["graph_replays"] > 0 and ops.launch_count() > n0
+    a, b = cases.engine(m, "cuda", BF), cases.engine(m, "cuda", BF, use_graphs=False)
+    t = cases.tokens(150, 3)
+    cases.assert_close(cases.feed_all(a, t, [120, 1]), cases.feed_all(b, t, [120, 1]).cpu(), BF)
+    assert a.stats["graph_replays"] > 0
 
 
 def test_logits_do_not_depend_on_the_batch():
