@@ -82,7 +82,7 @@ def linear_prefill(m, n: int) -> dict:
     assert int(status[0]) == 0
     C = 128
     flops = 2.0 * n * m.heads * (C / 2 * (m.dim + m.vdim) + 2 * m.dim * m.vdim)
-    return row(f"linear_chunk {x.name} rows {n} heads {m.heads} x {m.dim} x {m.vdim} (four launches)", us, 2.0 * n * m.heads * (2 * m.dim + 3 * m.vdim), flops)
+    return row(f"linear_chunk {x.name} rows {n} heads {m.heads} x {m.dim} x {m.vdim} (three launches)", us, 2.0 * n * m.heads * (2 * m.dim + 3 * m.vdim), flops)
 
 
 def gdn_prefill(n: int, heads: int, d: int) -> dict:

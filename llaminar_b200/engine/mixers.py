@@ -94,8 +94,10 @@ class MixerStack:
         L.post_mix = gain("post_attention")
         if isinstance(m, MatrixLSTM):
             L.left, L.right = None, self._build_lstm(w, p, m)
-            L.gate_proj = DenseLinear(torch.cat([self._mat(w, p + "lstm_i.weight"), self._mat(w, p + "lstm_f.weight")]))
-            L.proj = DenseLinear(torch.cat(L.right.rows))
+            gates = torch.cat([self._mat(w, p + "lstm_i.weight"), self._mat(w, p + "lstm_f.weight")])
+            L.gate_proj, L.gate_col = DenseLinear(gates), L.right.cols
+            # decode steps (float rows) take the gates from the one product
+            L.proj = DenseLinear(torch.cat(L.right.rows + [pad_to(gates, pad8(gates.shape[0]), gates.shape[1])]))
         else:
             L.left, L.right = self._build_attention(w, p, m.left), self._build_retention(w, p, m.right)
             L.right.offs = [x + L.left.cols for x in L.right.offs]
@@ -226,8 +228,8 @@ class MixerStack:
         rows = self._rows.view(plan.rows)[:T * L.proj.n_out].view(T, L.proj.n_out)
         L.proj(x, rows)
         if L.left is None:
-            gates = self._gates[:T * L.gate_proj.n_out].view(T, L.gate_proj.n_out)
-            L.gate_proj(x, gates)
+            n = L.gate_proj.n_out
+            gates = rows[:, L.gate_col:L.gate_col + n] if rows.dtype == torch.float32 else L.gate_proj(x, self._gates[:T * n].view(T, n))
             L.right.wo(self._linear(L.right, rows, gates, fb, plan, kv), y)
             ops.resid_norm(h, y, L.post_mix, copy0=x, center_post=True, eps=eps)
         else:

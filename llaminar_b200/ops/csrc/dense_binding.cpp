@@ -99,7 +99,7 @@ void gemv_dense(const Tensor& w, const Tensor& x, const Tensor& out, int64_t act
     p.out = out.data_ptr(); p.o_row = out.stride(1); p.o_z = out.stride(0);
     TORCH_CHECK(reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "gemv_dense operands must be 16-byte aligned");
     TORCH_CHECK((act == llm::ACT_GELU_SIDE) == table.has_value(), "a side table goes with the side activation");
-    p.side = side_table(table, first, cols, tokens, p.m, false);
+    p.side = side_table(table, first, cols, tokens, (int64_t)p.z * p.m, false);
     check(llm::launch_gemv_dense(p, stream()), "gemv_dense");
 }
 

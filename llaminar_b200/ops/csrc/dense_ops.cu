@@ -158,6 +158,107 @@ __global__ void __launch_bounds__(THREADS) resid_norm_kernel(const ResidNormPara
     }
 }
 
+// The same for rows that the threads hold in registers (NV x 4 values each): every load is on its way before the first sum.
+template <class T, int THREADS, int NV>
+__global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNormParams p) {
+    constexpr int W = THREADS / 32;
+    __shared__ float2 red[5][W];
+    pdl_trigger();
+    const size_t t = blockIdx.x;
+    const int d = p.d;
+    float* h = p.h + t * d;
+    auto at = [&](int n) { return (n * THREADS + (int)threadIdx.x) * 4; };
+    auto each = [&](auto f) {
+#pragma unroll
+        for (int n = 0; n < NV; ++n)
+            if (at(n) < d) f(n, at(n));
+    };
+    int used = 0;                                              // sums so far: each has its own place in `red`
+    auto block_sum2 = [&](float x, float y) {
+        x = warp_sum(x); y = warp_sum(y);
+        float2(&r)[W] = red[used++];
+        if ((threadIdx.x & 31) == 0) r[threadIdx.x >> 5] = make_float2(x, y);
+        __syncthreads();
+        float2 s = make_float2(0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < W; ++i) { s.x += r[i].x; s.y += r[i].y; }
+        return s;
+    };
+    float v[NV][4], a[NV][4] = {}, w[NV][4];
+    // mean (0 unless `center`) and 1 / root mean square around it
+    auto norm_of = [&](bool center, float& mean) {
+        float sum = 0.f, ss = 0.f;
+        each([&](int n, int) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) { sum += v[n][j]; ss += v[n][j] * v[n][j]; }
+        });
+        const float2 s = block_sum2(sum, ss);
+        mean = 0.f;
+        ss = s.y;
+        if (center) {
+            mean = s.x / (float)d;
+            float q = 0.f;
+            each([&](int n, int) {
+#pragma unroll
+                for (int j = 0; j < 4; ++j) q += (v[n][j] - mean) * (v[n][j] - mean);
+            });
+            ss = block_sum2(q, 0.f).x;
+        }
+        return 1.f / sqrtf(ss / (float)d + p.eps);
+    };
+    if (p.y && p.w_post) each([&](int n, int i) { Vec4<float>::load(p.w_post + i, w[n]); });
+    pdl_wait();
+    if (!p.y || p.add) each([&](int n, int i) { Vec4<float>::load(h + i, a[n]); });
+    if (p.y) {
+        const size_t r = p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[t], p.n_y_rows) : t;
+        const T* y = static_cast<const T*>(p.y) + r * p.y_stride;
+        each([&](int n, int i) { Vec4<T>::load(y + i, v[n]); });
+        if (p.y2) {
+            const T* y2 = static_cast<const T*>(p.y2) + t * p.y2_stride;
+            float u[NV][4], sa = 0.f, sb = 0.f;
+            each([&](int n, int i) {
+                Vec4<T>::load(y2 + i, u[n]);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) { sa += v[n][j] * v[n][j]; sb += u[n][j] * u[n][j]; }
+            });
+            const float2 s = block_sum2(sa, sb);
+            const float ia = 0.5f / sqrtf(s.x / (float)d + p.eps), ib = 0.5f / sqrtf(s.y / (float)d + p.eps);
+            each([&](int n, int i) {
+                float wa[4], wb[4];
+                Vec4<float>::load(p.w_y + i, wa); Vec4<float>::load(p.w_y2 + i, wb);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) v[n][j] = v[n][j] * ia * wa[j] + u[n][j] * ib * wb[j];
+            });
+        }
+        float mean = 0.f;
+        const float inv = p.w_post ? norm_of(p.center_post, mean) : p.factor;
+        each([&](int n, int i) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[n][j] = a[n][j] + (v[n][j] - mean) * inv * (p.w_post ? w[n][j] : 1.f);
+            Vec4<float>::store(h + i, v[n]);
+        });
+    } else {
+        each([&](int n, int) {
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[n][j] = a[n][j];
+        });
+    }
+    each([&](int n, int i) {
+        if (p.copy0) Vec4<T>::store(static_cast<T*>(p.copy0) + t * p.copy_stride + i, v[n]);
+        if (p.copy1) Vec4<T>::store(static_cast<T*>(p.copy1) + t * p.copy_stride + i, v[n]);
+    });
+    if (!p.w_next) return;
+    float mean;
+    const float inv = norm_of(p.center_next, mean);
+    T* xn = static_cast<T*>(p.xn) + t * d;
+    each([&](int n, int i) {
+        Vec4<float>::load(p.w_next + i, w[n]);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) v[n][j] = (v[n][j] - mean) * inv * w[n][j];
+        Vec4<T>::store(xn + i, v[n]);
+    });
+}
+
 // value `i` of row `t` of the activation of `x`; `u`: the second half's value (GELU_MUL)
 template <int ACT, class T>
 LLM_DEVICE float activated(float x, float u, const SideTable& s, int t, int i) {
@@ -268,7 +369,7 @@ __global__ void __launch_bounds__(32 * SKINNY_WARPS) gemv_dense_kernel(const Gem
         }
         // rounded like the stored projection of the unfused form
         if constexpr (ACT != ACT_NONE)
-            v = activated<ACT, __nv_bfloat16>(__bfloat162float(__float2bfloat16(v)), __bfloat162float(__float2bfloat16(v2)), p.side, m, n);
+            v = activated<ACT, __nv_bfloat16>(__bfloat162float(__float2bfloat16(v)), __bfloat162float(__float2bfloat16(v2)), p.side, blockIdx.y * p.m + m, n);
         static_cast<TO*>(p.out)[(size_t)blockIdx.y * p.o_z + m * p.o_row + n] = from_f<TO>(v);
     }
 }
@@ -287,7 +388,11 @@ cudaError_t resid_norm_any(const ResidNormParams& p, int rows, cudaStream_t st) 
         cudaError_t e = raise_smem(kernel, smem);
         return e != cudaSuccess ? e : launch_pdl(kernel, dim3(rows), dim3(threads), smem, st, p);
     };
-    if (vec && p.d <= 1024) return go(resid_norm_kernel<T, 4, 128>, 128);
+    auto go_reg = [&](auto kernel, int threads) { return launch_pdl(kernel, dim3(rows), dim3(threads), 0, st, p); };
+    if (vec && p.d <= 1024) return go_reg(resid_norm_reg_kernel<T, 128, 2>, 128);
+    if (vec && p.d <= 2048) return go_reg(resid_norm_reg_kernel<T, 256, 2>, 256);
+    if (vec && p.d <= 4096) return go_reg(resid_norm_reg_kernel<T, 512, 2>, 512);
+    if (vec && p.d <= 8192) return go_reg(resid_norm_reg_kernel<T, 512, 4>, 512);
     if (vec) return go(resid_norm_kernel<T, 4, 512>, 512);
     return go(resid_norm_kernel<T, 1, 256>, 256);
 }

@@ -12,7 +12,7 @@
 //
 //   chunk_state   per chunk and head: sum_j e^(a_j - A_L) v_j k_j^T           tcgen05, M = 128 values, N = dim, K = 128 rows
 //   chunk_scan    per head: the states in front of every chunk, one after the other, and the sequence's new state
-//   chunk_out     per chunk and head: scores, weights, o                     tcgen05, M = 128 rows, N = 128 rows / values
+//   chunk_out     per chunk and head: scores, weights, o, norm and gate      tcgen05, M = 128 rows, N = 128 rows / values
 //
 // What enters the state, the state and the weights stay at 32-bit accuracy: such operands are split into two bf16 numbers and
 // multiplied twice (q, k and v as projected are bf16 already).  Logarithms are to base 2 inside the kernels.
@@ -73,29 +73,49 @@ LLM_DEVICE Gates chunk_gates(const LinearParams& p, int h, int r0, int len, floa
     return r;
 }
 
-// values u * 8 .. u * 8 + 7 of head vector x (dim values), turned by the row's angles
-LLM_DEVICE void head_unit(const __nv_bfloat16* x, int u, int dim, const float2* ang, int half, float (&v)[8]) {
-    const int i0 = u * 8;
-    if (half % 8 == 0 && i0 < 2 * half) {
-        const bool first = i0 < half;
-        const int a0 = first ? i0 : i0 - half;
-        const uint4 own = *reinterpret_cast<const uint4*>(x + i0), other = *reinterpret_cast<const uint4*>(x + (first ? i0 + half : i0 - half));
-        const uint32_t a[4] = {own.x, own.y, own.z, own.w}, b[4] = {other.x, other.y, other.z, other.w};
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const float2 c0 = ang[a0 + 2 * j], c1 = ang[a0 + 2 * j + 1];
-            v[2 * j] = bf16_lo(a[j]) * c0.x + bf16_lo(b[j]) * (first ? -c0.y : c0.y);
-            v[2 * j + 1] = bf16_hi(a[j]) * c1.x + bf16_hi(b[j]) * (first ? -c1.y : c1.y);
-        }
-    } else if (i0 >= 2 * half) {
-        const uint4 own = *reinterpret_cast<const uint4*>(x + i0);
-        const uint32_t a[4] = {own.x, own.y, own.z, own.w};
+// The 16-byte units of a head's q or k row, turned by the row's angles, in work items: an item is one unit, or with rotated halves
+// of whole units the two units that turn into each other.
+struct RotItems { int pairs, count; };           // pairs: of units; items of a row
+template <bool ROT> LLM_DEVICE RotItems rot_items(int nu, int half) {
+    const int pairs = ROT && half % 8 == 0 ? half / 8 : 0;
+    return {pairs, nu - pairs};
+}
+// item `i` of row x (dim values, zero units behind): f(unit, values)
+template <bool ROT, class F> LLM_DEVICE void rot_item(const __nv_bfloat16* x, int i, const RotItems& it, int dim, const float2* ang, int half, F&& f) {
+    auto unpack = [](const uint4& w, float (&v)[8]) {
+        const uint32_t a[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
         for (int j = 0; j < 4; ++j) { v[2 * j] = bf16_lo(a[j]); v[2 * j + 1] = bf16_hi(a[j]); }
-    } else {
+    };
+    if (ROT && i < it.pairs) {
+        float u[8], w[8], a[8], b[8];
+        unpack(*reinterpret_cast<const uint4*>(x + i * 8), u);
+        unpack(*reinterpret_cast<const uint4*>(x + half + i * 8), w);
+        float4 cs[4];                                               // cos, sin of two pairs each; rows of 8 float2: 16-byte aligned
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] = rotated(x, i0 + j, ang, half);
+        for (int j = 0; j < 4; ++j) cs[j] = *reinterpret_cast<const float4*>(ang + i * 8 + 2 * j);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            a[2 * j] = u[2 * j] * cs[j].x - w[2 * j] * cs[j].y;
+            b[2 * j] = w[2 * j] * cs[j].x + u[2 * j] * cs[j].y;
+            a[2 * j + 1] = u[2 * j + 1] * cs[j].z - w[2 * j + 1] * cs[j].w;
+            b[2 * j + 1] = w[2 * j + 1] * cs[j].z + u[2 * j + 1] * cs[j].w;
+        }
+        f(i, a);
+        f(i + it.pairs, b);
+        return;
     }
+    const int u = i + it.pairs;
+    float v[8] = {};
+    if (u * 8 < dim) {
+        if (ROT && it.pairs == 0) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = rotated(x, u * 8 + j, ang, half);
+        } else {
+            unpack(*reinterpret_cast<const uint4*>(x + u * 8), v);
+        }
+    }
+    f(u, v);
 }
 // two bf16 numbers whose sum is x to 16 bits of mantissa
 LLM_DEVICE void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
@@ -162,25 +182,37 @@ __global__ void __launch_bounds__(THREADS, 2) chunk_state_kernel(const __grid_co
         __syncthreads();
     }
     const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(p.in) + (size_t)r0 * p.in_row + p.k_off + h * p.dim;
-    const int groups = THREADS / nu, u = tid % nu, grp = tid / nu;
-    float sum[8] = {};
+    const RotItems items = rot_items<ROT>(nu, p.half);
+    const int groups = THREADS / items.count, item = tid % items.count, grp = tid / items.count;
+    float sum[2][8] = {};                                             // of this thread's rows, by unit of the item
     for (int j = grp; j < C && grp < groups; j += groups) {
-        float v[8] = {};
-        if (j < len && u * 8 < p.dim) {
-            head_unit(kp + (size_t)j * p.in_row, u, p.dim, ROT ? p.angles + (size_t)(r0 + j) * p.half : nullptr, ROT ? p.half : 0, v);
-            const float w = s_w[j];
+        const float w = s_w[j];
+        int part = 0;
+        auto put = [&](int u, float (&v)[8]) {
+            uint32_t hi[4], lo[4];
 #pragma unroll
-            for (int e = 0; e < 8; ++e) { v[e] *= w; sum[e] += v[e]; }
+            for (int e = 0; e < 8; ++e) { v[e] *= w; sum[part][e] += v[e]; }
+#pragma unroll
+            for (int e = 0; e < 4; ++e) split_bf16(v[2 * e], v[2 * e + 1], hi[e], lo[e]);
+            st_shared_v4(atom_addr(sH + (u >> 3) * ATOM, j, u & 7), make_uint4(hi[0], hi[1], hi[2], hi[3]));
+            st_shared_v4(atom_addr(sL + (u >> 3) * ATOM, j, u & 7), make_uint4(lo[0], lo[1], lo[2], lo[3]));
+            part = 1;
+        };
+        if (j < len) {
+            rot_item<ROT>(kp + (size_t)j * p.in_row, item, items, p.dim, ROT ? p.angles + (size_t)(r0 + j) * p.half : nullptr, p.half, put);
+        } else {
+            float v[8] = {};
+            put(item < items.pairs ? item : item + items.pairs, v);
+            if (item < items.pairs) { float z[8] = {}; put(item + items.pairs, z); }
         }
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) split_bf16(v[2 * e], v[2 * e + 1], hi[e], lo[e]);
-        st_shared_v4(atom_addr(sH + (u >> 3) * ATOM, j, u & 7), make_uint4(hi[0], hi[1], hi[2], hi[3]));
-        st_shared_v4(atom_addr(sL + (u >> 3) * ATOM, j, u & 7), make_uint4(lo[0], lo[1], lo[2], lo[3]));
     }
     if (p.gates && v0 == 0 && grp < groups) {
+        if (item < items.pairs) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) s_red[grp * n16 + u * 8 + e] = sum[e];
+            for (int e = 0; e < 8; ++e) s_red[grp * n16 + (item + items.pairs) * 8 + e] = sum[1][e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s_red[grp * n16 + (item < items.pairs ? item : item + items.pairs) * 8 + e] = sum[0][e];
     }
     fence_proxy_async();
     __syncthreads();
@@ -208,16 +240,26 @@ __global__ void __launch_bounds__(THREADS, 2) chunk_state_kernel(const __grid_co
     ok = ok && mbar_wait_warp(bar_d, 0, abort_flag);
     if (ok) {
         tc_fence_after();
-        const int row = v0 + (warp & 3) * 32 + lane;
-        float* dst = c.state + (((size_t)blockIdx.x * p.heads + h) * p.vdim + row) * p.dim;
+        // through shared memory (the operands are done with): rows of 512 bytes, 16-byte units swizzled, then whole rows to memory
+        const int row = (warp & 3) * 32 + lane;
+        auto unit_at = [&](int r, int u) { return sV + r * 512 + (((u & ~7) | ((u ^ r) & 7)) << 4); };
         for (int c0 = (warp >> 2) * 16; c0 < n16; c0 += 32) {
             uint32_t r[16];
             tmem_ld_n<16>(tmem + ((uint32_t)((warp & 3) * 32) << 16) + c0, r);
-            if (row < p.vdim)
 #pragma unroll
-                for (int e = 0; e < 16; e += 4)
-                    if (c0 + e < p.dim) *reinterpret_cast<uint4*>(dst + c0 + e) = make_uint4(r[e], r[e + 1], r[e + 2], r[e + 3]);
+            for (int e = 0; e < 4; ++e) st_shared_v4(unit_at(row, c0 / 4 + e), make_uint4(r[4 * e], r[4 * e + 1], r[4 * e + 2], r[4 * e + 3]));
         }
+    }
+    __syncthreads();
+    if (ok) {
+        float* dst = c.state + (((size_t)blockIdx.x * p.heads + h) * p.vdim + v0) * p.dim;
+        const int rows = min(VS, p.vdim - v0);
+        for (int r = warp; r < rows; r += THREADS / 32)
+            if (lane * 4 < p.dim) {
+                uint4 w;
+                asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(w.x), "=r"(w.y), "=r"(w.z), "=r"(w.w) : "r"(sV + r * 512 + (((lane & ~7) | ((lane ^ r) & 7)) << 4)));
+                *reinterpret_cast<uint4*>(dst + (size_t)r * p.dim + lane * 4) = w;
+            }
     }
     end_cta(s_abort, c.status, tmem, 128);
 }
@@ -290,27 +332,43 @@ __global__ void __launch_bounds__(32 * SCAN_WARPS) chunk_scan_kernel(const Linea
 // (chunk_out runs behind chunk_scan and in front of any other use of the slots: the new stabilisers can be stored by it)
 
 // ---- outputs --------------------------------------------------------------------------------------------------------------------
-constexpr int T_S = 0, T_P = 128, T_O = 256, T_I = 384;              // TMEM columns: scores, weights (hi, lo), both parts of o
-enum OBar { B_QK = 0, B_V, B_ST, B_SC, B_IN, B_O, N_OBARS };
+// A CTA takes 256 values of a head (all of most heads) in two slices, so that the weights are computed once.  Shared memory, in atoms:
+// Q [na] | K, then V of slice 1 [2] | V of slice 0, then gate of slice 1 [2] | state [2 na: hi, lo], of one slice after the other |
+// gate of slice 0 [2].  With the whole head here (`fused`) the norm and the gate follow, otherwise head_gate does them.
+constexpr int T_S = 0, T_P = 128, T_O = 256, T_I = 384;              // TMEM columns: scores (then T_I of slice 1), weights (hi, lo), both parts of o
+// (a barrier that is waited for twice is not used again before every thread has seen its first phase)
+enum OBar { B_QK = 0, B_V, B_V1, B_G, B_G1, B_ST, B_SC, B_IN, B_IN1, B_O, N_OBARS };
 
 template <bool ROT>
 __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
-                                                               const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_s,
-                                                               const LinearParams p, const LinearChunks c) {
+                                                               const __grid_constant__ CUtensorMap map_v, const __grid_constant__ CUtensorMap map_g,
+                                                               const __grid_constant__ CUtensorMap map_s, const LinearParams p, const LinearChunks c) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t s_bars[N_OBARS];
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort[2];
-    __shared__ float s_tmp[2][4], s_top[C], s_keep[C], s_floor[C], s_x[2][C];
+    __shared__ float s_tmp[2][4], s_top[C], s_keep[C], s_floor[C], s_x[2][C], s_y[2][C];
     __shared__ __align__(16) float s_a[C], s_n[128];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int4 ck = c.chunks[blockIdx.x];
-    const int h = blockIdx.y, v0 = blockIdx.z * VS, r0 = ck.x, len = ck.y;
-    const int na = (p.dim + 63) / 64, ksteps = (p.dim + 15) / 16, nv = min(VS, (p.vdim - v0 + 15) / 16 * 16);
+    const int h = blockIdx.y, v0 = blockIdx.z * 2 * VS, r0 = ck.x, len = ck.y;
+    const int na = (p.dim + 63) / 64, nkv = max(na, 2), ksteps = (p.dim + 15) / 16;
+    const int slices = p.vdim - v0 > VS ? 2 : 1;
+    const bool lstm = p.gates != nullptr, fused = gridDim.z == 1;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
-    const uint32_t sQ = base, sK = sQ + na * ATOM, sV = sK + na * ATOM, sS = sV + 2 * ATOM;      // sS: hi atoms, then lo
+    const uint32_t sQ = base, sK = sQ + na * ATOM, sV = sK + nkv * ATOM, sS = sV + 2 * ATOM, sG = sS + 2 * na * ATOM;
     const uint32_t bars = smem_u32(s_bars);
     auto bar = [&](int i) { return bars + i * 8; };
+    auto width = [&](int s) { return min(VS, (p.vdim - v0 - s * VS + 15) / 16 * 16); };       // values of slice s, whole MMA steps
+    auto load_rows = [&](uint32_t dst, const CUtensorMap* map, int s, int b) {                 // [rows][128 values of slice s]
+        mbar_arrive_expect_tx(bar(b), 2 * ATOM);
+        for (int a = 0; a < 2; ++a) tma_load_3d(dst + a * ATOM, map, v0 + s * VS + a * 64, h, r0, bar(b));
+    };
+    auto load_state = [&](int s) {
+        mbar_arrive_expect_tx(bar(B_ST), 2 * na * ATOM);
+        for (int part = 0; part < 2; ++part)
+            for (int a = 0; a < na; ++a) tma_load_4d(sS + (part * na + a) * ATOM, &map_s, a * 64, part, v0 + s * VS, blockIdx.x * p.heads + h, bar(B_ST));
+    };
     begin_cta(s_bars, N_OBARS, &s_tmem, s_abort, 512);
     const uint32_t tmem = s_tmem;
     volatile int* abort_flag = s_abort;
@@ -323,24 +381,25 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
                 tma_load_3d(sK + a * ATOM, &map_k, a * 64, h, r0, bar(B_QK));
             }
         }
-        mbar_arrive_expect_tx(bar(B_ST), 2 * na * ATOM);
-        for (int part = 0; part < 2; ++part)
-            for (int a = 0; a < na; ++a) tma_load_4d(sS + (part * na + a) * ATOM, &map_s, a * 64, part, v0, blockIdx.x * p.heads + h, bar(B_ST));
-        mbar_arrive_expect_tx(bar(B_V), 2 * ATOM);
-        for (int a = 0; a < 2; ++a) tma_load_3d(sV + a * ATOM, &map_v, v0 + a * 64, h, r0, bar(B_V));
+        load_state(0);
+        load_rows(sV, &map_v, 0, B_V);
+        if (fused) load_rows(sG, &map_g, 0, B_G);
     }
     if constexpr (ROT) {
         const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.in) + (size_t)r0 * p.in_row + h * p.dim;
-        const int nu = ksteps * 2;
-        for (int i = tid; i < 2 * C * nu; i += THREADS) {
-            const int which = i / (C * nu), x = i - which * C * nu, j = x / nu, u = x - j * nu;
-            float v[8] = {};
-            if (j < len && u * 8 < p.dim) head_unit(in + (size_t)j * p.in_row + (which ? p.k_off : p.q_off), u, p.dim, p.angles + (size_t)(r0 + j) * p.half, p.half, v);
-            st_shared_v4(atom_addr((which ? sK : sQ) + (u >> 3) * ATOM, j, u & 7),
-                         make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7])));
+        const RotItems items = rot_items<true>(ksteps * 2, p.half);
+        const int n = 2 * items.count, groups = THREADS / n, item = tid % n, which = item >= items.count;
+        const uint32_t dst = which ? sK : sQ;
+        for (int j = tid / n; j < C && tid / n < groups; j += groups) {
+            auto put = [&](int u, float (&v)[8]) {
+                st_shared_v4(atom_addr(dst + (u >> 3) * ATOM, j, u & 7),
+                             make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7])));
+            };
+            // rows past the chunk repeat its last one (their results are not stored)
+            const int r = min(j, len - 1);
+            rot_item<true>(in + (size_t)r * p.in_row + (which ? p.k_off : p.q_off), item - which * items.count, items, p.dim, p.angles + (size_t)(r0 + r) * p.half, p.half, put);
         }
     }
-    const bool lstm = p.gates != nullptr;
     {
         const Gates g = chunk_gates(p, h, r0, len, s_tmp);
         if (tid < C) {
@@ -356,10 +415,40 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
     if (ROT) fence_proxy_async();
     __syncthreads();
     bool ok = true;
+    // one warp issues: o's part from the state of slice s into column t_i
+    auto issue_in = [&](int s, uint32_t t_i) {
+        ok = ok && mbar_wait_warp(bar(B_ST), s, abort_flag);
+        if (ok && elect_one()) {
+            const uint64_t q = smem_desc_sw128(sQ), st = smem_desc_sw128(sS);
+            const uint32_t idesc = instr_desc(width(s));
+            for (int ks = 0; ks < ksteps; ++ks) {
+                const uint32_t off = (ks >> 2) * (ATOM / 16) + 2 * (ks & 3);
+                mma_f16(tmem + t_i, q + off, st + off, idesc, ks > 0 ? 1u : 0u);
+                mma_f16(tmem + t_i, q + off, st + off + na * (ATOM / 16), idesc, 1u);
+            }
+            mma_commit(bar(s ? B_IN1 : B_IN));
+        }
+        __syncwarp();
+    };
+    auto issue_o = [&](int s) {
+        ok = ok && mbar_wait_warp(bar(s ? B_V1 : B_V), 0, abort_flag);
+        tc_fence_after();
+        if (ok && elect_one()) {
+            const uint64_t v = smem_desc_mn_sw128(s ? sK : sV, ATOM);
+            const uint32_t idesc = instr_desc(width(s)) | (1u << 16);
+#pragma unroll
+            for (int ks = 0; ks < C / 16; ++ks) {
+                mma_f16_ts(tmem + T_O, tmem + T_P + ks * 8, v + ks * (2048 / 16), idesc, ks > 0 ? 1u : 0u);
+                mma_f16_ts(tmem + T_O, tmem + T_P + 64 + ks * 8, v + ks * (2048 / 16), idesc, 1u);
+            }
+            mma_commit(bar(B_O));
+        }
+        __syncwarp();
+    };
     if (warp == 0) {
         if (!ROT) ok = mbar_wait_warp(bar(B_QK), 0, abort_flag);
-        const uint64_t q = smem_desc_sw128(sQ), k = smem_desc_sw128(sK), s = smem_desc_sw128(sS);
         if (ok && elect_one()) {
+            const uint64_t q = smem_desc_sw128(sQ), k = smem_desc_sw128(sK);
             for (int ks = 0; ks < ksteps; ++ks) {
                 const uint32_t off = (ks >> 2) * (ATOM / 16) + 2 * (ks & 3);
                 mma_f16(tmem + T_S, q + off, k + off, instr_desc(C), ks > 0 ? 1u : 0u);
@@ -367,16 +456,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
             mma_commit(bar(B_SC));
         }
         __syncwarp();
-        ok = ok && mbar_wait_warp(bar(B_ST), 0, abort_flag);
-        if (ok && elect_one()) {
-            for (int ks = 0; ks < ksteps; ++ks) {
-                const uint32_t off = (ks >> 2) * (ATOM / 16) + 2 * (ks & 3);
-                mma_f16(tmem + T_I, q + off, s + off, instr_desc(nv), ks > 0 ? 1u : 0u);
-                mma_f16(tmem + T_I, q + off, s + off + na * (ATOM / 16), instr_desc(nv), 1u);
-            }
-            mma_commit(bar(B_IN));
-        }
-        __syncwarp();
+        issue_in(0, T_I);
     }
     // weights: two threads per row (= TMEM lane), 64 columns each
     const int row = (warp & 3) * 32 + lane, half = warp >> 2;
@@ -385,6 +465,8 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
     ok = ok && mbar_wait_warp(bar(B_SC), 0, abort_flag);
     if (ok) {
         tc_fence_after();
+        if (slices == 2 && tid == 0) load_rows(sK, &map_v, 1, B_V1);      // the keys are done with
+        __syncwarp();
         const float top = s_top[row], scale = p.q_scale * p.k_scale;
         float sum = 0.f;
         uint32_t hi[32], lo[32];
@@ -429,42 +511,98 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
         tmem_wait_st();
         tc_fence_before();
     }
-    __syncthreads();
+    __syncthreads();                                                     // weights are in place, the scores have been read
     if (warp == 0) {
-        ok = ok && mbar_wait_warp(bar(B_V), 0, abort_flag);
-        tc_fence_after();
-        if (ok && elect_one()) {
-            const uint64_t v = smem_desc_mn_sw128(sV, ATOM);
-            const uint32_t idesc = instr_desc(nv) | (1u << 16);
-#pragma unroll
-            for (int ks = 0; ks < C / 16; ++ks) {
-                mma_f16_ts(tmem + T_O, tmem + T_P + ks * 8, v + ks * (2048 / 16), idesc, ks > 0 ? 1u : 0u);
-                mma_f16_ts(tmem + T_O, tmem + T_P + 64 + ks * 8, v + ks * (2048 / 16), idesc, 1u);
-            }
-            mma_commit(bar(B_O));
+        issue_o(0);
+        if (slices == 2) {
+            ok = ok && mbar_wait_warp(bar(B_IN), 0, abort_flag);         // the state of slice 0 is done with
+            if (ok && elect_one()) load_state(1);
+            __syncwarp();
+            issue_in(1, T_S);
         }
-        __syncwarp();
     }
-    ok = ok && mbar_wait_warp(bar(B_IN), 0, abort_flag) && mbar_wait_warp(bar(B_O), 0, abort_flag);
-    if (ok) {
-        tc_fence_after();
-        const float keep = s_keep[row];
-        const float inv = lstm ? 1.f / (fmaxf(fabsf(s_x[0][row] + s_x[1][row]), s_floor[row]) + NORM_FLOOR) : 1.f;
-        __nv_bfloat16* dst = c.o + (size_t)(r0 + row) * p.heads * p.vdim + (size_t)h * p.vdim + v0;
+    const float keep = s_keep[row];
+    const float inv = lstm ? 1.f / (fmaxf(fabsf(s_x[0][row] + s_x[1][row]), s_floor[row]) + NORM_FLOOR) : 1.f;
+    uint32_t o[2][32];
+    float ss = 0.f;
 #pragma unroll
-        for (int q = 0; q < 4; ++q) {
-            const int c0 = half * 64 + q * 16;
-            if (c0 >= nv) break;                                         // the same for all threads of the warp
-            uint32_t a[16], b[16];
-            tmem_ld_n<16>(t_lane + T_O + c0, a);
-            tmem_ld_n<16>(t_lane + T_I + c0, b);
-            uint32_t w[8];
+    for (int s = 0; s < 2; ++s) {
+        if (s < slices) {
+            ok = ok && mbar_wait_warp(bar(s ? B_IN1 : B_IN), 0, abort_flag) && mbar_wait_warp(bar(B_O), s, abort_flag);
+            if (ok) {
+                tc_fence_after();
+                if (fused && s == 0 && slices == 2 && tid == 0) load_rows(sV, &map_g, 1, B_G1);       // the values of slice 0 are done with
+                __syncwarp();
+                const int w = width(s);
 #pragma unroll
-            for (int i = 0; i < 8; ++i)
-                w[i] = pack_bf16((__uint_as_float(a[2 * i]) + keep * __uint_as_float(b[2 * i])) * inv, (__uint_as_float(a[2 * i + 1]) + keep * __uint_as_float(b[2 * i + 1])) * inv);
-            if (row < len) {
-                if (v0 + c0 < p.vdim) *reinterpret_cast<uint4*>(dst + c0) = make_uint4(w[0], w[1], w[2], w[3]);
-                if (v0 + c0 + 8 < p.vdim) *reinterpret_cast<uint4*>(dst + c0 + 8) = make_uint4(w[4], w[5], w[6], w[7]);
+                for (int q = 0; q < 4; ++q) {
+                    const int c0 = half * 64 + q * 16;
+                    if (c0 < w) {                                        // the same for all threads of the warp
+                        uint32_t a[16], b[16];
+                        tmem_ld_n<16>(t_lane + T_O + c0, a);
+                        tmem_ld_n<16>(t_lane + (s ? T_S : T_I) + c0, b);
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            const float x = (__uint_as_float(a[2 * i]) + keep * __uint_as_float(b[2 * i])) * inv;
+                            const float y = (__uint_as_float(a[2 * i + 1]) + keep * __uint_as_float(b[2 * i + 1])) * inv;
+                            ss += x * x + y * y;
+                            o[s][q * 8 + i] = pack_bf16(x, y);
+                        }
+                    }
+                }
+                tc_fence_before();
+            }
+            if (s == 0 && slices == 2) {
+                __syncthreads();                                         // slice 0 has been read out of tensor memory
+                if (warp == 0) issue_o(1);
+            }
+        }
+    }
+    s_y[half][row] = ss;
+    __syncthreads();
+    const float rms = fused ? 1.f / sqrtf((s_y[0][row] + s_y[1][row]) / (float)p.true_vdim + p.eps) : 1.f;
+#pragma unroll
+    for (int s = 0; s < 2; ++s) {
+        if (s < slices) {
+            // gated values into the gate's own place (fused), or o as it is; then whole rows to memory
+            const uint32_t tile = s ? sV : sG;
+            if (fused) ok = ok && mbar_wait_warp(bar(s ? B_G1 : B_G), 0, abort_flag);
+            const int w = width(s);
+            if (ok) {
+#pragma unroll
+                for (int q = 0; q < 8; ++q) {
+                    const int c0 = half * 64 + q * 8;
+                    if (c0 < w) {
+                        const uint32_t at = atom_addr(tile + half * ATOM, row, q);
+                        uint32_t r[4] = {o[s][4 * q], o[s][4 * q + 1], o[s][4 * q + 2], o[s][4 * q + 3]};
+                        if (fused) {
+                            uint32_t g[4];
+                            asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(g[0]), "=r"(g[1]), "=r"(g[2]), "=r"(g[3]) : "r"(at));
+                            const int col = v0 + s * VS + c0;
+#pragma unroll
+                            for (int i = 0; i < 4; ++i) {
+                                const float za = bf16_lo(g[i]), zb = bf16_hi(g[i]);
+                                float x = bf16_lo(r[i]) * rms * (p.silu ? za : 1.f) * __fdividef(1.f, 1.f + __expf(-za));
+                                float y = bf16_hi(r[i]) * rms * (p.silu ? zb : 1.f) * __fdividef(1.f, 1.f + __expf(-zb));
+                                if (p.norm_w && col < p.vdim) { x *= p.norm_w[h * p.vdim + col + 2 * i]; y *= p.norm_w[h * p.vdim + col + 2 * i + 1]; }
+                                r[i] = pack_bf16(x, y);
+                            }
+                        }
+                        st_shared_v4(at, make_uint4(r[0], r[1], r[2], r[3]));
+                    }
+                }
+            }
+            __syncthreads();
+            if (ok) {
+                __nv_bfloat16* dst = (fused ? static_cast<__nv_bfloat16*>(p.out) + (size_t)r0 * p.out_row : c.o + (size_t)r0 * p.heads * p.vdim) + (size_t)h * p.vdim + v0 + s * VS;
+                const size_t stride = fused ? p.out_row : (size_t)p.heads * p.vdim;
+                const int u = lane & 15;
+                for (int r = warp * 2 + (lane >> 4); r < len; r += THREADS / 16)
+                    if (v0 + s * VS + u * 8 < p.vdim) {
+                        uint4 x;
+                        asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(x.x), "=r"(x.y), "=r"(x.z), "=r"(x.w) : "r"(atom_addr(tile + (u >> 3) * ATOM, r, u & 7)));
+                        *reinterpret_cast<uint4*>(dst + (size_t)r * stride + u * 8) = x;
+                    }
             }
         }
     }
@@ -476,8 +614,11 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
     end_cta(s_abort, c.status, tmem, 512);
 }
 
-static size_t state_smem(int dim) { return (size_t)(2 + 2 * ((dim + 63) / 64)) * ATOM + 1024; }
-static size_t out_smem(int dim) { return (size_t)(2 + 4 * ((dim + 63) / 64)) * ATOM + 1024; }
+static size_t state_smem(int dim) { return (size_t)(2 + 2 * ((dim + 63) / 64)) * ATOM + 1024; }       // at least the 64 KB of the staged result
+static size_t out_smem(int dim) {
+    const int na = (dim + 63) / 64;
+    return (size_t)(3 * na + (na > 2 ? na : 2) + 4) * ATOM + 1024;
+}
 
 }  // namespace lin
 
@@ -486,11 +627,11 @@ bool linear_chunk_fits(int dim, int vdim) { return dim % 8 == 0 && vdim % 8 == 0
 cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cudaStream_t st) {
     using namespace lin;
     if (c.n_chunks == 0) return cudaSuccess;
-    if (!linear_chunk_fits(p.dim, p.vdim) || p.in_row % 8 || p.q_off % 8 || p.k_off % 8 || p.v_off % 8 || p.heads > 65535 || c.n_seqs > 65535 ||
-        (!p.gates == !p.decay))
+    if (!linear_chunk_fits(p.dim, p.vdim) || p.in_row % 8 || p.q_off % 8 || p.k_off % 8 || p.v_off % 8 || p.g_off % 8 || p.out_row % 8 || p.heads > 65535 || c.n_seqs > 65535 ||
+        (!p.gates == !p.decay) || (p.gates && p.half))
         return cudaErrorInvalidValue;
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.in);
-    CUtensorMap mq, mk, mv, ms;
+    CUtensorMap mq, mk, mv, mg, ms;
     auto rows_map = [&](CUtensorMap* m, int off, int size) {             // [T][heads][size]
         const cuuint64_t dims[3] = {(cuuint64_t)size, (cuuint64_t)p.heads, (cuuint64_t)c.rows}, strides[2] = {(cuuint64_t)size, (cuuint64_t)p.in_row};
         const cuuint32_t box[3] = {64, 1, C};
@@ -499,11 +640,11 @@ cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cu
     const cuuint64_t sd[4] = {(cuuint64_t)p.dim, 2, (cuuint64_t)p.vdim, (cuuint64_t)c.n_chunks * p.heads};
     const cuuint64_t ss[3] = {(cuuint64_t)p.dim, (cuuint64_t)2 * p.dim, (cuuint64_t)2 * p.dim * p.vdim};
     const cuuint32_t sb[4] = {64, 1, VS, 1};
-    if (!rows_map(&mq, p.q_off, p.dim) || !rows_map(&mk, p.k_off, p.dim) || !rows_map(&mv, p.v_off, p.vdim) || !make_map_nd<4>(&ms, c.state, sd, ss, sb))
+    if (!rows_map(&mq, p.q_off, p.dim) || !rows_map(&mk, p.k_off, p.dim) || !rows_map(&mv, p.v_off, p.vdim) ||
+        !rows_map(&mg, p.g_off, p.vdim) || !make_map_nd<4>(&ms, c.state, sd, ss, sb))
         return cudaErrorInvalidValue;
     const bool rot = p.half > 0;
-    const int slices = (p.vdim + VS - 1) / VS;
-    const dim3 grid(c.n_chunks, p.heads, slices);
+    const dim3 grid(c.n_chunks, p.heads, (p.vdim + VS - 1) / VS), out_grid(c.n_chunks, p.heads, (p.vdim + 2 * VS - 1) / (2 * VS));
     cudaError_t e;
     auto state = [&](auto kernel) {
         e = raise_smem(kernel, state_smem(p.dim));
@@ -515,9 +656,10 @@ cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cu
     if (e != cudaSuccess) return e;
     auto out = [&](auto kernel) {
         e = raise_smem(kernel, out_smem(p.dim));
-        return e != cudaSuccess ? e : launch_pdl(kernel, grid, dim3(THREADS), out_smem(p.dim), st, mq, mk, mv, ms, p, c);
+        return e != cudaSuccess ? e : launch_pdl(kernel, out_grid, dim3(THREADS), out_smem(p.dim), st, mq, mk, mv, mg, ms, p, c);
     };
-    return rot ? out(chunk_out_kernel<true>) : out(chunk_out_kernel<false>);
+    e = rot ? out(chunk_out_kernel<true>) : out(chunk_out_kernel<false>);
+    return e != cudaSuccess || out_grid.z == 1 ? e : launch_head_gate(p, c.o, c.rows, st);
 }
 
 int bounds_status_linear_tc(bool reset);

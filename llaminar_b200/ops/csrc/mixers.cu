@@ -169,13 +169,14 @@ LLM_DEVICE void lstm_gates(float zi, float zf, float cap, float& i, float& f) {
 }
 
 template <class TI, class TO>
-__global__ void __launch_bounds__(LIN_THREADS) linear_rows_kernel(const LinearParams p, int slice) {
+__global__ void __launch_bounds__(LIN_THREADS, 3) linear_rows_kernel(const LinearParams p, int slice) {
     extern __shared__ __align__(16) float sm[];
     __shared__ float red[LIN_THREADS / 32];
-    __shared__ float s_sum[2];                         // this CTA's sum of squares, by token parity
+    __shared__ float s_sum[2][8];                      // the cluster's sums of squares, by token parity
     pdl_trigger();
-    pdl_wait();
     cg::cluster_group cluster = cg::this_cluster();
+    const bool spread = gridDim.x > 1;                 // the head's rows are spread over the cluster
+    if (spread) asm volatile("barrier.cluster.arrive.aligned;" ::: "memory");
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = p.dim;
     const int h = blockIdx.y, b = blockIdx.z, v0 = blockIdx.x * slice, nv = min(slice, p.vdim - v0);
     float *s_q = sm, *s_k = s_q + D, *s_n = s_k + D, *s_v = s_n + D, *s_o = s_v + slice;
@@ -186,11 +187,28 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_rows_kernel(const LinearPa
     float* S = p.S + (((size_t)slot * p.heads + h) * p.vdim + v0) * D;
     float* n_pool = lstm ? p.n + ((size_t)slot * p.heads + h) * D : nullptr;
     float* m_pool = lstm ? p.m + (size_t)slot * p.heads + h : nullptr;
+    // a warp's first rows of the state are on their way before the rows in front of them are complete: slots, positions and the
+    // sequences' rows come from the host, the state from an earlier step
+    const bool one_pass = D <= 128;
+    const int c_own = lane * 4;
+    float nxt[LIN_ROWS][4];
+    auto fetch = [&](int r) {
+#pragma unroll
+        for (int j = 0; j < LIN_ROWS; ++j) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) nxt[j][e] = 0.f;
+            if (!fresh && r + j < nv && c_own < D) load4(S + (size_t)(r + j) * D + c_own, nxt[j]);
+        }
+    };
+    if (one_pass) fetch(warp * LIN_ROWS);
+    pdl_wait();
+    if (spread) asm volatile("barrier.cluster.wait.aligned;" ::: "memory");       // every CTA of the cluster runs: its memory may be written
     float m = lstm && !fresh ? *m_pool : 0.f;
     if (lstm) for (int i = threadIdx.x; i < D; i += LIN_THREADS) s_n[i] = fresh ? 0.f : n_pool[i];
     const TI* in = static_cast<const TI*>(p.in);
     TO* out = static_cast<TO*>(p.out);
     for (int t = r0; t < r1; ++t) {
+        if (one_pass && t > r0) fetch(warp * LIN_ROWS);
         const TI* row = in + (size_t)t * p.in_row;
         const TI *q = row + p.q_off + h * D, *k = row + p.k_off + h * D, *v = row + p.v_off + h * p.vdim + v0;
         const float2* ang = p.half ? p.angles + (size_t)t * p.half : nullptr;
@@ -222,13 +240,21 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_rows_kernel(const LinearPa
         else __syncthreads();
         for (int r = warp * LIN_ROWS; r < nv; r += LIN_THREADS / 32 * LIN_ROWS) {
             float acc[LIN_ROWS] = {};
-            for (int c = lane * 4; c < D; c += 128) {
+            for (int c = c_own; c < D; c += 128) {
                 float s[LIN_ROWS][4], kk[4], qq[4];
+                if (one_pass) {
 #pragma unroll
-                for (int j = 0; j < LIN_ROWS; ++j) {
+                    for (int j = 0; j < LIN_ROWS; ++j)
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-                    if (!fresh && r + j < nv) load4(S + (size_t)(r + j) * D + c, s[j]);
+                        for (int e = 0; e < 4; ++e) s[j][e] = nxt[j][e];
+                    fetch(r + LIN_THREADS / 32 * LIN_ROWS);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < LIN_ROWS; ++j) {
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
+                        if (!fresh && r + j < nv) load4(S + (size_t)(r + j) * D + c, s[j]);
+                    }
                 }
                 load4(s_k + c, kk); load4(s_q + c, qq);
 #pragma unroll
@@ -253,12 +279,12 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_rows_kernel(const LinearPa
         float ss = 0.f;
         for (int i = threadIdx.x; i < nv; i += LIN_THREADS) { const float o = s_o[i] * den; ss += o * o; }
         ss = block_sum<LIN_THREADS>(ss, red);
-        if (gridDim.x > 1) {                           // the head's rows are spread over the cluster
+        if (spread) {
             const int par = (t - r0) & 1;
-            if (threadIdx.x == 0) s_sum[par] = ss;
+            if (threadIdx.x < gridDim.x) *cluster.map_shared_rank(&s_sum[par][blockIdx.x], threadIdx.x) = ss;
             cluster.sync();
             ss = 0.f;
-            for (int c = 0; c < (int)gridDim.x; ++c) ss += *cluster.map_shared_rank(&s_sum[par], c);
+            for (int c = 0; c < (int)gridDim.x; ++c) ss += s_sum[par][c];
         }
         const float inv = den / sqrtf(ss / (float)p.true_vdim + p.eps);
         for (int i = threadIdx.x; i < nv; i += LIN_THREADS) {
@@ -271,7 +297,7 @@ __global__ void __launch_bounds__(LIN_THREADS) linear_rows_kernel(const LinearPa
         fresh = false;
         __syncthreads();                               // shared arrays are filled anew for the next token
     }
-    if (gridDim.x > 1) cluster.sync();                 // every CTA has read n and m, and the others' sums
+    if (spread) cluster.sync();                        // every CTA has read n and m
     if (lstm && blockIdx.x == 0 && r0 < r1) {
         for (int i = threadIdx.x; i < D; i += LIN_THREADS) n_pool[i] = s_n[i];
         if (threadIdx.x == 0) *m_pool = m;
@@ -345,7 +371,7 @@ cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, b
     if (p.dim % 8 || p.vdim % 8 || p.heads > 65535 || n_seqs > 65535 || (f32 && !in_f32) || (!p.gates == !p.decay)) return cudaErrorInvalidValue;
     // slices of at least 32 state rows: enough CTAs to fill the machine, clusters of at most eight
     int slices = 1;
-    while (slices < 8 && p.vdim > 32 * slices && p.heads * n_seqs * slices < 4 * 148) slices *= 2;
+    while (slices < 8 && p.vdim > 32 * slices && p.heads * n_seqs * slices < 2 * 148) slices *= 2;
     while ((p.vdim + slices - 1) / slices > 1024 && slices < 8) slices *= 2;
     const int slice = ((p.vdim + slices - 1) / slices + 7) / 8 * 8;
     slices = (p.vdim + slice - 1) / slice;

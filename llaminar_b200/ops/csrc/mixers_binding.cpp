@@ -194,7 +194,6 @@ void linear_chunk(const Tensor& in, const std::vector<int64_t>& offs, const OptT
     want(status, torch::kInt32, "status");
     c.status = status.data_ptr<int>();
     check(llm::launch_linear_chunk(p, c, stream()), "linear_chunk");
-    check(llm::launch_head_gate(p, c.o, c.rows, stream()), "head_gate");
 }
 
 }  // namespace

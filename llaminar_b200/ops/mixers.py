@@ -101,7 +101,7 @@ def linear_chunk(rows, offs, gates, decay, angles, q_scale: float, k_scale: floa
     f = lambda *s: torch.empty(*s, dtype=torch.float32, device=rows.device)
     ext().linear_chunk(rows, list(offs), *g, decay, angles, q_scale, k_scale, cu, positions, slots, list(state), true_vdim, norm_w, silu, out, eps,
                        chunks, seqs, f(n, h, v, d), f(n, h, d), f(n, h, 4), raw, status)
-    _count(4)
+    _count(4 if v > 256 else 3)
 
 
 def bounds_status(reset: bool = True) -> int:
