@@ -39,13 +39,12 @@ def tokens(n: int, seed: int, vocab: int = 97) -> list[int]:
 
 
 def tolerance(dtype) -> float:
-    return 2e-4 if dtype == torch.float32 else 0.2
+    return 2e-4 if dtype == torch.float32 else 0.1
 
 
 def assert_close(got, want, dtype, what="", factor=1.0) -> None:
     """Root mean square over the vocabulary of the centred difference, relative to the spread of the logits: its largest value
-    over the positions, and over more than a few its mean (random weights make single positions that amplify rounding, where the
-    normaliser of an mLSTM nearly cancels)."""
+    over the positions, and over more than a few its mean."""
     d = got.double().cpu() - want.double()
     d = (d - d.mean(-1, keepdim=True)).pow(2).mean(-1).sqrt() / want.double().std()
     ok = torch.isfinite(d).all() and d.max() < 1.5 * factor * tolerance(dtype) and (len(d) < 8 or d.mean() < factor * tolerance(dtype) / 5)
@@ -124,7 +123,7 @@ def mixed_batches(name, device, dtype):
 
 
 ASKS, ASKED = 7, 11
-SHARP = 0.25                   # where one key decides: a quarter of the tolerance, and a mistake moves the logits by more than all of it
+SHARP = 0.5                    # where one key decides: half the tolerance, and a mistake moves the logits by more than all of it
 
 
 def sharp_attention(window: int, seed: int = 0):

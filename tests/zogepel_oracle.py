@@ -186,6 +186,8 @@ def random_model(seed=0, vocab=97, width=48, layers=None, eps=1e-5, mult=0.4, em
         if e["type"] == "mlstm":
             H, d, ve = m["heads"], m["dim"], m["vdim"]
             mat(p + "mix.q", H * d, width, 1.5), mat(p + "mix.k", H * d, width, 1.5), mat(p + "mix.v", H * ve, width)
+            # a query lies along its own key: with n.q near zero the normaliser turns the sign of a rounding error into the output's
+            t[p + "mix.q"] = (0.6 * t[p + "mix.q"].float() + 0.8 * t[p + "mix.k"].float()).to(torch.bfloat16)
             mat(p + "mix.g", H * ve, width), mat(p + "mix.o", width, H * ve), vec(p + "mix.norm", H * ve)
             mat(p + "mix.i", H, width), vec(p + "mix.i.b", H, -1.0, 1.0)
             mat(p + "mix.f", H, width), vec(p + "mix.f.b", H, 3.0, 1.5)
