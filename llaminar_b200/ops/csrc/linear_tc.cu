@@ -37,12 +37,15 @@ LLM_DEVICE void lstm_gates2(float zi, float zf, float cap, float& i, float& f) {
 
 // The chunk's a_j, G_t and A_t (see above), for the first 128 threads; every thread calls it.  Rows past `len`: a = -inf.
 struct Gates { float a, g, top; };
+LLM_DEVICE Gates retention_gates(float decay, int t) {
+    const float g = (float)(t + 1) * log2_decay(decay);
+    return {-g, g, -g};
+}
 LLM_DEVICE Gates chunk_gates(const LinearParams& p, int h, int r0, int len, float (&s_tmp)[2][4]) {
     const int t = threadIdx.x, lane = t & 31, warp = t >> 5;
     Gates r = {-INFINITY, 0.f, -INFINITY};
     if (!p.gates) {
-        const float l = log2_decay(p.decay[h]);
-        if (t < len) { r.g = (float)(t + 1) * l; r.a = -r.g; r.top = r.a; }
+        if (t < len) r = retention_gates(p.decay[h], t);
         return r;
     }
     float i = -INFINITY, f = 0.f;
@@ -80,42 +83,63 @@ template <bool ROT> LLM_DEVICE RotItems rot_items(int nu, int half) {
     const int pairs = ROT && half % 8 == 0 ? half / 8 : 0;
     return {pairs, nu - pairs};
 }
-// item `i` of row x (dim values, zero units behind): f(unit, values)
-template <bool ROT, class F> LLM_DEVICE void rot_item(const __nv_bfloat16* x, int i, const RotItems& it, int dim, const float2* ang, int half, F&& f) {
+// What an item of row x needs from memory; loads of several items are issued together, ahead of the arithmetic
+template <bool ROT> struct RotRaw { uint4 a, b; float4 cs[4]; };
+template <> struct RotRaw<false> { uint4 a; };
+template <bool ROT> LLM_DEVICE void rot_load(const __nv_bfloat16* x, int i, const RotItems& it, int dim, const float2* ang, int half, RotRaw<ROT>& r) {
+    if constexpr (ROT) {
+        if (i < it.pairs) {
+            r.a = *reinterpret_cast<const uint4*>(x + i * 8);
+            r.b = *reinterpret_cast<const uint4*>(x + half + i * 8);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) r.cs[j] = *reinterpret_cast<const float4*>(ang + i * 8 + 2 * j);     // two pairs; rows of 8 float2: 16-byte aligned
+            return;
+        }
+        if (it.pairs == 0) return;                                   // single values: read where they are turned
+    }
+    const int u = i + it.pairs;
+    r.a = u * 8 < dim ? *reinterpret_cast<const uint4*>(x + u * 8) : make_uint4(0, 0, 0, 0);
+}
+// its values (zeros behind dim): f(unit, values)
+template <bool ROT, class F> LLM_DEVICE void rot_apply(const __nv_bfloat16* x, int i, const RotItems& it, int dim, const float2* ang, int half, const RotRaw<ROT>& r, F&& f) {
     auto unpack = [](const uint4& w, float (&v)[8]) {
         const uint32_t a[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
         for (int j = 0; j < 4; ++j) { v[2 * j] = bf16_lo(a[j]); v[2 * j + 1] = bf16_hi(a[j]); }
     };
-    if (ROT && i < it.pairs) {
-        float u[8], w[8], a[8], b[8];
-        unpack(*reinterpret_cast<const uint4*>(x + i * 8), u);
-        unpack(*reinterpret_cast<const uint4*>(x + half + i * 8), w);
-        float4 cs[4];                                               // cos, sin of two pairs each; rows of 8 float2: 16-byte aligned
-#pragma unroll
-        for (int j = 0; j < 4; ++j) cs[j] = *reinterpret_cast<const float4*>(ang + i * 8 + 2 * j);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            a[2 * j] = u[2 * j] * cs[j].x - w[2 * j] * cs[j].y;
-            b[2 * j] = w[2 * j] * cs[j].x + u[2 * j] * cs[j].y;
-            a[2 * j + 1] = u[2 * j + 1] * cs[j].z - w[2 * j + 1] * cs[j].w;
-            b[2 * j + 1] = w[2 * j + 1] * cs[j].z + u[2 * j + 1] * cs[j].w;
-        }
-        f(i, a);
-        f(i + it.pairs, b);
-        return;
-    }
     const int u = i + it.pairs;
     float v[8] = {};
-    if (u * 8 < dim) {
-        if (ROT && it.pairs == 0) {
+    if constexpr (ROT) {
+        if (i < it.pairs) {
+            float x0[8], x1[8], y[8];
+            unpack(r.a, x0);
+            unpack(r.b, x1);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) v[j] = rotated(x, u * 8 + j, ang, half);
-        } else {
-            unpack(*reinterpret_cast<const uint4*>(x + u * 8), v);
+            for (int j = 0; j < 4; ++j) {
+                v[2 * j] = x0[2 * j] * r.cs[j].x - x1[2 * j] * r.cs[j].y;
+                y[2 * j] = x1[2 * j] * r.cs[j].x + x0[2 * j] * r.cs[j].y;
+                v[2 * j + 1] = x0[2 * j + 1] * r.cs[j].z - x1[2 * j + 1] * r.cs[j].w;
+                y[2 * j + 1] = x1[2 * j + 1] * r.cs[j].z + x0[2 * j + 1] * r.cs[j].w;
+            }
+            f(i, v);
+            f(u, y);
+            return;
+        }
+        if (it.pairs == 0) {
+            if (u * 8 < dim) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) v[j] = rotated(x, u * 8 + j, ang, half);
+            }
+            f(u, v);
+            return;
         }
     }
+    unpack(r.a, v);
     f(u, v);
+}
+LLM_DEVICE void tmem_st8(uint32_t taddr, const uint32_t* r) {
+    asm volatile("tcgen05.st.sync.aligned.32x32b.x8.b32 [%0], {%1,%2,%3,%4,%5,%6,%7,%8};"
+                 ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]) : "memory");
 }
 // two bf16 numbers whose sum is x to 16 bits of mantissa
 LLM_DEVICE void split_bf16(float x, float y, uint32_t& hi, uint32_t& lo) {
@@ -171,8 +195,23 @@ __global__ void __launch_bounds__(THREADS, 2) chunk_state_kernel(const __grid_co
         mbar_arrive_expect_tx(bar_v, 2 * ATOM);
         for (int a = 0; a < 2; ++a) tma_load_3d(sV + a * ATOM, &map_v, v0 + a * 64, h, r0, bar_v);
     }
+    const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(p.in) + (size_t)r0 * p.in_row + p.k_off + h * p.dim;
+    const float2* ang = ROT ? p.angles + (size_t)r0 * p.half : nullptr;
+    const RotItems items = rot_items<ROT>(nu, p.half);
+    const int groups = THREADS / items.count, item = tid % items.count, grp = tid / items.count;
+    constexpr int BATCH = ROT ? 2 : 4;
+    RotRaw<ROT> raw[BATCH];
+    auto load = [&](int j0) {
+#pragma unroll
+        for (int i = 0; i < BATCH; ++i) {
+            const int j = min(j0 + i * groups, len - 1);               // rows past the chunk: any valid one, their weight is zero
+            rot_load<ROT>(kp + (size_t)j * p.in_row, item, items, p.dim, ROT ? ang + (size_t)j * p.half : nullptr, p.half, raw[i]);
+        }
+    };
+    load(grp);
     {
         const Gates g = chunk_gates(p, h, r0, len, s_tmp);
+        if (p.gates && v0 == 0 && tid < C) c.gate[((size_t)blockIdx.x * p.heads + h) * C + tid] = make_float4(g.a, g.g, g.top, 0.f);
         if (tid < C) s_w[tid] = g.top;
         __syncthreads();
         const float top = s_w[len - 1];                               // A_L
@@ -181,29 +220,27 @@ __global__ void __launch_bounds__(THREADS, 2) chunk_state_kernel(const __grid_co
         if (tid == len - 1 && v0 == 0) *reinterpret_cast<float4*>(c.scal + ((size_t)blockIdx.x * p.heads + h) * 4) = make_float4(g.g, top, 0.f, 0.f);
         __syncthreads();
     }
-    const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(p.in) + (size_t)r0 * p.in_row + p.k_off + h * p.dim;
-    const RotItems items = rot_items<ROT>(nu, p.half);
-    const int groups = THREADS / items.count, item = tid % items.count, grp = tid / items.count;
     float sum[2][8] = {};                                             // of this thread's rows, by unit of the item
-    for (int j = grp; j < C && grp < groups; j += groups) {
-        const float w = s_w[j];
-        int part = 0;
-        auto put = [&](int u, float (&v)[8]) {
-            uint32_t hi[4], lo[4];
+    for (int j0 = grp; j0 < C && grp < groups; j0 += BATCH * groups) {
+        if (j0 != grp) load(j0);
 #pragma unroll
-            for (int e = 0; e < 8; ++e) { v[e] *= w; sum[part][e] += v[e]; }
+        for (int i = 0; i < BATCH; ++i) {
+            const int j = j0 + i * groups;
+            if (j >= C) break;
+            const float w = s_w[j];
+            int part = 0;
+            auto put = [&](int u, float (&v)[8]) {
+                uint32_t hi[4], lo[4];
 #pragma unroll
-            for (int e = 0; e < 4; ++e) split_bf16(v[2 * e], v[2 * e + 1], hi[e], lo[e]);
-            st_shared_v4(atom_addr(sH + (u >> 3) * ATOM, j, u & 7), make_uint4(hi[0], hi[1], hi[2], hi[3]));
-            st_shared_v4(atom_addr(sL + (u >> 3) * ATOM, j, u & 7), make_uint4(lo[0], lo[1], lo[2], lo[3]));
-            part = 1;
-        };
-        if (j < len) {
-            rot_item<ROT>(kp + (size_t)j * p.in_row, item, items, p.dim, ROT ? p.angles + (size_t)(r0 + j) * p.half : nullptr, p.half, put);
-        } else {
-            float v[8] = {};
-            put(item < items.pairs ? item : item + items.pairs, v);
-            if (item < items.pairs) { float z[8] = {}; put(item + items.pairs, z); }
+                for (int e = 0; e < 8; ++e) { v[e] *= w; sum[part][e] += v[e]; }
+#pragma unroll
+                for (int e = 0; e < 4; ++e) split_bf16(v[2 * e], v[2 * e + 1], hi[e], lo[e]);
+                st_shared_v4(atom_addr(sH + (u >> 3) * ATOM, j, u & 7), make_uint4(hi[0], hi[1], hi[2], hi[3]));
+                st_shared_v4(atom_addr(sL + (u >> 3) * ATOM, j, u & 7), make_uint4(lo[0], lo[1], lo[2], lo[3]));
+                part = 1;
+            };
+            const int r = min(j, len - 1);
+            rot_apply<ROT>(kp + (size_t)r * p.in_row, item, items, p.dim, ROT ? ang + (size_t)r * p.half : nullptr, p.half, raw[i], put);
         }
     }
     if (p.gates && v0 == 0 && grp < groups) {
@@ -347,7 +384,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
     __shared__ __align__(8) uint64_t s_bars[N_OBARS];
     __shared__ uint32_t s_tmem;
     __shared__ int s_abort[2];
-    __shared__ float s_tmp[2][4], s_top[C], s_keep[C], s_floor[C], s_x[2][C], s_y[2][C];
+    __shared__ float s_top[C], s_keep[C], s_floor[C], s_x[2][C], s_y[2][C];
     __shared__ __align__(16) float s_a[C], s_n[128];
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int4 ck = c.chunks[blockIdx.x];
@@ -388,21 +425,37 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
     if constexpr (ROT) {
         const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.in) + (size_t)r0 * p.in_row + h * p.dim;
         const RotItems items = rot_items<true>(ksteps * 2, p.half);
-        const int n = 2 * items.count, groups = THREADS / n, item = tid % n, which = item >= items.count;
+        const int n = 2 * items.count, groups = THREADS / n, which = tid % n >= items.count, item = tid % n - which * items.count;
         const uint32_t dst = which ? sK : sQ;
-        for (int j = tid / n; j < C && tid / n < groups; j += groups) {
-            auto put = [&](int u, float (&v)[8]) {
-                st_shared_v4(atom_addr(dst + (u >> 3) * ATOM, j, u & 7),
-                             make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7])));
-            };
+        const __nv_bfloat16* x = in + (which ? p.k_off : p.q_off);
+        constexpr int BATCH = 4;
+        for (int j0 = tid / n; j0 < C && tid / n < groups; j0 += BATCH * groups) {
+            RotRaw<true> raw[BATCH];
             // rows past the chunk repeat its last one (their results are not stored)
-            const int r = min(j, len - 1);
-            rot_item<true>(in + (size_t)r * p.in_row + (which ? p.k_off : p.q_off), item - which * items.count, items, p.dim, p.angles + (size_t)(r0 + r) * p.half, p.half, put);
+            auto at = [&](int i) { return min(j0 + i * groups, len - 1); };
+#pragma unroll
+            for (int i = 0; i < BATCH; ++i) rot_load<true>(x + (size_t)at(i) * p.in_row, item, items, p.dim, p.angles + (size_t)(r0 + at(i)) * p.half, p.half, raw[i]);
+#pragma unroll
+            for (int i = 0; i < BATCH; ++i) {
+                const int j = j0 + i * groups;
+                if (j >= C) break;
+                auto put = [&](int u, float (&v)[8]) {
+                    st_shared_v4(atom_addr(dst + (u >> 3) * ATOM, j, u & 7),
+                                 make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7])));
+                };
+                rot_apply<true>(x + (size_t)at(i) * p.in_row, item, items, p.dim, p.angles + (size_t)(r0 + at(i)) * p.half, p.half, raw[i], put);
+            }
         }
     }
     {
-        const Gates g = chunk_gates(p, h, r0, len, s_tmp);
         if (tid < C) {
+            Gates g = {-INFINITY, 0.f, -INFINITY};
+            if (lstm) {
+                const float4 x = __ldcg(c.gate + ((size_t)blockIdx.x * p.heads + h) * C + tid);
+                g = {x.x, x.y, x.z};
+            } else if (tid < len) {
+                g = retention_gates(p.decay[h], tid);
+            }
             const float m = lstm ? __ldcg(c.scal + ((size_t)blockIdx.x * p.heads + h) * 4 + 2) : 0.f;
             const float top = lstm ? fmaxf(m, g.top) : g.top;
             s_a[tid] = g.a;
@@ -469,18 +522,16 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
         __syncwarp();
         const float top = s_top[row], scale = p.q_scale * p.k_scale;
         float sum = 0.f;
-        uint32_t hi[32], lo[32];
-        if (half * 64 > (warp & 3) * 32 + 31) {                          // nothing here for this warp's rows
+        const bool none = half * 64 > (warp & 3) * 32 + 31;              // nothing here for this warp's rows
+        // (rolled loops here and below: every instruction of a CTA is fetched once, and straight-line code of this size waited for that)
+#pragma unroll 1
+        for (int q = 0; q < 4; ++q) {
+            uint32_t r[16], hl[16];                                      // hl: hi words, then lo words
+            if (!none) {
+                tmem_ld_n<16>(t_lane + T_S + half * 64 + q * 16, r);
 #pragma unroll
-            for (int i = 0; i < 32; ++i) hi[i] = lo[i] = 0u;
-        } else {
-#pragma unroll
-            for (int q = 0; q < 2; ++q) {
-                uint32_t r[32];
-                tmem_ld_n<32>(t_lane + T_S + half * 64 + q * 32, r);
-#pragma unroll
-                for (int i = 0; i < 32; i += 4) {
-                    const int j = half * 64 + q * 32 + i;
+                for (int i = 0; i < 16; i += 4) {
+                    const int j = half * 64 + q * 16 + i;
                     const float4 a = *reinterpret_cast<const float4*>(s_a + j);
                     const float e[4] = {a.x, a.y, a.z, a.w};
                     float w[4];
@@ -489,13 +540,16 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
                         w[x] = j + x <= row ? __uint_as_float(r[i + x]) * scale * ex2(e[x] - top) : 0.f;
                         sum += w[x];
                     }
-                    split_bf16(w[0], w[1], hi[q * 16 + i / 2], lo[q * 16 + i / 2]);
-                    split_bf16(w[2], w[3], hi[q * 16 + i / 2 + 1], lo[q * 16 + i / 2 + 1]);
+                    split_bf16(w[0], w[1], hl[i / 2], hl[8 + i / 2]);
+                    split_bf16(w[2], w[3], hl[i / 2 + 1], hl[8 + i / 2 + 1]);
                 }
+            } else {
+#pragma unroll
+                for (int i = 0; i < 16; ++i) hl[i] = 0u;
             }
+            tmem_st8(t_lane + T_P + half * 32 + q * 8, hl);
+            tmem_st8(t_lane + T_P + 64 + half * 32 + q * 8, hl + 8);
         }
-        tmem_st32(t_lane + T_P + half * 32, hi);
-        tmem_st32(t_lane + T_P + 64 + half * 32, lo);
         if (lstm) {
             float dot = 0.f;
             for (int u = half; u * 8 < p.dim; u += 2) {
@@ -518,92 +572,95 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
             ok = ok && mbar_wait_warp(bar(B_IN), 0, abort_flag);         // the state of slice 0 is done with
             if (ok && elect_one()) load_state(1);
             __syncwarp();
-            issue_in(1, T_S);
         }
     }
     const float keep = s_keep[row];
     const float inv = lstm ? 1.f / (fmaxf(fabsf(s_x[0][row] + s_x[1][row]), s_floor[row]) + NORM_FLOOR) : 1.f;
-    uint32_t o[2][32];
     float ss = 0.f;
+    // both parts of o together; the sums stay in tensor memory (columns T_I of slice 0, T_O of slice 1) until the norm is known
+#pragma unroll 1
+    for (int s = 0; s < slices; ++s) {
+        ok = ok && mbar_wait_warp(bar(s ? B_IN1 : B_IN), 0, abort_flag) && mbar_wait_warp(bar(B_O), s, abort_flag);
+        if (ok) {
+            tc_fence_after();
+            if (fused && s == 0 && slices == 2 && tid == 0) load_rows(sV, &map_g, 1, B_G1);       // the values of slice 0 are done with
+            __syncwarp();
+            const int w = width(s);
+#pragma unroll 1
+            for (int c0 = half * 64; c0 < min(w, half * 64 + 64); c0 += 16) {        // the same for all threads of the warp
+                uint32_t a[16], b[16];
+                tmem_ld_n<16>(t_lane + T_O + c0, a);
+                tmem_ld_n<16>(t_lane + (s ? T_S : T_I) + c0, b);
 #pragma unroll
-    for (int s = 0; s < 2; ++s) {
-        if (s < slices) {
-            ok = ok && mbar_wait_warp(bar(s ? B_IN1 : B_IN), 0, abort_flag) && mbar_wait_warp(bar(B_O), s, abort_flag);
-            if (ok) {
-                tc_fence_after();
-                if (fused && s == 0 && slices == 2 && tid == 0) load_rows(sV, &map_g, 1, B_G1);       // the values of slice 0 are done with
-                __syncwarp();
-                const int w = width(s);
-#pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    const int c0 = half * 64 + q * 16;
-                    if (c0 < w) {                                        // the same for all threads of the warp
-                        uint32_t a[16], b[16];
-                        tmem_ld_n<16>(t_lane + T_O + c0, a);
-                        tmem_ld_n<16>(t_lane + (s ? T_S : T_I) + c0, b);
-#pragma unroll
-                        for (int i = 0; i < 8; ++i) {
-                            const float x = (__uint_as_float(a[2 * i]) + keep * __uint_as_float(b[2 * i])) * inv;
-                            const float y = (__uint_as_float(a[2 * i + 1]) + keep * __uint_as_float(b[2 * i + 1])) * inv;
-                            ss += x * x + y * y;
-                            o[s][q * 8 + i] = pack_bf16(x, y);
-                        }
-                    }
+                for (int i = 0; i < 16; ++i) {
+                    const float x = (__uint_as_float(a[i]) + keep * __uint_as_float(b[i])) * inv;
+                    ss += x * x;
+                    a[i] = __float_as_uint(x);
                 }
-                tc_fence_before();
+                tmem_st_n<16>(t_lane + (s ? T_O : T_I) + c0, a);
             }
-            if (s == 0 && slices == 2) {
-                __syncthreads();                                         // slice 0 has been read out of tensor memory
-                if (warp == 0) issue_o(1);
+            tmem_wait_st();
+            tc_fence_before();
+        }
+        if (s == 0 && slices == 2) {
+            __syncthreads();                                             // slice 0 has been read out of T_O
+            if (warp == 0) {
+                issue_in(1, T_S);
+                issue_o(1);
             }
         }
     }
     s_y[half][row] = ss;
     __syncthreads();
     const float rms = fused ? 1.f / sqrtf((s_y[0][row] + s_y[1][row]) / (float)p.true_vdim + p.eps) : 1.f;
+#pragma unroll 1
+    for (int s = 0; s < slices; ++s) {
+        // gated values into the gate's own place (fused), or o as it is; then whole rows to memory
+        const uint32_t tile = s ? sV : sG;
+        if (fused) ok = ok && mbar_wait_warp(bar(s ? B_G1 : B_G), 0, abort_flag);
+        const int w = width(s);
+        if (ok) {
+#pragma unroll 1
+            for (int c0 = half * 64; c0 < min(w, half * 64 + 64); c0 += 16) {
+                uint32_t o[16];
+                tmem_ld_n<16>(t_lane + (s ? T_O : T_I) + c0, o);
 #pragma unroll
-    for (int s = 0; s < 2; ++s) {
-        if (s < slices) {
-            // gated values into the gate's own place (fused), or o as it is; then whole rows to memory
-            const uint32_t tile = s ? sV : sG;
-            if (fused) ok = ok && mbar_wait_warp(bar(s ? B_G1 : B_G), 0, abort_flag);
-            const int w = width(s);
-            if (ok) {
+                for (int k = 0; k < 2; ++k) {
+                    const uint32_t at = atom_addr(tile + half * ATOM, row, (c0 & 63) / 8 + k);
+                    float v[8];
 #pragma unroll
-                for (int q = 0; q < 8; ++q) {
-                    const int c0 = half * 64 + q * 8;
-                    if (c0 < w) {
-                        const uint32_t at = atom_addr(tile + half * ATOM, row, q);
-                        uint32_t r[4] = {o[s][4 * q], o[s][4 * q + 1], o[s][4 * q + 2], o[s][4 * q + 3]};
-                        if (fused) {
-                            uint32_t g[4];
-                            asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(g[0]), "=r"(g[1]), "=r"(g[2]), "=r"(g[3]) : "r"(at));
-                            const int col = v0 + s * VS + c0;
-#pragma unroll
-                            for (int i = 0; i < 4; ++i) {
-                                const float za = bf16_lo(g[i]), zb = bf16_hi(g[i]);
-                                float x = bf16_lo(r[i]) * rms * (p.silu ? za : 1.f) * __fdividef(1.f, 1.f + __expf(-za));
-                                float y = bf16_hi(r[i]) * rms * (p.silu ? zb : 1.f) * __fdividef(1.f, 1.f + __expf(-zb));
-                                if (p.norm_w && col < p.vdim) { x *= p.norm_w[h * p.vdim + col + 2 * i]; y *= p.norm_w[h * p.vdim + col + 2 * i + 1]; }
-                                r[i] = pack_bf16(x, y);
-                            }
+                    for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(o[k * 8 + i]);
+                    if (fused) {
+                        uint32_t g[4];
+                        asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(g[0]), "=r"(g[1]), "=r"(g[2]), "=r"(g[3]) : "r"(at));
+                        const int col = v0 + s * VS + c0 + k * 8;
+                        float4 n0 = make_float4(1.f, 1.f, 1.f, 1.f), n1 = n0;
+                        if (p.norm_w && col < p.vdim) {
+                            n0 = *reinterpret_cast<const float4*>(p.norm_w + h * p.vdim + col);
+                            n1 = *reinterpret_cast<const float4*>(p.norm_w + h * p.vdim + col + 4);
                         }
-                        st_shared_v4(at, make_uint4(r[0], r[1], r[2], r[3]));
+                        const float n[8] = {n0.x, n0.y, n0.z, n0.w, n1.x, n1.y, n1.z, n1.w};
+#pragma unroll
+                        for (int i = 0; i < 8; ++i) {
+                            const float z = i & 1 ? bf16_hi(g[i >> 1]) : bf16_lo(g[i >> 1]);
+                            v[i] *= rms * n[i] * (p.silu ? z : 1.f) * __fdividef(1.f, 1.f + __expf(-z));
+                        }
                     }
+                    st_shared_v4(at, make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7])));
                 }
             }
-            __syncthreads();
-            if (ok) {
-                __nv_bfloat16* dst = (fused ? static_cast<__nv_bfloat16*>(p.out) + (size_t)r0 * p.out_row : c.o + (size_t)r0 * p.heads * p.vdim) + (size_t)h * p.vdim + v0 + s * VS;
-                const size_t stride = fused ? p.out_row : (size_t)p.heads * p.vdim;
-                const int u = lane & 15;
-                for (int r = warp * 2 + (lane >> 4); r < len; r += THREADS / 16)
-                    if (v0 + s * VS + u * 8 < p.vdim) {
-                        uint4 x;
-                        asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(x.x), "=r"(x.y), "=r"(x.z), "=r"(x.w) : "r"(atom_addr(tile + (u >> 3) * ATOM, r, u & 7)));
-                        *reinterpret_cast<uint4*>(dst + (size_t)r * stride + u * 8) = x;
-                    }
-            }
+        }
+        __syncthreads();
+        if (ok) {
+            __nv_bfloat16* dst = (fused ? static_cast<__nv_bfloat16*>(p.out) + (size_t)r0 * p.out_row : c.o + (size_t)r0 * p.heads * p.vdim) + (size_t)h * p.vdim + v0 + s * VS;
+            const size_t stride = fused ? p.out_row : (size_t)p.heads * p.vdim;
+            const int u = lane & 15;
+            for (int r = warp * 2 + (lane >> 4); r < len; r += THREADS / 16)
+                if (v0 + s * VS + u * 8 < p.vdim) {
+                    uint4 x;
+                    asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(x.x), "=r"(x.y), "=r"(x.z), "=r"(x.w) : "r"(atom_addr(tile + (u >> 3) * ATOM, r, u & 7)));
+                    *reinterpret_cast<uint4*>(dst + (size_t)r * stride + u * 8) = x;
+                }
         }
     }
     // the stabiliser behind the sequence's last chunk

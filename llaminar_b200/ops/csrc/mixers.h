@@ -57,13 +57,14 @@ struct LinearParams {
 cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, bool f32, cudaStream_t st);
 // Chunk-parallel form for prompts: bf16 rows, heads of at most 128 key values (linear_tc.cu).  Sequences are cut into chunks of
 // LINEAR_CHUNK rows; `chunks` holds (first row, rows, sequence, 0) of each, `seqs` (first chunk, chunks, 0, 0).  Scratch: state
-// [chunks][heads][vdim][dim] float, vec [chunks][heads][dim] float, scal [chunks][heads][4] float.  o
+// [chunks][heads][vdim][dim] float, vec [chunks][heads][dim] float, scal [chunks][heads][4] float, gate [chunks][heads][LINEAR_CHUNK].  o
 // [T, heads * vdim] bf16: the heads' outputs before norm and gate, where a head of more than 256 values is spread over CTAs.
 constexpr int LINEAR_CHUNK = 128;
 struct LinearChunks {
     const int4 *chunks, *seqs;
     int n_chunks, n_seqs, rows;
     float *state, *vec, *scal;
+    float4* gate;                                                // mLSTM: what the gates of every row come to, chunk_state to chunk_out
     __nv_bfloat16* o;
     int* status;                                                 // receives STATUS_TIMEOUT if a wait gave up
 };

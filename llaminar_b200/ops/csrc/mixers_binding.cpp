@@ -170,7 +170,7 @@ void linear_rows(const Tensor& in, const std::vector<int64_t>& offs, const OptTe
 void linear_chunk(const Tensor& in, const std::vector<int64_t>& offs, const OptTensor& gates, const OptTensor& bias_i, const OptTensor& bias_f, double cap,
                   const OptTensor& decay, const OptTensor& angles, double q_scale, double k_scale, const Tensor& cu, const Tensor& positions,
                   const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps,
-                  const Tensor& chunks, const Tensor& seqs, const Tensor& scratch, const Tensor& vec, const Tensor& scal, const Tensor& o, const Tensor& status) {
+                  const Tensor& chunks, const Tensor& seqs, const Tensor& scratch, const Tensor& vec, const Tensor& scal, const OptTensor& gate, const Tensor& o, const Tensor& status) {
     const llm::LinearParams p = linear_params(in, offs, gates, bias_i, bias_f, cap, decay, angles, q_scale, k_scale, cu, positions, slots, state, true_vdim, norm_w, silu, out, eps);
     bf16(in, "in"); bf16(out, "out");
     llm::LinearChunks c = {};
@@ -189,6 +189,7 @@ void linear_chunk(const Tensor& in, const std::vector<int64_t>& offs, const OptT
         return t.data_ptr<float>();
     };
     c.state = scratch_ptr(scratch, units * p.vdim * p.dim, "scratch"); c.vec = scratch_ptr(vec, units * p.dim, "vec"); c.scal = scratch_ptr(scal, units * 4, "scal");
+    if (p.gates) c.gate = reinterpret_cast<float4*>(scratch_ptr(gate.value(), units * llm::LINEAR_CHUNK * 4, "gate"));
     TORCH_CHECK(o.is_contiguous() && o.numel() >= (int64_t)c.rows * p.heads * p.vdim, "o too small");
     c.o = const_cast<__nv_bfloat16*>(bf16(o, "o"));
     want(status, torch::kInt32, "status");

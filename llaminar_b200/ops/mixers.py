@@ -100,7 +100,7 @@ def linear_chunk(rows, offs, gates, decay, angles, q_scale: float, k_scale: floa
     n = chunks.shape[0]
     f = lambda *s: torch.empty(*s, dtype=torch.float32, device=rows.device)
     ext().linear_chunk(rows, list(offs), *g, decay, angles, q_scale, k_scale, cu, positions, slots, list(state), true_vdim, norm_w, silu, out, eps,
-                       chunks, seqs, f(n, h, v, d), f(n, h, d), f(n, h, 4), raw, status)
+                       chunks, seqs, f(n, h, v, d), f(n, h, d), f(n, h, 4), f(n, h, ext().LINEAR_CHUNK, 4) if gates else None, raw, status)
     _count(4 if v > 256 else 3)
 
 
