@@ -133,7 +133,8 @@ def norms(cfg: ModelConfig, n: int) -> list[dict]:
 def products(cfg: ModelConfig, rows_list=(1, 4, 8, 32)) -> list[dict]:
     """Matrix products of a decode step: bf16 weights here, 8-bit blocks on the quantised kernels for comparison."""
     from . import ops as base
-    from .engine.latent import DenseLinear, PaddedSizes
+    from .engine.dense import DenseLinear
+    from .engine.latent import PaddedSizes
     from .gguf import GGMLType, quantize
     from .ops import latent as ops
     d, ff, m, dev = cfg.d_model, cfg.ff_width(0), cfg.mixers[0], "cuda"

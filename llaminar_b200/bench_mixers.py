@@ -104,7 +104,7 @@ def gdn_prefill(n: int, heads: int, d: int) -> dict:
 
 def attention(cfg: ModelConfig, gqa: ModelConfig) -> list[dict]:
     from . import ops as base
-    from .ops import mixers as ops
+    from .ops import grouped as ops
     m = next(x.left for x in cfg.mixers if isinstance(x, ParallelMixers))
     H, G, D, sc = m.heads, m.kv_heads, m.dim, base.scratch_for(torch.device("cuda", torch.cuda.current_device()))
     sink, out = torch.zeros(H, **F32), []

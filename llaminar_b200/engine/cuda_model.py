@@ -296,7 +296,7 @@ class CudaModel:
         self.qkv_dim = self.q_dim + 2 * self.kv_dim
         self.ff_local = pl.ff_stop - pl.ff_start
         self.stack = None
-        self.kv_row_widths = None
+        self.kv_layer_shapes = None
         if c.has_mixers:
             self._init_stack(weights, max_tokens)
             return
@@ -345,17 +345,17 @@ class CudaModel:
     def _init_stack(self, weights: ModelWeights, max_tokens: int) -> None:
         """Models whose layers have mixers and sizes of their own: unquantised matrices, cache and state layouts per layer."""
         from .dense import DenseLinear
-        from .latent import LatentStack
         from .mixers import MixerStack
+        from .stack import AttentionStack
         c = self.cfg
         if self.layer_ids != list(range(c.n_layers)):
             raise ValueError(f"a {c.arch} model cannot be cut into pipeline stages")
-        st = self.stack = (LatentStack if c.is_latent else MixerStack)(self, weights)
+        st = self.stack = (AttentionStack if c.is_attention_stack else MixerStack)(self, weights)
         self.layers = [st.build_layer(CudaLayer(), weights, i) for i in self.layer_ids]
-        self.out_norm = _f32(weights["output_norm.weight"], self.device)
-        self.head = DenseLinear(st._mat(weights, "output.weight"))
+        self.out_norm = _f32(weights["output_norm.weight"], self.device) * c.logit_scale
+        self.head = DenseLinear(st.head_matrix(weights))
         self.vocab_local = c.vocab_size
-        self.kv_row_widths, self.kv_head_shapes, self.state_shapes = st.kv_row_widths, st.kv_head_shapes, st.state_shapes
+        self.kv_layer_shapes, self.state_shapes = st.kv_layer_shapes, st.state_shapes
         self.n_kv_layers = self.mtp_kv_base = st.n_kv_layers
         self.mtp_layers, self.hybrid_dims, self.graph_safe, self.torch_attention = [], None, True, False
         self._kv_ids, self._gdn_ids = list(range(self.n_kv_layers)), []

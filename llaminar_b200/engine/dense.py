@@ -1,4 +1,4 @@
-"""Linear layers with unquantised matrices, shared by the models with per-layer mixers (engine/latent.py, engine/mixers.py)."""
+"""Linear layers with unquantised matrices, shared by the models with per-layer mixers (engine/stack.py, engine/mixers.py)."""
 from __future__ import annotations
 
 import torch
@@ -20,9 +20,9 @@ def pad_to(x: torch.Tensor, *shape: int) -> torch.Tensor:
 class DenseLinear:
     """y = x W^T with W as it is stored (bf16, or float in 32-bit mode)."""
 
-    def __init__(self, weight: torch.Tensor, gelu_pair: bool = False):
+    def __init__(self, weight: torch.Tensor):
         self.w = weight.contiguous()
-        self.n_out, self.k, self.gelu_pair = weight.shape[0], weight.shape[1], gelu_pair
+        self.n_out, self.k = weight.shape[0], weight.shape[1]
 
     def nbytes(self) -> int:
         return self.w.numel() * self.w.element_size()

@@ -104,8 +104,7 @@ class LLMEngine:
                 raise ValueError("the 8-bit KV cache is not available for hybrid (linear-attention) models: their gated "
                                  "attention blocks append to a bf16 cache")
             hybrid = HybridState(n_slots=max(1, max_batch), device=self.device, **hd)
-        row_widths = getattr(self.model, "kv_row_widths", None)      # latent attention: one shared row per token and layer
-        head_shapes = getattr(self.model, "kv_head_shapes", None)    # layers with keys and values of their own sizes
+        kv_shapes = getattr(self.model, "kv_layer_shapes", None)     # cache layers with sizes of their own
         if c.has_mixers and (kv_dtype == KV_Q8 or mtp is not None):
             raise ValueError(f"{c.arch} models have no 8-bit KV cache and no multi-token-prediction head")
         state_shapes = getattr(self.model, "state_shapes", None)
@@ -116,7 +115,7 @@ class LLMEngine:
             need = max_batch * self.max_pages_per_seq + 64
             if self.is_cuda:
                 free, _ = torch.cuda.mem_get_info(self.device)
-                per_page = max(1, PagedKVCache.bytes_per_page(n_kv_layers, self.model.n_kv_local, c.head_dim, 17 / 16 if kv_dtype == KV_Q8 else dtype.itemsize, row_widths, head_shapes))
+                per_page = max(1, PagedKVCache.bytes_per_page(n_kv_layers, self.model.n_kv_local, c.head_dim, 17 / 16 if kv_dtype == KV_Q8 else dtype.itemsize, kv_shapes))
                 kv_pages = int(min(need * 2, max(need // 4, int(free * kv_memory_fraction) // per_page)))
             else:
                 kv_pages = need
@@ -126,8 +125,7 @@ class LLMEngine:
         self._agree_group = agree_group if agree_group is not None else (tp.group if tp is not None and tp.size > 1 else None)
         kv_pages = self._agree_kv_pages(kv_pages, self._agree_group)
         self.kv = PagedKVCache(n_kv_layers, self.model.n_kv_local, c.head_dim, kv_pages, self.device,
-                               dtype=(KV_Q8 if kv_dtype == KV_Q8 else dtype) if self.is_cuda else (kv_dtype or torch.float32), row_widths=row_widths,
-                               head_shapes=head_shapes)
+                               dtype=(KV_Q8 if kv_dtype == KV_Q8 else dtype) if self.is_cuda else (kv_dtype or torch.float32), layer_shapes=kv_shapes)
         self.kv.hybrid = hybrid
         self.use_graphs = use_graphs and self.is_cuda and not debug_env().no_cuda_graphs and getattr(self.model, "graph_safe", True)
         self.perf = perf_stats()

@@ -146,24 +146,19 @@ Q8 = "q8_0"          # 8-bit cache: int8 values with one fp16 scale per 32 (CUDA
 
 
 class PagedKVCache:
-    """Pages of 64 tokens per cache layer.  Per-head layout: [2 (K, V), heads, 64, head size], with ``head_shapes`` the heads and
-    head size of every layer.  With ``row_widths`` (one per layer) a layer holds one row of that many values per token instead,
-    shared by all heads (latent attention)."""
+    """Pages of 64 tokens per cache layer.  Per-head layout: [2 (K, V), heads, 64, head size].  With ``layer_shapes`` every layer has
+    its own: (heads, head size), or (width,) for one row of that many values per token, shared by all heads (latent attention)."""
 
     def __init__(self, n_layers: int, n_kv_heads: int, head_dim: int, n_pages: int, device, dtype=torch.bfloat16,
-                 row_widths: list[int] | None = None, head_shapes: list[tuple[int, int]] | None = None):
+                 layer_shapes: list[tuple[int, ...]] | None = None):
         self.n_layers, self.n_kv_heads, self.head_dim, self.n_pages = n_layers, n_kv_heads, head_dim, n_pages
         self.device = torch.device(device)
         self.q8 = dtype == Q8
-        self.row_widths, self.head_shapes = row_widths, head_shapes
-        if head_shapes is not None:
-            if self.q8 or len(head_shapes) != n_layers:
-                raise ValueError("a cache of unequal layers takes one (heads, head size) per layer and float values")
-            self.layers = [torch.zeros(n_pages, 2, h, PAGE_SIZE, d, dtype=dtype, device=device) for h, d in head_shapes]
-        elif row_widths is not None:
-            if self.q8 or len(row_widths) != n_layers:
-                raise ValueError("a latent cache takes one row width per layer and float rows")
-            self.layers = [torch.zeros(n_pages, PAGE_SIZE, w, dtype=dtype, device=device) for w in row_widths]
+        self.layer_shapes = layer_shapes
+        if layer_shapes is not None:
+            if self.q8 or len(layer_shapes) != n_layers:
+                raise ValueError("a cache of unequal layers takes one shape per layer and float values")
+            self.layers = [torch.zeros(n_pages, *((PAGE_SIZE, *s) if len(s) == 1 else (2, s[0], PAGE_SIZE, s[1])), dtype=dtype, device=device) for s in layer_shapes]
         elif self.q8:
             # a page is [2][n_kv_heads][64][head_dim] int8 followed by [2][n_kv_heads][64][head_dim / 32] fp16 block scales;
             # zero bytes decode to zeros, so untouched positions stay finite
@@ -184,12 +179,9 @@ class PagedKVCache:
         return sum(l[0].numel() * l.element_size() for l in self.layers)
 
     @staticmethod
-    def bytes_per_page(n_layers: int, n_kv_heads: int, head_dim: int, itemsize: float = 2, row_widths: list[int] | None = None,
-                       head_shapes: list[tuple[int, int]] | None = None) -> int:
-        if head_shapes is not None:
-            return int(sum(2 * h * d for h, d in head_shapes) * PAGE_SIZE * itemsize)
-        if row_widths is not None:
-            return int(sum(row_widths) * PAGE_SIZE * itemsize)
+    def bytes_per_page(n_layers: int, n_kv_heads: int, head_dim: int, itemsize: float = 2, layer_shapes: list[tuple[int, ...]] | None = None) -> int:
+        if layer_shapes is not None:
+            return int(sum(s[0] if len(s) == 1 else 2 * s[0] * s[1] for s in layer_shapes) * PAGE_SIZE * itemsize)
         return int(n_layers * 2 * n_kv_heads * PAGE_SIZE * head_dim * itemsize)
 
     def ensure_capacity(self, seq: SequenceKV, n_tokens: int) -> None:
@@ -219,10 +211,10 @@ class PagedKVCache:
 
     # -- page payload movement for the RAM / disk prefix tiers -------------------------------
     def copy_page(self, page: int) -> torch.Tensor:
-        """One page over all layers, on the device: [layers, ...page], or one flat run where the layers' rows differ."""
+        """One page over all layers, on the device: [layers, ...page], or one flat run where the layers differ."""
         if not self.layers:                      # a pipeline stage of linear-attention blocks only: pages carry no bytes here
             return torch.empty(0)
-        if self.row_widths is not None or self.head_shapes is not None:
+        if self.layer_shapes is not None:
             return torch.cat([l[page].reshape(-1) for l in self.layers])
         return torch.stack([l[page] for l in self.layers])
 
@@ -230,7 +222,7 @@ class PagedKVCache:
         return self.copy_page(page).to("cpu", non_blocking=False)
 
     def import_page(self, page: int, payload: torch.Tensor) -> None:
-        if self.row_widths is not None or self.head_shapes is not None:
+        if self.layer_shapes is not None:
             payload = [x.view(l[page].shape) for x, l in zip(payload.split([l[page].numel() for l in self.layers]), self.layers)]
         for i, l in enumerate(self.layers):
             l[page].copy_(payload[i].to(self.device, non_blocking=True))

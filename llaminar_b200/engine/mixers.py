@@ -62,10 +62,9 @@ class MixerStack:
             torch.backends.cuda.matmul.allow_bf16_reduced_precision_reduction = False
         self.embed = self._mat(weights, "token_embd.weight")
         self.side = self._mat(weights, "side_embd.weight") if c.side_dim else None
-        self.kv_row_widths = None
-        self.kv_head_shapes = mixer_kv_shapes(c, self.head_pad)
+        self.kv_layer_shapes = mixer_kv_shapes(c, self.head_pad)
         self.state_shapes = mixer_state_shapes(c, 8)
-        self.n_kv_layers = len(self.kv_head_shapes)
+        self.n_kv_layers = len(self.kv_layer_shapes)
         from .. import ops
         self.scratch = ops.scratch_for(self.device)
         self.status = self.scratch.status                               # word that a kernel sets when a bounded wait runs out
@@ -75,13 +74,16 @@ class MixerStack:
 
     def head_pad(self, dim: int) -> int:
         """Head size of the attention kernels for heads of ``dim`` values."""
-        from ..ops import mixers as ops
+        from ..ops import grouped as ops
         if self.f32 or dim > max(ops.HEAD_SIZES):
             return pad8(dim)
         return min(s for s in ops.HEAD_SIZES if s >= dim)
 
     def _mat(self, w, name: str) -> torch.Tensor:
         return w[name].to_float().to(self.device).to(self.dtype)
+
+    def head_matrix(self, w) -> torch.Tensor:
+        return self._mat(w, "output.weight")
 
     def _vec(self, w, name: str) -> torch.Tensor:
         return w[name].to_float().to(device=self.device, dtype=torch.float32).contiguous()
@@ -247,7 +249,7 @@ class MixerStack:
             ops.resid_norm(h, y, L.side_norm, copy0=x, eps=eps)
 
     def _attention(self, P, rows: torch.Tensor, fb, plan: MixerPlan, kv) -> torch.Tensor:
-        from ..ops import mixers as ops
+        from ..ops import grouped as ops
         m, T = P.m, rows.shape[0]
         kvl, H, D = kv.layers[P.kv], m.heads, P.dim
         q, o = self.ws("q", T, H * D).view(T, H, D), self.ws("oa", T, H * D)
@@ -261,7 +263,7 @@ class MixerStack:
             tc = self.attn_tc and ops.prefill_tc(D, fb.max_q_len)
             ops.attn_prefill(q, kvl, o, fb.block_table, fb.cu_q, fb.ctx_lens, m.scale, fb.max_q_len, m.window, P.sink, gate, self.status if tc else None)
         else:
-            ops.window_plain(q, kvl, o, fb.positions, fb.seq_ids, fb.block_table, m.window, m.scale, P.sink, gate)
+            ops.attn_plain(q, kvl, o, fb.positions, fb.seq_ids, fb.block_table, m.window, m.scale, P.sink, gate)
         return o
 
     def _linear(self, P, rows: torch.Tensor, gates, fb, plan: MixerPlan, kv) -> torch.Tensor:

@@ -91,7 +91,7 @@ class PrefixCache:
         self.engine = engine
         kv = engine.kv
         el = kv.layers[0].element_size() if kv.layers else 2
-        self.page_bytes = kv.page_bytes if kv.row_widths is not None or kv.head_shapes is not None else kv.n_layers * 2 * kv.n_kv_heads * PAGE_SIZE * kv.head_dim * el
+        self.page_bytes = kv.page_bytes if kv.layer_shapes is not None else kv.n_layers * 2 * kv.n_kv_heads * PAGE_SIZE * kv.head_dim * el
         if kv.hybrid is not None:
             # state snapshots live on the device; between 1 and 64 of them, within the device budget of the cache
             self.max_states = max(1, min(64, self.cfg.vram_budget_mb * (1 << 20) // max(kv.hybrid.slot_bytes, 1)))
@@ -102,10 +102,8 @@ class PrefixCache:
         import torch.distributed as dist
         rank, world = (dist.get_rank(), dist.get_world_size()) if dist.is_available() and dist.is_initialized() else (0, 1)
         shard = f"{rank}/{world}/{kv.n_layers}/{kv.n_kv_heads}/{kv.head_dim}/{kv.layers[0].dtype if kv.layers else None}"
-        if kv.row_widths is not None:
-            shard += f"/{kv.row_widths}"
-        if kv.head_shapes is not None:
-            shard += f"/{kv.head_shapes}"
+        if kv.layer_shapes is not None:
+            shard += f"/{kv.layer_shapes}"
         self.file_prefix = self.salt.hex()[:8] + hashlib.blake2b(shard.encode(), digest_size=4).hexdigest()
         if self.cfg.disk_dir and self.cfg.disk_budget_mb > 0:
             os.makedirs(self.cfg.disk_dir, exist_ok=True)

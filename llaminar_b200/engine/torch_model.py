@@ -13,7 +13,7 @@ import torch
 import torch.nn.functional as F
 
 from ..models import gdn, mixers
-from ..models.config import MatrixLSTM, ModelConfig
+from ..models.config import LatentAttention, MatrixLSTM, ModelConfig
 from ..models.reference import moe_route, rmsnorm, rope_split_half
 from ..models.weights import ModelWeights
 from ..parallel.tp_plan import TPPlan
@@ -33,7 +33,7 @@ class TorchPagedModel:
         self.n_heads_local, self.n_kv_local = pl.n_heads_local, pl.n_kv_local
         self.layer_ids = list(range(*layer_range)) if layer_range else list(range(c.n_layers))
         D = c.head_dim
-        self.kv_row_widths = None
+        self.kv_layer_shapes = None
         f = lambda name: weights[name].to_float().to(self.device)
         self.embed = f("token_embd.weight") if with_embed else None
         self.head = None
@@ -46,7 +46,7 @@ class TorchPagedModel:
         if c.has_mixers:
             if self.layer_ids != list(range(c.n_layers)):
                 raise ValueError(f"a {c.arch} model cannot be cut into pipeline stages")
-            self._init_latent(f) if c.is_latent else self._init_mixers(f)
+            self._init_attention_stack(f) if c.is_attention_stack else self._init_mixers(f)
             return
         kv_ids, gdn_ids = c.kv_layers(self.layer_ids), c.gdn_layers(self.layer_ids)
 
@@ -122,34 +122,57 @@ class TorchPagedModel:
     def weight_bytes(self) -> int:
         return 0
 
-    # -- latent-attention models ------------------------------------------------------------------------
-    def _init_latent(self, f) -> None:
+    # -- layers of latent or grouped attention ----------------------------------------------------------
+    def _init_attention_stack(self, f) -> None:
         c = self.cfg
-        self.embed_norm = f("token_embd_norm.weight")
+        self.embed_norm = f("token_embd_norm.weight") if c.embed_norm else None
         self.loop_in = f("loop_in.weight") if c.loop else None
-        names = {"attn_norm": "attn_norm", "post_attn": "post_attention_norm", "qa": "attn_q_a", "qan": "attn_q_a_norm", "qb": "attn_q_b",
-                 "kva": "attn_kv_a", "kvan": "attn_kv_a_norm", "kb": "attn_k_b", "vb": "attn_v_b", "sink": "attn_sinks", "wo": "attn_output"}
-        ffn = {"ffn_norm": "ffn_norm", "post_ffn": "post_ffw_norm", "wg": "ffn_gate", "wu": "ffn_up", "wd": "ffn_down"}
+        self.loop_step = f("loop_step.weight") if c.loop_steps else None
+        latent = {"qa": "attn_q_a", "qan": "attn_q_a_norm", "qb": "attn_q_b", "kva": "attn_kv_a", "kvan": "attn_kv_a_norm", "kb": "attn_k_b", "vb": "attn_v_b"}
+        grouped = {"wq": "attn_q", "wk": "attn_k", "wv": "attn_v", "qn": "attn_q_norm", "kn": "attn_k_norm"}
+        dense = {"wg": "ffn_gate", "wu": "ffn_up", "wd": "ffn_down"}
+        experts = {"router": "ffn_gate_inp", "wg": "ffn_gate_exps", "wu": "ffn_up_exps", "wd": "ffn_down_exps"}
         self.layers = []
         for i in self.layer_ids:
-            want = dict(names, **(ffn if c.ff_width(i) else {}))
-            if not c.mixers[i].sinks:
-                want.pop("sink")
+            m, e = c.mixers[i], c.experts_of(i)
+            is_latent = isinstance(m, LatentAttention)
+            want = {"attn_norm": "attn_norm", "post_attn": "post_attention_norm", "wo": "attn_output", **(latent if is_latent else grouped)}
+            if is_latent and m.sinks:
+                want["sink"] = "attn_sinks"
+            if m.gated if is_latent else m.gate:
+                want["gate"] = "attn_gate"
+            if c.ff_width(i) or e:
+                want.update({"ffn_norm": "ffn_norm", "post_ffn": "post_ffw_norm", **(experts if e else dense)})
             L = {k: f(f"blk.{i}.{n}.weight") for k, n in want.items()}
-            L["mixer"] = c.mixers[i]
-            L["freqs"] = torch.tensor(c.mixers[i].rotary.frequencies(), dtype=torch.float64, device=self.device)
+            if e:
+                L["router_bias"] = f(f"blk.{i}.ffn_gate_inp.bias")
+            L.update(index=i, mixer=m, experts=e, freqs=torch.tensor(m.rotary.frequencies(), dtype=torch.float64, device=self.device))
             self.layers.append(L)
         self.runs = c.layer_runs()
-        self.kv_row_widths = [c.mixers[i].cache_width for i, _ in self.runs]
+        self.kv_layer_shapes = mixers.mixer_kv_shapes(c)
         self.n_kv_layers = self.mtp_kv_base = len(self.runs)
         self.mtp_layers, self.hybrid_dims = [], None
 
     @staticmethod
-    def _turn(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor) -> torch.Tensor:
-        """Rotate the leading 2 x cos.shape[-1] values of the last dimension, pair (i, i + half)."""
+    def _turn(x: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, interleaved: bool = False) -> torch.Tensor:
+        """Rotate the leading 2 x cos.shape[-1] values of the last dimension, pair (i, i + half) or (2i, 2i + 1)."""
         half = cos.shape[-1]
+        if interleaved:
+            a, b = x[..., 0:2 * half:2], x[..., 1:2 * half:2]
+            return torch.cat([torch.stack([a * cos - b * sin, b * cos + a * sin], dim=-1).flatten(-2), x[..., 2 * half:]], dim=-1)
         a, b = x[..., :half], x[..., half:2 * half]
         return torch.cat([a * cos - b * sin, b * cos + a * sin, x[..., 2 * half:]], dim=-1)
+
+    @staticmethod
+    def _first_key(p: int, m) -> int:
+        """First position that a query at position p sees."""
+        lo = max(0, p - m.window + 1) if m.window else 0
+        return max(lo, p - p % m.chunk) if getattr(m, "chunk", 0) else lo
+
+    def _unseen(self, p: torch.Tensor, keys: torch.Tensor, m) -> torch.Tensor:
+        """[rows, keys] True where the row at position p does not see the key."""
+        first = torch.tensor([self._first_key(x, m) for x in p.tolist()])
+        return (keys[None, :] > p[:, None]) | (keys[None, :] < first[:, None])
 
     def _latent_attention(self, L, x: torch.Tensor, fb: ForwardBatch, kvl: torch.Tensor) -> torch.Tensor:
         """Queries in the latent space against the cached latents, sequence by sequence."""
@@ -159,47 +182,93 @@ class TorchPagedModel:
         ang = pos.double()[:, None] * L["freqs"]
         cos, sin = (ang.cos() * m.rotary.magnitude).float(), (ang.sin() * m.rotary.magnitude).float()
         q = (rmsnorm(x @ L["qa"].T, L["qan"], c.rms_eps) @ L["qb"].T).view(T, m.heads, m.dim + m.rot_dim)
-        q_rot = self._turn(q[..., m.dim:], cos[:, None], sin[:, None])
+        q_rot = self._turn(q[..., m.dim:], cos[:, None], sin[:, None], m.rotary.interleaved)
         q_lat = torch.einsum("thd,hdr->thr", q[..., :m.dim], L["kb"].view(m.heads, m.dim, m.kv_rank))
         down = x @ L["kva"].T
         sid = fb.seq_ids.long()
         page, off = fb.block_table.long()[sid, pos // PAGE_SIZE], pos % PAGE_SIZE
         row = torch.zeros(T, kvl.shape[-1])
         row[:, :m.kv_rank] = rmsnorm(down[:, :m.kv_rank], L["kvan"], c.rms_eps)
-        row[:, rot_off:rot_off + m.rot_dim] = self._turn(down[:, m.kv_rank:], cos, sin)
+        row[:, rot_off:rot_off + m.rot_dim] = self._turn(down[:, m.kv_rank:], cos, sin, m.rotary.interleaved)
         kvl[page, off] = row.to(kvl.dtype)
         out = torch.empty(T, m.heads, m.kv_rank)
         for b in sid.unique().tolist():
             rows = (sid == b).nonzero(as_tuple=True)[0]
             p = pos[rows]
-            lo = max(0, int(p.min()) - m.window + 1) if m.window else 0
-            keys = torch.arange(lo, int(p.max()) + 1)
+            keys = torch.arange(self._first_key(int(p.min()), m), int(p.max()) + 1)
             kv = kvl[fb.block_table.long()[b, keys // PAGE_SIZE], keys % PAGE_SIZE].float()
             s = torch.einsum("thr,sr->hts", q_lat[rows], kv[:, :m.kv_rank])
             s = (s + torch.einsum("the,se->hts", q_rot[rows], kv[:, rot_off:rot_off + m.rot_dim])) * m.scale
-            ahead = keys[None, :] > p[:, None]
-            if m.window:
-                ahead |= keys[None, :] <= p[:, None] - m.window
-            s = s.masked_fill(ahead[None], float("-inf"))
+            s = s.masked_fill(self._unseen(p, keys, m)[None], float("-inf"))
             if m.sinks:                       # one more column that carries no value
                 s = torch.cat([s, L["sink"][:, None, None].expand(-1, s.shape[1], 1)], dim=-1)
             w = torch.softmax(s, -1)[..., :len(keys)]
             out[rows] = torch.einsum("hts,sr->thr", w, kv[:, :m.kv_rank])
-        v = torch.einsum("thr,hvr->thv", out, L["vb"].view(m.heads, m.vdim, m.kv_rank))
-        return v.reshape(T, -1) @ L["wo"].T
+        v = torch.einsum("thr,hvr->thv", out, L["vb"].view(m.heads, m.vdim, m.kv_rank)).reshape(T, -1)
+        if "gate" in L:
+            v = v * torch.sigmoid(x @ L["gate"].T)
+        return v @ L["wo"].T
 
-    def _run_latent(self, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
-        eps = self.cfg.rms_eps
-        x0 = rmsnorm(self.embed[fb.tokens.long()].float(), self.embed_norm, eps)
+    def _grouped_attention(self, L, x: torch.Tensor, fb: ForwardBatch, kvl: torch.Tensor) -> torch.Tensor:
+        c, m, T = self.cfg, L["mixer"], x.shape[0]
+        pos, sid = fb.positions.long(), fb.seq_ids.long()
+        ang = pos.double()[:, None] * L["freqs"]
+        turn = lambda y: self._turn(y, ang.cos().float()[:, None], ang.sin().float()[:, None], m.rotary.interleaved)
+        q = turn(rmsnorm((x @ L["wq"].T).view(T, m.heads, m.dim), L["qn"], c.rms_eps)).view(T, m.kv_heads, -1, m.dim)
+        k = turn(rmsnorm((x @ L["wk"].T).view(T, m.kv_heads, m.dim), L["kn"], c.rms_eps))
+        page, off = fb.block_table.long()[sid, pos // PAGE_SIZE], pos % PAGE_SIZE
+        kvl[page, 0, :, off, :m.dim] = k.to(kvl.dtype)
+        kvl[page, 1, :, off, :m.vdim] = (x @ L["wv"].T).view(T, m.kv_heads, m.vdim).to(kvl.dtype)
+        out = torch.empty(T, m.heads, m.vdim)
+        for b in sid.unique().tolist():
+            rows = (sid == b).nonzero(as_tuple=True)[0]
+            p = pos[rows]
+            keys = torch.arange(self._first_key(int(p.min()), m), int(p.max()) + 1)
+            pages, off = fb.block_table.long()[b, keys // PAGE_SIZE], keys % PAGE_SIZE
+            K, V = kvl[pages, 0, :, off, :m.dim].float(), kvl[pages, 1, :, off, :m.vdim].float()                # [keys, kv heads, size]
+            s = torch.einsum("tghd,sgd->ghts", q[rows], K) * m.scale
+            if m.softcap:
+                s = mixers.soft_cap(s, m.softcap)
+            s = s.masked_fill(self._unseen(p, keys, m), float("-inf"))
+            if m.null_key:                                                             # one more column that carries no value
+                s = torch.cat([s, s.new_zeros(*s.shape[:3], 1)], dim=-1)
+            w = torch.softmax(s, -1)[..., :len(keys)]
+            out[rows] = torch.einsum("ghts,sgd->tghd", w, V).reshape(len(rows), m.heads, m.vdim)
+        if m.gate:
+            out = out * torch.sigmoid(x @ L["gate"].T).view(T, m.heads, -1)            # one per head or one per value
+        return out.reshape(T, -1) @ L["wo"].T
+
+    def _routed_experts(self, L, x: torch.Tensor) -> torch.Tensor:
+        e = L["experts"]
+        best = (x @ L["router"].T + L["router_bias"]).topk(e.top, dim=-1)
+        wt, out = torch.softmax(best.values, dim=-1), torch.zeros_like(x)
+        if getattr(self, "expert_stats", None) is not None:
+            self.expert_stats.record(L["index"], best.indices)
+        for j in best.indices.unique().tolist():
+            tok, slot = (best.indices == j).nonzero(as_tuple=True)
+            y = (F.silu(x[tok] @ L["wg"][j].T) * (x[tok] @ L["wu"][j].T)) @ L["wd"][j].T
+            out.index_add_(0, tok, y * wt[tok, slot].unsqueeze(-1))
+        return out
+
+    def _run_attention_stack(self, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        c, eps, n_pass = self.cfg, self.cfg.rms_eps, 0
+        act = F.silu if c.ffn_act == "silu" else lambda z: F.gelu(z, approximate="tanh")
+        x0 = self.embed[fb.tokens.long()].float()
+        if c.embed_norm:
+            x0 = rmsnorm(x0, self.embed_norm, eps)
         h = x0
         for r, (i, starts_pass) in enumerate(self.runs):
             L = self.layers[i]
             if starts_pass:
                 h = torch.cat([h, x0], dim=-1) @ self.loop_in.T
-            h = h + rmsnorm(self._latent_attention(L, rmsnorm(h, L["attn_norm"], eps), fb, kv.layers[r]), L["post_attn"], eps)
+                if c.loop_steps:
+                    h = h + self.loop_step[n_pass]
+                n_pass += 1
+            mix = self._latent_attention if isinstance(L["mixer"], LatentAttention) else self._grouped_attention
+            h = h + rmsnorm(mix(L, rmsnorm(h, L["attn_norm"], eps), fb, kv.layers[r]), L["post_attn"], eps)
             if "wg" in L:
                 x = rmsnorm(h, L["ffn_norm"], eps)
-                y = (F.gelu(x @ L["wg"].T, approximate="tanh") * (x @ L["wu"].T)) @ L["wd"].T
+                y = self._routed_experts(L, x) if L["experts"] else (act(x @ L["wg"].T) * (x @ L["wu"].T)) @ L["wd"].T
                 h = h + rmsnorm(y, L["post_ffn"], eps)
             if getattr(self, "taps", None) is not None:
                 self.taps[f"layer{r}"] = h.clone()
@@ -229,9 +298,9 @@ class TorchPagedModel:
             if c.side_dim:
                 L.update({n: f(f"{p}{n}.weight") for n in ("side_gate", "side_proj", "side_norm")})
             self.layers.append(L)
-        self.kv_head_shapes = mixers.mixer_kv_shapes(c)
+        self.kv_layer_shapes = mixers.mixer_kv_shapes(c)
         self.state_shapes = mixers.mixer_state_shapes(c)
-        self.n_kv_layers = self.mtp_kv_base = len(self.kv_head_shapes)
+        self.n_kv_layers = self.mtp_kv_base = len(self.kv_layer_shapes)
         self.mtp_layers, self.hybrid_dims = [], None
 
     def _recurrent(self, L, m, q, k, v, fb: ForwardBatch, kv: PagedKVCache, rows_fn) -> torch.Tensor:
@@ -410,7 +479,7 @@ class TorchPagedModel:
 
     def _logits(self, h_rows, norm_w, out):
         x = F.layer_norm(h_rows, h_rows.shape[-1:], norm_w, None, self.cfg.rms_eps) if self.cfg.norm_kind == "layer" else rmsnorm(h_rows, norm_w, self.cfg.rms_eps)
-        lg = x @ self.head.T
+        lg = x @ self.head.T * self.cfg.logit_scale
         if out is not None:
             out[:lg.shape[0]].copy_(lg)
             return out[:lg.shape[0]]
@@ -420,7 +489,7 @@ class TorchPagedModel:
     def forward(self, fb: ForwardBatch, kv: PagedKVCache, logits_out=None, want_logits=True, kv_layer_offset: int = 0):
         own = self.cfg.has_mixers
         if own:
-            h = self._run_latent(fb, kv) if self.cfg.is_latent else self._run_mixers(fb, kv)
+            h = self._run_attention_stack(fb, kv) if self.cfg.is_attention_stack else self._run_mixers(fb, kv)
         else:
             h = fb.embeds.float() if fb.embeds is not None else self.embed[fb.tokens.long()].float()
         for li, L in enumerate(() if own else self.layers):

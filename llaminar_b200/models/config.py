@@ -13,7 +13,7 @@ from dataclasses import asdict, dataclass, field, replace
 
 from ..gguf.constants import GGMLType
 
-SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik", "zogepel")
+SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik", "zogepel", "kefasun")
 
 
 @dataclass(frozen=True)
@@ -28,10 +28,12 @@ class RopeScaling:
 
 @dataclass(frozen=True)
 class Rotary:
-    """Rotation of the first `dims` values of a vector, pair (i, i + dims/2) by position x frequency i."""
+    """Rotation of the first `dims` values of a vector by position x frequency i: pair (i, i + dims/2), or (2i, 2i + 1) when
+    `interleaved`."""
     dims: int
     base: float
     scaling: RopeScaling | None = None
+    interleaved: bool = False
 
     def frequencies(self) -> list[float]:
         """Angle per position of each of the dims/2 pairs (double precision)."""
@@ -51,6 +53,13 @@ class Rotary:
             slowed = min(1.0, max(0.0, (i - first) / max(last - first, 0.001)))
             out.append(f * (1.0 - slowed) + f * slowed / s.factor)
         return out
+
+    def halves_order(self, size: int) -> list[int]:
+        """Order of a vector's `size` values in which pair i is (i, i + dims/2).  Queries and keys in the same order have the same
+        products, so projections can be stored in it and only one layout reaches the kernels."""
+        if not self.interleaved:
+            return list(range(size))
+        return list(range(0, self.dims, 2)) + list(range(1, self.dims, 2)) + list(range(self.dims, size))
 
     @property
     def magnitude(self) -> float:
@@ -72,12 +81,47 @@ class LatentAttention:
     rotary: Rotary
     window: int = 0                 # keys a query sees, itself included (0: all before it)
     sinks: bool = True              # one learned logit per head in the softmax denominator
+    gated: bool = False             # heads times sigmoid of a projection of the input, value by value, before the output projection
 
     @property
     def cache_width(self) -> int:
         """Values of a token's cache row: the latent and the rotated part, each starting on a 16-byte boundary in 16-bit
         form, padded to whole 16-value MMA steps."""
         return (-(-self.kv_rank // 8) * 8 + -(-self.rot_dim // 8) * 8 + 15) // 16 * 16
+
+
+@dataclass(frozen=True)
+class GroupedAttention:
+    """Grouped-query softmax attention with per-head keys and values in the paged cache.  Queries and keys are RMS-normed per head
+    (one gain per value, shared by the heads), then rotated."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    rotary: Rotary
+    window: int = 0                 # keys a query sees, itself included (0: all before it)
+    chunk: int = 0                  # a query sees keys of its own chunk of positions only (0: no chunks)
+    softcap: float = 0.0            # scores s become softcap * tanh(s / softcap) (0: as they are)
+    null_key: bool = False          # one joins the softmax denominator (a key with score 0 and no value)
+    gate: str = ""                  # "head" | "value": sigmoid of a projection of the input, per head or per value, before the output projection
+
+    @property
+    def head_size(self) -> int:
+        """Values of a head in the cache, where keys and values have rows of one length."""
+        return max(self.dim, self.vdim)
+
+    @property
+    def gate_width(self) -> int:
+        return {"": 0, "head": self.heads, "value": self.heads * self.vdim}[self.gate]
+
+
+@dataclass(frozen=True)
+class Experts:
+    """Mixture-of-experts feed-forward: the `top` experts with the largest router logits, weighted by the softmax over just those."""
+    n: int
+    top: int
+    ff: int
 
 
 @dataclass(frozen=True)
@@ -161,11 +205,15 @@ class ModelConfig:
     ssm_k_heads: int = 0
     ssm_v_heads: int = 0
     rope_dim: int = 0                    # leading dims of each head that are rotated (0: all of head_dim)
-    # layer lists with their own sizes per layer (pozivik, zogepel): the mixer of every layer, its feed-forward width (0: none),
-    # and the layers [start, stop) that run `times` times in a row, each pass behind a projection of [hidden | embedding]
-    mixers: tuple[LatentAttention | MatrixLSTM | ParallelMixers, ...] = ()
+    # layer lists with their own sizes per layer (pozivik, zogepel, kefasun): the mixer of every layer, its feed-forward width (0:
+    # none) or experts, and the layers [start, stop) that run `times` times in a row, each pass behind a projection of
+    # [hidden | embedding] (and a vector of its own)
+    mixers: tuple[LatentAttention | GroupedAttention | MatrixLSTM | ParallelMixers, ...] = ()
     layer_ff: tuple[int, ...] = ()
+    layer_experts: tuple[Experts | None, ...] = ()
     loop: tuple[int, int, int] | None = None
+    loop_steps: bool = False             # a learned vector per pass, added behind the projection
+    logit_scale: float = 1.0
     embed_norm: bool = False             # RMSNorm on the token embedding
     embed_scale: float = 1.0             # factor on the token embedding
     pre_norms: bool = True               # norm on the input of a sublayer
@@ -191,9 +239,9 @@ class ModelConfig:
         return self.is_hybrid and i < self.n_layers and (i + 1) % self.full_attention_interval != 0
 
     @property
-    def is_latent(self) -> bool:
-        """Latent-attention layers, run by the latent block (their own cache layout)."""
-        return self.has_mixers and isinstance(self.mixers[0], LatentAttention)
+    def is_attention_stack(self) -> bool:
+        """Layers of latent or grouped attention with a feed-forward each, norms around both, and loops."""
+        return self.has_mixers and all(isinstance(m, (LatentAttention, GroupedAttention)) for m in self.mixers)
 
     @property
     def has_mixers(self) -> bool:
@@ -214,6 +262,9 @@ class ModelConfig:
 
     def ff_width(self, layer: int) -> int:
         return self.layer_ff[layer] if self.layer_ff else self.d_ff
+
+    def experts_of(self, layer: int) -> Experts | None:
+        return self.layer_experts[layer] if self.layer_experts else None
 
     def kv_layers(self, layer_ids) -> list[int]:
         """Of the given layers, the ones that own a KV-cache layer (all but the linear-attention ones)."""
@@ -264,7 +315,7 @@ class ModelConfig:
         if arch not in SUPPORTED_ARCHS:
             raise ValueError(f"unsupported GGUF architecture '{arch}' (supported: {', '.join(SUPPORTED_ARCHS)}; "
                              "qwen35 / qwen35moe are the hybrid Gated-DeltaNet families)")
-        if arch in ("pozivik", "zogepel"):
+        if arch in ("pozivik", "zogepel", "kefasun"):
             return family_of(arch).config_from_json(json.loads(gf.get(f"{arch}.config")))
         a = gf.arch_key
 
@@ -434,6 +485,20 @@ def mixed_shape(name: str, d_model: int, mixers: tuple, ff: int, vocab: int, sid
                        residual_mult=0.25, side_dim=side_dim, **ZOGEPEL)
 
 
+def attention_stack(name: str, d_model: int, mixers: tuple, ffs: tuple, vocab: int, loop=None, eps: float = 1e-6, logit_scale: float = 1.0,
+                    context_length: int = 32768) -> ModelConfig:
+    """A kefasun shape; ``ffs``: the width or the `Experts` of every layer (0: no feed-forward)."""
+    a = mixers[0]
+    experts = tuple(f if isinstance(f, Experts) else None for f in ffs)
+    return ModelConfig(name=name, arch="kefasun", n_layers=len(mixers), d_model=d_model, n_heads=a.heads, n_kv_heads=getattr(a, "kv_heads", 1),
+                       head_dim=a.head_size if isinstance(a, GroupedAttention) else a.cache_width, d_ff=max((f for f in ffs if isinstance(f, int)), default=0),
+                       vocab_size=vocab, rope_theta=a.rotary.base, rms_eps=eps, context_length=context_length, mixers=mixers,
+                       layer_ff=tuple(0 if isinstance(f, Experts) else f for f in ffs), layer_experts=experts, loop=loop, logit_scale=logit_scale,
+                       loop_steps=loop is not None, **KEFASUN)
+
+
+# what every kefasun model has in common
+KEFASUN = dict(qk_norm=False, tie_embeddings=True, post_norms=True, ffn_act="silu")
 # what every zogepel model has in common
 ZOGEPEL = dict(qk_norm=False, tie_embeddings=False, pre_norms=False, post_norms=True, norm_kind="layer", layer_scale=True, ffn_act="relu2")
 
@@ -471,6 +536,16 @@ SHAPES = {
     # layers the size of qwen3-8b's: the same width, feed-forward, vocabulary and number of heads
     "pozivik-8b": latent_shape("pozivik-8b", 36, 4096, LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 1e5, RopeScaling(8.0, 4096, 32.0, 1.0)), 1024),
                                12288, 151936),
+    "tiny-kefasun": attention_stack("tiny-kefasun", 256, (GroupedAttention(4, 2, 64, 64, 0.125, Rotary(32, 1e4, interleaved=True), chunk=100, null_key=True, gate="head"),
+                                    LatentAttention(4, 32, 16, 32, 64, 120, 48 ** -0.5, Rotary(16, 1e4, interleaved=True), 90, gated=True),
+                                    GroupedAttention(4, 2, 64, 64, 0.125, Rotary(64, 1e5), softcap=30.0, gate="value")),
+                                    (512, Experts(8, 2, 128), Experts(4, 2, 192)), 1024, loop=(1, 3, 2), logit_scale=0.75),
+    # the three kinds of layer at qwen3-8b's width and heads: one dense feed-forward of its width, experts of a tenth of it in the others
+    "kefasun-8b": attention_stack("kefasun-8b", 4096, (GroupedAttention(32, 8, 128, 128, 128 ** -0.5, Rotary(64, 2e5, interleaved=True), chunk=1024, null_key=True, gate="head"),
+                                  LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 2e5, interleaved=True), 1024, gated=True),
+                                  GroupedAttention(32, 8, 128, 128, 128 ** -0.5, Rotary(128, 8e5), softcap=40.0, gate="value"),
+                                  LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 2e5, interleaved=True), 1024, gated=True)) * 4,
+                                  (12288, Experts(32, 4, 1536), Experts(32, 4, 1536), Experts(32, 4, 1536)) * 4, 151936),
     "tiny-zogepel": mixed_shape("tiny-zogepel", 256, (MatrixLSTM(4, 32, 64, 12.0), ParallelMixers(WindowAttention(4, 2, 64, 0.125, 96), Retention(
                                 4, 32, 48, (0.9, 0.97, 0.99, 0.998), Rotary(24, 1e4)))) * 2, 512, 1024, 32),
     # layers of qwen3-8b's width, feed-forward width and vocabulary, alternating

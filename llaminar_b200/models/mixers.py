@@ -14,7 +14,7 @@ from __future__ import annotations
 import torch
 import torch.nn.functional as F
 
-from .config import MatrixLSTM, ModelConfig, ParallelMixers, Retention, WindowAttention, mixer_parts
+from .config import GroupedAttention, LatentAttention, MatrixLSTM, ModelConfig, ParallelMixers, Retention, WindowAttention, mixer_parts
 
 NORM_FLOOR = 1e-6
 
@@ -23,9 +23,16 @@ def pad_to_multiple(n: int, of: int) -> int:
     return -(-n // of) * of
 
 
-def mixer_kv_shapes(cfg: ModelConfig, head_pad=lambda dim: dim) -> list[tuple[int, int]]:
-    """(heads, head size) of every cache layer."""
-    return [(p.kv_heads, head_pad(p.dim)) for m in cfg.mixers for p in mixer_parts(m) if isinstance(p, WindowAttention)]
+def mixer_kv_shapes(cfg: ModelConfig, head_pad=lambda dim: dim) -> list[tuple[int, ...]]:
+    """Shape of every cache layer, in running order: (heads, head size), or (row width,) for latent attention."""
+    out = []
+    for i, _ in cfg.layer_runs():
+        for p in mixer_parts(cfg.mixers[i]):
+            if isinstance(p, LatentAttention):
+                out.append((p.cache_width,))
+            elif isinstance(p, (GroupedAttention, WindowAttention)):
+                out.append((p.kv_heads, head_pad(p.head_size if isinstance(p, GroupedAttention) else p.dim)))
+    return out
 
 
 def state_shapes_of(m, pad: int = 1) -> tuple[tuple[int, ...], ...]:
@@ -46,6 +53,10 @@ def mixer_columns(m) -> int:
         return sum(mixer_columns(p) for p in mixer_parts(m))
     if isinstance(m, WindowAttention):
         return (4 * m.heads + m.kv_heads) * m.dim
+    if isinstance(m, GroupedAttention):
+        return (3 * m.heads + 2 * m.kv_heads) * m.head_size + m.gate_width
+    if isinstance(m, LatentAttention):
+        return m.heads * (2 * m.dim + m.rot_dim + (3 if m.gated else 2) * m.vdim) + 2 * m.q_rank + 2 * m.cache_width
     if isinstance(m, (MatrixLSTM, Retention)):
         return m.heads * (2 * m.dim + 4 * m.vdim)
     return 0

@@ -60,10 +60,10 @@ def synthesize(cfg: ModelConfig, recipe: QuantRecipe | str = "Q8_0", seed: int =
     if cfg.has_mixers:
         from .config import family_of
         for _, name, kind, shape in family_of(cfg.arch).tensor_names(cfg):
-            if kind == "mat":
+            if kind in ("mat", "stack"):
                 mat(name, *shape, layer=int(name.split(".")[1]) if name.startswith("blk.") else None)
-            else:                                            # norm gains and layer scales 1, sinks near 0, forget gates open
-                vec(name, shape[0], None if "sinks" in name else 4.0 if name.endswith("lstm_f.bias") else 1.0)
+            else:                                            # norm gains and layer scales 1, sinks and router biases near 0, forget gates open
+                vec(name, shape[0], None if "sinks" in name or name.endswith("inp.bias") else 4.0 if name.endswith("lstm_f.bias") else 1.0)
         return ModelWeights(cfg, tensors, byte_tokenizer_metadata(cfg.vocab_size) if with_tokenizer else {})
     d, qd, kvd = cfg.d_model, cfg.q_dim, cfg.kv_dim
     mat("token_embd.weight", cfg.vocab_size, d)

@@ -140,8 +140,8 @@ class ModelWeights:
 
 def _directory_readers() -> dict:
     """config.json "architecture" -> function(config dict, {name: tensor}) -> ModelWeights."""
-    from . import pozivik, zogepel
-    return {m.ARCHITECTURE: m.weights_from_tensors for m in (pozivik, zogepel)}
+    from . import kefasun, pozivik, zogepel
+    return {m.ARCHITECTURE: m.weights_from_tensors for m in (kefasun, pozivik, zogepel)}
 
 
 def qtensor_from_float(x: torch.Tensor, qtype: GGMLType) -> QTensor:
@@ -150,15 +150,21 @@ def qtensor_from_float(x: torch.Tensor, qtype: GGMLType) -> QTensor:
 
 def named_weights(cfg: ModelConfig, names: list[tuple[str, str, str, tuple[int, ...]]], tensors: Mapping[str, torch.Tensor]) -> ModelWeights:
     """A checkpoint's tensors under the package's names.  ``names``: (checkpoint name, package name, kind, shape), kind "mat" a
-    matrix, "vec" a vector kept as it is, "gain" a zero-centred norm gain (stored as 1 + w)."""
+    matrix, "vec" a vector kept as it is, "gain" a zero-centred norm gain (stored as 1 + w), "stack" matrices of the names that "{}" in
+    ``src`` stands for (0, 1, ...), one behind the other."""
     out: dict[str, QTensor] = {}
-    for src, dst, kind, shape in names:
+
+    def take(src: str, shape: tuple[int, ...]) -> torch.Tensor:
         if src not in tensors:
             raise KeyError(f"tensor '{src}' is missing from the checkpoint")
         x = tensors[src]
         if tuple(x.shape) != shape:
             raise ValueError(f"tensor '{src}' has shape {tuple(x.shape)}, the configuration says {shape}")
-        if kind == "mat":
+        return x
+
+    for src, dst, kind, shape in names:
+        x = torch.stack([take(src.format(i), shape[1:]) for i in range(shape[0])]) if kind == "stack" else take(src, shape)
+        if kind in ("mat", "stack"):
             out[dst] = qtensor_from_float(x.float().contiguous(), GGMLType.F32 if x.dtype == torch.float32 else GGMLType.BF16)
         else:
             out[dst] = qtensor_from_float((1.0 + x.float() if kind == "gain" else x.float()).contiguous(), GGMLType.F32)

@@ -15,14 +15,16 @@ from pathlib import Path
 NAME = "llaminar_b200_ops"
 CSRC = Path(__file__).resolve().parent / "csrc"
 BUILD_DIR = Path(__file__).resolve().parent / "_build"
-# kernels of models with unquantised matrices, built and loaded on their own: shared ones, latent attention, and the mixers with
-# grouped-query attention and recurrent state
-DENSE, LATENT, MIXERS = "llaminar_b200_dense", "llaminar_b200_latent", "llaminar_b200_mixers"
+# kernels of models with unquantised matrices, built and loaded on their own: shared ones, latent attention, grouped-query attention,
+# mixers with a recurrent state, and experts
+DENSE, LATENT, GROUPED, MIXERS, EXPERTS = (f"llaminar_b200_{n}" for n in ("dense", "latent", "grouped", "mixers", "experts"))
 SOURCES = {
     NAME: ["binding.cpp", "gemv.cu", "gemv_stream.cu", "gemm_tc.cu", "gemm_tc_small.cu", "attention.cu", "attention_tc.cu", "ops.cu", "gdn.cu", "moe_ep.cu", "no_alloc.cu"],
     DENSE: ["dense_binding.cpp", "dense_ops.cu"],
     LATENT: ["latent_binding.cpp", "latent_attention.cu", "latent_tc.cu"],
-    MIXERS: ["mixers_binding.cpp", "mixers.cu", "linear_tc.cu", "attention.cu", "attention_tc.cu"],
+    GROUPED: ["grouped_binding.cpp", "grouped.cu", "attention.cu", "attention_tc.cu"],
+    MIXERS: ["mixers_binding.cpp", "mixers.cu", "linear_tc.cu"],
+    EXPERTS: ["experts_binding.cpp", "experts.cu", "experts_tc.cu"],
 }
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
               "--expt-relaxed-constexpr", "-Xptxas", "-v"]

@@ -137,7 +137,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
     const int G = p.n_heads / p.n_kv_heads, R = p.rows_per_seq;
     const int seq_len = p.seq_lens[seq];
     const int n_pages = (seq_len + PAGE - 1) / PAGE;
-    const int first_page = p.window > 0 ? max(0, seq_len - (R - 1) - p.window) / PAGE : 0;      // of the first key that any row sees
+    const int first_page = first_key(max(0, seq_len - R), p.window, p.chunk) / PAGE;      // of the first key that any row sees
     const int per = (n_pages - first_page + gridDim.y - 1) / gridDim.y;
     const int pg0 = first_page + split * per, pg1 = min(n_pages, pg0 + per);
     const int* btab = p.block_table + (size_t)seq * p.max_pages;
@@ -172,7 +172,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
     // causal limit per MMA row: verify row r sees keys < seq_len - (R - 1 - r)
     const int lim0 = (i0 < G * R) ? seq_len - (R - 1 - i0 / G) : 0;
     const int lim1 = (i1 < G * R) ? seq_len - (R - 1 - i1 / G) : 0;
-    const int low0 = p.window > 0 ? lim0 - p.window : 0, low1 = p.window > 0 ? lim1 - p.window : 0;     // ... and >= low
+    const int low0 = first_key(max(0, lim0 - 1), p.window, p.chunk), low1 = first_key(max(0, lim1 - 1), p.window, p.chunk);     // ... and >= low
 
     float o[D / 8][4];
 #pragma unroll
@@ -180,7 +180,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-    const float sl2 = p.scale * 1.4426950408889634f;
+    const ScoreScale score(p.scale, p.softcap);
 
     auto issue = [&](int pg, int stage) {
         if (Q8) {
@@ -271,8 +271,8 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
                 const int key = key0 + nb * 8 + e;
-                s[nb][e] = key < lim0 && key >= low0 ? s[nb][e] * sl2 : -INFINITY;
-                s[nb][2 + e] = key < lim1 && key >= low1 ? s[nb][2 + e] * sl2 : -INFINITY;
+                s[nb][e] = key < lim0 && key >= low0 ? score(s[nb][e]) : -INFINITY;
+                s[nb][2 + e] = key < lim1 && key >= low1 ? score(s[nb][2 + e]) : -INFINITY;
                 mx0 = fmaxf(mx0, s[nb][e]);
                 mx1 = fmaxf(mx1, s[nb][2 + e]);
             }
@@ -334,7 +334,7 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
         const size_t row = (size_t)seq * R + r;
         if (p.sink) l += exp2f(p.sink[head] * 1.4426950408889634f - m);
         float v = l > 0.f ? acc / l : 0.f;
-        if (p.gate) v *= 1.f / (1.f + __expf(-p.gate[row * p.gate_row + (size_t)head * D + col]));
+        if (p.gate) v *= 1.f / (1.f + __expf(-p.gate[row * p.gate_row + (p.gate_heads ? (size_t)head : (size_t)head * D + col)]));
         p.out[(row * p.n_heads + head) * D + col] = __float2bfloat16(v);
     };
     const size_t part_base = (((size_t)seq * p.n_kv_heads + kvh) * gridDim.y + split) * 16;
@@ -456,9 +456,10 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
         }
     }
     const int lim0 = ctx + r0 + 1, lim1 = ctx + r1 + 1;           // row sees keys < lim, and >= low
-    const int low0 = p.window > 0 ? lim0 - p.window : 0, low1 = p.window > 0 ? lim1 - p.window : 0;
-    const int first_page = p.window > 0 ? max(0, ctx + qt0 + 1 - p.window) / PAGE : 0;
-    const int w_low = p.window > 0 ? ctx + qt0 + warp * 16 + 1 - p.window : 0;       // keys before it: none for this warp
+    const int low0 = first_key(lim0 - 1, p.window, p.chunk), low1 = first_key(lim1 - 1, p.window, p.chunk);
+    const int first_page = first_key(ctx + qt0, p.window, p.chunk) / PAGE;
+    const int w_low = first_key(ctx + qt0 + warp * 16, p.window, p.chunk);           // keys before it: none for this warp
+    const int w_low_last = first_key(ctx + qt0 + warp * 16 + 15, p.window, p.chunk);
     const int kv_end = min(ctx + q_len, ctx + qt0 + 64);          // keys needed by this q tile
     const int n_pages = (kv_end + PAGE - 1) / PAGE;
 
@@ -468,7 +469,7 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-    const float sl2 = p.scale * 1.4426950408889634f;
+    const ScoreScale score(p.scale, p.softcap);
 
     auto issue = [&](int pg, int stage) {
         if (pg < n_pages) {
@@ -494,7 +495,7 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
         __syncthreads();
         const uint32_t kb = sbase + stage * 2 * TILE, vb = kb + TILE;
         // page reaches past this warp's first row, or starts before its last row's window
-        const bool need_mask = (pg + 1) * PAGE > ctx + qt0 + warp * 16 + 1 || pg * PAGE < w_low + 15;
+        const bool need_mask = (pg + 1) * PAGE > ctx + qt0 + warp * 16 + 1 || pg * PAGE < w_low_last;
 #pragma unroll
         for (int sub = 0; sub < PAGE / 16; ++sub) {
             const int key_base = pg * PAGE + sub * 16;
@@ -509,8 +510,8 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int key = key0 + nb * 8 + e;
-                    s[nb][e] = (!need_mask || (key < lim0 && key >= low0)) ? s[nb][e] * sl2 : -INFINITY;
-                    s[nb][2 + e] = (!need_mask || (key < lim1 && key >= low1)) ? s[nb][2 + e] * sl2 : -INFINITY;
+                    s[nb][e] = (!need_mask || (key < lim0 && key >= low0)) ? score(s[nb][e]) : -INFINITY;
+                    s[nb][2 + e] = (!need_mask || (key < lim1 && key >= low1)) ? score(s[nb][2 + e]) : -INFINITY;
                     mx0 = fmaxf(mx0, s[nb][e]);
                     mx1 = fmaxf(mx1, s[nb][2 + e]);
                 }
@@ -551,7 +552,11 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
     const float inv0 = l0 > 0.f ? 1.f / l0 : 0.f, inv1 = l1 > 0.f ? 1.f / l1 : 0.f;
     auto store = [&](int r, int col, float a, float b) {
         if (r >= q_len) return;
-        if (p.gate) {
+        if (p.gate && p.gate_heads) {
+            const float f = 1.f / (1.f + __expf(-__bfloat162float(p.gate[(size_t)(q_start + r) * p.gate_row + head])));
+            a *= f;
+            b *= f;
+        } else if (p.gate) {
             const uint32_t g = *reinterpret_cast<const uint32_t*>(p.gate + (size_t)(q_start + r) * p.gate_row + head * D + col);
             a *= 1.f / (1.f + __expf(-bf16_lo(g)));
             b *= 1.f / (1.f + __expf(-bf16_hi(g)));

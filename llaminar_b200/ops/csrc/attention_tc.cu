@@ -63,6 +63,7 @@ LLM_DEVICE void stmatrix_x4(uint32_t addr, uint32_t r0, uint32_t r1, uint32_t r2
 
 enum Bar { K_FULL = 0, K_EMPTY = 2, VT_FULL = 4, VT_EMPTY = 6, S_FULL = 8, S_EMPTY = 10, P_FULL = 12, O_FULL = 13, O_EMPTY = 14, LD_SYNC = 15, PAIR = 16, N_BARS = 20 };
 
+template <bool CAP>                                // scores are soft-capped
 __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const AttnPrefillParams p, int* status) {
     extern __shared__ uint8_t smem_raw[];
     __shared__ __align__(8) uint64_t s_bars[N_BARS];
@@ -81,7 +82,7 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
     const int ctx = p.ctx_lens[seq];                       // tokens already in the cache before this chunk
     const int rows = min(BQ, q_len - q0);
     const int kv_end = ctx + q0 + rows;                    // keys this query tile can see
-    const int tile0 = p.window > 0 ? max(0, ctx + q0 + 1 - p.window) / BK : 0;          // tile of the first key that the first row sees
+    const int tile0 = first_key(ctx + q0, p.window, p.chunk) / BK;          // tile of the first key that the first row sees
     const int nt = (kv_end + BK - 1) / BK - tile0, n_pages = (kv_end + PAGE - 1) / PAGE;
     const int* btab = p.block_table + (size_t)seq * p.max_pages;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
@@ -113,9 +114,10 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
         const int row = tid & 127, half = tid >> 7, q4 = warp & 3;
         const bool valid = row < rows;
         const int lim = ctx + min(q0 + row, q_len - 1) + 1;           // this row sees keys < lim, and >= low
-        const int low = p.window > 0 ? lim - p.window : 0;
+        const int low = first_key(lim - 1, p.window, p.chunk);
         const uint32_t t_lane = tmem + ((uint32_t)(q4 * 32) << 16) + half * 64;
-        const float sl2 = p.scale * 1.4426950408889634f;
+        const ScoreScale score(p.scale, p.softcap);
+        const float sl2 = score.mul;
         constexpr int HD = D / 2;
         float o[HD];
 #pragma unroll
@@ -159,7 +161,8 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             s_xchg[half][row] = mx;
             if (!pair_meet()) return false;
             mx = fmaxf(mx, s_xchg[half ^ 1][row]);
-            m_new = fmaxf(m, mx * sl2);
+            if constexpr (CAP) m_new = mx == -INFINITY ? m : fmaxf(m, score.capped(mx));        // the cap keeps the order
+            else m_new = fmaxf(m, mx * sl2);
             mb = m_new == -INFINITY ? 0.f : m_new;
             alpha = ex2(m - mb);
             return true;
@@ -199,21 +202,27 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
             tmem_wait_ld(ra);
             tmem_wait_ld(rb);
             float sum = 0.f;
+            const float c2 = -2.f * score.cap, c1 = score.cap - mb;
+            auto prob = [&](uint32_t r) {
+                const float s = __uint_as_float(r) * sl2;
+                if constexpr (CAP) return ex2(fmaf(c2, __fdividef(1.f, 1.f + ex2(s)), c1));
+                else return ex2(s - mb);
+            };
             auto probs_of = [&](int c, const uint32_t (&r)[32]) {
                 uint32_t w[16];
                 if (need_mask) {
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
                         const int key = key0 + c * 32 + i;
-                        const float p0 = key >= lim || key < low ? 0.f : ex2(__uint_as_float(r[i]) * sl2 - mb);
-                        const float p1 = key + 1 >= lim || key + 1 < low ? 0.f : ex2(__uint_as_float(r[i + 1]) * sl2 - mb);
+                        const float p0 = key >= lim || key < low ? 0.f : prob(r[i]);
+                        const float p1 = key + 1 >= lim || key + 1 < low ? 0.f : prob(r[i + 1]);
                         sum += p0 + p1;
                         w[i >> 1] = pack_bf16(p0, p1);
                     }
                 } else {
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {
-                        const float p0 = ex2(__uint_as_float(r[i]) * sl2 - mb), p1 = ex2(__uint_as_float(r[i + 1]) * sl2 - mb);
+                        const float p0 = prob(r[i]), p1 = prob(r[i + 1]);
                         sum += p0 + p1;
                         w[i >> 1] = pack_bf16(p0, p1);
                     }
@@ -242,12 +251,13 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
         if (ok && valid) {
             float lt = l + s_xchg[half ^ 1][row];
             if (p.sink) lt += exp2f(p.sink[head] * 1.4426950408889634f - m);
-            const float inv = lt > 0.f ? 1.f / lt : 0.f;
+            float inv = lt > 0.f ? 1.f / lt : 0.f;
+            if (p.gate && p.gate_heads) inv *= __fdividef(1.f, 1.f + __expf(-__bfloat162float(p.gate[(size_t)(q_start + q0 + row) * p.gate_row + head])));
             __nv_bfloat16* dst = p.out + ((size_t)(q_start + q0 + row) * p.n_heads + head) * D + half * HD;
 #pragma unroll
             for (int u = 0; u < HD / 8; ++u) {
                 uint4 v;
-                if (p.gate) {
+                if (p.gate && !p.gate_heads) {
                     const uint4 g = *reinterpret_cast<const uint4*>(p.gate + (size_t)(q_start + q0 + row) * p.gate_row + head * D + half * HD + 8 * u);
                     const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
@@ -386,15 +396,18 @@ __global__ void __launch_bounds__(THREADS, 1) paged_attn_prefill_tc_kernel(const
 cudaError_t launch_attn_prefill_tc(const AttnPrefillParams& p, int n_seqs, int max_q_len, int* status, cudaStream_t st) {
     if (n_seqs == 0 || max_q_len == 0) return cudaSuccess;
     if (p.head_dim != atc::D || p.n_heads % p.n_kv_heads) return cudaErrorInvalidValue;
-    static bool once = false;
-    if (!once) {
-        cudaError_t e = cudaFuncSetAttribute(atc::paged_attn_prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, atc::SMEM_BYTES);
-        if (e != cudaSuccess) return e;
-        once = true;
-    }
-    dim3 grid((max_q_len + atc::BQ - 1) / atc::BQ, p.n_heads, n_seqs);
-    atc::paged_attn_prefill_tc_kernel<<<grid, atc::THREADS, atc::SMEM_BYTES, st>>>(p, status);
-    return cudaGetLastError();
+    const dim3 grid((max_q_len + atc::BQ - 1) / atc::BQ, p.n_heads, n_seqs);
+    auto go = [&](auto kernel, bool& once) -> cudaError_t {
+        if (!once) {
+            cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, atc::SMEM_BYTES);
+            if (e != cudaSuccess) return e;
+            once = true;
+        }
+        kernel<<<grid, atc::THREADS, atc::SMEM_BYTES, st>>>(p, status);
+        return cudaGetLastError();
+    };
+    static bool plain = false, capped = false;
+    return p.softcap > 0.f ? go(atc::paged_attn_prefill_tc_kernel<true>, capped) : go(atc::paged_attn_prefill_tc_kernel<false>, plain);
 }
 
 LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_attention_tc)

@@ -94,6 +94,26 @@ LLM_DEVICE void pdl_wait() { asm volatile("griddepcontrol.wait;" ::: "memory"); 
 
 LLM_DEVICE uint32_t smem_u32(const void* p) { return static_cast<uint32_t>(__cvta_generic_to_shared(p)); }
 
+// position of the first key that a query at `pos` sees: a window of that many keys, itself included, and chunks of that many
+// positions (0: none)
+LLM_DEVICE int first_key(int pos, int window, int chunk) {
+    const int lo = window > 0 ? max(0, pos - window + 1) : 0;
+    return chunk > 0 ? max(lo, pos - pos % chunk) : lo;
+}
+
+// Attention scores in units of ln 2, as exp2 takes them: raw * scale, or soft-capped.  cap tanh(x / cap) is written
+// cap (1 - 2 / (1 + e^(2x / cap))); both ends of the quotient are right in the limit.
+struct ScoreScale {
+    float mul, cap;                 // cap > 0: capped
+    LLM_DEVICE ScoreScale(float scale, float softcap) {
+        cap = softcap * 1.4426950408889634f;
+        mul = (softcap > 0.f ? 2.f * scale / softcap : scale) * 1.4426950408889634f;
+    }
+    LLM_DEVICE float linear(float s) const { return s * mul; }
+    LLM_DEVICE float capped(float s) const { return fmaf(-2.f * cap, __fdividef(1.f, 1.f + exp2f(s * mul)), cap); }
+    LLM_DEVICE float operator()(float s) const { return cap > 0.f ? capped(s) : linear(s); }
+};
+
 // branch-free: the approximate division has no slow path for huge or infinite denominators (they give 0, the right limit)
 LLM_DEVICE float silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 

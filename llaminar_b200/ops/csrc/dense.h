@@ -8,13 +8,15 @@
 
 namespace llm {
 
-// v = y[row(t)], or half the sum of RMSNorm(y[t]) * w_y and RMSNorm(y2[t]) * w_y2
+// v = y[row(t)], or the sum of y[row(t, j)] * y_w[t, j] over j < n_parts, or half the sum of RMSNorm(y[t]) * w_y and RMSNorm(y2[t]) * w_y2
 // h[t] = (add ? h[t] : 0) + (norm of v) * w_post, or v * factor ; xn[t] = (norm of h[t]) * w_next ; copies of h[t] in the activation type
 struct ResidNormParams {
     const void* y;                 // activation type; nullptr: h is only read
     size_t y_stride;
-    const int* y_rows;             // optional gather (embedding lookup): row(t) = y_rows[t]
+    const int* y_rows;             // optional gather (embedding lookup, sorted experts): row(t) = y_rows[t], row(t, j) = y_rows[t * n_parts + j]
     int n_y_rows;                  // rows of y (bounds-check build)
+    const float* y_w;              // with n_parts > 0: weights of the parts (chosen experts)
+    int n_parts;
     const void* y2;                // optional second sublayer output [T, d]
     size_t y2_stride;
     const float *w_y, *w_y2;       // [d], with y2
@@ -32,17 +34,20 @@ struct ResidNormParams {
 };
 cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cudaStream_t st);
 
-// Activations behind a product.  GELU_MUL: gelu_tanh(first half of the columns) * second half; RELU2: squared relu;
-// GELU_SIDE: gelu_tanh times the token's row of a table (columns [0, side_cols), zero behind).
-enum Activation : int { ACT_NONE = 0, ACT_GELU_MUL = 1, ACT_RELU2 = 2, ACT_GELU_SIDE = 3 };
+// Activations behind a product.  GELU_MUL: gelu_tanh(first half of the columns) * second half, SILU_MUL the same with silu; RELU2: squared
+// relu; GELU_SIDE: gelu_tanh times the token's row of a table (columns [0, side_cols), zero behind); GATE: times the sigmoid of the row's
+// own row of the table (tokens unused).
+enum Activation : int { ACT_NONE = 0, ACT_GELU_MUL = 1, ACT_RELU2 = 2, ACT_GELU_SIDE = 3, ACT_SILU_MUL = 4, ACT_GATE = 5 };
+constexpr bool act_pairs(int act) { return act == ACT_GELU_MUL || act == ACT_SILU_MUL; }
 struct SideTable { const void* table; size_t row; int cols, n_rows; const int* tokens; };
-// act[t, 0..n) from x[t, 0..n) (GELU_MUL: 2n columns)
+// act[t, 0..n) from x[t, 0..n) (GELU_MUL, SILU_MUL: 2n columns)
 cudaError_t launch_activate(const void* x, void* act, int rows, int n, int kind, const SideTable& side, bool f32, cudaStream_t st);
 
 // out[t, i] = magnitude * (cos, sin)(positions[t] * freqs[i])
 cudaError_t launch_rope_angles(const int* positions, const double* freqs, double magnitude, float2* out, int rows, int half, cudaStream_t st);
 
-// out[z][m, :] = act(x[z][m, :] W[z]^T) for up to 8 rows, bf16 weights.  GELU_MUL: W holds 2n rows.
+// out[z][m, :] = act(x[z][m, :] W[z]^T) for up to 8 rows, bf16 weights.  GELU_MUL, SILU_MUL: W holds 2n rows.  GATE: the table's row m
+// holds the gates of all z, n columns each.
 struct GemvDenseParams {
     const __nv_bfloat16* w; size_t w_z; int ldw;
     const __nv_bfloat16* x; size_t x_row, x_z;

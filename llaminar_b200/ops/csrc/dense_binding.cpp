@@ -9,7 +9,7 @@ using namespace llm_binding;
 
 void resid_norm(const OptTensor& y, const OptTensor& y_rows, const OptTensor& w_post, const Tensor& h, bool add, const OptTensor& w_next,
                 const OptTensor& xn, const OptTensor& copy0, const OptTensor& copy1, double eps, const OptTensor& y2, const OptTensor& w_y,
-                const OptTensor& w_y2, double factor, bool center_post, bool center_next) {
+                const OptTensor& w_y2, double factor, bool center_post, bool center_next, const OptTensor& y_w) {
     llm::ResidNormParams p = {};
     want(h, torch::kFloat32, "h");
     const int64_t T = h.size(0), d = h.size(1);
@@ -26,11 +26,17 @@ void resid_norm(const OptTensor& y, const OptTensor& y_rows, const OptTensor& w_
         p.y = y->data_ptr(); p.y_stride = y->stride(0);
         if (w_post) p.w_post = floats(*w_post, d, "w_post");
         p.n_y_rows = y->size(0);
+        int64_t parts = 1;
+        if (y_w) {
+            TORCH_CHECK(y_w->dim() == 2 && y_w->size(0) == T && y_w->size(1) >= 1 && !y2, "y_w must be [tokens, parts]");
+            parts = y_w->size(1);
+            p.y_w = floats(*y_w, T * parts, "y_w"); p.n_parts = parts;
+        }
         if (y_rows) {
             p.y_rows = ints(*y_rows, "y_rows");
-            TORCH_CHECK(y_rows->numel() == T, "y_rows must name one row per token");
+            TORCH_CHECK(y_rows->numel() == T * parts, "y_rows must name one row per token and part");
         } else {
-            TORCH_CHECK(y->size(0) == T, "y must have as many rows as h");
+            TORCH_CHECK(y->size(0) == T * parts, "y must have a row per token and part");
         }
         if (y2) {
             elem(*y2, "y2");
@@ -61,18 +67,25 @@ llm::SideTable side_table(const OptTensor& table, int64_t first, int64_t cols, c
     if (!table) return s;
     want_like(*table, f32, "side table");
     TORCH_CHECK(table->dim() == 2 && table->stride(1) == 1 && first >= 0 && first + cols <= table->size(1), "side table columns");
-    TORCH_CHECK(tokens && tokens->numel() == rows, "one token per row");
+    TORCH_CHECK(tokens ? tokens->numel() == rows : table->size(0) == rows, "one token per row");
     s.table = static_cast<const char*>(table->data_ptr()) + first * table->element_size();
-    s.row = table->stride(0); s.cols = cols; s.n_rows = table->size(0); s.tokens = ints(*tokens, "tokens");
+    s.row = table->stride(0); s.cols = cols; s.n_rows = table->size(0);
+    if (tokens) s.tokens = ints(*tokens, "tokens");
     return s;
+}
+
+// the table of a side input names its rows by token, the one of a gate has the output's rows and columns
+void want_table(int64_t act, const OptTensor& table, int64_t cols, const OptTensor& tokens, int64_t n) {
+    TORCH_CHECK((act == llm::ACT_GELU_SIDE || act == llm::ACT_GATE) == table.has_value(), "a table goes with the side activation and the gate");
+    TORCH_CHECK((act == llm::ACT_GELU_SIDE) == tokens.has_value() && (act != llm::ACT_GATE || cols == n), "tokens / gate columns");
 }
 
 void activate(const Tensor& x, const Tensor& act, int64_t kind, const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens) {
     const bool f32 = is_f32(x, "x");
     want_like(act, f32, "act");
     TORCH_CHECK(x.is_contiguous() && act.is_contiguous() && x.size(0) == act.size(0), "activation rows");
-    TORCH_CHECK(x.size(1) == act.size(1) * (kind == llm::ACT_GELU_MUL ? 2 : 1), "activation columns");
-    TORCH_CHECK((kind == llm::ACT_GELU_SIDE) == table.has_value(), "a side table goes with the side activation");
+    TORCH_CHECK(x.size(1) == act.size(1) * (llm::act_pairs(kind) ? 2 : 1), "activation columns");
+    want_table(kind, table, cols, tokens, act.size(1));
     if (x.size(0) == 0) return;
     check(llm::launch_activate(x.data_ptr(), act.data_ptr(), x.size(0), act.size(1), kind, side_table(table, first, cols, tokens, x.size(0), f32), f32, stream()), "activate");
 }
@@ -86,20 +99,20 @@ void rope_angles(const Tensor& positions, const Tensor& freqs, double magnitude,
                                   rows, half, stream()), "rope_angles");
 }
 
-// w [z, n, k] (GELU_MUL: [z, 2n, k]), x [z, m, k], out [z, m, n]; the last dimension of each is dense
+// w [z, n, k] (GELU_MUL, SILU_MUL: [z, 2n, k]), x [z, m, k], out [z, m, n]; the last dimension of each is dense
 void gemv_dense(const Tensor& w, const Tensor& x, const Tensor& out, int64_t act, const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens) {
     TORCH_CHECK(w.is_cuda() && w.scalar_type() == torch::kBFloat16 && x.scalar_type() == torch::kBFloat16, "gemv_dense takes bf16 operands");
     TORCH_CHECK(w.dim() == 3 && x.dim() == 3 && out.dim() == 3 && w.stride(2) == 1 && x.stride(2) == 1 && out.stride(2) == 1, "gemv_dense layouts");
     llm::GemvDenseParams p = {};
-    p.z = w.size(0); p.n = act == llm::ACT_GELU_MUL ? w.size(1) / 2 : w.size(1); p.k = w.size(2); p.m = x.size(1);
+    p.z = w.size(0); p.n = llm::act_pairs(act) ? w.size(1) / 2 : w.size(1); p.k = w.size(2); p.m = x.size(1);
     TORCH_CHECK(x.size(0) == p.z && out.size(0) == p.z && x.size(2) == p.k && out.size(1) == p.m && out.size(2) == p.n, "gemv_dense shapes");
     p.out_f32 = is_f32(out, "out"); p.act = act;
     p.w = reinterpret_cast<const __nv_bfloat16*>(w.data_ptr()); p.w_z = w.stride(0); p.ldw = w.stride(1);
     p.x = reinterpret_cast<const __nv_bfloat16*>(x.data_ptr()); p.x_row = x.stride(1); p.x_z = x.stride(0);
     p.out = out.data_ptr(); p.o_row = out.stride(1); p.o_z = out.stride(0);
     TORCH_CHECK(reinterpret_cast<uintptr_t>(w.data_ptr()) % 16 == 0 && reinterpret_cast<uintptr_t>(x.data_ptr()) % 16 == 0, "gemv_dense operands must be 16-byte aligned");
-    TORCH_CHECK((act == llm::ACT_GELU_SIDE) == table.has_value(), "a side table goes with the side activation");
-    p.side = side_table(table, first, cols, tokens, (int64_t)p.z * p.m, false);
+    want_table(act, table, cols, tokens, (int64_t)p.z * p.n);
+    p.side = side_table(table, first, cols, tokens, act == llm::ACT_GATE ? p.m : (int64_t)p.z * p.m, false);
     check(llm::launch_gemv_dense(p, stream()), "gemv_dense");
 }
 

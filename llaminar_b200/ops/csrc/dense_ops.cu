@@ -18,6 +18,8 @@ LLM_DEVICE float gelu_tanh(float z) {
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
+LLM_DEVICE float logistic(float x) { return 1.f / (1.f + expf(-x)); }
+
 template <int THREADS>
 LLM_DEVICE float block_sum(float v, float* red) {
     v = warp_sum(v);
@@ -86,14 +88,24 @@ __global__ void __launch_bounds__(THREADS) resid_norm_kernel(const ResidNormPara
     };
     float inv_y = 0.f, mean_y = 0.f;
     const T* y = nullptr;
+    auto y_row = [&](size_t i) { return static_cast<const T*>(p.y) + (p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[i], p.n_y_rows) : i) * p.y_stride; };
     if (p.y) {
-        const size_t r = p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[t], p.n_y_rows) : t;
-        y = static_cast<const T*>(p.y) + r * p.y_stride;
+        y = y_row(p.n_parts ? t * p.n_parts : t);
         const T* y2 = p.y2 ? static_cast<const T*>(p.y2) + t * p.y2_stride : nullptr;
         float ss = 0.f, ss2 = 0.f, sum = 0.f;
         for (int i = threadIdx.x * VEC; i < p.d; i += THREADS * VEC) {
             float v[VEC];
             load_t(y + i, v);
+            if (p.n_parts) {
+                float u[VEC];
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) v[j] *= p.y_w[t * p.n_parts];
+                for (int q = 1; q < p.n_parts; ++q) {
+                    load_t(y_row(t * p.n_parts + q) + i, u);
+#pragma unroll
+                    for (int j = 0; j < VEC; ++j) v[j] = fmaf(u[j], p.y_w[t * p.n_parts + q], v[j]);
+                }
+            }
 #pragma unroll
             for (int j = 0; j < VEC; ++j) { ss += v[j] * v[j]; sum += v[j]; }
             store_f(row + i, v);
@@ -210,9 +222,24 @@ __global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNorm
     pdl_wait();
     if (!p.y || p.add) each([&](int n, int i) { Vec4<float>::load(h + i, a[n]); });
     if (p.y) {
-        const size_t r = p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[t], p.n_y_rows) : t;
-        const T* y = static_cast<const T*>(p.y) + r * p.y_stride;
-        each([&](int n, int i) { Vec4<T>::load(y + i, v[n]); });
+        auto y_row = [&](size_t i) { return static_cast<const T*>(p.y) + (p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[i], p.n_y_rows) : i) * p.y_stride; };
+        if (p.n_parts) {
+            each([&](int n, int) { v[n][0] = v[n][1] = v[n][2] = v[n][3] = 0.f; });
+#pragma unroll 4
+            for (int q = 0; q < p.n_parts; ++q) {
+                const T* y = y_row(t * p.n_parts + q);
+                const float w = p.y_w[t * p.n_parts + q];
+                each([&](int n, int i) {
+                    float u[4];
+                    Vec4<T>::load(y + i, u);
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) v[n][j] = fmaf(u[j], w, v[n][j]);
+                });
+            }
+        } else {
+            const T* y = y_row(t);
+            each([&](int n, int i) { Vec4<T>::load(y + i, v[n]); });
+        }
         if (p.y2) {
             const T* y2 = static_cast<const T*>(p.y2) + t * p.y2_stride;
             float u[NV][4], sa = 0.f, sb = 0.f;
@@ -259,10 +286,12 @@ __global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNorm
     });
 }
 
-// value `i` of row `t` of the activation of `x`; `u`: the second half's value (GELU_MUL)
+// value `i` of row `t` of the activation of `x`; `u`: the second half's value (GELU_MUL, SILU_MUL)
 template <int ACT, class T>
 LLM_DEVICE float activated(float x, float u, const SideTable& s, int t, int i) {
     if (ACT == ACT_GELU_MUL) return gelu_tanh(x) * u;
+    if (ACT == ACT_SILU_MUL) return x * logistic(x) * u;
+    if (ACT == ACT_GATE) return x * logistic(to_f(static_cast<const T*>(s.table)[(size_t)t * s.row + i]));
     if (ACT == ACT_RELU2) { x = fmaxf(x, 0.f); return x * x; }
     if (ACT == ACT_GELU_SIDE) return i < s.cols ? gelu_tanh(x) * to_f(static_cast<const T*>(s.table)[(size_t)LLM_CHECK_INDEX(s.tokens[t], s.n_rows) * s.row + i]) : 0.f;
     return x;
@@ -272,20 +301,20 @@ template <class T, int ACT>
 __global__ void __launch_bounds__(256) activate_kernel(const T* x, T* act, int n, const SideTable s) {
     pdl_trigger();
     pdl_wait();
-    const T* g = x + (size_t)blockIdx.y * n * (ACT == ACT_GELU_MUL ? 2 : 1);
+    const T* g = x + (size_t)blockIdx.y * n * (act_pairs(ACT) ? 2 : 1);
     T* a = act + (size_t)blockIdx.y * n;
     const int i0 = (blockIdx.x * 256 + threadIdx.x) * 4;
     if (n % 4 == 0) {
         if (i0 >= n) return;
         float v[4], u[4] = {};
         Vec4<T>::load(g + i0, v);
-        if (ACT == ACT_GELU_MUL) Vec4<T>::load(g + n + i0, u);
+        if (act_pairs(ACT)) Vec4<T>::load(g + n + i0, u);
 #pragma unroll
         for (int j = 0; j < 4; ++j) v[j] = activated<ACT, T>(v[j], u[j], s, blockIdx.y, i0 + j);
         Vec4<T>::store(a + i0, v);
     } else {
         for (int i = i0; i < min(n, i0 + 4); ++i)
-            a[i] = from_f<T>(activated<ACT, T>(to_f(g[i]), ACT == ACT_GELU_MUL ? to_f(g[n + i]) : 0.f, s, blockIdx.y, i));
+            a[i] = from_f<T>(activated<ACT, T>(to_f(g[i]), act_pairs(ACT) ? to_f(g[n + i]) : 0.f, s, blockIdx.y, i));
     }
 }
 
@@ -303,7 +332,7 @@ __global__ void rope_angles_kernel(const int* positions, const double* freqs, do
 // Up to eight rows of x against 16 weight rows per warp on the tensor cores (the weights are the M operand).  Thread (g, t) of
 // a warp loads 8 consecutive k of weight rows g and g + 8 and of x row g in one 16-byte access each; since both operands use
 // the same assignment of k to MMA slots, its order does not matter and no operand passes through shared memory.  `wk` warps
-// share the K range of a row block and add up in shared memory.  GELU_MUL: a second set of weight rows (n further down) per block.
+// share the K range of a row block and add up in shared memory.  GELU_MUL, SILU_MUL: a second set of weight rows (n further down) per block.
 constexpr int SKINNY_WARPS = 8;
 LLM_DEVICE void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -311,15 +340,15 @@ LLM_DEVICE void mma_bf16(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, u
 }
 template <int ACT, class TO>
 __global__ void __launch_bounds__(32 * SKINNY_WARPS) gemv_dense_kernel(const GemvDenseParams p, int wk) {
-    constexpr bool GELU = ACT == ACT_GELU_MUL;
-    __shared__ float s_acc[SKINNY_WARPS][GELU ? 2 : 1][16][9];
+    constexpr bool PAIR = act_pairs(ACT);
+    __shared__ float s_acc[SKINNY_WARPS][PAIR ? 2 : 1][16][9];
     pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, g = lane >> 2, t = lane & 3;
     const int part = warp % wk, n0 = (blockIdx.x * (SKINNY_WARPS / wk) + warp / wk) * 16;
     const int blocks = (p.k + 31) / 32, per = (blocks + wk - 1) / wk, kb0 = part * per, kb1 = min(blocks, kb0 + per);
-    constexpr int UN = GELU ? 4 : 8, NW = GELU ? 4 : 2;
+    constexpr int UN = PAIR ? 4 : 8, NW = PAIR ? 4 : 2;
     const uint4 zero = make_uint4(0, 0, 0, 0);
-    float acc[GELU ? 2 : 1][4] = {};
+    float acc[PAIR ? 2 : 1][4] = {};
     // rows past the end repeat the last one (never stored)
     const __nv_bfloat16* w[NW];
 #pragma unroll
@@ -365,11 +394,12 @@ __global__ void __launch_bounds__(32 * SKINNY_WARPS) gemv_dense_kernel(const Gem
         float v = 0.f, v2 = 0.f;
         for (int q = 0; q < wk; ++q) {
             v += s_acc[(c / 16) * wk + q][0][c % 16][m];
-            if constexpr (GELU) v2 += s_acc[(c / 16) * wk + q][1][c % 16][m];
+            if constexpr (PAIR) v2 += s_acc[(c / 16) * wk + q][1][c % 16][m];
         }
         // rounded like the stored projection of the unfused form
         if constexpr (ACT != ACT_NONE)
-            v = activated<ACT, __nv_bfloat16>(__bfloat162float(__float2bfloat16(v)), __bfloat162float(__float2bfloat16(v2)), p.side, blockIdx.y * p.m + m, n);
+            v = activated<ACT, __nv_bfloat16>(__bfloat162float(__float2bfloat16(v)), __bfloat162float(__float2bfloat16(v2)), p.side,
+                                              ACT == ACT_GATE ? m : blockIdx.y * p.m + m, ACT == ACT_GATE ? blockIdx.y * p.n + n : n);
         static_cast<TO*>(p.out)[(size_t)blockIdx.y * p.o_z + m * p.o_row + n] = from_f<TO>(v);
     }
 }
@@ -411,6 +441,8 @@ cudaError_t launch_activate(const void* x, void* act, int rows, int n, int kind,
         return launch_pdl(k16, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(act), n, side);
     };
     if (kind == ACT_GELU_MUL) return go(activate_kernel<float, ACT_GELU_MUL>, activate_kernel<__nv_bfloat16, ACT_GELU_MUL>);
+    if (kind == ACT_SILU_MUL) return go(activate_kernel<float, ACT_SILU_MUL>, activate_kernel<__nv_bfloat16, ACT_SILU_MUL>);
+    if (kind == ACT_GATE) return go(activate_kernel<float, ACT_GATE>, activate_kernel<__nv_bfloat16, ACT_GATE>);
     if (kind == ACT_RELU2) return go(activate_kernel<float, ACT_RELU2>, activate_kernel<__nv_bfloat16, ACT_RELU2>);
     if (kind == ACT_GELU_SIDE) return go(activate_kernel<float, ACT_GELU_SIDE>, activate_kernel<__nv_bfloat16, ACT_GELU_SIDE>);
     return cudaErrorInvalidValue;
@@ -432,6 +464,8 @@ cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st) {
     const dim3 grid((p.n + cols - 1) / cols, p.z);
     auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(32 * SKINNY_WARPS), 0, st, p, wk); };
     if (p.act == ACT_GELU_MUL) return go(gemv_dense_kernel<ACT_GELU_MUL, __nv_bfloat16>);
+    if (p.act == ACT_SILU_MUL) return go(gemv_dense_kernel<ACT_SILU_MUL, __nv_bfloat16>);
+    if (p.act == ACT_GATE) return go(gemv_dense_kernel<ACT_GATE, __nv_bfloat16>);
     if (p.act == ACT_RELU2) return go(gemv_dense_kernel<ACT_RELU2, __nv_bfloat16>);
     if (p.act == ACT_GELU_SIDE) return go(gemv_dense_kernel<ACT_GELU_SIDE, __nv_bfloat16>);
     return p.out_f32 ? go(gemv_dense_kernel<ACT_NONE, float>) : go(gemv_dense_kernel<ACT_NONE, __nv_bfloat16>);

@@ -1,0 +1,226 @@
+// Around grouped-query attention: the row-wise kernels.
+//
+//   attn_prep      norms of the queries and keys over all heads together, append to the paged cache
+//   head_prep      norms of queries and keys per head, rotation, append to the paged cache
+//   attn_plain     one row and head per CTA in float arithmetic
+#include "common.cuh"
+#include "grouped.h"
+#include "launch.h"
+
+namespace llm {
+
+namespace {
+
+constexpr int PAGE = 64;
+
+LLM_DEVICE float to_f(float v) { return v; }
+LLM_DEVICE float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
+template <class T> LLM_DEVICE T from_f(float v);
+template <> LLM_DEVICE float from_f<float>(float v) { return v; }
+template <> LLM_DEVICE __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
+LLM_DEVICE void load4(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+LLM_DEVICE void load4(const __nv_bfloat16* p, float (&v)[4]) {
+    const uint2 a = *reinterpret_cast<const uint2*>(p);
+    v[0] = bf16_lo(a.x); v[1] = bf16_hi(a.x); v[2] = bf16_lo(a.y); v[3] = bf16_hi(a.y);
+}
+LLM_DEVICE void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+LLM_DEVICE void store4(__nv_bfloat16* p, const float (&v)[4]) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3])); }
+
+template <int THREADS>
+LLM_DEVICE float block_sum(float v, float* red) {
+    v = warp_sum(v);
+    __syncthreads();                               // red may still be read from the sum before
+    if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+    __syncthreads();
+    float s = 0.f;
+#pragma unroll
+    for (int i = 0; i < THREADS / 32; ++i) s += red[i];
+    return s;
+}
+
+template <class TI, class T>
+__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrepParams p) {
+    __shared__ float red[8];
+    pdl_trigger();
+    pdl_wait();
+    const int t = blockIdx.x;
+    const TI* row = static_cast<const TI*>(p.in) + (size_t)t * p.in_row;
+    const TI *q = row + p.q_off, *k = row + p.k_off, *v = row + p.v_off;
+    const int nq = p.n_heads * p.dim, nk = p.n_kv_heads * p.dim;
+    const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
+    const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
+    float sq = 0.f, sk = 0.f, x[4], w[4];
+    for (int i = threadIdx.x * 4; i < nq; i += 1024) {
+        load4(q + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sq += x[j] * x[j];
+    }
+    for (int i = threadIdx.x * 4; i < nk; i += 1024) {
+        load4(k + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) sk += x[j] * x[j];
+    }
+    const float iq = 1.f / sqrtf(block_sum<256>(sq, red) / (float)(p.n_heads * p.true_dim) + p.eps);
+    const float ik = 1.f / sqrtf(block_sum<256>(sk, red) / (float)(p.n_kv_heads * p.true_dim) + p.eps);
+    T* qo = static_cast<T*>(p.q_out) + (size_t)t * nq;
+    for (int i = threadIdx.x * 4; i < nq; i += 1024) {
+        load4(q + i, x); load4(p.q_norm + i, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] *= iq * w[j];
+        store4(qo + i, x);
+    }
+    for (int i = threadIdx.x * 4; i < nk; i += 1024) {
+        const int g = i / p.dim, c = i - g * p.dim;
+        T* dst = static_cast<T*>(p.kv) + (((size_t)page * 2 * p.n_kv_heads + g) * PAGE + pos % PAGE) * p.dim + c;
+        load4(k + i, x); load4(p.k_norm + i, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] *= ik * w[j];
+        store4(dst, x);
+        load4(v + i, x);
+        store4(dst + (size_t)p.n_kv_heads * PAGE * p.dim, x);
+    }
+}
+
+// a warp per token and head: norm, rotation, and the append of keys and values
+template <class TI, class T>
+__global__ void __launch_bounds__(256) head_prep_kernel(const HeadPrepParams p) {
+    extern __shared__ __align__(16) float sm[];                // [8][dim]
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x, D = p.dim, H = p.n_heads, G = p.n_kv_heads;
+    const int u = blockIdx.y * 8 + warp;                       // queries, then keys, then values
+    if (u >= H + 2 * G) return;
+    const int kind = u < H ? 0 : u < H + G ? 1 : 2, h = u - (kind == 0 ? 0 : kind == 1 ? H : H + G);
+    T* dst = static_cast<T*>(p.q_out) + ((size_t)t * H + h) * D;
+    if (kind) {
+        const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
+        const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
+        dst = static_cast<T*>(p.kv) + ((((size_t)page * 2 + kind - 1) * G + h) * PAGE + pos % PAGE) * D;
+    }
+    pdl_wait();
+    const TI* src = static_cast<const TI*>(p.in) + (size_t)t * p.in_row + (kind == 0 ? p.q_off : kind == 1 ? p.k_off : p.v_off) + (size_t)h * D;
+    float x[4], w[4];
+    if (kind == 2) {
+        for (int i = lane * 4; i < D; i += 128) { load4(src + i, x); store4(dst + i, x); }
+        return;
+    }
+    float* row = sm + warp * D;
+    const float* gain = kind ? p.k_norm : p.q_norm;
+    float ss = 0.f;
+    for (int i = lane * 4; i < D; i += 128) {
+        load4(src + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss += x[j] * x[j];
+        store4(row + i, x);
+    }
+    const float inv = 1.f / sqrtf(warp_sum(ss) / (float)p.true_dim + p.eps);
+    for (int i = lane * 4; i < D; i += 128) {                  // every lane reads back what it wrote
+        load4(row + i, x); load4(gain + i, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) x[j] *= inv * w[j];
+        store4(row + i, x);
+    }
+    __syncwarp();
+    const float2* ang = p.angles + (size_t)t * p.half;
+    for (int i = lane * 4; i < D; i += 128) {
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int c = i + j;
+            x[j] = row[c];
+            if (c < p.half) x[j] = x[j] * ang[c].x - row[c + p.half] * ang[c].y;
+            else if (c < 2 * p.half) x[j] = x[j] * ang[c - p.half].x + row[c - p.half] * ang[c - p.half].y;
+        }
+        store4(dst + i, x);
+    }
+}
+
+template <class TG, class T>
+__global__ void __launch_bounds__(128) attn_plain_kernel(const AttnPlainParams p) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float s_score[64];
+    pdl_trigger();
+    pdl_wait();
+    const int h = blockIdx.x, t = blockIdx.y, D = p.dim, g = h / (p.n_heads / p.n_kv_heads);
+    float *sq = sm, *so = sm + D;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int pos = p.positions[t];
+    const int* btab = p.block_table + (size_t)LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs) * p.max_pages;
+    const T* q = static_cast<const T*>(p.q) + ((size_t)t * p.n_heads + h) * D;
+    for (int i = threadIdx.x; i < D; i += 128) { sq[i] = to_f(q[i]); so[i] = 0.f; }
+    __syncthreads();
+    auto key_row = [&](int key, int which) {
+        const int page = LLM_CHECK_INDEX(btab[key / PAGE], p.n_pages);
+        return static_cast<const T*>(p.kv) + ((((size_t)page * 2 + which) * p.n_kv_heads + g) * PAGE + key % PAGE) * D;
+    };
+    float m = p.sink ? p.sink[h] : -INFINITY, l = p.sink ? 1.f : 0.f;
+    for (int k0 = first_key(pos, p.window, p.chunk); k0 <= pos; k0 += 64) {
+        const int n = min(64, pos + 1 - k0);
+        for (int j = warp; j < n; j += 4) {
+            const T* row = key_row(k0 + j, 0);
+            float s = 0.f;
+            for (int i = lane; i < D; i += 32) s = fmaf(sq[i], to_f(row[i]), s);
+            s = warp_sum(s);
+            s *= p.scale;
+            if (lane == 0) s_score[j] = p.softcap > 0.f ? p.softcap * tanhf(s / p.softcap) : s;
+        }
+        __syncthreads();
+        float nm = m;
+        for (int j = 0; j < n; ++j) nm = fmaxf(nm, s_score[j]);
+        const float c = expf(m - nm);
+        __syncthreads();
+        if ((int)threadIdx.x < n) s_score[threadIdx.x] = expf(s_score[threadIdx.x] - nm);
+        __syncthreads();
+        float ps = 0.f;
+        for (int j = 0; j < n; ++j) ps += s_score[j];
+        l = l * c + ps;
+        m = nm;
+        for (int i = threadIdx.x; i < D; i += 128) {
+            float a = so[i] * c;
+            for (int j = 0; j < n; ++j) a = fmaf(s_score[j], to_f(key_row(k0 + j, 1)[i]), a);
+            so[i] = a;
+        }
+        __syncthreads();
+    }
+    T* o = static_cast<T*>(p.out) + ((size_t)t * p.n_heads + h) * D;
+    for (int i = threadIdx.x; i < D; i += 128) {
+        float v = so[i] / l;
+        if (p.gate) v *= 1.f / (1.f + expf(-to_f(static_cast<const TG*>(p.gate)[(size_t)t * p.gate_row + (p.gate_heads ? (size_t)h : (size_t)h * D + i)])));
+        o[i] = from_f<T>(v);
+    }
+}
+
+}  // namespace
+
+cudaError_t launch_head_prep(const HeadPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    const size_t smem = (size_t)8 * p.dim * 4;
+    if (p.dim % 8 || p.in_row % 4 || p.q_off % 4 || p.k_off % 4 || p.v_off % 4 || 2 * p.half > p.dim || smem > 48 * 1024 || (f32 && !in_f32)) return cudaErrorInvalidValue;
+    const dim3 grid(rows, (p.n_heads + 2 * p.n_kv_heads + 7) / 8);
+    auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(256), smem, st, p); };
+    if (f32) return go(head_prep_kernel<float, float>);
+    return in_f32 ? go(head_prep_kernel<float, __nv_bfloat16>) : go(head_prep_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
+
+cudaError_t launch_attn_prep(const AttnPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    if (p.dim % 8 || p.in_row % 4 || p.q_off % 4 || p.k_off % 4 || p.v_off % 4 || (f32 && !in_f32)) return cudaErrorInvalidValue;
+    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(256), 0, st, p); };
+    if (f32) return go(attn_prep_kernel<float, float>);
+    return in_f32 ? go(attn_prep_kernel<float, __nv_bfloat16>) : go(attn_prep_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
+
+cudaError_t launch_attn_plain(const AttnPlainParams& p, int rows, bool gate_f32, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    const size_t smem = (size_t)p.dim * 8;
+    if (rows > 65535 || smem > 48 * 1024 || p.n_heads % p.n_kv_heads) return cudaErrorInvalidValue;
+    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(p.n_heads, rows), dim3(128), smem, st, p); };
+    if (f32) return gate_f32 ? go(attn_plain_kernel<float, float>) : go(attn_plain_kernel<__nv_bfloat16, float>);
+    return gate_f32 ? go(attn_plain_kernel<float, __nv_bfloat16>) : go(attn_plain_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
+
+LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_grouped)
+
+}  // namespace llm

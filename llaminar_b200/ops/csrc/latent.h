@@ -66,6 +66,7 @@ struct LatentChunkParams {
     int dim, rot, vdim, n_heads, window;               // padded to multiples of 8
     float scale;
     const float* sink;
+    const __nv_bfloat16* gate; size_t gate_row;        // optional [token][head * vdim]: the result times its sigmoid (rows of whole 16-byte units)
 };
 cudaError_t launch_latent_chunk(const LatentChunkParams& p, int n_seqs, int max_q_len, cudaStream_t st);
 bool latent_chunk_has_kernel(int dk, int dv);

@@ -593,9 +593,18 @@ __global__ void __launch_bounds__(256) latent_chunk_kernel(const LatentChunkPara
     for (int n = 0; n < DV / 8; ++n) {
         const int col = n * 8 + (lane & 3) * 2;
         if (col >= p.vdim) continue;
-        __nv_bfloat16* out = p.out + (size_t)(sq.q_start + qt0) * p.out_row + (size_t)head * p.vdim + col;
-        if (i0 < n_rows) *reinterpret_cast<uint32_t*>(out + (size_t)i0 * p.out_row) = pack_bf16(o[n][0] * v0, o[n][1] * v0);
-        if (i1 < n_rows) *reinterpret_cast<uint32_t*>(out + (size_t)i1 * p.out_row) = pack_bf16(o[n][2] * v1, o[n][3] * v1);
+        auto store = [&](int i, float a, float b) {
+            if (i >= n_rows) return;
+            const size_t t = (size_t)sq.q_start + qt0 + i;
+            if (p.gate) {
+                const uint32_t g = *reinterpret_cast<const uint32_t*>(p.gate + t * p.gate_row + (size_t)head * p.vdim + col);
+                a *= 1.f / (1.f + __expf(-bf16_lo(g)));
+                b *= 1.f / (1.f + __expf(-bf16_hi(g)));
+            }
+            *reinterpret_cast<uint32_t*>(p.out + t * p.out_row + (size_t)head * p.vdim + col) = pack_bf16(a, b);
+        };
+        store(i0, o[n][0] * v0, o[n][1] * v0);
+        store(i1, o[n][2] * v1, o[n][3] * v1);
     }
 }
 

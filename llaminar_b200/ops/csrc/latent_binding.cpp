@@ -95,7 +95,7 @@ void latent_gather(const Tensor& kv, const Tensor& seqs, int64_t max_k_len, cons
 // k [keys, heads * dim]; v [keys, heads * vdim], or with status (the tcgen05 form) [heads * vdim, keys]
 void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& k, const Tensor& v, const Tensor& lat, int64_t rot_off, const Tensor& seqs,
                   int64_t max_q_len, const Tensor& out, int64_t dim, int64_t rot, int64_t vdim, int64_t window, double scale, const OptTensor& sink,
-                  const OptTensor& status) {
+                  const OptTensor& status, const OptTensor& gate) {
     for (auto& t : {q, k, v, lat, out}) want(t, torch::kBFloat16, "latent_chunk operand");
     const int64_t T = q.size(0), H = q.size(1), n = lat.size(0);
     TORCH_CHECK(q.dim() == 3 && q.size(2) == dim + rot, "q must be [tokens, heads, dim + rot]");
@@ -116,6 +116,12 @@ void latent_chunk(const Tensor& q, const Tensor& angles, const Tensor& k, const 
     p.out = reinterpret_cast<__nv_bfloat16*>(out.data_ptr()); p.out_row = out.size(1);
     p.dim = dim; p.rot = rot; p.vdim = vdim; p.n_heads = H; p.window = window; p.scale = scale;
     p.sink = sink ? floats(*sink, H, "sink") : nullptr;
+    if (gate) {
+        want_like(*gate, false, "gate");
+        TORCH_CHECK(gate->dim() == 2 && gate->size(0) == T && gate->size(1) == H * vdim && gate->stride(1) == 1 && gate->stride(0) % 8 == 0 &&
+                    reinterpret_cast<uintptr_t>(gate->data_ptr()) % 16 == 0, "gate must be [tokens, heads * vdim] in whole 16-byte units");
+        p.gate = b(*gate); p.gate_row = gate->stride(0);
+    }
     if (status) {
         want(*status, torch::kInt32, "status");
         check(llm::launch_latent_chunk_tc(p, n, seqs.size(0), max_q_len, status->data_ptr<int>(), stream()), "latent_chunk_tc");

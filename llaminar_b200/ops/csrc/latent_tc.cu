@@ -215,6 +215,15 @@ __global__ void __launch_bounds__(CHUNK_THREADS, 1) latent_chunk_tc_kernel(const
 #pragma unroll
             for (int u = 0; u < HD / 8; ++u) {
                 if (half * HD + u * 8 >= p.vdim) break;
+                if (p.gate) {
+                    const uint4 g = *reinterpret_cast<const uint4*>(p.gate + (size_t)(sq.q_start + q0 + row) * p.gate_row + (size_t)head * p.vdim + half * HD + 8 * u);
+                    const uint32_t gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                    for (int i = 0; i < 4; ++i) {
+                        o[8 * u + 2 * i] *= __fdividef(1.f, 1.f + __expf(-bf16_lo(gw[i])));
+                        o[8 * u + 2 * i + 1] *= __fdividef(1.f, 1.f + __expf(-bf16_hi(gw[i])));
+                    }
+                }
                 *reinterpret_cast<uint4*>(dst + 8 * u) = make_uint4(pack_bf16(o[8 * u] * inv, o[8 * u + 1] * inv), pack_bf16(o[8 * u + 2] * inv, o[8 * u + 3] * inv),
                                                                     pack_bf16(o[8 * u + 4] * inv, o[8 * u + 5] * inv), pack_bf16(o[8 * u + 6] * inv, o[8 * u + 7] * inv));
             }

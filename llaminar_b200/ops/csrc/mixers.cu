@@ -1,7 +1,5 @@
-// Mixers with grouped-query attention or a recurrent state: the row-wise kernels.
+// Mixers with a recurrent state: the row-wise kernels.
 //
-//   attn_prep      norms of the queries and keys over all heads together, append to the paged cache
-//   window_plain   one row and head per CTA in float arithmetic
 //   linear_rows    mLSTM and retention, row after row.  The state matrix S [vdim, dim] of a head is spread over a cluster of CTAs,
 //                  which take slices of its rows: a warp reads whole rows of S, scales them, adds v k^T and multiplies by q while
 //                  they pass through its registers, so the state is read and written once per token (what bounds a decode step).
@@ -19,7 +17,6 @@ namespace llm {
 namespace {
 
 namespace cg = cooperative_groups;
-constexpr int PAGE = 64;
 constexpr float NORM_FLOOR = 1e-6f;            // of the mLSTM normaliser
 
 LLM_DEVICE float to_f(float v) { return v; }
@@ -51,104 +48,6 @@ LLM_DEVICE float block_sum(float v, float* red) {
 #pragma unroll
     for (int i = 0; i < THREADS / 32; ++i) s += red[i];
     return s;
-}
-
-// ---- attention -----------------------------------------------------------------------------------------------------------
-template <class TI, class T>
-__global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrepParams p) {
-    __shared__ float red[8];
-    pdl_trigger();
-    pdl_wait();
-    const int t = blockIdx.x;
-    const TI* row = static_cast<const TI*>(p.in) + (size_t)t * p.in_row;
-    const TI *q = row + p.q_off, *k = row + p.k_off, *v = row + p.v_off;
-    const int nq = p.n_heads * p.dim, nk = p.n_kv_heads * p.dim;
-    const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
-    const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
-    float sq = 0.f, sk = 0.f, x[4], w[4];
-    for (int i = threadIdx.x * 4; i < nq; i += 1024) {
-        load4(q + i, x);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) sq += x[j] * x[j];
-    }
-    for (int i = threadIdx.x * 4; i < nk; i += 1024) {
-        load4(k + i, x);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) sk += x[j] * x[j];
-    }
-    const float iq = 1.f / sqrtf(block_sum<256>(sq, red) / (float)(p.n_heads * p.true_dim) + p.eps);
-    const float ik = 1.f / sqrtf(block_sum<256>(sk, red) / (float)(p.n_kv_heads * p.true_dim) + p.eps);
-    T* qo = static_cast<T*>(p.q_out) + (size_t)t * nq;
-    for (int i = threadIdx.x * 4; i < nq; i += 1024) {
-        load4(q + i, x); load4(p.q_norm + i, w);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) x[j] *= iq * w[j];
-        store4(qo + i, x);
-    }
-    for (int i = threadIdx.x * 4; i < nk; i += 1024) {
-        const int g = i / p.dim, c = i - g * p.dim;
-        T* dst = static_cast<T*>(p.kv) + (((size_t)page * 2 * p.n_kv_heads + g) * PAGE + pos % PAGE) * p.dim + c;
-        load4(k + i, x); load4(p.k_norm + i, w);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) x[j] *= ik * w[j];
-        store4(dst, x);
-        load4(v + i, x);
-        store4(dst + (size_t)p.n_kv_heads * PAGE * p.dim, x);
-    }
-}
-
-template <class TG, class T>
-__global__ void __launch_bounds__(128) window_plain_kernel(const WindowPlainParams p) {
-    extern __shared__ __align__(16) float sm[];
-    __shared__ float s_score[64];
-    pdl_trigger();
-    pdl_wait();
-    const int h = blockIdx.x, t = blockIdx.y, D = p.dim, g = h / (p.n_heads / p.n_kv_heads);
-    float *sq = sm, *so = sm + D;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int pos = p.positions[t];
-    const int* btab = p.block_table + (size_t)LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs) * p.max_pages;
-    const T* q = static_cast<const T*>(p.q) + ((size_t)t * p.n_heads + h) * D;
-    for (int i = threadIdx.x; i < D; i += 128) { sq[i] = to_f(q[i]); so[i] = 0.f; }
-    __syncthreads();
-    auto key_row = [&](int key, int which) {
-        const int page = LLM_CHECK_INDEX(btab[key / PAGE], p.n_pages);
-        return static_cast<const T*>(p.kv) + ((((size_t)page * 2 + which) * p.n_kv_heads + g) * PAGE + key % PAGE) * D;
-    };
-    float m = p.sink ? p.sink[h] : -INFINITY, l = p.sink ? 1.f : 0.f;
-    for (int k0 = p.window > 0 ? max(0, pos - p.window + 1) : 0; k0 <= pos; k0 += 64) {
-        const int n = min(64, pos + 1 - k0);
-        for (int j = warp; j < n; j += 4) {
-            const T* row = key_row(k0 + j, 0);
-            float s = 0.f;
-            for (int i = lane; i < D; i += 32) s = fmaf(sq[i], to_f(row[i]), s);
-            s = warp_sum(s);
-            if (lane == 0) s_score[j] = s * p.scale;
-        }
-        __syncthreads();
-        float nm = m;
-        for (int j = 0; j < n; ++j) nm = fmaxf(nm, s_score[j]);
-        const float c = expf(m - nm);
-        __syncthreads();
-        if ((int)threadIdx.x < n) s_score[threadIdx.x] = expf(s_score[threadIdx.x] - nm);
-        __syncthreads();
-        float ps = 0.f;
-        for (int j = 0; j < n; ++j) ps += s_score[j];
-        l = l * c + ps;
-        m = nm;
-        for (int i = threadIdx.x; i < D; i += 128) {
-            float a = so[i] * c;
-            for (int j = 0; j < n; ++j) a = fmaf(s_score[j], to_f(key_row(k0 + j, 1)[i]), a);
-            so[i] = a;
-        }
-        __syncthreads();
-    }
-    T* o = static_cast<T*>(p.out) + ((size_t)t * p.n_heads + h) * D;
-    for (int i = threadIdx.x; i < D; i += 128) {
-        float v = so[i] / l;
-        if (p.gate) v *= 1.f / (1.f + expf(-to_f(static_cast<const TG*>(p.gate)[(size_t)t * p.gate_row + (size_t)h * D + i])));
-        o[i] = from_f<T>(v);
-    }
 }
 
 // ---- linear attention ------------------------------------------------------------------------------------------------------
@@ -348,23 +247,6 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const LinearParams p, co
 }
 
 }  // namespace
-
-cudaError_t launch_attn_prep(const AttnPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {
-    if (rows == 0) return cudaSuccess;
-    if (p.dim % 8 || p.in_row % 4 || p.q_off % 4 || p.k_off % 4 || p.v_off % 4 || (f32 && !in_f32)) return cudaErrorInvalidValue;
-    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(256), 0, st, p); };
-    if (f32) return go(attn_prep_kernel<float, float>);
-    return in_f32 ? go(attn_prep_kernel<float, __nv_bfloat16>) : go(attn_prep_kernel<__nv_bfloat16, __nv_bfloat16>);
-}
-
-cudaError_t launch_window_plain(const WindowPlainParams& p, int rows, bool gate_f32, bool f32, cudaStream_t st) {
-    if (rows == 0) return cudaSuccess;
-    const size_t smem = (size_t)p.dim * 8;
-    if (rows > 65535 || smem > 48 * 1024 || p.n_heads % p.n_kv_heads) return cudaErrorInvalidValue;
-    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(p.n_heads, rows), dim3(128), smem, st, p); };
-    if (f32) return gate_f32 ? go(window_plain_kernel<float, float>) : go(window_plain_kernel<__nv_bfloat16, float>);
-    return gate_f32 ? go(window_plain_kernel<float, __nv_bfloat16>) : go(window_plain_kernel<__nv_bfloat16, __nv_bfloat16>);
-}
 
 cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, bool f32, cudaStream_t st) {
     if (n_seqs == 0) return cudaSuccess;

@@ -26,6 +26,9 @@ struct AttnDecodeParams {
     const float* sink;             // optional [n_heads]: one more logit in the softmax denominator, without a value
     const float* gate;             // optional [rows, gate_row]: head h of a row is multiplied by sigmoid(gate[h * head_dim ...])
     size_t gate_row;
+    int gate_heads;                // the gate has one number per head
+    int chunk;                     // a row sees keys of its own chunk of this many positions only (0: no chunks)
+    float softcap;                 // scores s become softcap * tanh(s / softcap) (0: as they are)
 };
 
 struct AttnPrefillParams {
@@ -42,6 +45,8 @@ struct AttnPrefillParams {
     const float* sink;
     const __nv_bfloat16* gate;
     size_t gate_row;               // even
+    int gate_heads, chunk;
+    float softcap;
 };
 
 int attn_decode_pick_splits(int batch, int n_kv_heads, int max_pages_in_use);

@@ -11,7 +11,7 @@ from . import _count
 from . import build as _build
 
 GEMV_MAX_ROWS = 8
-ACT_NONE, ACT_GELU_MUL, ACT_RELU2, ACT_GELU_SIDE = range(4)
+ACT_NONE, ACT_GELU_MUL, ACT_RELU2, ACT_GELU_SIDE, ACT_SILU_MUL, ACT_GATE = range(6)
 _ready = False
 
 
@@ -26,17 +26,19 @@ def ext():
 
 
 def resid_norm(h, y=None, w_post=None, *, add=True, y_rows=None, w_next=None, xn=None, copy0=None, copy1=None, eps: float, y2=None,
-               w_y=None, w_y2=None, factor: float = 1.0, center_post: bool = False, center_next: bool = False) -> None:
+               w_y=None, w_y2=None, factor: float = 1.0, center_post: bool = False, center_next: bool = False, y_w=None) -> None:
     """h = (h if add) + norm(y) * w_post (``y`` None: h is only read; ``y_rows`` gathers rows of y; ``w_post`` None: y * factor),
     then xn = norm(h) * w_next and copies of h in the activation type.  With ``y2``, y stands for half the sum of RMSNorm(y) * w_y
-    and RMSNorm(y2) * w_y2.  The norms are RMSNorms, or with ``center_post`` / ``center_next`` layer norms without a bias.  One launch."""
-    ext().resid_norm(y, y_rows, w_post, h, add, w_next, xn, copy0, copy1, eps, y2, w_y, w_y2, factor, center_post, center_next)
+    and RMSNorm(y2) * w_y2; with ``y_w`` [tokens, parts] for the sum of a token's rows of y (all of them, or those ``y_rows`` names) times their
+    weights.  The norms are RMSNorms, or with ``center_post`` / ``center_next`` layer norms without a bias.  One launch."""
+    ext().resid_norm(y, y_rows, w_post, h, add, w_next, xn, copy0, copy1, eps, y2, w_y, w_y2, factor, center_post, center_next, y_w)
     _count()
 
 
 def activate(x: torch.Tensor, act: torch.Tensor, kind: int, side=None) -> None:
-    """act = gelu_tanh(x[:, :n]) * x[:, n:] (ACT_GELU_MUL), squared relu (ACT_RELU2), or gelu_tanh(x) times columns of each token's
-    row of a table (ACT_GELU_SIDE; ``side``: table, first column, columns, tokens)."""
+    """act = gelu_tanh(x[:, :n]) * x[:, n:] (ACT_GELU_MUL), the same with silu (ACT_SILU_MUL), squared relu (ACT_RELU2), gelu_tanh(x) times
+    columns of each token's row of a table (ACT_GELU_SIDE; ``side``: table, first column, columns, tokens), or x times the sigmoid of
+    those columns of the row itself (ACT_GATE; tokens None).  ``act`` may be ``x``, except for the pairs."""
     ext().activate(x, act, kind, *(side or (None, 0, 0, None)))
     _count()
 
@@ -60,8 +62,8 @@ def gemv_fits(w: torch.Tensor, x: torch.Tensor) -> bool:
 
 
 def gemv_dense(w, x, out, gelu: bool = False, act: int = ACT_NONE, side=None) -> None:
-    """out[z] = x[z] @ w[z]^T for at most eight bf16 rows; ``act`` (see `activate`): applied to the result; ``gelu``: w stacks gate
-    and up, out = gelu_tanh(gate) * up."""
+    """out[z] = x[z] @ w[z]^T for at most eight bf16 rows; ``act`` (see `activate`): applied to the result (a gate's columns run over
+    all z); ``gelu``: w stacks gate and up, out = gelu_tanh(gate) * up."""
     ext().gemv_dense(w, x, out, ACT_GELU_MUL if gelu else act, *(side or (None, 0, 0, None)))
     _count()
 

@@ -9,7 +9,7 @@ import torch
 
 from . import _count
 from . import build as _build
-from .dense import GEMV_MAX_ROWS, gelu_mul, gemv_dense, gemv_fits, resid_norm, rope_angles  # noqa: F401
+from .dense import ACT_GATE, ACT_NONE, GEMV_MAX_ROWS, activate, gelu_mul, gemv_dense, gemv_fits, resid_norm, rope_angles  # noqa: F401
 from .dense import bounds_status as _dense_bounds_status
 
 _ready = False
@@ -71,10 +71,11 @@ def latent_gather(kv, seqs, max_k_len: int, block_table, out) -> None:
 
 
 def latent_chunk(q, angles, k, v, lat, rot_off: int, seqs, max_q_len: int, out, dim: int, rot: int, vdim: int, window: int,
-                 scale: float, sink, status=None) -> None:
+                 scale: float, sink, status=None, gate=None) -> None:
     """Attention of prompt chunks on keys and values written out per head and the shared rotated parts in ``lat``.  With
-    ``status`` the tcgen05 form runs, which takes the values transposed ([heads * vdim, keys])."""
-    ext().latent_chunk(q, angles, k, v, lat, rot_off, seqs, max_q_len, out, dim, rot, vdim, window, scale, sink, status)
+    ``status`` the tcgen05 form runs, which takes the values transposed ([heads * vdim, keys]).  ``gate`` [tokens, heads * vdim]: the result times its
+    sigmoid."""
+    ext().latent_chunk(q, angles, k, v, lat, rot_off, seqs, max_q_len, out, dim, rot, vdim, window, scale, sink, status, gate)
     _count()
 
 

@@ -1,5 +1,4 @@
-"""Python surface of the mixers extension (csrc/mixers.cu, linear_tc.cu, attention.cu, attention_tc.cu): grouped-query attention with a
-sliding window, sinks and an output gate, and linear attention with a recurrent state.
+"""Python surface of the mixers extension (csrc/mixers.cu, linear_tc.cu): linear attention with a recurrent state.
 
 As in :mod:`llaminar_b200.ops`, every call launches hand-written CUDA on the current stream; there is no fallback.
 """
@@ -7,11 +6,9 @@ from __future__ import annotations
 
 import torch
 
-from . import _attn_tc_default, _count
+from . import _count
 from . import build as _build
 
-DECODE_GROUP = 16              # query heads per key head that the decode kernel takes
-HEAD_SIZES = (64, 128)         # of the tensor-core attention kernels
 _ready = False
 
 
@@ -23,43 +20,6 @@ def ext():
         mod.set_pdl(bool(debug_env().pdl))
         _ready = True
     return mod
-
-
-def attn_prep(rows, q_off: int, k_off: int, v_off: int, q_norm, k_norm, positions, seq_ids, block_table, q_out, kv, true_dim: int, eps: float) -> None:
-    """Projected rows -> normed queries [tokens, heads, dim] and the tokens' entries of the paged cache (both norms over all heads
-    of a projection, and the append, in one launch).  ``v_off`` = ``k_off``: the values are the keys before their norm."""
-    ext().attn_prep(rows, q_off, k_off, v_off, q_norm, k_norm, positions, seq_ids, block_table, q_out, kv, true_dim, eps)
-    _count()
-
-
-def window_plain(q, kv, out, positions, seq_ids, block_table, window: int, scale: float, sink, gate) -> None:
-    """Attention of any rows in float arithmetic: 32-bit mode, and shapes without a tensor-core kernel."""
-    ext().window_plain(q, kv, out, positions, seq_ids, block_table, window, scale, sink, gate)
-    _count()
-
-
-def decode_splits(batch: int, kv_heads: int, dim: int, max_pages: int, window: int, scratch) -> int:
-    """Key splits of the decode kernel: about two CTAs per SM, at least two pages each, partial sums within the scratch."""
-    pages = min(max_pages, window // 64 + 2) if window else max_pages
-    n = max(1, min(16, 296 // max(1, batch * kv_heads), pages // 2))
-    n = min(n, scratch.part_o.numel() // (batch * kv_heads * 16 * dim), scratch.part_ml.numel() // (batch * kv_heads * 32))
-    return max(1, n) if batch * kv_heads <= scratch.attn_tickets.numel() else 1
-
-
-def attn_decode(q, kv, out, block_table, seq_lens, scale: float, n_splits: int, window: int, sink, gate, scratch) -> None:
-    """One row per sequence.  ``gate``: float rows whose sigmoid multiplies the result."""
-    ext().attn_decode(q, kv, out, block_table, seq_lens, scratch.part_o, scratch.part_ml, scratch.attn_tickets, scale, n_splits, window, sink, gate)
-    _count()
-
-
-def attn_prefill(q, kv, out, block_table, cu_q, ctx_lens, scale: float, max_q_len: int, window: int, sink, gate, status=None) -> None:
-    """Portions of prompts; with ``status`` the tcgen05 form."""
-    ext().attn_prefill(q, kv, out, block_table, cu_q, ctx_lens, scale, max_q_len, window, sink, gate, status)
-    _count()
-
-
-def prefill_tc(dim: int, max_q_len: int) -> bool:
-    return dim == 128 and max_q_len >= 128 and _attn_tc_default()
 
 
 def linear_rows(rows, offs, gates, decay, angles, q_scale: float, k_scale: float, cu, positions, slots, state, true_vdim: int, norm_w,

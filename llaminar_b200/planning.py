@@ -101,15 +101,12 @@ class ExecutionPlan:
 
 def layer_weight_bytes(cfg: ModelConfig, recipe: QuantRecipe, layer: int, tp: TPPlan) -> float:
     d, D = cfg.d_model, cfg.head_dim
-    if cfg.is_latent:                           # stored as 16-bit matrices whatever the file's format
-        m, ff = cfg.mixers[layer], cfg.ff_width(layer)
-        n = d * (m.q_rank + m.kv_rank + m.rot_dim) + m.heads * (m.dim + m.rot_dim) * m.q_rank
-        n += m.heads * (2 * m.dim + m.vdim) * m.kv_rank + d * m.heads * m.vdim + 3 * d * ff        # the key matrices are held twice
-        return 2.0 * n
-    if cfg.has_mixers:
-        from .models.config import family_of
-        return sum((2.0 if kind == "mat" else 4.0) * math.prod(shape) for _, name, kind, shape in family_of(cfg.arch).tensor_names(cfg)
-                   if name.startswith(f"blk.{layer}."))
+    if cfg.has_mixers:                          # stored as 16-bit matrices whatever the file's format
+        from .models.config import LatentAttention, family_of
+        m = cfg.mixers[layer]
+        twice = 2.0 * m.heads * m.dim * m.kv_rank if isinstance(m, LatentAttention) else 0.0        # the key matrices are held twice
+        return twice + sum((2.0 if kind in ("mat", "stack") else 4.0) * math.prod(shape) for _, name, kind, shape in family_of(cfg.arch).tensor_names(cfg)
+                           if name.startswith(f"blk.{layer}."))
     t = lambda name: recipe.for_tensor(f"blk.{layer}.{name}.weight", layer, cfg.n_layers)
     if cfg.is_gdn_layer(layer):
         # linear-attention block: q | k of every key head, this rank's value heads of v and z, alpha / b, output projection
@@ -168,14 +165,10 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
             pages = batch_size * ((ctx_size + 63) // 64 + 1) + 64
             stage_layers = range(first, last + 1)
             rp.kv_bytes = int(pages * len(cfg.kv_layers(stage_layers)) * 2 * tp.n_kv_local * 64 * cfg.head_dim * 2)
-            if cfg.is_latent:                   # one cache layer per layer run; input matrix of the looped layers
-                rp.kv_bytes = int(pages * sum(cfg.mixers[i].cache_width for i, _ in cfg.layer_runs()) * 64 * 2)
-                rp.weight_bytes += 4 * cfg.d_model * cfg.d_model if cfg.loop else 0
-            elif cfg.has_mixers:
-                rp.weight_bytes += 2 * cfg.vocab_size * cfg.side_dim * cfg.n_layers
-                from .engine.kv_cache import LayerStates
-                shapes = mixer_kv_shapes(cfg)
-                rp.kv_bytes = pages * sum(2 * h * d for h, d in shapes) * 64 * 2 + (batch_size + 1) * LayerStates.bytes_per_slot(mixer_state_shapes(cfg))
+            if cfg.has_mixers:                  # side embedding of the layers, input matrix of the looped ones
+                rp.weight_bytes += 2 * cfg.vocab_size * cfg.side_dim * cfg.n_layers + (4 * cfg.d_model * cfg.d_model if cfg.loop else 0)
+                from .engine.kv_cache import LayerStates, PagedKVCache
+                rp.kv_bytes = pages * PagedKVCache.bytes_per_page(0, 0, 0, layer_shapes=mixer_kv_shapes(cfg)) + (batch_size + 1) * LayerStates.bytes_per_slot(mixer_state_shapes(cfg))
             if cfg.is_hybrid:
                 # one fp32 state slot per batch lane (+1 scratch) for every linear-attention layer of the stage
                 from .engine.kv_cache import HybridState
@@ -186,12 +179,9 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
             ff = (tp.ff_stop - tp.ff_start) if not cfg.is_moe else cfg.expert_ff
             rp.activation_bytes = int(T * (cfg.d_model * (4 + 2) + (tp.n_heads_local + 2 * tp.n_kv_local) * cfg.head_dim * 2
                                            + 2 * tp.n_heads_local * cfg.head_dim * 2 + ff * 2))
-            if cfg.is_latent:
-                m = max(cfg.mixers, key=lambda m: m.heads * (2 * m.dim + m.rot_dim + 2 * m.vdim))
-                rp.activation_bytes = int(T * (cfg.d_model * (4 + 8) + 2 * (m.heads * (2 * m.dim + m.rot_dim + 2 * m.vdim) + 2 * m.q_rank
-                                                                            + 2 * m.cache_width + 3 * ff)))
-            elif cfg.has_mixers:
-                rp.activation_bytes = int(T * (cfg.d_model * (4 + 6) + 2 * (max(mixer_columns(m) for m in cfg.mixers) + 2 * max(cfg.layer_ff))))
+            if cfg.has_mixers:                  # every chosen expert has its rows
+                experts = max((e.top * (2 * cfg.d_model + 3 * e.ff) for e in cfg.layer_experts if e), default=0)
+                rp.activation_bytes = int(T * (cfg.d_model * (4 + 8) + 2 * (max(mixer_columns(m) for m in cfg.mixers) + max(3 * max(cfg.layer_ff), experts))))
             rp.workspace_bytes = int(256 * 65536 * 4 + (1 << 22) * 4 + batch_size * 4 * (tp.vocab_stop - tp.vocab_start) * 4)
             if rp.total_bytes > hbm_bytes * 0.95:
                 plan.errors.append(f"rank {rank} ({dev}): needs {rp.total_bytes / 1e9:.1f} GB, device has {hbm_bytes / 1e9:.0f} GB")

@@ -172,7 +172,7 @@ def test_rows_of_many_sequences():
 def test_attention_forms(heads, kv, dim, true_dim, window):
     """Prompt (tcgen05 and mma.sync), decode and plain kernel on pages in random order, behind cached context."""
     from llaminar_b200 import ops as base
-    from llaminar_b200.ops import mixers as ops
+    from llaminar_b200.ops import grouped as ops
     n, sc = 330, base.scratch_for(torch.device("cuda", 0))
     cols = (2 * heads + kv) * dim
     live = (torch.arange(cols, device="cuda") % dim) < true_dim                  # padding of a head is zero
@@ -197,7 +197,7 @@ def test_attention_forms(heads, kv, dim, true_dim, window):
     want = o * torch.sigmoid(x[:, (heads + kv) * dim:])
     gate = rows[:, (heads + kv) * dim:]
     out = torch.empty(n, heads * dim, dtype=BF, device="cuda")
-    ops.window_plain(q, cache, out, pos, sid, bt, window, scale, sink, gate)
+    ops.attn_plain(q, cache, out, pos, sid, bt, window, scale, sink, gate)
     assert err(out, want) < 1e-2, "plain"
     if dim in ops.HEAD_SIZES:
         for first in (0, 70):                                                    # rows from `first` on, the ones before are context

@@ -95,7 +95,7 @@ def test_rotation_keeps_relative_scores():
 def test_config_round_trip_and_errors():
     m = cases.model("mixed")
     c = config_from_json(m["config"])
-    assert c.is_latent and [x.window for x in c.mixers] == [20, 77, 64, 1000] and c.layer_ff == (56, 56, 0, 56)
+    assert c.is_attention_stack and [x.window for x in c.mixers] == [20, 77, 64, 1000] and c.layer_ff == (56, 56, 0, 56)
     again = config_from_json(config_to_json(c))
     assert again == c
     looped = config_from_json(cases.model("loop_middle")["config"])
@@ -132,8 +132,8 @@ def test_directory_and_gguf_round_trip(tmp_path):
 def test_cache_layout_per_layer_run():
     eng = cases.engine(cases.model("loop_all"), "cpu")
     assert [tuple(l.shape[1:]) for l in eng.kv.layers] == [(64, 48), (64, 48)] * 2 or len(eng.kv.layers) == 4
-    assert [l.shape[2] for l in eng.kv.layers] == eng.model.kv_row_widths
-    assert eng.kv.page_bytes == sum(eng.model.kv_row_widths) * 64 * 4
+    assert [(l.shape[2],) for l in eng.kv.layers] == eng.model.kv_layer_shapes
+    assert eng.kv.page_bytes == sum(w for w, in eng.model.kv_layer_shapes) * 64 * 4
 
 
 def test_feed_refuses_bad_steps():

@@ -113,7 +113,7 @@ def test_oracle_recurrences_written_out():
 def test_config_round_trip_and_errors():
     m = cases.model("both")
     c = config_from_json(m["config"])
-    assert c.has_mixers and c.has_state and not c.is_latent
+    assert c.has_mixers and c.has_state and not c.is_attention_stack
     assert [type(x) for x in c.mixers] == [MatrixLSTM, ParallelMixers] * 2 and c.mixers[3].left.window == 77 and c.mixers[2].gate_cap == 4.0
     assert config_from_json(config_to_json(c)) == c
     for name in cases.MODELS:
