@@ -155,6 +155,12 @@ def route(h, T, top):
     return best.indices, torch.softmax(best.values, dim=-1)
 
 
+def router_gap(h, T, top):
+    """[n] distance between the last logit that is chosen and the first that is not (infinite when all are)."""
+    z = torch.cat([h @ T("router").T + T("router.b"), h.new_full((h.shape[0], 1), float("-inf"))], dim=-1).sort(dim=-1, descending=True).values
+    return z[:, top - 1] - z[:, top]
+
+
 def experts_ffn(h, m, T):
     ids, weights = route(h, T, m["router"]["top"])
     out = torch.zeros_like(h)
@@ -164,7 +170,7 @@ def experts_ffn(h, m, T):
     return out
 
 
-def decoder_layer(x, i, model, W):
+def decoder_layer(x, i, model, W, gaps=None):
     entry, eps, p = model["config"]["layers"][i], model["config"]["norm"]["eps"], f"l{i}."
     mix, mlp = (lambda name: W(p + "mix." + name)), (lambda name: W(p + "mlp." + name))
     y = MIXERS[entry["type"]](rms_norm(x, W(p + "norm1"), eps), entry["mixer"], mix, eps)
@@ -172,6 +178,8 @@ def decoder_layer(x, i, model, W):
     f = entry.get("mlp")
     if f:
         h = rms_norm(x, W(p + "norm2"), eps)
+        if gaps is not None and f["kind"] == "moe":
+            gaps.append(router_gap(h, mlp, f["router"]["top"]))
         y = gated_ffn(h, mlp) if f["kind"] == "dense" else experts_ffn(h, f, mlp)
         x = x + rms_norm(y, W(p + "norm2b"), eps)
     return x
@@ -191,15 +199,16 @@ def run_order(cfg):
     return out + [(i, None) for i in range(stop, n)]
 
 
-def forward(tokens, model, dt=torch.float64, taps=None):
-    """Logits [n, vocab] of one sequence; `taps` (a list) receives the residual stream after every layer run."""
+def forward(tokens, model, dt=torch.float64, taps=None, gaps=None):
+    """Logits [n, vocab] of one sequence; `taps` (a list) receives the residual stream after every layer run, `gaps` how close every
+    choice of experts was."""
     cfg = model["config"]
     W = lambda name: model["tensors"][name].to(dt)
     x = x0 = W("embed")[torch.as_tensor(tokens).long()]
     for i, t in run_order(cfg):
         if t is not None:
             x = enter_pass(x, x0, t, W)
-        x = decoder_layer(x, i, model, W)
+        x = decoder_layer(x, i, model, W, gaps)
         if taps is not None:
             taps.append(x)
     return rms_norm(x, W("final.norm"), cfg["norm"]["eps"]) @ W("embed").T * cfg["logit_scale"]
