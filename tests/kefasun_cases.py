@@ -18,10 +18,10 @@ MODELS = {
     "kinds": ([C(chunk=20, mlp=moe()), L(window=20), G(softcap=3.0, mlp=moe(4, 1, 24))], {"start": 0, "stop": 2, "times": 2}),
     "order": ([G(heads=6, kv_heads=3, dim=33, vdim=12, rot_dims=6, softcap=20.0), L(heads=5, dim=16, rot_dim=12, vdim=24, kv_rank=33, q_rank=27, window=77, mlp=moe(3, 3, 20)),
                C(heads=3, kv_heads=1, dim=10, vdim=30, rot_dims=10, chunk=64, mlp=None), L(heads=1, window=1000), C(heads=2, kv_heads=2, dim=18, rot_dims=2, chunk=1)], None),
-    "loop_middle": ([C(chunk=70), G(mlp=moe(6, 4, 17)), L(window=31, mlp=moe(9, 2, 32)), C(chunk=130, dim=16)], {"start": 1, "stop": 3, "times": 3}),
+    "loop_middle": ([C(chunk=70), G(mlp=moe(6, 4, 17)), L(window=31, mlp=moe(9, 3, 32)), C(chunk=130, dim=16)], {"start": 1, "stop": 3, "times": 2}),
     "loop_all": ([L(window=65, mlp=None), C(chunk=33, heads=8, kv_heads=2, dim=8, vdim=8, rot_dims=4, mlp=moe(2, 1, 40))], {"start": 0, "stop": 2, "times": 2}),
     "loop_once": ([G(heads=2, kv_heads=1, softcap=50.0), C(chunk=1000, mlp=moe())], {"start": 0, "stop": 1, "times": 1}),
-    "loop_end": ([L(window=1, mlp=moe(8, 3, 16)), G(softcap=5.0, mlp=None), C(chunk=65)], {"start": 2, "stop": 3, "times": 4}),
+    "loop_end": ([L(window=1, mlp=moe(8, 3, 16)), G(softcap=5.0, mlp=None), C(chunk=65)], {"start": 2, "stop": 3, "times": 3}),
 }
 # sizes of the tcgen05 kernels (GPU only)
 WIDE = ([C(heads=4, kv_heads=2, dim=128, vdim=96, rot_dims=48, chunk=150, mlp=moe(6, 3, 136)), L(heads=20, dim=64, rot_dim=32, vdim=64, kv_rank=128, q_rank=64, window=90, mlp=dense(128)),

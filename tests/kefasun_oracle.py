@@ -231,7 +231,7 @@ def random_model(layers, seed=0, vocab=97, width=48, loop=None, eps=1e-5, sink_s
 
     t["embed"] = torch.randn(vocab, width, generator=g).to(torch.bfloat16)
     if loop:
-        mat("loop.in", width, 2 * width)
+        mat("loop.in", width, 2 * width, 1.4)
         t["loop.step"] = (torch.randn(loop["times"], width, generator=g) * 0.7).to(torch.bfloat16)
     for i, e in enumerate(layers):
         m, p = e["mixer"], f"l{i}."
@@ -247,7 +247,7 @@ def random_model(layers, seed=0, vocab=97, width=48, loop=None, eps=1e-5, sink_s
         else:
             G = m["kv_heads"]
             mat(p + "mix.q", H * dim, width), mat(p + "mix.k", G * dim, width), mat(p + "mix.v", G * vd, width)
-            vec(p + "mix.q.norm", dim, 1.5, 0.4), vec(p + "mix.k.norm", dim, 1.5, 0.4)
+            vec(p + "mix.q.norm", dim, 1.2, 0.4), vec(p + "mix.k.norm", dim, 1.2, 0.4)
         mat(p + "mix.g", H if e["type"] == "attention" else H * vd, width, 1.5)
         mat(p + "mix.o", width, H * vd)
         f = e.get("mlp")

@@ -59,7 +59,7 @@ right = {n: getattr(oracle, n) for n in dir(oracle) if callable(getattr(oracle, 
     ("enter_pass", lambda x, x0, t, W: right["enter_pass"](x, x0, 0, W)), ("enter_pass", lambda x, x0, t, W: right["enter_pass"](x, x, t, W))])
 def test_a_mistake_would_be_noticed(monkeypatch, where, wrong):
     """With one mechanism wrong in the oracle the 16-bit tolerance of the engine checks is exceeded."""
-    m, t = cases.model("kinds", seed=1), cases.tokens(230, 3)
+    m, t = cases.model("kinds", seed=1), cases.tokens(20 if where == "plain_softmax" else 230, 3)        # one in the denominator shows among few keys
     want = oracle.forward(t, m)
     monkeypatch.setattr(oracle, where, wrong)
     monkeypatch.setattr(oracle, "MIXERS", {"attention": oracle.chunked_attention, "latent_attention": oracle.latent_attention, "attention_2": oracle.capped_attention})
