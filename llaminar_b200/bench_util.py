@@ -124,5 +124,5 @@ def cut(cfg: ModelConfig, n_layers: int) -> ModelConfig:
     """The first layers of a shape, unlooped."""
     kw = dict(n_layers=n_layers)
     if cfg.has_mixers:
-        kw.update(mixers=cfg.mixers[:n_layers], layer_ff=cfg.layer_ff[:n_layers], loop=None)
+        kw.update(mixers=cfg.mixers[:n_layers], layer_ff=cfg.layer_ff[:n_layers], layer_experts=cfg.layer_experts[:n_layers], loop=None, loop_steps=False)
     return cfg.with_(**kw)
