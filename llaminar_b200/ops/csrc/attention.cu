@@ -127,7 +127,7 @@ LLM_DEVICE void q8_unit_to_f16(const uint4& w, __half2 sc2, __half2 off2, uint32
     }
 }
 
-template <int D, bool Q8>
+template <int D, bool Q8, bool CAP>                // CAP: scores are soft-capped
 __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecodeParams p) {
     extern __shared__ __align__(128) uint8_t smem[];
     pdl_trigger();
@@ -180,7 +180,11 @@ __global__ void __launch_bounds__(128) paged_attn_decode_kernel(const AttnDecode
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-    const ScoreScale score(p.scale, p.softcap);
+    const ScoreScale scaling(p.scale, p.softcap);
+    auto score = [&](float s) {
+        if constexpr (CAP) return scaling.capped(s);
+        else return scaling.linear(s);
+    };
 
     auto issue = [&](int pg, int stage) {
         if (Q8) {
@@ -413,20 +417,21 @@ cudaError_t launch_attn_decode(const AttnDecodeParams& p, int batch, int n_split
         return launch_pdl(kernel, grid, dim3(128), smem, st, p);
     };
     constexpr int SLACK = 1024;
-    if (p.head_dim == 128) {
-        if (p.kv_q8) return go(paged_attn_decode_kernel<128, true>, DecodeSmem<128, true>::BYTES + SLACK);
-        return go(paged_attn_decode_kernel<128, false>, DecodeSmem<128, false>::BYTES + SLACK);
-    } else if (p.head_dim == 64) {
-        if (p.kv_q8) return go(paged_attn_decode_kernel<64, true>, DecodeSmem<64, true>::BYTES + SLACK);
-        return go(paged_attn_decode_kernel<64, false>, DecodeSmem<64, false>::BYTES + SLACK);
-    }
+    if (p.kv_q8 && p.softcap > 0.f) return cudaErrorInvalidValue;
+    auto pick = [&](auto q8, auto plain, auto capped, int smem_q8, int smem) { return p.kv_q8 ? go(q8, smem_q8 + SLACK) : go(p.softcap > 0.f ? capped : plain, smem + SLACK); };
+    if (p.head_dim == 128)
+        return pick(paged_attn_decode_kernel<128, true, false>, paged_attn_decode_kernel<128, false, false>, paged_attn_decode_kernel<128, false, true>,
+                    DecodeSmem<128, true>::BYTES, DecodeSmem<128, false>::BYTES);
+    if (p.head_dim == 64)
+        return pick(paged_attn_decode_kernel<64, true, false>, paged_attn_decode_kernel<64, false, false>, paged_attn_decode_kernel<64, false, true>,
+                    DecodeSmem<64, true>::BYTES, DecodeSmem<64, false>::BYTES);
     return cudaErrorInvalidValue;
 }
 
 // ------------------------------------------------------------------------------------------------
 // prefill: 64 query rows per CTA, keys/values of one page per step
 // ------------------------------------------------------------------------------------------------
-template <int D>
+template <int D, bool CAP>
 __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefillParams p) {
     extern __shared__ __align__(128) uint8_t smem[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
@@ -469,7 +474,11 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
 #pragma unroll
         for (int i = 0; i < 4; ++i) o[n][i] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
-    const ScoreScale score(p.scale, p.softcap);
+    const ScoreScale scaling(p.scale, p.softcap);
+    auto score = [&](float s) {
+        if constexpr (CAP) return scaling.capped(s);
+        else return scaling.linear(s);
+    };
 
     auto issue = [&](int pg, int stage) {
         if (pg < n_pages) {
@@ -574,18 +583,15 @@ __global__ void __launch_bounds__(128) paged_attn_prefill_kernel(const AttnPrefi
 cudaError_t launch_attn_prefill(const AttnPrefillParams& p, int n_seqs, int max_q_len, cudaStream_t st) {
     if (p.n_heads % p.n_kv_heads) return cudaErrorInvalidValue;
     dim3 grid((max_q_len + 63) / 64, p.n_heads, n_seqs);
-    if (p.head_dim == 128) {
-        constexpr int smem = 4 * PAGE * 128 * 2;
-        static bool once = false;
-        if (!once) { cudaFuncSetAttribute(paged_attn_prefill_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem); once = true; }
-        paged_attn_prefill_kernel<128><<<grid, 128, smem, st>>>(p);
-    } else if (p.head_dim == 64) {
-        constexpr int smem = 4 * PAGE * 64 * 2;
-        paged_attn_prefill_kernel<64><<<grid, 128, smem, st>>>(p);
-    } else {
-        return cudaErrorInvalidValue;
-    }
-    return cudaGetLastError();
+    auto go = [&](auto kernel, int smem) {
+        cudaError_t e = smem > 48 * 1024 ? cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) : cudaSuccess;
+        if (e != cudaSuccess) return e;
+        kernel<<<grid, 128, smem, st>>>(p);
+        return cudaGetLastError();
+    };
+    if (p.head_dim == 128) return go(p.softcap > 0.f ? paged_attn_prefill_kernel<128, true> : paged_attn_prefill_kernel<128, false>, 4 * PAGE * 128 * 2);
+    if (p.head_dim == 64) return go(p.softcap > 0.f ? paged_attn_prefill_kernel<64, true> : paged_attn_prefill_kernel<64, false>, 4 * PAGE * 64 * 2);
+    return cudaErrorInvalidValue;
 }
 
 LLM_DEFINE_BOUNDS_STATUS_READER(bounds_status_attention)

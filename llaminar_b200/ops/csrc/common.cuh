@@ -111,7 +111,6 @@ struct ScoreScale {
     }
     LLM_DEVICE float linear(float s) const { return s * mul; }
     LLM_DEVICE float capped(float s) const { return fmaf(-2.f * cap, __fdividef(1.f, 1.f + exp2f(s * mul)), cap); }
-    LLM_DEVICE float operator()(float s) const { return cap > 0.f ? capped(s) : linear(s); }
 };
 
 // branch-free: the approximate division has no slow path for huge or infinite denominators (they give 0, the right limit)

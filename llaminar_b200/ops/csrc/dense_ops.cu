@@ -171,7 +171,7 @@ __global__ void __launch_bounds__(THREADS) resid_norm_kernel(const ResidNormPara
 }
 
 // The same for rows that the threads hold in registers (NV x 4 values each): every load is on its way before the first sum.
-template <class T, int THREADS, int NV>
+template <class T, int THREADS, int NV, bool PARTS>                         // PARTS: y is a weighted sum of rows
 __global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNormParams p) {
     constexpr int W = THREADS / 32;
     __shared__ float2 red[5][W];
@@ -223,7 +223,7 @@ __global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNorm
     if (!p.y || p.add) each([&](int n, int i) { Vec4<float>::load(h + i, a[n]); });
     if (p.y) {
         auto y_row = [&](size_t i) { return static_cast<const T*>(p.y) + (p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[i], p.n_y_rows) : i) * p.y_stride; };
-        if (p.n_parts) {
+        if constexpr (PARTS) {
             each([&](int n, int) { v[n][0] = v[n][1] = v[n][2] = v[n][3] = 0.f; });
 #pragma unroll 4
             for (int q = 0; q < p.n_parts; ++q) {
@@ -419,10 +419,10 @@ cudaError_t resid_norm_any(const ResidNormParams& p, int rows, cudaStream_t st) 
         return e != cudaSuccess ? e : launch_pdl(kernel, dim3(rows), dim3(threads), smem, st, p);
     };
     auto go_reg = [&](auto kernel, int threads) { return launch_pdl(kernel, dim3(rows), dim3(threads), 0, st, p); };
-    if (vec && p.d <= 1024) return go_reg(resid_norm_reg_kernel<T, 128, 2>, 128);
-    if (vec && p.d <= 2048) return go_reg(resid_norm_reg_kernel<T, 256, 2>, 256);
-    if (vec && p.d <= 4096) return go_reg(resid_norm_reg_kernel<T, 512, 2>, 512);
-    if (vec && p.d <= 8192) return go_reg(resid_norm_reg_kernel<T, 512, 4>, 512);
+    if (vec && p.d <= 1024) return go_reg(p.n_parts ? resid_norm_reg_kernel<T, 128, 2, true> : resid_norm_reg_kernel<T, 128, 2, false>, 128);
+    if (vec && p.d <= 2048) return go_reg(p.n_parts ? resid_norm_reg_kernel<T, 256, 2, true> : resid_norm_reg_kernel<T, 256, 2, false>, 256);
+    if (vec && p.d <= 4096) return go_reg(p.n_parts ? resid_norm_reg_kernel<T, 512, 2, true> : resid_norm_reg_kernel<T, 512, 2, false>, 512);
+    if (vec && p.d <= 8192) return go_reg(p.n_parts ? resid_norm_reg_kernel<T, 512, 4, true> : resid_norm_reg_kernel<T, 512, 4, false>, 512);
     if (vec) return go(resid_norm_kernel<T, 4, 512>, 512);
     return go(resid_norm_kernel<T, 1, 256>, 256);
 }

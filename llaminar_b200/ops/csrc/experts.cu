@@ -1,4 +1,6 @@
 // Mixture-of-experts feed-forwards with unquantised matrices: routing, sorting by expert, and the products of few rows.
+#include <cooperative_groups.h>
+
 #include "common.cuh"
 #include "experts.h"
 #include "launch.h"
@@ -6,6 +8,8 @@
 namespace llm {
 
 namespace {
+
+namespace cg = cooperative_groups;
 
 LLM_DEVICE float to_f(float v) { return v; }
 LLM_DEVICE float to_f(__nv_bfloat16 v) { return __bfloat162float(v); }
@@ -25,26 +29,34 @@ LLM_DEVICE void load8(const float* p, float (&v)[8]) {
 }
 
 // ---- routing -------------------------------------------------------------------------------------------------------------------
-// One warp: the `top` largest of z[0 .. n) (overwritten) and the softmax over them.  Every id it writes is a valid expert, whatever
-// the logits are.
-LLM_DEVICE void choose(float* z, const ExpertRouteParams& p, int t) {
+// One warp: the `top` largest of z[0 .. n) and the softmax over them.  Logits stay in registers as integers of the same order (NR per
+// lane), so a round is two warp-wide integer reductions.  Every id it writes is a valid expert, whatever the logits are.
+template <int NR>
+LLM_DEVICE void choose_of(const float* z, const ExpertRouteParams& p, int t) {
     const int lane = threadIdx.x & 31;
+    unsigned key[NR];
+#pragma unroll
+    for (int j = 0; j < NR; ++j) {
+        const int i = lane + j * 32;
+        const unsigned u = i < p.n ? __float_as_uint(z[i]) : 0u;
+        key[j] = i < p.n ? (u & 0x80000000u ? ~u : u | 0x80000000u) : 0u;
+    }
     float mine = -INFINITY;                        // lane r: the r-th largest logit
     int id = 0;
     for (int r = 0; r < p.top; ++r) {
-        float best = -INFINITY;
-        int at = lane < p.n ? lane : 0;
-        for (int i = lane; i < p.n; i += 32)
-            if (z[i] > best) { best = z[i]; at = i; }
+        unsigned best = 0;
 #pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float b = __shfl_xor_sync(0xffffffffu, best, o);
-            const int a = __shfl_xor_sync(0xffffffffu, at, o);
-            if (b > best || (b == best && a < at)) { best = b; at = a; }
-        }
-        if (lane == r) { mine = best; id = at; }
-        if (lane == 0) z[at] = -INFINITY;
-        __syncwarp();
+        for (int j = 0; j < NR; ++j) best = max(best, key[j]);
+        best = __reduce_max_sync(0xffffffffu, best);
+        unsigned at = 0xffffffffu;                 // the lowest expert that has it
+#pragma unroll
+        for (int j = 0; j < NR; ++j)
+            if (key[j] == best && lane + j * 32 < p.n) at = min(at, (unsigned)(lane + j * 32));
+        at = __reduce_min_sync(0xffffffffu, at);
+#pragma unroll
+        for (int j = 0; j < NR; ++j)
+            if ((unsigned)(lane + j * 32) == at) key[j] = 0;
+        if (lane == r) { mine = z[at]; id = at; }
     }
     const float top = warp_max(mine), e = lane < p.top ? expf(mine - top) : 0.f, sum = warp_sum(e);      // every lane takes part
     if (lane < p.top) {
@@ -54,18 +66,27 @@ LLM_DEVICE void choose(float* z, const ExpertRouteParams& p, int t) {
         if (p.counts) p.ranks[pair] = atomicAdd(&p.counts[id], 1);
     }
 }
+LLM_DEVICE void choose(const float* z, const ExpertRouteParams& p, int t) {
+    if (p.n <= 32) choose_of<1>(z, p, t);
+    else if (p.n <= 128) choose_of<4>(z, p, t);
+    else choose_of<EXPERTS_MAX / 32>(z, p, t);
+}
 
-// a CTA per token: its warps take the experts in turn, four at a time
-constexpr int ROUTE_THREADS = 512;
+// A cluster of CTAs per token: their warps take the experts in turn, four at a time, and leave the logits with the first CTA.
+constexpr int ROUTE_THREADS = 512, ROUTE_CLUSTER = 8;
 template <class T, bool VEC>
 __global__ void __launch_bounds__(ROUTE_THREADS) expert_route_kernel(const ExpertRouteParams p) {
     __shared__ float z[EXPERTS_MAX];
     pdl_trigger();
+    cg::cluster_group cluster = cg::this_cluster();
+    const bool spread = gridDim.x > 1;
+    if (spread) cluster.sync();                    // every CTA runs: its memory may be written
     pdl_wait();
-    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int t = blockIdx.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     constexpr int WARPS = ROUTE_THREADS / 32, NE = 4;
+    float* dst = spread ? cluster.map_shared_rank(z, 0) : z;
     const T* x = static_cast<const T*>(p.x) + (size_t)t * p.x_row;
-    for (int e0 = warp * NE; e0 < p.n; e0 += WARPS * NE) {
+    for (int e0 = (warp * gridDim.x + blockIdx.x) * NE; e0 < p.n; e0 += WARPS * NE * gridDim.x) {
         float acc[NE] = {};
         const T* w[NE];
 #pragma unroll
@@ -90,11 +111,11 @@ __global__ void __launch_bounds__(ROUTE_THREADS) expert_route_kernel(const Exper
 #pragma unroll
         for (int j = 0; j < NE; ++j) {
             const float s = warp_sum(acc[j]);
-            if (lane == 0 && e0 + j < p.n) z[e0 + j] = s + p.bias[e0 + j];
+            if (lane == 0 && e0 + j < p.n) dst[e0 + j] = s + p.bias[e0 + j];
         }
     }
-    __syncthreads();
-    if (warp == 0) choose(z, p, t);
+    if (spread) cluster.sync(); else __syncthreads();
+    if (warp == 0 && blockIdx.x == 0) choose(z, p, t);
 }
 
 // a warp per token, logits given
@@ -263,7 +284,22 @@ cudaError_t launch_expert_route(const ExpertRouteParams& p, int rows, bool f32, 
     if (p.n < 1 || p.n > EXPERTS_MAX || p.top < 1 || p.top > p.n || p.top > EXPERTS_MAX_TOP) return cudaErrorInvalidValue;
     if (p.logits) return launch_pdl(expert_choose_kernel, dim3((rows + 3) / 4), dim3(128), (size_t)4 * p.n * 4, st, p, rows);
     const bool vec = p.d % 8 == 0 && p.x_row % 8 == 0 && !((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.router)) & 15);
-    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(ROUTE_THREADS), 0, st, p); };
+    if (rows > 65535) return cudaErrorInvalidValue;
+    auto go = [&](auto kernel) {
+        cudaLaunchConfig_t cfg = {};
+        const int ctas = rows <= 16 && p.n >= 32 ? ROUTE_CLUSTER : 1;      // few tokens: the router's rows are read by more SMs
+        cfg.gridDim = dim3(ctas, rows);
+        cfg.blockDim = dim3(ROUTE_THREADS);
+        cfg.stream = st;
+        cudaLaunchAttribute attr[2];
+        attr[0].id = cudaLaunchAttributeClusterDimension;
+        attr[0].val.clusterDim.x = ctas; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+        attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+        attr[1].val.programmaticStreamSerializationAllowed = 1;
+        cfg.attrs = attr;
+        cfg.numAttrs = pdl_enabled() ? 2 : 1;
+        return cudaLaunchKernelEx(&cfg, kernel, p);
+    };
     if (f32) return vec ? go(expert_route_kernel<float, true>) : go(expert_route_kernel<float, false>);
     return vec ? go(expert_route_kernel<__nv_bfloat16, true>) : go(expert_route_kernel<__nv_bfloat16, false>);
 }

@@ -68,7 +68,7 @@ class Layer:
 
 # tokens, experts, chosen, width, expert width: one expert, all chosen, odd numbers of experts, tails of the MMA steps and tiles, more than
 # one tile per expert, experts without tokens
-SIZES = [(1, 8, 2, 256, 104), (5, 6, 3, 200, 72), (7, 40, 5, 136, 8), (33, 1, 1, 64, 64), (130, 5, 2, 1000, 200), (60, 3, 3, 128, 264), (300, 130, 2, 72, 136), (500, 4, 1, 512, 320)]
+SIZES = [(1, 8, 2, 256, 104), (5, 6, 3, 200, 72), (7, 40, 5, 136, 8), (33, 1, 1, 64, 64), (130, 5, 2, 1000, 200), (60, 3, 3, 128, 264), (300, 130, 2, 72, 136), (500, 4, 1, 512, 320), (9, 200, 6, 64, 16)]
 
 
 @pytest.mark.parametrize("T,E,top,d,ff", SIZES)
