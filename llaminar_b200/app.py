@@ -134,7 +134,7 @@ def build_engine(cfg: OrchestrationConfig):
     fp32 = v.get("activation_precision") == "fp32" and "activation_precision" in cfg.explicitly_set and torch.device(dev).type == "cuda"
     if fp32 and not mcfg.has_mixers:
         raise ConfigError(["--activation-precision fp32: the CUDA path of this model uses bf16 GEMM operands with an fp32 residual "
-                           "stream (fp32 is available for pozivik, zogepel and kefasun models, and with -d cpu)"])
+                           "stream (fp32 is available for pozivik, zogepel, kefasun and lagedra models, and with -d cpu)"])
     if mcfg.has_mixers:
         refused = [f"{flag} is not available for {mcfg.arch} models" for flag, on in
                    (("--kv-cache-precision q8_0", v.get("kv_cache_precision") in ("q8_0", "q8_1")), ("--mtp", v.get("mtp"))) if on]

@@ -37,7 +37,7 @@ def _o(*flags, **kw) -> OptionSpec:
 
 OPTIONS: list[OptionSpec] = [
     # -- model / general ------------------------------------------------------------------------------------
-    _o("-m", "--model", help="path to the .gguf checkpoint (first part of a split checkpoint), or to a checkpoint directory of a family served without conversion (pozivik, zogepel, kefasun)", category="model"),
+    _o("-m", "--model", help="path to the .gguf checkpoint (first part of a split checkpoint), or to a checkpoint directory of a family served without conversion (pozivik, zogepel, kefasun, lagedra)", category="model"),
     _o("-c", "--ctx-size", dest="ctx_size", type=int, default=4096, help="context window in tokens", category="model"),
     _o("--batch-size", type=int, default=1, help="concurrent request lanes (decode batch)", category="model"),
     _o("-p", "--prompt", help="prompt text (oneshot)", category="model"),
@@ -467,7 +467,7 @@ def validate(cfg: OrchestrationConfig) -> list[str]:
     if not on_cpu and v.get("kv_cache_precision") in ("fp16", "fp32") and "kv_cache_precision" in ex:
         errs.append(f"--kv-cache-precision {v['kv_cache_precision']}: the CUDA kernels keep the KV cache in bf16 (fp16 / fp32 are available with -d cpu)")
     if not on_cpu and v.get("activation_precision") == "fp16" and "activation_precision" in ex:
-        errs.append("--activation-precision fp16: the CUDA path uses bf16 GEMM operands with an fp32 residual stream (fp32: pozivik, zogepel and kefasun models, or any model with -d cpu)")
+        errs.append("--activation-precision fp16: the CUDA path uses bf16 GEMM operands with an fp32 residual stream (fp32: pozivik, zogepel, kefasun and lagedra models, or any model with -d cpu)")
     if v.get("kv_cache_precision") in ("tq4", "tq8"):
         errs.append(f"--kv-cache-precision {v['kv_cache_precision']}: the turbo-quantised KV caches are not built (bf16 / q8_0 on GPUs, bf16 / fp16 / fp32 with -d cpu)")
     if on_cpu and v.get("kv_cache_precision") in ("q8_0", "q8_1"):

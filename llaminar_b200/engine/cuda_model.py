@@ -346,11 +346,12 @@ class CudaModel:
         """Models whose layers have mixers and sizes of their own: unquantised matrices, cache and state layouts per layer."""
         from .dense import DenseLinear
         from .mixers import MixerStack
+        from .parallel_stack import ParallelStack
         from .stack import AttentionStack
         c = self.cfg
         if self.layer_ids != list(range(c.n_layers)):
             raise ValueError(f"a {c.arch} model cannot be cut into pipeline stages")
-        st = self.stack = (AttentionStack if c.is_attention_stack else MixerStack)(self, weights)
+        st = self.stack = (MixerStack if not c.is_attention_stack else ParallelStack if c.parallel_ff else AttentionStack)(self, weights)
         self.layers = [st.build_layer(CudaLayer(), weights, i) for i in self.layer_ids]
         self.out_norm = _f32(weights["output_norm.weight"], self.device) * c.logit_scale
         self.head = DenseLinear(st.head_matrix(weights))

@@ -79,6 +79,8 @@ class LLMEngine:
             device = "cuda" if torch.cuda.is_available() else "cpu"
         self.device = torch.device(device)
         self.is_cuda = self.device.type == "cuda"
+        if self.cfg.learned_positions:                  # no vector for positions behind the table
+            max_context = min(max_context, self.cfg.learned_positions)
         self.max_batch, self.max_context = max_batch, max_context
         self.max_prefill_tokens = max_prefill_tokens
         self.tp = tp

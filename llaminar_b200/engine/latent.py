@@ -106,7 +106,7 @@ class LatentMixer:
     def workspace(self) -> dict[str, int]:
         return {"rows": self.down.n_out, "cq": self.sizes.q_rank, "q": self.q_b.n_out, "o": self.wo.k}
 
-    def __call__(self, xn: torch.Tensor, fb, plan, kv_layer: torch.Tensor) -> torch.Tensor:
+    def __call__(self, xn: torch.Tensor, fb, plan, kv, kv_layer: torch.Tensor) -> torch.Tensor:
         """Normed input rows -> the gated heads, input of the output product."""
         from ..ops import latent as ops
         st, m, s, T, lp = self.stack, self.m, self.sizes, xn.shape[0], plan.latent

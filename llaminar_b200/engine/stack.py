@@ -1,9 +1,9 @@
-"""Decoder layers of latent or grouped attention with a dense or routed feed-forward each: weights, workspace and the kernel sequence of
+"""Decoder layers of latent, grouped or lightning attention with a dense or routed feed-forward each: weights, workspace and the kernel sequence of
 `CudaModel` for such models.
 
 Per layer (the residual stream h is fp32, everything else bf16, or float in 32-bit mode):
 
-    o = attention(xn)                                           engine/latent.py, engine/grouped.py
+    o = attention(xn)                                           engine/latent.py, grouped.py, linear.py
     y = Wo o ; h += norm(y) ; xn = norm(h)                      resid_norm
     act = a(Wg xn) * (Wu xn) ; y = Wd act                       fused into the product up to eight rows; or engine/experts.py
     h += norm(y) ; xn = norm(h) of the next layer               resid_norm (sums the chosen experts' rows first)
@@ -17,12 +17,13 @@ from dataclasses import dataclass
 
 import torch
 
-from ..models.config import GroupedAttention, LatentAttention, Rotary
-from ..models.mixers import mixer_kv_shapes
+from ..models.config import GroupedAttention, LatentAttention, LightningAttention, Rotary
+from ..models.mixers import has_state, mixer_kv_shapes, mixer_state_shapes, run_kv_layers
 from .dense import DenseLinear
 from .experts import RoutedExperts
 from .grouped import GroupedMixer, padded_head
 from .latent import PART_FLOATS, LatentMixer, LatentPlan
+from .linear import SHORT_ROWS, LightningMixer
 
 
 @dataclass
@@ -30,6 +31,8 @@ class StackPlan:
     """What the layers of one forward call share."""
     angles: list[torch.Tensor]                       # per distinct rotation: [T, dims/2, 2]
     latent: LatentPlan | None = None
+    chunks: tuple | None = None                      # how the chunk kernels of a recurrence cut the batch (None: row after row)
+    values: torch.Tensor | None = None               # of the first layer whose values later ones mix in
 
 
 class AttentionStack:
@@ -48,17 +51,21 @@ class AttentionStack:
         self.embed_norm = self.vec(weights, "token_embd_norm.weight") if c.embed_norm else None
         self.loop_in = DenseLinear(self.mat(weights, "loop_in.weight")) if c.loop else None
         self.loop_step = self.mat(weights, "loop_step.weight") if c.loop_steps else None
-        self.act = {"silu": ops.ACT_SILU_MUL, "gelu_tanh": ops.ACT_GELU_MUL}[c.ffn_act]
+        self.act = {"silu": ops.ACT_SILU_MUL, "gelu_tanh": ops.ACT_GELU_MUL, "gelu_up": ops.ACT_GELU}[c.ffn_act]
         from .. import ops as base
         self.scratch = base.scratch_for(self.device)
         self.status = self.scratch.status                               # word that a kernel sets when a bounded wait runs out
         self.runs = c.layer_runs()                                      # looped layers have a cache layer per pass
-        self.kv_layer_shapes = mixer_kv_shapes(c, lambda size: padded_head(size, self.f32))
-        self.state_shapes = None
-        self.n_kv_layers = len(self.runs)
+        head_pad = lambda size: padded_head(size, self.f32)
+        self.kv_layer_shapes, self.kv_index = mixer_kv_shapes(c, head_pad), run_kv_layers(c)
+        self.state_shapes = mixer_state_shapes(c, 8, head_pad)
+        self.state_index = [sum(has_state(m) for m in c.mixers[:i]) for i in range(c.n_layers)]
+        self.n_kv_layers = len(self.kv_layer_shapes)
+        self.linear_tc = True                                           # tcgen05 form of the recurrence over prompts where the sizes fit
         self.rotaries: list[Rotary] = []
         self.freqs: list[torch.Tensor] = []
-        self.has_latent = any(isinstance(m, LatentAttention) for m in c.mixers)
+        self.has_latent, self.has_linear = (any(isinstance(m, kind) for m in c.mixers) for kind in (LatentAttention, LightningAttention))
+        self.one = torch.ones(1, dtype=torch.float32, device=self.device)
 
     def mat(self, w, name: str) -> torch.Tensor:
         return w[name].to_float().to(self.device).to(self.dtype)
@@ -77,20 +84,29 @@ class AttentionStack:
         return self.embed if self.cfg.tie_embeddings else self.mat(w, "output.weight")
 
     # -- weights ---------------------------------------------------------------------------------------------
-    def build_layer(self, L, w, i: int):
+    def build_parts(self, L, w, i: int) -> None:
+        """A layer's mixer and feed-forward."""
         c, m, p = self.cfg, self.cfg.mixers[i], f"blk.{i}."
         L.index = i
-        L.attn_norm, L.post_attn_norm = self.vec(w, p + "attn_norm.weight"), self.vec(w, p + "post_attention_norm.weight")
-        L.mix = (GroupedMixer if isinstance(m, GroupedAttention) else LatentMixer)(self, w, p, m)
+        if isinstance(m, LightningAttention):
+            L.mix = LightningMixer(self, w, p, m, self.state_index[i])
+        else:
+            L.mix = GroupedMixer(self, w, p, m, self.state_index[i]) if isinstance(m, GroupedAttention) else LatentMixer(self, w, p, m)
         L.ff, e = c.ff_width(i), c.experts_of(i)
         L.experts = RoutedExperts(self, w, p, e) if e else None
         if L.experts:
             L.experts.layer = i
-        if L.ff or e:
-            L.ffn_norm, L.post_ffn_norm = self.vec(w, p + "ffn_norm.weight"), self.vec(w, p + "post_ffw_norm.weight")
         if L.ff:
-            L.gate_up = DenseLinear(torch.cat([self.mat(w, p + "ffn_gate.weight"), self.mat(w, p + "ffn_up.weight")]))
+            up = self.mat(w, p + "ffn_up.weight")
+            L.gate_up = DenseLinear(up if c.ffn_act == "gelu_up" else torch.cat([self.mat(w, p + "ffn_gate.weight"), up]))
             L.down = DenseLinear(self.mat(w, p + "ffn_down.weight"))
+
+    def build_layer(self, L, w, i: int):
+        p = f"blk.{i}."
+        self.build_parts(L, w, i)
+        L.attn_norm, L.post_attn_norm = self.vec(w, p + "attn_norm.weight"), self.vec(w, p + "post_attention_norm.weight")
+        if L.ff or L.experts:
+            L.ffn_norm, L.post_ffn_norm = self.vec(w, p + "ffn_norm.weight"), self.vec(w, p + "post_ffw_norm.weight")
         return L
 
     def nbytes(self, layers) -> int:
@@ -132,7 +148,7 @@ class AttentionStack:
             if r + 1 < len(self.runs):
                 to_pass = self.runs[r + 1][1]
                 nxt = None if to_pass else layers[self.runs[r + 1][0]].attn_norm
-            self.layer(L, h, fb, plan, kv.layers[r], nxt, to_pass)
+            self.layer(L, h, fb, plan, kv, r, nxt, to_pass)
             after_layer(r, h)
 
     def plan(self, fb, T: int, layers) -> StackPlan:
@@ -145,7 +161,15 @@ class AttentionStack:
         plan = StackPlan(angles)
         if self.has_latent:
             plan.latent = LatentPlan.build(fb, T, all(L.mix.chunk_fits for L in layers if isinstance(L.mix, LatentMixer)), self.device)
+        if self.has_linear and not self.f32 and not fb.is_decode and self.linear_tc and fb.max_q_len > SHORT_ROWS:
+            from ..ops import mixers as mixer_ops
+            plan.chunks = mixer_ops.chunk_tables(fb.host_cu if fb.host_cu is not None else fb.cu_q.tolist(), self.device)
         return plan
+
+    def mix(self, L, xn: torch.Tensor, fb, plan: StackPlan, kv, run: int) -> torch.Tensor:
+        """A layer run's mixer up to its output product."""
+        at = self.kv_index[run]
+        return L.mix(xn, fb, plan, kv, kv.layers[at] if at is not None else None)
 
     def embed_tokens(self, tokens: torch.Tensor, h: torch.Tensor, first_norm: torch.Tensor | None) -> None:
         """h = the (normed) embedding; ``first_norm``: the first layer's input norm (None: a loop pass comes first)."""
@@ -171,11 +195,11 @@ class AttentionStack:
         ops.resid_norm(h, y, w_post, w_next=w_next, xn=self.xn[:T] if w_next is not None else None,
                        copy0=self.cat[:T, :d] if to_pass else None, eps=self.cfg.rms_eps, y_rows=y_rows, y_w=y_w)
 
-    def layer(self, L, h: torch.Tensor, fb, plan: StackPlan, kv_layer: torch.Tensor, next_norm: torch.Tensor | None, to_pass: bool) -> None:
+    def layer(self, L, h: torch.Tensor, fb, plan: StackPlan, kv, run: int, next_norm: torch.Tensor | None, to_pass: bool) -> None:
         """xn holds the normed input; ``next_norm``: input norm of the layer that follows (None: a loop pass, or the end)."""
         T = h.shape[0]
         xn, y = self.xn[:T], self.y[:T]
-        L.mix.wo(L.mix(xn, fb, plan, kv_layer), y)
+        L.mix.wo(self.mix(L, xn, fb, plan, kv, run), y)
         if not L.ff and L.experts is None:
             self._join(h, y, L.post_attn_norm, next_norm, to_pass)
             return

@@ -13,7 +13,7 @@ import torch
 import torch.nn.functional as F
 
 from ..models import gdn, mixers
-from ..models.config import LatentAttention, MatrixLSTM, ModelConfig
+from ..models.config import LatentAttention, LightningAttention, MatrixLSTM, ModelConfig
 from ..models.reference import moe_route, rmsnorm, rope_split_half
 from ..models.weights import ModelWeights
 from ..parallel.tp_plan import TPPlan
@@ -122,35 +122,45 @@ class TorchPagedModel:
     def weight_bytes(self) -> int:
         return 0
 
-    # -- layers of latent or grouped attention ----------------------------------------------------------
+    # -- layers of latent, grouped or lightning attention ----------------------------------------------------------
     def _init_attention_stack(self, f) -> None:
         c = self.cfg
         self.embed_norm = f("token_embd_norm.weight") if c.embed_norm else None
         self.loop_in = f("loop_in.weight") if c.loop else None
         self.loop_step = f("loop_step.weight") if c.loop_steps else None
         latent = {"qa": "attn_q_a", "qan": "attn_q_a_norm", "qb": "attn_q_b", "kva": "attn_kv_a", "kvan": "attn_kv_a_norm", "kb": "attn_k_b", "vb": "attn_v_b"}
-        grouped = {"wq": "attn_q", "wk": "attn_k", "wv": "attn_v", "qn": "attn_q_norm", "kn": "attn_k_norm"}
-        dense = {"wg": "ffn_gate", "wu": "ffn_up", "wd": "ffn_down"}
+        self.positions = f("position_embd.weight") if c.learned_positions else None
+        dense = {"wu": "ffn_up", "wd": "ffn_down", **({} if c.ffn_act == "gelu_up" else {"wg": "ffn_gate"})}
         experts = {"router": "ffn_gate_inp", "wg": "ffn_gate_exps", "wu": "ffn_up_exps", "wd": "ffn_down_exps"}
-        self.layers = []
+        self.layers, n_states = [], 0
         for i in self.layer_ids:
             m, e = c.mixers[i], c.experts_of(i)
-            is_latent = isinstance(m, LatentAttention)
-            want = {"attn_norm": "attn_norm", "post_attn": "post_attention_norm", "wo": "attn_output", **(latent if is_latent else grouped)}
-            if is_latent and m.sinks:
-                want["sink"] = "attn_sinks"
-            if m.gated if is_latent else m.gate:
-                want["gate"] = "attn_gate"
+            want = {"attn_norm": "attn_norm", **({"post_attn": "post_attention_norm"} if c.post_norms else {})}
+            if isinstance(m, LatentAttention):
+                want.update(wo="attn_output", **latent, **({"sink": "attn_sinks"} if m.sinks else {}), **({"gate": "attn_gate"} if m.gated else {}))
+            elif isinstance(m, LightningAttention):
+                want.update(wq="lin_q", wk="lin_k", wv="lin_v", gate="lin_g", on="lin_norm", wo="lin_output")
+            else:
+                want.update(wq="attn_q", wk="attn_k", wv="attn_v", wo="attn_output")
+                for on, names in ((m.gate, {"gate": "attn_gate"}), (m.qk_norm, {"qn": "attn_q_norm", "kn": "attn_k_norm"}), (m.temperature, {"temp": "attn_temperature"}),
+                                  (m.conv, {"cq": "attn_q_conv", "ck": "attn_k_conv", "cv": "attn_v_conv"}), (m.value_mix, {"vmix": "attn_value_mix"})):
+                    want.update(names if on else {})
             if c.ff_width(i) or e:
-                want.update({"ffn_norm": "ffn_norm", "post_ffn": "post_ffw_norm", **(experts if e else dense)})
+                want.update({"ffn_norm": "ffn_norm", **({"post_ffn": "post_ffw_norm"} if c.post_norms else {}), **(experts if e else dense)})
+            if c.depth_average:
+                want["depth"] = "depth_average"
             L = {k: f(f"blk.{i}.{n}.weight") for k, n in want.items()}
             if e:
-                L["router_bias"] = f(f"blk.{i}.ffn_gate_inp.bias")
-            L.update(index=i, mixer=m, experts=e, freqs=torch.tensor(m.rotary.frequencies(), dtype=torch.float64, device=self.device))
+                L["router_bias"] = f(f"blk.{i}.ffn_gate_inp.bias") if e.bias else 0.0
+            L.update(index=i, mixer=m, experts=e, state=n_states)
+            n_states += mixers.has_state(m)
+            if not isinstance(m, LightningAttention):
+                L["freqs"] = torch.tensor(m.rotary.frequencies(), dtype=torch.float64, device=self.device)
             self.layers.append(L)
         self.runs = c.layer_runs()
-        self.kv_layer_shapes = mixers.mixer_kv_shapes(c)
-        self.n_kv_layers = self.mtp_kv_base = len(self.runs)
+        self.kv_layer_shapes, self.state_shapes = mixers.mixer_kv_shapes(c), mixers.mixer_state_shapes(c)
+        self.kv_index = mixers.run_kv_layers(c)
+        self.n_kv_layers = self.mtp_kv_base = len(self.kv_layer_shapes)
         self.mtp_layers, self.hybrid_dims = [], None
 
     @staticmethod
@@ -209,16 +219,43 @@ class TorchPagedModel:
             v = v * torch.sigmoid(x @ L["gate"].T)
         return v @ L["wo"].T
 
-    def _grouped_attention(self, L, x: torch.Tensor, fb: ForwardBatch, kvl: torch.Tensor) -> torch.Tensor:
+    def _conv_rows(self, L, u: torch.Tensor, w: torch.Tensor, at: int, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        """The convolution of projected rows u [T, n], channels ``at`` and on of the layer's; w [n, taps].  The state keeps the last
+        rows of a sequence, position p in place p mod taps."""
+        taps, n, out = w.shape[1], u.shape[1], torch.empty_like(u)
+        ring = kv.hybrid.layers[L["state"]][0][:, :, at:at + n]
+        for r0, r1, slot, _ in gdn.batch_sequences(fb.seq_ids, fb.positions, fb.state_slots):
+            p0 = int(fb.positions[r0])
+            past = torch.tensor([p for p in range(p0 - taps + 1, p0)], dtype=torch.long)
+            before = ring[slot, past % taps] * (past >= 0)[:, None]
+            out[r0:r1] = mixers.short_conv(u[r0:r1], before, w.T)
+            for r in range(max(r0, r1 - taps + 1), r1):
+                ring[slot, (p0 + r - r0) % taps] = u[r]
+        return out
+
+    def _grouped_attention(self, L, x: torch.Tensor, fb: ForwardBatch, kvl: torch.Tensor, kv: PagedKVCache | None = None, shared: dict | None = None) -> torch.Tensor:
+        """``shared``: what layers of one forward call hand on (the values that later ones mix in)."""
         c, m, T = self.cfg, L["mixer"], x.shape[0]
         pos, sid = fb.positions.long(), fb.seq_ids.long()
         ang = pos.double()[:, None] * L["freqs"]
-        turn = lambda y: self._turn(y, ang.cos().float()[:, None], ang.sin().float()[:, None], m.rotary.interleaved)
-        q = turn(rmsnorm((x @ L["wq"].T).view(T, m.heads, m.dim), L["qn"], c.rms_eps)).view(T, m.kv_heads, -1, m.dim)
-        k = turn(rmsnorm((x @ L["wk"].T).view(T, m.kv_heads, m.dim), L["kn"], c.rms_eps))
+        cos, sin = (ang.cos() * m.rotary.magnitude).float()[:, None], (ang.sin() * m.rotary.magnitude).float()[:, None]
+        turn = lambda y: self._turn(y, cos, sin, m.rotary.interleaved)
+        q, k, v = x @ L["wq"].T, x @ L["wk"].T, x @ L["wv"].T
+        if m.conv:
+            q, k, v = (self._conv_rows(L, u, L[w], at, fb, kv) for u, w, at in ((q, "cq", 0), (k, "ck", q.shape[1]), (v, "cv", q.shape[1] + k.shape[1])))
+        q, k = q.view(T, m.heads, m.dim), k.view(T, m.kv_heads, m.dim)
+        if m.qk_norm:
+            q, k = rmsnorm(q, L["qn"], c.rms_eps), rmsnorm(k, L["kn"], c.rms_eps)
+        q, k = turn(q), turn(k)
+        if m.temperature:
+            q = q * L["temp"][:, None]
+        q = q.view(T, m.kv_heads, -1, m.dim)
+        if m.value_mix:
+            first = shared.setdefault("values", v)
+            v = v if first is v else torch.lerp(v, first, L["vmix"])
         page, off = fb.block_table.long()[sid, pos // PAGE_SIZE], pos % PAGE_SIZE
         kvl[page, 0, :, off, :m.dim] = k.to(kvl.dtype)
-        kvl[page, 1, :, off, :m.vdim] = (x @ L["wv"].T).view(T, m.kv_heads, m.vdim).to(kvl.dtype)
+        kvl[page, 1, :, off, :m.vdim] = v.view(T, m.kv_heads, m.vdim).to(kvl.dtype)
         out = torch.empty(T, m.heads, m.vdim)
         for b in sid.unique().tolist():
             rows = (sid == b).nonzero(as_tuple=True)[0]
@@ -238,19 +275,61 @@ class TorchPagedModel:
             out = out * torch.sigmoid(x @ L["gate"].T).view(T, m.heads, -1)            # one per head or one per value
         return out.reshape(T, -1) @ L["wo"].T
 
+    def _lightning(self, L, x: torch.Tensor, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        m, T = L["mixer"], x.shape[0]
+        q, k, v = (F.silu(x @ L[n].T).view(T, m.heads, -1) for n in ("wq", "wk", "wv"))
+        decay, (S,), o = torch.tensor(m.decay), kv.hybrid.layers[L["state"]], torch.empty_like(v)
+        for r0, r1, slot, fresh in gdn.batch_sequences(fb.seq_ids, fb.positions, fb.state_slots):
+            if fresh:
+                S[slot].zero_()
+            o[r0:r1] = mixers.retention_rows(q[r0:r1], k[r0:r1], v[r0:r1], decay, S[slot])
+        return (rmsnorm(o.reshape(T, -1), L["on"], self.cfg.rms_eps) * torch.sigmoid(x @ L["gate"].T)) @ L["wo"].T
+
     def _routed_experts(self, L, x: torch.Tensor) -> torch.Tensor:
         e = L["experts"]
-        best = (x @ L["router"].T + L["router_bias"]).topk(e.top, dim=-1)
+        z = x @ L["router"].T + L["router_bias"]
+        if e.keep < e.groups:
+            groups = z.view(-1, e.groups, e.n // e.groups).amax(-1).topk(e.keep, dim=-1).indices
+            kept = torch.zeros(z.shape[0], e.groups, dtype=torch.bool).scatter_(1, groups, True)
+            z = z.masked_fill(~kept.repeat_interleave(e.n // e.groups, dim=1), float("-inf"))
+        best = z.topk(e.top, dim=-1)
         wt, out = torch.softmax(best.values, dim=-1), torch.zeros_like(x)
         if getattr(self, "expert_stats", None) is not None:
             self.expert_stats.record(L["index"], best.indices)
         for j in best.indices.unique().tolist():
             tok, slot = (best.indices == j).nonzero(as_tuple=True)
-            y = (F.silu(x[tok] @ L["wg"][j].T) * (x[tok] @ L["wu"][j].T)) @ L["wd"][j].T
+            g, u = x[tok] @ L["wg"][j].T, x[tok] @ L["wu"][j].T
+            y = (mixers.limited_pair(g, u, e.limit) if e.limit else F.silu(g) * u) @ L["wd"][j].T
             out.index_add_(0, tok, y * wt[tok, slot].unsqueeze(-1))
         return out
 
+    def _run_parallel_stack(self, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        """Mixer and feed-forward side by side on the same input, a weighted sum over depth behind every layer."""
+        c, eps, shared = self.cfg, self.cfg.rms_eps, {}
+        h = self.embed[fb.tokens.long()].float()
+        if c.learned_positions:
+            h = h + self.positions[fb.positions.long()]
+        streams = [h]
+        for r, L in enumerate(self.layers):
+            x = rmsnorm(h, L["attn_norm"], eps)
+            if isinstance(L["mixer"], LightningAttention):
+                y = self._lightning(L, x, fb, kv)
+            else:
+                y = self._grouped_attention(L, x, fb, kv.layers[self.kv_index[r]], kv, shared)
+            if "wu" in L:
+                x = rmsnorm(h, L["ffn_norm"], eps)
+                y = y + (self._routed_experts(L, x) if L["experts"] else F.gelu(x @ L["wu"].T, approximate="tanh") @ L["wd"].T)
+            h = h + y
+            if c.depth_average:
+                streams.append(h)
+                h = torch.einsum("j,jtd->td", L["depth"], torch.stack(streams))
+            if getattr(self, "taps", None) is not None:
+                self.taps[f"layer{r}"] = h.clone()
+        return h
+
     def _run_attention_stack(self, fb: ForwardBatch, kv: PagedKVCache) -> torch.Tensor:
+        if self.cfg.parallel_ff:
+            return self._run_parallel_stack(fb, kv)
         c, eps, n_pass = self.cfg, self.cfg.rms_eps, 0
         act = F.silu if c.ffn_act == "silu" else lambda z: F.gelu(z, approximate="tanh")
         x0 = self.embed[fb.tokens.long()].float()
@@ -265,7 +344,7 @@ class TorchPagedModel:
                     h = h + self.loop_step[n_pass]
                 n_pass += 1
             mix = self._latent_attention if isinstance(L["mixer"], LatentAttention) else self._grouped_attention
-            h = h + rmsnorm(mix(L, rmsnorm(h, L["attn_norm"], eps), fb, kv.layers[r]), L["post_attn"], eps)
+            h = h + rmsnorm(mix(L, rmsnorm(h, L["attn_norm"], eps), fb, kv.layers[self.kv_index[r]]), L["post_attn"], eps)
             if "wg" in L:
                 x = rmsnorm(h, L["ffn_norm"], eps)
                 y = self._routed_experts(L, x) if L["experts"] else (act(x @ L["wg"].T) * (x @ L["wu"].T)) @ L["wd"].T

@@ -13,7 +13,7 @@ from dataclasses import asdict, dataclass, field, replace
 
 from ..gguf.constants import GGMLType
 
-SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik", "zogepel", "kefasun")
+SUPPORTED_ARCHS = ("qwen2", "qwen3", "qwen3moe", "qwen35", "qwen35moe", "pozivik", "zogepel", "kefasun", "lagedra")
 
 
 @dataclass(frozen=True)
@@ -92,8 +92,8 @@ class LatentAttention:
 
 @dataclass(frozen=True)
 class GroupedAttention:
-    """Grouped-query softmax attention with per-head keys and values in the paged cache.  Queries and keys are RMS-normed per head
-    (one gain per value, shared by the heads), then rotated."""
+    """Grouped-query softmax attention with per-head keys and values in the paged cache.  Queries and keys are rotated, in front of
+    that RMS-normed per head (one gain per value, shared by the heads) or passed through a short causal convolution per channel."""
     heads: int
     kv_heads: int
     dim: int
@@ -105,6 +105,10 @@ class GroupedAttention:
     softcap: float = 0.0            # scores s become softcap * tanh(s / softcap) (0: as they are)
     null_key: bool = False          # one joins the softmax denominator (a key with score 0 and no value)
     gate: str = ""                  # "head" | "value": sigmoid of a projection of the input, per head or per value, before the output projection
+    qk_norm: bool = True
+    conv: int = 0                   # taps of the convolution over time on the projected queries, keys and values (0: none)
+    temperature: bool = False       # one learned factor per query head on the scores, before the soft cap
+    value_mix: bool = False         # the first such layer's values of a token join this layer's: v = (1 - share) v + share v_first
 
     @property
     def head_size(self) -> int:
@@ -118,10 +122,19 @@ class GroupedAttention:
 
 @dataclass(frozen=True)
 class Experts:
-    """Mixture-of-experts feed-forward: the `top` experts with the largest router logits, weighted by the softmax over just those."""
+    """Mixture-of-experts feed-forward: the `top` experts with the largest router logits, weighted by the softmax over just those (or
+    over all experts and divided by the chosen ones' sum: the same weights).  With several `groups` of neighbours only experts of
+    the `keep` groups whose best experts are largest can be chosen.
+
+    An expert is silu(gate) * up, or with a `limit` g sigmoid(1.702 g) (u + 1) of g = min(gate, limit) and u = up clamped to
+    [-limit, limit]."""
     n: int
     top: int
     ff: int
+    groups: int = 1
+    keep: int = 1
+    limit: float = 0.0
+    bias: bool = True               # on the router logits
 
 
 @dataclass(frozen=True)
@@ -147,6 +160,16 @@ class Retention:
     vdim: int
     decay: tuple[float, ...]        # per head
     rotary: Rotary
+
+
+@dataclass(frozen=True)
+class LightningAttention:
+    """Linear attention S_t = decay_h S_(t-1) + k_t v_t^T with silu on queries, keys and values, no rotation, scale or denominator; the
+    concatenated heads are RMS-normed together (a gain per value) and gated by a sigmoid."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: tuple[float, ...]        # per head
 
 
 @dataclass(frozen=True)
@@ -205,10 +228,10 @@ class ModelConfig:
     ssm_k_heads: int = 0
     ssm_v_heads: int = 0
     rope_dim: int = 0                    # leading dims of each head that are rotated (0: all of head_dim)
-    # layer lists with their own sizes per layer (pozivik, zogepel, kefasun): the mixer of every layer, its feed-forward width (0:
+    # layer lists with their own sizes per layer (pozivik, zogepel, kefasun, lagedra): the mixer of every layer, its feed-forward width (0:
     # none) or experts, and the layers [start, stop) that run `times` times in a row, each pass behind a projection of
     # [hidden | embedding] (and a vector of its own)
-    mixers: tuple[LatentAttention | GroupedAttention | MatrixLSTM | ParallelMixers, ...] = ()
+    mixers: tuple[LatentAttention | GroupedAttention | LightningAttention | MatrixLSTM | ParallelMixers, ...] = ()
     layer_ff: tuple[int, ...] = ()
     layer_experts: tuple[Experts | None, ...] = ()
     loop: tuple[int, int, int] | None = None
@@ -222,7 +245,11 @@ class ModelConfig:
     layer_scale: bool = False            # a gain per value on every sublayer's (normed) output
     residual_mult: float = 1.0           # factor on what joins the residual stream
     side_dim: int = 0                    # width of the per-layer token input behind the feed-forward (0: none)
-    ffn_act: str = "silu"                # silu | gelu_tanh: activation of the gated feed-forward; relu2: ungated, squared relu
+    ffn_act: str = "silu"                # silu | gelu_tanh: activation of the gated feed-forward; relu2 (squared relu), gelu_up (gelu_tanh): ungated
+    scalar_norms: bool = False           # one gain for all values in the norms of the residual stream
+    parallel_ff: bool = False            # mixer and feed-forward read the same input, each through a norm of its own
+    depth_average: bool = False          # behind layer i: a learned weighted sum of the embedding and the results of layers 0 .. i
+    learned_positions: int = 0           # rows of the table of position vectors that are added to the embedding (0: none)
     attn_gate: bool = False              # attn_q holds [q | gate] per head; the attention output is scaled by sigmoid(gate)
     name: str = "tiny-qwen3"
 
@@ -240,8 +267,8 @@ class ModelConfig:
 
     @property
     def is_attention_stack(self) -> bool:
-        """Layers of latent or grouped attention with a feed-forward each, norms around both, and loops."""
-        return self.has_mixers and all(isinstance(m, (LatentAttention, GroupedAttention)) for m in self.mixers)
+        """Layers of latent, grouped or lightning attention with a feed-forward each, norms around both, and loops."""
+        return self.has_mixers and all(isinstance(m, (LatentAttention, GroupedAttention, LightningAttention)) for m in self.mixers)
 
     @property
     def has_mixers(self) -> bool:
@@ -251,7 +278,8 @@ class ModelConfig:
     @property
     def has_state(self) -> bool:
         """Some layer carries a recurrent state from token to token, in a slot per sequence."""
-        return self.is_hybrid or any(isinstance(p, (Retention, MatrixLSTM)) for m in self.mixers for p in mixer_parts(m))
+        return self.is_hybrid or any(isinstance(p, (Retention, MatrixLSTM, LightningAttention)) or (isinstance(p, GroupedAttention) and p.conv > 0)
+                                     for m in self.mixers for p in mixer_parts(m))
 
     def layer_runs(self) -> list[tuple[int, bool]]:
         """The layers in the order they run: (layer, whether a pass over the looped layers starts before it).  Every run has a
@@ -315,7 +343,7 @@ class ModelConfig:
         if arch not in SUPPORTED_ARCHS:
             raise ValueError(f"unsupported GGUF architecture '{arch}' (supported: {', '.join(SUPPORTED_ARCHS)}; "
                              "qwen35 / qwen35moe are the hybrid Gated-DeltaNet families)")
-        if arch in ("pozivik", "zogepel", "kefasun"):
+        if arch in ("pozivik", "zogepel", "kefasun", "lagedra"):
             return family_of(arch).config_from_json(json.loads(gf.get(f"{arch}.config")))
         a = gf.arch_key
 
@@ -497,6 +525,19 @@ def attention_stack(name: str, d_model: int, mixers: tuple, ffs: tuple, vocab: i
                        loop_steps=loop is not None, **KEFASUN)
 
 
+def parallel_stack(name: str, d_model: int, mixers: tuple, ffs: tuple, vocab: int, max_positions: int, eps: float = 1e-6) -> ModelConfig:
+    """A lagedra shape; ``ffs``: the width or the `Experts` of every layer (0: no feed-forward)."""
+    a = next((m for m in mixers if isinstance(m, GroupedAttention)), None)
+    m = a or mixers[0]
+    return ModelConfig(name=name, arch="lagedra", n_layers=len(mixers), d_model=d_model, n_heads=m.heads, n_kv_heads=a.kv_heads if a else 1,
+                       head_dim=a.head_size if a else m.dim, d_ff=max((f for f in ffs if isinstance(f, int)), default=0), vocab_size=vocab,
+                       rope_theta=a.rotary.base if a else 1e4, rms_eps=eps, context_length=max_positions, mixers=mixers,
+                       layer_ff=tuple(0 if isinstance(f, Experts) else f for f in ffs),
+                       layer_experts=tuple(f if isinstance(f, Experts) else None for f in ffs), learned_positions=max_positions, **LAGEDRA)
+
+
+# what every lagedra model has in common
+LAGEDRA = dict(qk_norm=False, tie_embeddings=False, ffn_act="gelu_up", scalar_norms=True, parallel_ff=True, depth_average=True)
 # what every kefasun model has in common
 KEFASUN = dict(qk_norm=False, tie_embeddings=True, post_norms=True, ffn_act="silu")
 # what every zogepel model has in common
@@ -546,6 +587,13 @@ SHAPES = {
                                   GroupedAttention(32, 8, 128, 128, 128 ** -0.5, Rotary(128, 8e5), softcap=40.0, gate="value"),
                                   LatentAttention(32, 128, 64, 128, 1536, 512, 192 ** -0.5, Rotary(64, 2e5, interleaved=True), 1024, gated=True)) * 4,
                                   (12288, Experts(32, 4, 1536), Experts(32, 4, 1536), Experts(32, 4, 1536)) * 4, 151936),
+    "tiny-lagedra": parallel_stack("tiny-lagedra", 256, (LightningAttention(4, 32, 64, (0.8, 0.95, 0.99, 0.998)), GroupedAttention(
+                                   4, 2, 64, 48, 0.125, Rotary(64, 1e4, RopeScaling(4.0, 256, 32.0, 1.0)), 100, softcap=30.0, qk_norm=False, conv=4, temperature=True, value_mix=True)) * 2,
+                                   (512, Experts(8, 2, 128, 4, 2, 4.0, False), Experts(6, 3, 96, 2, 1, 7.0, False), 384), 1024, 4096),
+    # layers of qwen3-8b's width, heads, feed-forward width and vocabulary: lightning and windowed attention in turns, experts in every other layer
+    "lagedra-8b": parallel_stack("lagedra-8b", 4096, (LightningAttention(16, 128, 256, tuple(1.0 - 2.0 ** (-3.0 - i / 2) for i in range(16))), GroupedAttention(
+                                 32, 8, 128, 128, 128 ** -0.5, Rotary(128, 2e5, RopeScaling(8.0, 4096, 32.0, 1.0)), 1024, softcap=30.0, qk_norm=False, conv=4, temperature=True,
+                                 value_mix=True)) * 8, (12288, Experts(32, 4, 1536, 8, 4, 7.0, False), Experts(32, 4, 1536, 8, 4, 7.0, False), 12288) * 4, 151936, 32768),
     "tiny-zogepel": mixed_shape("tiny-zogepel", 256, (MatrixLSTM(4, 32, 64, 12.0), ParallelMixers(WindowAttention(4, 2, 64, 0.125, 96), Retention(
                                 4, 32, 48, (0.9, 0.97, 0.99, 0.998), Rotary(24, 1e4)))) * 2, 512, 1024, 32),
     # layers of qwen3-8b's width, feed-forward width and vocabulary, alternating

@@ -260,7 +260,7 @@ def requantize(w: ModelWeights, recipe: QuantRecipe | str) -> ModelWeights:
     cfg, out = w.config, {}
     for name, t in w.tensors.items():
         layer = int(name.split(".")[1]) if name.startswith("blk.") else None
-        if len(t.shape) < 2 or "ssm_conv1d" in name:
+        if len(t.shape) < 2 or "ssm_conv1d" in name or "_conv." in name:
             out[name] = t
         else:
             out[name] = t.transcoded(_fit(recipe.for_tensor(name, layer, cfg.n_layers), t.shape[-1]))

@@ -5,7 +5,7 @@ Per head, with log input gate i, log forget gate f and running maximum m (which 
 
     mLSTM       m' = max(f + m, i);  S' = e^(f+m-m') S + e^(i-m') v k^T;  n' = e^(f+m-m') n + e^(i-m') k
                 o = S' q / (max(|n'.q|, e^-m') + NORM_FLOOR)
-    retention   S' = decay S + v k^T;  o = S' q
+    retention   S' = decay S + v k^T;  o = S' q            (lightning attention the same)
 
 The state matrix is held as [vdim, dim]: a row per value, so that reading it out is a product with q along contiguous memory.
 """
@@ -14,7 +14,7 @@ from __future__ import annotations
 import torch
 import torch.nn.functional as F
 
-from .config import GroupedAttention, LatentAttention, MatrixLSTM, ModelConfig, ParallelMixers, Retention, WindowAttention, mixer_parts
+from .config import GroupedAttention, LatentAttention, LightningAttention, MatrixLSTM, ModelConfig, ParallelMixers, Retention, WindowAttention, mixer_parts
 
 NORM_FLOOR = 1e-6
 
@@ -35,16 +35,38 @@ def mixer_kv_shapes(cfg: ModelConfig, head_pad=lambda dim: dim) -> list[tuple[in
     return out
 
 
-def state_shapes_of(m, pad: int = 1) -> tuple[tuple[int, ...], ...]:
+def conv_columns(m: GroupedAttention, head_size: int) -> int:
+    """Channels of the convolution in front of an attention layer whose heads take `head_size` columns each."""
+    return (m.heads + 2 * m.kv_heads) * head_size
+
+
+def run_kv_layers(cfg: ModelConfig) -> list[int | None]:
+    """The cache layer of every layer run (None: its mixer has no cache)."""
+    out, n = [], 0
+    for i, _ in cfg.layer_runs():
+        cached = isinstance(cfg.mixers[i], (LatentAttention, GroupedAttention))
+        out.append(n if cached else None)
+        n += cached
+    return out
+
+
+def state_shapes_of(m, pad: int = 1, head_pad=lambda dim: dim) -> tuple[tuple[int, ...], ...]:
+    if isinstance(m, GroupedAttention):             # the last projected rows: position p in place p mod taps
+        return ((m.conv, conv_columns(m, head_pad(m.head_size))),)
     d, v = pad_to_multiple(m.dim, pad), pad_to_multiple(m.vdim, pad)
     if isinstance(m, MatrixLSTM):
         return (m.heads, v, d), (m.heads, d), (m.heads,)
     return ((m.heads, v, d),)
 
 
-def mixer_state_shapes(cfg: ModelConfig, pad: int = 1) -> list[tuple[tuple[int, ...], ...]]:
-    """Shapes of the state tensors of every recurrent mixer, in layer order; sizes rounded up to a multiple of ``pad``."""
-    return [state_shapes_of(p, pad) for m in cfg.mixers for p in mixer_parts(m) if isinstance(p, (MatrixLSTM, Retention))]
+def has_state(m) -> bool:
+    """Whether an elementary mixer carries something from token to token besides its cache entries."""
+    return isinstance(m, (MatrixLSTM, Retention, LightningAttention)) or (isinstance(m, GroupedAttention) and m.conv > 0)
+
+
+def mixer_state_shapes(cfg: ModelConfig, pad: int = 1, head_pad=lambda dim: dim) -> list[tuple[tuple[int, ...], ...]]:
+    """Shapes of the state tensors of every mixer with a state, in layer order; sizes rounded up to a multiple of ``pad``."""
+    return [state_shapes_of(p, pad, head_pad) for m in cfg.mixers for p in mixer_parts(m) if has_state(p)]
 
 
 def mixer_columns(m) -> int:
@@ -57,13 +79,19 @@ def mixer_columns(m) -> int:
         return (3 * m.heads + 2 * m.kv_heads) * m.head_size + m.gate_width
     if isinstance(m, LatentAttention):
         return m.heads * (2 * m.dim + m.rot_dim + (3 if m.gated else 2) * m.vdim) + 2 * m.q_rank + 2 * m.cache_width
-    if isinstance(m, (MatrixLSTM, Retention)):
+    if isinstance(m, (MatrixLSTM, Retention, LightningAttention)):
         return m.heads * (2 * m.dim + 4 * m.vdim)
     return 0
 
 
 def soft_cap(x: torch.Tensor, cap: float) -> torch.Tensor:
     return cap * torch.tanh(x / cap)
+
+
+def limited_pair(g: torch.Tensor, u: torch.Tensor, limit: float) -> torch.Tensor:
+    """Gated pair of clamped values (see `Experts.limit`)."""
+    g, u = g.clamp(max=limit), u.clamp(min=-limit, max=limit)
+    return g * torch.sigmoid(1.702 * g) * (u + 1.0)
 
 
 def mlstm_gates(zi: torch.Tensor, zf: torch.Tensor, cap: float) -> tuple[torch.Tensor, torch.Tensor]:
@@ -93,3 +121,10 @@ def retention_rows(q, k, v, decay, S):
         S.mul_(decay[:, None, None]).add_(v[t][:, :, None] * k[t][:, None, :])
         out[t] = (S @ q[t][:, :, None])[..., 0]
     return out
+
+
+def short_conv(u: torch.Tensor, before: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """Causal convolution over time per channel: u [T, channels] behind the rows ``before`` [taps - 1, channels], w [taps, channels]
+    with the newest tap last."""
+    T, x = u.shape[0], torch.cat([before, u])
+    return sum(w[j] * x[j:j + T] for j in range(w.shape[0]))

@@ -62,8 +62,14 @@ def synthesize(cfg: ModelConfig, recipe: QuantRecipe | str = "Q8_0", seed: int =
         for _, name, kind, shape in family_of(cfg.arch).tensor_names(cfg):
             if kind in ("mat", "stack"):
                 mat(name, *shape, layer=int(name.split(".")[1]) if name.startswith("blk.") else None)
+            elif kind == "taps":                             # mostly the newest one
+                x = torch.randn(*shape, generator=gen, device=dev, dtype=torch.float32) * 0.2
+                x[:, -1] += 1.0
+                tensors[name] = qtensor_from_float(x, GGMLType.F32)
+            elif name.endswith("depth_average.weight"):
+                tensors[name] = qtensor_from_float(torch.tensor([0.5 / (shape[0] - 1)] * (shape[0] - 1) + [0.5], device=dev), GGMLType.F32)
             else:                                            # norm gains and layer scales 1, sinks and router biases near 0, forget gates open
-                vec(name, shape[0], None if "sinks" in name or name.endswith("inp.bias") else 4.0 if name.endswith("lstm_f.bias") else 1.0)
+                vec(name, shape[0], None if "sinks" in name or name.endswith("inp.bias") else 4.0 if name.endswith("lstm_f.bias") else 0.5 if "value_mix" in name else 1.0)
         return ModelWeights(cfg, tensors, byte_tokenizer_metadata(cfg.vocab_size) if with_tokenizer else {})
     d, qd, kvd = cfg.d_model, cfg.q_dim, cfg.kv_dim
     mat("token_embd.weight", cfg.vocab_size, d)

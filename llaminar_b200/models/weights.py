@@ -140,8 +140,8 @@ class ModelWeights:
 
 def _directory_readers() -> dict:
     """config.json "architecture" -> function(config dict, {name: tensor}) -> ModelWeights."""
-    from . import kefasun, pozivik, zogepel
-    return {m.ARCHITECTURE: m.weights_from_tensors for m in (kefasun, pozivik, zogepel)}
+    from . import kefasun, lagedra, pozivik, zogepel
+    return {m.ARCHITECTURE: m.weights_from_tensors for m in (kefasun, lagedra, pozivik, zogepel)}
 
 
 def qtensor_from_float(x: torch.Tensor, qtype: GGMLType) -> QTensor:
@@ -150,8 +150,9 @@ def qtensor_from_float(x: torch.Tensor, qtype: GGMLType) -> QTensor:
 
 def named_weights(cfg: ModelConfig, names: list[tuple[str, str, str, tuple[int, ...]]], tensors: Mapping[str, torch.Tensor]) -> ModelWeights:
     """A checkpoint's tensors under the package's names.  ``names``: (checkpoint name, package name, kind, shape), kind "mat" a
-    matrix, "vec" a vector kept as it is, "gain" a zero-centred norm gain (stored as 1 + w), "stack" matrices of the names that "{}" in
-    ``src`` stands for (0, 1, ...), one behind the other."""
+    matrix, "vec" a vector kept as it is, "taps" small filters [channels, taps] kept likewise, "num" a single number (a vector of
+    one), "gain" a zero-centred norm gain (stored as 1 + w), "stack" matrices of the names that "{}" in ``src`` stands for (0, 1,
+    ...), one behind the other."""
     out: dict[str, QTensor] = {}
 
     def take(src: str, shape: tuple[int, ...]) -> torch.Tensor:
@@ -163,7 +164,7 @@ def named_weights(cfg: ModelConfig, names: list[tuple[str, str, str, tuple[int, 
         return x
 
     for src, dst, kind, shape in names:
-        x = torch.stack([take(src.format(i), shape[1:]) for i in range(shape[0])]) if kind == "stack" else take(src, shape)
+        x = torch.stack([take(src.format(i), shape[1:]) for i in range(shape[0])]) if kind == "stack" else take(src, () if kind == "num" else shape).reshape(shape)
         if kind in ("mat", "stack"):
             out[dst] = qtensor_from_float(x.float().contiguous(), GGMLType.F32 if x.dtype == torch.float32 else GGMLType.BF16)
         else:

@@ -116,4 +116,15 @@ struct ScoreScale {
 // branch-free: the approximate division has no slow path for huge or infinite denominators (they give 0, the right limit)
 LLM_DEVICE float silu(float x) { return __fdividef(x, 1.0f + __expf(-x)); }
 
+// A gated pair of clamped values: g sigmoid(1.702 g) (u + 1)
+template <class F> LLM_DEVICE float limited_pair(float g, float u, float limit, F&& sigmoid) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit);
+    return g * sigmoid(1.702f * g) * (u + 1.f);
+}
+// what an expert makes of its gate and up values
+LLM_DEVICE float expert_pair(float g, float u, float limit) {
+    return limit > 0.f ? limited_pair(g, u, limit, [](float z) { return __fdividef(1.f, 1.f + __expf(-z)); }) : silu(g) * u;
+}
+
 }  // namespace llm

@@ -61,6 +61,65 @@ void resid_norm(const OptTensor& y, const OptTensor& y_rows, const OptTensor& w_
     check(llm::launch_resid_norm(p, T, f32, stream()), "resid_norm");
 }
 
+// past [streams, tokens, d]: the first n_past streams are summed with weights w, stream n_past receives the update if there is one
+void depth_mix(const Tensor& h, bool add, const OptTensor& y, const OptTensor& y_rows, const OptTensor& z, const OptTensor& z_rows, const OptTensor& z_w,
+               const OptTensor& past, int64_t n_past, const OptTensor& w, const OptTensor& gain0, const OptTensor& xn0, const OptTensor& gain1, const OptTensor& xn1, double eps) {
+    llm::DepthMixParams p = {};
+    want(h, torch::kFloat32, "h");
+    TORCH_CHECK(h.dim() == 2, "h must be [tokens, width]");
+    const int64_t T = h.size(0), d = h.size(1);
+    if (T == 0) return;
+    bool f32 = false, typed = false;
+    auto elem = [&](const Tensor& t, const char* name) {
+        const bool f = is_f32(t, name);
+        TORCH_CHECK(!typed || f == f32, name, " has another element type than the other activations");
+        f32 = f; typed = true;
+        TORCH_CHECK(t.dim() == 2 && t.size(1) == d && t.stride(1) == 1, name, " must be rows of ", d, " values");
+        TORCH_CHECK(reinterpret_cast<uintptr_t>(t.data_ptr()) % 16 == 0, name, " must be 16-byte aligned");
+    };
+    if (y) {
+        elem(*y, "y");
+        p.y = y->data_ptr(); p.y_stride = y->stride(0); p.n_y_rows = y->size(0);
+        if (y_rows) p.y_rows = ints(*y_rows, "y_rows");
+        TORCH_CHECK((y_rows ? y_rows->numel() : y->size(0)) == T, "y must have a row per token");
+    }
+    if (z) {
+        elem(*z, "z");
+        p.z = z->data_ptr(); p.z_stride = z->stride(0); p.n_z_rows = z->size(0);
+        int64_t parts = 1;
+        if (z_w) {
+            TORCH_CHECK(z_w->dim() == 2 && z_w->size(0) == T && z_w->size(1) >= 1, "z_w must be [tokens, parts]");
+            parts = z_w->size(1);
+            p.z_w = floats(*z_w, T * parts, "z_w"); p.n_parts = parts;
+        }
+        if (z_rows) p.z_rows = ints(*z_rows, "z_rows");
+        TORCH_CHECK((z_rows ? z_rows->numel() : z->size(0)) == T * parts, "z must have a row per token and part");
+    }
+    p.h = h.data_ptr<float>(); p.add = add;
+    TORCH_CHECK(past.has_value() == w.has_value() && n_past >= 0 && (past || n_past == 0), "streams go with weights");
+    if (past) {
+        TORCH_CHECK(past->is_cuda() && past->scalar_type() == torch::kFloat32 && past->dim() == 3 && past->size(1) == T && past->size(2) == d && past->stride(2) == 1 &&
+                        past->stride(1) == d && n_past <= past->size(0) && reinterpret_cast<uintptr_t>(past->data_ptr()) % 16 == 0, "past must be float [streams, tokens, width]");
+        p.past = past->data_ptr<float>(); p.past_stride = past->stride(0); p.n_past = n_past;
+        p.keep = n_past < past->size(0) && (y || z);
+        p.w = floats(*w, n_past + 1, "w");
+    }
+    auto gain = [&](const OptTensor& g, const OptTensor& xn, const float*& gp, void*& xp) {
+        TORCH_CHECK(g.has_value() == xn.has_value(), "a norm has a gain and an output");
+        if (!g) return;
+        elem(*xn, "xn");
+        TORCH_CHECK(xn->is_contiguous() && xn->size(0) == T, "xn must be contiguous");
+        want(*g, torch::kFloat32, "gain");
+        const int step = g->numel() == 1 ? 0 : 1;
+        TORCH_CHECK((step == 0 || g->numel() == d) && (!p.gain0 || p.gain_step == step), "gains must be one number, or one per value, both of a kind");
+        p.gain_step = step; gp = g->data_ptr<float>(); xp = xn->data_ptr();
+    };
+    gain(gain0, xn0, p.gain0, p.xn0);
+    gain(gain1, xn1, p.gain1, p.xn1);
+    p.d = d; p.eps = eps;
+    check(llm::launch_depth_mix(p, T, f32, stream()), "depth_mix");
+}
+
 // table [vocabulary, columns]: columns [first, first + cols) belong to this layer
 llm::SideTable side_table(const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens, int64_t rows, bool f32) {
     llm::SideTable s = {};
@@ -83,11 +142,12 @@ void want_table(int64_t act, const OptTensor& table, int64_t cols, const OptTens
 void activate(const Tensor& x, const Tensor& act, int64_t kind, const OptTensor& table, int64_t first, int64_t cols, const OptTensor& tokens) {
     const bool f32 = is_f32(x, "x");
     want_like(act, f32, "act");
-    TORCH_CHECK(x.is_contiguous() && act.is_contiguous() && x.size(0) == act.size(0), "activation rows");
+    TORCH_CHECK(x.dim() == 2 && act.dim() == 2 && x.stride(1) == 1 && act.stride(1) == 1 && x.size(0) == act.size(0), "activation rows");
+    TORCH_CHECK((reinterpret_cast<uintptr_t>(x.data_ptr()) | reinterpret_cast<uintptr_t>(act.data_ptr())) % 16 == 0, "activations must be 16-byte aligned");
     TORCH_CHECK(x.size(1) == act.size(1) * (llm::act_pairs(kind) ? 2 : 1), "activation columns");
     want_table(kind, table, cols, tokens, act.size(1));
     if (x.size(0) == 0) return;
-    check(llm::launch_activate(x.data_ptr(), act.data_ptr(), x.size(0), act.size(1), kind, side_table(table, first, cols, tokens, x.size(0), f32), f32, stream()), "activate");
+    check(llm::launch_activate(x.data_ptr(), x.stride(0), act.data_ptr(), act.stride(0), x.size(0), act.size(1), kind, side_table(table, first, cols, tokens, x.size(0), f32), f32, stream()), "activate");
 }
 
 void rope_angles(const Tensor& positions, const Tensor& freqs, double magnitude, const Tensor& out) {
@@ -120,6 +180,7 @@ void gemv_dense(const Tensor& w, const Tensor& x, const Tensor& out, int64_t act
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("resid_norm", &resid_norm);
+    m.def("depth_mix", &depth_mix);
     m.def("activate", &activate);
     m.def("rope_angles", &rope_angles);
     m.def("gemv_dense", &gemv_dense);

@@ -286,6 +286,115 @@ __global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNorm
     });
 }
 
+// See DepthMixParams.  A CTA per row; a thread holds NV x VEC of its values (VEC = 1: of any alignment).
+template <class T, int VEC, int THREADS, int NV, bool PARTS>
+__global__ void __launch_bounds__(THREADS) depth_mix_kernel(const DepthMixParams p) {
+    constexpr int W = THREADS / 32;
+    __shared__ float red[W];
+    pdl_trigger();
+    const size_t t = blockIdx.x;
+    const int d = p.d;
+    auto at = [&](int n) { return (n * THREADS + (int)threadIdx.x) * VEC; };
+    auto each = [&](auto f) {
+#pragma unroll
+        for (int n = 0; n < NV; ++n)
+            if (at(n) < d) f(n, at(n));
+    };
+    auto load_t = [](const T* s, float (&v)[VEC]) {
+        if constexpr (VEC == 4) Vec4<T>::load(s, v); else v[0] = to_f(*s);
+    };
+    auto load_f = [](const float* s, float (&v)[VEC]) {
+        if constexpr (VEC == 4) Vec4<float>::load(s, v); else v[0] = *s;
+    };
+    auto store_t = [](T* s, const float (&v)[VEC]) {
+        if constexpr (VEC == 4) Vec4<T>::store(s, v); else *s = from_f<T>(v[0]);
+    };
+    auto store_f = [](float* s, const float (&v)[VEC]) {
+        if constexpr (VEC == 4) Vec4<float>::store(s, v); else *s = v[0];
+    };
+    pdl_wait();
+    float* h = p.h + t * d;
+    float v[NV][VEC] = {};
+    const bool update = p.y || p.z;
+    if (p.add || !update) each([&](int n, int i) { load_f(h + i, v[n]); });
+    if (p.y) {
+        const T* y = static_cast<const T*>(p.y) + (p.y_rows ? (size_t)LLM_CHECK_INDEX(p.y_rows[t], p.n_y_rows) : t) * p.y_stride;
+        float u[NV][VEC];
+        each([&](int n, int i) { load_t(y + i, u[n]); });
+        each([&](int n, int) {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[n][j] += u[n][j];
+        });
+    }
+    if (p.z) {
+        auto z_row = [&](size_t i) { return static_cast<const T*>(p.z) + (p.z_rows ? (size_t)LLM_CHECK_INDEX(p.z_rows[i], p.n_z_rows) : i) * p.z_stride; };
+        if constexpr (PARTS) {
+            float s[NV][VEC] = {};
+#pragma unroll 4
+            for (int q = 0; q < p.n_parts; ++q) {
+                const T* z = z_row(t * p.n_parts + q);
+                const float w = p.z_w[t * p.n_parts + q];
+                each([&](int n, int i) {
+                    float u[VEC];
+                    load_t(z + i, u);
+#pragma unroll
+                    for (int j = 0; j < VEC; ++j) s[n][j] = fmaf(u[j], w, s[n][j]);
+                });
+            }
+            each([&](int n, int) {
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) v[n][j] += s[n][j];
+            });
+        } else {
+            const T* z = z_row(t);
+            each([&](int n, int i) {
+                float u[VEC];
+                load_t(z + i, u);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) v[n][j] += u[j];
+            });
+        }
+    }
+    if (p.keep) each([&](int n, int i) { store_f(p.past + p.n_past * p.past_stride + t * d + i, v[n]); });
+    if (p.w) {
+        const float own = p.w[p.n_past];
+        each([&](int n, int) {
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[n][j] *= own;
+        });
+#pragma unroll 4
+        for (int q = 0; q < p.n_past; ++q) {
+            const float w = p.w[q];
+            const float* x = p.past + q * p.past_stride + t * d;
+            each([&](int n, int i) {
+                float u[VEC];
+                load_f(x + i, u);
+#pragma unroll
+                for (int j = 0; j < VEC; ++j) v[n][j] = fmaf(u[j], w, v[n][j]);
+            });
+        }
+    }
+    if (update) each([&](int n, int i) { store_f(h + i, v[n]); });
+    if (!p.xn0 && !p.xn1) return;
+    float ss = 0.f;
+    each([&](int n, int) {
+#pragma unroll
+        for (int j = 0; j < VEC; ++j) ss += v[n][j] * v[n][j];
+    });
+    const float inv = 1.f / sqrtf(block_sum<THREADS>(ss, red) / (float)d + p.eps);
+    auto norm = [&](const float* gain, void* xn) {
+        if (!xn) return;
+        each([&](int n, int i) {
+            float u[VEC];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) u[j] = v[n][j] * inv * gain[(i + j) * p.gain_step];
+            store_t(static_cast<T*>(xn) + t * d + i, u);
+        });
+    };
+    norm(p.gain0, p.xn0);
+    norm(p.gain1, p.xn1);
+}
+
 // value `i` of row `t` of the activation of `x`; `u`: the second half's value (GELU_MUL, SILU_MUL)
 template <int ACT, class T>
 LLM_DEVICE float activated(float x, float u, const SideTable& s, int t, int i) {
@@ -293,18 +402,20 @@ LLM_DEVICE float activated(float x, float u, const SideTable& s, int t, int i) {
     if (ACT == ACT_SILU_MUL) return x * logistic(x) * u;
     if (ACT == ACT_GATE) return x * logistic(to_f(static_cast<const T*>(s.table)[(size_t)t * s.row + i]));
     if (ACT == ACT_RELU2) { x = fmaxf(x, 0.f); return x * x; }
+    if (ACT == ACT_GELU) return gelu_tanh(x);
+    if (ACT == ACT_SILU) return x * logistic(x);
     if (ACT == ACT_GELU_SIDE) return i < s.cols ? gelu_tanh(x) * to_f(static_cast<const T*>(s.table)[(size_t)LLM_CHECK_INDEX(s.tokens[t], s.n_rows) * s.row + i]) : 0.f;
     return x;
 }
 
 template <class T, int ACT>
-__global__ void __launch_bounds__(256) activate_kernel(const T* x, T* act, int n, const SideTable s) {
+__global__ void __launch_bounds__(256) activate_kernel(const T* x, size_t x_row, T* act, size_t act_row, int n, const SideTable s) {
     pdl_trigger();
     pdl_wait();
-    const T* g = x + (size_t)blockIdx.y * n * (act_pairs(ACT) ? 2 : 1);
-    T* a = act + (size_t)blockIdx.y * n;
+    const T* g = x + (size_t)blockIdx.y * x_row;
+    T* a = act + (size_t)blockIdx.y * act_row;
     const int i0 = (blockIdx.x * 256 + threadIdx.x) * 4;
-    if (n % 4 == 0) {
+    if ((n | x_row | act_row) % 4 == 0) {
         if (i0 >= n) return;
         float v[4], u[4] = {};
         Vec4<T>::load(g + i0, v);
@@ -429,21 +540,42 @@ cudaError_t resid_norm_any(const ResidNormParams& p, int rows, cudaStream_t st) 
 
 }  // namespace
 
+cudaError_t launch_depth_mix(const DepthMixParams& p, int rows, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    const bool vec = p.d % 4 == 0 && p.y_stride % 4 == 0 && p.z_stride % 4 == 0 && p.past_stride % 4 == 0;
+    if (p.d < 1 || p.d > (vec ? 16384 : 8192) || (p.w == nullptr && p.n_past > 0)) return cudaErrorInvalidValue;
+    auto go = [&](auto plain, auto parts, int threads) { return launch_pdl(p.n_parts ? parts : plain, dim3(rows), dim3(threads), 0, st, p); };
+#define LLM_DEPTH_MIX(T, VEC, THREADS, NV) return go(depth_mix_kernel<T, VEC, THREADS, NV, false>, depth_mix_kernel<T, VEC, THREADS, NV, true>, THREADS)
+    auto any = [&](auto tag) {
+        using T = decltype(tag);
+        if (!vec) LLM_DEPTH_MIX(T, 1, 512, 16);
+        if (p.d <= 1024) LLM_DEPTH_MIX(T, 4, 128, 2);
+        if (p.d <= 2048) LLM_DEPTH_MIX(T, 4, 256, 2);
+        if (p.d <= 4096) LLM_DEPTH_MIX(T, 4, 512, 2);
+        if (p.d <= 8192) LLM_DEPTH_MIX(T, 4, 512, 4);
+        LLM_DEPTH_MIX(T, 4, 512, 8);
+    };
+#undef LLM_DEPTH_MIX
+    return f32 ? any(float()) : any(__nv_bfloat16());
+}
+
 cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cudaStream_t st) {
     return f32 ? resid_norm_any<float>(p, rows, st) : resid_norm_any<__nv_bfloat16>(p, rows, st);
 }
 
-cudaError_t launch_activate(const void* x, void* act, int rows, int n, int kind, const SideTable& side, bool f32, cudaStream_t st) {
+cudaError_t launch_activate(const void* x, size_t x_row, void* act, size_t act_row, int rows, int n, int kind, const SideTable& side, bool f32, cudaStream_t st) {
     const dim3 grid((n + 1023) / 1024, rows);
     if (rows > 65535) return cudaErrorInvalidValue;
     auto go = [&](auto k32, auto k16) {
-        if (f32) return launch_pdl(k32, grid, dim3(256), 0, st, static_cast<const float*>(x), static_cast<float*>(act), n, side);
-        return launch_pdl(k16, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(x), static_cast<__nv_bfloat16*>(act), n, side);
+        if (f32) return launch_pdl(k32, grid, dim3(256), 0, st, static_cast<const float*>(x), x_row, static_cast<float*>(act), act_row, n, side);
+        return launch_pdl(k16, grid, dim3(256), 0, st, static_cast<const __nv_bfloat16*>(x), x_row, static_cast<__nv_bfloat16*>(act), act_row, n, side);
     };
     if (kind == ACT_GELU_MUL) return go(activate_kernel<float, ACT_GELU_MUL>, activate_kernel<__nv_bfloat16, ACT_GELU_MUL>);
     if (kind == ACT_SILU_MUL) return go(activate_kernel<float, ACT_SILU_MUL>, activate_kernel<__nv_bfloat16, ACT_SILU_MUL>);
     if (kind == ACT_GATE) return go(activate_kernel<float, ACT_GATE>, activate_kernel<__nv_bfloat16, ACT_GATE>);
     if (kind == ACT_RELU2) return go(activate_kernel<float, ACT_RELU2>, activate_kernel<__nv_bfloat16, ACT_RELU2>);
+    if (kind == ACT_GELU) return go(activate_kernel<float, ACT_GELU>, activate_kernel<__nv_bfloat16, ACT_GELU>);
+    if (kind == ACT_SILU) return go(activate_kernel<float, ACT_SILU>, activate_kernel<__nv_bfloat16, ACT_SILU>);
     if (kind == ACT_GELU_SIDE) return go(activate_kernel<float, ACT_GELU_SIDE>, activate_kernel<__nv_bfloat16, ACT_GELU_SIDE>);
     return cudaErrorInvalidValue;
 }
@@ -455,6 +587,7 @@ cudaError_t launch_rope_angles(const int* positions, const double* freqs, double
 }
 
 cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st) {
+    if (p.act == ACT_SILU) return cudaErrorInvalidValue;
     if (p.m < 1 || p.m > 8 || p.n < 1 || p.k % 8 || p.ldw % 8 || p.w_z % 8 || p.x_row % 8 || p.x_z % 8 || (p.act != ACT_NONE && p.out_f32)) return cudaErrorInvalidValue;
     // split K until every warp has about eight blocks of 32 and the grid fills the machine
     const int blocks = (p.k + 31) / 32, tiles = (p.n + 15) / 16 * p.z;
@@ -467,6 +600,7 @@ cudaError_t launch_gemv_dense(const GemvDenseParams& p, cudaStream_t st) {
     if (p.act == ACT_SILU_MUL) return go(gemv_dense_kernel<ACT_SILU_MUL, __nv_bfloat16>);
     if (p.act == ACT_GATE) return go(gemv_dense_kernel<ACT_GATE, __nv_bfloat16>);
     if (p.act == ACT_RELU2) return go(gemv_dense_kernel<ACT_RELU2, __nv_bfloat16>);
+    if (p.act == ACT_GELU) return go(gemv_dense_kernel<ACT_GELU, __nv_bfloat16>);
     if (p.act == ACT_GELU_SIDE) return go(gemv_dense_kernel<ACT_GELU_SIDE, __nv_bfloat16>);
     return p.out_f32 ? go(gemv_dense_kernel<ACT_NONE, float>) : go(gemv_dense_kernel<ACT_NONE, __nv_bfloat16>);
 }

@@ -29,17 +29,40 @@ LLM_DEVICE void load8(const float* p, float (&v)[8]) {
 }
 
 // ---- routing -------------------------------------------------------------------------------------------------------------------
-// One warp: the `top` largest of z[0 .. n) and the softmax over them.  Logits stay in registers as integers of the same order (NR per
+// One warp: marks the `keep` groups of neighbours with the largest values in z[0 .. n) by a zero in g[0 .. groups).
+LLM_DEVICE unsigned ordered(float v) {             // integers of the same order; 0 is below all of them
+    const unsigned u = __float_as_uint(v);
+    return u & 0x80000000u ? ~u : u | 0x80000000u;
+}
+LLM_DEVICE void keep_groups(const float* z, unsigned* g, const ExpertRouteParams& p) {
+    const int lane = threadIdx.x & 31, size = p.n / p.groups;
+    for (int i = lane; i < p.groups; i += 32) {
+        unsigned best = 1;
+        for (int j = 0; j < size; ++j) best = max(best, ordered(z[i * size + j]));
+        g[i] = best;
+    }
+    __syncwarp();
+    for (int r = 0; r < p.keep; ++r) {
+        unsigned best = 0, at = 0xffffffffu;
+        for (int i = lane; i < p.groups; i += 32)
+            if (g[i] > best) { best = g[i]; at = i; }
+        const unsigned top = __reduce_max_sync(0xffffffffu, best);
+        at = __reduce_min_sync(0xffffffffu, best == top ? at : 0xffffffffu);
+        if (lane == 0 && at < (unsigned)p.groups) g[at] = 0;
+        __syncwarp();
+    }
+}
+
+// One warp: the `top` largest of z[0 .. n) (with g: of the groups that it marks) and the softmax over them.  Logits stay in registers as integers of the same order (NR per
 // lane), so a round is two warp-wide integer reductions.  Every id it writes is a valid expert, whatever the logits are.
 template <int NR>
-LLM_DEVICE void choose_of(const float* z, const ExpertRouteParams& p, int t) {
+LLM_DEVICE void choose_of(const float* z, const unsigned* g, const ExpertRouteParams& p, int t) {
     const int lane = threadIdx.x & 31;
     unsigned key[NR];
 #pragma unroll
     for (int j = 0; j < NR; ++j) {
         const int i = lane + j * 32;
-        const unsigned u = i < p.n ? __float_as_uint(z[i]) : 0u;
-        key[j] = i < p.n ? (u & 0x80000000u ? ~u : u | 0x80000000u) : 0u;
+        key[j] = i < p.n && !(g && g[i / (p.n / p.groups)]) ? ordered(z[i]) : 0u;
     }
     float mine = -INFINITY;                        // lane r: the r-th largest logit
     int id = 0;
@@ -66,10 +89,11 @@ LLM_DEVICE void choose_of(const float* z, const ExpertRouteParams& p, int t) {
         if (p.counts) p.ranks[pair] = atomicAdd(&p.counts[id], 1);
     }
 }
-LLM_DEVICE void choose(const float* z, const ExpertRouteParams& p, int t) {
-    if (p.n <= 32) choose_of<1>(z, p, t);
-    else if (p.n <= 128) choose_of<4>(z, p, t);
-    else choose_of<EXPERTS_MAX / 32>(z, p, t);
+LLM_DEVICE void choose(const float* z, unsigned* g, const ExpertRouteParams& p, int t) {       // g: workspace for the groups
+    if (p.keep < p.groups) keep_groups(z, g, p); else g = nullptr;
+    if (p.n <= 32) choose_of<1>(z, g, p, t);
+    else if (p.n <= 128) choose_of<4>(z, g, p, t);
+    else choose_of<EXPERTS_MAX / 32>(z, g, p, t);
 }
 
 // A cluster of CTAs per token: their warps take the experts in turn, four at a time, and leave the logits with the first CTA.
@@ -77,6 +101,7 @@ constexpr int ROUTE_THREADS = 512, ROUTE_CLUSTER = 8;
 template <class T, bool VEC>
 __global__ void __launch_bounds__(ROUTE_THREADS) expert_route_kernel(const ExpertRouteParams p) {
     __shared__ float z[EXPERTS_MAX];
+    __shared__ unsigned s_groups[EXPERTS_MAX];
     pdl_trigger();
     cg::cluster_group cluster = cg::this_cluster();
     const bool spread = gridDim.x > 1;
@@ -111,11 +136,11 @@ __global__ void __launch_bounds__(ROUTE_THREADS) expert_route_kernel(const Exper
 #pragma unroll
         for (int j = 0; j < NE; ++j) {
             const float s = warp_sum(acc[j]);
-            if (lane == 0 && e0 + j < p.n) dst[e0 + j] = s + p.bias[e0 + j];
+            if (lane == 0 && e0 + j < p.n) dst[e0 + j] = p.bias ? s + p.bias[e0 + j] : s;
         }
     }
     if (spread) cluster.sync(); else __syncthreads();
-    if (warp == 0 && blockIdx.x == 0) choose(z, p, t);
+    if (warp == 0 && blockIdx.x == 0) choose(z, s_groups, p, t);
 }
 
 // a warp per token, logits given
@@ -125,10 +150,10 @@ __global__ void __launch_bounds__(128) expert_choose_kernel(const ExpertRoutePar
     pdl_wait();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, t = blockIdx.x * 4 + warp;
     if (t >= rows) return;
-    float* z = sm + warp * p.n;
-    for (int i = lane; i < p.n; i += 32) z[i] = p.logits[(size_t)t * p.n + i] + p.bias[i];
+    float* z = sm + warp * (p.n + p.groups);
+    for (int i = lane; i < p.n; i += 32) z[i] = p.logits[(size_t)t * p.n + i] + (p.bias ? p.bias[i] : 0.f);
     __syncwarp();
-    choose(z, p, t);
+    choose(z, reinterpret_cast<unsigned*>(z + p.n), p, t);
 }
 
 // a CTA per token; warp j finds the row of the token's pair j, then all threads copy
@@ -249,7 +274,7 @@ __global__ void __launch_bounds__(32 * ROW_WARPS) expert_rows_kernel(const Exper
                     v += s_acc[(c / 16) * wk + a][0][c % 16][r];
                     if constexpr (PAIR) v2 += s_acc[(c / 16) * wk + a][1][c % 16][r];
                 }
-                if constexpr (PAIR) v = silu(v) * v2;
+                if constexpr (PAIR) v = expert_pair(v, v2, p.limit);
                 static_cast<__nv_bfloat16*>(p.out)[(size_t)s_pair[q0 + q * 8 + r] * p.n + n] = __float2bfloat16(v);
             }
         }
@@ -272,7 +297,7 @@ __global__ void __launch_bounds__(256) expert_plain_kernel(const ExpertRowsParam
             if (PAIR) b = fmaf(v, to_f(w[((size_t)p.n + n) * p.k + c]), b);
         }
         a = warp_sum(a);
-        if (PAIR) { b = warp_sum(b); a = a / (1.f + expf(-a)) * b; }
+        if (PAIR) { b = warp_sum(b); a = p.limit > 0.f ? limited_pair(a, b, p.limit, [](float z) { return 1.f / (1.f + expf(-z)); }) : a / (1.f + expf(-a)) * b; }
         if (lane == 0) static_cast<T*>(p.out)[(size_t)pair * p.n + n] = from_f<T>(a);
     }
 }
@@ -282,7 +307,8 @@ __global__ void __launch_bounds__(256) expert_plain_kernel(const ExpertRowsParam
 cudaError_t launch_expert_route(const ExpertRouteParams& p, int rows, bool f32, cudaStream_t st) {
     if (rows == 0) return cudaSuccess;
     if (p.n < 1 || p.n > EXPERTS_MAX || p.top < 1 || p.top > p.n || p.top > EXPERTS_MAX_TOP) return cudaErrorInvalidValue;
-    if (p.logits) return launch_pdl(expert_choose_kernel, dim3((rows + 3) / 4), dim3(128), (size_t)4 * p.n * 4, st, p, rows);
+    if (p.groups < 1 || p.n % p.groups || p.keep < 1 || p.keep > p.groups || p.top > p.n / p.groups * p.keep) return cudaErrorInvalidValue;
+    if (p.logits) return launch_pdl(expert_choose_kernel, dim3((rows + 3) / 4), dim3(128), (size_t)4 * (p.n + p.groups) * 4, st, p, rows);
     const bool vec = p.d % 8 == 0 && p.x_row % 8 == 0 && !((reinterpret_cast<uintptr_t>(p.x) | reinterpret_cast<uintptr_t>(p.router)) & 15);
     if (rows > 65535) return cudaErrorInvalidValue;
     auto go = [&](auto kernel) {

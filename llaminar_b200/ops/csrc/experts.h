@@ -11,7 +11,9 @@ namespace llm {
 constexpr int EXPERTS_MAX_TOP = 32, EXPERTS_MAX = 1024;
 
 // Router logits x W^T + bias (or given in `logits`), the `top` largest of them (the lower expert first when equal) and the softmax over
-// just those.  With `counts` (zeroed by the caller) the pairs of every expert are counted and numbered.
+// just those (what dividing their part of a softmax over all experts by its sum gives).  With `groups` > 1 the experts form that many
+// groups of neighbours, and only those of the `keep` groups with the largest logits (the lower group first when equal) can be chosen.
+// With `counts` (zeroed by the caller) the pairs of every expert are counted and numbered.
 struct ExpertRouteParams {
     const void* x; size_t x_row;                   // [T, d]
     const void* router;                            // [n, d]
@@ -19,7 +21,7 @@ struct ExpertRouteParams {
     const float* bias;                             // [n]
     int* ids; float* weights;                      // [T, top]
     int *counts, *ranks;                           // [n], [T * top]: number of a pair among those of its expert
-    int d, n, top;
+    int d, n, top, groups, keep;
 };
 cudaError_t launch_expert_route(const ExpertRouteParams& p, int rows, bool f32, cudaStream_t st);
 
@@ -33,7 +35,8 @@ struct ExpertPlaceParams {
 };
 cudaError_t launch_expert_place(const ExpertPlaceParams& p, int rows, cudaStream_t st);
 
-// out[pair] = x[pair / div] W_e^T with e = ids[pair]; `pair_act`: W_e stacks gate and up, out = silu(gate) * up.
+// out[pair] = x[pair / div] W_e^T with e = ids[pair]; `pair_act`: W_e stacks gate and up, out = silu(gate) * up, or with a `limit` g
+// sigmoid(1.702 g) (u + 1) of g = min(gate, limit) and u = up clamped to [-limit, limit].
 struct ExpertRowsParams {
     const void* w;                                 // [experts, n (pair_act: 2n), k]
     const void* x; size_t x_row;
@@ -41,6 +44,7 @@ struct ExpertRowsParams {
     void* out;                                     // [pairs, n]
     int pairs, div, n, k, experts;
     bool pair_act;
+    float limit;
 };
 // few pairs, bf16: the weights of every chosen expert are read once for all of its pairs (in groups of 8 to 32)
 constexpr int EXPERT_ROWS_MAX_PAIRS = 1024;
@@ -53,6 +57,7 @@ struct ExpertGroupedParams {
     const int* counts;
     __nv_bfloat16* out;                            // [pairs, n]
     int pairs, n, k, experts;
+    float limit;
 };
 bool expert_grouped_fits(int n, int k, int experts);
 cudaError_t launch_expert_grouped(const __nv_bfloat16* w, const __nv_bfloat16* x, const ExpertGroupedParams& p, bool pair_act, int* status, cudaStream_t st);

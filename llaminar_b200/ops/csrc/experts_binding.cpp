@@ -18,14 +18,15 @@ int* pair_ints(const Tensor& t, int64_t n, const char* name) {
 }
 
 // logits [tokens, experts], or x [tokens, d] and router [experts, d]; counts and ranks number the pairs of every expert
-void expert_route(const OptTensor& x, const OptTensor& router, const OptTensor& logits, const Tensor& bias, const Tensor& ids, const Tensor& weights,
-                  const OptTensor& counts, const OptTensor& ranks) {
+void expert_route(const OptTensor& x, const OptTensor& router, const OptTensor& logits, const OptTensor& bias, const Tensor& ids, const Tensor& weights,
+                  const OptTensor& counts, const OptTensor& ranks, int64_t groups, int64_t keep) {
     TORCH_CHECK(ids.dim() == 2 && weights.sizes() == ids.sizes(), "ids / weights must be [tokens, top]");
-    const int64_t T = ids.size(0), n = bias.numel();
+    TORCH_CHECK(logits || router, "logits, or x with router");
+    const int64_t T = ids.size(0), n = logits ? logits->size(-1) : router->size(0);
     if (T == 0) return;
     llm::ExpertRouteParams p = {};
-    p.n = n; p.top = ids.size(1);
-    p.bias = floats(bias, n, "bias");
+    p.n = n; p.top = ids.size(1); p.groups = groups; p.keep = keep;
+    if (bias) p.bias = floats(*bias, n, "bias");
     p.ids = pair_ints(ids, T * p.top, "ids"); p.weights = const_cast<float*>(floats(weights, T * p.top, "weights"));
     TORCH_CHECK(counts.has_value() == ranks.has_value() && logits.has_value() != x.has_value() && x.has_value() == router.has_value(), "counts with ranks; logits, or x with router");
     if (counts) { p.counts = pair_ints(*counts, n, "counts"); p.ranks = pair_ints(*ranks, T * p.top, "ranks"); }
@@ -54,28 +55,29 @@ void expert_place(const Tensor& x, const Tensor& ids, const Tensor& ranks, const
 }
 
 // w [experts, n (pair_act: 2n), k]; out [pairs, n]; pair p reads row p / div of x
-llm::ExpertRowsParams rows_params(const Tensor& w, const Tensor& x, const Tensor& ids, const Tensor& out, int64_t div, bool pair_act) {
+llm::ExpertRowsParams rows_params(const Tensor& w, const Tensor& x, const Tensor& ids, const Tensor& out, int64_t div, bool pair_act, double limit) {
     const bool f32 = is_f32(w, "w");
     want_like(x, f32, "x"); want_like(out, f32, "out");
     llm::ExpertRowsParams p = {};
     TORCH_CHECK(w.dim() == 3 && w.is_contiguous() && out.dim() == 2 && out.is_contiguous() && x.dim() == 2 && x.stride(1) == 1, "expert layouts");
-    p.w = w.data_ptr(); p.experts = w.size(0); p.n = out.size(1); p.k = w.size(2); p.pair_act = pair_act; p.div = div;
+    p.w = w.data_ptr(); p.experts = w.size(0); p.n = out.size(1); p.k = w.size(2); p.pair_act = pair_act; p.limit = limit; p.div = div;
     p.pairs = ids.numel();
     TORCH_CHECK(w.size(1) == p.n * (pair_act ? 2 : 1) && x.size(1) == p.k && out.size(0) == p.pairs && div >= 1 && x.size(0) * div >= p.pairs, "expert shapes");
     p.x = x.data_ptr(); p.x_row = x.stride(0); p.ids = ints(ids, "ids"); p.out = out.data_ptr();
     return p;
 }
-void expert_rows(const Tensor& w, const Tensor& x, const Tensor& ids, const Tensor& out, int64_t div, bool pair_act) {
+void expert_rows(const Tensor& w, const Tensor& x, const Tensor& ids, const Tensor& out, int64_t div, bool pair_act, double limit) {
     TORCH_CHECK(!is_f32(w, "w") && aligned16(w) && aligned16(x), "expert_rows takes 16-byte aligned bf16 operands");
-    check(llm::launch_expert_rows(rows_params(w, x, ids, out, div, pair_act), stream()), "expert_rows");
+    check(llm::launch_expert_rows(rows_params(w, x, ids, out, div, pair_act, limit), stream()), "expert_rows");
 }
-void expert_plain(const Tensor& w, const Tensor& x, const Tensor& ids, const Tensor& out, int64_t div, bool pair_act) {
-    check(llm::launch_expert_plain(rows_params(w, x, ids, out, div, pair_act), is_f32(w, "w"), stream()), "expert_plain");
+void expert_plain(const Tensor& w, const Tensor& x, const Tensor& ids, const Tensor& out, int64_t div, bool pair_act, double limit) {
+    check(llm::launch_expert_plain(rows_params(w, x, ids, out, div, pair_act, limit), is_f32(w, "w"), stream()), "expert_plain");
 }
 
 // x [pairs, k] and out [pairs, n] sorted by expert
-void expert_grouped(const Tensor& w, const Tensor& x, const Tensor& counts, const Tensor& out, bool pair_act, const Tensor& status) {
+void expert_grouped(const Tensor& w, const Tensor& x, const Tensor& counts, const Tensor& out, bool pair_act, const Tensor& status, double limit) {
     llm::ExpertGroupedParams p = {};
+    p.limit = limit;
     TORCH_CHECK(w.dim() == 3 && x.dim() == 2 && out.dim() == 2 && x.size(0) == out.size(0), "expert layouts");
     p.pairs = x.size(0); p.n = out.size(1); p.k = x.size(1); p.experts = w.size(0);
     TORCH_CHECK(w.size(1) == p.n * (pair_act ? 2 : 1) && w.size(2) == p.k, "expert shapes");

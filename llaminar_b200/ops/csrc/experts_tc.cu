@@ -3,7 +3,7 @@
 // Persistent CTAs walk the tiles (columns fastest, so that the CTAs at work share row and weight tiles in L2).  Row and weight tiles of
 // 64 columns arrive by TMA, 128-byte swizzled; one MMA of M = 128, N = 256 per 16 columns; two accumulators of 256 columns in TMEM, so
 // that the epilogue of a tile runs under the products of the next.  PAIR: the 256 weight rows are 128 rows of the gate and the 128 of
-// `up` at the same place, and the epilogue writes silu(gate) * up.  A row tile may reach into the next expert's rows: they are not stored.
+// `up` at the same place, and the epilogue writes silu(gate) * up, or its limited form.  A row tile may reach into the next expert's rows: they are not stored.
 // Warp 0 TMA, 1 MMA issue and TMEM allocation, 2 to 5 epilogue.  Every wait is bounded; on a timeout the status word is raised.
 #include "experts.h"
 #include "launch.h"
@@ -144,7 +144,7 @@ __global__ void __launch_bounds__(THREADS, 1) expert_grouped_kernel(const __grid
                 if constexpr (PAIR) {
                     tmem_wait_ld(u);
 #pragma unroll
-                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(silu(__uint_as_float(r[j])) * __uint_as_float(u[j]));
+                    for (int j = 0; j < 32; ++j) r[j] = __float_as_uint(expert_pair(__uint_as_float(r[j]), __uint_as_float(u[j]), p.limit));
                 }
                 if (row < t.rows) {
 #pragma unroll

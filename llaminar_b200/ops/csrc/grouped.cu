@@ -2,6 +2,8 @@
 //
 //   attn_prep      norms of the queries and keys over all heads together, append to the paged cache
 //   head_prep      norms of queries and keys per head, rotation, append to the paged cache
+//   conv_prep      short convolution over time, rotation, temperatures, mixing of values, append to the paged cache
+//   conv_keep      the last rows of prompt portions into the convolution's state
 //   attn_plain     one row and head per CTA in float arithmetic
 #include "common.cuh"
 #include "grouped.h"
@@ -137,6 +139,140 @@ __global__ void __launch_bounds__(256) head_prep_kernel(const HeadPrepParams p) 
     }
 }
 
+// A warp per head (queries, then keys, then values) and strip of N rows.  TAPS taps with at most four values per lane (dim <= 128): taps
+// and the rows before the current one stay in registers, the strip's rows are loaded together; TAPS = 0: any number and size.
+template <class TI, class T, int TAPS, int N>
+__global__ void __launch_bounds__(256) conv_prep_kernel(const ConvPrepParams p) {
+    extern __shared__ __align__(16) float sm[];                // [8][dim]
+    pdl_trigger();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = p.dim, H = p.n_heads, G = p.n_kv_heads, U = H + 2 * G;
+    const int u = blockIdx.y * 8 + warp, t0 = blockIdx.x * N, n_taps = TAPS ? TAPS : p.n_taps;
+    if (u >= U) return;
+    const int kind = u < H ? 0 : u < H + G ? 1 : 2, h = u - (kind == 0 ? 0 : kind == 1 ? H : H + G), col = u * D, cols = U * D;
+    float* out = sm + warp * D;
+    constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 1;
+    float w[TAPS ? TAPS : 1][4], past[KEEP][4], cur[N][4];     // past[j]: the row j + 1 before the current one
+    const int c_own = lane * 4;
+    if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+            w[j][0] = w[j][1] = w[j][2] = w[j][3] = 0.f;
+            if (c_own < D) load4(p.taps + (size_t)j * cols + col + c_own, w[j]);
+        }
+    }
+    const TI* in = static_cast<const TI*>(p.in) + col;
+    pdl_wait();
+    if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            cur[i][0] = cur[i][1] = cur[i][2] = cur[i][3] = 0.f;
+            if (t0 + i < p.rows && c_own < D) load4(in + (size_t)(t0 + i) * p.in_row + c_own, cur[i]);
+        }
+    }
+    const float gain = kind == 0 && p.q_gain ? p.q_gain[h] : 1.f, share = p.share ? *p.share : 0.f;
+#pragma unroll
+    for (int i = 0; i < N; ++i) {
+        const int t = t0 + i;
+        if (t >= p.rows) break;
+        const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
+        const int r0 = p.cu ? p.cu[seq] : t;                   // first row of the sequence's portion
+        float* ring = p.ring + (size_t)LLM_CHECK_INDEX(p.slots[seq], p.n_slots) * n_taps * cols + col;
+        // what stood `lag` rows before this one, zeros in front of the sequence
+        auto row_before = [&](int lag, int c, float (&x)[4]) {
+            x[0] = x[1] = x[2] = x[3] = 0.f;
+            if (c >= D || pos < lag) return;
+            if (t - lag >= r0) load4(in + (size_t)(t - lag) * p.in_row + c, x);
+            else load4(ring + (size_t)((pos - lag) % n_taps) * cols + c, x);
+        };
+        __syncwarp();                                          // the row of the token before has been read
+        if constexpr (TAPS > 0) {
+            if (i == 0 || t == r0) {
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) row_before(j + 1, c_own, past[j]);
+            }
+            if (c_own < D) {
+                float a[4];
+#pragma unroll
+                for (int e = 0; e < 4; ++e) a[e] = w[TAPS - 1][e] * cur[i][e];
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) a[e] = fmaf(w[TAPS - 2 - j][e], past[j][e], a[e]);
+                store4(out + c_own, a);
+                if (!p.cu) store4(ring + (size_t)(pos % n_taps) * cols + c_own, cur[i]);
+            }
+#pragma unroll
+            for (int j = KEEP - 1; j >= 0; --j)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) past[j][e] = j ? past[j - 1][e] : cur[i][e];
+        } else {
+            for (int c = c_own; c < D; c += 128) {
+                float a[4] = {}, x[4], k[4];
+                for (int lag = n_taps - 1; lag >= 0; --lag) {
+                    if (lag) row_before(lag, c, x);
+                    else load4(in + (size_t)t * p.in_row + c, x);
+                    load4(p.taps + (size_t)(n_taps - 1 - lag) * cols + col + c, k);
+#pragma unroll
+                    for (int e = 0; e < 4; ++e) a[e] = fmaf(k[e], x[e], a[e]);
+                }
+                store4(out + c, a);
+                if (!p.cu) store4(ring + (size_t)(pos % n_taps) * cols + c, x);
+            }
+        }
+        T* dst = static_cast<T*>(p.q_out) + ((size_t)t * H + h) * D;
+        if (kind) {
+            const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
+            dst = static_cast<T*>(p.kv) + ((((size_t)page * 2 + kind - 1) * G + h) * PAGE + pos % PAGE) * D;
+        }
+        float x[4];
+        if (kind == 2) {
+            float* first = p.first ? p.first + ((size_t)t * G + h) * p.first_dim : nullptr;
+            for (int c = c_own; c < D; c += 128) {             // every lane reads back what it wrote
+                load4(out + c, x);
+                if (first && c < p.first_dim) {
+                    if (p.share) {
+                        float f[4];
+                        load4(first + c, f);
+#pragma unroll
+                        for (int e = 0; e < 4; ++e) x[e] = (1.f - share) * x[e] + share * f[e];
+                    } else {
+                        store4(first + c, x);
+                    }
+                }
+                store4(dst + c, x);
+            }
+            continue;
+        }
+        __syncwarp();
+        const float2* ang = p.angles + (size_t)t * p.half;
+        for (int c = c_own; c < D; c += 128) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) {
+                const int k = c + e;
+                x[e] = out[k];
+                if (k < p.half) x[e] = x[e] * ang[k].x - out[k + p.half] * ang[k].y;
+                else if (k < 2 * p.half) x[e] = x[e] * ang[k - p.half].x + out[k - p.half] * ang[k - p.half].y;
+                x[e] *= gain;
+            }
+            store4(dst + c, x);
+        }
+    }
+}
+
+template <class TI>
+__global__ void __launch_bounds__(256) conv_keep_kernel(const ConvPrepParams p) {
+    pdl_trigger();
+    pdl_wait();
+    const int cols = (p.n_heads + 2 * p.n_kv_heads) * p.dim, c = (blockIdx.x * 256 + threadIdx.x) * 4, seq = blockIdx.y;
+    if (c >= cols) return;
+    float* ring = p.ring + (size_t)LLM_CHECK_INDEX(p.slots[seq], p.n_slots) * p.n_taps * cols + c;
+    for (int r = max(p.cu[seq], p.cu[seq + 1] - p.n_taps + 1); r < p.cu[seq + 1]; ++r) {
+        float x[4];
+        load4(static_cast<const TI*>(p.in) + (size_t)r * p.in_row + c, x);
+        store4(ring + (size_t)(p.positions[r] % p.n_taps) * cols, x);
+    }
+}
+
 template <class TG, class T>
 __global__ void __launch_bounds__(128) attn_plain_kernel(const AttnPlainParams p) {
     extern __shared__ __align__(16) float sm[];
@@ -202,6 +338,31 @@ cudaError_t launch_head_prep(const HeadPrepParams& p, int rows, bool in_f32, boo
     auto go = [&](auto kernel) { return launch_pdl(kernel, grid, dim3(256), smem, st, p); };
     if (f32) return go(head_prep_kernel<float, float>);
     return in_f32 ? go(head_prep_kernel<float, __nv_bfloat16>) : go(head_prep_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
+
+cudaError_t launch_conv_prep(const ConvPrepParams& p, bool in_f32, bool f32, cudaStream_t st) {
+    if (p.rows == 0) return cudaSuccess;
+    const size_t smem = (size_t)8 * p.dim * 4;
+    if (p.dim % 8 || p.in_row % 4 || p.first_dim % 4 || p.first_dim > p.dim || 2 * p.half > p.dim || p.n_taps < 1 || smem > 48 * 1024 || (f32 && !in_f32)) return cudaErrorInvalidValue;
+    constexpr int STRIP = 8;
+    const int groups = (p.n_heads + 2 * p.n_kv_heads + 7) / 8;
+    const bool strips = p.rows >= STRIP * 64 && !in_f32, few = p.dim <= 128 && !f32;
+    auto go = [&](auto kernel, int n) { return launch_pdl(kernel, dim3((p.rows + n - 1) / n, groups), dim3(256), smem, st, p); };
+    using B = __nv_bfloat16;
+#define LLM_CONV_PREP(TAPS) if (few && p.n_taps == TAPS) return in_f32 ? go(conv_prep_kernel<float, B, TAPS, 1>, 1) : strips ? go(conv_prep_kernel<B, B, TAPS, STRIP>, STRIP) : go(conv_prep_kernel<B, B, TAPS, 1>, 1)
+    LLM_CONV_PREP(2);
+    LLM_CONV_PREP(3);
+    LLM_CONV_PREP(4);
+#undef LLM_CONV_PREP
+    if (f32) return go(conv_prep_kernel<float, float, 0, 1>, 1);
+    return in_f32 ? go(conv_prep_kernel<float, B, 0, 1>, 1) : go(conv_prep_kernel<B, B, 0, 1>, 1);
+}
+
+cudaError_t launch_conv_keep(const ConvPrepParams& p, bool in_f32, cudaStream_t st) {
+    if (p.rows == 0 || p.n_taps == 1) return cudaSuccess;
+    if (!p.cu || p.n_seqs > 65535 || p.dim % 4 || p.in_row % 4) return cudaErrorInvalidValue;
+    const dim3 grid(((p.n_heads + 2 * p.n_kv_heads) * p.dim + 1023) / 1024, p.n_seqs);
+    return in_f32 ? launch_pdl(conv_keep_kernel<float>, grid, dim3(256), 0, st, p) : launch_pdl(conv_keep_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, p);
 }
 
 cudaError_t launch_attn_prep(const AttnPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {

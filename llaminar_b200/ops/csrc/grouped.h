@@ -38,6 +38,29 @@ struct HeadPrepParams {
 };
 cudaError_t launch_head_prep(const HeadPrepParams& p, int rows, bool in_f32, bool f32, cudaStream_t st);
 
+// Projected rows [q | k | v | ...] -> a causal convolution over time on each of their channels, then queries and keys rotated (pairs (i, i +
+// half)), queries times their head's temperature, values mixed with those of an earlier layer; appended to the cache like above.  The
+// last taps - 1 rows of a sequence come from `ring` [slots, taps, channels] (position p in place p mod taps, channels = (n_heads + 2
+// n_kv_heads) * dim).  One row per sequence (`cu` nullptr): the row enters the ring here; portions leave it to launch_conv_keep.
+struct ConvPrepParams {
+    const void* in; size_t in_row;                               // channels [0, (n_heads + 2 n_kv_heads) * dim) of a row
+    const float* taps; int n_taps;                               // [n_taps][channels], the newest tap last
+    float* ring; const int* slots; int n_slots;                  // [n_seqs]
+    const int* cu;                                               // [n_seqs + 1] first rows of the sequences, or nullptr
+    const float2* angles; int half;                              // [T, half] (half = 0: no rotation)
+    const float* q_gain;                                         // optional [n_heads]
+    float* first; int first_dim;                                 // optional [T, n_kv_heads, first_dim]: values of the earlier layer
+    const float* share;                                          // v = (1 - share) v + share first; nullptr: `first` receives v
+    const int *positions, *seq_ids, *block_table;
+    int max_pages, n_seqs, n_pages;
+    void* q_out;                                                 // [T, n_heads, dim]
+    void* kv;
+    int n_heads, n_kv_heads, dim, rows;
+};
+cudaError_t launch_conv_prep(const ConvPrepParams& p, bool in_f32, bool f32, cudaStream_t st);
+// the last rows of every portion into the ring (`cu` given)
+cudaError_t launch_conv_keep(const ConvPrepParams& p, bool in_f32, cudaStream_t st);
+
 // Attention of every row over the paged cache in float arithmetic, any size: the 32-bit mode, and shapes without a tensor-core kernel.
 struct AttnPlainParams {
     const void* q; const void* kv; void* out;                    // [T, n_heads, dim], cache, [T, n_heads, dim]

@@ -66,6 +66,48 @@ void head_prep(const Tensor& in, int64_t q_off, int64_t k_off, int64_t v_off, co
     check(llm::launch_head_prep(p, T, in_f32, f32, stream()), "head_prep");
 }
 
+// taps [n, channels], ring [slots, n, channels]; cu: portions of several rows; first [tokens, kv heads, values]
+void conv_prep(const Tensor& in, const Tensor& taps, const Tensor& ring, const Tensor& slots, const OptTensor& cu, const OptTensor& angles, const OptTensor& q_gain,
+               const OptTensor& first, const OptTensor& share, const Tensor& positions, const Tensor& seq_ids, const Tensor& block_table, const Tensor& q_out, const Tensor& kv) {
+    const bool in_f32 = is_f32(in, "in"), f32 = is_f32(kv, "kv");
+    want_like(q_out, f32, "q_out");
+    const int64_t T = in.size(0);
+    if (T == 0) return;
+    TORCH_CHECK(q_out.is_contiguous() && q_out.dim() == 3 && q_out.size(0) == T, "q_out must be [tokens, heads, dim]");
+    const int64_t H = q_out.size(1), D = q_out.size(2), G = kv.size(2), cols = (H + 2 * G) * D, n = taps.size(0);
+    want_cache(kv, D);
+    TORCH_CHECK(in.dim() == 2 && in.stride(1) == 1 && in.size(1) >= cols, "in: too few columns");
+    TORCH_CHECK(positions.numel() == T && seq_ids.numel() == T, "rows");
+    want_aligned(in, "in"); want_aligned(q_out, "q_out");
+    llm::ConvPrepParams p = {};
+    p.in = in.data_ptr(); p.in_row = in.stride(0); p.rows = T;
+    p.taps = floats(taps, n * cols, "taps"); p.n_taps = n;
+    want(ring, torch::kFloat32, "ring");
+    TORCH_CHECK(ring.dim() == 3 && ring.size(1) == n && ring.size(2) == cols, "ring must be [slots, taps, channels]");
+    p.ring = ring.data_ptr<float>(); p.n_slots = ring.size(0);
+    p.n_seqs = slots.numel(); p.slots = ints(slots, "slots");
+    TORCH_CHECK(block_table.size(0) >= p.n_seqs && (cu ? cu->numel() == p.n_seqs + 1 : p.n_seqs == T), "sequences");
+    if (cu) p.cu = ints(*cu, "cu");
+    if (angles) {
+        p.angles = angle_ptr(*angles, T); p.half = angles->size(1);
+        TORCH_CHECK(2 * p.half <= D, "more angles than a head has pairs");
+    }
+    if (q_gain) p.q_gain = floats(*q_gain, H, "q_gain");
+    TORCH_CHECK(!share || first, "shared values missing");
+    if (first) {
+        want(*first, torch::kFloat32, "first");
+        TORCH_CHECK(first->dim() == 3 && first->size(0) == T && first->size(1) == G, "first must be [tokens, kv heads, values]");
+        p.first = first->data_ptr<float>(); p.first_dim = first->size(2);
+        if (share) p.share = floats(*share, 1, "share");
+    }
+    p.positions = ints(positions, "positions"); p.seq_ids = ints(seq_ids, "seq_ids"); p.block_table = ints(block_table, "block_table");
+    p.max_pages = block_table.size(1); p.n_pages = kv.size(0);
+    p.q_out = q_out.data_ptr(); p.kv = kv.data_ptr();
+    p.n_heads = H; p.n_kv_heads = G; p.dim = D;
+    check(llm::launch_conv_prep(p, in_f32, f32, stream()), "conv_prep");
+    if (cu) check(llm::launch_conv_keep(p, in_f32, stream()), "conv_keep");
+}
+
 // gate [tokens, heads] (one number per head) or [tokens, heads * dim]; returns whether it is per head
 bool gate_rows(const OptTensor& gate, int64_t T, int64_t heads, int64_t dim) {
     if (!gate) return false;
@@ -152,6 +194,7 @@ void attn_prefill(const Tensor& q, const Tensor& kv, const Tensor& out, const Te
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("attn_prep", &attn_prep);
     m.def("head_prep", &head_prep);
+    m.def("conv_prep", &conv_prep);
     m.def("attn_plain", &attn_plain);
     m.def("attn_decode", &attn_decode);
     m.def("attn_prefill", &attn_prefill);

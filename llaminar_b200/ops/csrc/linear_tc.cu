@@ -371,7 +371,7 @@ __global__ void __launch_bounds__(32 * SCAN_WARPS) chunk_scan_kernel(const Linea
 // ---- outputs --------------------------------------------------------------------------------------------------------------------
 // A CTA takes 256 values of a head (all of most heads) in two slices, so that the weights are computed once.  Shared memory, in atoms:
 // Q [na] | K, then V of slice 1 [2] | V of slice 0, then gate of slice 1 [2] | state [2 na: hi, lo], of one slice after the other |
-// gate of slice 0 [2].  With the whole head here (`fused`) the norm and the gate follow, otherwise head_gate does them.
+// gate of slice 0 [2].  With the whole head here (`fused`) the norm and the gate follow, otherwise head_gate does them (`raw`: nobody).
 constexpr int T_S = 0, T_P = 128, T_O = 256, T_I = 384;              // TMEM columns: scores (then T_I of slice 1), weights (hi, lo), both parts of o
 // (a barrier that is waited for twice is not used again before every thread has seen its first phase)
 enum OBar { B_QK = 0, B_V, B_V1, B_G, B_G1, B_ST, B_SC, B_IN, B_IN1, B_O, N_OBARS };
@@ -391,7 +391,7 @@ __global__ void __launch_bounds__(THREADS, 1) chunk_out_kernel(const __grid_cons
     const int h = blockIdx.y, v0 = blockIdx.z * 2 * VS, r0 = ck.x, len = ck.y;
     const int na = (p.dim + 63) / 64, nkv = max(na, 2), ksteps = (p.dim + 15) / 16;
     const int slices = p.vdim - v0 > VS ? 2 : 1;
-    const bool lstm = p.gates != nullptr, fused = gridDim.z == 1;
+    const bool lstm = p.gates != nullptr, fused = gridDim.z == 1 && !p.raw;
     const uint32_t base = (smem_u32(smem_raw) + 1023u) & ~1023u;
     const uint32_t sQ = base, sK = sQ + na * ATOM, sV = sK + nkv * ATOM, sS = sV + 2 * ATOM, sG = sS + 2 * na * ATOM;
     const uint32_t bars = smem_u32(s_bars);
@@ -684,7 +684,7 @@ bool linear_chunk_fits(int dim, int vdim) { return dim % 8 == 0 && vdim % 8 == 0
 cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cudaStream_t st) {
     using namespace lin;
     if (c.n_chunks == 0) return cudaSuccess;
-    if (!linear_chunk_fits(p.dim, p.vdim) || p.in_row % 8 || p.q_off % 8 || p.k_off % 8 || p.v_off % 8 || p.g_off % 8 || p.out_row % 8 || p.heads > 65535 || c.n_seqs > 65535 ||
+    if (!linear_chunk_fits(p.dim, p.vdim) || p.in_row % 8 || p.q_off % 8 || p.k_off % 8 || p.v_off % 8 || p.g_off % 8 || p.out_row % 8 || p.silu_in || p.heads > 65535 || c.n_seqs > 65535 ||
         (!p.gates == !p.decay) || (p.gates && p.half))
         return cudaErrorInvalidValue;
     const __nv_bfloat16* in = static_cast<const __nv_bfloat16*>(p.in);
@@ -716,7 +716,7 @@ cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cu
         return e != cudaSuccess ? e : launch_pdl(kernel, out_grid, dim3(THREADS), out_smem(p.dim), st, mq, mk, mv, mg, ms, p, c);
     };
     e = rot ? out(chunk_out_kernel<true>) : out(chunk_out_kernel<false>);
-    return e != cudaSuccess || out_grid.z == 1 ? e : launch_head_gate(p, c.o, c.rows, st);
+    return e != cudaSuccess || p.raw || out_grid.z == 1 ? e : launch_head_gate(p, c.o, c.rows, st);
 }
 
 int bounds_status_linear_tc(bool reset);

@@ -6,6 +6,7 @@
 //                  The CTAs of a cluster exchange the sums of squares of their slices through distributed shared memory for the
 //                  norm of the head's output.
 //   head_gate      norm and gate of the heads' outputs behind the chunk kernels (linear_tc.cu)
+//   joint_gate     norm over all heads together and gate
 #include <cooperative_groups.h>
 
 #include "common.cuh"
@@ -52,6 +53,8 @@ LLM_DEVICE float block_sum(float v, float* red) {
 
 // ---- linear attention ------------------------------------------------------------------------------------------------------
 constexpr int LIN_THREADS = 256, LIN_ROWS = 4;         // state rows in flight per warp
+
+LLM_DEVICE float silu_exact(float x) { return x / (1.f + expf(-x)); }
 
 // value i of a head's q or k: pairs (i, i + half) turn, the rest passes
 template <class TI> LLM_DEVICE float rotated(const TI* x, int i, const float2* ang, int half) {
@@ -125,7 +128,9 @@ __global__ void __launch_bounds__(LIN_THREADS, 3) linear_rows_kernel(const Linea
         }
         float nq = 0.f;
         for (int i = threadIdx.x; i < D; i += LIN_THREADS) {
-            const float a = rotated(q, i, ang, p.half) * p.q_scale, c = rotated(k, i, ang, p.half) * p.k_scale;
+            float a = rotated(q, i, ang, p.half), c = rotated(k, i, ang, p.half);
+            if (p.silu_in) { a = silu_exact(a); c = silu_exact(c); }
+            a *= p.q_scale; c *= p.k_scale;
             s_q[i] = a;
             s_k[i] = c;
             if (lstm) {
@@ -134,7 +139,7 @@ __global__ void __launch_bounds__(LIN_THREADS, 3) linear_rows_kernel(const Linea
                 nq += x * a;
             }
         }
-        for (int i = threadIdx.x; i < nv; i += LIN_THREADS) s_v[i] = to_f(v[i]);
+        for (int i = threadIdx.x; i < nv; i += LIN_THREADS) s_v[i] = p.silu_in ? silu_exact(to_f(v[i])) : to_f(v[i]);
         if (lstm) den = 1.f / (fmaxf(fabsf(block_sum<LIN_THREADS>(nq, red)), expf(-m)) + NORM_FLOOR);
         else __syncthreads();
         for (int r = warp * LIN_ROWS; r < nv; r += LIN_THREADS / 32 * LIN_ROWS) {
@@ -175,6 +180,12 @@ __global__ void __launch_bounds__(LIN_THREADS, 3) linear_rows_kernel(const Linea
             }
         }
         __syncthreads();
+        if (p.raw) {
+            for (int i = threadIdx.x; i < nv; i += LIN_THREADS) out[(size_t)t * p.out_row + h * p.vdim + v0 + i] = from_f<TO>(s_o[i] * den);
+            fresh = false;
+            __syncthreads();
+            continue;
+        }
         float ss = 0.f;
         for (int i = threadIdx.x; i < nv; i += LIN_THREADS) { const float o = s_o[i] * den; ss += o * o; }
         ss = block_sum<LIN_THREADS>(ss, red);
@@ -246,7 +257,60 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const LinearParams p, co
     }
 }
 
+// a CTA per token
+template <class TI, class T>
+__global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p) {
+    __shared__ float red[8];
+    pdl_trigger();
+    pdl_wait();
+    const size_t t = blockIdx.x;
+    const TI *o = static_cast<const TI*>(p.o) + t * p.o_row, *g = static_cast<const TI*>(p.in) + t * p.in_row + p.g_off;
+    T* dst = static_cast<T*>(p.out) + t * p.out_row;
+    constexpr int UN = 4;                              // units of four values a thread keeps; the rest of wider rows is read again
+    float keep[UN][4], z[UN][4], x[4], y[4], w[4], ss = 0.f;
+#pragma unroll
+    for (int u = 0; u < UN; ++u) {
+        const int i = (u * 256 + threadIdx.x) * 4;
+        keep[u][0] = keep[u][1] = keep[u][2] = keep[u][3] = 0.f;
+        if (i < p.n) { load4(o + i, keep[u]); load4(g + i, z[u]); }
+    }
+#pragma unroll
+    for (int u = 0; u < UN; ++u)
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss += keep[u][j] * keep[u][j];
+    for (int i = (UN * 256 + threadIdx.x) * 4; i < p.n; i += 1024) {
+        load4(o + i, x);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss += x[j] * x[j];
+    }
+    const float inv = 1.f / sqrtf(block_sum<256>(ss, red) / (float)p.true_n + p.eps);
+    auto put = [&](int i, const float (&v)[4], const float (&s)[4]) {
+        load4(p.norm_w + i, w);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) y[j] = v[j] * inv * w[j] / (1.f + expf(-s[j]));
+        store4(dst + i, y);
+    };
+#pragma unroll
+    for (int u = 0; u < UN; ++u) {
+        const int i = (u * 256 + threadIdx.x) * 4;
+        if (i < p.n) put(i, keep[u], z[u]);
+    }
+    for (int i = (UN * 256 + threadIdx.x) * 4; i < p.n; i += 1024) {
+        float s[4];
+        load4(o + i, x); load4(g + i, s);
+        put(i, x, s);
+    }
+}
+
 }  // namespace
+
+cudaError_t launch_joint_gate(const JointGateParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {
+    if (rows == 0) return cudaSuccess;
+    if (p.n % 4 || p.o_row % 4 || p.in_row % 4 || p.g_off % 4 || p.out_row % 4 || (f32 && !in_f32)) return cudaErrorInvalidValue;
+    auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(256), 0, st, p); };
+    if (f32) return go(joint_gate_kernel<float, float>);
+    return in_f32 ? go(joint_gate_kernel<float, __nv_bfloat16>) : go(joint_gate_kernel<__nv_bfloat16, __nv_bfloat16>);
+}
 
 cudaError_t launch_linear_rows(const LinearParams& p, int n_seqs, bool in_f32, bool f32, cudaStream_t st) {
     if (n_seqs == 0) return cudaSuccess;

@@ -8,7 +8,7 @@
 
 namespace llm {
 
-// Linear attention with a recurrent state per head: mLSTM (with `gates`) or retention (with `decay`).
+// Linear attention with a recurrent state per head: mLSTM (with `gates`), or a fixed decay (retention, lightning attention).
 struct LinearParams {
     const void* in; size_t in_row;                               // projected rows; head h of q starts at q_off + h * dim
     int q_off, k_off, v_off, g_off;
@@ -24,6 +24,8 @@ struct LinearParams {
     int n_slots, heads, dim, vdim, true_vdim;                    // padded to multiples of 8
     const float* norm_w;                                         // optional [heads * vdim]
     int silu;                                                    // output gate: silu or sigmoid
+    int silu_in;                                                 // q, k and v pass through silu first (row-wise kernel; the chunk kernels want them so)
+    int raw;                                                     // o as it is, without norm and gate (`g_off` unused)
     void* out; size_t out_row;                                   // [T, heads * vdim]
     float eps;
 };
@@ -46,6 +48,17 @@ bool linear_chunk_fits(int dim, int vdim);
 cudaError_t launch_linear_chunk(const LinearParams& p, const LinearChunks& c, cudaStream_t st);
 // out[t, h] = o[t, h] / rms(o[t, h]) * norm_w * gate(in[t, g_off + ...]), bf16
 cudaError_t launch_head_gate(const LinearParams& p, const __nv_bfloat16* o, int rows, cudaStream_t st);
+
+// out[t] = o[t] / rms(o[t]) * norm_w * sigmoid(in[t, g_off + ...]): norm over all heads' n values together, `true_n` of them not padding.
+struct JointGateParams {
+    const void* o; size_t o_row;                                 // float or bf16, as `in`
+    const void* in; size_t in_row; int g_off;
+    const float* norm_w;                                         // [n]
+    void* out; size_t out_row;
+    int n, true_n;
+    float eps;
+};
+cudaError_t launch_joint_gate(const JointGateParams& p, int rows, bool in_f32, bool f32, cudaStream_t st);
 
 int bounds_status_mixers(bool reset);
 int bounds_status_linear_tc(bool reset);

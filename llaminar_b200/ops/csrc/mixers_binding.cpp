@@ -16,8 +16,9 @@ void want_aligned(const Tensor& t, const char* name) { TORCH_CHECK(reinterpret_c
 // What the linear-attention entry points share.  offs: first columns of q, k, v, g; state: S (, n, m); gates with bias_i, bias_f, cap: mLSTM; decay: retention
 llm::LinearParams linear_params(const Tensor& in, const std::vector<int64_t>& offs, const OptTensor& gates, const OptTensor& bias_i, const OptTensor& bias_f, double cap,
                                 const OptTensor& decay, const OptTensor& angles, double q_scale, double k_scale, const OptTensor& cu, const Tensor& positions,
-                                const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps) {
+                                const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps, bool silu_in, bool raw) {
     llm::LinearParams p = {};
+    p.silu_in = silu_in; p.raw = raw;
     is_f32(in, "in");
     const int64_t T = in.size(0);
     TORCH_CHECK(offs.size() == 4 && (state.size() == 1 || state.size() == 3), "offsets / state");
@@ -60,8 +61,8 @@ llm::LinearParams linear_params(const Tensor& in, const std::vector<int64_t>& of
 
 void linear_rows(const Tensor& in, const std::vector<int64_t>& offs, const OptTensor& gates, const OptTensor& bias_i, const OptTensor& bias_f, double cap,
                  const OptTensor& decay, const OptTensor& angles, double q_scale, double k_scale, const OptTensor& cu, const Tensor& positions,
-                 const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps) {
-    const llm::LinearParams p = linear_params(in, offs, gates, bias_i, bias_f, cap, decay, angles, q_scale, k_scale, cu, positions, slots, state, true_vdim, norm_w, silu, out, eps);
+                 const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps, bool silu_in, bool raw) {
+    const llm::LinearParams p = linear_params(in, offs, gates, bias_i, bias_f, cap, decay, angles, q_scale, k_scale, cu, positions, slots, state, true_vdim, norm_w, silu, out, eps, silu_in, raw);
     check(llm::launch_linear_rows(p, slots.numel(), is_f32(in, "in"), is_f32(out, "out"), stream()), "linear_rows");
 }
 
@@ -69,8 +70,8 @@ void linear_rows(const Tensor& in, const std::vector<int64_t>& offs, const OptTe
 void linear_chunk(const Tensor& in, const std::vector<int64_t>& offs, const OptTensor& gates, const OptTensor& bias_i, const OptTensor& bias_f, double cap,
                   const OptTensor& decay, const OptTensor& angles, double q_scale, double k_scale, const Tensor& cu, const Tensor& positions,
                   const Tensor& slots, const std::vector<Tensor>& state, int64_t true_vdim, const OptTensor& norm_w, bool silu, const Tensor& out, double eps,
-                  const Tensor& chunks, const Tensor& seqs, const Tensor& scratch, const Tensor& vec, const Tensor& scal, const OptTensor& gate, const Tensor& o, const Tensor& status) {
-    const llm::LinearParams p = linear_params(in, offs, gates, bias_i, bias_f, cap, decay, angles, q_scale, k_scale, cu, positions, slots, state, true_vdim, norm_w, silu, out, eps);
+                  const Tensor& chunks, const Tensor& seqs, const Tensor& scratch, const Tensor& vec, const Tensor& scal, const OptTensor& gate, const Tensor& o, const Tensor& status, bool raw) {
+    const llm::LinearParams p = linear_params(in, offs, gates, bias_i, bias_f, cap, decay, angles, q_scale, k_scale, cu, positions, slots, state, true_vdim, norm_w, silu, out, eps, false, raw);
     bf16(in, "in"); bf16(out, "out");
     llm::LinearChunks c = {};
     auto table = [](const Tensor& t, const char* name) {
@@ -96,11 +97,28 @@ void linear_chunk(const Tensor& in, const std::vector<int64_t>& offs, const OptT
     check(llm::launch_linear_chunk(p, c, stream()), "linear_chunk");
 }
 
+// o, in and out have a row per token; the gate stands in columns [g_off, g_off + n) of in
+void joint_gate(const Tensor& o, const Tensor& in, int64_t g_off, const Tensor& norm_w, int64_t true_n, const Tensor& out, double eps) {
+    llm::JointGateParams p = {};
+    const bool in_f32 = is_f32(in, "in"), f32 = is_f32(out, "out");
+    want_like(o, in_f32, "o");
+    const int64_t T = o.size(0), n = o.size(1);
+    TORCH_CHECK(o.dim() == 2 && out.sizes() == o.sizes() && in.dim() == 2 && in.size(0) == T && o.stride(1) == 1 && in.stride(1) == 1 && out.stride(1) == 1, "joint_gate rows");
+    TORCH_CHECK(g_off >= 0 && g_off + n <= in.size(1) && true_n >= 1 && true_n <= n, "joint_gate columns");
+    want_aligned(o, "o"); want_aligned(in, "in"); want_aligned(out, "out"); want_aligned(norm_w, "norm_w");
+    p.o = o.data_ptr(); p.o_row = o.stride(0); p.in = in.data_ptr(); p.in_row = in.stride(0); p.g_off = g_off;
+    p.norm_w = floats(norm_w, n, "norm_w");
+    p.out = out.data_ptr(); p.out_row = out.stride(0);
+    p.n = n; p.true_n = true_n; p.eps = eps;
+    check(llm::launch_joint_gate(p, T, in_f32, f32, stream()), "joint_gate");
+}
+
 }  // namespace
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
     m.def("linear_rows", &linear_rows);
     m.def("linear_chunk", &linear_chunk);
+    m.def("joint_gate", &joint_gate);
     m.def("linear_chunk_fits", &llm::linear_chunk_fits);
     m.attr("LINEAR_CHUNK") = llm::LINEAR_CHUNK;
     m.def("set_pdl", [](bool on) { llm::pdl_enabled() = on; });

@@ -11,7 +11,7 @@ from . import _count
 from . import build as _build
 
 GEMV_MAX_ROWS = 8
-ACT_NONE, ACT_GELU_MUL, ACT_RELU2, ACT_GELU_SIDE, ACT_SILU_MUL, ACT_GATE = range(6)
+ACT_NONE, ACT_GELU_MUL, ACT_RELU2, ACT_GELU_SIDE, ACT_SILU_MUL, ACT_GATE, ACT_GELU, ACT_SILU = range(8)
 _ready = False
 
 
@@ -35,8 +35,18 @@ def resid_norm(h, y=None, w_post=None, *, add=True, y_rows=None, w_next=None, xn
     _count()
 
 
+def depth_mix(h, y=None, z=None, *, add=True, y_rows=None, z_rows=None, z_w=None, past=None, n_past: int = 0, w=None, norms=(), eps: float) -> None:
+    """x = (h if add) + y + z, rows of either gathered by ``y_rows`` / ``z_rows``, z the sum of a token's rows times ``z_w`` [tokens,
+    parts] if given; h = sum of w[j] past[j] over j < n_past plus w[n_past] x, and past[n_past] = x if ``past`` [streams, tokens, d] has that
+    stream.  ``norms``: up to two (gain, output) pairs of RMSNorms of h, gains of one value or of d.  One launch."""
+    (g0, x0), (g1, x1) = (*norms, (None, None), (None, None))[:2]
+    ext().depth_mix(h, add, y, y_rows, z, z_rows, z_w, past, n_past, w, g0, x0, g1, x1, eps)
+    _count()
+
+
 def activate(x: torch.Tensor, act: torch.Tensor, kind: int, side=None) -> None:
-    """act = gelu_tanh(x[:, :n]) * x[:, n:] (ACT_GELU_MUL), the same with silu (ACT_SILU_MUL), squared relu (ACT_RELU2), gelu_tanh(x) times
+    """act = gelu_tanh(x[:, :n]) * x[:, n:] (ACT_GELU_MUL), the same with silu (ACT_SILU_MUL), both without a second half (ACT_GELU, ACT_SILU),
+    squared relu (ACT_RELU2), gelu_tanh(x) times
     columns of each token's row of a table (ACT_GELU_SIDE; ``side``: table, first column, columns, tokens), or x times the sigmoid of
     those columns of the row itself (ACT_GATE; tokens None).  ``act`` may be ``x``, except for the pairs."""
     ext().activate(x, act, kind, *(side or (None, 0, 0, None)))

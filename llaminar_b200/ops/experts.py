@@ -28,10 +28,10 @@ def max_pairs() -> int:
     return ext().MAX_PAIRS
 
 
-def expert_route(bias, ids, weights, x=None, router=None, logits=None, counts=None, ranks=None) -> None:
+def expert_route(bias, ids, weights, x=None, router=None, logits=None, counts=None, ranks=None, groups: int = 1, keep: int = 1) -> None:
     """Router logits (x router^T, or given) + bias in 32-bit -> the ``top`` largest (``ids`` [tokens, top]) and the softmax over just
-    those.  ``counts`` (zeroed) and ``ranks``: pairs per expert, and the number of a pair among those of its expert.  One launch."""
-    ext().expert_route(x, router, logits, bias, ids, weights, counts, ranks)
+    those.  With several ``groups`` of neighbours only the experts of the ``keep`` groups with the largest logits count.  ``counts`` (zeroed) and ``ranks``: pairs per expert, and the number of a pair among those of its expert.  One launch."""
+    ext().expert_route(x, router, logits, bias, ids, weights, counts, ranks, groups, keep)
     _count()
 
 
@@ -41,21 +41,22 @@ def expert_place(x, ids, ranks, counts, place, xs) -> None:
     _count()
 
 
-def expert_rows(w, x, ids, out, div: int, pair_act: bool) -> None:
-    """out[pair] = x[pair // div] w[ids[pair]]^T for few pairs (bf16); ``pair_act``: w stacks gate and up, out = silu(gate) * up."""
-    ext().expert_rows(w, x, ids, out, div, pair_act)
+def expert_rows(w, x, ids, out, div: int, pair_act: bool, limit: float = 0.0) -> None:
+    """out[pair] = x[pair // div] w[ids[pair]]^T for few pairs (bf16); ``pair_act``: w stacks gate and up, out = silu(gate) * up, or
+    with a ``limit`` g sigmoid(1.702 g) (u + 1) of the clamped values."""
+    ext().expert_rows(w, x, ids, out, div, pair_act, limit)
     _count()
 
 
-def expert_plain(w, x, ids, out, div: int, pair_act: bool) -> None:
+def expert_plain(w, x, ids, out, div: int, pair_act: bool, limit: float = 0.0) -> None:
     """As `expert_rows` in float arithmetic: 32-bit mode, and sizes without a tensor-core kernel."""
-    ext().expert_plain(w, x, ids, out, div, pair_act)
+    ext().expert_plain(w, x, ids, out, div, pair_act, limit)
     _count()
 
 
-def expert_grouped(w, x, counts, out, pair_act: bool, status) -> None:
+def expert_grouped(w, x, counts, out, pair_act: bool, status, limit: float = 0.0) -> None:
     """The same product for rows sorted by expert (tcgen05): ``counts`` rows of each."""
-    ext().expert_grouped(w, x, counts, out, pair_act, status)
+    ext().expert_grouped(w, x, counts, out, pair_act, status, limit)
     _count()
 
 

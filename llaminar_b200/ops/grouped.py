@@ -39,6 +39,15 @@ def head_prep(rows, q_off: int, k_off: int, v_off: int, q_norm, k_norm, angles, 
     _count()
 
 
+def conv_prep(rows, taps, ring, slots, cu, angles, q_gain, first, share, positions, seq_ids, block_table, q_out, kv) -> None:
+    """Projected rows [q | k | v | ...] -> queries [tokens, heads, dim] and the tokens' entries of the paged cache, every channel passed
+    through a causal convolution over time (``taps`` [n, channels], the last rows of each sequence in its slot of ``ring``), queries and
+    keys rotated, queries times ``q_gain`` of their head.  ``first`` [tokens, kv heads, values]: receives the values, or with ``share``
+    brings those of an earlier layer that are mixed in.  One launch; with ``cu`` (portions of prompts) another one for the ring."""
+    ext().conv_prep(rows, taps, ring, slots, cu, angles, q_gain, first, share, positions, seq_ids, block_table, q_out, kv)
+    _count(1 if cu is None or taps.shape[0] == 1 else 2)
+
+
 def attn_plain(q, kv, out, positions, seq_ids, block_table, window: int, scale: float, sink, gate, chunk: int = 0, softcap: float = 0.0) -> None:
     """Attention of any rows in float arithmetic: 32-bit mode, and shapes without a tensor-core kernel."""
     ext().attn_plain(q, kv, out, positions, seq_ids, block_table, window, scale, sink, gate, chunk, softcap)

@@ -23,11 +23,12 @@ def ext():
 
 
 def linear_rows(rows, offs, gates, decay, angles, q_scale: float, k_scale: float, cu, positions, slots, state, true_vdim: int, norm_w,
-                silu: bool, out, eps: float) -> None:
-    """mLSTM (``gates``: float rows of gate projections, input biases, forget biases, cap) or retention (``decay``), the rows of a
-    sequence one after the other; ``cu`` None: one row per sequence.  The state of ``slots`` is advanced in place."""
+                silu: bool, out, eps: float, silu_in: bool = False, raw: bool = False) -> None:
+    """mLSTM (``gates``: float rows of gate projections, input biases, forget biases, cap) or a fixed ``decay`` (retention, lightning
+    attention), the rows of a sequence one after the other; ``cu`` None: one row per sequence.  The state of ``slots`` is advanced in
+    place.  ``silu_in``: q, k and v pass through silu first; ``raw``: the outputs without norm and gate."""
     g = gates or (None, None, None, 1.0)
-    ext().linear_rows(rows, list(offs), *g, decay, angles, q_scale, k_scale, cu, positions, slots, list(state), true_vdim, norm_w, silu, out, eps)
+    ext().linear_rows(rows, list(offs), *g, decay, angles, q_scale, k_scale, cu, positions, slots, list(state), true_vdim, norm_w, silu, out, eps, silu_in, raw)
     _count()
 
 
@@ -51,17 +52,24 @@ def linear_chunk_fits(dim: int, vdim: int) -> bool:
 
 
 def linear_chunk(rows, offs, gates, decay, angles, q_scale: float, k_scale: float, cu, positions, slots, state, true_vdim: int, norm_w,
-                 silu: bool, out, eps: float, tables, raw, status) -> None:
+                 silu: bool, out, eps: float, tables, raw, status, only_raw: bool = False) -> None:
     """As `linear_rows` for prompts in bf16, chunk-parallel on the tensor cores.  ``tables``: see `chunk_tables`; ``raw``: workspace
-    like ``out``."""
+    like ``out``, with ``only_raw`` the result (without norm and gate; ``out`` is not written)."""
     g = gates or (None, None, None, 1.0)
     chunks, seqs = tables
     _, h, v, d = state[0].shape
     n = chunks.shape[0]
     f = lambda *s: torch.empty(*s, dtype=torch.float32, device=rows.device)
     ext().linear_chunk(rows, list(offs), *g, decay, angles, q_scale, k_scale, cu, positions, slots, list(state), true_vdim, norm_w, silu, out, eps,
-                       chunks, seqs, f(n, h, v, d), f(n, h, d), f(n, h, 4), f(n, h, ext().LINEAR_CHUNK, 4) if gates else None, raw, status)
-    _count(4 if v > 256 else 3)
+                       chunks, seqs, f(n, h, v, d), f(n, h, d), f(n, h, 4), f(n, h, ext().LINEAR_CHUNK, 4) if gates else None, raw, status, only_raw)
+    _count(4 if v > 256 and not only_raw else 3)
+
+
+def joint_gate(o, rows, g_off: int, norm_w, true_n: int, out, eps: float) -> None:
+    """out = o / rms(o) * norm_w * sigmoid(gate columns of ``rows``), the root mean square over a whole row (``true_n`` values that are
+    not padding)."""
+    ext().joint_gate(o, rows, g_off, norm_w, true_n, out, eps)
+    _count()
 
 
 def bounds_status(reset: bool = True) -> int:

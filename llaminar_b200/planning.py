@@ -165,8 +165,8 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
             pages = batch_size * ((ctx_size + 63) // 64 + 1) + 64
             stage_layers = range(first, last + 1)
             rp.kv_bytes = int(pages * len(cfg.kv_layers(stage_layers)) * 2 * tp.n_kv_local * 64 * cfg.head_dim * 2)
-            if cfg.has_mixers:                  # side embedding of the layers, input matrix of the looped ones
-                rp.weight_bytes += 2 * cfg.vocab_size * cfg.side_dim * cfg.n_layers + (4 * cfg.d_model * cfg.d_model if cfg.loop else 0)
+            if cfg.has_mixers:                  # side embedding of the layers, input matrix of the looped ones, table of positions
+                rp.weight_bytes += 2 * cfg.vocab_size * cfg.side_dim * cfg.n_layers + (4 * cfg.d_model * cfg.d_model if cfg.loop else 0) + 2 * cfg.learned_positions * cfg.d_model
                 from .engine.kv_cache import LayerStates, PagedKVCache
                 rp.kv_bytes = pages * PagedKVCache.bytes_per_page(0, 0, 0, layer_shapes=mixer_kv_shapes(cfg)) + (batch_size + 1) * LayerStates.bytes_per_slot(mixer_state_shapes(cfg))
             if cfg.is_hybrid:
@@ -181,7 +181,8 @@ def build_plan(cfg: ModelConfig, layout: dict, recipe: QuantRecipe | str = "Q4_K
                                            + 2 * tp.n_heads_local * cfg.head_dim * 2 + ff * 2))
             if cfg.has_mixers:                  # every chosen expert has its rows
                 experts = max((e.top * (2 * cfg.d_model + 3 * e.ff) for e in cfg.layer_experts if e), default=0)
-                rp.activation_bytes = int(T * (cfg.d_model * (4 + 8) + 2 * (max(mixer_columns(m) for m in cfg.mixers) + max(3 * max(cfg.layer_ff), experts))))
+                streams = cfg.n_layers + 1 if cfg.depth_average else 0          # results of all layers, kept for the average
+                rp.activation_bytes = int(T * (cfg.d_model * (4 + 8 + 4 * streams) + 2 * (max(mixer_columns(m) for m in cfg.mixers) + max(3 * max(cfg.layer_ff), experts))))
             rp.workspace_bytes = int(256 * 65536 * 4 + (1 << 22) * 4 + batch_size * 4 * (tp.vocab_stop - tp.vocab_start) * 4)
             if rp.total_bytes > hbm_bytes * 0.95:
                 plan.errors.append(f"rank {rank} ({dev}): needs {rp.total_bytes / 1e9:.1f} GB, device has {hbm_bytes / 1e9:.0f} GB")
