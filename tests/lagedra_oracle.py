@@ -251,7 +251,7 @@ def random_model(layers, seed=0, vocab=97, width=48, eps=1e-5, gain=1.0, max_pos
                 t[f"{p}mix.{x}.conv"] = (rnd(n, m["conv"]) * 0.5 + (torch.arange(m["conv"]) == m["conv"] - 1)).to(bf)
             t[p + "mix.temp"] = (rnd(H) * 0.4 + 1.2).to(bf)
             if m.get("v_mix"):
-                num(p + "mix.vmix", 0.5, 0.2)
+                num(p + "mix.vmix", 0.75, 0.1)
         mat(p + "mix.o", width, H * vd)
         f = e.get("mlp")
         if f:
@@ -263,7 +263,7 @@ def random_model(layers, seed=0, vocab=97, width=48, eps=1e-5, gain=1.0, max_pos
                 mat(p + "mlp.router", n, width, 3.0)
                 for x in range(n):
                     mat(f"{p}mlp.e{x}.gate", ff, width, 1.5), mat(f"{p}mlp.e{x}.up", ff, width, 1.5), mat(f"{p}mlp.e{x}.down", width, ff)
-        w = rnd(i + 2) * 0.3
+        w = rnd(i + 2) * 0.2
         w[i + 1] += 1.0
         t[p + "dwa"] = w.to(bf)
     num("final.norm")
@@ -275,7 +275,7 @@ def dense(ff=56):
     return {"kind": "dense", "ff": ff}
 
 
-def moe(experts=6, top=2, ff=40, count=3, keep=2, limit=1.5):
+def moe(experts=6, top=2, ff=40, count=2, keep=1, limit=1.5):
     return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": {"experts": experts, "top": top, "groups": {"count": count, "keep": keep}}}
 
 
