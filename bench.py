@@ -48,6 +48,7 @@ def parse_args():
     ap.add_argument("--latent", action="store_true", help="instead of the headline: kernels and models with latent attention beside the like parts of a grouped-query model")
     ap.add_argument("--experts", action="store_true", help="instead of the headline: kernels and models with routed experts and gated attention (kefasun) beside the like parts of the other families")
     ap.add_argument("--mixers", action="store_true", help="instead of the headline: kernels and models with recurrent mixers (zogepel) beside the like parts of the other families")
+    ap.add_argument("--parallel", action="store_true", help="instead of the headline: kernels and models with parallel layers, lightning and convolved attention (lagedra) beside the like parts of the other families")
     return ap.parse_args()
 
 
@@ -287,7 +288,7 @@ def log(msg: str) -> None:
 
 T_START = time.time()
 MODEL_DEFAULTS = {"qwen3-8b": ("Q4_K_M", 2048), "qwen3-32b": ("Q4_K_S", 1024),
-                  "pozivik-8b": ("BF16", 2048), "zogepel-8b": ("BF16", 2048), "kefasun-8b": ("BF16", 2048), "qwen3.5-27b": ("Q4_K_M", 512), "qwen3.5-35b-a3b": ("Q4_K_M", 512)}      # the hybrid shapes (--model ...)
+                  "pozivik-8b": ("BF16", 2048), "zogepel-8b": ("BF16", 2048), "kefasun-8b": ("BF16", 2048), "lagedra-8b": ("BF16", 2048), "qwen3.5-27b": ("Q4_K_M", 512), "qwen3.5-35b-a3b": ("Q4_K_M", 512)}      # the hybrid shapes (--model ...)
 
 
 def measure(model_name: str, recipe: str, S: int, args, tp, dev, world: int, rank: int, local: int, extras_on: bool) -> dict:
@@ -434,9 +435,9 @@ def main():
     _keep_stdout_for_the_result()
     if args.impl == "reference":
         return reference_arm(args)
-    if args.latent or args.mixers or args.experts:
+    what = next((w for w in ("latent", "mixers", "experts", "parallel") if getattr(args, w)), None)
+    if what:
         import importlib
-        what = "latent" if args.latent else "mixers" if args.mixers else "experts"
         sampler = ClockSampler(0)
         sampler.start()
         res = importlib.import_module(f"llaminar_b200.bench_{what}").run(args.layers or 8, log)
