@@ -286,6 +286,24 @@ __global__ void __launch_bounds__(THREADS) resid_norm_reg_kernel(const ResidNorm
     });
 }
 
+LLM_DEVICE void load8(const float* p, float (&v)[8]) {
+    const float4 a = *reinterpret_cast<const float4*>(p), b = *reinterpret_cast<const float4*>(p + 4);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+LLM_DEVICE void load8(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {a.x, a.y, a.z, a.w};
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { v[2 * j] = bf16_lo(w[j]); v[2 * j + 1] = bf16_hi(w[j]); }
+}
+LLM_DEVICE void store8(float* p, const float (&v)[8]) {
+    *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
+    *reinterpret_cast<float4*>(p + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+LLM_DEVICE void store8(__nv_bfloat16* p, const float (&v)[8]) {
+    *reinterpret_cast<uint4*>(p) = make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
+}
+
 // See DepthMixParams.  A CTA per row; a thread holds NV x VEC of its values (VEC = 1: of any alignment).
 template <class T, int VEC, int THREADS, int NV, bool PARTS>
 __global__ void __launch_bounds__(THREADS) depth_mix_kernel(const DepthMixParams p) {
@@ -395,16 +413,27 @@ __global__ void __launch_bounds__(THREADS) depth_mix_kernel(const DepthMixParams
     norm(p.gain1, p.xn1);
 }
 
+// For results that are rounded to 16 bits: approximate exponential and quotient (relative errors of some 1e-6).  gelu's
+// (1 + tanh(w)) / 2 is the logistic function of 2w.
+template <class T> LLM_DEVICE float logistic_for(float x) {
+    if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+    else return logistic(x);
+}
+template <class T> LLM_DEVICE float gelu_for(float z) {
+    if constexpr (sizeof(T) == 2) return z * logistic_for<T>(1.5957691216057308f * (z + 0.044715f * z * z * z));
+    else return gelu_tanh(z);
+}
+
 // value `i` of row `t` of the activation of `x`; `u`: the second half's value (GELU_MUL, SILU_MUL)
 template <int ACT, class T>
 LLM_DEVICE float activated(float x, float u, const SideTable& s, int t, int i) {
-    if (ACT == ACT_GELU_MUL) return gelu_tanh(x) * u;
-    if (ACT == ACT_SILU_MUL) return x * logistic(x) * u;
-    if (ACT == ACT_GATE) return x * logistic(to_f(static_cast<const T*>(s.table)[(size_t)t * s.row + i]));
+    if (ACT == ACT_GELU_MUL) return gelu_for<T>(x) * u;
+    if (ACT == ACT_SILU_MUL) return x * logistic_for<T>(x) * u;
+    if (ACT == ACT_GATE) return x * logistic_for<T>(to_f(static_cast<const T*>(s.table)[(size_t)t * s.row + i]));
     if (ACT == ACT_RELU2) { x = fmaxf(x, 0.f); return x * x; }
-    if (ACT == ACT_GELU) return gelu_tanh(x);
-    if (ACT == ACT_SILU) return x * logistic(x);
-    if (ACT == ACT_GELU_SIDE) return i < s.cols ? gelu_tanh(x) * to_f(static_cast<const T*>(s.table)[(size_t)LLM_CHECK_INDEX(s.tokens[t], s.n_rows) * s.row + i]) : 0.f;
+    if (ACT == ACT_GELU) return gelu_for<T>(x);
+    if (ACT == ACT_SILU) return x * logistic_for<T>(x);
+    if (ACT == ACT_GELU_SIDE) return i < s.cols ? gelu_for<T>(x) * to_f(static_cast<const T*>(s.table)[(size_t)LLM_CHECK_INDEX(s.tokens[t], s.n_rows) * s.row + i]) : 0.f;
     return x;
 }
 
@@ -414,17 +443,17 @@ __global__ void __launch_bounds__(256) activate_kernel(const T* x, size_t x_row,
     pdl_wait();
     const T* g = x + (size_t)blockIdx.y * x_row;
     T* a = act + (size_t)blockIdx.y * act_row;
-    const int i0 = (blockIdx.x * 256 + threadIdx.x) * 4;
-    if ((n | x_row | act_row) % 4 == 0) {
+    const int i0 = (blockIdx.x * 256 + threadIdx.x) * 8;
+    if ((n | x_row | act_row) % 8 == 0) {
         if (i0 >= n) return;
-        float v[4], u[4] = {};
-        Vec4<T>::load(g + i0, v);
-        if (act_pairs(ACT)) Vec4<T>::load(g + n + i0, u);
+        float v[8], u[8] = {};
+        load8(g + i0, v);
+        if (act_pairs(ACT)) load8(g + n + i0, u);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) v[j] = activated<ACT, T>(v[j], u[j], s, blockIdx.y, i0 + j);
-        Vec4<T>::store(a + i0, v);
+        for (int j = 0; j < 8; ++j) v[j] = activated<ACT, T>(v[j], u[j], s, blockIdx.y, i0 + j);
+        store8(a + i0, v);
     } else {
-        for (int i = i0; i < min(n, i0 + 4); ++i)
+        for (int i = i0; i < min(n, i0 + 8); ++i)
             a[i] = from_f<T>(activated<ACT, T>(to_f(g[i]), act_pairs(ACT) ? to_f(g[n + i]) : 0.f, s, blockIdx.y, i));
     }
 }
@@ -564,7 +593,7 @@ cudaError_t launch_resid_norm(const ResidNormParams& p, int rows, bool f32, cuda
 }
 
 cudaError_t launch_activate(const void* x, size_t x_row, void* act, size_t act_row, int rows, int n, int kind, const SideTable& side, bool f32, cudaStream_t st) {
-    const dim3 grid((n + 1023) / 1024, rows);
+    const dim3 grid((n + 2047) / 2048, rows);
     if (rows > 65535) return cudaErrorInvalidValue;
     auto go = [&](auto k32, auto k16) {
         if (f32) return launch_pdl(k32, grid, dim3(256), 0, st, static_cast<const float*>(x), x_row, static_cast<float*>(act), act_row, n, side);

@@ -29,13 +29,31 @@ LLM_DEVICE void load8(const float* p, float (&v)[8]) {
 }
 
 // ---- routing -------------------------------------------------------------------------------------------------------------------
+// A warp's view of which groups of experts may be chosen: up to 32 groups as a bit mask, more in shared memory.
+struct Groups {
+    unsigned mask;                                 // of the groups that stay
+    const unsigned* g;                             // zero where a group stays; nullptr: the mask holds
+    int size;                                      // experts of a group (0: all may be chosen)
+    LLM_DEVICE bool stays(int i) const { return size == 0 || (g ? g[i / size] == 0 : (mask >> (i / size)) & 1u); }
+};
+
 // One warp: marks the `keep` groups of neighbours with the largest values in z[0 .. n) by a zero in g[0 .. groups).
 LLM_DEVICE unsigned ordered(float v) {             // integers of the same order; 0 is below all of them
     const unsigned u = __float_as_uint(v);
     return u & 0x80000000u ? ~u : u | 0x80000000u;
 }
-LLM_DEVICE void keep_groups(const float* z, unsigned* g, const ExpertRouteParams& p) {
+LLM_DEVICE Groups keep_groups(const float* z, unsigned* g, const ExpertRouteParams& p) {
     const int lane = threadIdx.x & 31, size = p.n / p.groups;
+    if (p.groups <= 32) {                          // a group per lane: it stays if fewer than `keep` are ahead of it
+        unsigned best = 0;
+        if (lane < p.groups) for (int j = 0; j < size; ++j) best = max(best, ordered(z[lane * size + j]));
+        int ahead = 0;
+        for (int j = 0; j < p.groups; ++j) {
+            const unsigned other = __shfl_sync(0xffffffffu, best, j);
+            ahead += other > best || (other == best && j < lane);
+        }
+        return {__ballot_sync(0xffffffffu, lane < p.groups && ahead < p.keep), nullptr, size};
+    }
     for (int i = lane; i < p.groups; i += 32) {
         unsigned best = 1;
         for (int j = 0; j < size; ++j) best = max(best, ordered(z[i * size + j]));
@@ -51,18 +69,19 @@ LLM_DEVICE void keep_groups(const float* z, unsigned* g, const ExpertRouteParams
         if (lane == 0 && at < (unsigned)p.groups) g[at] = 0;
         __syncwarp();
     }
+    return {0u, g, size};
 }
 
-// One warp: the `top` largest of z[0 .. n) (with g: of the groups that it marks) and the softmax over them.  Logits stay in registers as integers of the same order (NR per
+// One warp: the `top` largest of z[0 .. n), of the groups that stay, and the softmax over them.  Logits stay in registers as integers of the same order (NR per
 // lane), so a round is two warp-wide integer reductions.  Every id it writes is a valid expert, whatever the logits are.
 template <int NR>
-LLM_DEVICE void choose_of(const float* z, const unsigned* g, const ExpertRouteParams& p, int t) {
+LLM_DEVICE void choose_of(const float* z, const Groups& groups, const ExpertRouteParams& p, int t) {
     const int lane = threadIdx.x & 31;
     unsigned key[NR];
 #pragma unroll
     for (int j = 0; j < NR; ++j) {
         const int i = lane + j * 32;
-        key[j] = i < p.n && !(g && g[i / (p.n / p.groups)]) ? ordered(z[i]) : 0u;
+        key[j] = i < p.n && groups.stays(i) ? ordered(z[i]) : 0u;
     }
     float mine = -INFINITY;                        // lane r: the r-th largest logit
     int id = 0;
@@ -90,10 +109,10 @@ LLM_DEVICE void choose_of(const float* z, const unsigned* g, const ExpertRoutePa
     }
 }
 LLM_DEVICE void choose(const float* z, unsigned* g, const ExpertRouteParams& p, int t) {       // g: workspace for the groups
-    if (p.keep < p.groups) keep_groups(z, g, p); else g = nullptr;
-    if (p.n <= 32) choose_of<1>(z, g, p, t);
-    else if (p.n <= 128) choose_of<4>(z, g, p, t);
-    else choose_of<EXPERTS_MAX / 32>(z, g, p, t);
+    const Groups groups = p.keep < p.groups ? keep_groups(z, g, p) : Groups{0u, nullptr, 0};
+    if (p.n <= 32) choose_of<1>(z, groups, p, t);
+    else if (p.n <= 128) choose_of<4>(z, groups, p, t);
+    else choose_of<EXPERTS_MAX / 32>(z, groups, p, t);
 }
 
 // A cluster of CTAs per token: their warps take the experts in turn, four at a time, and leave the logits with the first CTA.

@@ -87,6 +87,34 @@ __global__ void __launch_bounds__(256) attn_prep_kernel(const AttnPrepParams p) 
     }
 }
 
+// The angles of values c .. c + 3 where all four lie on one side of the pairs (half % 4 == 0, c < 2 half)
+struct Angles4 { float4 a, b; };
+LLM_DEVICE Angles4 angles4(const float2* ang, int c, int half) {
+    const int k = c < half ? c : c - half;
+    return {*reinterpret_cast<const float4*>(ang + k), *reinterpret_cast<const float4*>(ang + k + 2)};
+}
+LLM_DEVICE void turned4(const float* row, int c, int half, const Angles4& g, float (&x)[4]) {
+    const float co[4] = {g.a.x, g.a.z, g.b.x, g.b.z}, si[4] = {g.a.y, g.a.w, g.b.y, g.b.w};
+    float y[4];
+    load4(row + (c < half ? c + half : c - half), y);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] = x[e] * co[e] + (c < half ? -y[e] : y[e]) * si[e];
+}
+// values c .. c + 3 of a row, rotated: pairs (i, i + half) turn, the rest passes
+LLM_DEVICE void rotated4(const float* row, int c, int half, const float2* ang, float (&x)[4]) {
+    load4(row + c, x);
+    if (half % 4 == 0) {
+        if (c < 2 * half) turned4(row, c, half, angles4(ang, c, half), x);
+        return;
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        const int k = c + e;
+        if (k < half) x[e] = x[e] * ang[k].x - row[k + half] * ang[k].y;
+        else if (k < 2 * half) x[e] = x[e] * ang[k - half].x + row[k - half] * ang[k - half].y;
+    }
+}
+
 // a warp per token and head: norm, rotation, and the append of keys and values
 template <class TI, class T>
 __global__ void __launch_bounds__(256) head_prep_kernel(const HeadPrepParams p) {
@@ -128,30 +156,25 @@ __global__ void __launch_bounds__(256) head_prep_kernel(const HeadPrepParams p) 
     __syncwarp();
     const float2* ang = p.angles + (size_t)t * p.half;
     for (int i = lane * 4; i < D; i += 128) {
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int c = i + j;
-            x[j] = row[c];
-            if (c < p.half) x[j] = x[j] * ang[c].x - row[c + p.half] * ang[c].y;
-            else if (c < 2 * p.half) x[j] = x[j] * ang[c - p.half].x + row[c - p.half] * ang[c - p.half].y;
-        }
+        rotated4(row, i, p.half, ang, x);
         store4(dst + i, x);
     }
 }
 
 // A warp per head (queries, then keys, then values) and strip of N rows.  TAPS taps with at most four values per lane (dim <= 128): taps
-// and the rows before the current one stay in registers, the strip's rows are loaded together; TAPS = 0: any number and size.
+// and the rows before the current one stay in registers, the next row and its angles are on their way; TAPS = 0: any number and size,
+// N = 1.  Lane i looks up the strip's row i.
 template <class TI, class T, int TAPS, int N>
-__global__ void __launch_bounds__(256) conv_prep_kernel(const ConvPrepParams p) {
+__global__ void __launch_bounds__(256, N > 1 ? 3 : 4) conv_prep_kernel(const ConvPrepParams p) {
     extern __shared__ __align__(16) float sm[];                // [8][dim]
     pdl_trigger();
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, D = p.dim, H = p.n_heads, G = p.n_kv_heads, U = H + 2 * G;
-    const int u = blockIdx.y * 8 + warp, t0 = blockIdx.x * N, n_taps = TAPS ? TAPS : p.n_taps;
+    const int u = blockIdx.y * 8 + warp, t0 = blockIdx.x * N, t1 = min(t0 + N, p.rows), n_taps = TAPS ? TAPS : p.n_taps;
     if (u >= U) return;
     const int kind = u < H ? 0 : u < H + G ? 1 : 2, h = u - (kind == 0 ? 0 : kind == 1 ? H : H + G), col = u * D, cols = U * D;
     float* out = sm + warp * D;
     constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 1;
-    float w[TAPS ? TAPS : 1][4], past[KEEP][4], cur[N][4];     // past[j]: the row j + 1 before the current one
+    float w[TAPS ? TAPS : 1][4], past[KEEP][4], cur[4], nxt[4] = {};        // past[j]: the row j + 1 before the current one
     const int c_own = lane * 4;
     if constexpr (TAPS > 0) {
 #pragma unroll
@@ -161,22 +184,33 @@ __global__ void __launch_bounds__(256) conv_prep_kernel(const ConvPrepParams p) 
         }
     }
     const TI* in = static_cast<const TI*>(p.in) + col;
-    pdl_wait();
-    if constexpr (TAPS > 0) {
-#pragma unroll
-        for (int i = 0; i < N; ++i) {
-            cur[i][0] = cur[i][1] = cur[i][2] = cur[i][3] = 0.f;
-            if (t0 + i < p.rows && c_own < D) load4(in + (size_t)(t0 + i) * p.in_row + c_own, cur[i]);
-        }
+    // positions and sequences come from the host
+    int own_pos = 0, own_seq = 0, own_page = 0;
+    if (lane < t1 - t0) {
+        own_pos = p.positions[t0 + lane];
+        own_seq = LLM_CHECK_INDEX(p.seq_ids[t0 + lane], p.n_seqs);
+        if (kind) own_page = LLM_CHECK_INDEX(p.block_table[(size_t)own_seq * p.max_pages + own_pos / PAGE], p.n_pages);
     }
+    int seq = __shfl_sync(0xffffffffu, own_seq, 0), r0 = p.cu ? p.cu[seq] : t0;          // r0: first row of the sequence's portion
+    float* ring = p.ring + (size_t)LLM_CHECK_INDEX(p.slots[seq], p.n_slots) * n_taps * cols + col;
+    const bool ahead = TAPS > 0 && kind < 2 && p.half % 4 == 0 && c_own < 2 * p.half;    // this lane's angles come as two vectors
+    Angles4 ang_n = {};
     const float gain = kind == 0 && p.q_gain ? p.q_gain[h] : 1.f, share = p.share ? *p.share : 0.f;
-#pragma unroll
-    for (int i = 0; i < N; ++i) {
-        const int t = t0 + i;
-        if (t >= p.rows) break;
-        const int pos = p.positions[t], seq = LLM_CHECK_INDEX(p.seq_ids[t], p.n_seqs);
-        const int r0 = p.cu ? p.cu[seq] : t;                   // first row of the sequence's portion
-        float* ring = p.ring + (size_t)LLM_CHECK_INDEX(p.slots[seq], p.n_slots) * n_taps * cols + col;
+    pdl_wait();
+    if (TAPS > 0 && c_own < D) load4(in + (size_t)t0 * p.in_row + c_own, nxt);
+    if (ahead) ang_n = angles4(p.angles + (size_t)t0 * p.half, c_own, p.half);
+#pragma unroll 1
+    for (int t = t0; t < t1; ++t) {
+        const int pos = __shfl_sync(0xffffffffu, own_pos, t - t0), page = __shfl_sync(0xffffffffu, own_page, t - t0);
+        const int seq_t = __shfl_sync(0xffffffffu, own_seq, t - t0);
+        if (seq_t != seq) {                                    // the first row of another sequence's portion
+            seq = seq_t;
+            r0 = t;
+            ring = p.ring + (size_t)LLM_CHECK_INDEX(p.slots[seq], p.n_slots) * n_taps * cols + col;
+        }
+        T* dst = static_cast<T*>(p.q_out) + ((size_t)t * H + h) * D;
+        if (kind) dst = static_cast<T*>(p.kv) + ((((size_t)page * 2 + kind - 1) * G + h) * PAGE + pos % PAGE) * D;
+        const Angles4 ang_t = ang_n;
         // what stood `lag` rows before this one, zeros in front of the sequence
         auto row_before = [&](int lag, int c, float (&x)[4]) {
             x[0] = x[1] = x[2] = x[3] = 0.f;
@@ -184,27 +218,30 @@ __global__ void __launch_bounds__(256) conv_prep_kernel(const ConvPrepParams p) 
             if (t - lag >= r0) load4(in + (size_t)(t - lag) * p.in_row + c, x);
             else load4(ring + (size_t)((pos - lag) % n_taps) * cols + c, x);
         };
-        __syncwarp();                                          // the row of the token before has been read
         if constexpr (TAPS > 0) {
-            if (i == 0 || t == r0) {
+#pragma unroll
+            for (int e = 0; e < 4; ++e) cur[e] = nxt[e];
+            if (t + 1 < t1 && c_own < D) load4(in + (size_t)(t + 1) * p.in_row + c_own, nxt);
+            if (t + 1 < t1 && ahead) ang_n = angles4(p.angles + (size_t)(t + 1) * p.half, c_own, p.half);
+            if (t == t0 || t == r0) {
 #pragma unroll
                 for (int j = 0; j + 1 < TAPS; ++j) row_before(j + 1, c_own, past[j]);
             }
             if (c_own < D) {
                 float a[4];
 #pragma unroll
-                for (int e = 0; e < 4; ++e) a[e] = w[TAPS - 1][e] * cur[i][e];
+                for (int e = 0; e < 4; ++e) a[e] = w[TAPS - 1][e] * cur[e];
 #pragma unroll
                 for (int j = 0; j + 1 < TAPS; ++j)
 #pragma unroll
                     for (int e = 0; e < 4; ++e) a[e] = fmaf(w[TAPS - 2 - j][e], past[j][e], a[e]);
                 store4(out + c_own, a);
-                if (!p.cu) store4(ring + (size_t)(pos % n_taps) * cols + c_own, cur[i]);
+                if (!p.cu) store4(ring + (size_t)(pos % n_taps) * cols + c_own, cur);
             }
 #pragma unroll
             for (int j = KEEP - 1; j >= 0; --j)
 #pragma unroll
-                for (int e = 0; e < 4; ++e) past[j][e] = j ? past[j - 1][e] : cur[i][e];
+                for (int e = 0; e < 4; ++e) past[j][e] = j ? past[j - 1][e] : cur[e];
         } else {
             for (int c = c_own; c < D; c += 128) {
                 float a[4] = {}, x[4], k[4];
@@ -218,11 +255,6 @@ __global__ void __launch_bounds__(256) conv_prep_kernel(const ConvPrepParams p) 
                 store4(out + c, a);
                 if (!p.cu) store4(ring + (size_t)(pos % n_taps) * cols + c, x);
             }
-        }
-        T* dst = static_cast<T*>(p.q_out) + ((size_t)t * H + h) * D;
-        if (kind) {
-            const int page = LLM_CHECK_INDEX(p.block_table[(size_t)seq * p.max_pages + pos / PAGE], p.n_pages);
-            dst = static_cast<T*>(p.kv) + ((((size_t)page * 2 + kind - 1) * G + h) * PAGE + pos % PAGE) * D;
         }
         float x[4];
         if (kind == 2) {
@@ -241,20 +273,21 @@ __global__ void __launch_bounds__(256) conv_prep_kernel(const ConvPrepParams p) 
                 }
                 store4(dst + c, x);
             }
-            continue;
-        }
-        __syncwarp();
-        const float2* ang = p.angles + (size_t)t * p.half;
-        for (int c = c_own; c < D; c += 128) {
+        } else {
+            __syncwarp();
+            const float2* ang = p.angles + (size_t)t * p.half;
+            for (int c = c_own; c < D; c += 128) {
+                if (ahead) {
+                    load4(out + c, x);
+                    turned4(out, c, p.half, ang_t, x);
+                } else {
+                    rotated4(out, c, p.half, ang, x);
+                }
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int k = c + e;
-                x[e] = out[k];
-                if (k < p.half) x[e] = x[e] * ang[k].x - out[k + p.half] * ang[k].y;
-                else if (k < 2 * p.half) x[e] = x[e] * ang[k - p.half].x + out[k - p.half] * ang[k - p.half].y;
-                x[e] *= gain;
+                for (int e = 0; e < 4; ++e) x[e] *= gain;
+                store4(dst + c, x);
             }
-            store4(dst + c, x);
+            __syncwarp();                                      // the row has been read
         }
     }
 }

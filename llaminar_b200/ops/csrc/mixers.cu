@@ -37,7 +37,7 @@ LLM_DEVICE void load4(const __nv_bfloat16* p, float (&v)[4]) {
 LLM_DEVICE void store4(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
 LLM_DEVICE void store4(__nv_bfloat16* p, const float (&v)[4]) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3])); }
 
-LLM_DEVICE float sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
+LLM_DEVICE float sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 template <int THREADS>
 LLM_DEVICE float block_sum(float v, float* red) {
@@ -266,39 +266,51 @@ __global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p
     const size_t t = blockIdx.x;
     const TI *o = static_cast<const TI*>(p.o) + t * p.o_row, *g = static_cast<const TI*>(p.in) + t * p.in_row + p.g_off;
     T* dst = static_cast<T*>(p.out) + t * p.out_row;
-    constexpr int UN = 4;                              // units of four values a thread keeps; the rest of wider rows is read again
-    float keep[UN][4], z[UN][4], x[4], y[4], w[4], ss = 0.f;
+    constexpr int UN = 2;                              // units of eight values a thread keeps; the rest of wider rows is read again
+    auto load8 = [](const auto* s, float (&v)[8]) {
+        float a[4], b[4];
+        load4(s, a); load4(s + 4, b);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) { v[j] = a[j]; v[4 + j] = b[j]; }
+    };
+    float keep[UN][8], z[UN][8], w[UN][8], ss = 0.f;
 #pragma unroll
     for (int u = 0; u < UN; ++u) {
-        const int i = (u * 256 + threadIdx.x) * 4;
-        keep[u][0] = keep[u][1] = keep[u][2] = keep[u][3] = 0.f;
-        if (i < p.n) { load4(o + i, keep[u]); load4(g + i, z[u]); }
+        const int i = (u * 256 + threadIdx.x) * 8;
+#pragma unroll
+        for (int j = 0; j < 8; ++j) keep[u][j] = 0.f;
+        if (i < p.n) { load8(o + i, keep[u]); load8(g + i, z[u]); load8(p.norm_w + i, w[u]); }
     }
 #pragma unroll
     for (int u = 0; u < UN; ++u)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) ss += keep[u][j] * keep[u][j];
-    for (int i = (UN * 256 + threadIdx.x) * 4; i < p.n; i += 1024) {
-        load4(o + i, x);
+        for (int j = 0; j < 8; ++j) ss += keep[u][j] * keep[u][j];
+    for (int i = (UN * 256 + threadIdx.x) * 8; i < p.n; i += 2048) {
+        float x[8];
+        load8(o + i, x);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) ss += x[j] * x[j];
+        for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
     }
     const float inv = 1.f / sqrtf(block_sum<256>(ss, red) / (float)p.true_n + p.eps);
-    auto put = [&](int i, const float (&v)[4], const float (&s)[4]) {
-        load4(p.norm_w + i, w);
+    auto put = [&](int i, const float (&v)[8], const float (&s)[8], const float (&w)[8]) {
+        float a[4], b[4];
+        auto value = [&](int j) {
+            if constexpr (sizeof(T) == 2) return v[j] * inv * w[j] * sigmoid(s[j]);
+            else return v[j] * inv * w[j] / (1.f + expf(-s[j]));
+        };
 #pragma unroll
-        for (int j = 0; j < 4; ++j) y[j] = v[j] * inv * w[j] / (1.f + expf(-s[j]));
-        store4(dst + i, y);
+        for (int j = 0; j < 4; ++j) { a[j] = value(j); b[j] = value(4 + j); }
+        store4(dst + i, a); store4(dst + i + 4, b);
     };
 #pragma unroll
     for (int u = 0; u < UN; ++u) {
-        const int i = (u * 256 + threadIdx.x) * 4;
-        if (i < p.n) put(i, keep[u], z[u]);
+        const int i = (u * 256 + threadIdx.x) * 8;
+        if (i < p.n) put(i, keep[u], z[u], w[u]);
     }
-    for (int i = (UN * 256 + threadIdx.x) * 4; i < p.n; i += 1024) {
-        float s[4];
-        load4(o + i, x); load4(g + i, s);
-        put(i, x, s);
+    for (int i = (UN * 256 + threadIdx.x) * 8; i < p.n; i += 2048) {
+        float x[8], s[8], g8[8];
+        load8(o + i, x); load8(g + i, s); load8(p.norm_w + i, g8);
+        put(i, x, s, g8);
     }
 }
 
@@ -306,7 +318,7 @@ __global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p
 
 cudaError_t launch_joint_gate(const JointGateParams& p, int rows, bool in_f32, bool f32, cudaStream_t st) {
     if (rows == 0) return cudaSuccess;
-    if (p.n % 4 || p.o_row % 4 || p.in_row % 4 || p.g_off % 4 || p.out_row % 4 || (f32 && !in_f32)) return cudaErrorInvalidValue;
+    if (p.n % 8 || p.o_row % 8 || p.in_row % 8 || p.g_off % 8 || p.out_row % 8 || (f32 && !in_f32)) return cudaErrorInvalidValue;
     auto go = [&](auto kernel) { return launch_pdl(kernel, dim3(rows), dim3(256), 0, st, p); };
     if (f32) return go(joint_gate_kernel<float, float>);
     return in_f32 ? go(joint_gate_kernel<float, __nv_bfloat16>) : go(joint_gate_kernel<__nv_bfloat16, __nv_bfloat16>);

@@ -59,6 +59,21 @@ def test_kernel_forms_agree(off):
     eng.check_health()
 
 
+@pytest.mark.parametrize("few,many", [(0, 1 << 30), (1 << 30, 0)])
+def test_sublayers_one_after_the_other_or_at_the_same_time(few, many):
+    """Both orders, in prompts, portions and captured decode steps, twice with the same result."""
+    m = cases.model("wide", seed=8)
+    want, t = None, cases.tokens(330, 3)
+    eng = cases.engine(m, "cuda", BF)
+    st = eng.model.stack
+    st.beside_few, st.beside_few_experts, st.beside_many = few, few, many
+    for _ in range(2):
+        got = cases.feed_all(eng, t, [200, 5, 64, 1])
+        cases.assert_close(got, cases.expected(t, m), BF)
+        assert want is None or torch.equal(got, want)
+        want = got
+
+
 def test_long_context_many_tiles():
     """Windows of several key tiles and none at all, many chunks of the recurrence, over a few thousand tokens."""
     A, L = oracle.attention_entry, oracle.lightning_entry
