@@ -259,7 +259,7 @@ __global__ void __launch_bounds__(256) head_gate_kernel(const LinearParams p, co
 
 // a CTA per token
 template <class TI, class T>
-__global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p) {
+__global__ void __launch_bounds__(256, 5) joint_gate_kernel(const JointGateParams p) {
     __shared__ float red[8];
     pdl_trigger();
     pdl_wait();
@@ -273,13 +273,13 @@ __global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p
 #pragma unroll
         for (int j = 0; j < 4; ++j) { v[j] = a[j]; v[4 + j] = b[j]; }
     };
-    float keep[UN][8], z[UN][8], w[UN][8], ss = 0.f;
+    float keep[UN][8], z[UN][8], w[8], ss = 0.f;
 #pragma unroll
     for (int u = 0; u < UN; ++u) {
         const int i = (u * 256 + threadIdx.x) * 8;
 #pragma unroll
         for (int j = 0; j < 8; ++j) keep[u][j] = 0.f;
-        if (i < p.n) { load8(o + i, keep[u]); load8(g + i, z[u]); load8(p.norm_w + i, w[u]); }
+        if (i < p.n) { load8(o + i, keep[u]); load8(g + i, z[u]); }
     }
 #pragma unroll
     for (int u = 0; u < UN; ++u)
@@ -292,8 +292,9 @@ __global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p
         for (int j = 0; j < 8; ++j) ss += x[j] * x[j];
     }
     const float inv = 1.f / sqrtf(block_sum<256>(ss, red) / (float)p.true_n + p.eps);
-    auto put = [&](int i, const float (&v)[8], const float (&s)[8], const float (&w)[8]) {
+    auto put = [&](int i, const float (&v)[8], const float (&s)[8]) {
         float a[4], b[4];
+        load8(p.norm_w + i, w);
         auto value = [&](int j) {
             if constexpr (sizeof(T) == 2) return v[j] * inv * w[j] * sigmoid(s[j]);
             else return v[j] * inv * w[j] / (1.f + expf(-s[j]));
@@ -305,12 +306,12 @@ __global__ void __launch_bounds__(256) joint_gate_kernel(const JointGateParams p
 #pragma unroll
     for (int u = 0; u < UN; ++u) {
         const int i = (u * 256 + threadIdx.x) * 8;
-        if (i < p.n) put(i, keep[u], z[u], w[u]);
+        if (i < p.n) put(i, keep[u], z[u]);
     }
     for (int i = (UN * 256 + threadIdx.x) * 8; i < p.n; i += 2048) {
-        float x[8], s[8], g8[8];
-        load8(o + i, x); load8(g + i, s); load8(p.norm_w + i, g8);
-        put(i, x, s, g8);
+        float x[8], s[8];
+        load8(o + i, x); load8(g + i, s);
+        put(i, x, s);
     }
 }
 
