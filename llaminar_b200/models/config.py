@@ -108,7 +108,7 @@ class GroupedAttention:
     qk_norm: bool = True
     conv: int = 0                   # taps of the convolution over time on the projected queries, keys and values (0: none)
     temperature: bool = False       # one learned factor per query head on the scores, before the soft cap
-    value_mix: bool = False         # the first such layer's values of a token join this layer's: v = (1 - share) v + share v_first
+    value_mix: bool = False         # a token's values in the first layer that has this join those of the later ones, with a learned share
 
     @property
     def head_size(self) -> int:
@@ -164,8 +164,8 @@ class Retention:
 
 @dataclass(frozen=True)
 class LightningAttention:
-    """Linear attention S_t = decay_h S_(t-1) + k_t v_t^T with silu on queries, keys and values, no rotation, scale or denominator; the
-    concatenated heads are RMS-normed together (a gain per value) and gated by a sigmoid."""
+    """Linear attention S_t = decay_h S_(t-1) + k_t v_t^T with silu on queries, keys and values, no rotation, scale or denominator;
+    one RMS norm (a gain per value) spans the outputs of all heads, a sigmoid gates them."""
     heads: int
     dim: int
     vdim: int

@@ -101,7 +101,7 @@ def soft_cap(s, cap):
 
 
 def mix_values(v, first, share):
-    """The first layer's values of the same token join this layer's."""
+    """A token's values in the earlier layer take their share of this layer's."""
     return v if first is None else (1 - share) * v + share * first
 
 
